@@ -171,6 +171,12 @@ class EngineConfig:
     decode_stages: int = 0                 # decode attention pages in flight per warp: 0 = 3 (2 under attn_overlap), 2, 3
     gemm_shapes: Dict[str, Dict[str, int]] = field(default_factory=dict)   # "<op>.nb<k>" -> pinned launcher arguments
     decode_chunk_pages: int = 0            # 0 = choose per iteration
+    # layer-list models
+    state_slots: int = 0                   # recurrent-state slots; 0 = one per request of a full batch
+    max_sample_rows: int = 0               # most rows sampled in one iteration; 0 = max_batch_size
+    expand_rows: int = 0                   # rows of the expanded-key buffer of prefill attention; 0 = choose
+    expand_min_tokens: int = 17            # prompt portions of at least this many tokens expand their latents
+    tap_residual: bool = False             # debug: keep the residual stream after every layer run (engine.taps)
     use_cuda_graph: bool = False
     offload: bool = False
     fuse_gemm_rs: bool = False             # TP: K-split GEMMs push partial rows to their owners from the epilogue
@@ -218,9 +224,11 @@ def parse_config(raw: Dict[str, Any], *, tp: Optional[int] = None) -> NanoflowCo
     mc, pc, sc = raw["model_configs"], raw["pipeline_configs"], raw["serve_configs"]
     gpu_num = int(mc.get("gpu_num", 1))
     actual = int(sc.get("actual_gpu_num", gpu_num))
-    model = ModelConfig.from_hf(raw["model"], tp=tp or gpu_num, run_layers=int(mc.get("run_layer", 0)),
-                                name=sc.get("model", ""))
-    ptype = sc.get("pipeline_type", "PLLM")
+    from .models.registry import family_of
+    fam = family_of(raw["model"])
+    model = fam.parse_model(raw["model"], tp=tp or gpu_num, run_layers=int(mc.get("run_layer", 0)),
+                            name=sc.get("model", ""))
+    ptype = sc.get("pipeline_type", "NON_OVERLAP_LOCAL" if fam.listed_layers else "PLLM")
     if ptype not in PIPELINE_TYPES:
         raise ValueError(f"unknown pipeline_type '{ptype}' (known: {', '.join(PIPELINE_TYPES)})")
     gbs = int(pc.get("global_batch_size", mc.get("max_batch_size", 2048)))
@@ -261,6 +269,10 @@ def parse_config(raw: Dict[str, Any], *, tp: Optional[int] = None) -> NanoflowCo
         o_allgather_nanos=[int(k) for k in pc.get("o_allgather_nanos", [])],
         decode_impl=str(pc.get("decode_impl", "")),
         decode_stages=int(pc.get("decode_stages", 0)),
+        state_slots=int(mc.get("state_slots", 0)),
+        max_sample_rows=int(mc.get("max_sample_rows", 0)),
+        expand_rows=int(pc.get("expand_rows", 0)),
+        expand_min_tokens=int(pc.get("expand_min_tokens", 17)),
         model_id=sc.get("model", ""),
         weight_path=sc.get("weight_path", ""),
         hf_path=sc.get("hf_path", ""),
@@ -276,8 +288,31 @@ def parse_config(raw: Dict[str, Any], *, tp: Optional[int] = None) -> NanoflowCo
 
 
 def load_config(path, *, tp: Optional[int] = None) -> NanoflowConfig:
+    """``path``: a four-section JSON file, or a model folder (``config.json`` and safetensors), which gets default
+    serving sections."""
+    if Path(path).is_dir():
+        return folder_config(path, tp=tp)
     with open(path) as f:
         raw = json.load(f)
+    return parse_config(raw, tp=tp)
+
+
+def folder_config(path, *, tp: Optional[int] = None, dtype: str = "", global_batch_size: int = 2048,
+                  model_configs: Optional[Dict[str, Any]] = None,
+                  pipeline_configs: Optional[Dict[str, Any]] = None) -> NanoflowConfig:
+    """Configuration of a model folder. ``dtype`` "bfloat16" / "float32": what the engine stores and computes its
+    matrix products in (default: bfloat16)."""
+    with open(Path(path) / "config.json") as f:
+        hf = json.load(f)
+    if dtype:
+        hf["dtype"] = dtype
+    gpus = tp or 1
+    raw = {"model": hf,
+           "model_configs": {"gpu_num": gpus, "frame_page_size": 16, "max_batch_size": global_batch_size,
+                             **(model_configs or {})},
+           "pipeline_configs": {"global_batch_size": global_batch_size, **(pipeline_configs or {})},
+           "serve_configs": {"model": Path(path).name, "actual_gpu_num": gpus, "weight_path": "", "hf_path": str(path),
+                             "pipeline_type": "NON_OVERLAP" if gpus > 1 else "NON_OVERLAP_LOCAL"}}
     return parse_config(raw, tp=tp)
 
 
@@ -297,6 +332,11 @@ def _hf(hidden, ffn, layers, heads, kv, vocab, theta, *, mtype="llama", arch="Ll
     if extra:
         d.update(extra)
     return d
+
+
+def _volarax(*a, **kw):
+    from .models.volarax import builtin
+    return builtin(*a, **kw)
 
 
 _LLAMA31_SCALING = {"factor": 8.0, "low_freq_factor": 1.0, "high_freq_factor": 4.0,
@@ -320,6 +360,13 @@ MODEL_ARCHS: Dict[str, Dict[str, Any]] = {
     # attention shapes are kept so the config parses, experts are not modelled.
     "mixtral-8-7B": _hf(4096, 14336, 32, 32, 8, 32000, 1000000.0, mtype="mixtral", arch="MixtralForCausalLM",
                         max_pos=32768, extra={"num_local_experts": 8, "num_experts_per_tok": 2}),
+    # Layer-list models (layers, loop and all sizes are in the dictionary)
+    "volarax-tiny": _volarax(200, 1000, "ammaa", heads=3, dim=40, vdim=24, kv_rank=48, window=37, m_heads=3,
+                             m_dim=24, m_vdim=40, ff=136, loop=(1, 4, 2)),
+    "volarax-8B": _volarax(4096, 128256, "am" * 16, heads=32, dim=128, vdim=128, kv_rank=512, window=1024,
+                           m_heads=8, m_dim=256, m_vdim=512, ff=14336, m_ff=14336),
+    "volarax-2B": _volarax(2048, 32000, "am" * 12, heads=16, dim=128, vdim=128, kv_rank=256, window=512,
+                           m_heads=4, m_dim=256, m_vdim=512, ff=8192, m_ff=8192),
 }
 
 MODEL_IDS = {
@@ -328,6 +375,7 @@ MODEL_IDS = {
     "llama3.1-8B": "meta-llama/Meta-Llama-3.1-8B-Instruct", "qwen2-72B": "Qwen/Qwen2-72B-Instruct",
     "deepseek-67B": "deepseek-ai/deepseek-llm-67b-chat", "mixtral-8-7B": "mistralai/Mixtral-8x7B-Instruct-v0.1",
     "tiny": "nanoflow/tiny-llama-test", "tiny8": "nanoflow/tiny8-llama-test",
+    "volarax-tiny": "nanoflow/volarax-tiny-test",
 }
 
 
@@ -347,8 +395,12 @@ def make_config(model: str, *, gpu_num: int = 1, global_batch_size: int = 2048,
     if model not in MODEL_ARCHS:
         raise KeyError(f"unknown model '{model}' (known: {', '.join(MODEL_ARCHS)})")
     hf = copy.deepcopy(MODEL_ARCHS[model])
+    from .models.registry import family_of
+    listed = family_of(hf).listed_layers
     if pipeline_type is None:
-        if hf["model_type"] == "qwen2":
+        if listed:
+            pipeline_type = "NON_OVERLAP_LOCAL"
+        elif hf["model_type"] == "qwen2":
             pipeline_type = "KQVBIAS"
         else:
             pipeline_type = "PLLM" if gpu_num > 1 else "LOCAL"
@@ -356,7 +408,7 @@ def make_config(model: str, *, gpu_num: int = 1, global_batch_size: int = 2048,
     raw = {
         "model": hf,
         "model_configs": {
-            "gpu_num": gpu_num, "run_layer": run_layer or hf["num_hidden_layers"],
+            "gpu_num": gpu_num, "run_layer": run_layer or (0 if listed else hf["num_hidden_layers"]),
             "allocate_kv_data_batch": 0, "frame_page_size": 16, "max_batch_size": global_batch_size,
             "gpu_mem_fraction": 0.92,
         },
@@ -434,7 +486,7 @@ def write_shipped_configs(root: Optional[Path] = None) -> List[Path]:
     root = root or CONFIG_DIR
     written = []
     for model in MODEL_ARCHS:
-        if model.startswith("tiny"):
+        if model.startswith("tiny") or "layers" in MODEL_ARCHS[model]:
             continue
         for name, raw in shipped_variants(model).items():
             path = root / model / f"{name}.json"

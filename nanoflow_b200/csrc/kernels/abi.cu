@@ -22,6 +22,9 @@ extern "C" int nfk_gather_p(const nfk_gather_params* p, cudaStream_t s) {
 }
 extern "C" int nfk_argmax_p(const nfk_argmax_params* p, cudaStream_t s) {
   if (!p) return NF_ERR_BAD_ARG;
+  if (p->dtype == NFK_F32)
+    return nfk_argmax_f32(p->idx_out, p->val_out, reinterpret_cast<const float*>(p->logits), p->rows, p->cols, p->ld,
+                          p->col_offset, s);
   return nfk_argmax(p->idx_out, p->val_out, p->logits, p->rows, p->cols, p->ld, p->col_offset, s);
 }
 extern "C" int nfk_argmax_combine_p(const nfk_argmax_combine_params* p, cudaStream_t s) {

@@ -25,6 +25,12 @@
 // shared memory, 256 TMEM columns each). Every wait is bounded; a wait that runs out sets the status
 // word and all roles leave through the common exit, which frees TMEM.
 //
+// EXT adds what other attention designs need, in an instantiation of its own: a sliding window (tiles before
+// the first row's window are never loaded), a sink in the softmax denominator, K / V as columns of plain
+// rows instead of pool pages (keys expanded from a latent cache), and probabilities that enter the second
+// product as a bf16 pair: the high parts over the first half of the S accumulator, the low parts over the
+// second half.
+//
 // Takes the place of the reference's FlashInfer BatchPrefillWithPagedKVCacheKernel
 // (gemv/include/attention/prefill.cuh:1066-1374, mma.sync m16n16k16 + ldmatrix on sm_80).
 #include "common.cuh"
@@ -78,8 +84,10 @@ constexpr uint32_t kIdescBMnMajor = 1u << 16;
 
 struct Item {
   int req, tok0, ntok, kvh, pg0, np, kv_len, q_end, n_tiles;
+  int t_first;      // first key tile (EXT: the one the first row's window starts in)
   bool valid;
 };
+template <bool EXT>
 __device__ __forceinline__ Item read_item(const nfk_attn_params& p, long long w) {
   Item it;
   const int item = static_cast<int>(w / p.kv_heads);
@@ -95,9 +103,16 @@ __device__ __forceinline__ Item read_item(const nfk_attn_params& p, long long w)
   const int kv_hi = it.kv_len - (it.q_end - (it.tok0 + it.ntok - 1)) + 1;   // keys visible to the last row
   it.valid = it.ntok > 0 && it.np > 0 && kv_hi > 0;
   it.n_tiles = it.valid ? (kv_hi + kTile - 1) / kTile : 0;
+  it.t_first = 0;
+  if (EXT && p.window > 0 && it.valid) {
+    const int lo = it.kv_len - (it.q_end - it.tok0) - p.window + 1;     // first key of the first row
+    if (lo > 0) it.t_first = lo / kTile;
+    it.n_tiles -= it.t_first;
+  }
   return it;
 }
 
+template <bool EXT>
 __global__ void __launch_bounds__(kThreads, 2)
 attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                        nfk_attn_params p) {
@@ -151,14 +166,22 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       for (int b = 0; b < NUM_BARS; ++b) issued[b] = 0;
       bool ok = true;
       for (long long w = blockIdx.x; w < total && ok; w += gridDim.x) {
-        const Item it = read_item(p, w);
+        const Item it = read_item<EXT>(p, w);
         if (!it.valid) continue;
         if (!mbar_wait(&bars[Q_EMPTY], (n_item & 1) ^ 1) || *abort_flag) { fail(NF_ST_TIMEOUT_SMEM_EMPTY); break; }
+        if (EXT && p.q_rows > 0) {
+          // one head per query row tile: 128 rows in two boxes; rows past the item's tokens are other tokens' (or
+          // zero past the buffer) and are never stored
+          mbar_expect_tx(&bars[Q_FULL], 128u * HD * 2);
+          tma_load_2d(smem + Q_OFF, &tmQ, &bars[Q_FULL], it.kvh * HD, it.tok0);
+          tma_load_2d(smem + Q_OFF + 16384, &tmQ, &bars[Q_FULL], it.kvh * HD + 64, it.tok0);
+        } else {
         mbar_expect_tx(&bars[Q_FULL], static_cast<uint32_t>(it.ntok * group) * HD * 2);
         for (int tl = 0; tl < it.ntok; ++tl) {
           const int grow = (it.tok0 + tl) * p.q_heads + it.kvh * group;     // row of the [T*q_heads][128] view
           tma_load_2d(smem + Q_OFF + tl * group * 128, &tmQ, &bars[Q_FULL], 0, grow);
           tma_load_2d(smem + Q_OFF + 16384 + tl * group * 128, &tmQ, &bars[Q_FULL], 64, grow);
+        }
         }
         ++issued[Q_FULL];
         ++n_item;
@@ -166,7 +189,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         auto fetch_pages = [&](int t) {
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
-            int pslot = t * (kTile / kPage) + j;
+            int pslot = (it.t_first + t) * (kTile / kPage) + j;
             if (pslot >= it.np) pslot = 0;      // past the sequence: a valid page, masked by position
             int page = p.kv_indices[it.pg0 + pslot];
             if (page < 0 || page >= p.num_pages) {
@@ -186,20 +209,25 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           mbar_expect_tx(&bars[K_FULL0 + s], kStageBytes);
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
-            const int row0 = ((cur[j] * 2) * p.kv_heads + it.kvh) * kPage;   // of the [pages*2*kv_heads*16][128] view
+            // row of the [pages*2*kv_heads*16][128] view, or row and column of the plain [rows][kv_ld] one
+            const bool plain = EXT && p.kv_ld > 0;
+            const int row0 = plain ? cur[j] * kPage : ((cur[j] * 2) * p.kv_heads + it.kvh) * kPage;
+            const int col0 = plain ? p.k_col + it.kvh * HD : 0;
             uint8_t* dst = smem + K_OFF + s * kStageBytes + j * 2048;
-            tma_load_2d(dst, &tmKV, &bars[K_FULL0 + s], 0, row0);
-            tma_load_2d(dst + kHalfBytes, &tmKV, &bars[K_FULL0 + s], 64, row0);
+            tma_load_2d(dst, &tmKV, &bars[K_FULL0 + s], col0, row0);
+            tma_load_2d(dst + kHalfBytes, &tmKV, &bars[K_FULL0 + s], col0 + 64, row0);
           }
           ++issued[K_FULL0 + s];
           if (!mbar_wait(&bars[V_EMPTY0 + s], ph) || *abort_flag) { fail(NF_ST_TIMEOUT_SMEM_EMPTY); ok = false; break; }
           mbar_expect_tx(&bars[V_FULL0 + s], kStageBytes);
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
-            const int row0 = ((cur[j] * 2 + 1) * p.kv_heads + it.kvh) * kPage;
+            const bool plain = EXT && p.kv_ld > 0;
+            const int row0 = plain ? cur[j] * kPage : ((cur[j] * 2 + 1) * p.kv_heads + it.kvh) * kPage;
+            const int col0 = plain ? p.v_col + it.kvh * HD : 0;
             uint8_t* dst = smem + V_OFF + s * kStageBytes + j * 2048;
-            tma_load_2d(dst, &tmKV, &bars[V_FULL0 + s], 0, row0);
-            tma_load_2d(dst + kHalfBytes, &tmKV, &bars[V_FULL0 + s], 64, row0);
+            tma_load_2d(dst, &tmKV, &bars[V_FULL0 + s], col0, row0);
+            tma_load_2d(dst + kHalfBytes, &tmKV, &bars[V_FULL0 + s], col0 + 64, row0);
           }
           ++issued[V_FULL0 + s];
         }
@@ -239,7 +267,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       };
       bool ok = true;
       for (long long w = blockIdx.x; w < total && ok; w += gridDim.x) {
-        const Item it = read_item(p, w);
+        const Item it = read_item<EXT>(p, w);
         if (!it.valid) continue;
         if (!mbar_wait(&bars[Q_FULL], n_item & 1) || *abort_flag) { fail(NF_ST_TIMEOUT_SMEM_FULL); break; }
         if (!issue_s(g, g)) { fail(NF_ST_TIMEOUT_SMEM_FULL); break; }
@@ -264,6 +292,12 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           for (int k = 0; k < 4; ++k)
             umma_bf16_ts(tmem + 2 * kTile, tmem + s * kTile + k * 8,      // P(t): 16 tokens = 8 columns per step
                          umma_desc_mn_sw128(vb + k * 2048, kHalfBytes, 1024), idesc_o, (t | k) ? 1u : 0u);
+          if (EXT) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)                                   // the low parts of P(t)
+              umma_bf16_ts(tmem + 2 * kTile, tmem + s * kTile + 32 + k * 8,
+                           umma_desc_mn_sw128(vb + k * 2048, kHalfBytes, 1024), idesc_o, 1u);
+          }
           umma_commit(&bars[V_EMPTY0 + s]);
           umma_commit(&bars[PV_DONE0 + s]);
         }
@@ -280,7 +314,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     uint32_t g = 0, n_item = 0;
     bool ok = true;
     for (long long w = blockIdx.x; w < total && ok; w += gridDim.x) {
-      const Item it = read_item(p, w);
+      const Item it = read_item<EXT>(p, w);
       if (!it.valid) continue;
       const int tl = row / group, hh = row % group;
       const bool row_valid = tl < it.ntok;
@@ -295,12 +329,20 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld_32x32b_x32(t_lane + s * kTile, r0);
         tmem_ld_32x32b_x32(t_lane + s * kTile + 32, r1);
         tmem_ld_wait();
-        const int cbase = t * kTile;
+        const int cbase = (it.t_first + t) * kTile;
         if (cbase + kTile - 1 > pos) {                        // only tiles on the diagonal need the mask
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             if (cbase + j > pos) r0[j] = 0xff800000u;         // -inf
             if (cbase + 32 + j > pos) r1[j] = 0xff800000u;
+          }
+        }
+        if (EXT && p.window > 0 && cbase <= pos - p.window) {   // tiles on the window's lower edge
+          const int lo = pos - p.window + 1;
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            if (cbase + j < lo) r0[j] = 0xff800000u;
+            if (cbase + 32 + j < lo) r1[j] = 0xff800000u;
           }
         }
         float mxp = -INFINITY;
@@ -337,6 +379,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const float ms = m_ref == -INFINITY ? 0.f : m_ref;
         float rs = 0.f;
         uint32_t pk[32];                                      // column j: tokens 2j, 2j + 1 of the tile
+        uint32_t pl[EXT ? 32 : 1];                            // low parts
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           const float x0 = fast_exp2(fmaf(__uint_as_float(r0[2 * j]), scale, -ms));
@@ -346,11 +389,17 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           rs += (x0 + x1) + (y0 + y1);
           pk[j] = pack_bf16x2(x0, x1);
           pk[16 + j] = pack_bf16x2(y0, y1);
+          if (EXT) {
+            const float2 xh = unpack_bf16x2(pk[j]), yh = unpack_bf16x2(pk[16 + j]);
+            pl[EXT ? j : 0] = pack_bf16x2(x0 - xh.x, x1 - xh.y);
+            pl[EXT ? 16 + j : 0] = pack_bf16x2(y0 - yh.x, y1 - yh.y);
+          }
         }
         l += rs;
         // P(t) goes over the first half of the S accumulator it was computed from (all 64 scores are in
         // registers); the other accumulator holds P(t-1) / S(t+1), so nothing has to be waited for
         tmem_st_32x32b_x32(t_lane + s * kTile, pk);
+        if constexpr (EXT) tmem_st_32x32b_x32(t_lane + s * kTile + 32, pl);
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
@@ -363,6 +412,8 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       // outstanding here, which a single barrier's phase bit could not tell apart)
       if (!mbar_wait(&bars[PV_DONE0 + ((g - 1) & 1)], ((g - 1) >> 1) & 1) || *abort_flag) { fail(NF_ST_TIMEOUT_TMEM_FULL); break; }
       tc_fence_after();
+      // a far larger sink makes the sum infinite and the row zero, as it should be
+      if (EXT && p.sinks != nullptr && row_valid) l += fast_exp2(p.sinks[it.kvh * group + hh] * kLog2e - m_ref);
       const float inv = l > 0.f ? 1.f / l : 0.f;
       __nv_bfloat16* dst = outp + (static_cast<long long>(it.tok0 + tl) * p.q_heads + it.kvh * group + hh) * HD;
 #pragma unroll 1
@@ -413,22 +464,34 @@ extern "C" int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream
   // Q as [tokens * q_heads][128] (the token count is not known here: any row the items name is inside
   // the caller's buffer, the map's row bound only has to be large enough); the pool as
   // [pages * 2 * kv_heads * 16][128]. Boxes: the `group` rows of one token, one page of one head; 64 columns.
+  // With q_rows the queries are [q_rows][q_heads * 128] and a box is 128 tokens of one head; with kv_ld the
+  // keys and values are columns of [num_pages * 16][kv_ld] rows.
+  const bool ext = p->window > 0 || p->sinks != nullptr || p->kv_ld > 0 || p->q_rows > 0;
+  if (p->window < 0 || (p->q_rows > 0 && group != 1)) return NF_ERR_BAD_ARG;
+  if (p->kv_ld > 0 && (p->kv_ld % 8 != 0 || p->k_col < 0 || p->v_col < 0 || p->k_col % 8 != 0 || p->v_col % 8 != 0))
+    return NF_ERR_BAD_ARG;
   CUtensorMap tmQ, tmKV;
-  int rc = make_tmap_bf16_2d(&tmQ, p->q, 1ull << 26, HD, HD, static_cast<uint32_t>(group), 64);
+  int rc = p->q_rows > 0 ? make_tmap_bf16_2d(&tmQ, p->q, p->q_rows, static_cast<uint64_t>(p->q_heads) * HD,
+                                             p->ld_q > 0 ? p->ld_q : static_cast<uint64_t>(p->q_heads) * HD, 128, 64)
+                         : make_tmap_bf16_2d(&tmQ, p->q, 1ull << 26, HD, HD, static_cast<uint32_t>(group), 64);
   if (rc != NF_OK) return rc;
-  rc = make_tmap_bf16_2d(&tmKV, p->kv_pool, static_cast<uint64_t>(p->num_pages) * 2 * p->kv_heads * kPage, HD, HD, kPage, 64);
+  rc = p->kv_ld > 0 ? make_tmap_bf16_2d(&tmKV, p->kv_pool, static_cast<uint64_t>(p->num_pages) * kPage, p->kv_ld, p->kv_ld, kPage, 64)
+                    : make_tmap_bf16_2d(&tmKV, p->kv_pool, static_cast<uint64_t>(p->num_pages) * 2 * p->kv_heads * kPage, HD, HD, kPage, 64);
   if (rc != NF_OK) return rc;
   static bool attr_dev[kMaxDevices] = {false};   // the attribute is per device
   bool& attr = attr_dev[device_slot()];
   if (!attr) {
-    if (cudaFuncSetAttribute(attn_prefill_ws_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
-        cudaSuccess)
+    if (cudaFuncSetAttribute(attn_prefill_ws_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
+            cudaSuccess ||
+        cudaFuncSetAttribute(attn_prefill_ws_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
+            cudaSuccess)
       return NF_ERR_CUDA;
     attr = true;
   }
   const long long total = static_cast<long long>(p->num_items) * p->kv_heads;
   long long ctas = p->num_ctas > 0 ? p->num_ctas : 2LL * device_sm_count();   // two resident CTAs per SM
   if (ctas > total) ctas = total;
-  attn_prefill_ws_kernel<<<static_cast<int>(ctas), kThreads, kSmemBytes, stream>>>(tmQ, tmKV, *p);
+  if (ext) attn_prefill_ws_kernel<true><<<static_cast<int>(ctas), kThreads, kSmemBytes, stream>>>(tmQ, tmKV, *p);
+  else attn_prefill_ws_kernel<false><<<static_cast<int>(ctas), kThreads, kSmemBytes, stream>>>(tmQ, tmKV, *p);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }

@@ -190,31 +190,43 @@ __global__ void transpose_kernel(__nv_bfloat16* __restrict__ out,
 
 constexpr int kArgmaxThreads = 512;
 
+__device__ __forceinline__ void load_logits8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 a = *reinterpret_cast<const uint4*>(p);
+  const uint32_t aw[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 v = unpack_bf16x2(aw[j]);
+    f[2 * j] = v.x;
+    f[2 * j + 1] = v.y;
+  }
+}
+__device__ __forceinline__ void load_logits8(const float* p, float (&f)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
+template <class T>
 __global__ void __launch_bounds__(kArgmaxThreads)
 argmax_kernel(int* __restrict__ idx_out, float* __restrict__ val_out,
-              const __nv_bfloat16* __restrict__ logits, int rows, int cols, long long ld,
+              const T* __restrict__ logits, int rows, int cols, long long ld,
               int col_offset) {
   __shared__ float s_val[kArgmaxThreads / 32];
   __shared__ int s_idx[kArgmaxThreads / 32];
   for (int row = blockIdx.x; row < rows; row += gridDim.x) {
-    const __nv_bfloat16* lr = logits + static_cast<long long>(row) * ld;
+    const T* lr = logits + static_cast<long long>(row) * ld;
     float best = -INFINITY;
     int bi = 0x7fffffff;
     const int nvec = cols >> 3;
-    const uint4* lv = reinterpret_cast<const uint4*>(lr);
     for (int i = threadIdx.x; i < nvec; i += blockDim.x) {
-      const uint4 a = lv[i];
-      const uint32_t aw[4] = {a.x, a.y, a.z, a.w};
+      float f[8];
+      load_logits8(lr + i * 8, f);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float2 f = unpack_bf16x2(aw[j]);
-        const int c = i * 8 + 2 * j;
-        if (f.x > best) { best = f.x; bi = c; }
-        if (f.y > best) { best = f.y; bi = c + 1; }
-      }
+      for (int j = 0; j < 8; ++j)
+        if (f[j] > best) { best = f[j]; bi = i * 8 + j; }
     }
     for (int c = (nvec << 3) + threadIdx.x; c < cols; c += blockDim.x) {
-      const float f = __bfloat162float(lr[c]);
+      const float f = static_cast<float>(lr[c]);
       if (f > best || (f == best && c < bi)) { best = f; bi = c; }
     }
 #pragma unroll
@@ -385,8 +397,17 @@ extern "C" int nfk_argmax(int* idx_out, float* val_out, const void* logits, int 
   if (rows == 0) return NF_OK;
   if (!idx_out || !logits || rows < 0 || cols <= 0 || ld % 8 != 0 || !al16(logits))
     return NF_ERR_BAD_ARG;
-  argmax_kernel<<<grid_for(rows), kArgmaxThreads, 0, stream>>>(idx_out, val_out, (const bf16*)logits,
-                                                               rows, cols, ld, col_offset);
+  argmax_kernel<bf16><<<grid_for(rows), kArgmaxThreads, 0, stream>>>(idx_out, val_out, (const bf16*)logits,
+                                                                     rows, cols, ld, col_offset);
+  return ok_or_cuda();
+}
+
+extern "C" int nfk_argmax_f32(int* idx_out, float* val_out, const float* logits, int rows, int cols,
+                              long long ld, int col_offset, cudaStream_t stream) {
+  if (rows == 0) return NF_OK;
+  if (!idx_out || !logits || rows < 0 || cols <= 0 || ld % 4 != 0 || !al16(logits)) return NF_ERR_BAD_ARG;
+  argmax_kernel<float><<<grid_for(rows), kArgmaxThreads, 0, stream>>>(idx_out, val_out, logits, rows, cols, ld,
+                                                                      col_offset);
   return ok_or_cuda();
 }
 

@@ -2,7 +2,11 @@
 // by TMA into 128B-swizzled shared memory, persistent over output tiles with an explicit CTA budget.
 //
 //   D[M,N] = A[M,K] * B[N,K]^T (+ bias[N]) (+ beta * C[M,N])            (linear epilogue)
-//   D[M,F] = silu(A * Bg[F,K]^T) .* (A * Bu[F,K]^T)                      (SwiGLU epilogue)
+//   D[M,F] = act(A * Bg[F,K]^T) .* (A * Bu[F,K]^T)                       (gated epilogue: silu, relu, gelu)
+//
+// Columns from f32_col0 on can leave as fp32 into a second output (logits, gate pre-activations), and the
+// product can be block diagonal: with `groups` > 1 output columns of group g see only A's columns
+// [g * group_k, g * group_k + K), which is how per-head matrices are applied to all heads in one launch.
 //
 // Work units are whole output tiles, or with split-K (tile, k range) pairs whose fp32 partial tiles
 // a second pass adds up; with the stream-K tail only the tiles left over after the full waves are
@@ -147,7 +151,60 @@ struct DevParams {
   // gated input: see nfk_gemm_params::gate_flags
   const unsigned int* gate_flags;
   int gate_epoch, gate_nranks;
+  // columns from f32_col0 on go to D32 as fp32 (D32 null: none do)
+  float* D32;
+  long long ld32;
+  int f32_col0;
+  int act;                          // gated epilogue: NFK_ACT_*
+  int groups, group_n, group_k;     // block-diagonal product (groups 1: an ordinary one)
 };
+
+// First output column of column block `n_blk`, the column its group ends at, and where its group starts in
+// A's columns. A column block never straddles two groups.
+struct NBlock {
+  int col0, col_end, a_k0;
+};
+__host__ __device__ __forceinline__ int n_block_count(int groups, int group_n, int out_bn) {
+  return groups * ((group_n + out_bn - 1) / out_bn);
+}
+__device__ __forceinline__ NBlock n_block(const DevParams& p, int n_blk, int out_bn) {
+  NBlock b;
+  if (p.groups == 1) {
+    b.col0 = n_blk * out_bn;
+    b.a_k0 = 0;
+    b.col_end = min(p.N, b.col0 + out_bn);
+  } else {
+    const int per = (p.group_n + out_bn - 1) / out_bn;
+    const int g = n_blk / per;
+    b.col0 = g * p.group_n + (n_blk - g * per) * out_bn;
+    b.a_k0 = g * p.group_k;
+    b.col_end = min((g + 1) * p.group_n, b.col0 + out_bn);
+  }
+  return b;
+}
+
+// Activation of the gated epilogue.
+__device__ __forceinline__ float gated_act(float x, int act) {
+  if (act == NFK_ACT_RELU) return fmaxf(x, 0.f);
+  if (act == NFK_ACT_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+  return x / (1.0f + __expf(-x));
+}
+
+// Eight finished columns of one row: bf16 to D, or fp32 to D32 from f32_col0 on (a multiple of 8).
+__device__ __forceinline__ void store_cols8(const DevParams& p, int row, int col, const float* v) {
+  if (p.D32 != nullptr && col >= p.f32_col0) {
+    float4* dst = reinterpret_cast<float4*>(p.D32 + static_cast<long long>(row) * p.ld32 + (col - p.f32_col0));
+    dst[0] = make_float4(v[0], v[1], v[2], v[3]);
+    dst[1] = make_float4(v[4], v[5], v[6], v[7]);
+    return;
+  }
+  uint4 o;
+  o.x = pack_bf16x2(v[0], v[1]);
+  o.y = pack_bf16x2(v[2], v[3]);
+  o.z = pack_bf16x2(v[4], v[5]);
+  o.w = pack_bf16x2(v[6], v[7]);
+  *reinterpret_cast<uint4*>(p.D + static_cast<long long>(row) * p.ldd + col) = o;
+}
 
 // Tile index -> (m group, n block). Normally m groups vary fastest, so CTAs that run together share
 // weight panels in L2; with a gated input n blocks vary fastest, so the first wave of tiles needs only the
@@ -322,7 +379,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
   const int OUT_BN = (EPI == 1) ? BN / 2 : BN;
   const int m_tiles = (p.M + BM - 1) / BM;
   const int m_groups = (m_tiles + MT * CG - 1) / (MT * CG);
-  const int n_blocks = (p.N + OUT_BN - 1) / OUT_BN;
+  const int n_blocks = n_block_count(p.groups, p.group_n, OUT_BN);
   const int num_kb = (p.K + BK - 1) / BK;
   const int tiles = m_groups * n_blocks;
   const int sk = p.split_k;
@@ -372,6 +429,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       int m_grp, n_blk;
       tile_coords(p, sg.tile, m_groups, n_blocks, m_grp, n_blk);
       const int mt_valid = min(MT, m_tiles - m_grp * MT);
+      const NBlock nb = n_block(p, n_blk, OUT_BN);
       if (p.gate_flags != nullptr) {
         // last 128-row block of A that this CTA loads for the tile
         const int need = (CG == 2) ? min(m_tiles - 1, m_grp * 2 + static_cast<int>(rank)) : m_grp * MT + mt_valid - 1;
@@ -401,28 +459,28 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
           const uint32_t fb = mapa_shared(smem_u32(&full_bar[s]), 0);
           if (leader) mbar_expect_tx(&full_bar[s], 2 * (A_TILE_BYTES + B_BYTES));
           if (EPI == 1)
-            tma_load_2d_pair(sb, rank == 0 ? &tmB0 : &tmB1, fb, kb * BK, n_blk * OUT_BN);
+            tma_load_2d_pair(sb, rank == 0 ? &tmB0 : &tmB1, fb, kb * BK, nb.col0);
           else if (WIDE) {
             const int qrows = BN / 4;
-            tma_load_2d_pair(sb, &tmB0, fb, kb * BK, n_blk * BN + static_cast<int>(rank) * qrows);
+            tma_load_2d_pair(sb, &tmB0, fb, kb * BK, nb.col0 + static_cast<int>(rank) * qrows);
             tma_load_2d_pair(sb + qrows * (BK * 2), &tmB0, fb, kb * BK,
-                             n_blk * BN + BN / 2 + static_cast<int>(rank) * qrows);
+                             nb.col0 + BN / 2 + static_cast<int>(rank) * qrows);
           } else
-            tma_load_2d_pair(sb, &tmB0, fb, kb * BK, n_blk * BN + static_cast<int>(rank) * (BN / 2));
-          tma_load_2d_pair(sa, &tmA, fb, kb * BK, (m_grp * 2 + static_cast<int>(rank)) * BM);
+            tma_load_2d_pair(sb, &tmB0, fb, kb * BK, nb.col0 + static_cast<int>(rank) * (BN / 2));
+          tma_load_2d_pair(sa, &tmA, fb, nb.a_k0 + kb * BK, (m_grp * 2 + static_cast<int>(rank)) * BM);
           continue;
         }
         mbar_expect_tx(&full_bar[s], mt_valid * A_TILE_BYTES + B_BYTES);
         if (EPI == 1) {
-          tma_load_2d(sb, &tmB0, &full_bar[s], kb * BK, n_blk * OUT_BN);
-          tma_load_2d(sb + B_BYTES / 2, &tmB1, &full_bar[s], kb * BK, n_blk * OUT_BN);
+          tma_load_2d(sb, &tmB0, &full_bar[s], kb * BK, nb.col0);
+          tma_load_2d(sb + B_BYTES / 2, &tmB1, &full_bar[s], kb * BK, nb.col0);
         } else {
-          tma_load_2d(sb, &tmB0, &full_bar[s], kb * BK, n_blk * BN);
+          tma_load_2d(sb, &tmB0, &full_bar[s], kb * BK, nb.col0);
         }
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
           if (mt < mt_valid)
-            tma_load_2d(sa + mt * A_TILE_BYTES, &tmA, &full_bar[s], kb * BK, (m_grp * MT + mt) * BM);
+            tma_load_2d(sa + mt * A_TILE_BYTES, &tmA, &full_bar[s], nb.a_k0 + kb * BK, (m_grp * MT + mt) * BM);
       }
     }
     if (CG == 2 && ok) {
@@ -551,10 +609,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
           const int row = (m_first + mt) * BM + q * 32 + lane;
           const bool row_ok = row < p.M;
           const long long row_local = static_cast<long long>(mt * BM + q * 32 + lane) * BN;
-          __nv_bfloat16* drow = p.D + static_cast<long long>(row) * p.ldd;
           const __nv_bfloat16* crow =
               (EPI == 0 && p.C != nullptr) ? p.C + static_cast<long long>(row) * p.ldc : nullptr;
-          const int tile_col_end = min(p.N, (n_blk + 1) * OUT_BN);   // columns past it belong to the next tile
+          const NBlock nb = n_block(p, n_blk, OUT_BN);
+          const int tile_col_end = nb.col_end;   // columns past it belong to the next tile
 #pragma unroll 1
           for (int c = 0; c * 32 < OUT_BN; ++c) {
             uint32_t r[32];
@@ -589,7 +647,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 continue;
               }
 #pragma unroll
-              for (int j = 0; j < 32; ++j) v[j] = gsum[j] / (1.0f + __expf(-gsum[j])) * usum[j];
+              for (int j = 0; j < 32; ++j) v[j] = gated_act(gsum[j], p.act) * usum[j];
             } else {
               tmem_ld_wait();
 #pragma unroll
@@ -606,7 +664,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 continue;
               }
             }
-            const int col0 = n_blk * OUT_BN + c * 32;
+            const int col0 = nb.col0 + c * 32;
             if (EPI == 0 && p.partial != nullptr) {
               if (row_ok && col0 < tile_col_end) {
                 float* prow = p.partial + (static_cast<long long>(sg.ks) * p.M + row) * p.N;
@@ -709,12 +767,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                       }
                     }
                   }
-                  uint4 o;
-                  o.x = pack_bf16x2(vv[0], vv[1]);
-                  o.y = pack_bf16x2(vv[2], vv[3]);
-                  o.z = pack_bf16x2(vv[4], vv[5]);
-                  o.w = pack_bf16x2(vv[6], vv[7]);
-                  *reinterpret_cast<uint4*>(drow + col) = o;
+                  store_cols8(p, row, col, vv);
                 }
               }
             }
@@ -813,12 +866,7 @@ splitk_reduce_kernel(DevParams p) {
         v[2 * j + 1] += p.beta * f.y;
       }
     }
-    uint4 o;
-    o.x = pack_bf16x2(v[0], v[1]);
-    o.y = pack_bf16x2(v[2], v[3]);
-    o.z = pack_bf16x2(v[4], v[5]);
-    o.w = pack_bf16x2(v[6], v[7]);
-    *reinterpret_cast<uint4*>(p.D + static_cast<long long>(row) * p.ldd + col) = o;
+    store_cols8(p, row, col, v);
   }
 }
 
@@ -940,8 +988,9 @@ sk_fixup_kernel(DevParams p, FixupGeom f) {
     const int tile = p.sk_tiles_dp + t;
     const int m_grp = tile % f.m_groups, n_blk = tile / f.m_groups;
     const int row = (m_grp * f.cg + rank) * rows_cta + row_local;
-    const int col = n_blk * f.out_bn + gcol;
-    if (row >= p.M || col >= p.N) continue;
+    const NBlock nb = n_block(p, n_blk, f.out_bn);
+    const int col = nb.col0 + gcol;
+    if (row >= p.M || col >= nb.col_end) continue;
     const float* base = p.sk_partial + (static_cast<long long>(t) * p.sk_max_pieces * f.cg + rank) * slot_floats +
                         static_cast<long long>(row_local) * f.bn + gcol;
     float a[8] = {0, 0, 0, 0, 0, 0, 0, 0}, u[8] = {0, 0, 0, 0, 0, 0, 0, 0};
@@ -961,7 +1010,7 @@ sk_fixup_kernel(DevParams p, FixupGeom f) {
     }
     if (EPI == 1) {
 #pragma unroll
-      for (int j = 0; j < 8; ++j) a[j] = a[j] / (1.0f + __expf(-a[j])) * u[j];
+      for (int j = 0; j < 8; ++j) a[j] = gated_act(a[j], p.act) * u[j];
     } else {
       if (p.bias != nullptr) {
         const uint4 bv = *reinterpret_cast<const uint4*>(p.bias + col);
@@ -984,12 +1033,7 @@ sk_fixup_kernel(DevParams p, FixupGeom f) {
         }
       }
     }
-    uint4 o;
-    o.x = pack_bf16x2(a[0], a[1]);
-    o.y = pack_bf16x2(a[2], a[3]);
-    o.z = pack_bf16x2(a[4], a[5]);
-    o.w = pack_bf16x2(a[6], a[7]);
-    *reinterpret_cast<uint4*>(p.D + static_cast<long long>(row) * p.ldd + col) = o;
+    store_cols8(p, row, col, a);
   }
 }
 
@@ -1024,7 +1068,11 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
   const Geom geo = make_geom(bn, MT, EPI == 1, budget, CG, rs_staged ? kRsStageBytes : 0);
   if (geo.stages < 2) return NF_ERR_BAD_ARG;      // shared-memory budget too small for this tile
   CUtensorMap tmA, tmB0, tmB1;
-  int rc = make_tmap_bf16_2d(&tmA, g.A, g.M, g.K, g.lda, BM, BK);
+  const int groups = g.groups > 1 ? g.groups : 1;
+  const int group_n = g.N / groups;
+  // block-diagonal: a k block that runs past a group's K reads the next group's columns of A, which meet
+  // the zeros that fill B past its K columns
+  int rc = make_tmap_bf16_2d(&tmA, g.A, g.M, g.K + static_cast<uint64_t>(groups - 1) * g.group_k, g.lda, BM, BK);
   if (rc != NF_OK) return rc;
   // rows of B that one TMA copy brings in: a whole tile, a SwiGLU half, or a CTA pair's half
   // (wide tiles: a quarter of the tile per copy, two copies per CTA)
@@ -1076,7 +1124,7 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
   }
   const int m_tiles = (g.M + BM - 1) / BM;
   const int m_groups = (m_tiles + MT * CG - 1) / (MT * CG);
-  const int n_blocks = (g.N + geo.out_bn - 1) / geo.out_bn;
+  const int n_blocks = n_block_count(groups, group_n, geo.out_bn);
   const int units = m_groups * n_blocks * split_k;
   int workers = (g.num_ctas > 0 ? g.num_ctas : sm_count()) / CG;
   if (workers > max_workers) workers = max_workers;
@@ -1130,6 +1178,13 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
   p.gate_flags = g.gate_flags;
   p.gate_epoch = g.gate_epoch;
   p.gate_nranks = g.gate_nranks;
+  p.D32 = reinterpret_cast<float*>(g.D32);
+  p.ld32 = g.ld32;
+  p.f32_col0 = g.f32_col0;
+  p.act = g.act;
+  p.groups = groups;
+  p.group_n = group_n;
+  p.group_k = g.group_k;
   if (CG == 2) {
     cudaLaunchConfig_t lc = {};
     lc.gridDim = dim3(ctas);
@@ -1232,7 +1287,7 @@ Shape choose_shape(const nfk_gemm_params& g, bool swiglu) {
     if (cg == 2 && m_tiles < 2) continue;    // a pair covers two M tiles
     const int out_bn = swiglu ? bn / 2 : bn;
     const int m_groups = (m_tiles + mt * cg - 1) / (mt * cg);
-    const int n_blocks = (g.N + out_bn - 1) / out_bn;
+    const int n_blocks = n_block_count(g.groups > 1 ? g.groups : 1, g.N / (g.groups > 1 ? g.groups : 1), out_bn);
     const int tiles = m_groups * n_blocks;
     const int mt_eff = m_tiles < mt ? m_tiles : mt;
     // per k-block and SM: tensor time (us) at ~11 TFLOP/s, shared-memory fill at ~100 GB/s (a CTA
@@ -1343,7 +1398,7 @@ extern "C" int nfk_gemm_describe(const nfk_gemm_params* g, nfk_gemm_plan* out) {
   if (geo.stages < 2) return NF_ERR_BAD_ARG;
   const int m_tiles = (g->M + BM - 1) / BM;
   const int m_groups = (m_tiles + s.mt * s.cg - 1) / (s.mt * s.cg);
-  const int n_blocks = (g->N + geo.out_bn - 1) / geo.out_bn;
+  const int n_blocks = n_block_count(g->groups > 1 ? g->groups : 1, g->N / (g->groups > 1 ? g->groups : 1), geo.out_bn);
   const int tiles = m_groups * n_blocks;
   int workers = (g->num_ctas > 0 ? g->num_ctas : sm_count()) / s.cg;
   if (workers > sm_count() / s.cg) workers = sm_count() / s.cg;
@@ -1387,7 +1442,16 @@ extern "C" int nfk_gemm_bf16(const nfk_gemm_params* g, cudaStream_t stream) {
   }
   if (g->M == 0 || g->N == 0) return NF_OK;  // empty nano-batch: nothing to do
   if (g->A == nullptr || g->B == nullptr) return NF_ERR_BAD_ARG;
-  if (g->D == nullptr && g->epilogue != NFK_EPI_REDUCE_SCATTER) return NF_ERR_BAD_ARG;
+  if (g->D == nullptr && g->epilogue != NFK_EPI_REDUCE_SCATTER && !(g->D32 != nullptr && g->f32_col0 == 0))
+    return NF_ERR_BAD_ARG;
+  if (g->D32 != nullptr &&
+      (g->epilogue != NFK_EPI_LINEAR || g->f32_col0 < 0 || g->f32_col0 % 8 != 0 || g->ld32 % 4 != 0 ||
+       (reinterpret_cast<uintptr_t>(g->D32) & 15) != 0 || g->norm_w != nullptr))
+    return NF_ERR_BAD_ARG;
+  if (g->act < NFK_ACT_SILU || g->act > NFK_ACT_GELU_TANH) return NF_ERR_BAD_ARG;
+  if (g->groups > 1 && (g->epilogue != NFK_EPI_LINEAR || g->N % (8 * g->groups) != 0 || g->group_k % 8 != 0 ||
+                        g->group_k < 0 || g->gate_flags != nullptr))
+    return NF_ERR_BAD_ARG;
   if (g->M < 0 || g->N < 0 || g->K <= 0) return NF_ERR_BAD_ARG;
   if (g->K % 8 != 0 || g->N % 8 != 0 || g->lda % 8 != 0 || g->ldb % 8 != 0 || g->ldd % 8 != 0)
     return NF_ERR_BAD_ARG;

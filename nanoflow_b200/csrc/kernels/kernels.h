@@ -14,6 +14,8 @@ extern "C" {
 // GEMM (gemm.cu)
 // ------------------------------------------------------------------------------------------------
 enum { NFK_EPI_LINEAR = 0, NFK_EPI_SWIGLU = 1, NFK_EPI_REDUCE_SCATTER = 2 };
+enum { NFK_ACT_SILU = 0, NFK_ACT_RELU = 1, NFK_ACT_GELU_TANH = 2 };   // activation of the gated epilogue
+enum { NFK_BF16 = 0, NFK_F32 = 1 };                                    // storage type of activations and weights
 
 typedef struct nfk_gemm_params {
   const void* A;    // [M,K] bf16, row-major, leading dimension lda
@@ -69,9 +71,21 @@ typedef struct nfk_gemm_params {
   // epilogues; no split-K and no stream-K tail in this mode.
   const unsigned int* gate_flags;
   int gate_epoch, gate_nranks;
+  // Linear epilogue: output columns from f32_col0 on are written as fp32 to D32[row * ld32 + col - f32_col0]
+  // instead of bf16 to D (f32_col0 0: all of them, D may be null). Null = none.
+  void* D32;
+  long long ld32;
+  int f32_col0;         // multiple of 8
+  int act;              // gated epilogue: NFK_ACT_*
+  // Block-diagonal product (linear epilogue): `groups` > 1 cuts the N columns (and B's rows) into equal
+  // groups; group g reads A's columns [g * group_k, g * group_k + K). 0 or 1 = an ordinary product.
+  int groups, group_k;
 } nfk_gemm_params;
 
 int nfk_gemm_bf16(const nfk_gemm_params* p, cudaStream_t stream);
+// The same products with fp32 operands and outputs in fp32 FMA arithmetic (gemm_f32.cu): A, B, B2, D, C, bias
+// are fp32, D32 as above; tile / split / budget / gate fields are ignored, norm and reduce-scatter not built.
+int nfk_gemm_f32(const nfk_gemm_params* p, cudaStream_t stream);
 
 typedef struct nfk_gemm_plan {
   int tile_n, tile_m, cta_group, split_k, stream_k;
@@ -111,6 +125,9 @@ int nfk_transpose(void* out, const void* in, int rows, int cols, cudaStream_t st
 // val_out[r] (optional, fp32) = max. Ties resolve to the lowest index.
 int nfk_argmax(int* idx_out, float* val_out, const void* logits, int rows, int cols,
                long long ld, int col_offset, cudaStream_t stream);
+// The same over fp32 logits.
+int nfk_argmax_f32(int* idx_out, float* val_out, const float* logits, int rows, int cols, long long ld,
+                   int col_offset, cudaStream_t stream);
 // Combine per-shard (val, idx) candidates: cand_val/cand_idx are [shards, rows].
 int nfk_argmax_combine(int* idx_out, const float* cand_val, const int* cand_idx, int shards,
                        int rows, cudaStream_t stream);
@@ -178,6 +195,14 @@ typedef struct nfk_attn_params {
   int num_items;
   unsigned int* status;
   int decode_stages;       // decode: pages in flight per warp, 3 (0 means 3) or 2 (less shared memory per CTA)
+  // nfk_attn_prefill_ws only:
+  int window;              // > 0: position i sees j with 0 <= i - j < window
+  const float* sinks;      // [q_heads]: exp(sink) joins the softmax denominator; null = none
+  // kv_ld > 0: keys and values are not pool pages but columns of plain rows: page id x stands for rows
+  // 16 x .. 16 x + 15 of a [num_pages * 16][kv_ld] array, head h's key at column k_col + 128 h, value at v_col + 128 h
+  int kv_ld, k_col, v_col;
+  int q_rows;              // > 0 (one query head per KV head): rows of q, which is [q_rows][ld_q]
+  int ld_q;                // 0 = q_heads * 128
 } nfk_attn_params;
 int nfk_attn_decode(const nfk_attn_params* p, cudaStream_t stream);
 // The same with the pages copied by a TMA producer warp into a ring of decode_stages (2, 3 or 4) pages per
@@ -190,6 +215,141 @@ int nfk_attn_prefill_tc(const nfk_attn_params* p, cudaStream_t stream);
 // The same on a warp-specialised pipeline: a TMA load warp (whole pages, no transposes), an MMA warp that
 // issues the next tile's scores under this tile's softmax, four softmax warps (attention_ws.cu).
 int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream);
+
+// ------------------------------------------------------------------------------------------------
+// Layer-list models: residual step, latent attention, mLSTM (residual_norm.cu, latent.cu, mlstm.cu)
+// ------------------------------------------------------------------------------------------------
+enum { NFK_NORM_NONE = 0, NFK_NORM_RMS = 1, NFK_NORM_LAYER = 2 };
+// x <- (table ? 0 : x) + norm_in(src) (+ add);  h = norm_out(x). Rows of x, y, table and h are padded to a
+// multiple of 4 elements; weight vectors are padded with zeros to that length.
+typedef struct nfk_residual_norm_params {
+  float* x;                  // [*, ld_x] residual stream
+  long long ld_x;
+  const void* y;             // [*, ld_y] sublayer output, null: none
+  long long ld_y;
+  const void* table;         // [vocab, ld_table] embedding: the source is the token's row instead of y
+  long long ld_table;
+  const int* host_ids;       // token ids as in nfk_embedding
+  const int* feedback_src;
+  const int* prev_tokens;
+  int vocab;
+  const float* in_w;         // norm of the source
+  const float* in_b;
+  const float* add;          // [cols] added to the stream after the sum, null: none
+  void* h;                   // [rows, ld_h] normed stream for the next sublayer, null: none
+  long long ld_h;
+  const float* out_w;
+  const float* out_b;
+  const int* rows_idx;       // row r of h comes from row rows_idx[r] of x and y; x is not written back then
+  int in_rows;
+  int rows, cols;
+  float eps;
+  int in_kind, out_kind;     // NFK_NORM_*
+  int dtype;                 // NFK_BF16 / NFK_F32: y, table, h
+  unsigned int* status;
+} nfk_residual_norm_params;
+int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t stream);
+
+// Latent pool of one layer: [num_pages][page_size][ld] rows (ld = latent size padded to a multiple of 8, the
+// padding is zero). Token t's latent: RMS norm of src[t, 0:rank] times w, written to its page slot.
+// kv_first[req]: page slot of the sequence that the request's page list starts with (null: 0).
+typedef struct nfk_latent_append_params {
+  const void* src;
+  long long ld_src;
+  const float* w;
+  void* pool;
+  long long ld;
+  const int* positions;
+  const int* token_req;
+  const int* kv_indptr;
+  const int* kv_indices;
+  const int* kv_first;
+  int T, rank, page_size, num_pages;
+  float eps;
+  int dtype;
+  unsigned int* status;
+} nfk_latent_append_params;
+int nfk_latent_append(const nfk_latent_append_params* p, cudaStream_t stream);
+
+// Attention in latent space, for listed tokens: head h's query (already multiplied by its key matrix) meets
+// the cached latents, which are keys and values at once: out = sum_j softmax(scale q . c_j) c_j over the
+// positions i - window < j <= i (window 0: all j <= i), with exp(sink[h]) in the denominator (sinks null: none).
+typedef struct nfk_latent_attn_params {
+  const void* q;             // [*, ld_q]: head h of a token at column h * ld
+  long long ld_q;
+  const void* pool;
+  long long ld;              // padded latent size
+  void* out;                 // [*, ld_out]: head h at column h * ld
+  long long ld_out;
+  const int* tokens;         // [n_tokens] token rows
+  const int* positions;
+  const int* token_req;
+  const int* kv_indptr;
+  const int* kv_indices;
+  const int* kv_first;
+  const float* sinks;        // [heads]
+  int n_tokens, heads, page_size, num_pages, window;
+  float scale;
+  int dtype;
+  int impl;                  // 0 = choose, 1 = simple kernel, 2 = tensor-core kernel (bf16)
+  int splits;                // tensor-core kernel: key ranges per token, > 1 needs a workspace
+  float* workspace;          // [n_tokens][splits][heads][ld + 2] fp32
+  long long workspace_floats;
+  unsigned int* status;
+} nfk_latent_attn_params;
+int nfk_latent_attn(const nfk_latent_attn_params* p, cudaStream_t stream);
+
+// mLSTM. Per request slot and head: S [dim][vdim], n [2][dim], m [2], fp32. A launch reads one half of n and m
+// and writes the other, so that CTAs which share a head (each owns columns of S) can all read the old ones
+// while one of them writes the new ones; the caller flips the half with every step of the request. A request
+// whose first token of the launch is at position 0 starts from zero.
+typedef struct nfk_mlstm_params {
+  const void* qkv;           // [T, ld_qkv]: q at q_off + h * dim, k at k_off, v at v_off + h * vdim
+  long long ld_qkv;
+  int q_off, k_off, v_off;
+  const float* gates;        // [T, ld_gates]: input gate of head h at column h, forget gate at heads + h
+  long long ld_gates;
+  const float* i_bias;       // [heads]
+  const float* f_bias;
+  float* S;                  // [slots][heads][dim][vdim]
+  float* n;                  // [slots][heads][2][dim]
+  float* m;                  // [slots][heads][2]
+  float* out;                // [T, ld_out]: head h at column h * vdim
+  long long ld_out;
+  const int* positions;
+  const int* qo_indptr;
+  const int* state_slot;     // [B] 2 * slot + half of n / m to read
+  int req_begin, req_count;
+  int heads, dim, vdim;      // dim, vdim: padded to multiples of 8 (padding columns are zero)
+  int num_slots;
+  float gate_cap, q_scale;
+  int dtype;
+  int impl;                  // prefill: 0 = choose, 1 = token by token, 2 = chunked on tensor cores (bf16)
+  // chunked form: items [num_items][4] (request, first token, tokens, segment of the request) and scratch for
+  // the segments' states (see mlstm.cu)
+  const int* items;
+  int num_items;
+  float* scratch;
+  long long scratch_floats;
+  unsigned int* status;
+} nfk_mlstm_params;
+int nfk_mlstm_decode(const nfk_mlstm_params* p, cudaStream_t stream);    // one token per request
+int nfk_mlstm_prefill(const nfk_mlstm_params* p, cudaStream_t stream);   // any number of tokens per request
+
+// Output of a recurrent head group: out = RMS norm over each head's vdim values * w * sigmoid(g).
+typedef struct nfk_head_norm_gate_params {
+  const float* o;            // [T, ld_o]
+  long long ld_o;
+  const void* g;             // [T, ld_g]
+  long long ld_g;
+  const float* w;            // [heads * vdim_p]
+  void* out;                 // [T, ld_out]
+  long long ld_out;
+  int T, heads, vdim, vdim_p;   // vdim_p: columns per head (padded)
+  float eps;
+  int dtype;
+} nfk_head_norm_gate_params;
+int nfk_head_norm_gate(const nfk_head_norm_gate_params* p, cudaStream_t stream);
 
 // ------------------------------------------------------------------------------------------------
 // KV offload (kv_offload.cu): gather / scatter whole pages between the pool and a staging buffer
@@ -298,6 +458,7 @@ typedef struct nfk_gather_params {
 } nfk_gather_params;
 typedef struct nfk_argmax_params {
   int* idx_out; float* val_out; const void* logits; int rows, cols; long long ld; int col_offset;
+  int dtype;   // NFK_BF16 / NFK_F32
 } nfk_argmax_params;
 typedef struct nfk_argmax_combine_params {
   int* idx_out; const float* cand_val; const int* cand_idx; int shards, rows;

@@ -1,0 +1,786 @@
+// mLSTM: a recurrent mixer with a matrix memory per head, exponential input gate and sigmoid forget gate,
+// stabilised by a running maximum m (Beck et al., "xLSTM: Extended Long Short-Term Memory"):
+//
+//   m' = max(f + m, i);  S' = e^(f + m - m') S + e^(i - m') k v^T;  n' = e^(f + m - m') n + e^(i - m') k
+//   out = S'^T q / (max(|n' . q|, e^(-m')) + 1e-6)
+//
+// with i = cap tanh((x_i + b_i) / cap) and f = logsigmoid(cap tanh((x_f + b_f) / cap)). State, gates and
+// everything derived from them are fp32 (see kernels.h for where the state of a request lives).
+//
+// nfk_mlstm_decode   one token per request: a CTA streams 128 columns of one head's S through registers
+//                    (update, read out, write back in one pass). Bound by the state traffic.
+// nfk_mlstm_prefill  impl 1: token by token with 32 columns of S in shared memory; any size, bf16 or fp32.
+//                    impl 2 (bf16): chunks of 64 tokens on tensor cores. With F the running sum of f inside the
+//                    chunk, a_j = i_j - F_j and M_t = max(m_in, max_{j<=t} a_j), every weight of the chunk is
+//                    an exponential of a non-positive number: token j enters output t with e^(a_j - M_t), the
+//                    incoming state with e^(m_in - M_t), and m_t = F_t + M_t. Weights, weighted values and the
+//                    state enter the products as bf16 pairs (high and low part), so they keep about 16 bits.
+//                    Long prompts are cut into segments: their own contributions are computed side by side from
+//                    zero, a scan turns them into the state each segment starts from, and the outputs of all
+//                    segments are then computed side by side.
+// nfk_head_norm_gate RMS norm of each head's output, weight, output gate.
+#include "attn_mma.cuh"
+#include "elem_io.cuh"
+
+namespace nf {
+namespace {
+
+__device__ __forceinline__ float soft_cap(float x, float cap) { return cap * tanhf(x / cap); }
+__device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ void gate_values(const nfk_mlstm_params& p, long long tok, int head, float& li, float& lf) {
+  const float* g = p.gates + tok * p.ld_gates;
+  li = soft_cap(g[head] + p.i_bias[head], p.gate_cap);
+  lf = log_sigmoid(soft_cap(g[p.heads + head] + p.f_bias[head], p.gate_cap));
+}
+
+// Where a request's state is: slot index and which half of n / m to read (the other half is written).
+struct StateRef {
+  int slot, half;
+  bool ok, fresh;
+};
+__device__ __forceinline__ StateRef state_ref(const nfk_mlstm_params& p, int req) {
+  StateRef r;
+  const int v = p.state_slot[req];
+  r.slot = v >> 1;
+  r.half = v & 1;
+  r.ok = v >= 0 && r.slot < p.num_slots;
+  r.fresh = p.positions[p.qo_indptr[req]] == 0;
+  if (!r.ok) report_status(p.status, NF_ST_BAD_INDEX);
+  return r;
+}
+
+__device__ __forceinline__ float cta_sum256(float v, float* red) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __syncthreads();
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  return warp_sum(lane < 8 ? red[lane] : 0.f);
+}
+
+// ---- decode -----------------------------------------------------------------------------------------
+constexpr int kDecCols = 128;
+
+template <class T>
+__global__ void __launch_bounds__(256)
+mlstm_decode_kernel(nfk_mlstm_params p, int v_slices) {
+  extern __shared__ float dsm[];                 // k[dim] | q[dim]
+  __shared__ float red[8];
+  __shared__ float4 part[8][32];
+  float* k_s = dsm;
+  float* q_s = dsm + p.dim;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int vs = blockIdx.x % v_slices;
+  const int head = (blockIdx.x / v_slices) % p.heads;
+  const int req = p.req_begin + blockIdx.x / (v_slices * p.heads);
+  const StateRef st = state_ref(p, req);
+  if (!st.ok) return;
+  const long long tok = p.qo_indptr[req];
+  const long long sh = static_cast<long long>(st.slot) * p.heads + head;
+  const float* n_old = p.n + (sh * 2 + st.half) * p.dim;
+  float* n_new = p.n + (sh * 2 + (st.half ^ 1)) * p.dim;
+  float li, lf;
+  gate_values(p, tok, head, li, lf);
+  const float m_old = st.fresh ? 0.f : p.m[sh * 2 + st.half];
+  const float m_new = fmaxf(lf + m_old, li);
+  const float keep = expf(lf + m_old - m_new), write = expf(li - m_new);
+  const T* row = reinterpret_cast<const T*>(p.qkv) + tok * p.ld_qkv;
+  float nq = 0.f;
+  for (int d = threadIdx.x; d < p.dim; d += 256) {
+    const float k = to_f32(row[p.k_off + head * p.dim + d]), q = to_f32(row[p.q_off + head * p.dim + d]) * p.q_scale;
+    k_s[d] = k * write;
+    q_s[d] = q;
+    const float n = (st.fresh ? 0.f : keep * n_old[d]) + write * k;
+    if (vs == 0) n_new[d] = n;
+    nq += n * q;
+  }
+  nq = cta_sum256(nq, red);                      // also orders k_s / q_s
+  if (vs == 0 && threadIdx.x == 0) p.m[sh * 2 + (st.half ^ 1)] = m_new;
+  const float inv = 1.f / (fmaxf(fabsf(nq), expf(-m_new)) + 1e-6f);
+  const int col = vs * kDecCols + lane * 4;
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (col < p.vdim) {
+    const float4 v = load4(row + p.v_off + head * p.vdim + col);
+    float* S = p.S + sh * p.dim * p.vdim + col;
+#pragma unroll 8
+    for (int d = warp; d < p.dim; d += 8) {
+      float4* sp = reinterpret_cast<float4*>(S + static_cast<long long>(d) * p.vdim);
+      float4 s = st.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *sp;
+      const float kd = k_s[d], qd = q_s[d];
+      s.x = keep * s.x + kd * v.x;
+      s.y = keep * s.y + kd * v.y;
+      s.z = keep * s.z + kd * v.z;
+      s.w = keep * s.w + kd * v.w;
+      *sp = s;
+      acc.x += s.x * qd; acc.y += s.y * qd; acc.z += s.z * qd; acc.w += s.w * qd;
+    }
+  }
+  part[warp][lane] = acc;
+  __syncthreads();
+  if (warp == 0 && col < p.vdim) {
+#pragma unroll
+    for (int w = 1; w < 8; ++w) {
+      const float4 o = part[w][lane];
+      acc.x += o.x; acc.y += o.y; acc.z += o.z; acc.w += o.w;
+    }
+    acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
+    store4(p.out + tok * p.ld_out + head * p.vdim + col, acc);
+  }
+}
+
+// ---- prefill, token by token ---------------------------------------------------------------------------
+constexpr int kSeqCols = 32;
+
+template <class T>
+__global__ void __launch_bounds__(256)
+mlstm_seq_kernel(nfk_mlstm_params p, int v_slices) {
+  extern __shared__ float dsm[];                 // S[dim][32] | k[dim] | q[dim] | n[dim]
+  __shared__ float red[8];
+  __shared__ float part[8][32];
+  float* S_s = dsm;
+  float* k_s = S_s + p.dim * kSeqCols;
+  float* q_s = k_s + p.dim;
+  float* n_s = q_s + p.dim;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int vs = blockIdx.x % v_slices;
+  const int head = (blockIdx.x / v_slices) % p.heads;
+  const int req = p.req_begin + blockIdx.x / (v_slices * p.heads);
+  const StateRef st = state_ref(p, req);
+  if (!st.ok) return;
+  const int t0 = p.qo_indptr[req], t1 = p.qo_indptr[req + 1];
+  const long long sh = static_cast<long long>(st.slot) * p.heads + head;
+  const int col = vs * kSeqCols + lane;
+  const bool col_ok = col < p.vdim;
+  float* S = p.S + sh * p.dim * p.vdim + col;
+  for (int d = warp; d < p.dim; d += 8)
+    S_s[d * kSeqCols + lane] = (st.fresh || !col_ok) ? 0.f : S[static_cast<long long>(d) * p.vdim];
+  for (int d = threadIdx.x; d < p.dim; d += 256) n_s[d] = st.fresh ? 0.f : p.n[(sh * 2 + st.half) * p.dim + d];
+  float m = st.fresh ? 0.f : p.m[sh * 2 + st.half];
+  for (int t = t0; t < t1; ++t) {
+    float li, lf;
+    gate_values(p, t, head, li, lf);
+    const float m_new = fmaxf(lf + m, li);
+    const float keep = expf(lf + m - m_new), write = expf(li - m_new);
+    m = m_new;
+    const T* row = reinterpret_cast<const T*>(p.qkv) + static_cast<long long>(t) * p.ld_qkv;
+    __syncthreads();                             // the previous token's reads of k_s / q_s are done
+    float nq = 0.f;
+    for (int d = threadIdx.x; d < p.dim; d += 256) {
+      const float k = to_f32(row[p.k_off + head * p.dim + d]), q = to_f32(row[p.q_off + head * p.dim + d]) * p.q_scale;
+      k_s[d] = k * write;
+      q_s[d] = q;
+      const float n = keep * n_s[d] + write * k;
+      n_s[d] = n;
+      nq += n * q;
+    }
+    nq = cta_sum256(nq, red);
+    const float v = col_ok ? to_f32(row[p.v_off + head * p.vdim + col]) : 0.f;
+    float acc = 0.f;
+    for (int d = warp; d < p.dim; d += 8) {
+      const float s = keep * S_s[d * kSeqCols + lane] + k_s[d] * v;
+      S_s[d * kSeqCols + lane] = s;
+      acc += s * q_s[d];
+    }
+    part[warp][lane] = acc;
+    __syncthreads();
+    if (warp == 0 && col_ok) {
+      for (int w = 1; w < 8; ++w) acc += part[w][lane];
+      p.out[static_cast<long long>(t) * p.ld_out + head * p.vdim + col] =
+          acc / (fmaxf(fabsf(nq), expf(-m)) + 1e-6f);
+    }
+  }
+  __syncthreads();
+  for (int d = warp; d < p.dim; d += 8)
+    if (col_ok) S[static_cast<long long>(d) * p.vdim] = S_s[d * kSeqCols + lane];
+  if (vs == 0) {
+    for (int d = threadIdx.x; d < p.dim; d += 256) p.n[(sh * 2 + (st.half ^ 1)) * p.dim + d] = n_s[d];
+    if (threadIdx.x == 0) p.m[sh * 2 + (st.half ^ 1)] = m;
+  }
+}
+
+// ---- prefill, chunks of 64 tokens on tensor cores ----------------------------------------------------------
+constexpr int kChunk = 64, kVs = 64, kChThreads = 256;
+
+template <int DP>
+struct ChCfg {
+  static constexpr int QK_BYTES = kChunk * DP * 2;
+  static constexpr int V_BYTES = kChunk * kVs * 2;
+  static constexpr int S_BYTES = DP * kVs * 2;
+  static constexpr int P_BYTES = kChunk * kChunk * 2;
+  static constexpr int Q_OFF = 0;
+  static constexpr int K_OFF = Q_OFF + QK_BYTES;          // two buffers
+  static constexpr int V_OFF = K_OFF + 2 * QK_BYTES;      // two buffers
+  static constexpr int SH_OFF = V_OFF + 2 * V_BYTES;      // state, high part
+  static constexpr int SL_OFF = SH_OFF + S_BYTES;         // low part
+  static constexpr int PH_OFF = SL_OFF + S_BYTES;
+  static constexpr int PL_OFF = PH_OFF + P_BYTES;
+  static constexpr int WH_OFF = PL_OFF + P_BYTES;         // weighted values, high / low part
+  static constexpr int WL_OFF = WH_OFF + V_BYTES;
+  static constexpr int F_OFF = WL_OFF + V_BYTES;          // fp32 arrays
+  static constexpr int N_F32 = DP + 8 * kChunk + 8;
+  static constexpr int SMEM = F_OFF + N_F32 * 4;
+  static constexpr int WM = DP / 16 < 8 ? DP / 16 : 8;    // warps along dim in the state update
+  static constexpr int WN = 8 / WM;                       // ... and along the columns
+  static constexpr int MTS = DP / 16 / WM;                // 16-row tiles of S per warp
+  static constexpr int NTS = 8 / WN;                      // 8-column tiles of S per warp
+};
+
+__device__ __forceinline__ uint32_t swz(int row, int ch, int row_bytes) {
+  return static_cast<uint32_t>(row * row_bytes + ((ch ^ (row & 7)) << 4));
+}
+__device__ __forceinline__ void cp_async16_zfill(uint32_t smem_addr, const void* g, bool valid) {
+  const int n = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr), "l"(g), "r"(n) : "memory");
+}
+
+// Floats of scratch per (item, head): S [dim][vdim], n [dim], then m and the sum of f of the segment's own
+// contribution and m of the state it starts from.
+__host__ __device__ __forceinline__ long long seg_floats(int dim, int vdim) {
+  return static_cast<long long>(dim) * vdim + dim + 8;
+}
+
+// STATE_ONLY: the segment's own contribution to the state, from zero, into scratch. Otherwise: outputs, from the
+// request's state (first segment) or from scratch; the last segment leaves the state in the request's slot.
+template <int DP, bool STATE_ONLY>
+__global__ void __launch_bounds__(kChThreads, 1)
+mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
+  using C = ChCfg<DP>;
+  extern __shared__ __align__(128) uint8_t smem[];
+  const uint32_t sb = smem_u32(smem);
+  float* n_s = reinterpret_cast<float*>(smem + C::F_OFF);
+  float* a_s = n_s + DP;              // a_j
+  float* mx_s = a_s + kChunk;         // M_t
+  float* int_s = mx_s + kChunk;       // e^(m_in - M_t)
+  float* w_s = int_s + kChunk;        // e^(a_j - M_last)
+  float* em_s = w_s + kChunk;         // e^(-m_t)
+  float* rs_s = em_s + kChunk;        // [2][64] row sums of the weighted scores
+  float* nq_s = rs_s + 2 * kChunk;    // n . q_t
+  float* sc_s = nq_s + kChunk;        // decay, m_out, F_last
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int vs = blockIdx.x % v_slices;
+  const int head = (blockIdx.x / v_slices) % p.heads;
+  const int item = blockIdx.x / (v_slices * p.heads);
+  const int req = p.items[item * 4], tok0 = p.items[item * 4 + 1], ntok = p.items[item * 4 + 2], seg = p.items[item * 4 + 3];
+  const bool has_next = item + 1 < p.num_items && p.items[(item + 1) * 4] == req;
+  if (STATE_ONLY && !has_next) return;
+  const StateRef st = state_ref(p, req);
+  if (!st.ok || ntok <= 0) return;
+  const long long sh = static_cast<long long>(st.slot) * p.heads + head;
+  const __nv_bfloat16* qkv = reinterpret_cast<const __nv_bfloat16*>(p.qkv);
+  const int v0 = vs * kVs;
+  float* sc_S = p.scratch + (static_cast<long long>(item) * p.heads + head) * seg_floats(p.dim, p.vdim);
+  float* sc_n = sc_S + static_cast<long long>(p.dim) * p.vdim;
+  const int n_chunks = (ntok + kChunk - 1) / kChunk;
+
+  auto load_rows = [&](uint32_t dst, int c, int col0, int cols, int width, int row_bytes) {
+    // rows of chunk c, columns [col0, col0 + cols) of the head's block, zero past `cols` and past the last token
+    const int chs = width / 8;
+    for (int i = threadIdx.x; i < kChunk * chs; i += kChThreads) {
+      const int r = i / chs, ch = i % chs;
+      const int t = c * kChunk + r;
+      const bool ok = t < ntok && ch * 8 < cols;
+      cp_async16_zfill(dst + swz(r, ch, row_bytes),
+                       qkv + (ok ? static_cast<long long>(tok0 + t) * p.ld_qkv + col0 + ch * 8 : 0ll), ok);
+    }
+  };
+  auto load_kv = [&](int c) {
+    if (c < n_chunks) {
+      load_rows(sb + C::K_OFF + (c & 1) * C::QK_BYTES, c, p.k_off + head * p.dim, p.dim, DP, DP * 2);
+      load_rows(sb + C::V_OFF + (c & 1) * C::V_BYTES, c, p.v_off + head * p.vdim + v0, p.vdim - v0, kVs, kVs * 2);
+    }
+    cp_async_commit();
+  };
+  auto load_q = [&](int c) {
+    if (!STATE_ONLY && c < n_chunks) load_rows(sb + C::Q_OFF, c, p.q_off + head * p.dim, p.dim, DP, DP * 2);
+    cp_async_commit();
+  };
+  load_kv(0);
+  load_q(0);
+
+  // ---- incoming state ----
+  const bool from_zero = STATE_ONLY || (seg == 0 && st.fresh);
+  const float* S_in = seg == 0 ? p.S + sh * p.dim * p.vdim : sc_S;
+  const float* n_in = seg == 0 ? p.n + (sh * 2 + st.half) * p.dim : sc_n;
+  float m_in = STATE_ONLY ? -INFINITY : (seg == 0 ? (st.fresh ? 0.f : p.m[sh * 2 + st.half]) : sc_n[p.dim + 2]);
+  float F_total = 0.f;
+  const int wm = warp % C::WM, wn = warp / C::WM;
+  float S[C::MTS][C::NTS][4];
+#pragma unroll
+  for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+    for (int b = 0; b < C::NTS; ++b)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + (e >> 1) * 8;
+        const int v = v0 + (wn * C::NTS + b) * 8 + (lane & 3) * 2 + (e & 1);
+        S[a][b][e] = (from_zero || d >= p.dim || v >= p.vdim) ? 0.f : S_in[static_cast<long long>(d) * p.vdim + v];
+      }
+  for (int d = threadIdx.x; d < DP; d += kChThreads) n_s[d] = (from_zero || d >= p.dim) ? 0.f : n_in[d];
+  auto publish_state = [&]() {      // the state's bf16 pair, B operand of the next chunk's read-out
+#pragma unroll
+    for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+      for (int b = 0; b < C::NTS; ++b)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
+          const uint32_t off = swz(d, wn * C::NTS + b, kVs * 2) + (lane & 3) * 4;
+          const uint32_t hi = pack_bf16x2(S[a][b][2 * h], S[a][b][2 * h + 1]);
+          const float2 hf = unpack_bf16x2(hi);
+          *reinterpret_cast<uint32_t*>(smem + C::SH_OFF + off) = hi;
+          *reinterpret_cast<uint32_t*>(smem + C::SL_OFF + off) = pack_bf16x2(S[a][b][2 * h] - hf.x, S[a][b][2 * h + 1] - hf.y);
+        }
+  };
+  if (!STATE_ONLY) publish_state();
+
+  // gates of a chunk: two tokens per lane of warp 0, fetched one chunk ahead
+  float gi[2] = {-INFINITY, -INFINITY}, gf[2] = {0.f, 0.f};
+  auto load_gates = [&](int c) {
+    if (warp != 0) return;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = c * kChunk + lane * 2 + e;
+      gi[e] = -INFINITY;
+      gf[e] = 0.f;
+      if (c < n_chunks && t < ntok) gate_values(p, tok0 + t, head, gi[e], gf[e]);
+    }
+  };
+  load_gates(0);
+
+  for (int c = 0; c < n_chunks; ++c) {
+    if (warp == 0) {
+      // prefix sums of f, prefix maxima of a = i - F
+      float s = gf[0] + gf[1];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += up;
+      }
+      const float F1 = s, F0 = s - gf[1];
+      const float a0 = gi[0] - F0, a1 = gi[1] - F1;
+      float mx = fmaxf(a0, a1);
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, mx, o);
+        if (lane >= o) mx = fmaxf(mx, up);
+      }
+      float before = __shfl_up_sync(0xffffffffu, mx, 1);
+      if (lane == 0) before = -INFINITY;
+      const float M1 = fmaxf(m_in, mx), M0 = fmaxf(m_in, fmaxf(before, a0));
+      const float M_last = __shfl_sync(0xffffffffu, M1, 31), F_last = __shfl_sync(0xffffffffu, F1, 31);
+      const int t = lane * 2;
+      a_s[t] = a0; a_s[t + 1] = a1;
+      mx_s[t] = M0; mx_s[t + 1] = M1;
+      int_s[t] = expf(m_in - M0); int_s[t + 1] = expf(m_in - M1);
+      w_s[t] = expf(a0 - M_last); w_s[t + 1] = expf(a1 - M_last);
+      em_s[t] = expf(-(F0 + M0)); em_s[t + 1] = expf(-(F1 + M1));
+      if (lane == 0) {
+        sc_s[0] = expf(m_in - M_last);
+        sc_s[1] = F_last + M_last;
+        sc_s[2] = F_last;
+      }
+    }
+    cp_async_wait<0>();
+    __syncthreads();                 // chunk c's rows, gates and the state's bf16 pair are in shared memory
+    load_kv(c + 1);
+    load_gates(c + 1);
+    const float decay = sc_s[0];
+    m_in = sc_s[1];
+    F_total += sc_s[2];
+    const uint32_t kb = sb + C::K_OFF + (c & 1) * C::QK_BYTES;
+    const uint32_t vb = sb + C::V_OFF + (c & 1) * C::V_BYTES;
+    const int mt = warp & 3, half = warp >> 2;          // 16 tokens, 32 keys / columns
+    const int mm = lane >> 3, rr = lane & 7;
+    // ---- values weighted by e^(a_j - M_last), as a bf16 pair ----
+    for (int i = threadIdx.x; i < kChunk * kVs / 8; i += kChThreads) {
+      const int r = i / (kVs / 8), ch = i % (kVs / 8);
+      const uint32_t off = swz(r, ch, kVs * 2);
+      const uint4 v = *reinterpret_cast<const uint4*>(smem + C::V_OFF + (c & 1) * C::V_BYTES + off);
+      const uint32_t vw[4] = {v.x, v.y, v.z, v.w};
+      const float w = w_s[r];
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float2 f = unpack_bf16x2(vw[j]);
+        f.x *= w;
+        f.y *= w;
+        hi[j] = pack_bf16x2(f.x, f.y);
+        const float2 hf = unpack_bf16x2(hi[j]);
+        lo[j] = pack_bf16x2(f.x - hf.x, f.y - hf.y);
+      }
+      *reinterpret_cast<uint4*>(smem + C::WH_OFF + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(smem + C::WL_OFF + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    float qs[4][4];
+    if (!STATE_ONLY) {
+      // ---- n . q ----
+      {
+        const int t = threadIdx.x >> 2, part = threadIdx.x & 3;
+        float d = 0.f;
+#pragma unroll 2
+        for (int ch = part; ch < DP / 8; ch += 4) {
+          const uint4 q = *reinterpret_cast<const uint4*>(smem + C::Q_OFF + swz(t, ch, DP * 2));
+          const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float2 f = unpack_bf16x2(qw[j]);
+            d += f.x * n_s[ch * 8 + 2 * j] + f.y * n_s[ch * 8 + 2 * j + 1];
+          }
+        }
+        d = quad_sum(d);
+        if (part == 0) nq_s[t] = d;
+      }
+      // ---- scores Q K^T and read-out Q S of this warp's 16 tokens ----
+      float sc[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[j][e] = qs[j][e] = 0.f;
+      const bool keys_seen = half * 32 <= mt * 16 + 15;       // some of this half's keys are not in the future
+#pragma unroll 2
+      for (int ks = 0; ks < DP / 16; ++ks) {
+        uint32_t a[4], b0, b1, b2, b3;
+        ldsm_x4(sb + C::Q_OFF + swz(mt * 16 + (lane & 15), 2 * ks + (lane >> 4), DP * 2), a[0], a[1], a[2], a[3]);
+        if (keys_seen) {
+#pragma unroll
+          for (int g = 0; g < 2; ++g) {
+            ldsm_x4(kb + swz(half * 32 + g * 16 + (mm >> 1) * 8 + rr, 2 * ks + (mm & 1), DP * 2), b0, b1, b2, b3);
+            mma_bf16(sc[2 * g], a, b0, b1);
+            mma_bf16(sc[2 * g + 1], a, b2, b3);
+          }
+        }
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+          const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, half * 4 + 2 * g + (mm >> 1), kVs * 2);
+          ldsm_x4_trans(sb + C::SH_OFF + off, b0, b1, b2, b3);
+          mma_bf16(qs[2 * g], a, b0, b1);
+          mma_bf16(qs[2 * g + 1], a, b2, b3);
+          ldsm_x4_trans(sb + C::SL_OFF + off, b0, b1, b2, b3);
+          mma_bf16(qs[2 * g], a, b0, b1);
+          mma_bf16(qs[2 * g + 1], a, b2, b3);
+        }
+      }
+      // ---- weights, row sums, bf16 pair of the weighted scores ----
+      const int r0 = mt * 16 + (lane >> 2), r1 = r0 + 8;
+      const float M0 = mx_s[r0], M1 = mx_s[r1];
+      float sum0 = 0.f, sum1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int col = half * 32 + j * 8 + (lane & 3) * 2;
+        const float ac0 = a_s[col], ac1 = a_s[col + 1];
+        const float x0 = col <= r0 ? sc[j][0] * p.q_scale * expf(ac0 - M0) : 0.f;
+        const float x1 = col + 1 <= r0 ? sc[j][1] * p.q_scale * expf(ac1 - M0) : 0.f;
+        const float y0 = col <= r1 ? sc[j][2] * p.q_scale * expf(ac0 - M1) : 0.f;
+        const float y1 = col + 1 <= r1 ? sc[j][3] * p.q_scale * expf(ac1 - M1) : 0.f;
+        sum0 += x0 + x1;
+        sum1 += y0 + y1;
+        const uint32_t h0 = pack_bf16x2(x0, x1), h1 = pack_bf16x2(y0, y1);
+        const float2 f0 = unpack_bf16x2(h0), f1 = unpack_bf16x2(h1);
+        const uint32_t o0 = swz(r0, half * 4 + j, kChunk * 2) + (lane & 3) * 4;
+        const uint32_t o1 = swz(r1, half * 4 + j, kChunk * 2) + (lane & 3) * 4;
+        *reinterpret_cast<uint32_t*>(smem + C::PH_OFF + o0) = h0;
+        *reinterpret_cast<uint32_t*>(smem + C::PH_OFF + o1) = h1;
+        *reinterpret_cast<uint32_t*>(smem + C::PL_OFF + o0) = pack_bf16x2(x0 - f0.x, x1 - f0.y);
+        *reinterpret_cast<uint32_t*>(smem + C::PL_OFF + o1) = pack_bf16x2(y0 - f1.x, y1 - f1.y);
+      }
+      sum0 = quad_sum(sum0);
+      sum1 = quad_sum(sum1);
+      if ((lane & 3) == 0) {
+        rs_s[half * kChunk + r0] = sum0;
+        rs_s[half * kChunk + r1] = sum1;
+      }
+    }
+    __syncthreads();                 // weighted scores and values are in shared memory; Q and the old state are free
+    load_q(c + 1);
+    if (!STATE_ONLY) {
+      // ---- P V, then the outputs of these 16 tokens x 32 columns ----
+      float pv[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) pv[j][0] = pv[j][1] = pv[j][2] = pv[j][3] = 0.f;
+      for (int ks = 0; ks <= mt; ++ks) {
+        uint32_t ph[4], pl[4], b0, b1, b2, b3;
+        const uint32_t ao = swz(mt * 16 + (lane & 15), 2 * ks + (lane >> 4), kChunk * 2);
+        ldsm_x4(sb + C::PH_OFF + ao, ph[0], ph[1], ph[2], ph[3]);
+        ldsm_x4(sb + C::PL_OFF + ao, pl[0], pl[1], pl[2], pl[3]);
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+          ldsm_x4_trans(vb + swz(ks * 16 + (mm & 1) * 8 + rr, half * 4 + 2 * g + (mm >> 1), kVs * 2), b0, b1, b2, b3);
+          mma_bf16(pv[2 * g], ph, b0, b1);
+          mma_bf16(pv[2 * g], pl, b0, b1);
+          mma_bf16(pv[2 * g + 1], ph, b2, b3);
+          mma_bf16(pv[2 * g + 1], pl, b2, b3);
+        }
+      }
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int r = mt * 16 + (lane >> 2) + h * 8, t = c * kChunk + r;
+        if (t >= ntok) continue;
+        const float inter = int_s[r] * p.q_scale;
+        const float den = rs_s[r] + rs_s[kChunk + r] + inter * nq_s[r];
+        const float inv = 1.f / (fmaxf(fabsf(den), em_s[r]) + 1e-6f);
+        float* dst = p.out + static_cast<long long>(tok0 + t) * p.ld_out + head * p.vdim;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int v = v0 + half * 32 + j * 8 + (lane & 3) * 2;
+          if (v < p.vdim)
+            *reinterpret_cast<float2*>(dst + v) = make_float2((inter * qs[j][2 * h] + pv[j][2 * h]) * inv,
+                                                              (inter * qs[j][2 * h + 1] + pv[j][2 * h + 1]) * inv);
+        }
+      }
+    }
+    // ---- state update: S = decay S + K^T (w V), n = decay n + K^T w ----
+#pragma unroll
+    for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+      for (int b = 0; b < C::NTS; ++b)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[a][b][e] *= decay;
+#pragma unroll
+    for (int ks = 0; ks < kChunk / 16; ++ks) {
+      uint32_t ak[C::MTS][4];
+#pragma unroll
+      for (int a = 0; a < C::MTS; ++a)
+        ldsm_x4_trans(kb + swz(ks * 16 + (mm >> 1) * 8 + rr, (wm * C::MTS + a) * 2 + (mm & 1), DP * 2), ak[a][0], ak[a][1],
+                      ak[a][2], ak[a][3]);
+#pragma unroll
+      for (int b = 0; b < C::NTS; b += 2) {
+        const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, wn * C::NTS + b + (mm >> 1), kVs * 2);
+        uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+        ldsm_x4_trans(sb + C::WH_OFF + off, h0, h1, h2, h3);
+        ldsm_x4_trans(sb + C::WL_OFF + off, l0, l1, l2, l3);
+#pragma unroll
+        for (int a = 0; a < C::MTS; ++a) {
+          mma_bf16(S[a][b], ak[a], h0, h1);
+          mma_bf16(S[a][b], ak[a], l0, l1);
+          mma_bf16(S[a][b + 1], ak[a], h2, h3);
+          mma_bf16(S[a][b + 1], ak[a], l2, l3);
+        }
+      }
+    }
+    if (threadIdx.x < DP) {
+      const int d = threadIdx.x;
+      float n = decay * n_s[d];
+      const uint8_t* kp = smem + C::K_OFF + (c & 1) * C::QK_BYTES + (d & 7) * 2;
+#pragma unroll 8
+      for (int j = 0; j < kChunk; ++j)
+        n += w_s[j] * __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(kp + swz(j, d >> 3, DP * 2)));
+      n_s[d] = n;
+    }
+    if (!STATE_ONLY && c + 1 < n_chunks) publish_state();
+    __syncthreads();                 // gate arrays and n are free for the next chunk
+  }
+  cp_async_wait<0>();
+
+  // ---- state out ----
+  if (!STATE_ONLY && has_next) return;
+  float* S_out = STATE_ONLY ? sc_S : p.S + sh * p.dim * p.vdim;
+  float* n_out = STATE_ONLY ? sc_n : p.n + (sh * 2 + (st.half ^ 1)) * p.dim;
+#pragma unroll
+  for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+    for (int b = 0; b < C::NTS; ++b)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
+        const int v = v0 + (wn * C::NTS + b) * 8 + (lane & 3) * 2;
+        if (d < p.dim && v < p.vdim)
+          *reinterpret_cast<float2*>(S_out + static_cast<long long>(d) * p.vdim + v) = make_float2(S[a][b][2 * h], S[a][b][2 * h + 1]);
+      }
+  if (vs == 0) {
+    for (int d = threadIdx.x; d < p.dim; d += kChThreads) n_out[d] = n_s[d];
+    if (threadIdx.x == 0) {
+      if (STATE_ONLY) {
+        sc_n[p.dim] = m_in;
+        sc_n[p.dim + 1] = F_total;
+      } else {
+        p.m[sh * 2 + (st.half ^ 1)] = m_in;
+      }
+    }
+  }
+}
+
+// Segment contributions -> incoming states, in place, for requests with more than one segment. One thread per
+// four elements of (S, n) of a head; all threads follow the same m.
+__global__ void __launch_bounds__(256)
+mlstm_scan_kernel(nfk_mlstm_params p, int e_blocks) {
+  const int eb = blockIdx.x % e_blocks;
+  const int head = (blockIdx.x / e_blocks) % p.heads;
+  const int item0 = blockIdx.x / (e_blocks * p.heads);
+  const int req = p.items[item0 * 4];
+  if (p.items[item0 * 4 + 3] != 0) return;                                   // not a request's first segment
+  if (item0 + 1 >= p.num_items || p.items[(item0 + 1) * 4] != req) return;   // its only segment
+  const StateRef st = state_ref(p, req);
+  if (!st.ok) return;
+  const long long sh = static_cast<long long>(st.slot) * p.heads + head;
+  const long long ns = static_cast<long long>(p.dim) * p.vdim, total = ns + p.dim;
+  const long long e = (static_cast<long long>(eb) * 256 + threadIdx.x) * 4;
+  const bool in = e < total;
+  float4 R = make_float4(0.f, 0.f, 0.f, 0.f);
+  float m = 0.f;
+  if (!st.fresh) {
+    m = p.m[sh * 2 + st.half];
+    if (in) R = e < ns ? load4(p.S + sh * ns + e) : load4(p.n + (sh * 2 + st.half) * p.dim + (e - ns));
+  }
+  for (int it = item0; it < p.num_items && p.items[it * 4] == req; ++it) {
+    float* sc = p.scratch + (static_cast<long long>(it) * p.heads + head) * seg_floats(p.dim, p.vdim);
+    const bool last = it + 1 >= p.num_items || p.items[(it + 1) * 4] != req;
+    float m_loc = 0.f, F = 0.f;
+    float4 L = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (!last) {
+      m_loc = sc[total];
+      F = sc[total + 1];
+      if (in) L = load4(sc + e);
+    }
+    if (it != item0) {
+      if (in) store4(sc + e, R);
+      // m of the incoming state goes to a word of its own: the contribution's m and F are still being read
+      if (eb == 0 && threadIdx.x == 0) sc[total + 2] = m;
+    }
+    if (last) break;
+    const float m_new = fmaxf(F + m, m_loc);
+    const float ka = expf(F + m - m_new), kb = expf(m_loc - m_new);
+    R.x = ka * R.x + kb * L.x;
+    R.y = ka * R.y + kb * L.y;
+    R.z = ka * R.z + kb * L.z;
+    R.w = ka * R.w + kb * L.w;
+    m = m_new;
+  }
+}
+
+// ---- head norm + output gate ---------------------------------------------------------------------------
+template <class T>
+__global__ void __launch_bounds__(256)
+head_norm_gate_kernel(nfk_head_norm_gate_params p) {
+  const int lane = threadIdx.x & 31;
+  const long long total = static_cast<long long>(p.T) * p.heads;
+  for (long long i = blockIdx.x * 8ll + (threadIdx.x >> 5); i < total; i += gridDim.x * 8ll) {
+    const long long t = i / p.heads;
+    const int c0 = static_cast<int>(i % p.heads) * p.vdim_p;
+    const float* o = p.o + t * p.ld_o + c0;
+    float ss = 0.f;
+    for (int c = lane * 4; c < p.vdim_p; c += 128) {       // padding columns are zero
+      const float4 v = load4(o + c);
+      ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+    }
+    const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(p.vdim) + p.eps);
+    const T* g = reinterpret_cast<const T*>(p.g) + t * p.ld_g + c0;
+    T* dst = reinterpret_cast<T*>(p.out) + t * p.ld_out + c0;
+    for (int c = lane * 4; c < p.vdim_p; c += 128) {
+      float4 v = load4(o + c);
+      const float4 w = load4(p.w + c0 + c), gg = load4(g + c);
+      v.x = v.x * inv * w.x / (1.f + expf(-gg.x));
+      v.y = v.y * inv * w.y / (1.f + expf(-gg.y));
+      v.z = v.z * inv * w.z / (1.f + expf(-gg.z));
+      v.w = v.w * inv * w.w / (1.f + expf(-gg.w));
+      store4(dst + c, v);
+    }
+  }
+}
+
+int check_mlstm(const nfk_mlstm_params* p) {
+  if (p == nullptr) return NF_ERR_BAD_ARG;
+  if (!p->qkv || !p->gates || !p->i_bias || !p->f_bias || !p->S || !p->n || !p->m || !p->out || !p->positions ||
+      !p->qo_indptr || !p->state_slot)
+    return NF_ERR_BAD_ARG;
+  if (p->heads <= 0 || p->dim <= 0 || p->vdim <= 0 || p->dim % 8 != 0 || p->vdim % 8 != 0 || p->num_slots <= 0 ||
+      p->req_begin < 0 || p->req_count < 0 || !(p->gate_cap > 0.f))
+    return NF_ERR_BAD_ARG;
+  if (p->ld_qkv % 8 != 0 || p->q_off % 8 != 0 || p->k_off % 8 != 0 || p->v_off % 8 != 0 || p->ld_out % 4 != 0)
+    return NF_ERR_BAD_ARG;
+  return NF_OK;
+}
+
+template <class K>
+int set_smem(K kernel, size_t bytes) {
+  if (bytes > 227 * 1024) return NF_ERR_UNSUPPORTED;
+  if (bytes > 48 * 1024 &&
+      cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)) != cudaSuccess)
+    return NF_ERR_CUDA;
+  return NF_OK;
+}
+
+template <int DP>
+int launch_chunk(const nfk_mlstm_params& p, cudaStream_t stream) {
+  using C = ChCfg<DP>;
+  static bool attr_dev[kMaxDevices] = {false};
+  bool& attr = attr_dev[device_slot()];
+  if (!attr) {
+    int rc = set_smem(mlstm_chunk_kernel<DP, false>, C::SMEM);
+    if (rc == NF_OK) rc = set_smem(mlstm_chunk_kernel<DP, true>, C::SMEM);
+    if (rc != NF_OK) return rc;
+    attr = true;
+  }
+  const int v_slices = (p.vdim + kVs - 1) / kVs;
+  const int grid = p.num_items * p.heads * v_slices;
+  if (p.num_items > p.req_count) {       // some request has several segments
+    mlstm_chunk_kernel<DP, true><<<grid, kChThreads, C::SMEM, stream>>>(p, v_slices);
+    if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
+    const int e_blocks = (p.dim * p.vdim + p.dim + 1023) / 1024;
+    mlstm_scan_kernel<<<p.num_items * p.heads * e_blocks, 256, 0, stream>>>(p, e_blocks);
+    if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
+  }
+  mlstm_chunk_kernel<DP, false><<<grid, kChThreads, C::SMEM, stream>>>(p, v_slices);
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+}  // namespace
+}  // namespace nf
+
+extern "C" int nfk_mlstm_decode(const nfk_mlstm_params* p, cudaStream_t stream) {
+  using namespace nf;
+  const int rc = check_mlstm(p);
+  if (rc != NF_OK) return rc;
+  if (p->req_count == 0) return NF_OK;
+  const int v_slices = (p->vdim + kDecCols - 1) / kDecCols;
+  const long long grid = static_cast<long long>(p->req_count) * p->heads * v_slices;
+  const size_t sm = static_cast<size_t>(p->dim) * 8;
+  if (grid > 0x7fffffffll || sm > 40 * 1024) return NF_ERR_BAD_ARG;
+  if (p->dtype == NFK_F32) mlstm_decode_kernel<float><<<static_cast<int>(grid), 256, sm, stream>>>(*p, v_slices);
+  else mlstm_decode_kernel<__nv_bfloat16><<<static_cast<int>(grid), 256, sm, stream>>>(*p, v_slices);
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+extern "C" int nfk_mlstm_prefill(const nfk_mlstm_params* p, cudaStream_t stream) {
+  using namespace nf;
+  int rc = check_mlstm(p);
+  if (rc != NF_OK) return rc;
+  if (p->req_count == 0) return NF_OK;
+  const bool chunk_ok = p->dtype == NFK_BF16 && p->dim <= 256 && p->items != nullptr && p->num_items >= p->req_count &&
+                        (reinterpret_cast<uintptr_t>(p->qkv) & 15) == 0 &&
+                        (p->num_items == p->req_count ||
+                         (p->scratch != nullptr && p->num_items * p->heads * seg_floats(p->dim, p->vdim) <= p->scratch_floats));
+  if (p->impl == 2 && !chunk_ok) return NF_ERR_UNSUPPORTED;
+  if (p->impl != 1 && chunk_ok) {
+    if (p->dim <= 64) return launch_chunk<64>(*p, stream);
+    if (p->dim <= 128) return launch_chunk<128>(*p, stream);
+    return launch_chunk<256>(*p, stream);
+  }
+  const int v_slices = (p->vdim + kSeqCols - 1) / kSeqCols;
+  const size_t sm = static_cast<size_t>(p->dim) * (kSeqCols + 3) * 4;
+  const long long grid = static_cast<long long>(p->req_count) * p->heads * v_slices;
+  if (grid > 0x7fffffffll) return NF_ERR_BAD_ARG;
+  if (p->dtype == NFK_F32) {
+    rc = set_smem(mlstm_seq_kernel<float>, sm);
+    if (rc == NF_OK) mlstm_seq_kernel<float><<<static_cast<int>(grid), 256, sm, stream>>>(*p, v_slices);
+  } else {
+    rc = set_smem(mlstm_seq_kernel<__nv_bfloat16>, sm);
+    if (rc == NF_OK) mlstm_seq_kernel<__nv_bfloat16><<<static_cast<int>(grid), 256, sm, stream>>>(*p, v_slices);
+  }
+  if (rc != NF_OK) return rc;
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+extern "C" int nfk_head_norm_gate(const nfk_head_norm_gate_params* p, cudaStream_t stream) {
+  using namespace nf;
+  if (p == nullptr) return NF_ERR_BAD_ARG;
+  if (p->T == 0) return NF_OK;
+  if (!p->o || !p->g || !p->w || !p->out || p->T < 0 || p->heads <= 0 || p->vdim <= 0 || p->vdim_p < p->vdim ||
+      p->vdim_p % 4 != 0 || p->ld_o % 4 != 0 || p->ld_g % 4 != 0 || p->ld_out % 4 != 0)
+    return NF_ERR_BAD_ARG;
+  long long grid = (static_cast<long long>(p->T) * p->heads + 7) / 8;
+  if (grid > 16ll * device_sm_count()) grid = 16ll * device_sm_count();
+  if (p->dtype == NFK_F32) head_norm_gate_kernel<float><<<static_cast<int>(grid), 256, 0, stream>>>(*p);
+  else head_norm_gate_kernel<__nv_bfloat16><<<static_cast<int>(grid), 256, 0, stream>>>(*p);
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}

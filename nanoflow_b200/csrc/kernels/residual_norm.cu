@@ -1,0 +1,161 @@
+// The step between two sublayers in one pass over the row: norm of the sublayer's output, residual sum in
+// fp32, an optional vector added to the stream, and the norm that the next sublayer reads.
+//
+//   x <- (table ? 0 : x) + norm_in(src) (+ add);   h = norm_out(x)
+//
+// `src` is the sublayer's output row, or the embedding row of the token (ids as in nfk_embedding, with the
+// previous iteration's tokens fed back on the device). Norms are RMS or layer norms with fp32 weights. The
+// stream x is fp32; src and h are bf16 or fp32. One CTA per row, the row stays in registers.
+#include "elem_io.cuh"
+
+namespace nf {
+namespace {
+
+constexpr int kRnThreads = 256;
+
+// Sum over the CTA of one value per thread; every thread gets the result.
+__device__ __forceinline__ float cta_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __syncthreads();                       // readers of the previous sum are done with `red`
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  return warp_sum(lane < (kRnThreads >> 5) ? red[lane] : 0.f);
+}
+
+// In-place norm of the row held in v (elements at or past `cols` are zero and stay zero).
+template <int NV>
+__device__ __forceinline__ void norm_row(float4 (&v)[NV], int kind, const float* w, const float* b, int cols, int nvec,
+                                         float eps, float* red) {
+  if (kind == NFK_NORM_NONE) return;
+  const float inv_n = 1.f / static_cast<float>(cols);
+  float mean = 0.f;
+  if (kind == NFK_NORM_LAYER) {
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    mean = cta_sum(s, red) * inv_n;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (threadIdx.x + i * kRnThreads) * 4;
+    float* e = reinterpret_cast<float*>(&v[i]);
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (c + j < cols) {
+        e[j] -= mean;
+        ss += e[j] * e[j];
+      }
+  }
+  const float inv = rsqrtf(cta_sum(ss, red) * inv_n + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int vi = threadIdx.x + i * kRnThreads;
+    if (vi < nvec) {
+      const float4 ww = load4(w + vi * 4);            // zero past `cols`
+      const float4 bb = b != nullptr ? load4(b + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[i].x = v[i].x * inv * ww.x + bb.x;
+      v[i].y = v[i].y * inv * ww.y + bb.y;
+      v[i].z = v[i].z * inv * ww.z + bb.z;
+      v[i].w = v[i].w * inv * ww.w + bb.w;
+    }
+  }
+}
+
+template <class T, int NV>
+__global__ void __launch_bounds__(kRnThreads)
+residual_norm_kernel(nfk_residual_norm_params p) {
+  __shared__ float red[kRnThreads / 32];
+  const int nvec = (p.cols + 3) >> 2;
+  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+    int src_row = row;
+    if (p.rows_idx != nullptr) {
+      src_row = p.rows_idx[row];
+      if (src_row < 0 || src_row >= p.in_rows) {
+        if (threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
+        src_row = 0;
+      }
+    }
+    const T* src = nullptr;
+    if (p.table != nullptr) {
+      int id = p.host_ids != nullptr ? p.host_ids[row] : 0;
+      if (p.feedback_src != nullptr && p.prev_tokens != nullptr) {
+        const int f = p.feedback_src[row];
+        if (f >= 0) id = p.prev_tokens[f];
+      }
+      if (id < 0 || id >= p.vocab) {
+        if (threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
+        id = 0;
+      }
+      src = reinterpret_cast<const T*>(p.table) + static_cast<long long>(id) * p.ld_table;
+    } else if (p.y != nullptr) {
+      src = reinterpret_cast<const T*>(p.y) + static_cast<long long>(src_row) * p.ld_y;
+    }
+    float* xr = p.x + static_cast<long long>(src_row) * p.ld_x;
+    float4 v[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int vi = threadIdx.x + i * kRnThreads;
+      v[i] = (src != nullptr && vi < nvec) ? load4(src + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (src != nullptr) norm_row<NV>(v, p.in_kind, p.in_w, p.in_b, p.cols, nvec, p.eps, red);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int vi = threadIdx.x + i * kRnThreads;
+      if (vi < nvec) {
+        if (p.table == nullptr) {
+          const float4 x = load4(xr + vi * 4);
+          v[i].x += x.x; v[i].y += x.y; v[i].z += x.z; v[i].w += x.w;
+        }
+        if (p.add != nullptr) {
+          const float4 a = load4(p.add + vi * 4);
+          v[i].x += a.x; v[i].y += a.y; v[i].z += a.z; v[i].w += a.w;
+        }
+        if (p.rows_idx == nullptr) store4(xr + vi * 4, v[i]);
+      }
+    }
+    if (p.h != nullptr) {
+      norm_row<NV>(v, p.out_kind, p.out_w, p.out_b, p.cols, nvec, p.eps, red);
+      T* hr = reinterpret_cast<T*>(p.h) + static_cast<long long>(row) * p.ld_h;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int vi = threadIdx.x + i * kRnThreads;
+        if (vi < nvec) store4(hr + vi * 4, v[i]);
+      }
+    }
+  }
+}
+
+template <class T>
+int launch_rn(const nfk_residual_norm_params& p, cudaStream_t stream) {
+  const int nvec = (p.cols + 3) / 4, per = (nvec + kRnThreads - 1) / kRnThreads;
+  const int cap = device_sm_count() * 16;
+  const int grid = p.rows < cap ? p.rows : cap;
+  if (per <= 1) residual_norm_kernel<T, 1><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 2) residual_norm_kernel<T, 2><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 4) residual_norm_kernel<T, 4><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 8) residual_norm_kernel<T, 8><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 16) residual_norm_kernel<T, 16><<<grid, kRnThreads, 0, stream>>>(p);
+  else return NF_ERR_UNSUPPORTED;
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+}  // namespace
+}  // namespace nf
+
+extern "C" int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t stream) {
+  using namespace nf;
+  if (p == nullptr) return NF_ERR_BAD_ARG;
+  if (p->rows == 0) return NF_OK;
+  if (!p->x || p->rows < 0 || p->cols <= 0 || p->ld_x % 4 != 0 || p->ld_x < p->cols) return NF_ERR_BAD_ARG;
+  if (p->table && (p->rows_idx || p->vocab <= 0 || p->ld_table % 4 != 0)) return NF_ERR_BAD_ARG;
+  if (p->table && !p->host_ids && !(p->feedback_src && p->prev_tokens)) return NF_ERR_BAD_ARG;
+  if ((p->y && p->ld_y % 4 != 0) || (p->h && p->ld_h % 4 != 0)) return NF_ERR_BAD_ARG;
+  if (p->rows_idx && (p->in_rows <= 0 || !p->h)) return NF_ERR_BAD_ARG;
+  for (int kind : {p->in_kind, p->out_kind})
+    if (kind != NFK_NORM_NONE && kind != NFK_NORM_RMS && kind != NFK_NORM_LAYER) return NF_ERR_BAD_ARG;
+  if ((p->table || p->y) && p->in_kind != NFK_NORM_NONE && !p->in_w) return NF_ERR_BAD_ARG;
+  if (p->h && p->out_kind != NFK_NORM_NONE && !p->out_w) return NF_ERR_BAD_ARG;
+  return p->dtype == NFK_F32 ? launch_rn<float>(*p, stream) : launch_rn<__nv_bfloat16>(*p, stream);
+}

@@ -41,7 +41,9 @@ class GemmParams(Structure):
                 ("rs_rows_cap", c_int), ("rs_flag_off", c_longlong), ("rs_epoch", c_int), ("smem_budget_kb", c_int),
                 ("cta_group", c_int), ("stream_k", c_int),
                 ("norm_w", c_void_p), ("norm_out", c_void_p), ("norm_ld", c_longlong), ("norm_eps", c_float),
-                ("rs_staged", c_int), ("gate_flags", c_void_p), ("gate_epoch", c_int), ("gate_nranks", c_int)]
+                ("rs_staged", c_int), ("gate_flags", c_void_p), ("gate_epoch", c_int), ("gate_nranks", c_int),
+                ("D32", c_void_p), ("ld32", c_longlong), ("f32_col0", c_int), ("act", c_int),
+                ("groups", c_int), ("group_k", c_int)]
 
 
 class RopeAppendParams(Structure):
@@ -67,7 +69,64 @@ class AttnParams(Structure):
                 ("page_size", c_int), ("num_pages", c_int), ("sm_scale", c_float),
                 ("num_ctas", c_int), ("req_begin", c_int), ("req_count", c_int),
                 ("chunk_pages", c_int), ("workspace", c_void_p), ("max_chunks", c_int),
-                ("items", c_void_p), ("num_items", c_int), ("status", c_void_p), ("decode_stages", c_int)]
+                ("items", c_void_p), ("num_items", c_int), ("status", c_void_p), ("decode_stages", c_int),
+                ("window", c_int), ("sinks", c_void_p), ("kv_ld", c_int), ("k_col", c_int), ("v_col", c_int),
+                ("q_rows", c_int), ("ld_q", c_int)]
+
+
+BF16, F32 = 0, 1                                        # storage type of a kernel's activations and weights
+ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 2}           # activation of the gated GEMM epilogue
+NORMS = {None: 0, "rms": 1, "layer": 2}
+
+
+def dtype_code(dtype: torch.dtype) -> int:
+    if dtype == torch.bfloat16:
+        return BF16
+    if dtype == torch.float32:
+        return F32
+    raise RuntimeError(f"kernels store activations as bfloat16 or float32, not {dtype}")
+
+
+class ResidualNormParams(Structure):
+    _fields_ = [("x", c_void_p), ("ld_x", c_longlong), ("y", c_void_p), ("ld_y", c_longlong),
+                ("table", c_void_p), ("ld_table", c_longlong), ("host_ids", c_void_p), ("feedback_src", c_void_p),
+                ("prev_tokens", c_void_p), ("vocab", c_int), ("in_w", c_void_p), ("in_b", c_void_p),
+                ("add", c_void_p), ("h", c_void_p), ("ld_h", c_longlong), ("out_w", c_void_p), ("out_b", c_void_p),
+                ("rows_idx", c_void_p), ("in_rows", c_int), ("rows", c_int), ("cols", c_int), ("eps", c_float),
+                ("in_kind", c_int), ("out_kind", c_int), ("dtype", c_int), ("status", c_void_p)]
+
+
+class LatentAppendParams(Structure):
+    _fields_ = [("src", c_void_p), ("ld_src", c_longlong), ("w", c_void_p), ("pool", c_void_p), ("ld", c_longlong),
+                ("positions", c_void_p), ("token_req", c_void_p), ("kv_indptr", c_void_p), ("kv_indices", c_void_p),
+                ("kv_first", c_void_p), ("T", c_int), ("rank", c_int), ("page_size", c_int), ("num_pages", c_int),
+                ("eps", c_float), ("dtype", c_int), ("status", c_void_p)]
+
+
+class LatentAttnParams(Structure):
+    _fields_ = [("q", c_void_p), ("ld_q", c_longlong), ("pool", c_void_p), ("ld", c_longlong), ("out", c_void_p),
+                ("ld_out", c_longlong), ("tokens", c_void_p), ("positions", c_void_p), ("token_req", c_void_p),
+                ("kv_indptr", c_void_p), ("kv_indices", c_void_p), ("kv_first", c_void_p), ("sinks", c_void_p),
+                ("n_tokens", c_int), ("heads", c_int), ("page_size", c_int), ("num_pages", c_int), ("window", c_int),
+                ("scale", c_float), ("dtype", c_int), ("impl", c_int), ("splits", c_int), ("workspace", c_void_p),
+                ("workspace_floats", c_longlong), ("status", c_void_p)]
+
+
+class MlstmParams(Structure):
+    _fields_ = [("qkv", c_void_p), ("ld_qkv", c_longlong), ("q_off", c_int), ("k_off", c_int), ("v_off", c_int),
+                ("gates", c_void_p), ("ld_gates", c_longlong), ("i_bias", c_void_p), ("f_bias", c_void_p),
+                ("S", c_void_p), ("n", c_void_p), ("m", c_void_p), ("out", c_void_p), ("ld_out", c_longlong),
+                ("positions", c_void_p), ("qo_indptr", c_void_p), ("state_slot", c_void_p),
+                ("req_begin", c_int), ("req_count", c_int), ("heads", c_int), ("dim", c_int), ("vdim", c_int),
+                ("num_slots", c_int), ("gate_cap", c_float), ("q_scale", c_float), ("dtype", c_int), ("impl", c_int),
+                ("items", c_void_p), ("num_items", c_int), ("scratch", c_void_p), ("scratch_floats", c_longlong),
+                ("status", c_void_p)]
+
+
+class HeadNormGateParams(Structure):
+    _fields_ = [("o", c_void_p), ("ld_o", c_longlong), ("g", c_void_p), ("ld_g", c_longlong), ("w", c_void_p),
+                ("out", c_void_p), ("ld_out", c_longlong), ("T", c_int), ("heads", c_int), ("vdim", c_int),
+                ("vdim_p", c_int), ("eps", c_float), ("dtype", c_int)]
 
 
 def library_path() -> Path:

@@ -126,6 +126,18 @@ def build_executor_host(verbose: bool = False, sanitize: str = "") -> Path:
     return out
 
 
+def build_runtime(verbose: bool = False) -> None:
+    """What running a model needs: the kernel library and the executor, if they are missing or out of date. A
+    lock file keeps processes that start together from compiling twice."""
+    import fcntl
+
+    BUILD_DIR.mkdir(exist_ok=True)
+    with open(BUILD_DIR / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        build_kernels(verbose)
+        build_executor(verbose)
+
+
 def build_all(verbose: bool = False) -> None:
     build_kernels(verbose)
     build_executor(verbose)

@@ -42,8 +42,11 @@ DECODE_SPLIT_ROWS = 8192       # workspace rows (request x q head) reserved for 
 class MetaLayout:
     """Offsets (int32 words) of every per-iteration array inside one contiguous metadata block."""
 
-    def __init__(self, T: int, B: int, nano_sizes: List[int], num_pages: int, offload_cap: int = 0):
-        self.T, self.B = T, B
+    def __init__(self, T: int, B: int, nano_sizes: List[int], num_pages: int, offload_cap: int = 0,
+                 sample_rows: int = 0, extra: Optional[Dict[str, int]] = None):
+        """``sample_rows``: most rows sampled in one iteration (0 = one per request). ``extra``: further arrays
+        of a model family, name -> words."""
+        self.T, self.B, self.sample_cap = T, B, sample_rows or B
         off = 0
         self.off: Dict[str, int] = {}
         self.size: Dict[str, int] = {}
@@ -58,17 +61,22 @@ class MetaLayout:
         put("qo_indptr", B + 1)
         put("kv_indptr", B + 1)
         put("kv_last_page_len", B)
-        put("sample_rows", B)
+        put("sample_rows", self.sample_cap)
         self.item_caps = [s + 2 for s in nano_sizes]
         for k, cap in enumerate(self.item_caps):
             put(f"items{k}", cap * 3)
         put("offload_pages", offload_cap)
+        for name, n in (extra or {}).items():
+            put(name, n)
         self.fixed_words = off
         put("kv_indices", num_pages + B)
         self.total_words = off
 
 
 class Engine:
+    """The Llama family's engine, and through the ``_setup`` and ``_stage_model`` hooks the step
+    machinery (staging ring, launches, token feedback, status) of every other family's."""
+
     def __init__(self, cfg: NanoflowConfig, weights: RankWeights, *, device: Optional[torch.device] = None,
                  collectives: Optional[CollectiveHooks] = None, num_pages: Optional[int] = None,
                  executor: str = "auto"):
@@ -79,83 +87,25 @@ class Engine:
         self.device = device or torch.device("cuda", torch.cuda.current_device())
         self.w = weights
         self.coll = collectives or CollectiveHooks()
-        m, e = self.model, self.eng
+        e = self.eng
         if e.page_size != 16:
             raise ValueError("the attention kernels are built for 16-token pages")
-        T, B = e.global_batch_size, e.max_batch_size
         self.nano_sizes = e.resolved_nanobatches()
-        dev, bf = self.device, torch.bfloat16
-
-        def alloc(*shape, dtype=bf):
-            return self.coll.alloc(shape, dtype) if hasattr(self.coll, "alloc") else \
-                torch.zeros(*shape, dtype=dtype, device=dev)
-
         # debug_guards: every local activation buffer sits between guard words that check_status()
         # compares after the iteration (utils/guards.py)
         self.guards = None
         if e.debug_guards:
             from ..utils.guards import GuardedArena
-            self.guards = GuardedArena(dev)
-
-        def plain(*shape, dtype=bf, name="activation"):
-            if self.guards is not None:
-                return self.guards.zeros(name, shape, dtype)
-            return torch.zeros(*shape, dtype=dtype, device=dev)
-
-        # x[0]: residual stream (local). x[1]: under TP the symmetric buffer the K-split GEMMs write
-        # their partial products into (peers pull from it); on one GPU it aliases x[0].
-        x0 = plain(T, m.hidden_size, name="x")
-        x = [x0, alloc(T + 8 * len(self.nano_sizes), m.hidden_size) if weights.tp > 1 else x0]
-        self.num_pages = int(num_pages or e.num_pages or self._derive_num_pages(T, B))
-        # KV offload: pages of requests retired in an iteration are gathered layer by layer and
-        # copied to pinned host memory; at most offload_cap pages per iteration.
-        self.page_bytes_layer = 2 * m.kv_heads_local * e.page_size * m.head_dim * 2
-        self.offload_cap = 0
-        if e.offload:
-            self.offload_cap = max(16, min(2048, OFFLOAD_HOST_BYTES // (m.run_layers * self.page_bytes_layer)))
-        layout = MetaLayout(T, B, self.nano_sizes, self.num_pages, self.offload_cap)
-        self.layout = layout
-        self.meta_dev = torch.zeros(layout.total_words, dtype=torch.int32, device=dev)
-        self.meta_host = [torch.zeros(layout.total_words, dtype=torch.int32).pin_memory() for _ in range(RING)]
-        self.meta_np = [t.numpy() for t in self.meta_host]
-        view = lambda name: self.meta_dev[layout.off[name]:layout.off[name] + layout.size[name]]
-        meta = {n: view(n) for n in ("host_ids", "feedback_src", "positions", "token_req", "qo_indptr",
-                                     "kv_indptr", "kv_last_page_len", "sample_rows", "kv_indices")}
-        nano_items = [view(f"items{k}").view(-1, 3) for k in range(len(self.nano_sizes))]
-        kv_pool = [torch.zeros(self.num_pages, 2, m.kv_heads_local, e.page_size, m.head_dim, dtype=bf, device=dev)
-                   for _ in range(m.run_layers)]
-        self.bufs = Buffers(
-            x=x, h=alloc(T, m.hidden_size) if weights.tp > 1 else plain(T, m.hidden_size, name="h"),
-            qkv=plain(T, m.qkv_size_local, name="qkv"), q_rot=plain(T, m.q_size_local, name="q_rot"),
-            attn_out=plain(T, m.q_size_local, name="attn_out"), act=plain(T, m.ffn_local, name="act"),
-            sample_h=plain(B, m.hidden_size, name="sample_h"), sample_hn=plain(B, m.hidden_size, name="sample_hn"),
-            logits=plain(B, weights.lm_head.shape[0], name="logits"),
-            cand_val=alloc(weights.tp, B, dtype=torch.float32), cand_idx=alloc(weights.tp, B, dtype=torch.int32),
-            sampled=plain(B, dtype=torch.int32, name="sampled"), kv_pool=kv_pool,
-            inv_freq=ref.rope_inv_freq(m.head_dim, m.rope_theta, m.rope_scaling).to(dev),
-            status=torch.zeros(1, dtype=torch.int32, device=dev),
-            decode_ws=torch.empty(DECODE_SPLIT_ROWS * DECODE_MAX_CHUNKS * (m.head_dim + 2), dtype=torch.float32,
-                                  device=dev),
-            meta=meta, nano_items=nano_items,
-            gemm_ws=torch.zeros(GEMM_WS_BYTES // 4, dtype=torch.float32, device=dev),
-            rope_table=torch.zeros(T, m.head_dim // 2, 2, dtype=torch.float32, device=dev),
-            attn_full=alloc(T, m.q_size_local * weights.tp) if (weights.tp > 1 and e.o_allgather_nanos) else None)
-        io = IoSpec(self.meta_dev, layout.fixed_words, layout.off["kv_indices"])
-        self.offload_host = None
-        if self.offload_cap:
-            io.offload_staging = torch.zeros(self.offload_cap, self.page_bytes_layer // 2, dtype=bf, device=dev)
-            io.offload_pages = view("offload_pages")
-            self.offload_host = [torch.zeros(m.run_layers, self.offload_cap, self.page_bytes_layer // 2,
-                                             dtype=bf).pin_memory() for _ in range(RING)]
+            self.guards = GuardedArena(self.device)
         self.gemm_tuning: Dict[str, dict] = {}
-        if e.autotune_gemm:
-            self._autotune_gemms()
-        self.graph: OpGraph = build_graph(m, e, weights, self.bufs, self.coll, io)
-        self.tokens_host = [torch.zeros(B, dtype=torch.int32).pin_memory() for _ in range(RING)]
+        self.offload_cap, self.offload_host = 0, None
+        self._setup(num_pages)
+        S = self.layout.sample_cap
+        self.tokens_host = [torch.zeros(S, dtype=torch.int32).pin_memory() for _ in range(RING)]
         self.tokens_np = [t.numpy() for t in self.tokens_host]
         self.status_host = [torch.zeros(1, dtype=torch.int32).pin_memory() for _ in range(RING)]
         self.status_np = [t.numpy() for t in self.status_host]
-        self.stream = torch.cuda.Stream(device=dev)
+        self.stream = torch.cuda.Stream(device=self.device)
         self.done_events = [torch.cuda.Event() for _ in range(RING)]
         self._staged: Optional[dict] = None
         self._inflight: List[dict] = []
@@ -167,6 +117,79 @@ class Engine:
         self.launches_per_iteration = len(self.graph.ops)
         self.executor_kind = executor
         self._make_executor(executor)
+
+    def _plain(self, *shape, dtype=torch.bfloat16, name="activation") -> torch.Tensor:
+        """A local activation buffer, zeroed (between guard words with debug_guards)."""
+        if self.guards is not None:
+            return self.guards.zeros(name, shape, dtype)
+        return torch.zeros(*shape, dtype=dtype, device=self.device)
+
+    def _make_metadata(self, layout: "MetaLayout") -> None:
+        self.layout = layout
+        self.meta_dev = torch.zeros(layout.total_words, dtype=torch.int32, device=self.device)
+        self.meta_host = [torch.zeros(layout.total_words, dtype=torch.int32).pin_memory() for _ in range(RING)]
+        self.meta_np = [t.numpy() for t in self.meta_host]
+
+    def _meta_view(self, name: str) -> torch.Tensor:
+        lay = self.layout
+        return self.meta_dev[lay.off[name]:lay.off[name] + lay.size[name]]
+
+    def _setup(self, num_pages: Optional[int]) -> None:
+        """Buffers, page pool, metadata block and op graph of the model."""
+        m, e, weights = self.model, self.eng, self.w
+        T, B = e.global_batch_size, e.max_batch_size
+        S = e.max_sample_rows or B
+        dev, bf = self.device, torch.bfloat16
+
+        def alloc(*shape, dtype=bf):
+            return self.coll.alloc(shape, dtype) if hasattr(self.coll, "alloc") else \
+                torch.zeros(*shape, dtype=dtype, device=dev)
+
+        plain = self._plain
+
+        # x[0]: residual stream (local). x[1]: under TP the symmetric buffer the K-split GEMMs write
+        # their partial products into (peers pull from it); on one GPU it aliases x[0].
+        x0 = plain(T, m.hidden_size, name="x")
+        x = [x0, alloc(T + 8 * len(self.nano_sizes), m.hidden_size) if weights.tp > 1 else x0]
+        self.num_pages = int(num_pages or e.num_pages or self._derive_num_pages(T, B))
+        # KV offload: pages of requests retired in an iteration are gathered layer by layer and
+        # copied to pinned host memory; at most offload_cap pages per iteration.
+        self.page_bytes_layer = 2 * m.kv_heads_local * e.page_size * m.head_dim * 2
+        if e.offload:
+            self.offload_cap = max(16, min(2048, OFFLOAD_HOST_BYTES // (m.run_layers * self.page_bytes_layer)))
+        layout = MetaLayout(T, B, self.nano_sizes, self.num_pages, self.offload_cap, S)
+        self._make_metadata(layout)
+        view = self._meta_view
+        meta = {n: view(n) for n in ("host_ids", "feedback_src", "positions", "token_req", "qo_indptr",
+                                     "kv_indptr", "kv_last_page_len", "sample_rows", "kv_indices")}
+        nano_items = [view(f"items{k}").view(-1, 3) for k in range(len(self.nano_sizes))]
+        kv_pool = [torch.zeros(self.num_pages, 2, m.kv_heads_local, e.page_size, m.head_dim, dtype=bf, device=dev)
+                   for _ in range(m.run_layers)]
+        self.bufs = Buffers(
+            x=x, h=alloc(T, m.hidden_size) if weights.tp > 1 else plain(T, m.hidden_size, name="h"),
+            qkv=plain(T, m.qkv_size_local, name="qkv"), q_rot=plain(T, m.q_size_local, name="q_rot"),
+            attn_out=plain(T, m.q_size_local, name="attn_out"), act=plain(T, m.ffn_local, name="act"),
+            sample_h=plain(S, m.hidden_size, name="sample_h"), sample_hn=plain(S, m.hidden_size, name="sample_hn"),
+            logits=plain(S, weights.lm_head.shape[0], name="logits"),
+            cand_val=alloc(weights.tp, S, dtype=torch.float32), cand_idx=alloc(weights.tp, S, dtype=torch.int32),
+            sampled=plain(S, dtype=torch.int32, name="sampled"), kv_pool=kv_pool,
+            inv_freq=ref.rope_inv_freq(m.head_dim, m.rope_theta, m.rope_scaling).to(dev),
+            status=torch.zeros(1, dtype=torch.int32, device=dev),
+            decode_ws=torch.empty(DECODE_SPLIT_ROWS * DECODE_MAX_CHUNKS * (m.head_dim + 2), dtype=torch.float32,
+                                  device=dev),
+            meta=meta, nano_items=nano_items,
+            gemm_ws=torch.zeros(GEMM_WS_BYTES // 4, dtype=torch.float32, device=dev),
+            rope_table=torch.zeros(T, m.head_dim // 2, 2, dtype=torch.float32, device=dev),
+            attn_full=alloc(T, m.q_size_local * weights.tp) if (weights.tp > 1 and e.o_allgather_nanos) else None)
+        io = IoSpec(self.meta_dev, layout.fixed_words, layout.off["kv_indices"])
+        if self.offload_cap:
+            io.offload_staging = torch.zeros(self.offload_cap, self.page_bytes_layer // 2, dtype=bf, device=dev)
+            io.offload_pages = view("offload_pages")
+            self.offload_host = [torch.zeros(m.run_layers, self.offload_cap, self.page_bytes_layer // 2,
+                                             dtype=bf).pin_memory() for _ in range(RING)]
+        if e.autotune_gemm:
+            self._autotune_gemms()
+        self.graph: OpGraph = build_graph(m, e, weights, self.bufs, self.coll, io)
 
     # ---- GEMM shapes --------------------------------------------------------------------------------
     def _autotune_gemms(self) -> None:
@@ -284,10 +307,14 @@ class Engine:
             host = self.offload_host[slot]
             for l in range(self.model.run_layers):
                 sym[f"offload_dst_{l}"] = host.data_ptr() + l * host.stride(0) * host.element_size()
-        cp, mc = self._decode_split(plan)
-        sym["decode_chunk_pages"], sym["decode_max_chunks"] = cp, mc
+        self._stage_model(plan, put, sym)
         self._staged = dict(slot=slot, sym=sym, n_sample=int(plan.sample_rows.size),
                             kv_words=int(plan.kv_indices.size), plan=plan, n_offload=n_off)
+
+    def _stage_model(self, plan: BatchPlan, put, sym: Dict[str, int]) -> None:
+        """Metadata arrays and symbols that only this family's ops use."""
+        cp, mc = self._decode_split(plan)
+        sym["decode_chunk_pages"], sym["decode_max_chunks"] = cp, mc
 
     def _decode_split(self, plan: BatchPlan):
         if self.eng.decode_chunk_pages > 0:
@@ -368,6 +395,11 @@ class Engine:
         self.update(plan)
         self.run_async()
         return self.run_async_wait()
+
+    def last_logits(self, n: int) -> torch.Tensor:
+        """Logits [n, vocab] of the first ``n`` sampled rows of the last iteration (this rank's vocabulary shard)."""
+        torch.cuda.synchronize(self.device)
+        return self.bufs.logits[:n, :self.model.vocab_size].float()
 
     def getPipelineOutput(self) -> np.ndarray:
         return self._last_tokens

@@ -45,7 +45,7 @@ class GatherParams(Structure):
 
 class ArgmaxParams(Structure):
     _fields_ = [("idx_out", c_void_p), ("val_out", c_void_p), ("logits", c_void_p), ("rows", c_int),
-                ("cols", c_int), ("ld", c_longlong), ("col_offset", c_int)]
+                ("cols", c_int), ("ld", c_longlong), ("col_offset", c_int), ("dtype", c_int)]
 
 
 class ArgmaxCombineParams(Structure):
@@ -81,12 +81,19 @@ GemmParams = _ops.GemmParams
 RopeAppendParams = _ops.RopeAppendParams
 RopeTableParams = _ops.RopeTableParams
 AttnParams = _ops.AttnParams
+ResidualNormParams = _ops.ResidualNormParams
+LatentAppendParams = _ops.LatentAppendParams
+LatentAttnParams = _ops.LatentAttnParams
+MlstmParams = _ops.MlstmParams
+HeadNormGateParams = _ops.HeadNormGateParams
 
 KERNEL_OF = {
     GemmParams: "nfk_gemm_bf16", RopeAppendParams: "nfk_rope_append", RopeTableParams: "nfk_rope_table",
     NormParams: "nfk_norm_p",
     EmbeddingParams: "nfk_embedding_p", GatherParams: "nfk_gather_p", ArgmaxParams: "nfk_argmax_p",
     ArgmaxCombineParams: "nfk_argmax_combine_p", CopyColsParams: "nfk_copy_cols_p",
+    ResidualNormParams: "nfk_residual_norm", LatentAppendParams: "nfk_latent_append",
+    LatentAttnParams: "nfk_latent_attn", HeadNormGateParams: "nfk_head_norm_gate",
     MemcpyParams: "nfk_memcpy_p", Memcpy2DParams: "nfk_memcpy2d_p", KvMoveParams: "nfk_kv_move_p", SleepParams: "nfk_sleep_p",
 }
 

@@ -1,0 +1,507 @@
+"""Engine of layer-list models (:mod:`..models.layer_list`): buffers, caches and the op graph of one iteration.
+
+Everything around the graph (staging of the batch metadata, launches, token feedback on the device,
+status word) is :class:`.engine.Engine`; this module says what an iteration consists of. One nano-batch,
+one GPU, one stream. Per layer run:
+
+* the packed input projection of the mixer (gate pre-activations leave it in fp32);
+* latent attention: latents normed into the paged pool, then two ways to attend, chosen per portion when the
+  batch is staged. Single tokens and short portions (and everything in 32-bit) stay in latent space: the
+  queries are multiplied by their heads' key matrices (one block-diagonal GEMM), the kernel reads the cached
+  rows as keys and values at once, and a second block-diagonal GEMM applies the value matrices. Longer
+  portions gather the latents they can see, expand them to keys and values of all heads with one GEMM, and
+  run the tcgen05 prefill kernel over those;
+* mLSTM: one kernel for requests with one token, one for longer portions, then head norm and output gate;
+* output projection, and one kernel for: norm of the sublayer's output, residual sum in fp32, the step
+  vector of a loop pass, and the norm the next sublayer reads.
+
+A new kind of mixer needs a spec and weights in ``models/layer_list.py`` and a builder in ``MIXERS``.
+"""
+from __future__ import annotations
+
+from ctypes import c_void_p
+from typing import Dict, List, Optional, Tuple
+
+import numpy as np
+import torch
+
+from .. import ops
+from ..models.layer_list import PREFILL_HEAD_DIM, LayerListConfig, NormWeights, round8
+from ..ops import ACTS, NORMS, dtype_code
+from ..serving.scheduler import BatchPlan
+from .engine import GEMM_WS_BYTES, Engine, MetaLayout
+from .graph import (ArgmaxParams, AttnParams, GemmParams, HeadNormGateParams, KvMoveParams, LatentAppendParams,
+                    LatentAttnParams, MemcpyParams, MlstmParams, OpGraph, ResidualNormParams)
+from .pipeline import _ptr
+
+PAGE = 16
+QUERY_TILE = 128             # query tokens per work item of the prefill attention kernel
+MLSTM_CHUNK = 64             # tokens per chunk of the chunked mLSTM kernel
+MLSTM_COLS = 64              # columns of the state per CTA of that kernel
+SEGMENT_ITEMS = 48           # most segments that prompt portions are cut into for the mLSTM kernel
+
+
+class PathGroup:
+    """Latent-attention layers that share their work lists: same window, same choice of paths."""
+
+    def __init__(self, index: int, window: int, expands: bool):
+        self.index, self.window, self.expands = index, window, expands
+
+    def name(self, what: str) -> str:
+        return f"{what}{self.index}"
+
+
+class LayerListEngine(Engine):
+    model: LayerListConfig
+
+    # ---- set-up -------------------------------------------------------------------------------------
+    def _setup(self, num_pages: Optional[int]) -> None:
+        m, e = self.model, self.eng
+        if len(self.nano_sizes) != 1 or e.overlap:
+            raise ValueError("layer-list models run in one nano-batch on one stream (pipeline_type NON_OVERLAP_LOCAL)")
+        if e.offload:
+            raise ValueError("KV offload is not built for layer-list models")
+        T, B = e.global_batch_size, e.max_batch_size
+        self.T, self.B = T, B
+        self.S_cap = e.max_sample_rows or B
+        self.code = dtype_code(m.dtype)
+        self.gemm_kernel = "nfk_gemm_f32" if m.dtype == torch.float32 else "nfk_gemm_bf16"
+        self.num_slots = (e.state_slots or B) if m.has_state else 0
+        self.groups: List[PathGroup] = []
+        for s in m.run_specs("latent_attention"):
+            key = (s.window or 0, m.expands(s))
+            if not any((g.window, g.expands) == key for g in self.groups):
+                self.groups.append(PathGroup(len(self.groups), *key))
+        self.x_pages = self._expand_pages()
+        self._alloc_state()
+        self.num_pages = int(num_pages or e.num_pages or self._derive_num_pages(T, B))
+        extra = {"kv_first": B, "state_ref": B}
+        for g in self.groups:
+            extra[g.name("abs")] = T
+            if g.expands:
+                extra.update({g.name("xptr"): B + 1, g.name("xpage"): self.x_pages, g.name("xitem"): 3 * (T // QUERY_TILE + B + 1)})
+        if m.has_state:
+            extra["segs"] = 4 * max(B, SEGMENT_ITEMS)
+        self._make_metadata(MetaLayout(T, B, self.nano_sizes, self.num_pages, 0, self.S_cap, extra))
+        self.meta = {n: self._meta_view(n) for n in self.layout.off}
+        self._alloc_buffers()
+        if e.autotune_gemm and m.dtype == torch.bfloat16:
+            self._autotune()
+        self.graph = self._build_graph()
+
+    def _expand_pages(self) -> int:
+        """Pages of latents that one iteration can expand to keys and values."""
+        if not any(g.expands for g in self.groups):
+            return 0
+        rows = self.eng.expand_rows
+        if rows <= 0:
+            window = max(g.window for g in self.groups if g.expands)
+            if any(g.expands and g.window == 0 for g in self.groups):
+                window = 8192
+            rows = self.T + 8 * (window + 2 * PAGE)
+        return max(2, (rows + PAGE - 1) // PAGE)
+
+    def _alloc_state(self) -> None:
+        m, dev = self.model, self.device
+        self.state: List[Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]]] = []
+        for r in m.runs:
+            s = m.layers[r.layer].mixer
+            if s.kind != "mlstm":
+                self.state.append(None)
+                continue
+            d, v, n = round8(s.dim), round8(s.vdim), self.num_slots
+            z = lambda *shape: torch.zeros(*shape, dtype=torch.float32, device=dev)
+            self.state.append((z(n, s.heads, d, v), z(n, s.heads, 2, d), z(n, s.heads, 2)))
+
+    def _widths(self) -> Dict[str, int]:
+        """Columns of the shared activation buffers (the widest layer's)."""
+        m = self.model
+        w = dict(proj=8, gates=8, attn=8, q_lat=0, o_lat=0, o_rec=8, act=8, kv=0, cg=0)
+        up = lambda k, n: w.__setitem__(k, max(w[k], n))
+        for lay in m.layers:
+            s = lay.mixer
+            if s.kind == "latent_attention":
+                dq, dv = m.head_pads(s)
+                ld = m.latent_ld(s)
+                up("proj", s.heads * dq + round8(s.kv_rank))
+                up("attn", s.heads * dv)
+                up("q_lat", s.heads * ld)
+                if m.expands(s):
+                    up("kv", s.heads * 2 * PREFILL_HEAD_DIM)
+                    up("cg", ld)
+            else:
+                d, v = round8(s.dim), round8(s.vdim)
+                up("proj", s.heads * 2 * (d + v))
+                up("gates", round8(2 * s.heads))
+                up("o_rec", s.heads * v)
+                up("attn", s.heads * v)
+            if lay.mlp is not None:
+                up("act", round8(lay.mlp.ff))
+        return w
+
+    def _derive_num_pages(self, T: int, B: int) -> int:
+        m, e = self.model, self.eng
+        free, total = torch.cuda.mem_get_info(self.device)
+        w = self._widths()
+        es = m.elem_bytes
+        act = T * (4 * m.width_p + es * (2 * m.width_p + w["proj"] + w["attn"] + 2 * w["q_lat"] + w["act"]) +
+                   4 * (w["gates"] + w["o_rec"]))
+        act += self.x_pages * PAGE * (w["kv"] + w["cg"]) * es + self.S_cap * (es * m.width_p + 4 * m.vocab_p)
+        budget = free - total * (1.0 - e.gpu_mem_fraction) - act - (1 << 30)
+        per_page = max(1, m.kv_bytes_per_token_local()) * PAGE
+        n = int(min(budget // per_page, 1 << 22))
+        if n < 64:
+            raise RuntimeError(f"not enough GPU memory for a latent pool ({free >> 20} MiB free)")
+        return n
+
+    def _alloc_buffers(self) -> None:
+        m, T, dev = self.model, self.T, self.device
+        dt, f32, w = m.dtype, torch.float32, self._widths()
+        P = lambda rows, cols, dtype=dt, name="": self._plain(rows, cols, dtype=dtype, name=name)
+        self.x = P(T, m.width_p, f32, "x")
+        self.h = P(T, m.width_p, dt, "h")
+        self.y = P(T, m.width_p, dt, "y")
+        flat = lambda k, dtype, rows=T: P(1, max(8, rows * w[k]), dtype, k).view(-1)
+        self.flat = {"proj": flat("proj", dt), "attn": flat("attn", dt), "act": flat("act", dt), "gates": flat("gates", f32),
+                     "o_rec": flat("o_rec", f32), "q_lat": flat("q_lat", dt), "o_lat": flat("q_lat", dt),
+                     "kv": flat("kv", dt, self.x_pages * PAGE), "cg": flat("cg", dt, self.x_pages * PAGE)}
+        self.h_s = P(self.S_cap, m.width_p, dt, "sample_h")
+        self.logits = P(self.S_cap, m.vocab_p, f32, "logits")
+        self.pools = [torch.zeros(self.num_pages, PAGE, m.latent_ld(s.mixer), dtype=dt, device=dev)
+                      if s.mixer.kind == "latent_attention" else None for s in (m.layers[r.layer] for r in m.runs)]
+        self.arange = torch.arange(self.x_pages + 1, dtype=torch.int32, device=dev)
+        heads = max([s.heads * (m.latent_ld(s) + 2) for s in m.run_specs("latent_attention")], default=0)
+        self.latent_ws = torch.empty(max(8, 160 * heads), dtype=f32, device=dev)
+        seg = max([s.heads * (round8(s.dim) * round8(s.vdim) + round8(s.dim) + 8) for s in m.run_specs("mlstm")], default=0)
+        self.seg_ws = torch.empty(max(8, SEGMENT_ITEMS * seg if dt == torch.bfloat16 else 8), dtype=f32, device=dev)
+        self.gemm_ws = torch.zeros(GEMM_WS_BYTES // 4, dtype=f32, device=dev) if dt == torch.bfloat16 else None
+        self.taps = P(len(m.runs) * T, m.width_p, f32, "taps").view(len(m.runs), T, m.width_p) \
+            if self.eng.tap_residual else None
+
+        class _Bufs:                      # the members Engine reads
+            pass
+        self.bufs = _Bufs()
+        self.bufs.sampled = self._plain(self.S_cap, dtype=torch.int32, name="sampled")
+        self.bufs.status = torch.zeros(1, dtype=torch.int32, device=dev)
+        self.bufs.logits = self.logits
+
+    def view(self, name: str, cols: int, rows: Optional[int] = None) -> torch.Tensor:
+        rows = rows or self.T
+        return self.flat[name][:rows * cols].view(rows, cols)
+
+    # ---- graph --------------------------------------------------------------------------------------
+    def _build_graph(self) -> OpGraph:
+        m, w = self.model, self.w
+        g = self.g = OpGraph()
+        self.last_op: Optional[int] = None
+        T = g.symbol("T")
+        for s in ("nb0_T", "nb0_items", "nb0_dec_begin", "nb0_dec_count", "n_sample", "n_dec", "n_pre"):
+            g.symbol(s)
+        lay = self.layout
+        self._op("meta_h2d", MemcpyParams(dst=_ptr(self.meta_dev), src=c_void_p(0), elem_bytes=4, count=lay.fixed_words),
+                 dyn=[("src", g.symbol("meta_src"))])
+        self._op("kv_indices_h2d", MemcpyParams(dst=c_void_p(self.meta_dev.data_ptr() + 4 * lay.off["kv_indices"]),
+                                                src=c_void_p(0), elem_bytes=4, count=0),
+                 dyn=[("src", g.symbol("kv_src")), ("count", g.symbol("kv_words"))])
+        # the stream's step before each run, as (vector added, norm of its mixer's input)
+        step = lambda r: None if m.runs[r].step is None else w.loop_steps[m.runs[r].step]
+        self._residual("embedding", None, w.embed_norm, w.layers[m.runs[0].layer].norm_in, step(0), embed=True)
+        for r, run in enumerate(m.runs):
+            spec, lw = m.layers[run.layer], w.layers[run.layer]
+            last = r + 1 == len(m.runs)
+            nxt = None if last else w.layers[m.runs[r + 1].layer].norm_in
+            add = None if last else step(r + 1)
+            MIXERS[spec.mixer.kind](self, r, run.layer, spec.mixer, lw.mixer)
+            if spec.mlp is not None:
+                self._residual(f"R{r}.mid", self.y, lw.norm_out, lw.mlp_in, None, layer=r)
+                act = self.view("act", round8(spec.mlp.ff))
+                self._gemm(f"R{r}.gate_up", self.h, lw.w_gate, act, rows=T, up=lw.w_up, act=spec.mlp.act,
+                           key=f"l{run.layer}.gate_up", layer=r)
+                self._gemm(f"R{r}.down", act, lw.w_down, self.y, rows=T, key=f"l{run.layer}.down", layer=r)
+            out = lw.mlp_out if spec.mlp is not None else lw.norm_out
+            if last and self.taps is None:
+                # only the sampled rows go on
+                self._residual("final", self.y, out, w.final_norm, None, sampled=True)
+            else:
+                tap_add = add if self.taps is None else None
+                self._residual(f"R{r}.out", self.y, out, None if (last or self.taps is not None) else nxt, tap_add, layer=r)
+                if self.taps is not None:
+                    self._op(f"R{r}.tap", MemcpyParams(dst=_ptr(self.taps[r]), src=_ptr(self.x), elem_bytes=4 * m.width_p,
+                                                       count=0), dyn=[("count", T)], layer=r)
+                    if last:
+                        self._residual("final", None, None, w.final_norm, None, sampled=True)
+                    else:
+                        self._residual(f"R{r}.next", None, None, nxt, add, layer=r)
+        S = g.symbol("n_sample")
+        self._gemm("lm_head", self.h_s, w.lm_head, None, rows=S, d32=self.logits)
+        self._op("argmax", ArgmaxParams(idx_out=_ptr(self.bufs.sampled), val_out=c_void_p(0), logits=_ptr(self.logits),
+                                        rows=0, cols=m.vocab_size, ld=self.logits.stride(0), col_offset=0, dtype=ops.F32),
+                 dyn=[("rows", S)])
+        self._op("tokens_d2h", MemcpyParams(dst=c_void_p(0), src=_ptr(self.bufs.sampled), elem_bytes=4, count=0),
+                 dyn=[("dst", g.symbol("tokens_dst")), ("count", S)])
+        self._op("status_d2h", MemcpyParams(dst=c_void_p(0), src=_ptr(self.bufs.status), elem_bytes=4, count=1),
+                 dyn=[("dst", g.symbol("status_dst"))])
+        return g
+
+    def _op(self, name, params, *, dyn=(), kernel=None, layer=-1) -> None:
+        self.last_op = self.g.add(name, params, "gemm", deps=[] if self.last_op is None else [self.last_op], dyn=dyn,
+                                  kernel=kernel, layer=layer, nano=0)
+
+    def _residual(self, name, y, norm_in: Optional[NormWeights], norm_out: Optional[NormWeights], add, *, embed=False,
+                  sampled=False, layer=-1) -> None:
+        m, kind = self.model, NORMS[self.model.norm_kind]
+        p = ResidualNormParams()
+        p.x, p.ld_x = _ptr(self.x), self.x.stride(0)
+        if embed:
+            p.table, p.ld_table, p.vocab = _ptr(self.w.embed), self.w.embed.stride(0), m.vocab_size
+            p.host_ids, p.feedback_src = _ptr(self.meta["host_ids"]), _ptr(self.meta["feedback_src"])
+            p.prev_tokens = _ptr(self.bufs.sampled)
+        elif y is not None:
+            p.y, p.ld_y = _ptr(y), y.stride(0)
+        if norm_in is not None:
+            p.in_w, p.in_b, p.in_kind = _ptr(norm_in.w), _ptr(norm_in.b), kind
+        p.add = _ptr(add)
+        if norm_out is not None:
+            h = self.h_s if sampled else self.h
+            p.h, p.ld_h, p.out_w, p.out_b, p.out_kind = _ptr(h), h.stride(0), _ptr(norm_out.w), _ptr(norm_out.b), kind
+        if sampled:
+            p.rows_idx, p.in_rows = _ptr(self.meta["sample_rows"]), self.T
+        p.cols, p.eps, p.dtype, p.status = m.hidden_size, m.norm_eps, self.code, _ptr(self.bufs.status)
+        self._op(name, p, dyn=[("rows", "n_sample" if sampled else "T")], layer=layer)
+
+    def _gemm(self, name, a, wt, out, *, rows: str, up=None, act="silu", d32=None, f32_col0=0, groups=1, group_k=0, k=0,
+              key="", layer=-1) -> None:
+        """out[rows, N] = a @ wt^T. ``d32``: columns from ``f32_col0`` on leave as fp32; ``groups`` > 1:
+        block-diagonal (each group of rows of ``wt`` sees ``k`` columns of ``a``, ``group_k`` apart)."""
+        p = GemmParams()
+        p.A, p.B, p.B2, p.D = _ptr(a), _ptr(wt), _ptr(up), _ptr(out)
+        p.lda, p.ldb, p.ldd = a.stride(0), wt.stride(0), (out.stride(0) if out is not None else wt.shape[0])
+        p.N, p.K = wt.shape[0], k or wt.shape[1]
+        p.epilogue, p.act = (1 if up is not None else 0), ACTS[act]
+        if d32 is not None:
+            p.D32, p.ld32, p.f32_col0 = _ptr(d32), d32.stride(0), f32_col0
+        p.groups, p.group_k = groups, group_k
+        p.status = _ptr(self.bufs.status)
+        if self.gemm_ws is not None:
+            p.workspace, p.workspace_bytes = _ptr(self.gemm_ws), self.gemm_ws.numel() * 4
+        shape = self.eng.gemm_shapes.get(key)
+        if shape is not None:
+            p.tile_m, p.tile_n, p.cta_group = shape["tile_m"], shape["tile_n"], shape["cta_group"]
+            p.split_k, p.stream_k = shape["split_k"], shape["stream_k"]
+        self._op(name, p, dyn=[("M", rows)], kernel=self.gemm_kernel, layer=layer)
+
+    # ---- mixers: read self.h, leave their output projection in self.y ---------------------------------
+    def _latent_attention(self, r: int, layer: int, s, lw) -> None:
+        m, g, T = self.model, self.g, "T"
+        dq, dv = m.head_pads(s)
+        H, ld, pool = s.heads, m.latent_ld(s), self.pools[r]
+        pg = next(x for x in self.groups if (x.window, x.expands) == (s.window or 0, m.expands(s)))
+        meta, st = self.meta, _ptr(self.bufs.status)
+        proj = self.view("proj", H * dq + round8(s.kv_rank))
+        self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, key=f"l{layer}.in", layer=r)
+        ap = LatentAppendParams(src=c_void_p(proj.data_ptr() + H * dq * proj.element_size()), ld_src=proj.stride(0),
+                                w=_ptr(lw.dkv_norm), pool=_ptr(pool), ld=ld, positions=_ptr(meta["positions"]),
+                                token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
+                                kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), T=0, rank=s.kv_rank,
+                                page_size=PAGE, num_pages=self.num_pages, eps=m.norm_eps, dtype=self.code, status=st)
+        self._op(f"R{r}.latent_append", ap, dyn=[("T", T)], layer=r)
+        # in latent space
+        rows, n_abs = g.symbol(pg.name("abs_rows")), g.symbol(pg.name("n_abs"))
+        q_lat, o_lat, attn = self.view("q_lat", H * ld), self.view("o_lat", H * ld), self.view("attn", H * dv)
+        self._gemm(f"R{r}.q_latent", proj, lw.w_qk, q_lat, rows=rows, groups=H, group_k=dq, layer=r)
+        lp = LatentAttnParams(q=_ptr(q_lat), ld_q=q_lat.stride(0), pool=_ptr(pool), ld=ld, out=_ptr(o_lat),
+                              ld_out=o_lat.stride(0), tokens=_ptr(meta[pg.name("abs")]), positions=_ptr(meta["positions"]),
+                              token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
+                              kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), sinks=_ptr(lw.sinks),
+                              n_tokens=0, heads=H, page_size=PAGE, num_pages=self.num_pages, window=s.window or 0,
+                              scale=s.scale, dtype=self.code, impl=0, splits=1, workspace=_ptr(self.latent_ws),
+                              workspace_floats=self.latent_ws.numel(), status=st)
+        self._op(f"R{r}.latent_attn", lp, dyn=[("n_tokens", n_abs), ("splits", g.symbol(pg.name("splits")))], layer=r)
+        self._gemm(f"R{r}.v_latent", o_lat, lw.w_ov, attn, rows=rows, groups=H, group_k=ld, layer=r)
+        # expanded keys and values
+        if pg.expands:
+            n_x = g.symbol(pg.name("n_xpages"))
+            kv_cols = H * 2 * PREFILL_HEAD_DIM
+            cg, kv = self.view("cg", ld, self.x_pages * PAGE), self.view("kv", kv_cols, self.x_pages * PAGE)
+            mp = KvMoveParams(pool=_ptr(pool), staging=_ptr(cg), page_ids=_ptr(meta[pg.name("xpage")]), n_pages=0,
+                              page_bytes=PAGE * ld * pool.element_size(), num_pages=self.num_pages, direction=0,
+                              num_ctas=8 * ops.sm_count(self.device), status=st)
+            self._op(f"R{r}.latent_gather", mp, dyn=[("n_pages", n_x)], layer=r)
+            self._gemm(f"R{r}.expand", cg, lw.w_kv, kv, rows=g.symbol(pg.name("x_rows")), layer=r)
+            pp = AttnParams()
+            pp.q, pp.out, pp.kv_pool = _ptr(proj), _ptr(attn), _ptr(kv)
+            pp.qo_indptr, pp.kv_indptr = _ptr(meta["qo_indptr"]), _ptr(meta[pg.name("xptr")])
+            pp.kv_indices, pp.kv_last_page_len = _ptr(self.arange), _ptr(meta["kv_last_page_len"])
+            pp.q_heads = pp.kv_heads = H
+            pp.head_dim, pp.page_size, pp.num_pages, pp.sm_scale = PREFILL_HEAD_DIM, PAGE, self.x_pages, s.scale
+            pp.items, pp.status = _ptr(meta[pg.name("xitem")]), st
+            pp.window, pp.sinks = s.window or 0, _ptr(lw.sinks)
+            pp.kv_ld, pp.k_col, pp.v_col = kv_cols, 0, H * PREFILL_HEAD_DIM
+            pp.q_rows, pp.ld_q = self.T, proj.stride(0)
+            self._op(f"R{r}.attn_prefill", pp, kernel="nfk_attn_prefill_ws", dyn=[("num_items", g.symbol(pg.name("n_xitems")))],
+                     layer=r)
+        self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
+
+    def _mlstm(self, r: int, layer: int, s, lw) -> None:
+        m, T, meta = self.model, "T", self.meta
+        H, d, v = s.heads, round8(s.dim), round8(s.vdim)
+        main = H * 2 * (d + v)
+        proj, gates = self.view("proj", main), self.view("gates", round8(2 * H))
+        o_rec, attn = self.view("o_rec", H * v), self.view("attn", H * v)
+        self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, d32=gates, f32_col0=main, key=f"l{layer}.in", layer=r)
+        S, n, mx = self.state[r]
+
+        def params() -> MlstmParams:
+            return MlstmParams(
+                qkv=_ptr(proj), ld_qkv=proj.stride(0), q_off=0, k_off=H * d, v_off=2 * H * d, gates=_ptr(gates),
+                ld_gates=gates.stride(0), i_bias=_ptr(lw.i_b), f_bias=_ptr(lw.f_b), S=_ptr(S), n=_ptr(n), m=_ptr(mx),
+                out=_ptr(o_rec), ld_out=o_rec.stride(0), positions=_ptr(meta["positions"]),
+                qo_indptr=_ptr(meta["qo_indptr"]), state_slot=_ptr(meta["state_ref"]), req_begin=0, req_count=0, heads=H,
+                dim=d, vdim=v, num_slots=self.num_slots, gate_cap=s.gate_cap, q_scale=s.dim ** -0.5, dtype=self.code,
+                impl=0, items=_ptr(meta["segs"]), num_items=0, scratch=_ptr(self.seg_ws),
+                scratch_floats=self.seg_ws.numel(), status=_ptr(self.bufs.status))
+
+        self._op(f"R{r}.mlstm_decode", params(), kernel="nfk_mlstm_decode", dyn=[("req_count", "n_dec")], layer=r)
+        self._op(f"R{r}.mlstm_prefill", params(), kernel="nfk_mlstm_prefill",
+                 dyn=[("req_begin", "n_dec"), ("req_count", "n_pre"), ("num_items", self.g.symbol("n_segs"))], layer=r)
+        g_cols = c_void_p(proj.data_ptr() + (2 * H * d + H * v) * proj.element_size())
+        hp = HeadNormGateParams(o=_ptr(o_rec), ld_o=o_rec.stride(0), g=g_cols, ld_g=proj.stride(0), w=_ptr(lw.norm),
+                                out=_ptr(attn), ld_out=attn.stride(0), T=0, heads=H, vdim=s.vdim, vdim_p=v, eps=m.norm_eps,
+                                dtype=self.code)
+        self._op(f"R{r}.head_norm", hp, dyn=[("T", T)], layer=r)
+        self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
+
+    # ---- GEMM shapes ----------------------------------------------------------------------------------
+    def _autotune(self) -> None:
+        """Measured shapes for the dense products of every distinct layer at the full batch size."""
+        from ..ops import autotune
+        m, T, done = self.model, self.T, {}
+        self.h.normal_()
+        for k in ("attn", "act"):
+            self.flat[k].normal_()
+        for i, lay in enumerate(m.layers):
+            lw = self.w.layers[i]
+            specs = [("in", self.h, lw.mixer.w_in, None, self.flat["proj"]), ("o", None, lw.mixer.w_o, None, None)]
+            if lay.mlp is not None:
+                specs += [("gate_up", self.h, lw.w_gate, lw.w_up, self.flat["act"]), ("down", None, lw.w_down, None, None)]
+            for key, a, wt, up, out in specs:
+                name = f"l{i}.{key}"
+                if name in self.eng.gemm_shapes:
+                    continue
+                if a is None:
+                    a = self.view("attn" if key == "o" else "act", wt.shape[1])
+                n = wt.shape[0]
+                if out is not None and T * n > out.numel():
+                    n = out.numel() // T // 8 * 8          # the fp32 gate columns have no place in the bf16 buffer
+                    wt = wt[:n]
+                dst = self.y if out is None else out[:T * n].view(T, n)
+                sig = (key, n, wt.shape[1], up is not None)
+                if sig not in done:
+                    done[sig] = autotune.tune_gemm(a, [wt], dst, weights_up=None if up is None else [up], workspace=self.gemm_ws)
+                res = done[sig]
+                self.eng.gemm_shapes[name] = dict(res["best"])
+                self.gemm_tuning[name] = dict(M=T, best=res["best"], us=res["us"], auto_us=res["auto_us"])
+        torch.cuda.synchronize(self.device)
+        for t in (self.h, self.y, *self.flat.values()):
+            t.zero_()
+
+    # ---- per iteration ----------------------------------------------------------------------------------
+    def _stage_model(self, plan: BatchPlan, put, sym: Dict[str, int]) -> None:
+        if plan.num_tail_decode:
+            raise ValueError("layer-list models take their decode requests at the front of the batch")
+        m, D, P, B = self.model, plan.num_decode, len(plan.prefill), plan.num_requests
+        put("kv_first", plan.kv_first)
+        put("state_ref", plan.state_ref)
+        sym["n_dec"], sym["n_pre"] = D, P
+        qo, span = plan.qo_indptr, np.diff(plan.qo_indptr)
+        if m.has_state:
+            segs = mlstm_segments(qo, D, self._segment_ctas(), ops.sm_count(self.device))
+            put("segs", segs.reshape(-1))
+            sym["n_segs"] = segs.shape[0]
+        for g in self.groups:
+            work = route_attention(plan, g.window, g.expands, self.x_pages, self.eng.expand_min_tokens)
+            put(g.name("abs"), work["abs"])
+            n_abs = int(work["abs"].size)
+            sym[g.name("n_abs")] = n_abs
+            sym[g.name("abs_rows")] = int(work["abs"].max()) + 1 if n_abs else 0
+            ctx = plan.max_kv_pages * PAGE
+            sym[g.name("splits")] = self._latent_splits(n_abs, min(ctx, g.window + PAGE) if g.window else ctx)
+            if g.expands:
+                put(g.name("xptr"), work["xptr"])
+                put(g.name("xpage"), work["xpage"])
+                put(g.name("xitem"), work["items"].reshape(-1))
+                sym[g.name("n_xpages")] = int(work["xpage"].size)
+                sym[g.name("x_rows")] = int(work["xpage"].size) * PAGE
+                sym[g.name("n_xitems")] = int(work["items"].shape[0])
+
+    def _segment_ctas(self) -> int:
+        """CTAs of the chunked mLSTM kernel per segment (of the layer with the fewest)."""
+        return min(s.heads * ((s.vdim + MLSTM_COLS - 1) // MLSTM_COLS) for s in self.model.run_specs("mlstm"))
+
+    def _latent_splits(self, n_abs: int, ctx: int) -> int:
+        """Key ranges per token, so that a few tokens still occupy the SMs (at least four 64-key tiles each)."""
+        if n_abs == 0:
+            return 1
+        groups = max((s.heads + 31) // 32 for s in self.model.run_specs("latent_attention"))
+        return int(max(1, min(16, ctx // 256, ops.sm_count(self.device) // (n_abs * groups))))
+
+    def last_logits(self, n: int) -> torch.Tensor:
+        """fp32 logits [n, vocab] of the first ``n`` sampled rows of the last iteration."""
+        torch.cuda.synchronize(self.device)
+        return self.logits[:n, :self.model.vocab_size]
+
+
+MIXERS = {"latent_attention": LayerListEngine._latent_attention, "mlstm": LayerListEngine._mlstm}
+
+
+# --------------------------------------------------------------------------------------------------
+# Work lists (host side, no GPU needed)
+# --------------------------------------------------------------------------------------------------
+def mlstm_segments(qo_indptr: np.ndarray, n_dec: int, ctas_per_segment: int, sms: int) -> np.ndarray:
+    """Rows (request, first token, tokens, segment) for the chunked mLSTM kernel. A portion is one segment unless
+    the portions alone leave most SMs idle; then long ones are cut into equal runs of whole chunks."""
+    reqs = np.arange(n_dec, qo_indptr.size - 1)
+    lens = np.diff(qo_indptr)[n_dec:]
+    if reqs.size == 0:
+        return np.zeros((0, 4), dtype=np.int32)
+    target = 2 * sms // max(1, ctas_per_segment)
+    seg_len = int(lens.max())
+    if reqs.size < target and reqs.size < SEGMENT_ITEMS:
+        room = min(target, SEGMENT_ITEMS) - reqs.size
+        seg_len = max(4 * MLSTM_CHUNK, -(-int(lens.sum()) // room))
+        seg_len = (seg_len + MLSTM_CHUNK - 1) // MLSTM_CHUNK * MLSTM_CHUNK
+    out = []
+    for b, n in zip(reqs, lens):
+        for k, t in enumerate(range(0, int(n), seg_len)):
+            out.append((b, qo_indptr[b] + t, min(seg_len, n - t), k))
+    return np.asarray(out, dtype=np.int32)
+
+
+def route_attention(plan: BatchPlan, window: int, expands: bool, page_cap: int, min_tokens: int) -> dict:
+    """Which tokens attend in latent space (``abs``) and, for the portions that do not, the latent pages to
+    expand (``xpage``, per-request ranges ``xptr`` of the expanded pages) and the prefill kernel's work items.
+    A portion whose pages do not fit what is left of ``page_cap`` stays in latent space."""
+    D, B, qo = plan.num_decode, plan.num_requests, plan.qo_indptr
+    if not expands:
+        return dict(abs=np.arange(plan.num_tokens, dtype=np.int32))
+    toks = [np.arange(qo[D], dtype=np.int32)]
+    pages, items = [], []
+    xptr = np.zeros(B + 1, dtype=np.int32)
+    used = 0
+    for b in range(D, B):
+        q0, q1 = int(qo[b]), int(qo[b + 1])
+        start, end = int(plan.positions[q0]), int(plan.positions[q1 - 1])
+        lo = max(0, start - window + 1) if window else 0
+        first, n = lo // PAGE, end // PAGE - lo // PAGE + 1
+        if q1 - q0 < min_tokens or used + n > page_cap:
+            toks.append(np.arange(q0, q1, dtype=np.int32))
+        else:
+            p0 = int(plan.kv_indptr[b]) + first - int(plan.kv_first[b])
+            pages.append(plan.kv_indices[p0:p0 + n])
+            t = np.arange(q0, q1, QUERY_TILE, dtype=np.int32)
+            items.append(np.stack([np.full_like(t, b), t, np.minimum(QUERY_TILE, q1 - t)], axis=1))
+            used += n
+        xptr[b + 1] = used
+    cat = lambda parts, empty: np.concatenate(parts).astype(np.int32, copy=False) if parts else empty
+    return dict(abs=np.concatenate(toks), xptr=xptr, xpage=cat(pages, np.zeros(0, dtype=np.int32)),
+                items=cat(items, np.zeros((0, 3), dtype=np.int32)))

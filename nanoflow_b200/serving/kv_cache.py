@@ -10,7 +10,7 @@ raises :class:`KVPoolExhausted` instead of tripping an ``assert``, and batch fla
 """
 from __future__ import annotations
 
-from typing import List, Sequence
+from typing import List, Optional, Sequence
 
 import numpy as np
 
@@ -65,16 +65,49 @@ class DistKVPool:
         self.free_pages([idx])
 
 
+class StateSlotsExhausted(KVPoolExhausted):
+    """Raised when a request needs a recurrent-state slot and none is free."""
+
+
+class StateSlotPool:
+    """Slots of the recurrent state of models that carry one: a request owns one slot from its first
+    scheduled token until it is released. Lowest free slot first."""
+
+    def __init__(self, num_slots: int):
+        self.num_slots = int(num_slots)
+        self._free = list(range(self.num_slots - 1, -1, -1))
+
+    @property
+    def num_free(self) -> int:
+        return len(self._free)
+
+    def alloc(self) -> int:
+        if not self._free:
+            raise StateSlotsExhausted(f"all {self.num_slots} state slots are in use")
+        return self._free.pop()
+
+    def free(self, slot: int) -> None:
+        if not 0 <= slot < self.num_slots or slot in self._free:
+            raise ValueError(f"state slot {slot} is invalid or already free")
+        self._free.append(slot)
+
+
 class DistKVCache:
-    """Page list and length of one request. ``allocate_tokens`` grows it, ``release`` frees it."""
+    """What one request holds on the device: its page list and length, and with a ``state_pool`` a slot of
+    recurrent state. ``allocate_tokens`` grows it, ``trim`` gives back pages that no window reaches any more,
+    ``release`` frees everything."""
 
-    __slots__ = ("_pool", "_pages", "_npages", "_seqlen")
+    __slots__ = ("_pool", "_pages", "_npages", "_seqlen", "_first", "_state_pool", "state_slot", "_state_half")
 
-    def __init__(self, pool: DistKVPool):
+    def __init__(self, pool: DistKVPool, state_pool: Optional[StateSlotPool] = None):
         self._pool = pool
         self._pages = np.empty(8, dtype=np.int32)
         self._npages = 0
         self._seqlen = 0
+        self._first = 0                     # page slots before this one have been given back
+        self._state_pool = state_pool
+        self.state_slot = -1
+        self._state_half = 0
 
     @property
     def seqlen(self) -> int:
@@ -82,13 +115,28 @@ class DistKVCache:
 
     @property
     def indicies(self) -> np.ndarray:  # spelling kept from the reference API
-        return self._pages[:self._npages]
+        return self._pages[self._first:self._npages]
 
     indices = indicies
 
     @property
     def num_pages(self) -> int:
-        return self._npages
+        """Pages held."""
+        return self._npages - self._first
+
+    @property
+    def first_page_slot(self) -> int:
+        """Page slot of the sequence (position // page size) that the held pages start with."""
+        return self._first
+
+    def state_ref(self) -> int:
+        """``2 * slot + half`` for the step being formed, -1 without recurrent state. The step reads that half
+        of the small per-head vectors and writes the other one, so every call flips it."""
+        if self.state_slot < 0:
+            return -1
+        ref = 2 * self.state_slot + self._state_half
+        self._state_half ^= 1
+        return ref
 
     @property
     def last_page_offset(self) -> int:
@@ -101,6 +149,18 @@ class DistKVCache:
     def allocate_tokens(self, num_tokens: int) -> None:
         if num_tokens <= 0:
             raise ValueError("allocate_tokens needs a positive token count")
+        if self._state_pool is not None and self.state_slot < 0:
+            slot = self._state_pool.alloc()
+            try:
+                self._grow(num_tokens)
+            except KVPoolExhausted:
+                self._state_pool.free(slot)
+                raise
+            self.state_slot, self._state_half = slot, 0
+        else:
+            self._grow(num_tokens)
+
+    def _grow(self, num_tokens: int) -> None:
         need = self.pages_needed(num_tokens)
         if need > 0:
             new = self._pool.alloc_pages(need)
@@ -112,10 +172,25 @@ class DistKVCache:
             self._npages += need
         self._seqlen += num_tokens
 
+    def trim(self, first_position: int) -> int:
+        """Give back the pages all of whose positions are below ``first_position`` (no later token reads
+        them). Returns how many."""
+        keep = min(max(0, first_position) // self._pool.page_size, self._npages)
+        n = keep - self._first
+        if n <= 0:
+            return 0
+        self._pool.free_pages(self._pages[self._first:keep])
+        self._first = keep
+        return n
+
     def release(self) -> None:
-        self._pool.free_pages(self._pages[:self._npages])
+        self._pool.free_pages(self._pages[self._first:self._npages])
         self._npages = 0
+        self._first = 0
         self._seqlen = 0
+        if self.state_slot >= 0:
+            self._state_pool.free(self.state_slot)
+            self.state_slot = -1
 
 
 class BatchedDistKVCache:

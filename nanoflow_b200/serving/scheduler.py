@@ -31,7 +31,7 @@ from typing import List, Optional, Sequence, Tuple
 
 import numpy as np
 
-from .kv_cache import DistKVCache, DistKVPool, KVPoolExhausted
+from .kv_cache import DistKVCache, DistKVPool, KVPoolExhausted, StateSlotPool
 from .request import FlyRequestInfo, NewRequestInfo, NewRequestQueue
 
 
@@ -92,10 +92,70 @@ class BatchPlan:
     # ``num_tail_decode`` decode requests whose tokens are the last of the batch (they fall into the last
     # nano-batch). ``decode`` lists head then tail.
     num_tail_decode: int = 0
+    # Per request: page slot its page list starts with (pages before it have left every window), and its
+    # recurrent-state reference (see DistKVCache.state_ref; -1 without state).
+    kv_first: Optional[np.ndarray] = None
+    state_ref: Optional[np.ndarray] = None
 
     @property
     def num_requests(self) -> int:
         return len(self.decode) + len(self.prefill)
+
+
+def request_arrays(kvs: Sequence[DistKVCache]) -> dict:
+    """Page tables and state references of a batch's requests, in batch order."""
+    B = len(kvs)
+    counts = np.fromiter((kv.num_pages for kv in kvs), dtype=np.int32, count=B)
+    kv_indptr = np.zeros(B + 1, dtype=np.int32)
+    np.cumsum(counts, out=kv_indptr[1:])
+    return dict(
+        kv_indptr=kv_indptr,
+        kv_indices=np.concatenate([kv.indicies for kv in kvs]).astype(np.int32, copy=False),
+        kv_last_page_len=np.fromiter((kv.last_page_offset for kv in kvs), dtype=np.int32, count=B),
+        kv_first=np.fromiter((kv.first_page_slot for kv in kvs), dtype=np.int32, count=B),
+        state_ref=np.fromiter((kv.state_ref() for kv in kvs), dtype=np.int32, count=B),
+        max_kv_pages=int(counts.max()) if B else 0)
+
+
+@dataclass
+class Portion:
+    """Given tokens of one request for one step (trace replay): they continue the sequence held in ``kv``, which
+    already has room for them, and the rows listed in ``want`` are sampled."""
+    kv: DistKVCache
+    tokens: np.ndarray
+    want: Sequence[int] = ()
+
+
+def plan_portions(portions: Sequence[Portion], iteration: int = 0, tile_tokens: int = 128) -> BatchPlan:
+    """One step over given tokens, laid out as :meth:`Scheduler.schedule` lays out a batch (single decoded
+    tokens first, then longer portions) in one nano-batch. ``sample_rows`` follows the order of
+    ``portions`` and of their ``want`` lists, whatever order the tokens take. ``tile_tokens``: query tokens
+    per prefill work item (128 / query heads per KV head)."""
+    order = sorted(range(len(portions)), key=lambda i: len(portions[i].tokens) > 1)     # stable
+    D = sum(len(p.tokens) == 1 for p in portions)
+    row0, t = {}, 0
+    qo_indptr = np.zeros(len(order) + 1, dtype=np.int32)
+    positions, ids, token_req = [], [], []
+    for b, i in enumerate(order):
+        p = portions[i]
+        n = len(p.tokens)
+        row0[i] = t
+        t += n
+        qo_indptr[b + 1] = t
+        positions.append(np.arange(p.kv.seqlen - n, p.kv.seqlen, dtype=np.int32))
+        ids.append(np.asarray(p.tokens, dtype=np.int32))
+        token_req.append(np.full(n, b, dtype=np.int32))
+    arrays = request_arrays([portions[i].kv for i in order])
+    rows = [row0[i] + int(w) for i, p in enumerate(portions) for w in p.want]
+    items = [(b, q, min(tile_tokens, int(qo_indptr[b + 1]) - q)) for b in range(D, len(order))
+             for q in range(int(qo_indptr[b]), int(qo_indptr[b + 1]), tile_tokens)]
+    return BatchPlan(iteration=iteration, decode=[None] * D, prefill=[(None, int(positions[b][0]), len(ids[b]))
+                                                                      for b in range(D, len(order))],
+                     num_tokens=t, num_decode=D, host_ids=np.concatenate(ids),
+                     feedback_src=np.full(t, -1, dtype=np.int32), positions=np.concatenate(positions),
+                     token_req=np.concatenate(token_req), qo_indptr=qo_indptr,
+                     sample_rows=np.asarray(rows, dtype=np.int32), sample_reqs=[],
+                     nano=[NanoBatchPlan(0, t, 0, D, np.asarray(items, dtype=np.int32).reshape(-1, 3))], **arrays)
 
 
 class Scheduler:
@@ -104,8 +164,14 @@ class Scheduler:
                  max_batch_size: Optional[int] = None, average_prefill_length: int = 1024,
                  average_decode_length: int = 512, group_size: int = 8, eos_token_id: Optional[int] = None,
                  stop_on_eos: bool = False, hold_retired_pages: bool = False, prefill_ctas: int = 296,
-                 decode_tail_fraction: float = 0.0):
+                 decode_tail_fraction: float = 0.0, state_pool: Optional[StateSlotPool] = None,
+                 kv_window: int = 0):
+        """``state_pool``: slots of recurrent state, one per request in flight (models that carry one).
+        ``kv_window``: > 0 if no token of the model sees further back than this many positions; pages that
+        have left the window are then given back while the request runs."""
         self._memory_pool = memory_pool
+        self._state_pool = state_pool
+        self.kv_window = int(kv_window)
         self._request_queue = request_queue
         self.global_batch_size = int(global_batch_size)
         self.nanobatch_sizes = list(nanobatch_sizes) if nanobatch_sizes else [self.global_batch_size]
@@ -322,7 +388,8 @@ class Scheduler:
             curve = curve + one
             new = self._request_queue.get()
             req = FlyRequestInfo(req_idx=new.req_idx, prompt=np.asarray(new.prompt, dtype=np.int32),
-                                 output_len=new.output_len, kv_cache=DistKVCache(self._memory_pool),
+                                 output_len=new.output_len,
+                                 kv_cache=DistKVCache(self._memory_pool, self._state_pool),
                                  request_comein_time=new.start_time)
             n = min(req.input_len, idle)
             try:
@@ -385,11 +452,12 @@ class Scheduler:
         sample_rows.extend(range(t, t + Dt))
         sample_reqs.extend(tail)
         kvs = [r.kv_cache for r in head] + [r.kv_cache for r, _, _ in prefill] + [r.kv_cache for r in tail]
-        counts = np.fromiter((kv.num_pages for kv in kvs), dtype=np.int32, count=B)
-        kv_indptr = np.zeros(B + 1, dtype=np.int32)
-        np.cumsum(counts, out=kv_indptr[1:])
-        kv_indices = np.concatenate([kv.indicies for kv in kvs]).astype(np.int32, copy=False)
-        kv_last = np.fromiter((kv.last_page_offset for kv in kvs), dtype=np.int32, count=B)
+        if self.kv_window > 0:
+            # The step's first token of a request sees kv_window - 1 positions back. Pages before that may
+            # still be read by the iteration in flight; whoever gets them writes them in a later one.
+            for kv, n in zip(kvs, np.diff(qo_indptr)):
+                kv.trim(kv.seqlen - int(n) - self.kv_window + 1)
+        arrays = request_arrays(kvs)
 
         # 5. state transitions for the launched work
         for slot, req in enumerate(sample_reqs):
@@ -406,10 +474,9 @@ class Scheduler:
 
         plan = BatchPlan(iteration=self.iteration, decode=decode, prefill=prefill, num_tokens=T, num_decode=D,
                          host_ids=host_ids, feedback_src=feedback, positions=positions, token_req=token_req,
-                         qo_indptr=qo_indptr, kv_indptr=kv_indptr, kv_indices=kv_indices,
-                         kv_last_page_len=kv_last, sample_rows=np.asarray(sample_rows, dtype=np.int32),
-                         sample_reqs=sample_reqs, nano=nano, max_kv_pages=int(counts.max()) if B else 0,
-                         retired_reqs=retired_now, num_tail_decode=Dt)
+                         qo_indptr=qo_indptr, sample_rows=np.asarray(sample_rows, dtype=np.int32),
+                         sample_reqs=sample_reqs, nano=nano,
+                         retired_reqs=retired_now, num_tail_decode=Dt, **arrays)
         if self.hold_retired_pages and retired_now:
             plan.retired_pages = np.concatenate([r.kv_cache.indicies for r in retired_now]).astype(np.int32)
         self._finish_retire_log(retired_now, plan)
