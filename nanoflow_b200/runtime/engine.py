@@ -98,7 +98,7 @@ class Engine:
             from ..utils.guards import GuardedArena
             self.guards = GuardedArena(self.device)
         self.gemm_tuning: Dict[str, dict] = {}
-        self.offload_cap, self.offload_host = 0, None
+        self.offload_cap, self.offload_host, self.page_bytes_layer = 0, None, 0
         self._setup(num_pages)
         S = self.layout.sample_cap
         self.tokens_host = [torch.zeros(S, dtype=torch.int32).pin_memory() for _ in range(RING)]
