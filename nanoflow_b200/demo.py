@@ -21,7 +21,8 @@ import os
 import sys
 from typing import List
 
-MODELS = ["llama2-70B", "llama3-70B", "llama3.1-70B", "llama3-8B", "llama3.1-8B", "qwen2-72B", "tiny"]
+MODELS = ["llama2-70B", "llama3-70B", "llama3.1-70B", "llama3-8B", "llama3.1-8B", "qwen2-72B", "tiny",
+          "volarax-tiny", "volarax-2B", "volarax-8B"]
 
 
 def _serve(a) -> int:
@@ -35,6 +36,8 @@ def _serve(a) -> int:
         raise SystemExit(f"unknown model {a.model}; choose from {', '.join(m for m in MODELS if m in MODEL_ARCHS)}")
     if a.model == "tiny":
         cfg = make_config("tiny", gpu_num=a.gpus, global_batch_size=48)
+    elif "layers" in MODEL_ARCHS[a.model]:
+        cfg = make_config(a.model, gpu_num=a.gpus, global_batch_size=48 if a.model.endswith("tiny") else 1024)
     else:
         variants = shipped_variants(a.model)
         cfg = variants["1024" if "1024" in variants and MODEL_ARCHS[a.model]["hidden_size"] <= 4096 else "2048"]

@@ -129,3 +129,79 @@ def paged_attention(q, kv_pool, qo_indptr, kv_indptr, kv_indices, kv_last_page_l
 
 def argmax(logits, col_offset=0):
     return logits.float().argmax(dim=-1).int() + col_offset
+
+
+# ---- layer-list models ---------------------------------------------------------------------------------
+def layernorm(x, w, b, eps):
+    return torch.nn.functional.layer_norm(x.float(), (x.shape[-1],), w.float(), b.float(), eps)
+
+
+def gated_mlp(h, w_gate, w_up, w_down, act: str):
+    f = {"silu": torch.nn.functional.silu, "relu": torch.relu,
+         "gelu_tanh": lambda z: torch.nn.functional.gelu(z, approximate="tanh")}[act]
+    return (f(h.float() @ w_gate.float().t()) * (h.float() @ w_up.float().t())) @ w_down.float().t()
+
+
+def _pool_rows(positions, req, kv_indptr, kv_indices, kv_first, page_size):
+    """Row numbers of ``positions`` of one request in a pool flattened to [pages * page_size, ...]."""
+    slot = positions // page_size - int(kv_first[req])
+    assert (slot >= 0).all() and (slot < int(kv_indptr[req + 1] - kv_indptr[req])).all(), "position without a page"
+    pages = torch.as_tensor(kv_indices).long()[int(kv_indptr[req]) + slot]
+    return pages * page_size + positions % page_size
+
+
+def latent_append(src, w, pool, positions, token_req, kv_indptr, kv_indices, kv_first, eps):
+    """Latents [T, rank] -> RMS norm -> page slots of pool [pages, page_size, ld] (in place)."""
+    c = rmsnorm(src, w, eps)
+    flat = pool.view(-1, pool.shape[-1])
+    for t in range(src.shape[0]):
+        row = _pool_rows(torch.as_tensor([int(positions[t])]), int(token_req[t]), kv_indptr, kv_indices, kv_first, pool.shape[1])
+        flat[row, :src.shape[1]] = c[t].to(pool.dtype)
+
+
+def latent_attention(q, pool, positions, token_req, kv_indptr, kv_indices, kv_first, *, scale, window=0, sinks=None):
+    """q [T, H, ld] in latent space -> [T, H, ld]: the pool's rows are keys and values."""
+    T, H, ld = q.shape
+    out = torch.zeros(T, H, ld)
+    flat = pool.view(-1, pool.shape[-1]).float()
+    for t in range(T):
+        pos = int(positions[t])
+        keys = torch.arange(max(0, pos - window + 1) if window else 0, pos + 1)
+        c = flat[_pool_rows(keys, int(token_req[t]), kv_indptr, kv_indices, kv_first, pool.shape[1])]
+        s = q[t].float() @ c.t() * scale
+        if sinks is not None:
+            s = torch.cat([s, sinks.float()[:, None]], dim=1)
+        p = torch.softmax(s, dim=-1)
+        out[t] = p[:, :keys.numel()] @ c
+    return out
+
+
+def mlstm(q, k, v, i_pre, f_pre, cap, state, positions, qo_indptr, state_ref):
+    """q (scaled), k [T, H, d], v [T, H, vd], gate pre-activations [T, H]; ``state`` = (S, n, m) of all slots, updated in
+    place: requests at position 0 start from zero, half ``ref & 1`` of n and m is read, the other written."""
+    S_all, n_all, m_all = state
+    li = cap * torch.tanh(i_pre.float() / cap)
+    lf = torch.nn.functional.logsigmoid(cap * torch.tanh(f_pre.float() / cap))
+    out = torch.zeros(v.shape)
+    for b in range(len(qo_indptr) - 1):
+        t0, t1 = int(qo_indptr[b]), int(qo_indptr[b + 1])
+        slot, half = int(state_ref[b]) >> 1, int(state_ref[b]) & 1
+        S, n, m = S_all[slot].clone(), n_all[slot, :, half].clone(), m_all[slot, :, half].clone()
+        if int(positions[t0]) == 0:
+            S, n, m = torch.zeros_like(S), torch.zeros_like(n), torch.zeros_like(m)
+        for t in range(t0, t1):
+            mn = torch.maximum(lf[t] + m, li[t])
+            keep, write = torch.exp(lf[t] + m - mn), torch.exp(li[t] - mn)
+            S = keep[:, None, None] * S + write[:, None, None] * k[t].float()[:, :, None] * v[t].float()[:, None, :]
+            n = keep[:, None] * n + write[:, None] * k[t].float()
+            m = mn
+            den = torch.maximum((n * q[t].float()).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            out[t] = torch.einsum("hdv,hd->hv", S, q[t].float()) / den[:, None]
+        S_all[slot], n_all[slot, :, half ^ 1], m_all[slot, :, half ^ 1] = S, n, m
+    return out
+
+
+def head_norm_gate(o, g, w, vdim, eps):
+    """o, g [T, H, vd_padded], w [H, vd_padded]: RMS norm over each head's ``vdim`` values, weight, sigmoid gate."""
+    inv = torch.rsqrt(o.float().pow(2).sum(-1, keepdim=True) / vdim + eps)
+    return o.float() * inv * w.float() * torch.sigmoid(g.float())

@@ -28,7 +28,8 @@ def build_parser() -> argparse.ArgumentParser:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("-t", "--trace_path", type=str, required=True, help="request trace CSV")
     ap.add_argument("-r", "--run_cycles", type=int, default=20)
-    ap.add_argument("-c", "--config_path", type=str, required=True, help="four-section config JSON")
+    ap.add_argument("-c", "--config_path", type=str, required=True,
+                    help="four-section config JSON, or a model folder (config.json + safetensors)")
     ap.add_argument("-s", "--skip_cycles", type=int, default=0)
     ap.add_argument("--est_cycle_time", type=float, default=0.175)
     ap.add_argument("-o", "--output_prefix", type=str, default="")
@@ -51,10 +52,11 @@ def main(argv=None) -> int:
     args = build_parser().parse_args(argv)
     import torch
 
-    from .config import load_config
-    from .models import random_full_weights, random_rank_weights, shard_weights
+    from .config import load_config, parse_config
+    from .models import random_full_weights, shard_weights
+    from .models.registry import family_of, is_model_folder
     from .models.weights import ensure_converted, load_rank_weights, load_weights
-    from .serving import DistKVPool, RequestManager, Scheduler
+    from .serving import DistKVPool, RequestManager, Scheduler, StateSlotPool
     from .serving.loop import ServingLoop
     from .serving.stats import summarize, write_outputs
 
@@ -62,6 +64,10 @@ def main(argv=None) -> int:
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local = int(os.environ.get("LOCAL_RANK", "0"))
     cfg = load_config(args.config_path, tp=world if world > 1 else None)
+    fam = family_of(cfg.raw["model"])
+    if fam.listed_layers and args.backend == "cpu" and cfg.raw["model"].get("dtype") != "float32":
+        cfg.raw["model"]["dtype"] = "float32"          # the CPU backend computes in fp32
+        cfg = parse_config(cfg.raw)
     model, eng_cfg = cfg.model, cfg.engine
     if world > 1 and world != model.tp:
         raise SystemExit(f"config is for tp={model.tp} but WORLD_SIZE={world}")
@@ -82,8 +88,6 @@ def main(argv=None) -> int:
 
     coll = None
     if args.backend == "gpu":
-        from .runtime.engine import Engine
-
         torch.cuda.set_device(local)
         dev = torch.device("cuda", local)
         if world > 1:
@@ -92,33 +96,40 @@ def main(argv=None) -> int:
 
             dist.init_process_group("nccl", device_id=dev)
             coll = TpCollectives(rank, world, dev)
-        have_files = False
-        if not args.empty_weight and eng_cfg.weight_path:
+        have_files, folder = False, ""
+        if fam.listed_layers:
+            # these models are read from their checkpoint folder as it is
+            folder = next((p for p in (eng_cfg.hf_path, eng_cfg.weight_path) if is_model_folder(p)), "")
+        elif not args.empty_weight and eng_cfg.weight_path:
             # converted per-rank files; written first from the Hugging Face snapshot if they are missing
             if rank == 0:
                 have_files = ensure_converted(eng_cfg.weight_path, eng_cfg.hf_path, max(1, world))
             if world > 1:
                 torch.distributed.barrier()
             have_files = ensure_converted(eng_cfg.weight_path, "", max(1, world))
-        if not have_files:
-            weights = random_rank_weights(model, rank, max(1, world), dev, o1=bool(eng_cfg.o_allgather_nanos))
+        if folder and not args.empty_weight:
+            weights = fam.load_folder(cfg, folder, dev)
+        elif not have_files:
+            weights = fam.random_weights(cfg, rank, max(1, world), dev)
         else:
             weights = load_rank_weights(eng_cfg.weight_path, model, rank, max(1, world), device=dev,
                                         o1=bool(eng_cfg.o_allgather_nanos))
-        engine = Engine(cfg, weights, device=dev, collectives=coll, num_pages=args.allocate_page_num or None)
+        engine = fam.engine(cfg, weights, device=dev, collectives=coll, num_pages=args.allocate_page_num or None)
         num_pages = engine.num_pages
     else:
-        from .runtime.cpu_backend import CpuEngine
-
         tp = model.tp
         num_pages = args.allocate_page_num or 4096
-        if not args.empty_weight and eng_cfg.weight_path and ensure_converted(eng_cfg.weight_path, eng_cfg.hf_path, tp,
+        if fam.listed_layers:
+            folder = next((p for p in (eng_cfg.hf_path, eng_cfg.weight_path) if is_model_folder(p)), "")
+            shards = [fam.load_folder(cfg, folder, "cpu") if folder and not args.empty_weight
+                      else fam.random_weights(cfg, 0, 1, "cpu")]
+        elif not args.empty_weight and eng_cfg.weight_path and ensure_converted(eng_cfg.weight_path, eng_cfg.hf_path, tp,
                                                                                 dtype=torch.float32):
             shards = load_weights(tp, eng_cfg.weight_path, model, dtype=torch.float32)
         else:
             fw = random_full_weights(model, seed=0)
             shards = [shard_weights(fw, model, r, tp, dtype=torch.float32) for r in range(tp)]
-        engine = CpuEngine(cfg, shards, num_pages=num_pages)
+        engine = fam.cpu_engine(cfg, shards, num_pages=num_pages)
 
     pool = DistKVPool(model.run_layers, model.num_kv_heads, model.head_dim, num_pages, eng_cfg.page_size, model.tp)
     sch = Scheduler(pool, rm.avaliable_request_queue, global_batch_size=eng_cfg.global_batch_size,
@@ -126,7 +137,9 @@ def main(argv=None) -> int:
                     average_prefill_length=rm.average_prefill_length, average_decode_length=rm.average_decode_length,
                     group_size=model.group_size, eos_token_id=model.eos_token_id, stop_on_eos=args.stop_on_eos,
                     hold_retired_pages=bool(eng_cfg.offload and args.backend == "gpu"),
-                    decode_tail_fraction=eng_cfg.decode_tail_fraction)
+                    decode_tail_fraction=eng_cfg.decode_tail_fraction,
+                    state_pool=StateSlotPool(engine.num_slots) if getattr(engine, "num_slots", 0) else None,
+                    kv_window=getattr(model, "kv_window", 0))
     sch.keep_schedule_log = bool(args.output_prefix)
     offload = None
     if eng_cfg.offload and args.backend == "gpu":
