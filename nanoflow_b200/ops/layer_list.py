@@ -1,0 +1,149 @@
+"""Python entry points for the layer-list kernels (residual step, latent attention, mLSTM, general GEMM forms).
+
+Like the functions of :mod:`nanoflow_b200.ops` they take torch CUDA tensors, check what the C ABI cannot and
+launch on the current stream; engines do not call them but put the same parameter blocks into their op graph.
+"""
+from __future__ import annotations
+
+from ctypes import byref
+from typing import Optional
+
+import torch
+
+from . import (ACTS, NORMS, AttnParams, GemmParams, HeadNormGateParams, LatentAppendParams, LatentAttnParams, MlstmParams,
+               ResidualNormParams, _check, _i32, _p, _stream, dtype_code, lib)
+
+
+def _f32(t: Optional[torch.Tensor], name: str) -> None:
+    if t is not None and (t.dtype != torch.float32 or not t.is_cuda or t.stride(-1) != 1):
+        raise RuntimeError(f"{name} must be a CUDA float32 tensor with unit inner stride")
+
+
+def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None, up: Optional[torch.Tensor] = None,
+         act: str = "silu", out32: Optional[torch.Tensor] = None, f32_col0: int = 0, groups: int = 1, group_k: int = 0,
+         k: int = 0, workspace: Optional[torch.Tensor] = None, status=None, **shape) -> Optional[torch.Tensor]:
+    """a @ w^T in the storage type of the operands (bf16: tensor cores, fp32: FMA). ``up``: act(a @ w^T) * (a @ up^T).
+    ``out32``: columns from ``f32_col0`` on are written there as fp32. ``groups``: block-diagonal product."""
+    M, N, p = a.shape[0], w.shape[0], GemmParams()
+    if a.dtype != w.dtype or a.stride(1) != 1 or w.stride(1) != 1:
+        raise RuntimeError("gemm: operands of one type with unit inner stride expected")
+    _f32(out32, "out32")
+    if out is None and not (out32 is not None and f32_col0 == 0):
+        out = torch.zeros(M, f32_col0 if out32 is not None else N, dtype=a.dtype, device=a.device)
+    p.A, p.B, p.B2, p.D = _p(a), _p(w), _p(up), _p(out)
+    p.lda, p.ldb, p.ldd = a.stride(0), w.stride(0), out.stride(0) if out is not None else N
+    p.M, p.N, p.K = M, N, k or w.shape[1]
+    p.epilogue, p.act, p.groups, p.group_k = (1 if up is not None else 0), ACTS[act], groups, group_k
+    if out32 is not None:
+        p.D32, p.ld32, p.f32_col0 = _p(out32), out32.stride(0), f32_col0
+    if workspace is not None:
+        p.workspace, p.workspace_bytes = _p(workspace), workspace.numel() * workspace.element_size()
+    p.status = _p(status)
+    for key, v in shape.items():
+        setattr(p, key, v)
+    name = "nfk_gemm_f32" if a.dtype == torch.float32 else "nfk_gemm_bf16"
+    _check(getattr(lib(), name)(byref(p), _stream()), name)
+    return out
+
+
+def residual_norm(x: torch.Tensor, *, y=None, table=None, ids=None, feedback_src=None, prev_tokens=None, norm_in=None,
+                  add=None, h=None, norm_out=None, rows_idx=None, cols: int, eps: float, rows: Optional[int] = None,
+                  status=None) -> None:
+    """x <- (table ? 0 : x) + norm_in(y or table[ids]) (+ add); h <- norm_out(x). Norms: (kind, weight, bias)."""
+    p = ResidualNormParams()
+    _f32(x, "x")
+    p.x, p.ld_x = _p(x), x.stride(0)
+    typed = next(t for t in (y, table, h) if t is not None)
+    p.dtype = dtype_code(typed.dtype)
+    if y is not None:
+        p.y, p.ld_y = _p(y), y.stride(0)
+    if table is not None:
+        p.table, p.ld_table, p.vocab = _p(table), table.stride(0), table.shape[0]
+        p.host_ids, p.feedback_src, p.prev_tokens = _p(ids), _p(feedback_src), _p(prev_tokens)
+    if norm_in is not None:
+        p.in_kind, p.in_w, p.in_b = NORMS[norm_in[0]], _p(norm_in[1]), _p(norm_in[2])
+    p.add = _p(add)
+    if h is not None:
+        p.h, p.ld_h = _p(h), h.stride(0)
+        if norm_out is not None:
+            p.out_kind, p.out_w, p.out_b = NORMS[norm_out[0]], _p(norm_out[1]), _p(norm_out[2])
+    if rows_idx is not None:
+        _i32(rows_idx, "rows_idx")
+        p.rows_idx, p.in_rows = _p(rows_idx), x.shape[0]
+    p.rows = rows if rows is not None else (rows_idx.numel() if rows_idx is not None else x.shape[0])
+    p.cols, p.eps, p.status = cols, eps, _p(status)
+    _check(lib().nfk_residual_norm(byref(p), _stream()), "nfk_residual_norm")
+
+
+def latent_append(src, w, pool, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, rank: int, eps: float,
+                  status=None) -> None:
+    """RMS-normed latents of src[:, :rank] into their slots of pool [pages, page size, row size]."""
+    _f32(w, "w")
+    p = LatentAppendParams(src=_p(src), ld_src=src.stride(0), w=_p(w), pool=_p(pool), ld=pool.shape[2],
+                           positions=_p(positions), token_req=_p(token_req), kv_indptr=_p(kv_indptr),
+                           kv_indices=_p(kv_indices), kv_first=_p(kv_first), T=src.shape[0], rank=rank,
+                           page_size=pool.shape[1], num_pages=pool.shape[0], eps=eps, dtype=dtype_code(pool.dtype),
+                           status=_p(status))
+    _check(lib().nfk_latent_append(byref(p), _stream()), "nfk_latent_append")
+
+
+def latent_attention(q, pool, out, tokens, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, heads: int,
+                     scale: float, window: int = 0, sinks=None, impl: int = 0, splits: int = 1, workspace=None,
+                     status=None) -> None:
+    """Attention of the listed token rows over latent rows; q and out are [T, heads * row size]."""
+    _i32(tokens, "tokens")
+    _f32(sinks, "sinks")
+    p = LatentAttnParams(q=_p(q), ld_q=q.stride(0), pool=_p(pool), ld=pool.shape[2], out=_p(out), ld_out=out.stride(0),
+                         tokens=_p(tokens), positions=_p(positions), token_req=_p(token_req), kv_indptr=_p(kv_indptr),
+                         kv_indices=_p(kv_indices), kv_first=_p(kv_first), sinks=_p(sinks), n_tokens=tokens.numel(),
+                         heads=heads, page_size=pool.shape[1], num_pages=pool.shape[0], window=window, scale=scale,
+                         dtype=dtype_code(pool.dtype), impl=impl, splits=splits, workspace=_p(workspace),
+                         workspace_floats=0 if workspace is None else workspace.numel(), status=_p(status))
+    _check(lib().nfk_latent_attn(byref(p), _stream()), "nfk_latent_attn")
+
+
+def attn_prefill_rows(q, kv, out, qo_indptr, kv_indptr, page_ids, kv_last_page_len, items, *, heads: int, scale: float,
+                      window: int = 0, sinks=None, k_col: int = 0, v_col: Optional[int] = None, status=None) -> None:
+    """The tcgen05 prefill kernel over expanded rows: q [T, >= heads * 128], kv [rows, ...] with head h's key at column
+    k_col + 128 h and value at v_col + 128 h; page id x of a request stands for rows 16 x ... of kv."""
+    p = AttnParams()
+    p.q, p.out, p.kv_pool = _p(q), _p(out), _p(kv)
+    p.qo_indptr, p.kv_indptr, p.kv_indices = _p(qo_indptr), _p(kv_indptr), _p(page_ids)
+    p.kv_last_page_len, p.items, p.num_items = _p(kv_last_page_len), _p(items), items.shape[0]
+    p.q_heads = p.kv_heads = heads
+    p.head_dim, p.page_size, p.num_pages, p.sm_scale = 128, 16, kv.shape[0] // 16, scale
+    p.window, p.sinks, p.status = window, _p(sinks), _p(status)
+    p.kv_ld, p.k_col, p.v_col = kv.stride(0), k_col, heads * 128 if v_col is None else v_col
+    p.q_rows, p.ld_q = q.shape[0], q.stride(0)
+    _check(lib().nfk_attn_prefill_ws(byref(p), _stream()), "nfk_attn_prefill_ws")
+
+
+def mlstm(qkv, gates, i_bias, f_bias, state, out, positions, qo_indptr, state_ref, *, heads: int, dim: int, vdim: int,
+          gate_cap: float, q_scale: float, req_begin: int = 0, req_count: Optional[int] = None, decode: bool = False,
+          impl: int = 0, items=None, scratch=None, status=None) -> None:
+    """qkv rows are q | k | v of all heads; ``state`` = (S, n, m) of all slots (see kernels.h); out fp32 [T, heads * vdim].
+    ``decode``: every request has one token. ``items`` [n, 4]: segments for the chunked form."""
+    for t, nm in ((gates, "gates"), (i_bias, "i_bias"), (f_bias, "f_bias"), (out, "out")):
+        _f32(t, nm)
+    S, n, m = state
+    p = MlstmParams(qkv=_p(qkv), ld_qkv=qkv.stride(0), q_off=0, k_off=heads * dim, v_off=2 * heads * dim, gates=_p(gates),
+                    ld_gates=gates.stride(0), i_bias=_p(i_bias), f_bias=_p(f_bias), S=_p(S), n=_p(n), m=_p(m), out=_p(out),
+                    ld_out=out.stride(0), positions=_p(positions), qo_indptr=_p(qo_indptr), state_slot=_p(state_ref),
+                    req_begin=req_begin, req_count=qo_indptr.numel() - 1 if req_count is None else req_count, heads=heads,
+                    dim=dim, vdim=vdim, num_slots=S.shape[0], gate_cap=gate_cap, q_scale=q_scale,
+                    dtype=dtype_code(qkv.dtype), impl=impl, items=_p(items), num_items=0 if items is None else items.shape[0],
+                    scratch=_p(scratch), scratch_floats=0 if scratch is None else scratch.numel(), status=_p(status))
+    name = "nfk_mlstm_decode" if decode else "nfk_mlstm_prefill"
+    _check(getattr(lib(), name)(byref(p), _stream()), name)
+
+
+def mlstm_scratch_floats(items: int, heads: int, dim: int, vdim: int) -> int:
+    return items * heads * (dim * vdim + dim + 8)
+
+
+def head_norm_gate(o, g, w, out, *, heads: int, vdim: int, eps: float) -> None:
+    """out = RMS norm of each head's values * w * sigmoid(g); o fp32 [T, heads * padded vdim]."""
+    _f32(o, "o"); _f32(w, "w")
+    p = HeadNormGateParams(o=_p(o), ld_o=o.stride(0), g=_p(g), ld_g=g.stride(0), w=_p(w), out=_p(out), ld_out=out.stride(0),
+                           T=o.shape[0], heads=heads, vdim=vdim, vdim_p=w.numel() // heads, eps=eps, dtype=dtype_code(out.dtype))
+    _check(lib().nfk_head_norm_gate(byref(p), _stream()), "nfk_head_norm_gate")
