@@ -1,0 +1,267 @@
+"""Volarax on the GPU: every kernel against the plain oracle of its mechanism, then the engine against the oracle
+model in 32-bit (tight) and bf16, however prompts are cut and batched, and greedy generation through the serving
+loop. All sizes and weights are the tests' own."""
+import numpy as np
+import pytest
+import torch
+
+pytestmark = pytest.mark.gpu
+
+import volarax_cases as cases
+import volarax_oracle as oracle
+from nanoflow_b200 import ops
+from nanoflow_b200.models import volarax
+from nanoflow_b200.models.registry import family
+from nanoflow_b200.ops import layer_list as K
+from nanoflow_b200.replay import TraceReplay
+from nanoflow_b200.runtime.layer_list import mlstm_segments
+from nanoflow_b200.serving import DistKVPool, RequestManager, Scheduler, StateSlotPool
+from nanoflow_b200.serving.loop import ServingLoop
+
+BOTH = [torch.float32, torch.bfloat16]
+TOL = {torch.float32: 2e-5, torch.bfloat16: 1.2e-2}
+
+
+def i32(v):
+    return torch.as_tensor(np.asarray(v), dtype=torch.int32).cuda()
+
+
+def rnd(*shape, seed=0, dtype=torch.float32, scale=1.0):
+    g = torch.Generator().manual_seed(seed)
+    return (torch.randn(*shape, generator=g) * scale).to(dtype).cuda()
+
+
+def rel(got, want):
+    got, want = got.double().cpu(), want.double().cpu()
+    return float((got - want).abs().max() / want.pow(2).mean().sqrt())
+
+
+# ---- GEMM forms ---------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("M,N,Kd", [(1, 8, 8), (5, 216, 104), (130, 72, 200), (300, 520, 1000)])
+def test_gemm_with_fp32_columns(dtype, M, N, Kd):
+    a, w = rnd(M, Kd, seed=1, dtype=dtype), rnd(N, Kd, seed=2, dtype=dtype, scale=Kd ** -0.5)
+    want = a.double() @ w.double().T
+    split = N // 16 * 8
+    for col0 in {0, split}:
+        out32 = torch.full((M, N - col0 + 4), -7.0, device="cuda")
+        out = K.gemm(a, w, out32=out32, f32_col0=col0)
+        assert rel(out32[:, :N - col0], want[:, col0:]) < 2e-5 and (out32[:, N - col0:] == -7.0).all()
+        if col0:
+            assert rel(out, want[:, :col0]) < TOL[dtype] * 2
+
+
+@pytest.mark.parametrize("split_k,stream_k", [(2, 0), (1, 1)])
+def test_fp32_columns_survive_split_k_and_the_stream_k_tail(split_k, stream_k):
+    a, w = rnd(200, 2048, seed=1, dtype=torch.bfloat16), rnd(1000, 2048, seed=2, dtype=torch.bfloat16, scale=0.02)
+    ws = torch.zeros(1 << 24, device="cuda")
+    out32 = torch.zeros(200, 40, device="cuda")
+    out = K.gemm(a, w, out32=out32, f32_col0=960, workspace=ws, tile_n=128, tile_m=1, split_k=split_k, stream_k=stream_k)
+    want = a.double() @ w.double().T
+    assert rel(out32, want[:, 960:]) < 2e-5 and rel(out, want[:, :960]) < 0.02
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("act", ["silu", "relu", "gelu_tanh"])
+def test_gated_gemm_activations(dtype, act):
+    a = rnd(70, 136, seed=1, dtype=dtype)
+    g, u = (rnd(88, 136, seed=s, dtype=dtype, scale=136 ** -0.5) for s in (2, 3))
+    f = {"silu": torch.nn.functional.silu, "relu": torch.relu,
+         "gelu_tanh": lambda z: torch.nn.functional.gelu(z, approximate="tanh")}[act]
+    want = f(a.double() @ g.double().T) * (a.double() @ u.double().T)
+    assert rel(K.gemm(a, g, up=u, act=act), want) < TOL[dtype] * 4
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("M,groups,gn,gk", [(3, 3, 48, 40), (200, 5, 72, 16), (140, 2, 520, 136), (64, 33, 512, 128)])
+def test_block_diagonal_gemm(dtype, M, groups, gn, gk):
+    """Every group of output columns sees only its own columns of the input (which has more behind them)."""
+    a = rnd(M, groups * gk + 24, seed=1, dtype=dtype)
+    w = rnd(groups * gn, gk, seed=2, dtype=dtype, scale=gk ** -0.5)
+    want = torch.einsum("mgk,gnk->mgn", a[:, :groups * gk].double().reshape(M, groups, gk),
+                        w.double().reshape(groups, gn, gk)).reshape(M, -1)
+    assert rel(K.gemm(a, w, groups=groups, group_k=gk, k=gk), want) < TOL[dtype] * 2
+
+
+# ---- residual step ----------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("cols", [5, 50, 104, 1032, 4096, 9000])
+@pytest.mark.parametrize("kind", ["layer", "rms"])
+def test_residual_step(dtype, cols, kind):
+    ld, rows, eps = (cols + 7) // 8 * 8, 37, 1e-3
+    pad = lambda t: torch.nn.functional.pad(t, (0, ld - cols)).contiguous()
+    x, y = pad(rnd(rows, cols, seed=1) + 3.0), pad(rnd(rows, cols, seed=2, dtype=dtype) + 1.5)
+    vec = [rnd(cols, seed=s) for s in range(3, 8)]
+    w1, b1, w2, b2, add = (pad(v[None])[0] for v in vec)
+    nrm = (lambda t, w, b: oracle.layer_norm(t, w.double(), b.double(), eps)) if kind == "layer" else \
+        (lambda t, w, b: oracle.rms_norm(t, eps, w.double()))
+    if kind == "rms":
+        b1 = b2 = None
+    d = lambda t: t.double()[..., :cols]
+    want_x = d(x) + nrm(d(y), vec[0], vec[1]) + d(add)
+    want_h = nrm(want_x, vec[2], vec[3])
+    h = torch.zeros(rows, ld, dtype=dtype, device="cuda")
+    # gathered rows: the stream stays as it is
+    idx = i32([36, 0, 5, 5])
+    hs, before = torch.zeros(4, ld, dtype=dtype, device="cuda"), x.clone()
+    K.residual_norm(x, y=y, norm_in=(kind, w1, b1), add=add, h=hs, norm_out=(kind, w2, b2), rows_idx=idx, cols=cols, eps=eps)
+    assert torch.equal(x, before) and rel(hs[:, :cols], want_h[idx.long()]) < TOL[dtype] * 4
+    K.residual_norm(x, y=y, norm_in=(kind, w1, b1), add=add, h=h, norm_out=(kind, w2, b2), cols=cols, eps=eps)
+    assert rel(x[:, :cols], want_x) < 2e-5 and rel(h[:, :cols], want_h) < TOL[dtype] * 4
+    assert (h[:, cols:] == 0).all() and (x[:, cols:] == 0).all()
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+def test_embedding_step_takes_fed_back_tokens(dtype):
+    table, w, b = rnd(67, 56, seed=1, dtype=dtype), rnd(56, seed=2), rnd(56, seed=3)
+    x, h = torch.full((4, 56), 9.0, device="cuda"), torch.zeros(4, 56, dtype=dtype, device="cuda")
+    K.residual_norm(x, table=table, ids=i32([3, 0, 66, 1]), feedback_src=i32([-1, 2, -1, 0]), prev_tokens=i32([5, 6, 7]),
+                    norm_in=("layer", w, b), add=b, h=h, norm_out=("layer", w, b), cols=56, eps=1e-5)
+    want = oracle.layer_norm(table.double()[[3, 7, 66, 5]], w.double(), b.double(), 1e-5) + b.double()
+    assert rel(x, want) < 2e-5 and rel(h, oracle.layer_norm(want, w.double(), b.double(), 1e-5)) < TOL[dtype] * 4
+
+
+# ---- latent attention ---------------------------------------------------------------------------------------------
+class Paged:
+    """Sequences in a paged latent pool, pages handed out in a shuffled order, leading pages possibly given back."""
+
+    def __init__(self, lens, ld, dtype, seed=0, first=None):
+        rng = np.random.default_rng(seed)
+        self.lens, self.ld = lens, ld
+        pages = [(n + 15) // 16 for n in lens]
+        ids = rng.permutation(sum(pages) + 5)
+        self.pool = torch.full((sum(pages) + 5, 16, ld), 0.0, dtype=dtype, device="cuda")
+        self.first = first or [0] * len(lens)
+        rows = [ids[sum(pages[:b]):sum(pages[:b + 1])] for b in range(len(lens))]
+        self.page_rows = rows
+        kept = [r[f:] for r, f in zip(rows, self.first)]
+        self.indptr = i32(np.concatenate([[0], np.cumsum([len(r) for r in kept])]))
+        self.indices, self.kv_first = i32(np.concatenate(kept)), i32(self.first)
+
+    def fill(self, b, rows):
+        ids = torch.as_tensor(self.page_rows[b].astype(np.int64)).cuda()
+        pos = torch.arange(rows.shape[0], device="cuda")
+        self.pool[ids[pos // 16], pos % 16] = rows.to(self.pool.dtype)
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("rank", [13, 64, 200])
+def test_latents_are_normed_into_their_page_slots(dtype, rank):
+    ld = (rank + 7) // 8 * 8
+    pg = Paged([40, 20], ld, dtype, first=[1, 0])
+    src = rnd(7, rank + 3, seed=1, dtype=dtype)
+    w = rnd(rank, seed=2)
+    pos, req = [16, 17, 31, 32, 39, 0, 19], [0, 0, 0, 0, 0, 1, 1]
+    st = ops.new_status()
+    K.latent_append(src, w, pg.pool, i32(pos), i32(req), pg.indptr, pg.indices, pg.kv_first, rank=rank, eps=1e-3, status=st)
+    ops.check_status(st)
+    want = oracle.rms_norm(src.double()[:, :rank], 1e-3, w.double())
+    got = torch.stack([pg.pool[pg.page_rows[r][p // 16], p % 16] for p, r in zip(pos, req)])
+    assert rel(got[:, :rank], want) < TOL[dtype] * 2 and (got[:, rank:] == 0).all()
+    assert pg.pool.count_nonzero() <= 7 * rank
+
+
+def latent_case(dtype, impl, heads, ld, window, scale, positions, lens, splits=1, sink_value=None, standout=(), first=None,
+                seed=0):
+    """Run the kernel over tokens at ``positions`` [(request, position)]; returns (got, want). ``standout``: (token, key
+    position) pairs whose key is made to match that token's first head far better than any other."""
+    pg = Paged(lens, ld, dtype, seed, first)
+    lat = [rnd(n, ld, seed=seed + 10 + b).to(dtype).float() for b, n in enumerate(lens)]
+    q = rnd(len(positions), heads, ld, seed=seed + 5, scale=0.3).to(dtype)
+    for t, key in standout:
+        b = positions[t][0]
+        q[t, 0] = (lat[b][key] * 2.0).to(dtype)
+    for b, rows in enumerate(lat):
+        pg.fill(b, rows)
+    sinks = None if sink_value is None else (rnd(heads, seed=3) + sink_value)
+    out = torch.zeros(len(positions), heads * ld, dtype=dtype, device="cuda")
+    order = np.random.default_rng(seed).permutation(len(positions))       # listed in any order
+    ws = torch.zeros(len(positions) * max(splits, 1) * heads * (ld + 2), device="cuda")
+    st = ops.new_status()
+    K.latent_attention(q.reshape(len(positions), -1), pg.pool, out, i32(order), i32([p for _, p in positions]),
+                       i32([b for b, _ in positions]), pg.indptr, pg.indices, pg.kv_first, heads=heads, scale=scale,
+                       window=window, sinks=sinks, impl=impl, splits=splits, workspace=ws, status=st)
+    ops.check_status(st)
+    want = torch.zeros(len(positions), heads, ld, dtype=torch.float64)
+    for t, (b, p) in enumerate(positions):
+        c = lat[b][:p + 1].double().cpu()[:, None, :].expand(-1, heads, -1)
+        qq = torch.zeros(p + 1, heads, ld, dtype=torch.float64)
+        qq[p] = q[t].double().cpu()
+        lo = max(0, p - window + 1) if window else 0
+        sk = torch.full((heads,), -1e30, dtype=torch.float64) if sinks is None else sinks.double().cpu()
+        want[t] = oracle.windowed_sink_attention(qq[lo:], c[lo:], c[lo:], scale, window or None, sk)[-1]
+    return out.reshape(want.shape).double().cpu(), want
+
+
+VARIANTS = [(torch.float32, 1, 40), (torch.bfloat16, 1, 72), (torch.bfloat16, 2, 64), (torch.bfloat16, 2, 192),
+            (torch.bfloat16, 2, 512)]
+
+
+@pytest.mark.parametrize("dtype,impl,ld", VARIANTS)
+@pytest.mark.parametrize("heads", [1, 5, 16, 33])
+def test_latent_attention_random(dtype, impl, ld, heads):
+    lens = [1, 16, 17, 150]
+    pos = [(0, 0), (1, 15), (2, 16), (3, 149), (3, 100), (3, 64), (3, 63)]
+    for window, sink in ((0, None), (37, 0.0), (64, 2.0), (1, 1.0)):
+        got, want = latent_case(dtype, impl, heads, ld, window, ld ** -0.5, pos, lens, sink_value=sink)
+        assert rel(got, want) < TOL[dtype] * 3, (window, sink)
+
+
+@pytest.mark.parametrize("dtype,impl,ld", VARIANTS)
+@pytest.mark.parametrize("window", [1, 16, 17, 48, 65, 200])
+def test_latent_attention_window_edges(dtype, impl, ld, window):
+    """The last key inside the window and the first one outside it, each made to stand out for one token: taking
+    one too many or one too few changes the output entirely."""
+    n = 420
+    tests = [(p, p - d) for p in (window + 15, window + 16, 300, 415, n - 1) for d in (window - 1, window) if p - d >= 0]
+    pos = [(0, p) for p, _ in tests]
+    got, want = latent_case(dtype, impl, 3, ld, window, 0.5, pos, [n], sink_value=-2.0, standout=list(enumerate(k for _, k in tests)))
+    assert rel(got, want) < TOL[dtype] * 3
+
+
+@pytest.mark.parametrize("dtype,impl,ld", VARIANTS)
+def test_latent_attention_far_key_among_hundreds(dtype, impl, ld):
+    keys = [0, 1, 15, 16, 63, 64, 300, 511, 512, 640]
+    got, want = latent_case(dtype, impl, 2, ld, 0, 0.5, [(0, 699)] * len(keys), [700], standout=list(enumerate(keys)), sink_value=0.0)
+    assert rel(got, want) < TOL[dtype] * 3
+    # the key that stands out is the output
+    assert float((want[0, 0] - want[1, 0]).abs().max()) > 0.5
+
+
+@pytest.mark.parametrize("dtype,impl,ld", VARIANTS)
+def test_latent_attention_sinks_take_their_share(dtype, impl, ld):
+    """A sink that outweighs every key pulls the output to zero; a very low one changes nothing."""
+    pos, lens = [(0, 70), (0, 3), (1, 0)], [71, 1]
+    none, _ = latent_case(dtype, impl, 4, ld, 20, ld ** -0.5, pos, lens)
+    low, _ = latent_case(dtype, impl, 4, ld, 20, ld ** -0.5, pos, lens, sink_value=-60.0)
+    got, want = latent_case(dtype, impl, 4, ld, 20, ld ** -0.5, pos, lens, sink_value=3.0)
+    high, _ = latent_case(dtype, impl, 4, ld, 20, ld ** -0.5, pos, lens, sink_value=200.0)
+    assert torch.allclose(none, low, atol=1e-6) and float(high.abs().max()) < 1e-6
+    assert rel(got, want) < TOL[dtype] * 3 and rel(none, want) > 0.2
+
+
+@pytest.mark.parametrize("ld,heads", [(64, 4), (256, 20), (512, 33)])
+@pytest.mark.parametrize("splits", [2, 3, 7])
+def test_latent_attention_split_over_key_ranges(ld, heads, splits):
+    lens = [30, 700, 65]
+    pos = [(0, 29), (1, 699), (1, 64), (2, 64), (2, 0)]
+    for window in (0, 100):
+        got, want = latent_case(torch.bfloat16, 2, heads, ld, window, ld ** -0.5, pos, lens, splits=splits, sink_value=0.5)
+        assert rel(got, want) < TOL[torch.bfloat16] * 3
+
+
+@pytest.mark.parametrize("dtype,impl,ld", VARIANTS)
+def test_latent_attention_with_leading_pages_given_back(dtype, impl, ld):
+    pos = [(0, 99), (0, 80), (1, 40)]
+    got, want = latent_case(dtype, impl, 3, ld, 33, ld ** -0.5, pos, [100, 41], first=[3, 0], sink_value=0.0)
+    assert rel(got, want) < TOL[dtype] * 3
+
+
+def test_latent_attention_rejects_what_it_is_not_built_for():
+    t = torch.zeros(1, 4096, device="cuda")
+    one = i32([0])
+    with pytest.raises(RuntimeError, match="bad argument"):
+        K.latent_attention(t, torch.zeros(1, 16, 4096, device="cuda"), t, one, one, one, i32([0, 1]), one, heads=1, scale=1.0)
+    with pytest.raises(RuntimeError, match="unsupported"):
+        K.latent_attention(t[:, :40], torch.zeros(1, 16, 40, device="cuda"), t, one, one, one, i32([0, 1]), one, heads=1,
+                           scale=1.0, impl=2)
