@@ -265,3 +265,192 @@ def test_latent_attention_rejects_what_it_is_not_built_for():
     with pytest.raises(RuntimeError, match="unsupported"):
         K.latent_attention(t[:, :40], torch.zeros(1, 16, 40, device="cuda"), t, one, one, one, i32([0, 1]), one, heads=1,
                            scale=1.0, impl=2)
+
+
+def prefill_case(spans, heads, window, sink, scale=0.2, standout=(), seed=0):
+    """Expanded keys and values of requests [(context, tokens)] through the tcgen05 kernel. Returns (got, want)."""
+    kv_len = [c + n for c, n in spans]
+    pages = [(n + 15) // 16 for n in kv_len]
+    base = np.concatenate([[0], np.cumsum(pages)])
+    T = sum(n for _, n in spans)
+    ld_q = heads * 128 + 72
+    q = rnd(T, ld_q, seed=seed + 1, dtype=torch.bfloat16)
+    kv = rnd(int(base[-1]) * 16, heads * 256, seed=seed + 2, dtype=torch.bfloat16)
+    qo = np.concatenate([[0], np.cumsum([n for _, n in spans])])
+    for tok, key in standout:                       # token's first head matches that key of its request
+        b = int(np.searchsorted(qo, tok, side="right") - 1)
+        q[tok, :128] = kv[int(base[b]) * 16 + key, :128] * 1.5
+    sinks = None if sink is None else rnd(heads, seed=3) + sink
+    items = [(b, t, min(128, int(qo[b + 1]) - t)) for b in range(len(spans)) for t in range(int(qo[b]), int(qo[b + 1]), 128)]
+    out = torch.zeros(T, heads * 128, dtype=torch.bfloat16, device="cuda")
+    st = ops.new_status()
+    K.attn_prefill_rows(q, kv, out, i32(qo), i32(base), torch.arange(int(base[-1]), dtype=torch.int32, device="cuda"),
+                        i32([(n - 1) % 16 + 1 for n in kv_len]), i32(items), heads=heads, scale=scale, window=window, sinks=sinks,
+                        status=st)
+    ops.check_status(st)
+    want = torch.zeros(T, heads, 128, dtype=torch.float64)
+    for b, (c, n) in enumerate(spans):
+        rows = kv[int(base[b]) * 16:int(base[b]) * 16 + kv_len[b]].double().cpu()
+        k, v = rows[:, :heads * 128].reshape(-1, heads, 128), rows[:, heads * 128:].reshape(-1, heads, 128)
+        qq = q[qo[b]:qo[b + 1], :heads * 128].double().cpu().reshape(n, heads, 128)
+        s = torch.einsum("thd,khd->htk", qq, k) * scale
+        i, j = torch.arange(c, c + n)[:, None], torch.arange(c + n)[None, :]
+        seen = (j <= i) & ((i - j < window) if window else True)
+        s = s.masked_fill(~seen[None], float("-inf"))
+        if sinks is not None:
+            s = torch.cat([s, sinks.double().cpu()[:, None, None].expand(-1, n, 1)], dim=2)
+        want[qo[b]:qo[b + 1]] = torch.einsum("htk,khd->thd", torch.softmax(s, -1)[..., :c + n], v)
+    return out.reshape(want.shape).double().cpu(), want
+
+
+@pytest.mark.parametrize("window", [0, 1, 16, 37, 64, 65, 300])
+@pytest.mark.parametrize("heads", [1, 3])
+def test_prefill_attention_over_expanded_rows(window, heads):
+    for spans in ([(0, 1)], [(0, 200)], [(5, 40), (0, 129), (333, 70)], [(63, 64), (64, 65), (500, 17)]):
+        for sink in (None, 1.0):
+            got, want = prefill_case(spans, heads, window, sink)
+            assert rel(got, want) < 0.03, (spans, sink)
+
+
+@pytest.mark.parametrize("window", [1, 16, 50, 64, 129, 400])
+def test_prefill_attention_window_edges_and_far_keys(window):
+    spans = [(520, 300)]
+    marks = [(t, 520 + t - d) for t in (0, 1, 63, 64, 127, 128, 200, 299) for d in (window - 1, window)]
+    for half in (marks[0::2], marks[1::2]):
+        got, want = prefill_case(spans, 2, window, 0.0, scale=1.0, standout=half)
+        assert rel(got, want) < 0.03
+    got, want = prefill_case(spans, 2, 0, 0.0, scale=1.0, standout=[(299, 0), (298, 1), (297, 15), (0, 16), (130, 511)])
+    assert rel(got, want) < 0.03
+    high, _ = prefill_case(spans, 2, window, 500.0)
+    assert float(high.abs().max()) < 1e-6
+
+
+# ---- mLSTM -----------------------------------------------------------------------------------------------------------
+class MlstmCase:
+    def __init__(self, lens, heads, dim, vdim, dtype, cap=9.0, seed=0, f_bias=4.0):
+        self.lens, self.H, self.d, self.v, self.dtype, self.cap = lens, heads, dim, vdim, dtype, cap
+        self.q, self.k = (rnd(sum(lens), heads, dim, seed=seed + s, dtype=dtype) for s in (1, 2))
+        self.vv = rnd(sum(lens), heads, vdim, seed=seed + 3, dtype=dtype)
+        self.gates = rnd(sum(lens), 2 * heads + 2, seed=seed + 4, scale=2.0)
+        self.i_b, self.f_b = rnd(heads, seed=seed + 5), rnd(heads, seed=seed + 6) + f_bias
+        self.slots = len(lens) + 2
+        z = lambda *s: torch.full(s, 77.0, device="cuda")        # what an earlier owner of the slot left behind
+        self.state = (z(self.slots, heads, dim, vdim), z(self.slots, heads, 2, dim), z(self.slots, heads, 2))
+        self.at = [0] * len(lens)
+        self.half = [0] * len(lens)
+        self.out = [torch.zeros(n, heads * vdim) for n in lens]
+        self.row0 = np.concatenate([[0], np.cumsum(lens)])
+
+    def want(self):
+        outs = []
+        for b, n in enumerate(self.lens):
+            r = slice(int(self.row0[b]), int(self.row0[b + 1]))
+            d = lambda t: t[r].double().cpu()
+            li = oracle.soft_cap(d(self.gates)[:, :self.H] + self.i_b.double().cpu(), self.cap)
+            lf = oracle.log_sigmoid(oracle.soft_cap(d(self.gates)[:, self.H:2 * self.H] + self.f_b.double().cpu(), self.cap))
+            o, s = oracle.mlstm_recurrence(d(self.q) * self.d ** -0.5, d(self.k), d(self.vv), li, lf)
+            outs.append((o.reshape(n, -1), s))
+        return outs
+
+    def step(self, parts, decode=False, impl=0, seg_ctas=4):
+        """Run the next ``n`` tokens of each request in ``parts`` {request: n} as one launch."""
+        reqs = list(parts)
+        rows = np.concatenate([np.arange(self.row0[b] + self.at[b], self.row0[b] + self.at[b] + parts[b]) for b in reqs])
+        idx = torch.as_tensor(rows).cuda()
+        qkv = torch.cat([self.q[idx].flatten(1), self.k[idx].flatten(1), self.vv[idx].flatten(1)], dim=1).contiguous()
+        qo = np.concatenate([[0], np.cumsum([parts[b] for b in reqs])]).astype(np.int32)
+        pos = np.concatenate([np.arange(self.at[b], self.at[b] + parts[b]) for b in reqs])
+        items = mlstm_segments(qo, 0, seg_ctas, 148)
+        scratch = torch.zeros(K.mlstm_scratch_floats(len(items), self.H, self.d, self.v), device="cuda")
+        out = torch.zeros(len(rows), self.H * self.v, device="cuda")
+        st = ops.new_status()
+        K.mlstm(qkv, self.gates[idx].contiguous(), self.i_b, self.f_b, self.state, out, i32(pos), i32(qo),
+                i32([2 * (b + 1) + self.half[b] for b in reqs]), heads=self.H, dim=self.d, vdim=self.v, gate_cap=self.cap,
+                q_scale=self.d ** -0.5, decode=decode, impl=impl, items=i32(items), scratch=scratch, status=st)
+        ops.check_status(st)
+        for j, b in enumerate(reqs):
+            n = parts[b]
+            self.out[b][self.at[b]:self.at[b] + n] = out[int(qo[j]):int(qo[j + 1])].cpu()
+            self.at[b] += n
+            self.half[b] ^= 1
+
+    def check(self, tol):
+        for b, (o, (S, n, m)) in enumerate(self.want()):
+            assert self.at[b] == self.lens[b]
+            # relative to each head's output: a denominator near zero makes a row large and its error with it
+            err, o = (self.out[b].double() - o).reshape(-1, self.v), o.reshape(-1, self.v)
+            assert float((err.norm(dim=1) / o.norm(dim=1)).max()) < tol
+            got_m = self.state[2][b + 1, :, self.half[b]].double().cpu()
+            assert torch.allclose(got_m, m, atol=2e-4)
+            assert rel(self.state[0][b + 1], S) < tol * 4 and rel(self.state[1][b + 1, :, self.half[b]], n) < tol * 4
+
+
+MLSTM = [(torch.float32, 1, 3e-4), (torch.bfloat16, 1, 3e-4), (torch.bfloat16, 2, 1e-3)]
+SIZES = [(2, 32, 64), (3, 8, 8), (1, 136, 72), (2, 256, 200)]
+
+
+@pytest.mark.parametrize("dtype,impl,tol", MLSTM)
+@pytest.mark.parametrize("heads,dim,vdim", SIZES)
+def test_mlstm_prompts(dtype, impl, tol, heads, dim, vdim):
+    c = MlstmCase([1, 63, 64, 65, 200], heads, dim, vdim, dtype)
+    c.step({b: n for b, n in enumerate(c.lens)}, impl=impl)
+    c.check(tol)
+
+
+@pytest.mark.parametrize("dtype,impl,tol", MLSTM)
+def test_mlstm_portions_and_single_tokens(dtype, impl, tol):
+    """Prompts in portions that end inside chunks, decoding in between, requests that sit out steps."""
+    c = MlstmCase([150, 40, 7, 129], 2, 40, 72, dtype, seed=5)
+    c.step({0: 2, 1: 30}, impl=impl)
+    c.step({0: 1, 2: 1}, decode=True)
+    c.step({0: 64, 1: 3, 3: 128}, impl=impl)
+    c.step({2: 1, 1: 1, 3: 1}, decode=True)
+    c.step({0: 70, 2: 2}, impl=impl)
+    for _ in range(3):
+        c.step({0: 1, 1: 1, 2: 1}, decode=True)
+    c.step({0: 10, 1: 3}, impl=impl)
+    c.check(tol)
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+def test_mlstm_token_by_token(dtype):
+    c = MlstmCase([90, 33], 3, 24, 136, dtype, seed=7)
+    for t in range(90):
+        c.step({b: 1 for b in range(2) if t < c.lens[b]}, decode=True)
+    c.check(3e-4)
+
+
+@pytest.mark.parametrize("cap,f_bias", [(1.5, 0.0), (30.0, -20.0), (30.0, 25.0)])
+def test_mlstm_gate_extremes(cap, f_bias):
+    """Quick forgetting, no forgetting and a tight cap: the running maximum and the floor of the denominator."""
+    for dtype, impl, tol in MLSTM:
+        c = MlstmCase([260], 2, 32, 40, dtype, cap=cap, f_bias=f_bias, seed=3)
+        c.step({0: 130}, impl=impl)
+        c.step({0: 130}, impl=impl)
+        c.check(tol * 4)
+
+
+@pytest.mark.parametrize("n,seg_ctas", [(1000, 4), (777, 30), (3000, 8)])
+def test_mlstm_segments_carry_the_state(n, seg_ctas):
+    """A long portion cut into segments (a first token written strongly and asked for at the end), after and before
+    other portions of the request."""
+    c = MlstmCase([n + 40, 70], 2, 64, 64, torch.bfloat16, seed=9, f_bias=9.0)
+    c.gates[3, :2] = 8.0                           # an early token that stays
+    c.q[n + 20] = c.k[3] * 3.0
+    assert len(mlstm_segments(np.asarray([0, n, n + 50], dtype=np.int32), 0, seg_ctas, 148)) > 2
+    c.step({0: 13}, impl=2)
+    c.step({0: n, 1: 50}, impl=2, seg_ctas=seg_ctas)
+    c.step({0: 27, 1: 20}, impl=2)
+    c.check(1e-3)
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("heads,vdim", [(3, 40), (1, 5), (2, 512)])
+def test_head_norm_and_gate(dtype, heads, vdim):
+    vp = (vdim + 7) // 8 * 8
+    pad = lambda t: torch.nn.functional.pad(t, (0, vp - vdim)).flatten(-2).contiguous()
+    o, g, w = rnd(9, heads, vdim, seed=1), rnd(9, heads, vdim, seed=2, dtype=dtype), rnd(heads, vdim, seed=3)
+    out = torch.zeros(9, heads * vp, dtype=dtype, device="cuda")
+    K.head_norm_gate(pad(o), pad(g), pad(w), out, heads=heads, vdim=vdim, eps=1e-2)
+    want = oracle.rms_norm(o.double(), 1e-2) * w.double() * torch.sigmoid(g.double())
+    assert rel(out.reshape(9, heads, vp)[..., :vdim], want) < TOL[dtype] * 2
