@@ -155,6 +155,9 @@ def main():
     ap.add_argument("--skip-cycles", type=int, default=1600)
     ap.add_argument("--executor", default="auto", help="auto | native | graph (native executor, iterations "
                     "captured and launched as CUDA graphs) | python")
+    ap.add_argument("--layer-list", default="", help="instead of the headline workload: prefill and decode throughput of the "
+                    "layer-list model (Volarax) beside the Llama of equal size, comma-separated sizes out of 2B, 8B")
+    ap.add_argument("--layer-list-only", default="", help="with --layer-list: only workloads whose name holds this text")
     ap.add_argument("--timeline", default="", help="after the timed regions, time every op of one iteration "
                     "with CUDA events and write the aggregate + Chrome trace to this file")
     args = ap.parse_args()
@@ -166,6 +169,20 @@ def main():
     if args.impl == "reference":
         if rank == 0:
             print(json.dumps({"impl": "reference", "unavailable": REF_UNAVAILABLE}))
+        return 0
+    if args.layer_list:
+        if world != 1:
+            raise SystemExit("--layer-list runs on one GPU")
+        from nanoflow_b200.eval import layer_bench
+
+        sampler = ClockSampler(local_rank)
+        sampler.start()
+        t0 = time.perf_counter()
+        res = layer_bench.run(args.layer_list.split(","), args.steps, args.warmup, args.layer_list_only)
+        clocks = sampler.stop(t0, time.perf_counter())
+        print(layer_bench.report(res), file=sys.stderr)
+        print(json.dumps({"benchmark": "layer-list", "n_gpus": 1, "steps": args.steps, "dtype": "bf16",
+                          "data": "synthetic (random token ids, random-init weights)", "results": res, "clocks": clocks}))
         return 0
     if world != args.gpus:
         if args.gpus == 1 and world == 1:

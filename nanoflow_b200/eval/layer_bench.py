@@ -1,0 +1,198 @@
+"""Prefill and decode throughput of a layer-list model beside the Llama model of equal size, layer by layer.
+
+    python bench.py --layer-list 8B            (or 2B, or both: 2B,8B)
+
+Both models get the same width, feed-forward, head count and number of layers, random weights, and the same
+batches: whole prompts in one iteration, and single-token decoding over a given context. Engines, kernels
+and step function are those of serving; each workload has an engine of its own batch size, so that both models'
+GEMM shapes are the tuned ones. Time: CUDA events around repeated iterations (CUDA graphs, weights far larger than
+L2), then one iteration with an event pair around every op for the per-kernel table. Each kernel is set against
+its roofline, the larger of FLOPs over the measured GEMM rate and bytes over the measured copy bandwidth.
+"""
+from __future__ import annotations
+
+import json
+from pathlib import Path
+from typing import Any, Dict, List, Tuple
+
+import numpy as np
+import torch
+
+SIZES = {
+    # name: (width, ff, heads, kv heads of the Llama, vocab, latent rank, window, mLSTM heads, dim, vdim)
+    "8B": dict(width=4096, ff=14336, heads=32, kv=8, vocab=128256, rank=512, window=1024, mh=8, md=256, mv=512),
+    "2B": dict(width=2048, ff=8192, heads=16, kv=4, vocab=32000, rank=256, window=512, mh=4, md=256, mv=512),
+}
+WORKLOADS = [("prefill 4 x 1024", [(0, 1024)] * 4), ("prefill 1 x 4096", [(0, 4096)]),
+             ("decode 256 at 1280", [(1280, 1)] * 256), ("decode 32 at 4096", [(4096, 1)] * 32)]
+LAYERS = 4
+
+
+def peaks() -> Tuple[float, float]:
+    """(FLOP/s, bytes/s) measured on this machine's GPUs, or the earlier measurement if the file is missing."""
+    f = Path(__file__).resolve().parents[2] / "MEASURED_PEAKS.json"
+    if f.exists():
+        d = json.loads(f.read_text())
+        return d["bf16_tflops"] * 1e12, d["hbm_gbs"] * 1e9
+    return 1.59e15, 6.65e12
+
+
+def model_dict(kind: str, s: Dict[str, int]) -> Dict[str, Any]:
+    from ..config import _hf
+    from ..models.volarax import builtin
+    if kind == "llama":
+        return _hf(s["width"], s["ff"], LAYERS, s["heads"], s["kv"], s["vocab"], 500000.0)
+    return builtin(s["width"], s["vocab"], "am" * (LAYERS // 2), heads=s["heads"], dim=128, vdim=128, kv_rank=s["rank"],
+                   window=s["window"], m_heads=s["mh"], m_dim=s["md"], m_vdim=s["mv"], ff=s["ff"], m_ff=s["ff"])
+
+
+def make_engine(kind: str, size: Dict[str, int], spans, device, pages: int, **pipeline):
+    from ..config import parse_config
+    from ..models.registry import family_of
+    T, B = sum(n for _, n in spans), len(spans)
+    hf = model_dict(kind, size)
+    cfg = parse_config({"model": hf, "model_configs": {"gpu_num": 1, "max_batch_size": B, "num_pages": pages},
+                        "pipeline_configs": {"global_batch_size": T, **pipeline},
+                        "serve_configs": {"model": kind, "actual_gpu_num": 1, "pipeline_type": "NON_OVERLAP_LOCAL"}})
+    fam = family_of(hf)
+    return fam.engine(cfg, fam.random_weights(cfg, 0, 1, device), device=device, executor="graph")
+
+
+def make_plan(engine, spans, pages: int):
+    from ..serving import DistKVCache, DistKVPool, Portion, StateSlotPool, plan_portions
+    m = engine.model
+    pool = DistKVPool(m.run_layers, m.num_kv_heads, m.head_dim, pages, 16, 1)
+    slots = StateSlotPool(len(spans)) if getattr(m, "has_state", False) else None
+    window = getattr(m, "kv_window", 0)
+    parts = []
+    for ctx, n in spans:
+        kv = DistKVCache(pool, slots)
+        if ctx:
+            kv.allocate_tokens(ctx)
+        if window:
+            kv.trim(ctx - window + 1)
+        kv.allocate_tokens(n)
+        parts.append(Portion(kv, np.random.default_rng(0).integers(0, m.vocab_size, n), [n - 1]))
+    return plan_portions(parts, tile_tokens=max(1, 128 // m.group_size))
+
+
+def op_work(engine, op, spans) -> Tuple[float, float]:
+    """(FLOPs, bytes) an op has to do; (0, 0) for ops that are not set against a roofline."""
+    from ..runtime import graph as G
+    m, p = engine.model, op.params
+    T = sum(n for _, n in spans)
+    es = 2
+    sees = lambda w: sum(sum(min(c + t + 1, w or c + t + 1) for t in range(n)) for c, n in spans)
+    if isinstance(p, G.GemmParams):
+        dyn = dict(op.dyn)["M"]
+        M = engine._last_sym.get(dyn, 0)
+        if M == 0:
+            return 0.0, 0.0
+        gated = 2 if p.epilogue == 1 else 1
+        groups = max(1, p.groups)
+        return 2.0 * M * p.N * p.K * gated, es * (gated * p.N * p.K + M * (p.K * groups + p.N))
+    if isinstance(p, G.AttnParams):
+        pre = "prefill" in op.kernel
+        if (spans[0][1] == 1) == pre:
+            return 0.0, 0.0
+        w = p.window
+        pairs = sees(w)
+        keys = sum(min(c + n, (w + n - 1) if w else c + n) for c, n in spans)
+        return 4.0 * pairs * p.q_heads * p.head_dim, es * (2 * keys * p.kv_heads * p.head_dim + 2 * T * p.q_heads * p.head_dim)
+    if isinstance(p, G.LatentAttnParams):
+        if spans[0][1] != 1:
+            return 0.0, 0.0
+        pairs = sees(p.window)
+        return 4.0 * pairs * p.heads * p.ld, es * (pairs * p.ld + 2 * T * p.heads * p.ld)
+    if isinstance(p, G.MlstmParams):
+        dec = "decode" in op.kernel
+        if (spans[0][1] == 1) != dec:
+            return 0.0, 0.0
+        state = len(spans) * p.heads * (p.dim * p.vdim + 2 * p.dim) * 4
+        io = T * p.heads * ((2 * p.dim + p.vdim) * es + p.vdim * 4)
+        chunk = 0 if dec else 64
+        return T * p.heads * (chunk * (p.dim + p.vdim) + 4.0 * p.dim * p.vdim), (2 if dec else 1) * state + io
+    if isinstance(p, G.ResidualNormParams):
+        rows = T if not p.rows_idx else len(spans)
+        return 0.0, rows * p.cols * (8 + 2 * es)
+    if isinstance(p, G.HeadNormGateParams):
+        return 0.0, T * p.heads * p.vdim * (4 + 2 * es)
+    if isinstance(p, G.LatentAppendParams):
+        return 0.0, T * p.rank * 2 * es
+    if isinstance(p, G.RopeAppendParams):
+        return 0.0, T * (2 * p.q_heads + 4 * p.kv_heads) * p.head_dim * es
+    if isinstance(p, G.KvMoveParams):
+        return 0.0, 2.0 * engine._last_sym.get(dict(op.dyn)["n_pages"], 0) * p.page_bytes
+    if isinstance(p, G.NormParams):
+        return 0.0, 2 * T * p.cols * es
+    return 0.0, 0.0
+
+
+def measure(engine, plan, spans, steps: int, warmup: int) -> Dict[str, Any]:
+    flops_peak, bw_peak = peaks()
+    for _ in range(max(3, warmup)):
+        engine.run(plan)
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    e0.record(engine.stream)
+    for i in range(steps):
+        engine.update(plan)
+        engine.run_async()
+        if i:
+            engine.run_async_wait()
+    engine.run_async_wait()
+    e1.record(engine.stream)
+    torch.cuda.synchronize()
+    ms = e0.elapsed_time(e1) / steps
+    engine.check_status()
+    # one op at a time, best of three iterations
+    best: Dict[int, float] = {}
+    for _ in range(3):
+        engine.update(plan)
+        engine._last_sym = dict(engine._staged["sym"])
+        engine.run_async(timed=True)
+        engine.run_async_wait()
+        for i, (_, _, a, b) in enumerate(engine.timeline()):
+            best[i] = min(best.get(i, 1e9), b - a)
+    table: Dict[str, List[float]] = {}
+    for i, op in enumerate(engine.graph.ops):
+        fl, by = op_work(engine, op, spans)
+        if fl == 0 and by == 0:
+            continue
+        name = op.name.split(".")[-1]
+        if op.name.startswith("R") and name in ("in", "o", "gate_up", "down"):
+            spec = engine.model.layers[engine.model.runs[op.layer].layer].mixer.kind
+            name = f"{spec[:6]}.{name}" if name in ("in", "o") else name
+        r = table.setdefault(name, [0, 0.0, 0.0])
+        r[0] += 1
+        r[1] += best[i]
+        r[2] += max(fl / flops_peak, by / bw_peak) * 1e6
+    T = sum(n for _, n in spans)
+    return {"ms": round(ms, 3), "tokens_per_s": round(T / ms * 1e3),
+            "ops": {k: {"us": round(us / n, 1), "of_roofline": round(roof / us, 3)} for k, (n, us, roof) in table.items()}}
+
+
+def run(sizes: List[str], steps: int, warmup: int, only: str = "") -> Dict[str, Any]:
+    device = torch.device("cuda", torch.cuda.current_device())
+    out: Dict[str, Any] = {}
+    for size in sizes:
+        for label, spans in WORKLOADS:
+            if only and only not in label:
+                continue
+            pages = sum((c + n + 15) // 16 for c, n in spans) + 8
+            for kind in ("llama", "volarax"):
+                engine = make_engine(kind, SIZES[size], spans, device, pages)
+                res = measure(engine, make_plan(engine, spans, pages), spans, steps, warmup)
+                engine.finalize()
+                del engine
+                torch.cuda.empty_cache()
+                out[f"{size} {label} {kind}"] = res
+    return out
+
+
+def report(out: Dict[str, Any]) -> str:
+    lines = [f"{LAYERS} layers, random weights, one GPU; kernel columns: us per launch (fraction of roofline)", ""]
+    for key, r in out.items():
+        ops = ", ".join(f"{k} {v['us']} ({v['of_roofline']})" for k, v in r["ops"].items())
+        lines.append(f"{key}: {r['ms']} ms, {r['tokens_per_s']} tokens/s\n    {ops}")
+    return "\n".join(lines)
