@@ -7,10 +7,12 @@
 //                     Used for decoding, for prompt tokens whose keys are not expanded, and in 32-bit.
 //
 // Two kernels for the attention. The tensor-core one (bf16): a CTA takes one token, 16 or 32 of its heads (the
-// rows of its MMA tiles) and a range of keys; every latent row is fetched once for all those heads. Per tile
-// of 64 keys the eight warps first split the scores by key, then the softmax by row, then the output by
-// column; probabilities enter the second product as a bf16 pair (high and low part), which keeps them to about
-// 16 bits. The simple one (bf16 or fp32, any size): one CTA per token and head.
+// rows of its MMA tiles) and a range of keys; every latent row is fetched once for all those heads, in whole
+// pages by TMA. Two groups of eight warps work on 16 heads each (or on alternate key tiles of the same heads),
+// so that one group's softmax runs under the other's products. Per tile of 64 keys a group first splits the
+// scores by (column quarter, half of the keys), with the warp's part of the queries in registers, then the
+// softmax by row, then the output by column. Probabilities enter the second product as a bf16 pair (high and
+// low part), which keeps them to about 16 bits. The simple one (bf16 or fp32, any size): one CTA per token and head.
 #include "attn_mma.cuh"
 #include "elem_io.cuh"
 
@@ -22,20 +24,32 @@ template <class T>
 __global__ void __launch_bounds__(128)
 latent_append_kernel(nfk_latent_append_params p) {
   const int lane = threadIdx.x & 31;
+  // columns moved four at a time: all whole groups of four when every row starts on such a group
+  const bool vec = p.ld_src % 4 == 0 && p.ld % 4 == 0 && (reinterpret_cast<uintptr_t>(p.src) & 15) == 0 &&
+                   (reinterpret_cast<uintptr_t>(p.w) & 15) == 0 && (reinterpret_cast<uintptr_t>(p.pool) & 15) == 0;
+  const int n4 = vec ? p.rank / 4 * 4 : 0;
   for (int t = blockIdx.x * 4 + (threadIdx.x >> 5); t < p.T; t += gridDim.x * 4) {
     const T* src = reinterpret_cast<const T*>(p.src) + static_cast<long long>(t) * p.ld_src;
+    const int pos = p.positions[t];
+    const int page = page_of(pos, p.token_req[t], p.page_size, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages,
+                             p.status);
     float ss = 0.f;
-    for (int c = lane; c < p.rank; c += 32) {
+    for (int c = lane * 4; c < n4; c += 128) {
+      const float4 v = load4(src + c);
+      ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+    }
+    for (int c = n4 + lane; c < p.rank; c += 32) {
       const float v = to_f32(src[c]);
       ss += v * v;
     }
     const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(p.rank) + p.eps);
-    const int pos = p.positions[t];
-    const int page = page_of(pos, p.token_req[t], p.page_size, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages,
-                             p.status);
     if (page < 0) continue;
     T* dst = reinterpret_cast<T*>(p.pool) + (static_cast<long long>(page) * p.page_size + pos % p.page_size) * p.ld;
-    for (int c = lane; c < p.rank; c += 32) put(dst + c, to_f32(src[c]) * inv * p.w[c]);
+    for (int c = lane * 4; c < n4; c += 128) {
+      const float4 v = load4(src + c), w = load4(p.w + c);
+      store4(dst + c, make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w));
+    }
+    for (int c = n4 + lane; c < p.rank; c += 32) put(dst + c, to_f32(src[c]) * inv * p.w[c]);
   }
 }
 
@@ -110,253 +124,334 @@ latent_attn_simple_kernel(nfk_latent_attn_params p) {
 }
 
 // ---- tensor-core kernel -------------------------------------------------------------------------------
-constexpr int kLThreads = 256, kLTile = 64;
+constexpr int kLTile = 64;
+constexpr int kLGroup = 256, kLThreads = 2 * kLGroup;   // two groups of eight warps
 
-template <int DW, int MT>
+template <int DW, bool KSPLIT>
 struct LCfg {
   static constexpr int D = DW * 64;                       // latent columns
-  static constexpr int ROWS = MT * 16;
-  static constexpr int TILE_BYTES = kLTile * D * 2;
-  static constexpr int Q_BYTES = ROWS * D * 2;
-  static constexpr int S_LD = kLTile + 4;
-  static constexpr int S_BYTES = ROWS * S_LD * 4;
-  static constexpr int P_BYTES = ROWS * kLTile * 2;       // one part (high or low)
-  static constexpr int FIXED = Q_BYTES + S_BYTES + 2 * P_BYTES + 2 * ROWS * 4;
-  static constexpr int STAGES = 3 * TILE_BYTES + FIXED <= 110 * 1024 ? 3 : 2;
-  static constexpr int SMEM = FIXED + STAGES * TILE_BYTES;
+  static constexpr int ROWS = KSPLIT ? 16 : 32;           // heads per CTA, 16 per group
+  static constexpr int TILE_BYTES = kLTile * D * 2;       // [DW][64 keys][64 columns], 128-byte swizzle
+  static constexpr int S_LD = kLTile + 8;
+  static constexpr int S_BYTES = 4 * 16 * S_LD * 4;       // per group: score parts of the four column quarters
+  static constexpr int P_BYTES = 16 * kLTile * 2;         // per group: one part (high or low)
+  static constexpr int O_LD = D + 4;
+  static constexpr int GROUP_BYTES = S_BYTES + 2 * P_BYTES + 2 * 16 * 4;
+  static constexpr int FIXED = 2 * GROUP_BYTES + 128;
+  static constexpr int STAGES = 4 * TILE_BYTES + FIXED <= 200 * 1024 ? 4 : (3 * TILE_BYTES + FIXED <= 200 * 1024 ? 3 : 2);
+  static constexpr int SMEM = FIXED + STAGES * TILE_BYTES + 1024;
+  static_assert(16 * O_LD * 4 <= STAGES * TILE_BYTES, "the merge of the two groups reuses the key tiles");
 };
 
 // Byte offset of 16-byte chunk `ch` of row `row` in a tile of `row_bytes`-byte rows.
 __device__ __forceinline__ uint32_t sw_off(int row, int ch, int row_bytes) {
   return static_cast<uint32_t>(row * row_bytes + ((ch ^ (row & 7)) << 4));
 }
+// ... in a key tile: blocks of 64 columns, 128 bytes per key.
+__device__ __forceinline__ uint32_t key_off(int key, int ch) {
+  return static_cast<uint32_t>((ch >> 3) * (kLTile * 128) + key * 128 + (((ch ^ key) & 7) << 4));
+}
 // A fragment (16 rows x 16 k) of a row-major tile.
 __device__ __forceinline__ void load_a(uint32_t (&a)[4], uint32_t base, int row0, int ks, int row_bytes) {
   const int lane = threadIdx.x & 31;
   ldsm_x4(base + sw_off(row0 + (lane & 15), 2 * ks + (lane >> 4), row_bytes), a[0], a[1], a[2], a[3]);
 }
+__device__ __forceinline__ void group_sync(int g) { asm volatile("bar.sync %0, 256;" ::"r"(g + 1) : "memory"); }
+// Count of the warps that are done with a key tile; orders their reads before what the last one does next.
+__device__ __forceinline__ int count_done(uint32_t addr) {
+  int old;
+  asm volatile("atom.acq_rel.cta.shared::cta.add.s32 %0, [%1], 1;" : "=r"(old) : "r"(addr) : "memory");
+  return old + 1;
+}
 
-template <int DW, int MT>
+// KSPLIT false: the groups take different heads (rows 0-15 and 16-31) over the same key tiles; true (at most 16
+// heads): they take alternate key tiles and are merged at the end. Either way they only share the tiles, so
+// one group's softmax runs under the other's products. The warp that is last to finish with a tile starts
+// the copy of the tile that takes its place.
+template <int DW, bool KSPLIT>
 __global__ void __launch_bounds__(kLThreads, 1)
-latent_attn_mma_kernel(nfk_latent_attn_params p) {
-  using Cfg = LCfg<DW, MT>;
+latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_params p) {
+  using Cfg = LCfg<DW, KSPLIT>;
   constexpr int D = Cfg::D, ROWS = Cfg::ROWS;
-  extern __shared__ __align__(128) uint8_t smem[];
+  constexpr int kDone = KSPLIT ? kLGroup / 32 : kLThreads / 32;    // warps that read a tile
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const uint32_t sb = smem_u32(smem);
-  const uint32_t q_base = sb + Cfg::STAGES * Cfg::TILE_BYTES;
-  float* s_s = reinterpret_cast<float*>(smem + Cfg::STAGES * Cfg::TILE_BYTES + Cfg::Q_BYTES);
-  const uint32_t p_hi = q_base + Cfg::Q_BYTES + Cfg::S_BYTES, p_lo = p_hi + Cfg::P_BYTES;
-  uint8_t* p_ptr = smem + Cfg::STAGES * Cfg::TILE_BYTES + Cfg::Q_BYTES + Cfg::S_BYTES;
+  const int warp = (threadIdx.x >> 5) & 7, lane = threadIdx.x & 31, grp = threadIdx.x / kLGroup;
+  uint8_t* fixed = smem + Cfg::STAGES * Cfg::TILE_BYTES;
+  float* s_s = reinterpret_cast<float*>(fixed + grp * Cfg::GROUP_BYTES);
+  uint8_t* p_ptr = fixed + grp * Cfg::GROUP_BYTES + Cfg::S_BYTES;
+  const uint32_t p_hi = smem_u32(p_ptr), p_lo = p_hi + Cfg::P_BYTES;
   float* alpha_s = reinterpret_cast<float*>(p_ptr + 2 * Cfg::P_BYTES);
-  float* l_s = alpha_s + ROWS;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* l_s = alpha_s + 16;
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(fixed + 2 * Cfg::GROUP_BYTES);
+  int* done_s = reinterpret_cast<int*>(full_bar + 4);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(done_s + 4);
   const int hgroups = (p.heads + ROWS - 1) / ROWS;
   const int hg = blockIdx.x % hgroups;
   const int split = (blockIdx.x / hgroups) % p.splits;
   const int ti = blockIdx.x / (hgroups * p.splits);
   const int tok = p.tokens[ti];
   const int pos = p.positions[tok], req = p.token_req[tok];
-  const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
   const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
   const int key0 = lo / kPage * kPage;                         // tiles start on a page
   const int n_all = (pos - key0) / kLTile + 1;
   const int per = (n_all + p.splits - 1) / p.splits;
-  const int t_begin = split * per, t_end = min(n_all, t_begin + per);
+  const int t_begin = min(n_all, split * per), n_tiles = min(n_all, t_begin + per) - t_begin;
+  const int head0 = hg * ROWS + (KSPLIT ? 0 : grp * 16);       // first head of this group
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < Cfg::STAGES; ++s) {
+      mbar_init(&full_bar[s], 1);
+      done_s[s] = 0;
+    }
+    *abort_flag = 0;
+    mbar_fence_init();
+    tma_prefetch_desc(&tmC);
+  }
+  __syncthreads();
+
+  // ---- copies: whole pages, lanes 0-3 one page of the tile each ----
   const int pg0 = p.kv_indptr[req], np = p.kv_indptr[req + 1] - pg0;
   const int first = p.kv_first != nullptr ? p.kv_first[req] : 0;
-
-  // queries of this CTA's heads (rows past the last head are zero)
-  for (int i = threadIdx.x; i < ROWS * (D / 8); i += kLThreads) {
-    const int r = i / (D / 8), ch = i % (D / 8), head = hg * ROWS + r;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (head < p.heads)
-      v = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.q) +
-                                          static_cast<long long>(tok) * p.ld_q + static_cast<long long>(head) * D + ch * 8);
-    *reinterpret_cast<uint4*>(smem + Cfg::STAGES * Cfg::TILE_BYTES + sw_off(r, ch, D * 2)) = v;
-  }
-  auto issue = [&](int t) {
-    if (t < t_end) {
-      const uint32_t st = sb + ((t - t_begin) % Cfg::STAGES) * Cfg::TILE_BYTES;
-#pragma unroll
-      for (int j = 0; j < kLTile * (D / 8) / kLThreads; ++j) {
-        const int idx = threadIdx.x + kLThreads * j;
-        const int row = idx / (D / 8), ch = idx % (D / 8);
-        const int key = min(key0 + t * kLTile + row, pos);     // past the last key: any valid row, masked below
-        int slot = key / kPage - first;
-        if (slot < 0 || slot >= np) {
-          report_status(p.status, NF_ST_BAD_INDEX);
-          slot = 0;
-        }
-        int page = p.kv_indices[pg0 + slot];
-        if (page < 0 || page >= p.num_pages) {
-          report_status(p.status, NF_ST_BAD_INDEX);
-          page = 0;
-        }
-        cp_async16(st + sw_off(row, ch, D * 2),
-                   pool + (static_cast<long long>(page) * kPage + key % kPage) * D + ch * 8);
-      }
-    }
-    cp_async_commit();
+  auto page_at = [&](int t) {
+    // past the last key: the last page again, masked by position
+    const int slot = min((key0 + (t_begin + t) * kLTile) / kPage + lane, pos / kPage) - first;
+    return (slot >= 0 && slot < np) ? p.kv_indices[pg0 + slot] : -1;    // looked at when the copy starts, not before
   };
+  auto copy_tile = [&](int t, int page) {       // one whole warp
+    const int s = t % Cfg::STAGES;
+    if (page < 0 || page >= p.num_pages) {
+      report_status(p.status, NF_ST_BAD_INDEX);
+      page = 0;
+    }
+    if (lane == 0) mbar_expect_tx(&full_bar[s], Cfg::TILE_BYTES);
+    __syncwarp();
+    if (lane < 4) {
 #pragma unroll
-  for (int s = 0; s < Cfg::STAGES - 1; ++s) issue(t_begin + s);
+      for (int b = 0; b < DW; ++b)
+        tma_load_2d(smem + s * Cfg::TILE_BYTES + b * (kLTile * 128) + lane * (kPage * 128), &tmC, &full_bar[s], b * 64,
+                    page * kPage);
+    }
+  };
+  if (threadIdx.x < 32) {
+    for (int t = 0; t < min(n_tiles, Cfg::STAGES); ++t) copy_tile(t, lane < 4 ? page_at(t) : 0);
+  }
 
-  float o[MT][DW][4];
-#pragma unroll
-  for (int a = 0; a < MT; ++a)
-#pragma unroll
-    for (int b = 0; b < DW; ++b) o[a][b][0] = o[a][b][1] = o[a][b][2] = o[a][b][3] = 0.f;
-  // softmax rows of this warp: 2 * MT of them, state replicated in its lanes
-  constexpr int RW = ROWS / 8;
-  float m_r[RW], l_r[RW];
-#pragma unroll
-  for (int r = 0; r < RW; ++r) {
-    const int head = hg * ROWS + warp * RW + r;
-    const bool sink = p.sinks != nullptr && head < p.heads && split == 0;
-    m_r[r] = sink ? p.sinks[head] * kLog2e : -INFINITY;
-    l_r[r] = sink ? 1.f : 0.f;
-  }
-  const float scale = p.scale * kLog2e;
-
-  for (int t = t_begin; t < t_end; ++t) {
-    cp_async_wait<Cfg::STAGES - 2>();
-    __syncthreads();           // tile t is in shared memory, every warp is done with tile t - 1
-    issue(t + Cfg::STAGES - 1);
-    const uint32_t st = sb + ((t - t_begin) % Cfg::STAGES) * Cfg::TILE_BYTES;
-    // 1. scores: MT = 2: 16 keys x one row tile per warp; MT = 1: 8 keys per warp
-    {
-      const int mt = MT == 2 ? (warp & 1) : 0;
-      const int k0 = MT == 2 ? (warp >> 1) * 16 : warp * 8;
-      float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-      const int mm = lane >> 3, rr = lane & 7;
-#pragma unroll 4
-      for (int ks = 0; ks < D / 16; ks += 2) {
-        uint32_t a0[4], a1[4], b0, b1, b2, b3;
-        load_a(a0, q_base, mt * 16, ks, D * 2);
-        load_a(a1, q_base, mt * 16, ks + 1, D * 2);
-        if (MT == 2) {
-          ldsm_x4(st + sw_off(k0 + (mm >> 1) * 8 + rr, 2 * ks + (mm & 1), D * 2), b0, b1, b2, b3);
-          mma_bf16(s0, a0, b0, b1);
-          mma_bf16(s1, a0, b2, b3);
-          ldsm_x4(st + sw_off(k0 + (mm >> 1) * 8 + rr, 2 * ks + 2 + (mm & 1), D * 2), b0, b1, b2, b3);
-          mma_bf16(s0, a1, b0, b1);
-          mma_bf16(s1, a1, b2, b3);
-        } else {
-          ldsm_x4(st + sw_off(k0 + rr, 2 * ks + mm, D * 2), b0, b1, b2, b3);
-          mma_bf16(s0, a0, b0, b1);
-          mma_bf16(s0, a1, b2, b3);
-        }
-      }
-      const int r0 = mt * 16 + (lane >> 2), c0 = k0 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(s_s + r0 * Cfg::S_LD + c0) = make_float2(s0[0], s0[1]);
-      *reinterpret_cast<float2*>(s_s + (r0 + 8) * Cfg::S_LD + c0) = make_float2(s0[2], s0[3]);
-      if (MT == 2) {
-        *reinterpret_cast<float2*>(s_s + r0 * Cfg::S_LD + c0 + 8) = make_float2(s1[0], s1[1]);
-        *reinterpret_cast<float2*>(s_s + (r0 + 8) * Cfg::S_LD + c0 + 8) = make_float2(s1[2], s1[3]);
-      }
-    }
-    __syncthreads();
-    // 2. softmax of this warp's rows, two keys per lane
-    {
-      const int key = key0 + t * kLTile + lane * 2;
-      const bool in0 = key >= lo && key <= pos, in1 = key + 1 >= lo && key + 1 <= pos;
-#pragma unroll
-      for (int r = 0; r < RW; ++r) {
-        const int row = warp * RW + r;
-        const float2 s = *reinterpret_cast<const float2*>(s_s + row * Cfg::S_LD + lane * 2);
-        const float x0 = in0 ? s.x * scale : -INFINITY, x1 = in1 ? s.y * scale : -INFINITY;
-        float mx = fmaxf(x0, x1);
-#pragma unroll
-        for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-        const float mn = fmaxf(m_r[r], mx);
-        const float ms = mn == -INFINITY ? 0.f : mn;
-        const float al = exp2f(m_r[r] - ms);
-        m_r[r] = mn;
-        const float e0 = exp2f(x0 - ms), e1 = exp2f(x1 - ms);
-        l_r[r] = l_r[r] * al + warp_sum(e0 + e1);
-        const uint32_t hi = pack_bf16x2(e0, e1);
-        const float2 hf = unpack_bf16x2(hi);
-        const uint32_t off = sw_off(row, lane >> 2, kLTile * 2) + (lane & 3) * 4;
-        *reinterpret_cast<uint32_t*>(p_ptr + off) = hi;
-        *reinterpret_cast<uint32_t*>(p_ptr + Cfg::P_BYTES + off) = pack_bf16x2(e0 - hf.x, e1 - hf.y);
-        if (lane == 0) alpha_s[row] = al;
-      }
-    }
-    __syncthreads();
-    // 3. output: DW * 8 columns per warp
-    {
-      const int mm = lane >> 3, rr = lane & 7;
-#pragma unroll
-      for (int a = 0; a < MT; ++a) {
-        const float al0 = alpha_s[a * 16 + (lane >> 2)], al1 = alpha_s[a * 16 + 8 + (lane >> 2)];
-#pragma unroll
-        for (int b = 0; b < DW; ++b) {
-          o[a][b][0] *= al0; o[a][b][1] *= al0; o[a][b][2] *= al1; o[a][b][3] *= al1;
-        }
-      }
-#pragma unroll
-      for (int ks = 0; ks < kLTile / 16; ++ks) {
-        uint32_t ph[MT][4], pl[MT][4];
-#pragma unroll
-        for (int a = 0; a < MT; ++a) {
-          load_a(ph[a], p_hi, a * 16, ks, kLTile * 2);
-          load_a(pl[a], p_lo, a * 16, ks, kLTile * 2);
-        }
-        const int key = ks * 16 + (mm & 1) * 8 + rr;
-#pragma unroll
-        for (int b = 0; b < DW; b += 2) {
-          const int ch = min(warp * DW + b + (mm >> 1), D / 8 - 1);   // odd DW: the second half is not used
-          uint32_t b0, b1, b2, b3;
-          ldsm_x4_trans(st + sw_off(key, ch, D * 2), b0, b1, b2, b3);
-#pragma unroll
-          for (int a = 0; a < MT; ++a) {
-            mma_bf16(o[a][b], ph[a], b0, b1);
-            mma_bf16(o[a][b], pl[a], b0, b1);
-            if (b + 1 < DW) {
-              mma_bf16(o[a][b + 1 < DW ? b + 1 : b], ph[a], b2, b3);
-              mma_bf16(o[a][b + 1 < DW ? b + 1 : b], pl[a], b2, b3);
-            }
-          }
-        }
-      }
-    }
-  }
-  cp_async_wait<0>();
-  // row sums (and reference maxima, for the merge) to every warp
-  __syncthreads();
-  if (lane == 0) {
-#pragma unroll
-    for (int r = 0; r < RW; ++r) {
-      l_s[warp * RW + r] = l_r[r];
-      alpha_s[warp * RW + r] = m_r[r];
-    }
-  }
-  __syncthreads();
-#pragma unroll
-  for (int a = 0; a < MT; ++a)
+  // ---- scores by (column quarter, key half), softmax by row, output by column ----
+  const int kq = warp >> 1, kh = warp & 1;
+  uint32_t qa[DW][4];                                          // this quarter's columns of the group's rows
+  {
+    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + static_cast<long long>(tok) * p.ld_q;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const int row = a * 16 + half * 8 + (lane >> 2), head = hg * ROWS + row;
-      if (head >= p.heads) continue;
-      const float l = l_s[row], inv = l > 0.f ? 1.f / l : 0.f;
-      const int c0 = warp * DW * 8 + (lane & 3) * 2;
-      if (p.splits == 1) {
-        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(tok) * p.ld_out +
-                             static_cast<long long>(head) * D;
+      const int head = head0 + half * 8 + (lane >> 2);
+      const __nv_bfloat16* row = q + static_cast<long long>(head) * D + kq * (DW * 16) + (lane & 3) * 2;
 #pragma unroll
-        for (int b = 0; b < DW; ++b)
-          *reinterpret_cast<uint32_t*>(dst + c0 + b * 8) = pack_bf16x2(o[a][b][2 * half] * inv, o[a][b][2 * half + 1] * inv);
-      } else {
-        float* ws = p.workspace + ((static_cast<long long>(ti) * p.splits + split) * p.heads + head) * (D + 2);
+      for (int ks = 0; ks < DW; ++ks) {
+        qa[ks][half] = head < p.heads ? *reinterpret_cast<const uint32_t*>(row + ks * 16) : 0u;
+        qa[ks][half + 2] = head < p.heads ? *reinterpret_cast<const uint32_t*>(row + ks * 16 + 8) : 0u;
+      }
+    }
+  }
+  float o[DW][4];
 #pragma unroll
-        for (int b = 0; b < DW; ++b)
-          *reinterpret_cast<float2*>(ws + c0 + b * 8) = make_float2(o[a][b][2 * half], o[a][b][2 * half + 1]);
-        if (warp == 0 && (lane & 3) == 0) {
-          ws[D] = alpha_s[row];
-          ws[D + 1] = l;
+  for (int b = 0; b < DW; ++b) o[b][0] = o[b][1] = o[b][2] = o[b][3] = 0.f;
+  const int row_r = warp * 2 + (lane >> 4);                    // softmax row of this half warp
+  float m_r = -INFINITY, l_r = 0.f;
+  {
+    const int head = head0 + row_r;
+    if (p.sinks != nullptr && head < p.heads && split == 0 && !(KSPLIT && grp == 1)) {
+      m_r = p.sinks[head] * kLog2e;
+      l_r = (lane & 15) == 0 ? 1.f : 0.f;
+    }
+  }
+  const float scale = p.scale * kLog2e;
+  const int mm = lane >> 3, rr = lane & 7;
+
+  for (int t = KSPLIT ? grp : 0; t < n_tiles; t += KSPLIT ? 2 : 1) {
+    const int s = t % Cfg::STAGES;
+    const uint32_t st = sb + s * Cfg::TILE_BYTES;
+    // page of the tile that will take this one's place, in case this warp is the one to copy it
+    const int page = (lane < 4 && t + Cfg::STAGES < n_tiles) ? page_at(t + Cfg::STAGES) : 0;
+    // a wait that runs out is reported; the warps go on in step, so that they meet at their barriers
+    if (*abort_flag == 0 && !mbar_wait(&full_bar[s], (t / Cfg::STAGES) & 1)) {
+      if (lane == 0) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
+      *abort_flag = 1;
+    }
+    __syncwarp();
+    // 1. scores of 32 keys over a quarter of the columns
+    {
+      float sc[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < DW; ++ks) {
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+          uint32_t b0, b1, b2, b3;
+          ldsm_x4(st + key_off(kh * 32 + g * 16 + (mm >> 1) * 8 + rr, (kq * DW + ks) * 2 + (mm & 1)), b0, b1, b2, b3);
+          mma_bf16(sc[2 * g], qa[ks], b0, b1);
+          mma_bf16(sc[2 * g + 1], qa[ks], b2, b3);
+        }
+      }
+      float* dst = s_s + (kq * 16 + (lane >> 2)) * Cfg::S_LD + kh * 32 + (lane & 3) * 2;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        *reinterpret_cast<float2*>(dst + j * 8) = make_float2(sc[j][0], sc[j][1]);
+        *reinterpret_cast<float2*>(dst + 8 * Cfg::S_LD + j * 8) = make_float2(sc[j][2], sc[j][3]);
+      }
+    }
+    group_sync(grp);
+    // 2. softmax of this warp's two rows: half a warp per row, four keys per lane
+    {
+      const int key = key0 + (t_begin + t) * kLTile + (lane & 15) * 4;
+      const float* src = s_s + row_r * Cfg::S_LD + (lane & 15) * 4;
+      float4 v = *reinterpret_cast<const float4*>(src);
+#pragma unroll
+      for (int k = 1; k < 4; ++k) {
+        const float4 w = *reinterpret_cast<const float4*>(src + k * 16 * Cfg::S_LD);
+        v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+      }
+      v.x = (key >= lo && key <= pos) ? v.x * scale : -INFINITY;
+      v.y = (key + 1 >= lo && key + 1 <= pos) ? v.y * scale : -INFINITY;
+      v.z = (key + 2 >= lo && key + 2 <= pos) ? v.z * scale : -INFINITY;
+      v.w = (key + 3 >= lo && key + 3 <= pos) ? v.w * scale : -INFINITY;
+      float mx = fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w));
+#pragma unroll
+      for (int off = 8; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      const float mn = fmaxf(m_r, mx);
+      const float ms = mn == -INFINITY ? 0.f : mn;
+      const float al = exp2f(m_r - ms);
+      m_r = mn;
+      const float e0 = exp2f(v.x - ms), e1 = exp2f(v.y - ms), e2 = exp2f(v.z - ms), e3 = exp2f(v.w - ms);
+      l_r = l_r * al + ((e0 + e1) + (e2 + e3));      // this lane's keys; the row's lanes are added up at the end
+      const uint32_t h0 = pack_bf16x2(e0, e1), h1 = pack_bf16x2(e2, e3);
+      const float2 f0 = unpack_bf16x2(h0), f1 = unpack_bf16x2(h1);
+      const uint32_t off = sw_off(row_r, (lane & 15) >> 1, kLTile * 2) + (lane & 1) * 8;
+      *reinterpret_cast<uint2*>(p_ptr + off) = make_uint2(h0, h1);
+      *reinterpret_cast<uint2*>(p_ptr + Cfg::P_BYTES + off) =
+          make_uint2(pack_bf16x2(e0 - f0.x, e1 - f0.y), pack_bf16x2(e2 - f1.x, e3 - f1.y));
+      if ((lane & 15) == 0) alpha_s[row_r] = al;
+    }
+    group_sync(grp);
+    // 3. output: DW * 8 columns per warp
+    {
+      const float al0 = alpha_s[lane >> 2], al1 = alpha_s[8 + (lane >> 2)];
+      if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {
+#pragma unroll
+        for (int b = 0; b < DW; ++b) {
+          o[b][0] *= al0; o[b][1] *= al0; o[b][2] *= al1; o[b][3] *= al1;
         }
       }
     }
+#pragma unroll
+    for (int ks = 0; ks < kLTile / 16; ++ks) {
+      uint32_t ph[4], pl[4];
+      load_a(ph, p_hi, 0, ks, kLTile * 2);
+      load_a(pl, p_lo, 0, ks, kLTile * 2);
+      const int key = ks * 16 + (mm & 1) * 8 + rr;
+#pragma unroll
+      for (int b = 0; b < DW; b += 2) {
+        const int ch = min(warp * DW + b + (mm >> 1), D / 8 - 1);   // odd DW: the second half is not used
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4_trans(st + key_off(key, ch), b0, b1, b2, b3);
+        mma_bf16(o[b], ph, b0, b1);
+        if (b + 1 < DW) mma_bf16(o[b + 1 < DW ? b + 1 : b], ph, b2, b3);
+        mma_bf16(o[b], pl, b0, b1);
+        if (b + 1 < DW) mma_bf16(o[b + 1 < DW ? b + 1 : b], pl, b2, b3);
+      }
+    }
+    __syncwarp();
+    int last = 0;
+    if (lane == 0) {
+      last = count_done(smem_u32(&done_s[s])) == kDone;
+      if (last) done_s[s] = 0;
+    }
+    if (__shfl_sync(0xffffffffu, last, 0) != 0 && t + Cfg::STAGES < n_tiles) copy_tile(t + Cfg::STAGES, page);
+  }
+  if (*abort_flag != 0 && threadIdx.x == 0) {
+    // a wait ran out: give copies still in flight a bounded chance to land before the CTA ends
+    for (int t = max(0, n_tiles - Cfg::STAGES); t < n_tiles; ++t) (void)mbar_wait(&full_bar[t % Cfg::STAGES], (t / Cfg::STAGES) & 1);
+  }
+  // row sums and reference maxima to every warp of the group
+#pragma unroll
+  for (int off = 8; off > 0; off >>= 1) l_r += __shfl_xor_sync(0xffffffffu, l_r, off);
+  group_sync(grp);            // the last tile's rescaling factors have been read
+  if ((lane & 15) == 0) {
+    l_s[row_r] = l_r;
+    alpha_s[row_r] = m_r;
+  }
+  if (KSPLIT) {
+    // merge: group 1 leaves its output over the key tiles, group 0 brings both to the larger maximum
+    __syncthreads();
+    float* mo = reinterpret_cast<float*>(smem);
+    const float* other_m = reinterpret_cast<const float*>(fixed + Cfg::GROUP_BYTES + Cfg::S_BYTES + 2 * Cfg::P_BYTES);
+    const int c0 = warp * DW * 8 + (lane & 3) * 2;
+    if (grp == 1) {
+#pragma unroll
+      for (int half = 0; half < 2; ++half)
+#pragma unroll
+        for (int b = 0; b < DW; ++b)
+          *reinterpret_cast<float2*>(mo + (half * 8 + (lane >> 2)) * Cfg::O_LD + c0 + b * 8) = make_float2(o[b][2 * half], o[b][2 * half + 1]);
+    }
+    __syncthreads();
+    if (grp == 1) return;
+    float ms[2], f0[2], f1[2];
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int row = half * 8 + (lane >> 2);
+      const float m0 = alpha_s[row], m1 = other_m[row];
+      ms[half] = fmaxf(m0, m1);
+      const float msafe = ms[half] == -INFINITY ? 0.f : ms[half];
+      f0[half] = exp2f(m0 - msafe);
+      f1[half] = exp2f(m1 - msafe);
+#pragma unroll
+      for (int b = 0; b < DW; ++b) {
+        const float2 v = *reinterpret_cast<const float2*>(mo + row * Cfg::O_LD + c0 + b * 8);
+        o[b][2 * half] = o[b][2 * half] * f0[half] + v.x * f1[half];
+        o[b][2 * half + 1] = o[b][2 * half + 1] * f0[half] + v.y * f1[half];
+      }
+    }
+    float l[2];
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int row = half * 8 + (lane >> 2);
+      l[half] = l_s[row] * f0[half] + other_m[16 + row] * f1[half];
+    }
+    group_sync(0);            // everyone has read the maxima and sums
+    if (warp == 0 && (lane & 3) == 0) {
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        l_s[half * 8 + (lane >> 2)] = l[half];
+        alpha_s[half * 8 + (lane >> 2)] = ms[half];
+      }
+    }
+  }
+  group_sync(grp);
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int row = half * 8 + (lane >> 2), head = head0 + row;
+    if (head >= p.heads) continue;
+    const float l = l_s[row], inv = l > 0.f ? 1.f / l : 0.f;
+    const int c0 = warp * DW * 8 + (lane & 3) * 2;
+    if (p.splits == 1) {
+      __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(tok) * p.ld_out +
+                           static_cast<long long>(head) * D;
+#pragma unroll
+      for (int b = 0; b < DW; ++b)
+        *reinterpret_cast<uint32_t*>(dst + c0 + b * 8) = pack_bf16x2(o[b][2 * half] * inv, o[b][2 * half + 1] * inv);
+    } else {
+      float* ws = p.workspace + ((static_cast<long long>(ti) * p.splits + split) * p.heads + head) * (D + 2);
+#pragma unroll
+      for (int b = 0; b < DW; ++b)
+        *reinterpret_cast<float2*>(ws + c0 + b * 8) = make_float2(o[b][2 * half], o[b][2 * half + 1]);
+      if (warp == 0 && (lane & 3) == 0) {
+        ws[D] = alpha_s[row];
+        ws[D + 1] = l;
+      }
+    }
+  }
 }
 
 __global__ void __launch_bounds__(128)
@@ -385,21 +480,24 @@ latent_attn_merge_kernel(nfk_latent_attn_params p) {
   }
 }
 
-template <int DW, int MT>
+template <int DW, bool KSPLIT>
 int launch_latent(const nfk_latent_attn_params& p, cudaStream_t stream) {
-  using Cfg = LCfg<DW, MT>;
+  using Cfg = LCfg<DW, KSPLIT>;
   static bool attr_dev[kMaxDevices] = {false};
   bool& attr = attr_dev[device_slot()];
   if (!attr) {
-    if (cudaFuncSetAttribute(latent_attn_mma_kernel<DW, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) !=
+    if (cudaFuncSetAttribute(latent_attn_mma_kernel<DW, KSPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) !=
         cudaSuccess)
       return NF_ERR_CUDA;
     attr = true;
   }
+  CUtensorMap tm;
+  const int rc = make_tmap_bf16_2d(&tm, p.pool, static_cast<uint64_t>(p.num_pages) * kPage, Cfg::D, Cfg::D, kPage, 64);
+  if (rc != NF_OK) return rc;
   const int hgroups = (p.heads + Cfg::ROWS - 1) / Cfg::ROWS;
   const long long grid = static_cast<long long>(p.n_tokens) * p.splits * hgroups;
   if (grid > 0x7fffffffll) return NF_ERR_BAD_ARG;
-  latent_attn_mma_kernel<DW, MT><<<static_cast<int>(grid), kLThreads, Cfg::SMEM, stream>>>(p);
+  latent_attn_mma_kernel<DW, KSPLIT><<<static_cast<int>(grid), kLThreads, Cfg::SMEM, stream>>>(tm, p);
   if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
   if (p.splits > 1) {
     latent_attn_merge_kernel<<<p.n_tokens * p.heads, 128, 0, stream>>>(p);
@@ -409,7 +507,7 @@ int launch_latent(const nfk_latent_attn_params& p, cudaStream_t stream) {
 }
 template <int DW>
 int launch_latent_mt(const nfk_latent_attn_params& p, cudaStream_t stream) {
-  return p.heads <= 16 ? launch_latent<DW, 1>(p, stream) : launch_latent<DW, 2>(p, stream);
+  return p.heads <= 16 ? launch_latent<DW, true>(p, stream) : launch_latent<DW, false>(p, stream);
 }
 
 bool mma_ok(const nfk_latent_attn_params& p) {

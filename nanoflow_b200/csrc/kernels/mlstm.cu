@@ -422,10 +422,12 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
         for (int ch = part; ch < DP / 8; ch += 4) {
           const uint4 q = *reinterpret_cast<const uint4*>(smem + C::Q_OFF + swz(t, ch, DP * 2));
           const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
+          const float4 n0 = *reinterpret_cast<const float4*>(n_s + ch * 8), n1 = *reinterpret_cast<const float4*>(n_s + ch * 8 + 4);
+          const float nn[8] = {n0.x, n0.y, n0.z, n0.w, n1.x, n1.y, n1.z, n1.w};
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
             const float2 f = unpack_bf16x2(qw[j]);
-            d += f.x * n_s[ch * 8 + 2 * j] + f.y * n_s[ch * 8 + 2 * j + 1];
+            d += f.x * nn[2 * j] + f.y * nn[2 * j + 1];
           }
         }
         d = quad_sum(d);
@@ -451,15 +453,14 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
           }
         }
 #pragma unroll
-        for (int g = 0; g < 2; ++g) {
-          const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, half * 4 + 2 * g + (mm >> 1), kVs * 2);
-          ldsm_x4_trans(sb + C::SH_OFF + off, b0, b1, b2, b3);
-          mma_bf16(qs[2 * g], a, b0, b1);
-          mma_bf16(qs[2 * g + 1], a, b2, b3);
-          ldsm_x4_trans(sb + C::SL_OFF + off, b0, b1, b2, b3);
-          mma_bf16(qs[2 * g], a, b0, b1);
-          mma_bf16(qs[2 * g + 1], a, b2, b3);
-        }
+        for (int hl = 0; hl < 2; ++hl)        // high parts of all columns, then low parts
+#pragma unroll
+          for (int g = 0; g < 2; ++g) {
+            const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, half * 4 + 2 * g + (mm >> 1), kVs * 2);
+            ldsm_x4_trans(sb + (hl == 0 ? C::SH_OFF : C::SL_OFF) + off, b0, b1, b2, b3);
+            mma_bf16(qs[2 * g], a, b0, b1);
+            mma_bf16(qs[2 * g + 1], a, b2, b3);
+          }
       }
       // ---- weights, row sums, bf16 pair of the weighted scores ----
       const int r0 = mt * 16 + (lane >> 2), r1 = r0 + 8;
@@ -552,8 +553,11 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
 #pragma unroll
         for (int a = 0; a < C::MTS; ++a) {
           mma_bf16(S[a][b], ak[a], h0, h1);
-          mma_bf16(S[a][b], ak[a], l0, l1);
           mma_bf16(S[a][b + 1], ak[a], h2, h3);
+        }
+#pragma unroll
+        for (int a = 0; a < C::MTS; ++a) {
+          mma_bf16(S[a][b], ak[a], l0, l1);
           mma_bf16(S[a][b + 1], ak[a], l2, l3);
         }
       }
