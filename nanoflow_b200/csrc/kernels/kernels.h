@@ -325,10 +325,12 @@ typedef struct nfk_mlstm_params {
   float gate_cap, q_scale;
   int dtype;
   int impl;                  // prefill: 0 = choose, 1 = token by token, 2 = chunked on tensor cores (bf16)
-  // chunked form: items [num_items][4] (request, first token, tokens, segment of the request) and scratch for
-  // the segments' states (see mlstm.cu)
+  // chunked form: items [num_items][4] (request, first token, tokens, segment of the request), in token order, and
+  // scratch: (num_tokens / 64 + num_items + 1) * heads * 192 floats of gate values, and if a request has several
+  // segments num_items * heads * (dim * vdim + dim + 8) floats for their states
   const int* items;
   int num_items;
+  int num_tokens;            // rows of qkv that hold tokens of this iteration
   float* scratch;
   long long scratch_floats;
   unsigned int* status;

@@ -12,7 +12,8 @@
 // nfk_mlstm_prefill  impl 1: token by token with 32 columns of S in shared memory; any size, bf16 or fp32.
 //                    impl 2 (bf16): chunks of 64 tokens on tensor cores. With F the running sum of f inside the
 //                    chunk, a_j = i_j - F_j and M_t = max(m_in, max_{j<=t} a_j), every weight of the chunk is
-//                    an exponential of a non-positive number: token j enters output t with e^(a_j - M_t), the
+//                    an exponential of a non-positive number (a small kernel computes a, its running maximum and F
+//                    of all chunks first): token j enters output t with e^(a_j - M_t), the
 //                    incoming state with e^(m_in - M_t), and m_t = F_t + M_t. Weights, weighted values and the
 //                    state enter the products as bf16 pairs (high and low part), so they keep about 16 bits.
 //                    Long prompts are cut into segments: their own contributions are computed side by side from
@@ -203,7 +204,7 @@ constexpr int kChunk = 64, kVs = 64, kChThreads = 256;
 
 template <int DP>
 struct ChCfg {
-  static constexpr int QK_BYTES = kChunk * DP * 2;
+  static constexpr int QK_BYTES = kChunk * DP * 2;        // [DP / 64][64 tokens][64 columns], 128-byte swizzle
   static constexpr int V_BYTES = kChunk * kVs * 2;
   static constexpr int S_BYTES = DP * kVs * 2;
   static constexpr int P_BYTES = kChunk * kChunk * 2;
@@ -217,20 +218,29 @@ struct ChCfg {
   static constexpr int WH_OFF = PL_OFF + P_BYTES;         // weighted values, high / low part
   static constexpr int WL_OFF = WH_OFF + V_BYTES;
   static constexpr int F_OFF = WL_OFF + V_BYTES;          // fp32 arrays
-  static constexpr int N_F32 = DP + 8 * kChunk + 8;
-  static constexpr int SMEM = F_OFF + N_F32 * 4;
+  static constexpr int NPARTS = 2 * kChThreads / DP;      // partial sums that n is kept in
+  static constexpr int N_F32 = NPARTS * DP + 10 * kChunk;
+  static constexpr int BAR_OFF = F_OFF + N_F32 * 4;
+  static constexpr int SMEM = BAR_OFF + 64 + 1024;
   static constexpr int WM = DP / 16 < 8 ? DP / 16 : 8;    // warps along dim in the state update
   static constexpr int WN = 8 / WM;                       // ... and along the columns
   static constexpr int MTS = DP / 16 / WM;                // 16-row tiles of S per warp
   static constexpr int NTS = 8 / WN;                      // 8-column tiles of S per warp
 };
 
-__device__ __forceinline__ uint32_t swz(int row, int ch, int row_bytes) {
-  return static_cast<uint32_t>(row * row_bytes + ((ch ^ (row & 7)) << 4));
+// Byte offset of 16-byte chunk `ch` of row `row`: 128-byte rows, and blocks of 64 columns of 64-row tiles.
+__device__ __forceinline__ uint32_t swz(int row, int ch) {
+  return static_cast<uint32_t>(row * 128 + ((ch ^ (row & 7)) << 4));
 }
-__device__ __forceinline__ void cp_async16_zfill(uint32_t smem_addr, const void* g, bool valid) {
-  const int n = valid ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr), "l"(g), "r"(n) : "memory");
+__device__ __forceinline__ uint32_t swz_blk(int row, int ch) {
+  return static_cast<uint32_t>((ch >> 3) * (kChunk * 128) + row * 128 + (((ch ^ row) & 7) << 4));
+}
+__device__ __forceinline__ void tma_load_3d(void* smem_dst, const CUtensorMap* tm, uint64_t* bar, int x, int y, int z) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes"
+      " [%0], [%1, {%3, %4, %5}], [%2];" ::"r"(smem_u32(smem_dst)),
+      "l"(reinterpret_cast<uint64_t>(tm)), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z)
+      : "memory");
 }
 
 // Floats of scratch per (item, head): S [dim][vdim], n [dim], then m and the sum of f of the segment's own
@@ -238,24 +248,78 @@ __device__ __forceinline__ void cp_async16_zfill(uint32_t smem_addr, const void*
 __host__ __device__ __forceinline__ long long seg_floats(int dim, int vdim) {
   return static_cast<long long>(dim) * vdim + dim + 8;
 }
+// Gate values of all chunks: [chunk][head][a | running maximum of a | F][64]. A chunk's index is its distance from
+// the launch's first token in chunks plus the number of its item, which no two chunks share.
+__host__ __device__ __forceinline__ long long gate_floats(int tokens, int items, int heads) {
+  return static_cast<long long>(tokens / kChunk + items + 1) * heads * (3 * kChunk);
+}
+__device__ __forceinline__ float* chunk_gates(const nfk_mlstm_params& p, int item, int tok0, int c, int head) {
+  return p.scratch + (static_cast<long long>(tok0 / kChunk + item + c) * p.heads + head) * (3 * kChunk);
+}
+
+// a_j = i_j - F_j, its running maximum and F_j inside every chunk: one warp per (item, head, chunk), two tokens per
+// lane. Tokens past the item's last one get a = -inf.
+__global__ void __launch_bounds__(256)
+mlstm_gates_kernel(nfk_mlstm_params p) {
+  const int lane = threadIdx.x & 31;
+  const int head = blockIdx.x % p.heads, item = blockIdx.x / p.heads;
+  const int tok0 = p.items[item * 4 + 1], ntok = p.items[item * 4 + 2];
+  for (int c = threadIdx.x >> 5; c * kChunk < ntok; c += 8) {
+    float gi[2], gf[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = c * kChunk + lane * 2 + e;
+      gi[e] = -INFINITY;
+      gf[e] = 0.f;
+      if (t < ntok) gate_values(p, tok0 + t, head, gi[e], gf[e]);
+    }
+    float s = gf[0] + gf[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, s, o);
+      if (lane >= o) s += up;
+    }
+    const float F1 = s, F0 = s - gf[1];
+    const float a0 = gi[0] - F0, a1 = gi[1] - F1;
+    float mx = fmaxf(a0, a1);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, mx, o);
+      if (lane >= o) mx = fmaxf(mx, up);
+    }
+    const float before = __shfl_up_sync(0xffffffffu, mx, 1);
+    float2* dst = reinterpret_cast<float2*>(chunk_gates(p, item, tok0, c, head)) + lane;
+    dst[0] = make_float2(a0, a1);
+    dst[32] = make_float2(lane == 0 ? a0 : fmaxf(before, a0), mx);
+    dst[64] = make_float2(F0, F1);
+  }
+}
 
 // STATE_ONLY: the segment's own contribution to the state, from zero, into scratch. Otherwise: outputs, from the
 // request's state (first segment) or from scratch; the last segment leaves the state in the request's slot.
+// Tiles of q, k, v come by TMA (columns past a head's are filled with zeros; rows past the segment's last token
+// are other tokens' and get zero weights). Per chunk: scores and read-out of the old state by (32 tokens, 16 keys
+// or columns) per warp, outputs by (32 tokens, 16 columns), state update by 16-row tiles of S, which stays in
+// registers; its bf16 pair goes to shared memory for the next chunk's read-out.
 template <int DP, bool STATE_ONLY>
 __global__ void __launch_bounds__(kChThreads, 1)
-mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
+mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                   const __grid_constant__ CUtensorMap tmV, nfk_mlstm_params p, int v_slices, long long seg_off) {
   using C = ChCfg<DP>;
-  extern __shared__ __align__(128) uint8_t smem[];
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const uint32_t sb = smem_u32(smem);
-  float* n_s = reinterpret_cast<float*>(smem + C::F_OFF);
-  float* a_s = n_s + DP;              // a_j
+  float* n_s = reinterpret_cast<float*>(smem + C::F_OFF);   // [NPARTS][DP]: n is their sum
+  float* a_s = n_s + C::NPARTS * DP;  // a_j
   float* mx_s = a_s + kChunk;         // M_t
   float* int_s = mx_s + kChunk;       // e^(m_in - M_t)
   float* w_s = int_s + kChunk;        // e^(a_j - M_last)
   float* em_s = w_s + kChunk;         // e^(-m_t)
-  float* rs_s = em_s + kChunk;        // [2][64] row sums of the weighted scores
-  float* nq_s = rs_s + 2 * kChunk;    // n . q_t
-  float* sc_s = nq_s + kChunk;        // decay, m_out, F_last
+  float* rs_s = em_s + kChunk;        // [4][64] row sums of the weighted scores
+  float* nq_s = rs_s + 4 * kChunk;    // n . q_t
+  uint64_t* q_full = reinterpret_cast<uint64_t*>(smem + C::BAR_OFF);
+  uint64_t* kv_full = q_full + 1;     // two
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(q_full + 3);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int vs = blockIdx.x % v_slices;
@@ -267,36 +331,50 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
   const StateRef st = state_ref(p, req);
   if (!st.ok || ntok <= 0) return;
   const long long sh = static_cast<long long>(st.slot) * p.heads + head;
-  const __nv_bfloat16* qkv = reinterpret_cast<const __nv_bfloat16*>(p.qkv);
   const int v0 = vs * kVs;
-  float* sc_S = p.scratch + (static_cast<long long>(item) * p.heads + head) * seg_floats(p.dim, p.vdim);
+  float* sc_S = p.scratch + seg_off + (static_cast<long long>(item) * p.heads + head) * seg_floats(p.dim, p.vdim);
   float* sc_n = sc_S + static_cast<long long>(p.dim) * p.vdim;
   const int n_chunks = (ntok + kChunk - 1) / kChunk;
 
-  auto load_rows = [&](uint32_t dst, int c, int col0, int cols, int width, int row_bytes) {
-    // rows of chunk c, columns [col0, col0 + cols) of the head's block, zero past `cols` and past the last token
-    const int chs = width / 8;
-    for (int i = threadIdx.x; i < kChunk * chs; i += kChThreads) {
-      const int r = i / chs, ch = i % chs;
-      const int t = c * kChunk + r;
-      const bool ok = t < ntok && ch * 8 < cols;
-      cp_async16_zfill(dst + swz(r, ch, row_bytes),
-                       qkv + (ok ? static_cast<long long>(tok0 + t) * p.ld_qkv + col0 + ch * 8 : 0ll), ok);
-    }
-  };
-  auto load_kv = [&](int c) {
-    if (c < n_chunks) {
-      load_rows(sb + C::K_OFF + (c & 1) * C::QK_BYTES, c, p.k_off + head * p.dim, p.dim, DP, DP * 2);
-      load_rows(sb + C::V_OFF + (c & 1) * C::V_BYTES, c, p.v_off + head * p.vdim + v0, p.vdim - v0, kVs, kVs * 2);
-    }
-    cp_async_commit();
+  if (threadIdx.x == 0) {
+    mbar_init(q_full, 1);
+    mbar_init(kv_full, 1);
+    mbar_init(kv_full + 1, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  __syncthreads();
+  auto load_kv = [&](int c) {        // one thread
+    uint64_t* bar = kv_full + (c & 1);
+    mbar_expect_tx(bar, C::QK_BYTES + C::V_BYTES);
+#pragma unroll
+    for (int b = 0; b < DP / 64; ++b)
+      tma_load_3d(smem + C::K_OFF + (c & 1) * C::QK_BYTES + b * (kChunk * 128), &tmK, bar, b * 64, head, tok0 + c * kChunk);
+    tma_load_3d(smem + C::V_OFF + (c & 1) * C::V_BYTES, &tmV, bar, v0, head, tok0 + c * kChunk);
   };
   auto load_q = [&](int c) {
-    if (!STATE_ONLY && c < n_chunks) load_rows(sb + C::Q_OFF, c, p.q_off + head * p.dim, p.dim, DP, DP * 2);
-    cp_async_commit();
+    if (STATE_ONLY) return;
+    mbar_expect_tx(q_full, C::QK_BYTES);
+#pragma unroll
+    for (int b = 0; b < DP / 64; ++b)
+      tma_load_3d(smem + C::Q_OFF + b * (kChunk * 128), &tmQ, q_full, b * 64, head, tok0 + c * kChunk);
   };
-  load_kv(0);
-  load_q(0);
+  if (threadIdx.x == 0) {
+    load_kv(0);
+    load_q(0);
+  }
+  // gates of a chunk, fetched one chunk ahead: token threadIdx.x & 63, and the chunk's last maximum and sum
+  float ga, gm, gF, gm_last, gF_last;
+  auto fetch_gates = [&](int c) {
+    const float* g = chunk_gates(p, item, tok0, c < n_chunks ? c : n_chunks - 1, head);
+    const int t = threadIdx.x & 63;
+    ga = g[t];
+    gm = g[kChunk + t];
+    gF = g[2 * kChunk + t];
+    gm_last = g[2 * kChunk - 1];
+    gF_last = g[3 * kChunk - 1];
+  };
+  fetch_gates(0);
 
   // ---- incoming state ----
   const bool from_zero = STATE_ONLY || (seg == 0 && st.fresh);
@@ -311,12 +389,15 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
 #pragma unroll
     for (int b = 0; b < C::NTS; ++b)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + (e >> 1) * 8;
-        const int v = v0 + (wn * C::NTS + b) * 8 + (lane & 3) * 2 + (e & 1);
-        S[a][b][e] = (from_zero || d >= p.dim || v >= p.vdim) ? 0.f : S_in[static_cast<long long>(d) * p.vdim + v];
+      for (int h = 0; h < 2; ++h) {
+        const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
+        const int v = v0 + (wn * C::NTS + b) * 8 + (lane & 3) * 2;
+        float2 x = make_float2(0.f, 0.f);
+        if (!from_zero && d < p.dim && v < p.vdim) x = *reinterpret_cast<const float2*>(S_in + static_cast<long long>(d) * p.vdim + v);
+        S[a][b][2 * h] = x.x;
+        S[a][b][2 * h + 1] = x.y;
       }
-  for (int d = threadIdx.x; d < DP; d += kChThreads) n_s[d] = (from_zero || d >= p.dim) ? 0.f : n_in[d];
+  for (int i = threadIdx.x; i < C::NPARTS * DP; i += kChThreads) n_s[i] = (from_zero || i >= p.dim) ? 0.f : n_in[i];
   auto publish_state = [&]() {      // the state's bf16 pair, B operand of the next chunk's read-out
 #pragma unroll
     for (int a = 0; a < C::MTS; ++a)
@@ -325,7 +406,7 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
           const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
-          const uint32_t off = swz(d, wn * C::NTS + b, kVs * 2) + (lane & 3) * 4;
+          const uint32_t off = swz(d, wn * C::NTS + b) + (lane & 3) * 4;
           const uint32_t hi = pack_bf16x2(S[a][b][2 * h], S[a][b][2 * h + 1]);
           const float2 hf = unpack_bf16x2(hi);
           *reinterpret_cast<uint32_t*>(smem + C::SH_OFF + off) = hi;
@@ -334,68 +415,35 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
   };
   if (!STATE_ONLY) publish_state();
 
-  // gates of a chunk: two tokens per lane of warp 0, fetched one chunk ahead
-  float gi[2] = {-INFINITY, -INFINITY}, gf[2] = {0.f, 0.f};
-  auto load_gates = [&](int c) {
-    if (warp != 0) return;
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int t = c * kChunk + lane * 2 + e;
-      gi[e] = -INFINITY;
-      gf[e] = 0.f;
-      if (c < n_chunks && t < ntok) gate_values(p, tok0 + t, head, gi[e], gf[e]);
-    }
-  };
-  load_gates(0);
-
+  const int th = warp & 1, cq = warp >> 1;              // 32 tokens, 16 keys / columns
+  const int mm = lane >> 3, rr = lane & 7;
   for (int c = 0; c < n_chunks; ++c) {
-    if (warp == 0) {
-      // prefix sums of f, prefix maxima of a = i - F
-      float s = gf[0] + gf[1];
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, s, o);
-        if (lane >= o) s += up;
-      }
-      const float F1 = s, F0 = s - gf[1];
-      const float a0 = gi[0] - F0, a1 = gi[1] - F1;
-      float mx = fmaxf(a0, a1);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, mx, o);
-        if (lane >= o) mx = fmaxf(mx, up);
-      }
-      float before = __shfl_up_sync(0xffffffffu, mx, 1);
-      if (lane == 0) before = -INFINITY;
-      const float M1 = fmaxf(m_in, mx), M0 = fmaxf(m_in, fmaxf(before, a0));
-      const float M_last = __shfl_sync(0xffffffffu, M1, 31), F_last = __shfl_sync(0xffffffffu, F1, 31);
-      const int t = lane * 2;
-      a_s[t] = a0; a_s[t + 1] = a1;
-      mx_s[t] = M0; mx_s[t + 1] = M1;
-      int_s[t] = expf(m_in - M0); int_s[t + 1] = expf(m_in - M1);
-      w_s[t] = expf(a0 - M_last); w_s[t + 1] = expf(a1 - M_last);
-      em_s[t] = expf(-(F0 + M0)); em_s[t + 1] = expf(-(F1 + M1));
-      if (lane == 0) {
-        sc_s[0] = expf(m_in - M_last);
-        sc_s[1] = F_last + M_last;
-        sc_s[2] = F_last;
-      }
+    const float M_last = fmaxf(m_in, gm_last);
+    const float decay = expf(m_in - M_last);
+    if (threadIdx.x < kChunk) {
+      const float M = fmaxf(m_in, gm);
+      a_s[threadIdx.x] = ga;
+      mx_s[threadIdx.x] = M;
+      int_s[threadIdx.x] = expf(m_in - M);
+      w_s[threadIdx.x] = expf(ga - M_last);
+      em_s[threadIdx.x] = expf(-(gF + M));
     }
-    cp_async_wait<0>();
-    __syncthreads();                 // chunk c's rows, gates and the state's bf16 pair are in shared memory
-    load_kv(c + 1);
-    load_gates(c + 1);
-    const float decay = sc_s[0];
-    m_in = sc_s[1];
-    F_total += sc_s[2];
+    m_in = gF_last + M_last;
+    F_total += gF_last;
+    // a wait that runs out is reported; the warps go on in step, so that they meet at their barriers
+    if (*abort_flag == 0 && (!mbar_wait(kv_full + (c & 1), (c >> 1) & 1) || (!STATE_ONLY && !mbar_wait(q_full, c & 1)))) {
+      if (lane == 0) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
+      *abort_flag = 1;
+    }
+    __syncthreads();                 // chunk c's gates and the state's bf16 pair are in shared memory
+    if (threadIdx.x == 0 && c + 1 < n_chunks) load_kv(c + 1);
+    fetch_gates(c + 1);
     const uint32_t kb = sb + C::K_OFF + (c & 1) * C::QK_BYTES;
     const uint32_t vb = sb + C::V_OFF + (c & 1) * C::V_BYTES;
-    const int mt = warp & 3, half = warp >> 2;          // 16 tokens, 32 keys / columns
-    const int mm = lane >> 3, rr = lane & 7;
     // ---- values weighted by e^(a_j - M_last), as a bf16 pair ----
     for (int i = threadIdx.x; i < kChunk * kVs / 8; i += kChThreads) {
       const int r = i / (kVs / 8), ch = i % (kVs / 8);
-      const uint32_t off = swz(r, ch, kVs * 2);
+      const uint32_t off = swz(r, ch);
       const uint4 v = *reinterpret_cast<const uint4*>(smem + C::V_OFF + (c & 1) * C::V_BYTES + off);
       const uint32_t vw[4] = {v.x, v.y, v.z, v.w};
       const float w = w_s[r];
@@ -412,7 +460,7 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
       *reinterpret_cast<uint4*>(smem + C::WH_OFF + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
       *reinterpret_cast<uint4*>(smem + C::WL_OFF + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
-    float qs[4][4];
+    float qs[2][2][4];
     if (!STATE_ONLY) {
       // ---- n . q ----
       {
@@ -420,9 +468,15 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
         float d = 0.f;
 #pragma unroll 2
         for (int ch = part; ch < DP / 8; ch += 4) {
-          const uint4 q = *reinterpret_cast<const uint4*>(smem + C::Q_OFF + swz(t, ch, DP * 2));
+          const uint4 q = *reinterpret_cast<const uint4*>(smem + C::Q_OFF + swz_blk(t, ch));
           const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
-          const float4 n0 = *reinterpret_cast<const float4*>(n_s + ch * 8), n1 = *reinterpret_cast<const float4*>(n_s + ch * 8 + 4);
+          float4 n0 = *reinterpret_cast<const float4*>(n_s + ch * 8), n1 = *reinterpret_cast<const float4*>(n_s + ch * 8 + 4);
+#pragma unroll
+          for (int k = 1; k < C::NPARTS; ++k) {
+            const float4 x0 = *reinterpret_cast<const float4*>(n_s + k * DP + ch * 8), x1 = *reinterpret_cast<const float4*>(n_s + k * DP + ch * 8 + 4);
+            n0.x += x0.x; n0.y += x0.y; n0.z += x0.z; n0.w += x0.w;
+            n1.x += x1.x; n1.y += x1.y; n1.z += x1.z; n1.w += x1.w;
+          }
           const float nn[8] = {n0.x, n0.y, n0.z, n0.w, n1.x, n1.y, n1.z, n1.w};
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
@@ -433,102 +487,117 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
         d = quad_sum(d);
         if (part == 0) nq_s[t] = d;
       }
-      // ---- scores Q K^T and read-out Q S of this warp's 16 tokens ----
-      float sc[4][4];
+      // ---- scores Q K^T (16 keys) and read-out Q S (16 columns) of this warp's 32 tokens ----
+      float sc[2][2][4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
+      for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[j][e] = qs[j][e] = 0.f;
-      const bool keys_seen = half * 32 <= mt * 16 + 15;       // some of this half's keys are not in the future
-#pragma unroll 2
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sc[i][j][e] = qs[i][j][e] = 0.f;
+      const bool keys_seen = cq * 16 <= th * 32 + 31;          // some of these keys are not in the future
+#pragma unroll 4
       for (int ks = 0; ks < DP / 16; ++ks) {
-        uint32_t a[4], b0, b1, b2, b3;
-        ldsm_x4(sb + C::Q_OFF + swz(mt * 16 + (lane & 15), 2 * ks + (lane >> 4), DP * 2), a[0], a[1], a[2], a[3]);
-        if (keys_seen) {
+        uint32_t a[2][4], b0, b1, b2, b3, h0, h1, h2, h3, l0, l1, l2, l3;
 #pragma unroll
-          for (int g = 0; g < 2; ++g) {
-            ldsm_x4(kb + swz(half * 32 + g * 16 + (mm >> 1) * 8 + rr, 2 * ks + (mm & 1), DP * 2), b0, b1, b2, b3);
-            mma_bf16(sc[2 * g], a, b0, b1);
-            mma_bf16(sc[2 * g + 1], a, b2, b3);
+        for (int i = 0; i < 2; ++i)
+          ldsm_x4(sb + C::Q_OFF + swz_blk(th * 32 + i * 16 + (lane & 15), 2 * ks + (lane >> 4)), a[i][0], a[i][1], a[i][2], a[i][3]);
+        const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, cq * 2 + (mm >> 1));
+        ldsm_x4_trans(sb + C::SH_OFF + off, h0, h1, h2, h3);
+        ldsm_x4_trans(sb + C::SL_OFF + off, l0, l1, l2, l3);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          mma_bf16(qs[i][0], a[i], h0, h1);
+          mma_bf16(qs[i][1], a[i], h2, h3);
+        }
+        if (keys_seen) {
+          ldsm_x4(kb + swz_blk(cq * 16 + (mm >> 1) * 8 + rr, 2 * ks + (mm & 1)), b0, b1, b2, b3);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            mma_bf16(sc[i][0], a[i], b0, b1);
+            mma_bf16(sc[i][1], a[i], b2, b3);
           }
         }
 #pragma unroll
-        for (int hl = 0; hl < 2; ++hl)        // high parts of all columns, then low parts
-#pragma unroll
-          for (int g = 0; g < 2; ++g) {
-            const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, half * 4 + 2 * g + (mm >> 1), kVs * 2);
-            ldsm_x4_trans(sb + (hl == 0 ? C::SH_OFF : C::SL_OFF) + off, b0, b1, b2, b3);
-            mma_bf16(qs[2 * g], a, b0, b1);
-            mma_bf16(qs[2 * g + 1], a, b2, b3);
-          }
+        for (int i = 0; i < 2; ++i) {
+          mma_bf16(qs[i][0], a[i], l0, l1);
+          mma_bf16(qs[i][1], a[i], l2, l3);
+        }
       }
       // ---- weights, row sums, bf16 pair of the weighted scores ----
-      const int r0 = mt * 16 + (lane >> 2), r1 = r0 + 8;
-      const float M0 = mx_s[r0], M1 = mx_s[r1];
-      float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int col = half * 32 + j * 8 + (lane & 3) * 2;
-        const float ac0 = a_s[col], ac1 = a_s[col + 1];
-        const float x0 = col <= r0 ? sc[j][0] * p.q_scale * expf(ac0 - M0) : 0.f;
-        const float x1 = col + 1 <= r0 ? sc[j][1] * p.q_scale * expf(ac1 - M0) : 0.f;
-        const float y0 = col <= r1 ? sc[j][2] * p.q_scale * expf(ac0 - M1) : 0.f;
-        const float y1 = col + 1 <= r1 ? sc[j][3] * p.q_scale * expf(ac1 - M1) : 0.f;
-        sum0 += x0 + x1;
-        sum1 += y0 + y1;
-        const uint32_t h0 = pack_bf16x2(x0, x1), h1 = pack_bf16x2(y0, y1);
-        const float2 f0 = unpack_bf16x2(h0), f1 = unpack_bf16x2(h1);
-        const uint32_t o0 = swz(r0, half * 4 + j, kChunk * 2) + (lane & 3) * 4;
-        const uint32_t o1 = swz(r1, half * 4 + j, kChunk * 2) + (lane & 3) * 4;
-        *reinterpret_cast<uint32_t*>(smem + C::PH_OFF + o0) = h0;
-        *reinterpret_cast<uint32_t*>(smem + C::PH_OFF + o1) = h1;
-        *reinterpret_cast<uint32_t*>(smem + C::PL_OFF + o0) = pack_bf16x2(x0 - f0.x, x1 - f0.y);
-        *reinterpret_cast<uint32_t*>(smem + C::PL_OFF + o1) = pack_bf16x2(y0 - f1.x, y1 - f1.y);
-      }
-      sum0 = quad_sum(sum0);
-      sum1 = quad_sum(sum1);
-      if ((lane & 3) == 0) {
-        rs_s[half * kChunk + r0] = sum0;
-        rs_s[half * kChunk + r1] = sum1;
-      }
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int r = th * 32 + i * 16 + h * 8 + (lane >> 2);
+          const float M = mx_s[r];
+          float sum = 0.f;
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            const int col = cq * 16 + j * 8 + (lane & 3) * 2;
+            const float2 ac = *reinterpret_cast<const float2*>(a_s + col);
+            const float x0 = col <= r ? sc[i][j][2 * h] * p.q_scale * expf(ac.x - M) : 0.f;
+            const float x1 = col + 1 <= r ? sc[i][j][2 * h + 1] * p.q_scale * expf(ac.y - M) : 0.f;
+            sum += x0 + x1;
+            const uint32_t hi = pack_bf16x2(x0, x1);
+            const float2 hf = unpack_bf16x2(hi);
+            const uint32_t o = swz(r, cq * 2 + j) + (lane & 3) * 4;
+            *reinterpret_cast<uint32_t*>(smem + C::PH_OFF + o) = hi;
+            *reinterpret_cast<uint32_t*>(smem + C::PL_OFF + o) = pack_bf16x2(x0 - hf.x, x1 - hf.y);
+          }
+          sum = quad_sum(sum);
+          if ((lane & 3) == 0) rs_s[cq * kChunk + r] = sum;
+        }
     }
     __syncthreads();                 // weighted scores and values are in shared memory; Q and the old state are free
-    load_q(c + 1);
+    if (threadIdx.x == 0 && c + 1 < n_chunks) load_q(c + 1);
     if (!STATE_ONLY) {
-      // ---- P V, then the outputs of these 16 tokens x 32 columns ----
-      float pv[4][4];
+      // ---- P V, then the outputs of these 32 tokens x 16 columns ----
+      float pv[2][2][4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) pv[j][0] = pv[j][1] = pv[j][2] = pv[j][3] = 0.f;
-      for (int ks = 0; ks <= mt; ++ks) {
-        uint32_t ph[4], pl[4], b0, b1, b2, b3;
-        const uint32_t ao = swz(mt * 16 + (lane & 15), 2 * ks + (lane >> 4), kChunk * 2);
-        ldsm_x4(sb + C::PH_OFF + ao, ph[0], ph[1], ph[2], ph[3]);
-        ldsm_x4(sb + C::PL_OFF + ao, pl[0], pl[1], pl[2], pl[3]);
+      for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int g = 0; g < 2; ++g) {
-          ldsm_x4_trans(vb + swz(ks * 16 + (mm & 1) * 8 + rr, half * 4 + 2 * g + (mm >> 1), kVs * 2), b0, b1, b2, b3);
-          mma_bf16(pv[2 * g], ph, b0, b1);
-          mma_bf16(pv[2 * g], pl, b0, b1);
-          mma_bf16(pv[2 * g + 1], ph, b2, b3);
-          mma_bf16(pv[2 * g + 1], pl, b2, b3);
+        for (int j = 0; j < 2; ++j) pv[i][j][0] = pv[i][j][1] = pv[i][j][2] = pv[i][j][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks) {
+        if (ks * 16 > th * 32 + 31) continue;
+        uint32_t ph[2][4], pl[2][4], b0, b1, b2, b3;
+        ldsm_x4_trans(vb + swz(ks * 16 + (mm & 1) * 8 + rr, cq * 2 + (mm >> 1)), b0, b1, b2, b3);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const uint32_t ao = swz(th * 32 + i * 16 + (lane & 15), 2 * ks + (lane >> 4));
+          ldsm_x4(sb + C::PH_OFF + ao, ph[i][0], ph[i][1], ph[i][2], ph[i][3]);
+          ldsm_x4(sb + C::PL_OFF + ao, pl[i][0], pl[i][1], pl[i][2], pl[i][3]);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          mma_bf16(pv[i][0], ph[i], b0, b1);
+          mma_bf16(pv[i][1], ph[i], b2, b3);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          mma_bf16(pv[i][0], pl[i], b0, b1);
+          mma_bf16(pv[i][1], pl[i], b2, b3);
         }
       }
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int r = mt * 16 + (lane >> 2) + h * 8, t = c * kChunk + r;
-        if (t >= ntok) continue;
-        const float inter = int_s[r] * p.q_scale;
-        const float den = rs_s[r] + rs_s[kChunk + r] + inter * nq_s[r];
-        const float inv = 1.f / (fmaxf(fabsf(den), em_s[r]) + 1e-6f);
-        float* dst = p.out + static_cast<long long>(tok0 + t) * p.ld_out + head * p.vdim;
+      for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const int v = v0 + half * 32 + j * 8 + (lane & 3) * 2;
-          if (v < p.vdim)
-            *reinterpret_cast<float2*>(dst + v) = make_float2((inter * qs[j][2 * h] + pv[j][2 * h]) * inv,
-                                                              (inter * qs[j][2 * h + 1] + pv[j][2 * h + 1]) * inv);
+        for (int h = 0; h < 2; ++h) {
+          const int r = th * 32 + i * 16 + h * 8 + (lane >> 2), t = c * kChunk + r;
+          if (t >= ntok) continue;
+          const float inter = int_s[r] * p.q_scale;
+          const float den = (rs_s[r] + rs_s[kChunk + r]) + (rs_s[2 * kChunk + r] + rs_s[3 * kChunk + r]) + inter * nq_s[r];
+          const float inv = 1.f / (fmaxf(fabsf(den), em_s[r]) + 1e-6f);
+          float* dst = p.out + static_cast<long long>(tok0 + t) * p.ld_out + head * p.vdim;
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            const int v = v0 + cq * 16 + j * 8 + (lane & 3) * 2;
+            if (v < p.vdim)
+              *reinterpret_cast<float2*>(dst + v) = make_float2((inter * qs[i][j][2 * h] + pv[i][j][2 * h]) * inv,
+                                                                (inter * qs[i][j][2 * h + 1] + pv[i][j][2 * h + 1]) * inv);
+          }
         }
-      }
     }
     // ---- state update: S = decay S + K^T (w V), n = decay n + K^T w ----
 #pragma unroll
@@ -542,11 +611,11 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
       uint32_t ak[C::MTS][4];
 #pragma unroll
       for (int a = 0; a < C::MTS; ++a)
-        ldsm_x4_trans(kb + swz(ks * 16 + (mm >> 1) * 8 + rr, (wm * C::MTS + a) * 2 + (mm & 1), DP * 2), ak[a][0], ak[a][1],
+        ldsm_x4_trans(kb + swz_blk(ks * 16 + (mm >> 1) * 8 + rr, (wm * C::MTS + a) * 2 + (mm & 1)), ak[a][0], ak[a][1],
                       ak[a][2], ak[a][3]);
 #pragma unroll
       for (int b = 0; b < C::NTS; b += 2) {
-        const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, wn * C::NTS + b + (mm >> 1), kVs * 2);
+        const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, wn * C::NTS + b + (mm >> 1));
         uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
         ldsm_x4_trans(sb + C::WH_OFF + off, h0, h1, h2, h3);
         ldsm_x4_trans(sb + C::WL_OFF + off, l0, l1, l2, l3);
@@ -562,19 +631,37 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
         }
       }
     }
-    if (threadIdx.x < DP) {
-      const int d = threadIdx.x;
-      float n = decay * n_s[d];
-      const uint8_t* kp = smem + C::K_OFF + (c & 1) * C::QK_BYTES + (d & 7) * 2;
-#pragma unroll 8
-      for (int j = 0; j < kChunk; ++j)
-        n += w_s[j] * __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(kp + swz(j, d >> 3, DP * 2)));
-      n_s[d] = n;
+    {
+      // two columns and kChunk / NPARTS tokens per thread; each part of n is a sum of its own
+      constexpr int TOKS = kChunk / C::NPARTS;
+      const int dp = threadIdx.x % (DP / 2), part = threadIdx.x / (DP / 2);
+      float2* np = reinterpret_cast<float2*>(n_s + part * DP) + dp;
+      float2 n = *np;
+      n.x *= decay;
+      n.y *= decay;
+      const uint8_t* kp = smem + C::K_OFF + (c & 1) * C::QK_BYTES + (dp & 3) * 4;
+#pragma unroll
+      for (int j4 = 0; j4 < TOKS; j4 += 4) {
+        const int j0 = part * TOKS + j4;
+        const float4 w = *reinterpret_cast<const float4*>(w_s + j0);
+        const float ww[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(kp + swz_blk(j0 + j, dp >> 2)));
+          n.x += ww[j] * k.x;
+          n.y += ww[j] * k.y;
+        }
+      }
+      *np = n;
     }
     if (!STATE_ONLY && c + 1 < n_chunks) publish_state();
     __syncthreads();                 // gate arrays and n are free for the next chunk
   }
-  cp_async_wait<0>();
+  if (*abort_flag != 0 && threadIdx.x == 0) {
+    // a wait ran out: give copies still in flight a bounded chance to land before the CTA ends
+    for (int c = n_chunks > 1 ? n_chunks - 2 : 0; c < n_chunks; ++c) (void)mbar_wait(kv_full + (c & 1), (c >> 1) & 1);
+    if (!STATE_ONLY) (void)mbar_wait(q_full, (n_chunks - 1) & 1);
+  }
 
   // ---- state out ----
   if (!STATE_ONLY && has_next) return;
@@ -592,7 +679,12 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
           *reinterpret_cast<float2*>(S_out + static_cast<long long>(d) * p.vdim + v) = make_float2(S[a][b][2 * h], S[a][b][2 * h + 1]);
       }
   if (vs == 0) {
-    for (int d = threadIdx.x; d < p.dim; d += kChThreads) n_out[d] = n_s[d];
+    for (int d = threadIdx.x; d < p.dim; d += kChThreads) {
+      float n = n_s[d];
+#pragma unroll
+      for (int k = 1; k < C::NPARTS; ++k) n += n_s[k * DP + d];
+      n_out[d] = n;
+    }
     if (threadIdx.x == 0) {
       if (STATE_ONLY) {
         sc_n[p.dim] = m_in;
@@ -607,7 +699,7 @@ mlstm_chunk_kernel(nfk_mlstm_params p, int v_slices) {
 // Segment contributions -> incoming states, in place, for requests with more than one segment. One thread per
 // four elements of (S, n) of a head; all threads follow the same m.
 __global__ void __launch_bounds__(256)
-mlstm_scan_kernel(nfk_mlstm_params p, int e_blocks) {
+mlstm_scan_kernel(nfk_mlstm_params p, int e_blocks, long long seg_off) {
   const int eb = blockIdx.x % e_blocks;
   const int head = (blockIdx.x / e_blocks) % p.heads;
   const int item0 = blockIdx.x / (e_blocks * p.heads);
@@ -627,7 +719,7 @@ mlstm_scan_kernel(nfk_mlstm_params p, int e_blocks) {
     if (in) R = e < ns ? load4(p.S + sh * ns + e) : load4(p.n + (sh * 2 + st.half) * p.dim + (e - ns));
   }
   for (int it = item0; it < p.num_items && p.items[it * 4] == req; ++it) {
-    float* sc = p.scratch + (static_cast<long long>(it) * p.heads + head) * seg_floats(p.dim, p.vdim);
+    float* sc = p.scratch + seg_off + (static_cast<long long>(it) * p.heads + head) * seg_floats(p.dim, p.vdim);
     const bool last = it + 1 >= p.num_items || p.items[(it + 1) * 4] != req;
     float m_loc = 0.f, F = 0.f;
     float4 L = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -704,6 +796,20 @@ int set_smem(K kernel, size_t bytes) {
   return NF_OK;
 }
 
+// [num_tokens][heads][cols] view of a column block of qkv; box: 64 tokens of one head, 64 columns.
+int head_tmap(CUtensorMap* out, const nfk_mlstm_params& p, int col0, int cols) {
+  nf_encode_tiled_fn enc = get_encode_tiled();
+  if (enc == nullptr) return NF_ERR_CUDA;
+  cuuint64_t dim[3] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(p.heads), static_cast<cuuint64_t>(p.num_tokens)};
+  cuuint64_t stride[2] = {static_cast<cuuint64_t>(cols) * 2, static_cast<cuuint64_t>(p.ld_qkv) * 2};
+  cuuint32_t box[3] = {64, 1, kChunk}, estr[3] = {1, 1, 1};
+  const __nv_bfloat16* base = reinterpret_cast<const __nv_bfloat16*>(p.qkv) + col0;
+  return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<__nv_bfloat16*>(base), dim, stride, box, estr,
+             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS
+             ? NF_OK : NF_ERR_CUDA;
+}
+
 template <int DP>
 int launch_chunk(const nfk_mlstm_params& p, cudaStream_t stream) {
   using C = ChCfg<DP>;
@@ -715,16 +821,24 @@ int launch_chunk(const nfk_mlstm_params& p, cudaStream_t stream) {
     if (rc != NF_OK) return rc;
     attr = true;
   }
+  CUtensorMap tq, tk, tv;
+  int rc = head_tmap(&tq, p, p.q_off, p.dim);
+  if (rc == NF_OK) rc = head_tmap(&tk, p, p.k_off, p.dim);
+  if (rc == NF_OK) rc = head_tmap(&tv, p, p.v_off, p.vdim);
+  if (rc != NF_OK) return rc;
   const int v_slices = (p.vdim + kVs - 1) / kVs;
   const int grid = p.num_items * p.heads * v_slices;
+  const long long seg_off = gate_floats(p.num_tokens, p.num_items, p.heads);
+  mlstm_gates_kernel<<<p.num_items * p.heads, 256, 0, stream>>>(p);
+  if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
   if (p.num_items > p.req_count) {       // some request has several segments
-    mlstm_chunk_kernel<DP, true><<<grid, kChThreads, C::SMEM, stream>>>(p, v_slices);
+    mlstm_chunk_kernel<DP, true><<<grid, kChThreads, C::SMEM, stream>>>(tq, tk, tv, p, v_slices, seg_off);
     if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
     const int e_blocks = (p.dim * p.vdim + p.dim + 1023) / 1024;
-    mlstm_scan_kernel<<<p.num_items * p.heads * e_blocks, 256, 0, stream>>>(p, e_blocks);
+    mlstm_scan_kernel<<<p.num_items * p.heads * e_blocks, 256, 0, stream>>>(p, e_blocks, seg_off);
     if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
   }
-  mlstm_chunk_kernel<DP, false><<<grid, kChThreads, C::SMEM, stream>>>(p, v_slices);
+  mlstm_chunk_kernel<DP, false><<<grid, kChThreads, C::SMEM, stream>>>(tq, tk, tv, p, v_slices, seg_off);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 
@@ -750,10 +864,12 @@ extern "C" int nfk_mlstm_prefill(const nfk_mlstm_params* p, cudaStream_t stream)
   int rc = check_mlstm(p);
   if (rc != NF_OK) return rc;
   if (p->req_count == 0) return NF_OK;
-  const bool chunk_ok = p->dtype == NFK_BF16 && p->dim <= 256 && p->items != nullptr && p->num_items >= p->req_count &&
-                        (reinterpret_cast<uintptr_t>(p->qkv) & 15) == 0 &&
-                        (p->num_items == p->req_count ||
-                         (p->scratch != nullptr && p->num_items * p->heads * seg_floats(p->dim, p->vdim) <= p->scratch_floats));
+  const bool chunk_ok =
+      p->dtype == NFK_BF16 && p->dim <= 256 && p->items != nullptr && p->num_items >= p->req_count && p->num_tokens > 0 &&
+      (reinterpret_cast<uintptr_t>(p->qkv) & 15) == 0 && p->scratch != nullptr &&
+      (reinterpret_cast<uintptr_t>(p->scratch) & 15) == 0 &&
+      gate_floats(p->num_tokens, p->num_items, p->heads) +
+              (p->num_items > p->req_count ? p->num_items * p->heads * seg_floats(p->dim, p->vdim) : 0ll) <= p->scratch_floats;
   if (p->impl == 2 && !chunk_ok) return NF_ERR_UNSUPPORTED;
   if (p->impl != 1 && chunk_ok) {
     if (p->dim <= 64) return launch_chunk<64>(*p, stream);

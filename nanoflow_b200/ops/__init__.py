@@ -119,7 +119,7 @@ class MlstmParams(Structure):
                 ("positions", c_void_p), ("qo_indptr", c_void_p), ("state_slot", c_void_p),
                 ("req_begin", c_int), ("req_count", c_int), ("heads", c_int), ("dim", c_int), ("vdim", c_int),
                 ("num_slots", c_int), ("gate_cap", c_float), ("q_scale", c_float), ("dtype", c_int), ("impl", c_int),
-                ("items", c_void_p), ("num_items", c_int), ("scratch", c_void_p), ("scratch_floats", c_longlong),
+                ("items", c_void_p), ("num_items", c_int), ("num_tokens", c_int), ("scratch", c_void_p), ("scratch_floats", c_longlong),
                 ("status", c_void_p)]
 
 

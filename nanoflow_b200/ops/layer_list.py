@@ -132,13 +132,15 @@ def mlstm(qkv, gates, i_bias, f_bias, state, out, positions, qo_indptr, state_re
                     req_begin=req_begin, req_count=qo_indptr.numel() - 1 if req_count is None else req_count, heads=heads,
                     dim=dim, vdim=vdim, num_slots=S.shape[0], gate_cap=gate_cap, q_scale=q_scale,
                     dtype=dtype_code(qkv.dtype), impl=impl, items=_p(items), num_items=0 if items is None else items.shape[0],
+                    num_tokens=qkv.shape[0],
                     scratch=_p(scratch), scratch_floats=0 if scratch is None else scratch.numel(), status=_p(status))
     name = "nfk_mlstm_decode" if decode else "nfk_mlstm_prefill"
     _check(getattr(lib(), name)(byref(p), _stream()), name)
 
 
-def mlstm_scratch_floats(items: int, heads: int, dim: int, vdim: int) -> int:
-    return items * heads * (dim * vdim + dim + 8)
+def mlstm_scratch_floats(items: int, heads: int, dim: int, vdim: int, tokens: int, segmented: bool = True) -> int:
+    gates = (tokens // 64 + items + 1) * heads * 192
+    return gates + (items * heads * (dim * vdim + dim + 8) if segmented else 0)
 
 
 def head_norm_gate(o, g, w, out, *, heads: int, vdim: int, eps: float) -> None:

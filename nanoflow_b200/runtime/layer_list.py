@@ -28,6 +28,7 @@ import torch
 from .. import ops
 from ..models.layer_list import PREFILL_HEAD_DIM, LayerListConfig, NormWeights, round8
 from ..ops import ACTS, NORMS, dtype_code
+from ..ops.layer_list import mlstm_scratch_floats
 from ..serving.scheduler import BatchPlan
 from .engine import GEMM_WS_BYTES, Engine, MetaLayout
 from .graph import (ArgmaxParams, AttnParams, GemmParams, HeadNormGateParams, KvMoveParams, LatentAppendParams,
@@ -172,8 +173,9 @@ class LayerListEngine(Engine):
         self.arange = torch.arange(self.x_pages + 1, dtype=torch.int32, device=dev)
         heads = max([s.heads * (m.latent_ld(s) + 2) for s in m.run_specs("latent_attention")], default=0)
         self.latent_ws = torch.empty(max(8, 160 * heads), dtype=f32, device=dev)
-        seg = max([s.heads * (round8(s.dim) * round8(s.vdim) + round8(s.dim) + 8) for s in m.run_specs("mlstm")], default=0)
-        self.seg_ws = torch.empty(max(8, SEGMENT_ITEMS * seg if dt == torch.bfloat16 else 8), dtype=f32, device=dev)
+        seg = max([mlstm_scratch_floats(SEGMENT_ITEMS, s.heads, round8(s.dim), round8(s.vdim), T) +
+                   mlstm_scratch_floats(self.B, s.heads, 8, 8, T, False) for s in m.run_specs("mlstm")], default=0)
+        self.seg_ws = torch.empty(max(8, seg if dt == torch.bfloat16 else 8), dtype=f32, device=dev)
         self.gemm_ws = torch.zeros(GEMM_WS_BYTES // 4, dtype=f32, device=dev) if dt == torch.bfloat16 else None
         self.taps = P(len(m.runs) * T, m.width_p, f32, "taps").view(len(m.runs), T, m.width_p) \
             if self.eng.tap_residual else None
@@ -358,12 +360,13 @@ class LayerListEngine(Engine):
                 out=_ptr(o_rec), ld_out=o_rec.stride(0), positions=_ptr(meta["positions"]),
                 qo_indptr=_ptr(meta["qo_indptr"]), state_slot=_ptr(meta["state_ref"]), req_begin=0, req_count=0, heads=H,
                 dim=d, vdim=v, num_slots=self.num_slots, gate_cap=s.gate_cap, q_scale=s.dim ** -0.5, dtype=self.code,
-                impl=0, items=_ptr(meta["segs"]), num_items=0, scratch=_ptr(self.seg_ws),
+                impl=0, items=_ptr(meta["segs"]), num_items=0, num_tokens=0, scratch=_ptr(self.seg_ws),
                 scratch_floats=self.seg_ws.numel(), status=_ptr(self.bufs.status))
 
         self._op(f"R{r}.mlstm_decode", params(), kernel="nfk_mlstm_decode", dyn=[("req_count", "n_dec")], layer=r)
         self._op(f"R{r}.mlstm_prefill", params(), kernel="nfk_mlstm_prefill",
-                 dyn=[("req_begin", "n_dec"), ("req_count", "n_pre"), ("num_items", self.g.symbol("n_segs"))], layer=r)
+                 dyn=[("req_begin", "n_dec"), ("req_count", "n_pre"), ("num_items", self.g.symbol("n_segs")),
+                      ("num_tokens", T)], layer=r)
         g_cols = c_void_p(proj.data_ptr() + (2 * H * d + H * v) * proj.element_size())
         hp = HeadNormGateParams(o=_ptr(o_rec), ld_o=o_rec.stride(0), g=g_cols, ld_g=proj.stride(0), w=_ptr(lw.norm),
                                 out=_ptr(attn), ld_out=attn.stride(0), T=0, heads=H, vdim=s.vdim, vdim_p=v, eps=m.norm_eps,

@@ -361,7 +361,7 @@ class MlstmCase:
         qo = np.concatenate([[0], np.cumsum([parts[b] for b in reqs])]).astype(np.int32)
         pos = np.concatenate([np.arange(self.at[b], self.at[b] + parts[b]) for b in reqs])
         items = mlstm_segments(qo, 0, seg_ctas, 148)
-        scratch = torch.zeros(K.mlstm_scratch_floats(len(items), self.H, self.d, self.v), device="cuda")
+        scratch = torch.zeros(K.mlstm_scratch_floats(len(items), self.H, self.d, self.v, len(rows)), device="cuda")
         out = torch.zeros(len(rows), self.H * self.v, device="cuda")
         st = ops.new_status()
         K.mlstm(qkv, self.gates[idx].contiguous(), self.i_b, self.f_b, self.state, out, i32(pos), i32(qo),
