@@ -217,9 +217,11 @@ struct ChCfg {
   static constexpr int PL_OFF = PH_OFF + P_BYTES;
   static constexpr int WH_OFF = PL_OFF + P_BYTES;         // weighted values, high / low part
   static constexpr int WL_OFF = WH_OFF + V_BYTES;
-  static constexpr int F_OFF = WL_OFF + V_BYTES;          // fp32 arrays
-  static constexpr int NPARTS = 2 * kChThreads / DP;      // partial sums that n is kept in
-  static constexpr int N_F32 = NPARTS * DP + 10 * kChunk;
+  static constexpr int N_OFF = WL_OFF + V_BYTES;          // n as a ninth column tile of the state, [DP][8]: columns
+                                                          // 0-2 are three bf16 parts that add up to it
+  static constexpr int U_OFF = N_OFF + DP * 16;           // its weighted values: the weights in three parts, [64][8]
+  static constexpr int F_OFF = U_OFF + kChunk * 16;       // fp32 arrays
+  static constexpr int N_F32 = 13 * kChunk;
   static constexpr int BAR_OFF = F_OFF + N_F32 * 4;
   static constexpr int SMEM = BAR_OFF + 64 + 1024;
   static constexpr int WM = DP / 16 < 8 ? DP / 16 : 8;    // warps along dim in the state update
@@ -234,6 +236,19 @@ __device__ __forceinline__ uint32_t swz(int row, int ch) {
 }
 __device__ __forceinline__ uint32_t swz_blk(int row, int ch) {
   return static_cast<uint32_t>((ch >> 3) * (kChunk * 128) + row * 128 + (((ch ^ row) & 7) << 4));
+}
+__device__ __forceinline__ void ldsm_x2_trans(uint32_t addr, uint32_t& r0, uint32_t& r1) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
+}
+// Three bf16 values that add up to v, in the first three places of a row.
+__device__ __forceinline__ void store_parts(uint8_t* row, float v) {
+  const __nv_bfloat16 a = __float2bfloat16(v);
+  const float r = v - __bfloat162float(a);
+  const __nv_bfloat16 b = __float2bfloat16(r);
+  __nv_bfloat16* p = reinterpret_cast<__nv_bfloat16*>(row);
+  p[0] = a;
+  p[1] = b;
+  p[2] = __float2bfloat16(r - __bfloat162float(b));
 }
 __device__ __forceinline__ void tma_load_3d(void* smem_dst, const CUtensorMap* tm, uint64_t* bar, int x, int y, int z) {
   asm volatile(
@@ -300,7 +315,9 @@ mlstm_gates_kernel(nfk_mlstm_params p) {
 // Tiles of q, k, v come by TMA (columns past a head's are filled with zeros; rows past the segment's last token
 // are other tokens' and get zero weights). Per chunk: scores and read-out of the old state by (32 tokens, 16 keys
 // or columns) per warp, outputs by (32 tokens, 16 columns), state update by 16-row tiles of S, which stays in
-// registers; its bf16 pair goes to shared memory for the next chunk's read-out.
+// registers; its bf16 pair goes to shared memory for the next chunk's read-out. n rides along as one more column
+// of S (its values are all ones), in three bf16 parts: the products n . q and K^T w come out of the same
+// instructions in full fp32 accuracy.
 template <int DP, bool STATE_ONLY>
 __global__ void __launch_bounds__(kChThreads, 1)
 mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
@@ -309,14 +326,13 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const uint32_t sb = smem_u32(smem);
-  float* n_s = reinterpret_cast<float*>(smem + C::F_OFF);   // [NPARTS][DP]: n is their sum
-  float* a_s = n_s + C::NPARTS * DP;  // a_j
-  float* mx_s = a_s + kChunk;         // M_t
-  float* int_s = mx_s + kChunk;       // e^(m_in - M_t)
+  float* a_s = reinterpret_cast<float*>(smem + C::F_OFF);   // a_j log2(e)
+  float* mx_s = a_s + kChunk;         // M_t log2(e) - log2(q_scale)
+  float* int_s = mx_s + kChunk;       // q_scale e^(m_in - M_t)
   float* w_s = int_s + kChunk;        // e^(a_j - M_last)
   float* em_s = w_s + kChunk;         // e^(-m_t)
   float* rs_s = em_s + kChunk;        // [4][64] row sums of the weighted scores
-  float* nq_s = rs_s + 4 * kChunk;    // n . q_t
+  float* nq_s = rs_s + 4 * kChunk;    // [4][64] parts of n . q_t
   uint64_t* q_full = reinterpret_cast<uint64_t*>(smem + C::BAR_OFF);
   uint64_t* kv_full = q_full + 1;     // two
   volatile int* abort_flag = reinterpret_cast<volatile int*>(q_full + 3);
@@ -397,7 +413,22 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         S[a][b][2 * h] = x.x;
         S[a][b][2 * h + 1] = x.y;
       }
-  for (int i = threadIdx.x; i < C::NPARTS * DP; i += kChThreads) n_s[i] = (from_zero || i >= p.dim) ? 0.f : n_in[i];
+  // n is the sum of columns 0-2 of the ninth tile, the others stay zero
+  float Sn[C::MTS][4];
+#pragma unroll
+  for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + (e >> 1) * 8;
+      Sn[a][e] = (from_zero || d >= p.dim || (lane & 3) != 0 || (e & 1) != 0) ? 0.f : n_in[d];
+    }
+  for (int i = threadIdx.x; i < (C::F_OFF - C::N_OFF) / 16; i += kChThreads)
+    *reinterpret_cast<uint4*>(smem + C::N_OFF + i * 16) = make_uint4(0u, 0u, 0u, 0u);
+  __syncthreads();
+  auto n_of = [&](int a, int h) {   // n of row (lane >> 2) + 8 h of row tile a, in every lane of its quad
+    const float x = (lane & 3) == 0 ? Sn[a][2 * h] + Sn[a][2 * h + 1] : (lane & 3) == 1 ? Sn[a][2 * h] : 0.f;
+    return quad_sum(x);
+  };
   auto publish_state = [&]() {      // the state's bf16 pair, B operand of the next chunk's read-out
 #pragma unroll
     for (int a = 0; a < C::MTS; ++a)
@@ -412,7 +443,18 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           *reinterpret_cast<uint32_t*>(smem + C::SH_OFF + off) = hi;
           *reinterpret_cast<uint32_t*>(smem + C::SL_OFF + off) = pack_bf16x2(S[a][b][2 * h] - hf.x, S[a][b][2 * h + 1] - hf.y);
         }
+    if (wn == 0) {
+#pragma unroll
+      for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const float n = n_of(a, h);
+          if ((lane & 3) == 0)
+            store_parts(smem + C::N_OFF + ((wm * C::MTS + a) * 16 + (lane >> 2) + h * 8) * 16, n);
+        }
+    }
   };
+  const float log2_qs = log2f(p.q_scale);
   if (!STATE_ONLY) publish_state();
 
   const int th = warp & 1, cq = warp >> 1;              // 32 tokens, 16 keys / columns
@@ -422,11 +464,13 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     const float decay = expf(m_in - M_last);
     if (threadIdx.x < kChunk) {
       const float M = fmaxf(m_in, gm);
-      a_s[threadIdx.x] = ga;
-      mx_s[threadIdx.x] = M;
-      int_s[threadIdx.x] = expf(m_in - M);
-      w_s[threadIdx.x] = expf(ga - M_last);
+      a_s[threadIdx.x] = ga * kLog2e;
+      mx_s[threadIdx.x] = M * kLog2e - log2_qs;
+      int_s[threadIdx.x] = p.q_scale * expf(m_in - M);
       em_s[threadIdx.x] = expf(-(gF + M));
+      const float w = expf(ga - M_last);
+      w_s[threadIdx.x] = w;
+      store_parts(smem + C::U_OFF + threadIdx.x * 16, w);
     }
     m_in = gF_last + M_last;
     F_total += gF_last;
@@ -462,39 +506,14 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     }
     float qs[2][2][4];
     if (!STATE_ONLY) {
-      // ---- n . q ----
-      {
-        const int t = threadIdx.x >> 2, part = threadIdx.x & 3;
-        float d = 0.f;
-#pragma unroll 2
-        for (int ch = part; ch < DP / 8; ch += 4) {
-          const uint4 q = *reinterpret_cast<const uint4*>(smem + C::Q_OFF + swz_blk(t, ch));
-          const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
-          float4 n0 = *reinterpret_cast<const float4*>(n_s + ch * 8), n1 = *reinterpret_cast<const float4*>(n_s + ch * 8 + 4);
-#pragma unroll
-          for (int k = 1; k < C::NPARTS; ++k) {
-            const float4 x0 = *reinterpret_cast<const float4*>(n_s + k * DP + ch * 8), x1 = *reinterpret_cast<const float4*>(n_s + k * DP + ch * 8 + 4);
-            n0.x += x0.x; n0.y += x0.y; n0.z += x0.z; n0.w += x0.w;
-            n1.x += x1.x; n1.y += x1.y; n1.z += x1.z; n1.w += x1.w;
-          }
-          const float nn[8] = {n0.x, n0.y, n0.z, n0.w, n1.x, n1.y, n1.z, n1.w};
-#pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const float2 f = unpack_bf16x2(qw[j]);
-            d += f.x * nn[2 * j] + f.y * nn[2 * j + 1];
-          }
-        }
-        d = quad_sum(d);
-        if (part == 0) nq_s[t] = d;
-      }
       // ---- scores Q K^T (16 keys) and read-out Q S (16 columns) of this warp's 32 tokens ----
-      float sc[2][2][4];
+      float sc[2][2][4], nq[2][4];
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) sc[i][j][e] = qs[i][j][e] = 0.f;
+          for (int e = 0; e < 4; ++e) sc[i][j][e] = qs[i][j][e] = nq[i][e] = 0.f;
       const bool keys_seen = cq * 16 <= th * 32 + 31;          // some of these keys are not in the future
 #pragma unroll 4
       for (int ks = 0; ks < DP / 16; ++ks) {
@@ -523,6 +542,11 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           mma_bf16(qs[i][0], a[i], l0, l1);
           mma_bf16(qs[i][1], a[i], l2, l3);
         }
+        if ((ks & 3) == cq) {              // n . q: every fourth step of the columns per warp
+          ldsm_x2_trans(sb + C::N_OFF + (ks * 16 + (lane & 15)) * 16, b0, b1);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) mma_bf16(nq[i], a[i], b0, b1);
+        }
       }
       // ---- weights, row sums, bf16 pair of the weighted scores ----
 #pragma unroll
@@ -536,8 +560,8 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           for (int j = 0; j < 2; ++j) {
             const int col = cq * 16 + j * 8 + (lane & 3) * 2;
             const float2 ac = *reinterpret_cast<const float2*>(a_s + col);
-            const float x0 = col <= r ? sc[i][j][2 * h] * p.q_scale * expf(ac.x - M) : 0.f;
-            const float x1 = col + 1 <= r ? sc[i][j][2 * h + 1] * p.q_scale * expf(ac.y - M) : 0.f;
+            const float x0 = col <= r ? sc[i][j][2 * h] * fast_exp2(ac.x - M) : 0.f;
+            const float x1 = col + 1 <= r ? sc[i][j][2 * h + 1] * fast_exp2(ac.y - M) : 0.f;
             sum += x0 + x1;
             const uint32_t hi = pack_bf16x2(x0, x1);
             const float2 hf = unpack_bf16x2(hi);
@@ -546,7 +570,11 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             *reinterpret_cast<uint32_t*>(smem + C::PL_OFF + o) = pack_bf16x2(x0 - hf.x, x1 - hf.y);
           }
           sum = quad_sum(sum);
-          if ((lane & 3) == 0) rs_s[cq * kChunk + r] = sum;
+          const float nqr = quad_sum((lane & 3) == 0 ? nq[i][2 * h] + nq[i][2 * h + 1] : (lane & 3) == 1 ? nq[i][2 * h] : 0.f);
+          if ((lane & 3) == 0) {
+            rs_s[cq * kChunk + r] = sum;
+            nq_s[cq * kChunk + r] = nqr;
+          }
         }
     }
     __syncthreads();                 // weighted scores and values are in shared memory; Q and the old state are free
@@ -586,8 +614,9 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         for (int h = 0; h < 2; ++h) {
           const int r = th * 32 + i * 16 + h * 8 + (lane >> 2), t = c * kChunk + r;
           if (t >= ntok) continue;
-          const float inter = int_s[r] * p.q_scale;
-          const float den = (rs_s[r] + rs_s[kChunk + r]) + (rs_s[2 * kChunk + r] + rs_s[3 * kChunk + r]) + inter * nq_s[r];
+          const float inter = int_s[r];
+          const float den = (rs_s[r] + rs_s[kChunk + r]) + (rs_s[2 * kChunk + r] + rs_s[3 * kChunk + r]) +
+                            inter * ((nq_s[r] + nq_s[kChunk + r]) + (nq_s[2 * kChunk + r] + nq_s[3 * kChunk + r]));
           const float inv = 1.f / (fmaxf(fabsf(den), em_s[r]) + 1e-6f);
           float* dst = p.out + static_cast<long long>(tok0 + t) * p.ld_out + head * p.vdim;
 #pragma unroll
@@ -607,12 +636,22 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
         for (int e = 0; e < 4; ++e) S[a][b][e] *= decay;
 #pragma unroll
+    for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) Sn[a][e] *= decay;
+#pragma unroll
     for (int ks = 0; ks < kChunk / 16; ++ks) {
       uint32_t ak[C::MTS][4];
 #pragma unroll
       for (int a = 0; a < C::MTS; ++a)
         ldsm_x4_trans(kb + swz_blk(ks * 16 + (mm >> 1) * 8 + rr, (wm * C::MTS + a) * 2 + (mm & 1)), ak[a][0], ak[a][1],
                       ak[a][2], ak[a][3]);
+      if (wn == 0) {
+        uint32_t u0, u1;
+        ldsm_x2_trans(sb + C::U_OFF + (ks * 16 + (lane & 15)) * 16, u0, u1);
+#pragma unroll
+        for (int a = 0; a < C::MTS; ++a) mma_bf16(Sn[a], ak[a], u0, u1);
+      }
 #pragma unroll
       for (int b = 0; b < C::NTS; b += 2) {
         const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, wn * C::NTS + b + (mm >> 1));
@@ -631,31 +670,8 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         }
       }
     }
-    {
-      // two columns and kChunk / NPARTS tokens per thread; each part of n is a sum of its own
-      constexpr int TOKS = kChunk / C::NPARTS;
-      const int dp = threadIdx.x % (DP / 2), part = threadIdx.x / (DP / 2);
-      float2* np = reinterpret_cast<float2*>(n_s + part * DP) + dp;
-      float2 n = *np;
-      n.x *= decay;
-      n.y *= decay;
-      const uint8_t* kp = smem + C::K_OFF + (c & 1) * C::QK_BYTES + (dp & 3) * 4;
-#pragma unroll
-      for (int j4 = 0; j4 < TOKS; j4 += 4) {
-        const int j0 = part * TOKS + j4;
-        const float4 w = *reinterpret_cast<const float4*>(w_s + j0);
-        const float ww[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(kp + swz_blk(j0 + j, dp >> 2)));
-          n.x += ww[j] * k.x;
-          n.y += ww[j] * k.y;
-        }
-      }
-      *np = n;
-    }
     if (!STATE_ONLY && c + 1 < n_chunks) publish_state();
-    __syncthreads();                 // gate arrays and n are free for the next chunk
+    __syncthreads();                 // gate arrays are free for the next chunk
   }
   if (*abort_flag != 0 && threadIdx.x == 0) {
     // a wait ran out: give copies still in flight a bounded chance to land before the CTA ends
@@ -679,11 +695,15 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           *reinterpret_cast<float2*>(S_out + static_cast<long long>(d) * p.vdim + v) = make_float2(S[a][b][2 * h], S[a][b][2 * h + 1]);
       }
   if (vs == 0) {
-    for (int d = threadIdx.x; d < p.dim; d += kChThreads) {
-      float n = n_s[d];
+    if (wn == 0) {
 #pragma unroll
-      for (int k = 1; k < C::NPARTS; ++k) n += n_s[k * DP + d];
-      n_out[d] = n;
+      for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
+          const float n = n_of(a, h);
+          if ((lane & 3) == 0 && d < p.dim) n_out[d] = n;
+        }
     }
     if (threadIdx.x == 0) {
       if (STATE_ONLY) {
@@ -865,7 +885,7 @@ extern "C" int nfk_mlstm_prefill(const nfk_mlstm_params* p, cudaStream_t stream)
   if (rc != NF_OK) return rc;
   if (p->req_count == 0) return NF_OK;
   const bool chunk_ok =
-      p->dtype == NFK_BF16 && p->dim <= 256 && p->items != nullptr && p->num_items >= p->req_count && p->num_tokens > 0 &&
+      p->dtype == NFK_BF16 && p->dim <= 256 && p->items != nullptr && p->num_items >= p->req_count && p->num_tokens > 0 && p->q_scale > 0.f &&
       (reinterpret_cast<uintptr_t>(p->qkv) & 15) == 0 && p->scratch != nullptr &&
       (reinterpret_cast<uintptr_t>(p->scratch) & 15) == 0 &&
       gate_floats(p->num_tokens, p->num_items, p->heads) +
