@@ -200,7 +200,7 @@ mlstm_seq_kernel(nfk_mlstm_params p, int v_slices) {
 }
 
 // ---- prefill, chunks of 64 tokens on tensor cores ----------------------------------------------------------
-constexpr int kChunk = 64, kVs = 64, kChThreads = 256;
+constexpr int kChunk = 64, kVs = 64, kGroup = 256, kChThreads = 2 * kGroup;   // output warps, state warps
 
 template <int DP>
 struct ChCfg {
@@ -221,7 +221,7 @@ struct ChCfg {
                                                           // 0-2 are three bf16 parts that add up to it
   static constexpr int U_OFF = N_OFF + DP * 16;           // its weighted values: the weights in three parts, [64][8]
   static constexpr int F_OFF = U_OFF + kChunk * 16;       // fp32 arrays
-  static constexpr int N_F32 = 13 * kChunk;
+  static constexpr int N_F32 = 12 * kChunk;
   static constexpr int BAR_OFF = F_OFF + N_F32 * 4;
   static constexpr int SMEM = BAR_OFF + 64 + 1024;
   static constexpr int WM = DP / 16 < 8 ? DP / 16 : 8;    // warps along dim in the state update
@@ -310,12 +310,18 @@ mlstm_gates_kernel(nfk_mlstm_params p) {
   }
 }
 
+// Named barriers: one per group, and two that hand the state's bf16 pair back and forth between the groups.
+enum : int { kBarOut = 1, kBarState = 2, kBarPublished = 3, kBarRead = 4 };
+__device__ __forceinline__ void bar_sync(int id, int n) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(n) : "memory"); }
+__device__ __forceinline__ void bar_arrive(int id, int n) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(n) : "memory"); }
+
 // STATE_ONLY: the segment's own contribution to the state, from zero, into scratch. Otherwise: outputs, from the
 // request's state (first segment) or from scratch; the last segment leaves the state in the request's slot.
 // Tiles of q, k, v come by TMA (columns past a head's are filled with zeros; rows past the segment's last token
-// are other tokens' and get zero weights). Per chunk: scores and read-out of the old state by (32 tokens, 16 keys
-// or columns) per warp, outputs by (32 tokens, 16 columns), state update by 16-row tiles of S, which stays in
-// registers; its bf16 pair goes to shared memory for the next chunk's read-out. n rides along as one more column
+// are other tokens' and get zero weights). Two groups of eight warps work side by side. The state warps keep S in
+// registers (16-row tiles), update it chunk by chunk and publish its bf16 pair in shared memory once the output
+// warps have read the previous one. The output warps compute scores and the read-out of the published state by
+// (32 tokens, 16 keys or columns), then the outputs by (32 tokens, 16 columns). n rides along as one more column
 // of S (its values are all ones), in three bf16 parts: the products n . q and K^T w come out of the same
 // instructions in full fp32 accuracy.
 template <int DP, bool STATE_ONLY>
@@ -329,15 +335,15 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   float* a_s = reinterpret_cast<float*>(smem + C::F_OFF);   // a_j log2(e)
   float* mx_s = a_s + kChunk;         // M_t log2(e) - log2(q_scale)
   float* int_s = mx_s + kChunk;       // q_scale e^(m_in - M_t)
-  float* w_s = int_s + kChunk;        // e^(a_j - M_last)
-  float* em_s = w_s + kChunk;         // e^(-m_t)
+  float* em_s = int_s + kChunk;       // e^(-m_t)
   float* rs_s = em_s + kChunk;        // [4][64] row sums of the weighted scores
   float* nq_s = rs_s + 4 * kChunk;    // [4][64] parts of n . q_t
   uint64_t* q_full = reinterpret_cast<uint64_t*>(smem + C::BAR_OFF);
   uint64_t* kv_full = q_full + 1;     // two
   volatile int* abort_flag = reinterpret_cast<volatile int*>(q_full + 3);
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = (threadIdx.x >> 5) & 7, lane = threadIdx.x & 31, tid = threadIdx.x % kGroup;
+  const bool state_warp = threadIdx.x >= kGroup;
   const int vs = blockIdx.x % v_slices;
   const int head = (blockIdx.x / v_slices) % p.heads;
   const int item = blockIdx.x / (v_slices * p.heads);
@@ -351,6 +357,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   float* sc_S = p.scratch + seg_off + (static_cast<long long>(item) * p.heads + head) * seg_floats(p.dim, p.vdim);
   float* sc_n = sc_S + static_cast<long long>(p.dim) * p.vdim;
   const int n_chunks = (ntok + kChunk - 1) / kChunk;
+  const int mm = lane >> 3, rr = lane & 7;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -359,6 +366,8 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     *abort_flag = 0;
     mbar_fence_init();
   }
+  for (int i = threadIdx.x; i < (C::F_OFF - C::N_OFF) / 16; i += kChThreads)
+    *reinterpret_cast<uint4*>(smem + C::N_OFF + i * 16) = make_uint4(0u, 0u, 0u, 0u);
   __syncthreads();
   auto load_kv = [&](int c) {        // one thread
     uint64_t* bar = kv_full + (c & 1);
@@ -369,67 +378,32 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     tma_load_3d(smem + C::V_OFF + (c & 1) * C::V_BYTES, &tmV, bar, v0, head, tok0 + c * kChunk);
   };
   auto load_q = [&](int c) {
-    if (STATE_ONLY) return;
     mbar_expect_tx(q_full, C::QK_BYTES);
 #pragma unroll
     for (int b = 0; b < DP / 64; ++b)
       tma_load_3d(smem + C::Q_OFF + b * (kChunk * 128), &tmQ, q_full, b * 64, head, tok0 + c * kChunk);
   };
+  // A wait that runs out is reported; the warps go on in step, so that they meet at their barriers.
+  auto wait_tile = [&](uint64_t* bar, int parity) {
+    if (*abort_flag == 0 && !mbar_wait(bar, parity)) {
+      if (lane == 0) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
+      *abort_flag = 1;
+    }
+  };
   if (threadIdx.x == 0) {
     load_kv(0);
-    load_q(0);
+    if (!STATE_ONLY) load_q(0);
   }
-  // gates of a chunk, fetched one chunk ahead: token threadIdx.x & 63, and the chunk's last maximum and sum
-  float ga, gm, gF, gm_last, gF_last;
-  auto fetch_gates = [&](int c) {
-    const float* g = chunk_gates(p, item, tok0, c < n_chunks ? c : n_chunks - 1, head);
-    const int t = threadIdx.x & 63;
-    ga = g[t];
-    gm = g[kChunk + t];
-    gF = g[2 * kChunk + t];
-    gm_last = g[2 * kChunk - 1];
-    gF_last = g[3 * kChunk - 1];
-  };
-  fetch_gates(0);
-
-  // ---- incoming state ----
   const bool from_zero = STATE_ONLY || (seg == 0 && st.fresh);
-  const float* S_in = seg == 0 ? p.S + sh * p.dim * p.vdim : sc_S;
-  const float* n_in = seg == 0 ? p.n + (sh * 2 + st.half) * p.dim : sc_n;
   float m_in = STATE_ONLY ? -INFINITY : (seg == 0 ? (st.fresh ? 0.f : p.m[sh * 2 + st.half]) : sc_n[p.dim + 2]);
-  float F_total = 0.f;
-  const int wm = warp % C::WM, wn = warp / C::WM;
-  float S[C::MTS][C::NTS][4];
-#pragma unroll
-  for (int a = 0; a < C::MTS; ++a)
-#pragma unroll
-    for (int b = 0; b < C::NTS; ++b)
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
-        const int v = v0 + (wn * C::NTS + b) * 8 + (lane & 3) * 2;
-        float2 x = make_float2(0.f, 0.f);
-        if (!from_zero && d < p.dim && v < p.vdim) x = *reinterpret_cast<const float2*>(S_in + static_cast<long long>(d) * p.vdim + v);
-        S[a][b][2 * h] = x.x;
-        S[a][b][2 * h + 1] = x.y;
-      }
-  // n is the sum of columns 0-2 of the ninth tile, the others stay zero
-  float Sn[C::MTS][4];
-#pragma unroll
-  for (int a = 0; a < C::MTS; ++a)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + (e >> 1) * 8;
-      Sn[a][e] = (from_zero || d >= p.dim || (lane & 3) != 0 || (e & 1) != 0) ? 0.f : n_in[d];
-    }
-  for (int i = threadIdx.x; i < (C::F_OFF - C::N_OFF) / 16; i += kChThreads)
-    *reinterpret_cast<uint4*>(smem + C::N_OFF + i * 16) = make_uint4(0u, 0u, 0u, 0u);
-  __syncthreads();
-  auto n_of = [&](int a, int h) {   // n of row (lane >> 2) + 8 h of row tile a, in every lane of its quad
-    const float x = (lane & 3) == 0 ? Sn[a][2 * h] + Sn[a][2 * h + 1] : (lane & 3) == 1 ? Sn[a][2 * h] : 0.f;
-    return quad_sum(x);
-  };
-  auto publish_state = [&]() {      // the state's bf16 pair, B operand of the next chunk's read-out
+  auto gates_of = [&](int c) { return chunk_gates(p, item, tok0, c < n_chunks ? c : n_chunks - 1, head); };
+
+  if (state_warp) {
+    // ------------------------------------------------------------------ state
+    const float* S_in = seg == 0 ? p.S + sh * p.dim * p.vdim : sc_S;
+    const float* n_in = seg == 0 ? p.n + (sh * 2 + st.half) * p.dim : sc_n;
+    const int wm = warp % C::WM, wn = warp / C::WM;
+    float S[C::MTS][C::NTS][4];
 #pragma unroll
     for (int a = 0; a < C::MTS; ++a)
 #pragma unroll
@@ -437,77 +411,215 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
           const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
-          const uint32_t off = swz(d, wn * C::NTS + b) + (lane & 3) * 4;
-          const uint32_t hi = pack_bf16x2(S[a][b][2 * h], S[a][b][2 * h + 1]);
-          const float2 hf = unpack_bf16x2(hi);
-          *reinterpret_cast<uint32_t*>(smem + C::SH_OFF + off) = hi;
-          *reinterpret_cast<uint32_t*>(smem + C::SL_OFF + off) = pack_bf16x2(S[a][b][2 * h] - hf.x, S[a][b][2 * h + 1] - hf.y);
+          const int v = v0 + (wn * C::NTS + b) * 8 + (lane & 3) * 2;
+          float2 x = make_float2(0.f, 0.f);
+          if (!from_zero && d < p.dim && v < p.vdim) x = *reinterpret_cast<const float2*>(S_in + static_cast<long long>(d) * p.vdim + v);
+          S[a][b][2 * h] = x.x;
+          S[a][b][2 * h + 1] = x.y;
         }
-    if (wn == 0) {
+    // n is the sum of columns 0-2 of the ninth tile, the others stay zero
+    float Sn[C::MTS][4];
+#pragma unroll
+    for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + (e >> 1) * 8;
+        Sn[a][e] = (from_zero || d >= p.dim || (lane & 3) != 0 || (e & 1) != 0) ? 0.f : n_in[d];
+      }
+    auto n_of = [&](int a, int h) {   // n of row (lane >> 2) + 8 h of row tile a, in every lane of its quad
+      const float x = (lane & 3) == 0 ? Sn[a][2 * h] + Sn[a][2 * h + 1] : (lane & 3) == 1 ? Sn[a][2 * h] : 0.f;
+      return quad_sum(x);
+    };
+    auto publish_state = [&]() {      // the state's bf16 pair, B operand of the next chunk's read-out
 #pragma unroll
       for (int a = 0; a < C::MTS; ++a)
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const float n = n_of(a, h);
-          if ((lane & 3) == 0)
-            store_parts(smem + C::N_OFF + ((wm * C::MTS + a) * 16 + (lane >> 2) + h * 8) * 16, n);
-        }
-    }
-  };
-  const float log2_qs = log2f(p.q_scale);
-  if (!STATE_ONLY) publish_state();
-
-  const int th = warp & 1, cq = warp >> 1;              // 32 tokens, 16 keys / columns
-  const int mm = lane >> 3, rr = lane & 7;
-  for (int c = 0; c < n_chunks; ++c) {
-    const float M_last = fmaxf(m_in, gm_last);
-    const float decay = expf(m_in - M_last);
-    if (threadIdx.x < kChunk) {
-      const float M = fmaxf(m_in, gm);
-      a_s[threadIdx.x] = ga * kLog2e;
-      mx_s[threadIdx.x] = M * kLog2e - log2_qs;
-      int_s[threadIdx.x] = p.q_scale * expf(m_in - M);
-      em_s[threadIdx.x] = expf(-(gF + M));
-      const float w = expf(ga - M_last);
-      w_s[threadIdx.x] = w;
-      store_parts(smem + C::U_OFF + threadIdx.x * 16, w);
-    }
-    m_in = gF_last + M_last;
-    F_total += gF_last;
-    // a wait that runs out is reported; the warps go on in step, so that they meet at their barriers
-    if (*abort_flag == 0 && (!mbar_wait(kv_full + (c & 1), (c >> 1) & 1) || (!STATE_ONLY && !mbar_wait(q_full, c & 1)))) {
-      if (lane == 0) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
-      *abort_flag = 1;
-    }
-    __syncthreads();                 // chunk c's gates and the state's bf16 pair are in shared memory
-    if (threadIdx.x == 0 && c + 1 < n_chunks) load_kv(c + 1);
-    fetch_gates(c + 1);
-    const uint32_t kb = sb + C::K_OFF + (c & 1) * C::QK_BYTES;
-    const uint32_t vb = sb + C::V_OFF + (c & 1) * C::V_BYTES;
-    // ---- values weighted by e^(a_j - M_last), as a bf16 pair ----
-    for (int i = threadIdx.x; i < kChunk * kVs / 8; i += kChThreads) {
-      const int r = i / (kVs / 8), ch = i % (kVs / 8);
-      const uint32_t off = swz(r, ch);
-      const uint4 v = *reinterpret_cast<const uint4*>(smem + C::V_OFF + (c & 1) * C::V_BYTES + off);
-      const uint32_t vw[4] = {v.x, v.y, v.z, v.w};
-      const float w = w_s[r];
-      uint32_t hi[4], lo[4];
+        for (int b = 0; b < C::NTS; ++b)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        float2 f = unpack_bf16x2(vw[j]);
-        f.x *= w;
-        f.y *= w;
-        hi[j] = pack_bf16x2(f.x, f.y);
-        const float2 hf = unpack_bf16x2(hi[j]);
-        lo[j] = pack_bf16x2(f.x - hf.x, f.y - hf.y);
+          for (int h = 0; h < 2; ++h) {
+            const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
+            const uint32_t off = swz(d, wn * C::NTS + b) + (lane & 3) * 4;
+            const uint32_t hi = pack_bf16x2(S[a][b][2 * h], S[a][b][2 * h + 1]);
+            const float2 hf = unpack_bf16x2(hi);
+            *reinterpret_cast<uint32_t*>(smem + C::SH_OFF + off) = hi;
+            *reinterpret_cast<uint32_t*>(smem + C::SL_OFF + off) = pack_bf16x2(S[a][b][2 * h] - hf.x, S[a][b][2 * h + 1] - hf.y);
+          }
+      if (wn == 0) {
+#pragma unroll
+        for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            const float n = n_of(a, h);
+            if ((lane & 3) == 0)
+              store_parts(smem + C::N_OFF + ((wm * C::MTS + a) * 16 + (lane >> 2) + h * 8) * 16, n);
+          }
       }
-      *reinterpret_cast<uint4*>(smem + C::WH_OFF + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-      *reinterpret_cast<uint4*>(smem + C::WL_OFF + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-    }
-    float qs[2][2][4];
+    };
     if (!STATE_ONLY) {
+      publish_state();
+      bar_arrive(kBarPublished, kChThreads);
+    }
+    // gates of a chunk, fetched one chunk ahead: of the token rows this thread weights, and the chunk's last ones
+    float ga[2], gm_last, gF_last, F_total = 0.f;
+    auto fetch_gates = [&](int c) {
+      const float* g = gates_of(c);
+      ga[0] = g[tid >> 3];
+      ga[1] = g[32 + (tid >> 3)];
+      gm_last = g[2 * kChunk - 1];
+      gF_last = g[3 * kChunk - 1];
+    };
+    fetch_gates(0);
+    for (int c = 0; c < n_chunks; ++c) {
+      const float M_last = fmaxf(m_in, gm_last);
+      const float decay = expf(m_in - M_last);
+      m_in = gF_last + M_last;
+      F_total += gF_last;
+      const float w[2] = {expf(ga[0] - M_last), expf(ga[1] - M_last)};
+      fetch_gates(c + 1);
+      const uint32_t kb = sb + C::K_OFF + (c & 1) * C::QK_BYTES;
+      wait_tile(kv_full + (c & 1), (c >> 1) & 1);
+      // values weighted by e^(a_j - M_last), as a bf16 pair, and the weights as values of n
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int r = i * 32 + (tid >> 3);
+        const uint32_t off = swz(r, tid & 7);
+        const uint4 v = *reinterpret_cast<const uint4*>(smem + C::V_OFF + (c & 1) * C::V_BYTES + off);
+        const uint32_t vw[4] = {v.x, v.y, v.z, v.w};
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          float2 f = unpack_bf16x2(vw[j]);
+          f.x *= w[i];
+          f.y *= w[i];
+          hi[j] = pack_bf16x2(f.x, f.y);
+          const float2 hf = unpack_bf16x2(hi[j]);
+          lo[j] = pack_bf16x2(f.x - hf.x, f.y - hf.y);
+        }
+        *reinterpret_cast<uint4*>(smem + C::WH_OFF + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(smem + C::WL_OFF + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        if ((tid & 7) == 0) store_parts(smem + C::U_OFF + r * 16, w[i]);
+      }
+      bar_sync(kBarState, kGroup);
+      if (STATE_ONLY && tid == 0 && c + 1 < n_chunks) load_kv(c + 1);
+      // S = decay S + K^T (w V), n = decay n + K^T w
+#pragma unroll
+      for (int a = 0; a < C::MTS; ++a) {
+#pragma unroll
+        for (int b = 0; b < C::NTS; ++b)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) S[a][b][e] *= decay;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) Sn[a][e] *= decay;
+      }
+#pragma unroll
+      for (int ks = 0; ks < kChunk / 16; ++ks) {
+        uint32_t ak[C::MTS][4];
+#pragma unroll
+        for (int a = 0; a < C::MTS; ++a)
+          ldsm_x4_trans(kb + swz_blk(ks * 16 + (mm >> 1) * 8 + rr, (wm * C::MTS + a) * 2 + (mm & 1)), ak[a][0], ak[a][1],
+                        ak[a][2], ak[a][3]);
+        if (wn == 0) {
+          uint32_t u0, u1;
+          ldsm_x2_trans(sb + C::U_OFF + (ks * 16 + (lane & 15)) * 16, u0, u1);
+#pragma unroll
+          for (int a = 0; a < C::MTS; ++a) mma_bf16(Sn[a], ak[a], u0, u1);
+        }
+#pragma unroll
+        for (int b = 0; b < C::NTS; b += 2) {
+          const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, wn * C::NTS + b + (mm >> 1));
+          uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+          ldsm_x4_trans(sb + C::WH_OFF + off, h0, h1, h2, h3);
+          ldsm_x4_trans(sb + C::WL_OFF + off, l0, l1, l2, l3);
+#pragma unroll
+          for (int a = 0; a < C::MTS; ++a) {
+            mma_bf16(S[a][b], ak[a], h0, h1);
+            mma_bf16(S[a][b + 1], ak[a], h2, h3);
+          }
+#pragma unroll
+          for (int a = 0; a < C::MTS; ++a) {
+            mma_bf16(S[a][b], ak[a], l0, l1);
+            mma_bf16(S[a][b + 1], ak[a], l2, l3);
+          }
+        }
+      }
+      if (!STATE_ONLY && c + 1 < n_chunks) {
+        bar_sync(kBarRead, kChThreads);        // the output warps have read the previous state
+        publish_state();
+        bar_arrive(kBarPublished, kChThreads);
+      } else {
+        bar_sync(kBarState, kGroup);           // weighted values are free for the next chunk
+      }
+    }
+    // ---- state out ----
+    if (STATE_ONLY || !has_next) {
+      float* S_out = STATE_ONLY ? sc_S : p.S + sh * p.dim * p.vdim;
+      float* n_out = STATE_ONLY ? sc_n : p.n + (sh * 2 + (st.half ^ 1)) * p.dim;
+#pragma unroll
+      for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+        for (int b = 0; b < C::NTS; ++b)
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
+            const int v = v0 + (wn * C::NTS + b) * 8 + (lane & 3) * 2;
+            if (d < p.dim && v < p.vdim)
+              *reinterpret_cast<float2*>(S_out + static_cast<long long>(d) * p.vdim + v) = make_float2(S[a][b][2 * h], S[a][b][2 * h + 1]);
+          }
+      if (vs == 0) {
+        if (wn == 0) {
+#pragma unroll
+          for (int a = 0; a < C::MTS; ++a)
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+              const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
+              const float n = n_of(a, h);
+              if ((lane & 3) == 0 && d < p.dim) n_out[d] = n;
+            }
+        }
+        if (tid == 0) {
+          if (STATE_ONLY) {
+            sc_n[p.dim] = m_in;
+            sc_n[p.dim + 1] = F_total;
+          } else {
+            p.m[sh * 2 + (st.half ^ 1)] = m_in;
+          }
+        }
+      }
+    }
+  } else if (!STATE_ONLY) {
+    // ------------------------------------------------------------------ outputs
+    const int th = warp & 1, cq = warp >> 1;              // 32 tokens, 16 keys / columns
+    const float log2_qs = log2f(p.q_scale);
+    float ga, gm, gF, gm_last, gF_last;
+    auto fetch_gates = [&](int c) {
+      const float* g = gates_of(c);
+      const int t = tid & 63;
+      ga = g[t];
+      gm = g[kChunk + t];
+      gF = g[2 * kChunk + t];
+      gm_last = g[2 * kChunk - 1];
+      gF_last = g[3 * kChunk - 1];
+    };
+    fetch_gates(0);
+    for (int c = 0; c < n_chunks; ++c) {
+      if (tid < kChunk) {
+        const float M = fmaxf(m_in, gm);
+        a_s[tid] = ga * kLog2e;
+        mx_s[tid] = M * kLog2e - log2_qs;
+        int_s[tid] = p.q_scale * expf(m_in - M);
+        em_s[tid] = expf(-(gF + M));
+      }
+      m_in = gF_last + fmaxf(m_in, gm_last);
+      fetch_gates(c + 1);
+      wait_tile(q_full, c & 1);
+      wait_tile(kv_full + (c & 1), (c >> 1) & 1);
+      // chunk c's gates and the state before it are in shared memory; chunk c - 1's k and v have been used up
+      bar_sync(kBarPublished, kChThreads);
+      if (tid == 0 && c + 1 < n_chunks) load_kv(c + 1);
+      const uint32_t kb = sb + C::K_OFF + (c & 1) * C::QK_BYTES;
+      const uint32_t vb = sb + C::V_OFF + (c & 1) * C::V_BYTES;
       // ---- scores Q K^T (16 keys) and read-out Q S (16 columns) of this warp's 32 tokens ----
-      float sc[2][2][4], nq[2][4];
+      float sc[2][2][4], qs[2][2][4], nq[2][4];
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -515,7 +627,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
           for (int e = 0; e < 4; ++e) sc[i][j][e] = qs[i][j][e] = nq[i][e] = 0.f;
       const bool keys_seen = cq * 16 <= th * 32 + 31;          // some of these keys are not in the future
-#pragma unroll 4
+#pragma unroll 2
       for (int ks = 0; ks < DP / 16; ++ks) {
         uint32_t a[2][4], b0, b1, b2, b3, h0, h1, h2, h3, l0, l1, l2, l3;
 #pragma unroll
@@ -548,6 +660,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           for (int i = 0; i < 2; ++i) mma_bf16(nq[i], a[i], b0, b1);
         }
       }
+      if (c + 1 < n_chunks) bar_arrive(kBarRead, kChThreads);
       // ---- weights, row sums, bf16 pair of the weighted scores ----
 #pragma unroll
       for (int i = 0; i < 2; ++i)
@@ -576,10 +689,8 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             nq_s[cq * kChunk + r] = nqr;
           }
         }
-    }
-    __syncthreads();                 // weighted scores and values are in shared memory; Q and the old state are free
-    if (threadIdx.x == 0 && c + 1 < n_chunks) load_q(c + 1);
-    if (!STATE_ONLY) {
+      bar_sync(kBarOut, kGroup);         // weighted scores are in shared memory, Q is free
+      if (tid == 0 && c + 1 < n_chunks) load_q(c + 1);
       // ---- P V, then the outputs of these 32 tokens x 16 columns ----
       float pv[2][2][4];
 #pragma unroll
@@ -627,92 +738,13 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
                                                                 (inter * qs[i][j][2 * h + 1] + pv[i][j][2 * h + 1]) * inv);
           }
         }
+      bar_sync(kBarOut, kGroup);         // gate arrays, sums and weighted scores are free for the next chunk
     }
-    // ---- state update: S = decay S + K^T (w V), n = decay n + K^T w ----
-#pragma unroll
-    for (int a = 0; a < C::MTS; ++a)
-#pragma unroll
-      for (int b = 0; b < C::NTS; ++b)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) S[a][b][e] *= decay;
-#pragma unroll
-    for (int a = 0; a < C::MTS; ++a)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) Sn[a][e] *= decay;
-#pragma unroll
-    for (int ks = 0; ks < kChunk / 16; ++ks) {
-      uint32_t ak[C::MTS][4];
-#pragma unroll
-      for (int a = 0; a < C::MTS; ++a)
-        ldsm_x4_trans(kb + swz_blk(ks * 16 + (mm >> 1) * 8 + rr, (wm * C::MTS + a) * 2 + (mm & 1)), ak[a][0], ak[a][1],
-                      ak[a][2], ak[a][3]);
-      if (wn == 0) {
-        uint32_t u0, u1;
-        ldsm_x2_trans(sb + C::U_OFF + (ks * 16 + (lane & 15)) * 16, u0, u1);
-#pragma unroll
-        for (int a = 0; a < C::MTS; ++a) mma_bf16(Sn[a], ak[a], u0, u1);
-      }
-#pragma unroll
-      for (int b = 0; b < C::NTS; b += 2) {
-        const uint32_t off = swz(ks * 16 + (mm & 1) * 8 + rr, wn * C::NTS + b + (mm >> 1));
-        uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
-        ldsm_x4_trans(sb + C::WH_OFF + off, h0, h1, h2, h3);
-        ldsm_x4_trans(sb + C::WL_OFF + off, l0, l1, l2, l3);
-#pragma unroll
-        for (int a = 0; a < C::MTS; ++a) {
-          mma_bf16(S[a][b], ak[a], h0, h1);
-          mma_bf16(S[a][b + 1], ak[a], h2, h3);
-        }
-#pragma unroll
-        for (int a = 0; a < C::MTS; ++a) {
-          mma_bf16(S[a][b], ak[a], l0, l1);
-          mma_bf16(S[a][b + 1], ak[a], l2, l3);
-        }
-      }
-    }
-    if (!STATE_ONLY && c + 1 < n_chunks) publish_state();
-    __syncthreads();                 // gate arrays are free for the next chunk
+    if (*abort_flag != 0 && tid == 0) (void)mbar_wait(q_full, (n_chunks - 1) & 1);
   }
-  if (*abort_flag != 0 && threadIdx.x == 0) {
+  if (*abort_flag != 0 && state_warp && tid == 0) {
     // a wait ran out: give copies still in flight a bounded chance to land before the CTA ends
     for (int c = n_chunks > 1 ? n_chunks - 2 : 0; c < n_chunks; ++c) (void)mbar_wait(kv_full + (c & 1), (c >> 1) & 1);
-    if (!STATE_ONLY) (void)mbar_wait(q_full, (n_chunks - 1) & 1);
-  }
-
-  // ---- state out ----
-  if (!STATE_ONLY && has_next) return;
-  float* S_out = STATE_ONLY ? sc_S : p.S + sh * p.dim * p.vdim;
-  float* n_out = STATE_ONLY ? sc_n : p.n + (sh * 2 + (st.half ^ 1)) * p.dim;
-#pragma unroll
-  for (int a = 0; a < C::MTS; ++a)
-#pragma unroll
-    for (int b = 0; b < C::NTS; ++b)
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
-        const int v = v0 + (wn * C::NTS + b) * 8 + (lane & 3) * 2;
-        if (d < p.dim && v < p.vdim)
-          *reinterpret_cast<float2*>(S_out + static_cast<long long>(d) * p.vdim + v) = make_float2(S[a][b][2 * h], S[a][b][2 * h + 1]);
-      }
-  if (vs == 0) {
-    if (wn == 0) {
-#pragma unroll
-      for (int a = 0; a < C::MTS; ++a)
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const int d = (wm * C::MTS + a) * 16 + (lane >> 2) + h * 8;
-          const float n = n_of(a, h);
-          if ((lane & 3) == 0 && d < p.dim) n_out[d] = n;
-        }
-    }
-    if (threadIdx.x == 0) {
-      if (STATE_ONLY) {
-        sc_n[p.dim] = m_in;
-        sc_n[p.dim + 1] = F_total;
-      } else {
-        p.m[sh * 2 + (st.half ^ 1)] = m_in;
-      }
-    }
   }
 }
 
