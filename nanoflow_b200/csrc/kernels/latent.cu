@@ -322,9 +322,9 @@ latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_
       for (int off = 8; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
       const float mn = fmaxf(m_r, mx);
       const float ms = mn == -INFINITY ? 0.f : mn;
-      const float al = exp2f(m_r - ms);
+      const float al = fast_exp2(m_r - ms);
       m_r = mn;
-      const float e0 = exp2f(v.x - ms), e1 = exp2f(v.y - ms), e2 = exp2f(v.z - ms), e3 = exp2f(v.w - ms);
+      const float e0 = fast_exp2(v.x - ms), e1 = fast_exp2(v.y - ms), e2 = fast_exp2(v.z - ms), e3 = fast_exp2(v.w - ms);
       l_r = l_r * al + ((e0 + e1) + (e2 + e3));      // this lane's keys; the row's lanes are added up at the end
       const uint32_t h0 = pack_bf16x2(e0, e1), h1 = pack_bf16x2(e2, e3);
       const float2 f0 = unpack_bf16x2(h0), f1 = unpack_bf16x2(h1);
@@ -404,8 +404,8 @@ latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_
       const float m0 = alpha_s[row], m1 = other_m[row];
       ms[half] = fmaxf(m0, m1);
       const float msafe = ms[half] == -INFINITY ? 0.f : ms[half];
-      f0[half] = exp2f(m0 - msafe);
-      f1[half] = exp2f(m1 - msafe);
+      f0[half] = fast_exp2(m0 - msafe);
+      f1[half] = fast_exp2(m1 - msafe);
 #pragma unroll
       for (int b = 0; b < DW; ++b) {
         const float2 v = *reinterpret_cast<const float2*>(mo + row * Cfg::O_LD + c0 + b * 8);
@@ -463,7 +463,7 @@ latent_attn_merge_kernel(nfk_latent_attn_params p) {
   float m = -INFINITY, l = 0.f;
   for (int s = 0; s < p.splits; ++s) m = fmaxf(m, ws[s * step + D]);
   const float ms = m == -INFINITY ? 0.f : m;
-  for (int s = 0; s < p.splits; ++s) l += ws[s * step + D + 1] * exp2f(ws[s * step + D] - ms);
+  for (int s = 0; s < p.splits; ++s) l += ws[s * step + D + 1] * fast_exp2(ws[s * step + D] - ms);
   const float inv = l > 0.f ? 1.f / l : 0.f;
   const int tok = p.tokens[ti];
   __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(tok) * p.ld_out +
@@ -471,7 +471,7 @@ latent_attn_merge_kernel(nfk_latent_attn_params p) {
   for (int c = threadIdx.x * 2; c < D; c += 256) {
     float x = 0.f, y = 0.f;
     for (int s = 0; s < p.splits; ++s) {
-      const float w = exp2f(ws[s * step + D] - ms);
+      const float w = fast_exp2(ws[s * step + D] - ms);
       const float2 v = *reinterpret_cast<const float2*>(ws + s * step + c);
       x += v.x * w;
       y += v.y * w;

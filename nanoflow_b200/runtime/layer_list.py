@@ -462,14 +462,15 @@ MIXERS = {"latent_attention": LayerListEngine._latent_attention, "mlstm": LayerL
 # --------------------------------------------------------------------------------------------------
 def mlstm_segments(qo_indptr: np.ndarray, n_dec: int, ctas_per_segment: int, sms: int) -> np.ndarray:
     """Rows (request, first token, tokens, segment) for the chunked mLSTM kernel. A portion is one segment unless
-    the portions alone leave most SMs idle; then long ones are cut into equal runs of whole chunks."""
+    the portions alone leave SMs idle; then long ones are cut into equal runs of whole chunks, enough of them to
+    keep the last wave short (segments cost an extra pass over the keys and values)."""
     reqs = np.arange(n_dec, qo_indptr.size - 1)
     lens = np.diff(qo_indptr)[n_dec:]
     if reqs.size == 0:
         return np.zeros((0, 4), dtype=np.int32)
-    target = 2 * sms // max(1, ctas_per_segment)
+    target = 4 * sms // max(1, ctas_per_segment)
     seg_len = int(lens.max())
-    if reqs.size < target and reqs.size < SEGMENT_ITEMS:
+    if 2 * reqs.size * ctas_per_segment < 3 * sms and reqs.size < min(target, SEGMENT_ITEMS):
         room = min(target, SEGMENT_ITEMS) - reqs.size
         seg_len = max(4 * MLSTM_CHUNK, -(-int(lens.sum()) // room))
         seg_len = (seg_len + MLSTM_CHUNK - 1) // MLSTM_CHUNK * MLSTM_CHUNK
