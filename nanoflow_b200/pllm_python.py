@@ -63,13 +63,16 @@ def setModelConfig(config, *, backend: Optional[str] = None) -> NanoflowConfig:
 def createModelWeight(seed: int = 0):
     """Random-init weights of the configured architecture: this rank's shard on the GPU backend, all
     ranks' shards (a list) on the CPU backend, which runs every rank in one process."""
-    from .models import random_full_weights, random_rank_weights, shard_weights
+    from .models import random_full_weights, shard_weights
+    from .models.registry import family_of
 
     cfg = _need("cfg", "setModelConfig")
-    m = cfg.model
+    m, fam = cfg.model, family_of(cfg.raw["model"])
     if _state["backend"] == "gpu":
         dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
-        return random_rank_weights(m, _state["rank"], m.tp, dev, seed=seed)
+        return fam.random_weights(cfg, _state["rank"], m.tp, dev, seed=seed)
+    if fam.listed_layers:
+        return [fam.random_weights(cfg, 0, 1, "cpu", seed=seed)]
     fw = random_full_weights(m, seed=seed)
     return [shard_weights(fw, m, r, m.tp, dtype=torch.float32) for r in range(m.tp)]
 
@@ -92,9 +95,10 @@ def config(config_data=None) -> None:
     cfg, weights = _need("cfg", "setModelConfig"), _need("weights", "init")
     if config_data and config_data.get("nanobatch_sizes"):
         cfg.engine.nanobatch_sizes = list(config_data["nanobatch_sizes"])
-    if _state["backend"] == "gpu":
-        from .runtime.engine import Engine
+    from .models.registry import family_of
 
+    fam = family_of(cfg.raw["model"])
+    if _state["backend"] == "gpu":
         local = int(os.environ.get("LOCAL_RANK", "0"))
         torch.cuda.set_device(local)
         dev = torch.device("cuda", local)
@@ -106,11 +110,9 @@ def config(config_data=None) -> None:
             if not dist.is_initialized():
                 dist.init_process_group("nccl", device_id=dev)
             _state["coll"] = TpCollectives(_state["rank"], _state["world"], dev)
-        _state["engine"] = Engine(cfg, weights, device=dev, collectives=_state["coll"], num_pages=_state["pages"])
+        _state["engine"] = fam.engine(cfg, weights, device=dev, collectives=_state["coll"], num_pages=_state["pages"])
     else:
-        from .runtime.cpu_backend import CpuEngine
-
-        _state["engine"] = CpuEngine(cfg, weights, num_pages=_state["pages"] or 4096)
+        _state["engine"] = fam.cpu_engine(cfg, weights, num_pages=_state["pages"] or 4096)
 
 
 def num_pages() -> int:

@@ -44,9 +44,8 @@ def main(argv=None) -> int:
     import torch
 
     from .config import load_config
-    from .models import random_rank_weights
-    from .runtime.engine import Engine
-    from .serving import DistKVPool, RequestManager, Scheduler
+    from .models.registry import family_of
+    from .serving import DistKVPool, RequestManager, Scheduler, StateSlotPool
     from .serving.loop import ServingLoop
 
     rank, world = int(os.environ.get("RANK", "0")), int(os.environ.get("WORLD_SIZE", "1"))
@@ -75,8 +74,9 @@ def main(argv=None) -> int:
         m.num_layers = m.run_layers = a.layers
     gbs = e.global_batch_size
     e.max_batch_size = max(e.max_batch_size, gbs)
-    w = random_rank_weights(m, rank, tp, dev)
-    eng = Engine(cfg, w, collectives=coll, num_pages=a.pages or None)
+    fam = family_of(cfg.raw["model"])
+    w = fam.random_weights(cfg, rank, tp, dev)
+    eng = fam.engine(cfg, w, collectives=coll, num_pages=a.pages or None)
     n_req = int((a.skip_cycles + 4 * a.iters + 64) * gbs / (a.input_len + a.output_len)) + 256
     rm = RequestManager(vocab_size=m.vocab_size, random_ids=True, seed=0)
     for _ in range(n_req):
@@ -86,7 +86,9 @@ def main(argv=None) -> int:
     sch = Scheduler(pool, rm.avaliable_request_queue, global_batch_size=gbs, nanobatch_sizes=e.resolved_nanobatches(),
                     max_batch_size=e.max_batch_size, average_prefill_length=a.input_len,
                     average_decode_length=a.output_len, group_size=m.group_size,
-                    decode_tail_fraction=e.decode_tail_fraction)
+                    decode_tail_fraction=e.decode_tail_fraction,
+                    state_pool=StateSlotPool(eng.num_slots) if getattr(eng, "num_slots", 0) else None,
+                    kv_window=getattr(m, "kv_window", 0))
     loop = ServingLoop(eng, sch, rm, simulated_time=True, est_cycle_time=1.0)
     loop.skip_cycles(a.skip_cycles)
     loop.step()
