@@ -194,7 +194,7 @@ def latent_case(dtype, impl, heads, ld, window, scale, positions, lens, splits=1
 
 
 VARIANTS = [(torch.float32, 1, 40), (torch.bfloat16, 1, 72), (torch.bfloat16, 2, 64), (torch.bfloat16, 2, 192),
-            (torch.bfloat16, 2, 512)]
+            (torch.bfloat16, 2, 512), (torch.bfloat16, 3, 128), (torch.bfloat16, 3, 384), (torch.bfloat16, 3, 512)]
 
 
 @pytest.mark.parametrize("dtype,impl,ld", VARIANTS)
@@ -240,13 +240,13 @@ def test_latent_attention_sinks_take_their_share(dtype, impl, ld):
     assert rel(got, want) < TOL[dtype] * 3 and rel(none, want) > 0.2
 
 
-@pytest.mark.parametrize("ld,heads", [(64, 4), (256, 20), (512, 33)])
+@pytest.mark.parametrize("impl,ld,heads", [(2, 64, 4), (2, 256, 20), (3, 256, 20), (3, 512, 33)])
 @pytest.mark.parametrize("splits", [2, 3, 7])
-def test_latent_attention_split_over_key_ranges(ld, heads, splits):
+def test_latent_attention_split_over_key_ranges(impl, ld, heads, splits):
     lens = [30, 700, 65]
     pos = [(0, 29), (1, 699), (1, 64), (2, 64), (2, 0)]
     for window in (0, 100):
-        got, want = latent_case(torch.bfloat16, 2, heads, ld, window, ld ** -0.5, pos, lens, splits=splits, sink_value=0.5)
+        got, want = latent_case(torch.bfloat16, impl, heads, ld, window, ld ** -0.5, pos, lens, splits=splits, sink_value=0.5)
         assert rel(got, want) < TOL[torch.bfloat16] * 3
 
 
@@ -624,3 +624,21 @@ def test_greedy_generation_in_bf16_stays_near_the_oracle_arg_max():
         logits = oracle.forward(raw, t, p.tolist() + out[i][:-1])[len(p) - 1:]
         gap = logits.max(-1).values - logits[torch.arange(12), torch.tensor(out[i])]
         assert float(gap.max()) < 0.25 * float(logits.std())
+
+
+def test_latent_attention_maxima_that_keep_growing():
+    """Scores that rise from tile to tile, far beyond what exponentials of the first reference maximum could hold."""
+    for impl in (2, 3):
+        ld, heads, n = 256, 5, 400
+        pg = Paged([n], ld, torch.bfloat16)
+        lat = rnd(n, ld, seed=1, dtype=torch.bfloat16)
+        lat[:, 0] = torch.arange(n, device="cuda") * 0.5
+        q = rnd(1, heads, ld, seed=2, scale=0.2).bfloat16()
+        q[0, :, 0] = torch.tensor([1.0, -1.0, 0.3, 0.0, 4.0])
+        pg.fill(0, lat)
+        out, st = torch.zeros(1, heads * ld, dtype=torch.bfloat16, device="cuda"), ops.new_status()
+        K.latent_attention(q.reshape(1, -1), pg.pool, out, i32([0]), i32([n - 1]), i32([0]), pg.indptr, pg.indices, heads=heads,
+                           scale=1.0, impl=impl, status=st)
+        ops.check_status(st)
+        p = torch.softmax(q[0].double() @ lat.double().T, dim=-1)
+        assert torch.allclose(out.reshape(heads, ld).double(), p @ lat.double(), rtol=1e-2, atol=0.02), impl
