@@ -23,6 +23,15 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
   *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
 }
 
+// Latent pool pages: whether they are stored in 8 x 64 tiles, and the element offset of (row, column) of a page.
+__host__ __device__ __forceinline__ bool latent_tiled(int dtype, long long ld, int page_size) {
+  return dtype == NFK_BF16 && ld % 64 == 0 && page_size % 8 == 0;
+}
+__device__ __forceinline__ long long latent_offset(int page, int row, int col, int page_size, long long ld, bool tiled) {
+  if (!tiled) return (static_cast<long long>(page) * page_size + row) * ld + col;
+  return static_cast<long long>(page) * page_size * ld + (row >> 3) * 8 * ld + (col >> 6) * 512 + (row & 7) * 64 + (col & 63);
+}
+
 // Index of the page that holds position `pos` of request `req` in kv_indices, or -1 (reported): a request's
 // page list starts at page slot kv_first[req] of its sequence (earlier pages have been given back).
 __device__ __forceinline__ int page_of(int pos, int req, int page_size, const int* kv_indptr, const int* kv_indices,

@@ -250,8 +250,10 @@ typedef struct nfk_residual_norm_params {
 } nfk_residual_norm_params;
 int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t stream);
 
-// Latent pool of one layer: [num_pages][page_size][ld] rows (ld = latent size padded to a multiple of 8, the
-// padding is zero). Token t's latent: RMS norm of src[t, 0:rank] times w, written to its page slot.
+// Latent pool of one layer: pages of page_size rows of ld elements (ld = latent size padded to a multiple of 8, the
+// padding is zero). bf16 pages whose ld is a multiple of 64 are stored in tiles, [page_size / 8][ld / 64][8 rows][64
+// columns], so that one TMA copy brings in a whole page in the layout the tensor cores read; all others row by
+// row. Token t's latent: RMS norm of src[t, 0:rank] times w, written to its page slot.
 // kv_first[req]: page slot of the sequence that the request's page list starts with (null: 0).
 typedef struct nfk_latent_append_params {
   const void* src;
@@ -270,6 +272,17 @@ typedef struct nfk_latent_append_params {
   unsigned int* status;
 } nfk_latent_append_params;
 int nfk_latent_append(const nfk_latent_append_params* p, cudaStream_t stream);
+
+// Pages of a latent pool -> plain rows: out[i * page_size + r, :] = row r of page page_ids[i].
+typedef struct nfk_latent_gather_params {
+  const void* pool;
+  void* out;                 // [n_pages * page_size, ld]
+  const int* page_ids;
+  long long ld;
+  int n_pages, page_size, num_pages, dtype;
+  unsigned int* status;
+} nfk_latent_gather_params;
+int nfk_latent_gather(const nfk_latent_gather_params* p, cudaStream_t stream);
 
 // Attention in latent space, for listed tokens: head h's query (already multiplied by its key matrix) meets
 // the cached latents, which are keys and values at once: out = sum_j softmax(scale q . c_j) c_j over the

@@ -2,6 +2,7 @@
 // pool layout).
 //
 // nfk_latent_append   RMS norm of a token's latent row, written to its page slot
+// nfk_latent_gather   pages back to plain rows (for the expansion to keys and values)
 // nfk_latent_attn     attention of listed tokens in latent space (queries already multiplied by their heads'
 //                     key matrices, so the cached row is key and value at once), sliding window, sink.
 //                     Used for decoding, for prompt tokens whose keys are not expanded, and in 32-bit.
@@ -30,6 +31,7 @@ latent_append_kernel(nfk_latent_append_params p) {
   const bool vec = p.ld_src % 4 == 0 && p.ld % 4 == 0 && (reinterpret_cast<uintptr_t>(p.src) & 15) == 0 &&
                    (reinterpret_cast<uintptr_t>(p.w) & 15) == 0 && (reinterpret_cast<uintptr_t>(p.pool) & 15) == 0;
   const int n4 = vec ? p.rank / 4 * 4 : 0;
+  const bool tiled = latent_tiled(p.dtype, p.ld, p.page_size);
   for (int t = blockIdx.x * 4 + (threadIdx.x >> 5); t < p.T; t += gridDim.x * 4) {
     const T* src = reinterpret_cast<const T*>(p.src) + static_cast<long long>(t) * p.ld_src;
     const int pos = p.positions[t];
@@ -46,12 +48,34 @@ latent_append_kernel(nfk_latent_append_params p) {
     }
     const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(p.rank) + p.eps);
     if (page < 0) continue;
-    T* dst = reinterpret_cast<T*>(p.pool) + (static_cast<long long>(page) * p.page_size + pos % p.page_size) * p.ld;
+    T* pool = reinterpret_cast<T*>(p.pool);
+    auto at = [&](int c) { return pool + latent_offset(page, pos % p.page_size, c, p.page_size, p.ld, tiled); };
     for (int c = lane * 4; c < n4; c += 128) {
       const float4 v = load4(src + c), w = load4(p.w + c);
-      store4(dst + c, make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w));
+      store4(at(c), make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w));
     }
-    for (int c = n4 + lane; c < p.rank; c += 32) put(dst + c, to_f32(src[c]) * inv * p.w[c]);
+    for (int c = n4 + lane; c < p.rank; c += 32) put(at(c), to_f32(src[c]) * inv * p.w[c]);
+  }
+}
+
+// ---- gather -----------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(nfk_latent_gather_params p, int elem_bytes) {
+  const int per16 = 16 / elem_bytes, chunks = static_cast<int>(p.ld) / per16;
+  const bool tiled = latent_tiled(p.dtype, p.ld, p.page_size);
+  for (int i = blockIdx.x; i < p.n_pages; i += gridDim.x) {
+    const int page = p.page_ids[i];
+    if (page < 0 || page >= p.num_pages) {
+      if (threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
+      continue;
+    }
+    for (int k = threadIdx.x; k < p.page_size * chunks; k += blockDim.x) {
+      const int r = k / chunks, ch = k % chunks;
+      const long long src = latent_offset(page, r, ch * per16, p.page_size, p.ld, tiled);
+      const long long dst = (static_cast<long long>(i) * p.page_size + r) * p.ld + ch * per16;
+      *reinterpret_cast<uint4*>(reinterpret_cast<char*>(p.out) + dst * elem_bytes) =
+          *reinterpret_cast<const uint4*>(reinterpret_cast<const char*>(p.pool) + src * elem_bytes);
+    }
   }
 }
 
@@ -63,7 +87,7 @@ __global__ void __launch_bounds__(kSimpleThreads)
 latent_attn_simple_kernel(nfk_latent_attn_params p) {
   extern __shared__ float q_s[];                      // [ld]
   __shared__ float s_s[kSimpleTile];
-  __shared__ int row_s[kSimpleTile];
+  __shared__ int row_s[kSimpleTile];                  // page * page_size + row, or -1
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int ld = static_cast<int>(p.ld);
   const T* pool = reinterpret_cast<const T*>(p.pool);
@@ -76,6 +100,8 @@ latent_attn_simple_kernel(nfk_latent_attn_params p) {
 #pragma unroll
   for (int i = 0; i < kSimpleCols; ++i) acc[i] = 0.f;
   float m = p.sinks != nullptr ? p.sinks[head] : -INFINITY, l = p.sinks != nullptr ? 1.f : 0.f;
+  const bool tiled = latent_tiled(p.dtype, p.ld, p.page_size);
+  auto at = [&](int k, int c) { return pool + latent_offset(row_s[k] / p.page_size, row_s[k] % p.page_size, c, p.page_size, ld, tiled); };
   const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
   for (int j0 = lo; j0 <= pos; j0 += kSimpleTile) {
     const int n = min(kSimpleTile, pos + 1 - j0);
@@ -89,8 +115,7 @@ latent_attn_simple_kernel(nfk_latent_attn_params p) {
     for (int k = warp; k < n; k += kSimpleThreads / 32) {
       float d = 0.f;
       if (row_s[k] >= 0) {
-        const T* c = pool + static_cast<long long>(row_s[k]) * ld;
-        for (int i = lane; i < ld; i += 32) d += q_s[i] * to_f32(c[i]);
+        for (int i = lane; i < ld; i += 32) d += q_s[i] * to_f32(*at(k, i));
       }
       d = warp_sum(d);
       if (lane == 0) s_s[k] = row_s[k] >= 0 ? d * p.scale : -INFINITY;
@@ -108,11 +133,10 @@ latent_attn_simple_kernel(nfk_latent_attn_params p) {
       if (row_s[k] < 0) continue;
       const float w = expf(s_s[k] - m);
       l += w;
-      const T* c = pool + static_cast<long long>(row_s[k]) * ld;
 #pragma unroll
       for (int i = 0; i < kSimpleCols; ++i) {
         const int col = threadIdx.x + i * kSimpleThreads;
-        if (col < ld) acc[i] += w * to_f32(c[col]);
+        if (col < ld) acc[i] += w * to_f32(*at(k, col));
       }
     }
   }
@@ -133,7 +157,7 @@ template <int DW, bool KSPLIT>
 struct LCfg {
   static constexpr int D = DW * 64;                       // latent columns
   static constexpr int ROWS = KSPLIT ? 16 : 32;           // heads per CTA, 16 per group
-  static constexpr int TILE_BYTES = kLTile * D * 2;       // [DW][64 keys][64 columns], 128-byte swizzle
+  static constexpr int TILE_BYTES = kLTile * D * 2;       // 128-byte swizzle, see key_off
   static constexpr int S_LD = kLTile + 8;
   static constexpr int S_BYTES = 4 * 16 * S_LD * 4;       // per group: score parts of the four column quarters
   static constexpr int P_BYTES = 16 * kLTile * 2;         // per group: one part (high or low)
@@ -149,9 +173,10 @@ struct LCfg {
 __device__ __forceinline__ uint32_t sw_off(int row, int ch, int row_bytes) {
   return static_cast<uint32_t>(row * row_bytes + ((ch ^ (row & 7)) << 4));
 }
-// ... in a key tile: blocks of 64 columns, 128 bytes per key.
+// ... in a key tile: pages as the pool stores them, [8-key group][64-column block][8 keys][128 bytes].
+template <int DW>
 __device__ __forceinline__ uint32_t key_off(int key, int ch) {
-  return static_cast<uint32_t>((ch >> 3) * (kLTile * 128) + key * 128 + (((ch ^ key) & 7) << 4));
+  return static_cast<uint32_t>((key >> 3) * (DW * 1024) + (ch >> 3) * 1024 + (key & 7) * 128 + (((ch ^ key) & 7) << 4));
 }
 // A fragment (16 rows x 16 k) of a row-major tile.
 __device__ __forceinline__ void load_a(uint32_t (&a)[4], uint32_t base, int row0, int ks, int row_bytes) {
@@ -230,10 +255,7 @@ latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_
     if (lane == 0) mbar_expect_tx(&full_bar[s], Cfg::TILE_BYTES);
     __syncwarp();
     if (lane < 4) {
-#pragma unroll
-      for (int b = 0; b < DW; ++b)
-        tma_load_2d(smem + s * Cfg::TILE_BYTES + b * (kLTile * 128) + lane * (kPage * 128), &tmC, &full_bar[s], b * 64,
-                    page * kPage);
+      tma_load_2d(smem + s * Cfg::TILE_BYTES + lane * (kPage * D * 2), &tmC, &full_bar[s], 0, page * (kPage * DW));
     }
   };
   if (threadIdx.x < 32) {
@@ -292,7 +314,7 @@ latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_
 #pragma unroll
         for (int g = 0; g < 2; ++g) {
           uint32_t b0, b1, b2, b3;
-          ldsm_x4(st + key_off(kh * 32 + g * 16 + (mm >> 1) * 8 + rr, (kq * DW + ks) * 2 + (mm & 1)), b0, b1, b2, b3);
+          ldsm_x4(st + key_off<DW>(kh * 32 + g * 16 + (mm >> 1) * 8 + rr, (kq * DW + ks) * 2 + (mm & 1)), b0, b1, b2, b3);
           mma_bf16(sc[2 * g], qa[ks], b0, b1);
           mma_bf16(sc[2 * g + 1], qa[ks], b2, b3);
         }
@@ -357,7 +379,7 @@ latent_attn_mma_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_
       for (int b = 0; b < DW; b += 2) {
         const int ch = min(warp * DW + b + (mm >> 1), D / 8 - 1);   // odd DW: the second half is not used
         uint32_t b0, b1, b2, b3;
-        ldsm_x4_trans(st + key_off(key, ch), b0, b1, b2, b3);
+        ldsm_x4_trans(st + key_off<DW>(key, ch), b0, b1, b2, b3);
         mma_bf16(o[b], ph, b0, b1);
         if (b + 1 < DW) mma_bf16(o[b + 1 < DW ? b + 1 : b], ph, b2, b3);
         mma_bf16(o[b], pl, b0, b1);
@@ -494,7 +516,7 @@ int launch_latent(const nfk_latent_attn_params& p, cudaStream_t stream) {
     attr = true;
   }
   CUtensorMap tm;
-  const int rc = make_tmap_bf16_2d(&tm, p.pool, static_cast<uint64_t>(p.num_pages) * kPage, Cfg::D, Cfg::D, kPage, 64);
+  const int rc = make_tmap_bf16_2d(&tm, p.pool, static_cast<uint64_t>(p.num_pages) * kPage * DW, 64, 64, kPage * DW, 64);
   if (rc != NF_OK) return rc;
   const int hgroups = (p.heads + Cfg::ROWS - 1) / Cfg::ROWS;
   const long long grid = static_cast<long long>(p.n_tokens) * p.splits * hgroups;
@@ -532,6 +554,20 @@ extern "C" int nfk_latent_append(const nfk_latent_append_params* p, cudaStream_t
   if (grid > 16 * device_sm_count()) grid = 16 * device_sm_count();
   if (p->dtype == NFK_F32) latent_append_kernel<float><<<grid, 128, 0, stream>>>(*p);
   else latent_append_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(*p);
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+extern "C" int nfk_latent_gather(const nfk_latent_gather_params* p, cudaStream_t stream) {
+  using namespace nf;
+  if (p == nullptr) return NF_ERR_BAD_ARG;
+  if (p->n_pages == 0) return NF_OK;
+  const int es = p->dtype == NFK_F32 ? 4 : 2;
+  if (!p->pool || !p->out || !p->page_ids || p->n_pages < 0 || p->page_size <= 0 || p->num_pages <= 0 || p->ld <= 0 ||
+      p->ld * es % 16 != 0 || (reinterpret_cast<uintptr_t>(p->pool) & 15) != 0 || (reinterpret_cast<uintptr_t>(p->out) & 15) != 0)
+    return NF_ERR_BAD_ARG;
+  int grid = 8 * device_sm_count();
+  if (grid > p->n_pages) grid = p->n_pages;
+  latent_gather_kernel<<<grid, 256, 0, stream>>>(*p, es);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 

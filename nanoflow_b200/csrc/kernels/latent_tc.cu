@@ -7,7 +7,7 @@
 // A CTA takes one token, 32 of its heads and a range of keys, in tiles of 64 keys (whole pages, by TMA). P^T has 64
 // columns: the high bf16 parts of the 32 heads' probabilities and their low parts, which go to columns of their own
 // and are added at the end, so the second product keeps about 16 bits without a second pass over the tile.
-// Rows 64-127 of the score product read whatever follows the tile's column block; nobody looks at them.
+// Rows 64-127 of the score product read whatever follows the tile; nobody looks at them.
 //
 // Roles (12 warps): 0, 1 and 4, 5 softmax of 16 heads each, one thread per key (TMEM lanes 0-63; maxima over keys by
 // shuffles, the reference maximum of a head moves only when it is outgrown by 2^8); 2 MMA issue and TMEM; 3 TMA;
@@ -24,16 +24,19 @@ constexpr float kGap = 8.f;
 
 template <int D>
 struct TcCfg {
-  static constexpr int BLK = kTile * 128;                 // one block of 64 columns of a key tile
-  static constexpr int TILE = D / 64 * BLK;
-  static constexpr int STAGES = D <= 256 ? 4 : 2;
+  // a key tile holds pages as the pool stores them: [8-key group][64-column block][8 keys][128 bytes]
+  static constexpr int BLK = 1024, GRP = D / 64 * BLK;
+  static constexpr int TILE = kTile / 8 * GRP;
+  static constexpr int STAGES = D <= 256 ? 4 : (D == 384 ? 3 : 2);
   static constexpr int QBLK = kHeads * 128;
   static constexpr int Q_OFF = STAGES * TILE;
   static constexpr int P_OFF = Q_OFF + D / 64 * QBLK;     // two buffers [64 keys][64]
   static constexpr int F_OFF = P_OFF + 2 * kTile * 128;
   // fp32: maxima [2 groups][2 warps][16], alpha [2 parities][32], l [2 groups][2 warps][16], inverse [32], m [32]
   static constexpr int BAR_OFF = F_OFF + (64 + 64 + 64 + 64) * 4;
-  static constexpr int SMEM = BAR_OFF + 256 + 1024;
+  // rows 64-127 of the last stage's score product read one tile further: that has to be shared memory, too
+  static constexpr int END = BAR_OFF + 256 > (STAGES + 1) * TILE ? BAR_OFF + 256 : (STAGES + 1) * TILE;
+  static constexpr int SMEM = END + 1024;
   static constexpr int O_COL = 64;                        // TMEM: S^T of even / odd tiles, then O^T blocks of 64
   static constexpr int NCB = D / 128;
   static constexpr int TMEM_COLS = O_COL + NCB * 64 <= 128 ? 128 : (O_COL + NCB * 64 <= 256 ? 256 : 512);
@@ -41,6 +44,17 @@ struct TcCfg {
 
 enum TBar : int { FULL0 = 0, EMPTY0 = 4, S_FULL0 = 8, P_FULL0 = 10, CORR0 = 12, PV0 = 14, NUM_TBARS = 16 };
 
+// K-major operand in the 128-byte swizzle, `sbo` bytes between groups of eight rows.
+__device__ __forceinline__ uint64_t desc_k(uint32_t addr, uint32_t sbo) {
+  uint64_t d = 0;
+  d |= static_cast<uint64_t>((addr & 0x3FFFF) >> 4);
+  d |= static_cast<uint64_t>(1) << 16;
+  d |= static_cast<uint64_t>((sbo >> 4) & 0x3FFF) << 32;
+  d |= static_cast<uint64_t>(1) << 46;
+  d |= static_cast<uint64_t>(2) << 61;
+  return d;
+}
+// MN-major operand: `lbo` bytes between blocks of 64 along M / N, `sbo` between groups of eight k indices.
 __device__ __forceinline__ uint64_t desc_mn(uint32_t addr, uint32_t lbo, uint32_t sbo) {
   uint64_t d = 0;
   d |= static_cast<uint64_t>((addr & 0x3FFFF) >> 4);
@@ -166,9 +180,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_p
           report_status(p.status, NF_ST_BAD_INDEX);
           page = 0;
         }
-#pragma unroll
-        for (int b = 0; b < D / 64; ++b)
-          tma_load_2d(smem + s * C::TILE + b * C::BLK + lane * (kPage * 128), &tmC, &bars[FULL0 + s], b * 64, page * kPage);
+        tma_load_2d(smem + s * C::TILE + lane * (kPage * D * 2), &tmC, &bars[FULL0 + s], 0, page * (kPage * D / 64));
       }
       ++issued;
     }
@@ -187,7 +199,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_p
         const uint32_t kb = sb + s * C::TILE;
 #pragma unroll 8
         for (int k = 0; k < D / 16; ++k)
-          umma_bf16_ss(tmem + (t & 1) * kHeads, umma_desc_k_sw128(kb + (k >> 2) * C::BLK + (k & 3) * 32),
+          umma_bf16_ss(tmem + (t & 1) * kHeads, desc_k(kb + (k >> 2) * C::BLK + (k & 3) * 32, C::GRP),
                        umma_desc_k_sw128(sb + C::Q_OFF + (k >> 2) * C::QBLK + (k & 3) * 32), idesc_s, k ? 1u : 0u);
         umma_commit(&bars[S_FULL0 + (t & 1)]);
         return true;
@@ -204,8 +216,8 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tmC, nfk_latent_attn_p
         for (int cb = 0; cb < C::NCB; ++cb)
 #pragma unroll
           for (int k = 0; k < kTile / 16; ++k)
-            umma_bf16_ss(tmem + C::O_COL + cb * (2 * kHeads), desc_mn(kb + 2 * cb * C::BLK + k * 2048, C::BLK, 1024),
-                         desc_mn(pb + k * 2048, C::BLK, 1024), idesc_o, (t | k) ? 1u : 0u);
+            umma_bf16_ss(tmem + C::O_COL + cb * (2 * kHeads), desc_mn(kb + 2 * cb * C::BLK + k * 2 * C::GRP, C::BLK, C::GRP),
+                         desc_mn(pb + k * 2048, 8192, 1024), idesc_o, (t | k) ? 1u : 0u);
         umma_commit(&bars[EMPTY0 + s]);
         umma_commit(&bars[PV0 + par]);
       }
@@ -379,7 +391,7 @@ int launch(const nfk_latent_attn_params& p, cudaStream_t stream) {
     attr = true;
   }
   CUtensorMap tm;
-  const int rc = make_tmap_bf16_2d(&tm, p.pool, static_cast<uint64_t>(p.num_pages) * kPage, D, D, kPage, 64);
+  const int rc = make_tmap_bf16_2d(&tm, p.pool, static_cast<uint64_t>(p.num_pages) * kPage * (D / 64), 64, 64, kPage * (D / 64), 64);
   if (rc != NF_OK) return rc;
   const long long grid = static_cast<long long>(p.n_tokens) * p.splits * ((p.heads + kHeads - 1) / kHeads);
   if (grid > 0x7fffffffll) return NF_ERR_BAD_ARG;

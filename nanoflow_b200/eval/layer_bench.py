@@ -121,8 +121,8 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
         return 0.0, T * p.rank * 2 * es
     if isinstance(p, G.RopeAppendParams):
         return 0.0, T * (2 * p.q_heads + 4 * p.kv_heads) * p.head_dim * es
-    if isinstance(p, G.KvMoveParams):
-        return 0.0, 2.0 * engine._last_sym.get(dict(op.dyn)["n_pages"], 0) * p.page_bytes
+    if isinstance(p, G.LatentGatherParams):
+        return 0.0, 2.0 * engine._last_sym.get(dict(op.dyn)["n_pages"], 0) * p.page_size * p.ld * es
     if isinstance(p, G.NormParams):
         return 0.0, 2 * T * p.cols * es
     return 0.0, 0.0

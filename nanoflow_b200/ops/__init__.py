@@ -103,6 +103,11 @@ class LatentAppendParams(Structure):
                 ("eps", c_float), ("dtype", c_int), ("status", c_void_p)]
 
 
+class LatentGatherParams(Structure):
+    _fields_ = [("pool", c_void_p), ("out", c_void_p), ("page_ids", c_void_p), ("ld", c_longlong), ("n_pages", c_int),
+                ("page_size", c_int), ("num_pages", c_int), ("dtype", c_int), ("status", c_void_p)]
+
+
 class LatentAttnParams(Structure):
     _fields_ = [("q", c_void_p), ("ld_q", c_longlong), ("pool", c_void_p), ("ld", c_longlong), ("out", c_void_p),
                 ("ld_out", c_longlong), ("tokens", c_void_p), ("positions", c_void_p), ("token_req", c_void_p),

@@ -11,7 +11,7 @@ from typing import Optional
 import torch
 
 from . import (ACTS, NORMS, AttnParams, GemmParams, HeadNormGateParams, LatentAppendParams, LatentAttnParams, MlstmParams,
-               ResidualNormParams, _check, _i32, _p, _stream, dtype_code, lib)
+               ResidualNormParams, LatentGatherParams, _check, _i32, _p, _stream, dtype_code, lib)
 
 
 def _f32(t: Optional[torch.Tensor], name: str) -> None:
@@ -85,6 +85,33 @@ def latent_append(src, w, pool, positions, token_req, kv_indptr, kv_indices, kv_
                            page_size=pool.shape[1], num_pages=pool.shape[0], eps=eps, dtype=dtype_code(pool.dtype),
                            status=_p(status))
     _check(lib().nfk_latent_append(byref(p), _stream()), "nfk_latent_append")
+
+
+def pool_to_rows(pool: torch.Tensor) -> torch.Tensor:
+    """A latent pool [pages, page size, row size] as plain rows in the same shape: bf16 pages whose row size is a multiple
+    of 64 are stored in tiles of 8 rows x 64 columns (see kernels.h)."""
+    n, ps, ld = pool.shape
+    if pool.dtype != torch.bfloat16 or ld % 64 or ps % 8:
+        return pool
+    return pool.reshape(n, ps // 8, ld // 64, 8, 64).permute(0, 1, 3, 2, 4).reshape(n, ps, ld)
+
+
+def rows_to_pool(rows: torch.Tensor) -> torch.Tensor:
+    """The inverse of :func:`pool_to_rows`."""
+    n, ps, ld = rows.shape
+    if rows.dtype != torch.bfloat16 or ld % 64 or ps % 8:
+        return rows
+    return rows.reshape(n, ps // 8, 8, ld // 64, 64).permute(0, 1, 3, 2, 4).reshape(n, ps, ld)
+
+
+def latent_gather(pool: torch.Tensor, page_ids: torch.Tensor, status=None) -> torch.Tensor:
+    """Pages of a latent pool as plain rows [n * page size, row size]."""
+    _i32(page_ids, "page_ids")
+    out = torch.zeros(page_ids.numel() * pool.shape[1], pool.shape[2], dtype=pool.dtype, device=pool.device)
+    p = LatentGatherParams(pool=_p(pool), out=_p(out), page_ids=_p(page_ids), ld=pool.shape[2], n_pages=page_ids.numel(),
+                           page_size=pool.shape[1], num_pages=pool.shape[0], dtype=dtype_code(pool.dtype), status=_p(status))
+    _check(lib().nfk_latent_gather(byref(p), _stream()), "nfk_latent_gather")
+    return out
 
 
 def latent_attention(q, pool, out, tokens, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, heads: int,

@@ -84,6 +84,7 @@ AttnParams = _ops.AttnParams
 ResidualNormParams = _ops.ResidualNormParams
 LatentAppendParams = _ops.LatentAppendParams
 LatentAttnParams = _ops.LatentAttnParams
+LatentGatherParams = _ops.LatentGatherParams
 MlstmParams = _ops.MlstmParams
 HeadNormGateParams = _ops.HeadNormGateParams
 
@@ -93,7 +94,7 @@ KERNEL_OF = {
     EmbeddingParams: "nfk_embedding_p", GatherParams: "nfk_gather_p", ArgmaxParams: "nfk_argmax_p",
     ArgmaxCombineParams: "nfk_argmax_combine_p", CopyColsParams: "nfk_copy_cols_p",
     ResidualNormParams: "nfk_residual_norm", LatentAppendParams: "nfk_latent_append",
-    LatentAttnParams: "nfk_latent_attn", HeadNormGateParams: "nfk_head_norm_gate",
+    LatentGatherParams: "nfk_latent_gather", LatentAttnParams: "nfk_latent_attn", HeadNormGateParams: "nfk_head_norm_gate",
     MemcpyParams: "nfk_memcpy_p", Memcpy2DParams: "nfk_memcpy2d_p", KvMoveParams: "nfk_kv_move_p", SleepParams: "nfk_sleep_p",
 }
 

@@ -31,8 +31,8 @@ from ..ops import ACTS, NORMS, dtype_code
 from ..ops.layer_list import mlstm_scratch_floats
 from ..serving.scheduler import BatchPlan
 from .engine import GEMM_WS_BYTES, Engine, MetaLayout
-from .graph import (ArgmaxParams, AttnParams, GemmParams, HeadNormGateParams, KvMoveParams, LatentAppendParams,
-                    LatentAttnParams, MemcpyParams, MlstmParams, OpGraph, ResidualNormParams)
+from .graph import (ArgmaxParams, AttnParams, GemmParams, HeadNormGateParams, LatentAppendParams,
+                    LatentAttnParams, LatentGatherParams, MemcpyParams, MlstmParams, OpGraph, ResidualNormParams)
 from .pipeline import _ptr
 
 PAGE = 16
@@ -325,9 +325,8 @@ class LayerListEngine(Engine):
             n_x = g.symbol(pg.name("n_xpages"))
             kv_cols = H * 2 * PREFILL_HEAD_DIM
             cg, kv = self.view("cg", ld, self.x_pages * PAGE), self.view("kv", kv_cols, self.x_pages * PAGE)
-            mp = KvMoveParams(pool=_ptr(pool), staging=_ptr(cg), page_ids=_ptr(meta[pg.name("xpage")]), n_pages=0,
-                              page_bytes=PAGE * ld * pool.element_size(), num_pages=self.num_pages, direction=0,
-                              num_ctas=8 * ops.sm_count(self.device), status=st)
+            mp = LatentGatherParams(pool=_ptr(pool), out=_ptr(cg), page_ids=_ptr(meta[pg.name("xpage")]), ld=ld, n_pages=0,
+                                    page_size=PAGE, num_pages=self.num_pages, dtype=self.code, status=st)
             self._op(f"R{r}.latent_gather", mp, dyn=[("n_pages", n_x)], layer=r)
             self._gemm(f"R{r}.expand", cg, lw.w_kv, kv, rows=g.symbol(pg.name("x_rows")), layer=r)
             pp = AttnParams()

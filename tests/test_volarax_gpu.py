@@ -141,11 +141,13 @@ class Paged:
     def fill(self, b, rows):
         ids = torch.as_tensor(self.page_rows[b].astype(np.int64)).cuda()
         pos = torch.arange(rows.shape[0], device="cuda")
-        self.pool[ids[pos // 16], pos % 16] = rows.to(self.pool.dtype)
+        plain = K.pool_to_rows(self.pool).clone()
+        plain[ids[pos // 16], pos % 16] = rows.to(self.pool.dtype)
+        self.pool.copy_(K.rows_to_pool(plain))
 
 
 @pytest.mark.parametrize("dtype", BOTH)
-@pytest.mark.parametrize("rank", [13, 64, 200])
+@pytest.mark.parametrize("rank", [13, 64, 190, 200])
 def test_latents_are_normed_into_their_page_slots(dtype, rank):
     ld = (rank + 7) // 8 * 8
     pg = Paged([40, 20], ld, dtype, first=[1, 0])
@@ -156,9 +158,12 @@ def test_latents_are_normed_into_their_page_slots(dtype, rank):
     K.latent_append(src, w, pg.pool, i32(pos), i32(req), pg.indptr, pg.indices, pg.kv_first, rank=rank, eps=1e-3, status=st)
     ops.check_status(st)
     want = oracle.rms_norm(src.double()[:, :rank], 1e-3, w.double())
-    got = torch.stack([pg.pool[pg.page_rows[r][p // 16], p % 16] for p, r in zip(pos, req)])
+    plain = K.pool_to_rows(pg.pool)
+    got = torch.stack([plain[pg.page_rows[r][p // 16], p % 16] for p, r in zip(pos, req)])
     assert rel(got[:, :rank], want) < TOL[dtype] * 2 and (got[:, rank:] == 0).all()
     assert pg.pool.count_nonzero() <= 7 * rank
+    ids = i32(pg.page_rows[0][::-1].copy())
+    assert torch.equal(K.latent_gather(pg.pool, ids), plain[ids.long()].reshape(-1, ld))
 
 
 def latent_case(dtype, impl, heads, ld, window, scale, positions, lens, splits=1, sink_value=None, standout=(), first=None,
