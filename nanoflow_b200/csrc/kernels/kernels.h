@@ -304,8 +304,8 @@ typedef struct nfk_latent_attn_params {
   int n_tokens, heads, page_size, num_pages, window;
   float scale;
   int dtype;
-  int impl;                  // 0 = choose, 1 = simple kernel, 2 = mma.sync kernel (bf16), 3 = tcgen05 kernel (bf16)
-  int splits;                // tensor-core kernels: key ranges per token, > 1 needs a workspace
+  int impl;                  // 0 = choose, 1 = simple kernel, 2 = tensor-core kernel (bf16)
+  int splits;                // tensor-core kernel: key ranges per token, > 1 needs a workspace
   float* workspace;          // [n_tokens][splits][heads][ld + 2] fp32
   long long workspace_floats;
   unsigned int* status;

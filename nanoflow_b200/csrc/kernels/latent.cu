@@ -7,8 +7,7 @@
 //                     key matrices, so the cached row is key and value at once), sliding window, sink.
 //                     Used for decoding, for prompt tokens whose keys are not expanded, and in 32-bit.
 //
-// Three kernels for the attention. latent_tc.cu (bf16, row sizes that are multiples of 128) runs on tcgen05. The
-// mma.sync one (bf16, the other row sizes): a CTA takes one token, 16 or 32 of its heads (the
+// Two kernels for the attention. The tensor-core one (bf16): a CTA takes one token, 16 or 32 of its heads (the
 // rows of its MMA tiles) and a range of keys; every latent row is fetched once for all those heads, in whole
 // pages by TMA. Two groups of eight warps work on 16 heads each (or on alternate key tiles of the same heads),
 // so that one group's softmax runs under the other's products. Per tile of 64 keys a group first splits the
@@ -17,7 +16,6 @@
 // low part), which keeps them to about 16 bits. The simple one (bf16 or fp32, any size): one CTA per token and head.
 #include "attn_mma.cuh"
 #include "elem_io.cuh"
-#include "latent_tc.h"
 
 namespace nf {
 namespace {
@@ -581,19 +579,12 @@ extern "C" int nfk_latent_attn(const nfk_latent_attn_params* pp, cudaStream_t st
       p.num_pages <= 0 || p.window < 0)
     return NF_ERR_BAD_ARG;
   if (p.splits < 1) p.splits = 1;
-  if (p.impl < 0 || p.impl > 3) return NF_ERR_BAD_ARG;
-  if (p.impl >= 2 && !mma_ok(p)) return NF_ERR_UNSUPPORTED;
-  if (p.impl == 3 && !latent_tc_built(p.ld)) return NF_ERR_UNSUPPORTED;
+  if (p.impl < 0 || p.impl > 2) return NF_ERR_BAD_ARG;
+  if (p.impl == 2 && !mma_ok(p)) return NF_ERR_UNSUPPORTED;
   if (p.impl != 1 && mma_ok(p)) {
     if (p.splits > 1 && (p.workspace == nullptr || static_cast<long long>(p.n_tokens) * p.splits * p.heads * (p.ld + 2) >
                                                        p.workspace_floats))
       p.splits = 1;
-    if (p.impl != 2 && latent_tc_built(p.ld)) {
-      const int rc = latent_tc_launch(p, stream);
-      if (rc != NF_OK || p.splits == 1) return rc;
-      latent_attn_merge_kernel<<<p.n_tokens * p.heads, 128, 0, stream>>>(p);
-      return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
-    }
     switch (p.ld / 64) {
       case 1: return launch_latent_mt<1>(p, stream);
       case 2: return launch_latent_mt<2>(p, stream);

@@ -199,7 +199,7 @@ def latent_case(dtype, impl, heads, ld, window, scale, positions, lens, splits=1
 
 
 VARIANTS = [(torch.float32, 1, 40), (torch.bfloat16, 1, 72), (torch.bfloat16, 2, 64), (torch.bfloat16, 2, 192),
-            (torch.bfloat16, 2, 512), (torch.bfloat16, 3, 128), (torch.bfloat16, 3, 384), (torch.bfloat16, 3, 512)]
+            (torch.bfloat16, 2, 384), (torch.bfloat16, 2, 512)]
 
 
 @pytest.mark.parametrize("dtype,impl,ld", VARIANTS)
@@ -245,13 +245,13 @@ def test_latent_attention_sinks_take_their_share(dtype, impl, ld):
     assert rel(got, want) < TOL[dtype] * 3 and rel(none, want) > 0.2
 
 
-@pytest.mark.parametrize("impl,ld,heads", [(2, 64, 4), (2, 256, 20), (3, 256, 20), (3, 512, 33)])
+@pytest.mark.parametrize("ld,heads", [(64, 4), (256, 20), (512, 33)])
 @pytest.mark.parametrize("splits", [2, 3, 7])
-def test_latent_attention_split_over_key_ranges(impl, ld, heads, splits):
+def test_latent_attention_split_over_key_ranges(ld, heads, splits):
     lens = [30, 700, 65]
     pos = [(0, 29), (1, 699), (1, 64), (2, 64), (2, 0)]
     for window in (0, 100):
-        got, want = latent_case(torch.bfloat16, impl, heads, ld, window, ld ** -0.5, pos, lens, splits=splits, sink_value=0.5)
+        got, want = latent_case(torch.bfloat16, 2, heads, ld, window, ld ** -0.5, pos, lens, splits=splits, sink_value=0.5)
         assert rel(got, want) < TOL[torch.bfloat16] * 3
 
 
@@ -633,7 +633,7 @@ def test_greedy_generation_in_bf16_stays_near_the_oracle_arg_max():
 
 def test_latent_attention_maxima_that_keep_growing():
     """Scores that rise from tile to tile, far beyond what exponentials of the first reference maximum could hold."""
-    for impl in (2, 3):
+    for impl in (1, 2):
         ld, heads, n = 256, 5, 400
         pg = Paged([n], ld, torch.bfloat16)
         lat = rnd(n, ld, seed=1, dtype=torch.bfloat16)
