@@ -224,8 +224,12 @@ def parse_config(raw: Dict[str, Any], *, tp: Optional[int] = None) -> NanoflowCo
     mc, pc, sc = raw["model_configs"], raw["pipeline_configs"], raw["serve_configs"]
     gpu_num = int(mc.get("gpu_num", 1))
     actual = int(sc.get("actual_gpu_num", gpu_num))
-    from .models.registry import family_of
+    from .models.registry import family_of, is_model_folder
     fam = family_of(raw["model"])
+    if fam.complete is not None:
+        folder = next((p for p in (sc.get("hf_path", ""), sc.get("weight_path", "")) if p and Path(p).is_dir() and is_model_folder(p)), "")
+        if folder:
+            raw = dict(raw, model=fam.complete(raw["model"], folder))
     model = fam.parse_model(raw["model"], tp=tp or gpu_num, run_layers=int(mc.get("run_layer", 0)),
                             name=sc.get("model", ""))
     ptype = sc.get("pipeline_type", "NON_OVERLAP_LOCAL" if fam.listed_layers else "PLLM")
@@ -339,6 +343,11 @@ def _volarax(*a, **kw):
     return builtin(*a, **kw)
 
 
+def _zubedra(*a, **kw):
+    from .models.zubedra import builtin
+    return builtin(*a, **kw)
+
+
 _LLAMA31_SCALING = {"factor": 8.0, "low_freq_factor": 1.0, "high_freq_factor": 4.0,
                     "original_max_position_embeddings": 8192, "rope_type": "llama3"}
 
@@ -367,6 +376,13 @@ MODEL_ARCHS: Dict[str, Dict[str, Any]] = {
                            m_heads=8, m_dim=256, m_vdim=512, ff=14336, m_ff=14336),
     "volarax-2B": _volarax(2048, 32000, "am" * 12, heads=16, dim=128, vdim=128, kv_rank=256, window=512,
                            m_heads=4, m_dim=256, m_vdim=512, ff=8192, m_ff=8192),
+    # named by what a token uses: the experts' feed-forwards add up to those of the dense models of that size
+    "zubedra-tiny": _zubedra(200, 1000, "awaw", heads=6, kv_heads=2, dim=40, vdim=24, softcap=20.0, w_heads=3, w_dim=24,
+                             rank=12, experts=12, top=3, ff=40, groups=3, keep=2, shared_ff=72),
+    "zubedra-8B": _zubedra(4096, 128256, "aw" * 16, heads=32, kv_heads=8, dim=128, vdim=128, softcap=50.0, w_heads=64,
+                           w_dim=64, rank=128, experts=64, top=6, ff=2048, groups=8, keep=4, shared_ff=2048),
+    "zubedra-2B": _zubedra(2048, 32000, "aw" * 12, heads=16, kv_heads=4, dim=128, vdim=128, softcap=50.0, w_heads=32,
+                           w_dim=64, rank=64, experts=64, top=6, ff=1024, groups=8, keep=4, shared_ff=2048),
 }
 
 MODEL_IDS = {
@@ -375,7 +391,7 @@ MODEL_IDS = {
     "llama3.1-8B": "meta-llama/Meta-Llama-3.1-8B-Instruct", "qwen2-72B": "Qwen/Qwen2-72B-Instruct",
     "deepseek-67B": "deepseek-ai/deepseek-llm-67b-chat", "mixtral-8-7B": "mistralai/Mixtral-8x7B-Instruct-v0.1",
     "tiny": "nanoflow/tiny-llama-test", "tiny8": "nanoflow/tiny8-llama-test",
-    "volarax-tiny": "nanoflow/volarax-tiny-test",
+    "volarax-tiny": "nanoflow/volarax-tiny-test", "zubedra-tiny": "nanoflow/zubedra-tiny-test",
 }
 
 

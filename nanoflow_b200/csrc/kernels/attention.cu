@@ -69,6 +69,28 @@ __device__ __forceinline__ void pv_16tok(float (&o)[HD / 8][4], const uint32_t (
   }
 }
 
+// The same with P as a bf16 pair.
+template <int HD>
+__device__ __forceinline__ void pv_16tok_pair(float (&o)[HD / 8][4], const uint32_t (&pa)[4], const uint32_t (&pl)[4],
+                                              uint32_t v_base, int row0) {
+  const int lane = threadIdx.x & 31;
+  const int m = lane >> 3, r = lane & 7;
+  const int tok = row0 + (m & 1) * 8 + r;
+#pragma unroll
+  for (int c = 0; c < HD / 8; c += 2) {
+    uint32_t b0, b1, b2, b3;
+    ldsm_x4_trans(v_base + tile_off<HD>(tok, c + (m >> 1)), b0, b1, b2, b3);
+    mma_bf16(o[c], pa, b0, b1);
+    mma_bf16(o[c + 1], pa, b2, b3);
+    mma_bf16(o[c], pl, b0, b1);
+    mma_bf16(o[c + 1], pl, b2, b3);
+  }
+}
+// tanh x = 1 - 2 / (e^(2x) + 1): within a few 1e-7 absolute everywhere, and +-1 at the far ends.
+__device__ __forceinline__ float tanh_by_exp(float x) {
+  return 1.f - __fdividef(2.f, fast_exp2(x * (2.f * kLog2e)) + 1.f);
+}
+
 // ================================================================================================
 // Decode
 // ================================================================================================
@@ -94,8 +116,9 @@ struct DecCfg {
 constexpr int kDecodeCounterSlots = 64;
 __device__ unsigned int g_decode_counters[kDecodeCounterSlots][2];
 
-template <int HD, int ST>
-__global__ void __launch_bounds__(kDecThreads, 3)
+// EXT: sink in the denominator, capped scores, probabilities as a bf16 pair (in an instantiation of its own).
+template <int HD, int ST, bool EXT>
+__global__ void __launch_bounds__(kDecThreads, EXT ? 2 : 3)
 attn_decode_kernel(nfk_attn_params p, int slot) {
   using Cfg = DecCfg<HD, ST>;
   constexpr int kDecStages = ST;
@@ -183,6 +206,14 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
       const int pslot = c_begin + warp + 4 * i;
       const int valid = (pslot == np - 1) ? last_len : kPage;
       const int c0 = (lane & 3) * 2;
+      if (EXT && p.softcap > 0.f) {
+        const float cap_in = p.sm_scale / p.softcap, cap_out = p.softcap / p.sm_scale;   // `scale` follows below
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          s0[e] = cap_out * tanh_by_exp(s0[e] * cap_in);
+          s1[e] = cap_out * tanh_by_exp(s1[e] * cap_in);
+        }
+      }
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         s0[e] = (c0 + (e & 1) < valid) ? s0[e] * scale : -INFINITY;
@@ -211,7 +242,17 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
       pa[1] = pack_bf16x2(pr[2], pr[3]);
       pa[2] = pack_bf16x2(pr[4], pr[5]);
       pa[3] = pack_bf16x2(pr[6], pr[7]);
-      pv_16tok<HD>(o, pa, st + Cfg::PAGE_BYTES, 0);
+      if (EXT) {
+        uint32_t pl[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 h = unpack_bf16x2(pa[j]);
+          pl[j] = pack_bf16x2(pr[2 * j] - h.x, pr[2 * j + 1] - h.y);
+        }
+        pv_16tok_pair<HD>(o, pa, pl, st + Cfg::PAGE_BYTES, 0);
+      } else {
+        pv_16tok<HD>(o, pa, st + Cfg::PAGE_BYTES, 0);
+      }
       __syncwarp();
       issue(i + kDecStages - 1);
     }
@@ -254,8 +295,10 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
         x += v.x * sc;
         y += v.y * sc;
       }
-      const float inv = L > 0.f ? 1.f / L : 0.f;
       const int head = kvh * group + r;
+      // a far larger sink makes the sum infinite and the row zero, as it should be; with several chunks the merge adds it
+      if (EXT && p.sinks != nullptr && n_chunks == 1) L += fast_exp2(p.sinks[head] * kLog2e - msafe);
+      const float inv = L > 0.f ? 1.f / L : 0.f;
       if (n_chunks == 1) {
         *reinterpret_cast<uint32_t*>(outp + (static_cast<long long>(tok) * p.q_heads + head) * HD + c) =
             pack_bf16x2(x * inv, y * inv);
@@ -295,8 +338,9 @@ __global__ void attn_decode_merge_kernel(nfk_attn_params p) {
   const float msafe = mm == -INFINITY ? 0.f : mm;
   const int tok = p.qo_indptr[req];
   __nv_bfloat16* outp = reinterpret_cast<__nv_bfloat16*>(p.out);
+  const float sink = p.sinks != nullptr ? fast_exp2(p.sinks[head] * kLog2e - msafe) : 0.f;
   for (int d = threadIdx.x; d < HD; d += blockDim.x) {
-    float acc = 0.f, W = 0.f;
+    float acc = 0.f, W = sink;
     for (int c = 0; c < n_chunks; ++c) {
       const float w = exp2f(ws[c * (HD + 2) + HD] - msafe);
       W += w;
@@ -477,26 +521,29 @@ attn_prefill_kernel(nfk_attn_params p) {
 
 inline int sm_count_attn() { return device_sm_count(); }
 
-int check_common(const nfk_attn_params* p) {
+bool decode_ext(const nfk_attn_params& p) { return p.sinks != nullptr || p.softcap > 0.f || p.precise != 0; }
+
+int check_common(const nfk_attn_params* p, bool decode = false) {
   if (p == nullptr) return NF_ERR_BAD_ARG;
   if (!p->q || !p->out || !p->kv_pool || !p->qo_indptr || !p->kv_indptr || !p->kv_indices ||
       !p->kv_last_page_len)
     return NF_ERR_BAD_ARG;
   if (p->kv_heads <= 0 || p->q_heads % p->kv_heads != 0) return NF_ERR_BAD_ARG;
   const int group = p->q_heads / p->kv_heads;
-  if (group > 16 || (16 % group) != 0) return NF_ERR_UNSUPPORTED;
-  if (p->page_size != kPage) return NF_ERR_UNSUPPORTED;
+  // the extended decode kernel takes any number of query heads that fits its 16-row tile
+  if (group > 16 || ((16 % group) != 0 && !(decode && decode_ext(*p)))) return NF_ERR_UNSUPPORTED;
+  if (p->page_size != kPage || p->softcap < 0.f || (!decode && (p->sinks != nullptr || p->softcap > 0.f))) return NF_ERR_UNSUPPORTED;
   if (p->head_dim != 128 && p->head_dim != 64) return NF_ERR_UNSUPPORTED;
   return NF_OK;
 }
 
-template <int HD, int ST>
+template <int HD, int ST, bool EXT>
 int launch_decode_st(const nfk_attn_params* p, cudaStream_t stream) {
   using Cfg = DecCfg<HD, ST>;
   static bool attr_dev[kMaxDevices] = {false};   // the attribute is per device
   bool& attr = attr_dev[device_slot()];
   if (!attr) {
-    if (cudaFuncSetAttribute(attn_decode_kernel<HD, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attn_decode_kernel<HD, ST, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              Cfg::SMEM_BYTES) != cudaSuccess)
       return NF_ERR_CUDA;
     attr = true;
@@ -507,7 +554,7 @@ int launch_decode_st(const nfk_attn_params* p, cudaStream_t stream) {
   if (ctas > total) ctas = total;
   static std::atomic<unsigned int> launch_seq{0};
   const int slot = static_cast<int>(launch_seq.fetch_add(1u) % kDecodeCounterSlots);
-  attn_decode_kernel<HD, ST><<<static_cast<int>(ctas), kDecThreads, Cfg::SMEM_BYTES, stream>>>(*p, slot);
+  attn_decode_kernel<HD, ST, EXT><<<static_cast<int>(ctas), kDecThreads, Cfg::SMEM_BYTES, stream>>>(*p, slot);
   if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
   if (p->chunk_pages > 0 && max_chunks > 1) {
     attn_decode_merge_kernel<HD><<<p->req_count * p->q_heads, HD, 0, stream>>>(*p);
@@ -518,7 +565,9 @@ int launch_decode_st(const nfk_attn_params* p, cudaStream_t stream) {
 
 template <int HD>
 int launch_decode(const nfk_attn_params* p, cudaStream_t stream) {
-  return p->decode_stages == 2 ? launch_decode_st<HD, 2>(p, stream) : launch_decode_st<HD, 3>(p, stream);
+  if (decode_ext(*p))
+    return p->decode_stages == 2 ? launch_decode_st<HD, 2, true>(p, stream) : launch_decode_st<HD, 3, true>(p, stream);
+  return p->decode_stages == 2 ? launch_decode_st<HD, 2, false>(p, stream) : launch_decode_st<HD, 3, false>(p, stream);
 }
 
 template <int HD>
@@ -544,7 +593,7 @@ int launch_prefill(const nfk_attn_params* p, cudaStream_t stream) {
 
 extern "C" int nfk_attn_decode(const nfk_attn_params* p, cudaStream_t stream) {
   using namespace nf;
-  const int rc = check_common(p);
+  const int rc = check_common(p, true);
   if (rc != NF_OK) return rc;
   if (p->req_count == 0) return NF_OK;
   if (p->req_count < 0 || p->req_begin < 0) return NF_ERR_BAD_ARG;
@@ -587,7 +636,7 @@ int static_scratch_for_current_device(float** out) {
 
 extern "C" int nfk_attn_decode_static(const nfk_attn_params* p, cudaStream_t stream) {
   using namespace nf;
-  const int rc = check_common(p);
+  const int rc = check_common(p, true);
   if (rc != NF_OK) return rc;
   if (p->req_count == 0) return NF_OK;
   if (p->req_count < 0 || p->req_begin < 0 || p->chunk_pages < 0) return NF_ERR_BAD_ARG;

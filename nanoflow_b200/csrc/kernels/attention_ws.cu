@@ -29,7 +29,7 @@
 // the first row's window are never loaded), a sink in the softmax denominator, K / V as columns of plain
 // rows instead of pool pages (keys expanded from a latent cache), and probabilities that enter the second
 // product as a bf16 pair: the high parts over the first half of the S accumulator, the low parts over the
-// second half.
+// second half. CAP adds capped scores (cap tanh(score / cap)); with either, head_dim 64 is built as well.
 //
 // Takes the place of the reference's FlashInfer BatchPrefillWithPagedKVCacheKernel
 // (gemv/include/attention/prefill.cuh:1066-1374, mma.sync m16n16k16 + ldmatrix on sm_80).
@@ -39,21 +39,25 @@
 namespace nf {
 namespace {
 
-constexpr int HD = 128;
 constexpr int kPage = 16;
 constexpr int kTile = 64;             // kv tokens per tile
 constexpr int kThreads = 192;         // warps 0-3 softmax (TMEM lane quarter = warp index), 4 loads, 5 MMA
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kRescaleGap = 8.0f;   // log2 of how far a row maximum may outgrow its reference
 
-// shared-memory map (bytes from the 1024-aligned base); every operand region is 1024-aligned
-constexpr int Q_OFF = 0;                       // 2 halves x [128 rows][64 hd]                 32 KB
-constexpr int K_OFF = 32768;                   // 2 stages x 2 halves x [64 tok][64 hd]        32 KB
-constexpr int V_OFF = K_OFF + 32768;           // 2 stages x 2 halves x [64 tok][64 hd]        32 KB
-constexpr int BAR_OFF = V_OFF + 32768;
-constexpr int kSmemBytes = BAR_OFF + 256;
-constexpr int kStageBytes = 16384;             // one K (or V) tile
+// Shared-memory map (bytes from the 1024-aligned base); every operand region is 1024-aligned. Operands are cut into
+// blocks of 64 columns ("halves" at head_dim 128).
 constexpr int kHalfBytes = 8192;               // [64 tok][64 hd]
+template <int HD>
+struct WsCfg {
+  static constexpr int NH = HD / 64;
+  static constexpr int Q_OFF = 0;                       // NH x [128 rows][64 hd]
+  static constexpr int K_OFF = NH * 16384;              // 2 stages x NH x [64 tok][64 hd]
+  static constexpr int kStageBytes = NH * kHalfBytes;   // one K (or V) tile
+  static constexpr int V_OFF = K_OFF + 2 * kStageBytes; // 2 stages x NH x [64 tok][64 hd]
+  static constexpr int BAR_OFF = V_OFF + 2 * kStageBytes;
+  static constexpr int kSmemBytes = BAR_OFF + 256;
+};
 
 enum Bar : int {
   Q_FULL = 0, Q_EMPTY, K_FULL0, K_FULL1, K_EMPTY0, K_EMPTY1, V_FULL0, V_FULL1, V_EMPTY0, V_EMPTY1,
@@ -64,6 +68,10 @@ __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+// tanh x = 1 - 2 / (e^(2x) + 1): within a few 1e-7 absolute everywhere, and +-1 at the far ends.
+__device__ __forceinline__ float tanh_by_exp(float x) {
+  return 1.f - __fdividef(2.f, fast_exp2(x * (2.f * kLog2e)) + 1.f);
 }
 __device__ __forceinline__ void st_shared_v4(uint32_t addr, uint32_t a, uint32_t b, uint32_t c, uint32_t d) {
   asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(a), "r"(b), "r"(c), "r"(d) : "memory");
@@ -112,10 +120,13 @@ __device__ __forceinline__ Item read_item(const nfk_attn_params& p, long long w)
   return it;
 }
 
-template <bool EXT>
+template <int HD, bool EXT, bool CAP>
 __global__ void __launch_bounds__(kThreads, 2)
 attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                        nfk_attn_params p) {
+  using C = WsCfg<HD>;
+  constexpr int NH = C::NH, Q_OFF = C::Q_OFF, K_OFF = C::K_OFF, V_OFF = C::V_OFF, BAR_OFF = C::BAR_OFF;
+  constexpr int kStageBytes = C::kStageBytes;
   extern __shared__ __align__(1024) uint8_t smem[];
   const uint32_t sb = smem_u32(smem);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + BAR_OFF);
@@ -173,14 +184,16 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           // one head per query row tile: 128 rows in two boxes; rows past the item's tokens are other tokens' (or
           // zero past the buffer) and are never stored
           mbar_expect_tx(&bars[Q_FULL], 128u * HD * 2);
-          tma_load_2d(smem + Q_OFF, &tmQ, &bars[Q_FULL], it.kvh * HD, it.tok0);
-          tma_load_2d(smem + Q_OFF + 16384, &tmQ, &bars[Q_FULL], it.kvh * HD + 64, it.tok0);
+#pragma unroll
+          for (int h = 0; h < NH; ++h)
+            tma_load_2d(smem + Q_OFF + h * 16384, &tmQ, &bars[Q_FULL], it.kvh * HD + h * 64, it.tok0);
         } else {
         mbar_expect_tx(&bars[Q_FULL], static_cast<uint32_t>(it.ntok * group) * HD * 2);
         for (int tl = 0; tl < it.ntok; ++tl) {
           const int grow = (it.tok0 + tl) * p.q_heads + it.kvh * group;     // row of the [T*q_heads][128] view
-          tma_load_2d(smem + Q_OFF + tl * group * 128, &tmQ, &bars[Q_FULL], 0, grow);
-          tma_load_2d(smem + Q_OFF + 16384 + tl * group * 128, &tmQ, &bars[Q_FULL], 64, grow);
+#pragma unroll
+          for (int h = 0; h < NH; ++h)
+            tma_load_2d(smem + Q_OFF + h * 16384 + tl * group * 128, &tmQ, &bars[Q_FULL], h * 64, grow);
         }
         }
         ++issued[Q_FULL];
@@ -214,8 +227,8 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             const int row0 = plain ? cur[j] * kPage : ((cur[j] * 2) * p.kv_heads + it.kvh) * kPage;
             const int col0 = plain ? p.k_col + it.kvh * HD : 0;
             uint8_t* dst = smem + K_OFF + s * kStageBytes + j * 2048;
-            tma_load_2d(dst, &tmKV, &bars[K_FULL0 + s], col0, row0);
-            tma_load_2d(dst + kHalfBytes, &tmKV, &bars[K_FULL0 + s], col0 + 64, row0);
+#pragma unroll
+            for (int h = 0; h < NH; ++h) tma_load_2d(dst + h * kHalfBytes, &tmKV, &bars[K_FULL0 + s], col0 + h * 64, row0);
           }
           ++issued[K_FULL0 + s];
           if (!mbar_wait(&bars[V_EMPTY0 + s], ph) || *abort_flag) { fail(NF_ST_TIMEOUT_SMEM_EMPTY); ok = false; break; }
@@ -226,8 +239,8 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             const int row0 = plain ? cur[j] * kPage : ((cur[j] * 2 + 1) * p.kv_heads + it.kvh) * kPage;
             const int col0 = plain ? p.v_col + it.kvh * HD : 0;
             uint8_t* dst = smem + V_OFF + s * kStageBytes + j * 2048;
-            tma_load_2d(dst, &tmKV, &bars[V_FULL0 + s], col0, row0);
-            tma_load_2d(dst + kHalfBytes, &tmKV, &bars[V_FULL0 + s], col0 + 64, row0);
+#pragma unroll
+            for (int h = 0; h < NH; ++h) tma_load_2d(dst + h * kHalfBytes, &tmKV, &bars[V_FULL0 + s], col0 + h * 64, row0);
           }
           ++issued[V_FULL0 + s];
         }
@@ -256,7 +269,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tc_fence_after();
         const uint32_t kb = sb + K_OFF + s * kStageBytes;
 #pragma unroll
-        for (int h = 0; h < 2; ++h)
+        for (int h = 0; h < NH; ++h)
 #pragma unroll
           for (int k = 0; k < 4; ++k)
             umma_bf16_ss(tmem + s * kTile, umma_desc_k_sw128(sb + Q_OFF + h * 16384 + k * 32),
@@ -310,7 +323,9 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int row = warp * 32 + lane;                  // query row = TMEM lane
     const uint32_t t_lane = tmem + (static_cast<uint32_t>(warp * 32) << 16);
     __nv_bfloat16* outp = reinterpret_cast<__nv_bfloat16*>(p.out);
-    const float scale = p.sm_scale * kLog2e;
+    // CAP: capped scores carry the scale themselves
+    const float scale = CAP ? 1.f : p.sm_scale * kLog2e;
+    const float cap_in = CAP ? p.sm_scale / p.softcap : 0.f, cap_out = CAP ? p.softcap * kLog2e : 0.f;
     uint32_t g = 0, n_item = 0;
     bool ok = true;
     for (long long w = blockIdx.x; w < total && ok; w += gridDim.x) {
@@ -329,6 +344,13 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld_32x32b_x32(t_lane + s * kTile, r0);
         tmem_ld_32x32b_x32(t_lane + s * kTile + 32, r1);
         tmem_ld_wait();
+        if (CAP) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            r0[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r0[j]) * cap_in));
+            r1[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r1[j]) * cap_in));
+          }
+        }
         const int cbase = (it.t_first + t) * kTile;
         if (cbase + kTile - 1 > pos) {                        // only tiles on the diagonal need the mask
 #pragma unroll
@@ -364,7 +386,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           tc_fence_after();
           const float alpha = grow ? (m_ref == -INFINITY ? 0.f : fast_exp2(m_ref - mx)) : 1.f;
 #pragma unroll 1
-          for (int c = 0; c < 4; ++c) {
+          for (int c = 0; c < HD / 32; ++c) {
             uint32_t ov[32];
             tmem_ld_32x32b_x32(t_lane + 2 * kTile + c * 32, ov);
             tmem_ld_wait();
@@ -417,7 +439,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       const float inv = l > 0.f ? 1.f / l : 0.f;
       __nv_bfloat16* dst = outp + (static_cast<long long>(it.tok0 + tl) * p.q_heads + it.kvh * group + hh) * HD;
 #pragma unroll 1
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < HD / 32; ++c) {
         uint32_t r[32];
         tmem_ld_32x32b_x32(t_lane + 2 * kTile + c * 32, r);
         tmem_ld_wait();
@@ -448,6 +470,24 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   }
 }
 
+template <int HD, bool EXT, bool CAP>
+int launch_ws(const nfk_attn_params& p, const CUtensorMap& tmQ, const CUtensorMap& tmKV, cudaStream_t stream) {
+  constexpr int bytes = WsCfg<HD>::kSmemBytes;
+  static bool attr_dev[kMaxDevices] = {false};   // the attribute is per device
+  bool& attr = attr_dev[device_slot()];
+  if (!attr) {
+    if (cudaFuncSetAttribute(attn_prefill_ws_kernel<HD, EXT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) !=
+        cudaSuccess)
+      return NF_ERR_CUDA;
+    attr = true;
+  }
+  const long long total = static_cast<long long>(p.num_items) * p.kv_heads;
+  long long ctas = p.num_ctas > 0 ? p.num_ctas : 2LL * device_sm_count();   // two resident CTAs per SM
+  if (ctas > total) ctas = total;
+  attn_prefill_ws_kernel<HD, EXT, CAP><<<static_cast<int>(ctas), kThreads, bytes, stream>>>(tmQ, tmKV, p);
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
 }  // namespace
 }  // namespace nf
 
@@ -458,7 +498,13 @@ extern "C" int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream
     return NF_ERR_BAD_ARG;
   if (p->kv_heads <= 0 || p->q_heads % p->kv_heads != 0 || p->num_pages <= 0) return NF_ERR_BAD_ARG;
   const int group = p->q_heads / p->kv_heads;
-  if (p->head_dim != HD || p->page_size != kPage || group > 16 || (16 % group) != 0) return NF_ERR_UNSUPPORTED;
+  // `precise` and the extensions run in the EXT instantiations, capped scores and head_dim 64 in one of their own
+  const bool cap = p->softcap > 0.f;
+  const bool ext = p->window > 0 || p->sinks != nullptr || p->kv_ld > 0 || p->q_rows > 0 || cap || p->precise != 0;
+  if (p->page_size != kPage || p->softcap < 0.f) return NF_ERR_UNSUPPORTED;
+  if (p->head_dim != 128 && !(p->head_dim == 64 && ext)) return NF_ERR_UNSUPPORTED;
+  if (ext ? group > 128 : (group > 16 || (16 % group) != 0)) return NF_ERR_UNSUPPORTED;
+  const uint64_t HD = static_cast<uint64_t>(p->head_dim);
   if (p->num_items == 0) return NF_OK;
   if (p->num_items < 0 || p->items == nullptr) return NF_ERR_BAD_ARG;
   // Q as [tokens * q_heads][128] (the token count is not known here: any row the items name is inside
@@ -466,7 +512,6 @@ extern "C" int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream
   // [pages * 2 * kv_heads * 16][128]. Boxes: the `group` rows of one token, one page of one head; 64 columns.
   // With q_rows the queries are [q_rows][q_heads * 128] and a box is 128 tokens of one head; with kv_ld the
   // keys and values are columns of [num_pages * 16][kv_ld] rows.
-  const bool ext = p->window > 0 || p->sinks != nullptr || p->kv_ld > 0 || p->q_rows > 0;
   if (p->window < 0 || (p->q_rows > 0 && group != 1)) return NF_ERR_BAD_ARG;
   if (p->kv_ld > 0 && (p->kv_ld % 8 != 0 || p->k_col < 0 || p->v_col < 0 || p->k_col % 8 != 0 || p->v_col % 8 != 0))
     return NF_ERR_BAD_ARG;
@@ -478,20 +523,7 @@ extern "C" int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream
   rc = p->kv_ld > 0 ? make_tmap_bf16_2d(&tmKV, p->kv_pool, static_cast<uint64_t>(p->num_pages) * kPage, p->kv_ld, p->kv_ld, kPage, 64)
                     : make_tmap_bf16_2d(&tmKV, p->kv_pool, static_cast<uint64_t>(p->num_pages) * 2 * p->kv_heads * kPage, HD, HD, kPage, 64);
   if (rc != NF_OK) return rc;
-  static bool attr_dev[kMaxDevices] = {false};   // the attribute is per device
-  bool& attr = attr_dev[device_slot()];
-  if (!attr) {
-    if (cudaFuncSetAttribute(attn_prefill_ws_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
-            cudaSuccess ||
-        cudaFuncSetAttribute(attn_prefill_ws_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
-            cudaSuccess)
-      return NF_ERR_CUDA;
-    attr = true;
-  }
-  const long long total = static_cast<long long>(p->num_items) * p->kv_heads;
-  long long ctas = p->num_ctas > 0 ? p->num_ctas : 2LL * device_sm_count();   // two resident CTAs per SM
-  if (ctas > total) ctas = total;
-  if (ext) attn_prefill_ws_kernel<true><<<static_cast<int>(ctas), kThreads, kSmemBytes, stream>>>(tmQ, tmKV, *p);
-  else attn_prefill_ws_kernel<false><<<static_cast<int>(ctas), kThreads, kSmemBytes, stream>>>(tmQ, tmKV, *p);
-  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+  if (p->head_dim == 64) return cap ? launch_ws<64, true, true>(*p, tmQ, tmKV, stream) : launch_ws<64, true, false>(*p, tmQ, tmKV, stream);
+  if (cap) return launch_ws<128, true, true>(*p, tmQ, tmKV, stream);
+  return ext ? launch_ws<128, true, false>(*p, tmQ, tmKV, stream) : launch_ws<128, false, false>(*p, tmQ, tmKV, stream);
 }

@@ -77,6 +77,29 @@ NF_DEVICE bool mbar_wait(uint64_t* bar, uint32_t parity) {
   return false;
 }
 
+// Wait of a role of a persistent kernel: bounded by wall clock (globaltimer) and by the CTA abort flag.
+NF_DEVICE bool wait_or_abort(uint64_t* bar, uint32_t parity, volatile int* abort_flag) {
+  const uint32_t addr = smem_u32(bar);
+  uint64_t t0 = 0;
+  for (uint32_t it = 0;; ++it) {
+    uint32_t ok;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(ok)
+        : "r"(addr), "r"(parity)
+        : "memory");
+    if (ok) return true;
+    if ((it & 255u) == 255u) {
+      if (*abort_flag) return false;
+      uint64_t now;
+      asm volatile("mov.u64 %0, %globaltimer;" : "=l"(now));
+      if (t0 == 0) t0 = now;
+      if (now - t0 > 2000000000ull || it > (1u << 30)) return false;  // 2 s
+    }
+  }
+}
 
 NF_DEVICE void report_status(unsigned int* status, unsigned int code) {
   if (status != nullptr) atomicCAS(status, 0u, code);

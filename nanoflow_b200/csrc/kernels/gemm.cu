@@ -2,7 +2,7 @@
 // by TMA into 128B-swizzled shared memory, persistent over output tiles with an explicit CTA budget.
 //
 //   D[M,N] = A[M,K] * B[N,K]^T (+ bias[N]) (+ beta * C[M,N])            (linear epilogue)
-//   D[M,F] = act(A * Bg[F,K]^T) .* (A * Bu[F,K]^T)                       (gated epilogue: silu, relu, gelu)
+//   D[M,F] = act(A * Bg[F,K]^T, A * Bu[F,K]^T)                           (gated epilogue, see gated_act.cuh)
 //
 // Columns from f32_col0 on can leave as fp32 into a second output (logits, gate pre-activations), and the
 // product can be block diagonal: with `groups` > 1 output columns of group g see only A's columns
@@ -23,6 +23,7 @@
 // (pipeline/include/cutlassGemmWrapperImpl.cuh:68-125: D = alpha*A*B + beta*C, residual or
 // replicated bias as C) and of its DualGemm + SiLU-mul epilogue (pipeline/include/dualWrapper.cuh:47-144).
 #include "common.cuh"
+#include "gated_act.cuh"
 #include "kernels.h"
 
 #include <mutex>
@@ -155,7 +156,8 @@ struct DevParams {
   float* D32;
   long long ld32;
   int f32_col0;
-  int act;                          // gated epilogue: NFK_ACT_*
+  GatedAct act;                     // gated epilogue
+  int lin_act;                      // linear epilogue: NFK_LIN_*
   int groups, group_n, group_k;     // block-diagonal product (groups 1: an ordinary one)
 };
 
@@ -183,15 +185,12 @@ __device__ __forceinline__ NBlock n_block(const DevParams& p, int n_blk, int out
   return b;
 }
 
-// Activation of the gated epilogue.
-__device__ __forceinline__ float gated_act(float x, int act) {
-  if (act == NFK_ACT_RELU) return fmaxf(x, 0.f);
-  if (act == NFK_ACT_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-  return x / (1.0f + __expf(-x));
-}
-
 // Eight finished columns of one row: bf16 to D, or fp32 to D32 from f32_col0 on (a multiple of 8).
-__device__ __forceinline__ void store_cols8(const DevParams& p, int row, int col, const float* v) {
+__device__ __forceinline__ void store_cols8(const DevParams& p, int row, int col, float* v) {
+  if (p.lin_act == NFK_LIN_TANH) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = tanhf(v[j]);
+  }
   if (p.D32 != nullptr && col >= p.f32_col0) {
     float4* dst = reinterpret_cast<float4*>(p.D32 + static_cast<long long>(row) * p.ld32 + (col - p.f32_col0));
     dst[0] = make_float4(v[0], v[1], v[2], v[3]);
@@ -244,30 +243,6 @@ __device__ __forceinline__ bool wait_gate(const DevParams& p, int m_tile, volati
   }
   asm volatile("fence.proxy.async;" ::: "memory");
   return true;
-}
-
-// Wait helper shared by all roles: bounded by wall clock (globaltimer) and by the CTA abort flag.
-__device__ __forceinline__ bool wait_or_abort(uint64_t* bar, uint32_t parity, volatile int* abort_flag) {
-  const uint32_t addr = smem_u32(bar);
-  uint64_t t0 = 0;
-  for (uint32_t it = 0;; ++it) {
-    uint32_t ok;
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(ok)
-        : "r"(addr), "r"(parity)
-        : "memory");
-    if (ok) return true;
-    if ((it & 255u) == 255u) {
-      if (*abort_flag) return false;
-      uint64_t now;
-      asm volatile("mov.u64 %0, %globaltimer;" : "=l"(now));
-      if (t0 == 0) t0 = now;
-      if (now - t0 > 2000000000ull || it > (1u << 30)) return false;  // 2 s
-    }
-  }
 }
 
 // ---- work distribution -----------------------------------------------------------------------------
@@ -647,7 +622,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 continue;
               }
 #pragma unroll
-              for (int j = 0; j < 32; ++j) v[j] = gated_act(gsum[j], p.act) * usum[j];
+              for (int j = 0; j < 32; ++j) v[j] = gated_act(gsum[j], usum[j], p.act);
             } else {
               tmem_ld_wait();
 #pragma unroll
@@ -1010,7 +985,7 @@ sk_fixup_kernel(DevParams p, FixupGeom f) {
     }
     if (EPI == 1) {
 #pragma unroll
-      for (int j = 0; j < 8; ++j) a[j] = gated_act(a[j], p.act) * u[j];
+      for (int j = 0; j < 8; ++j) a[j] = gated_act(a[j], u[j], p.act);
     } else {
       if (p.bias != nullptr) {
         const uint4 bv = *reinterpret_cast<const uint4*>(p.bias + col);
@@ -1181,7 +1156,8 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
   p.D32 = reinterpret_cast<float*>(g.D32);
   p.ld32 = g.ld32;
   p.f32_col0 = g.f32_col0;
-  p.act = g.act;
+  p.act = GatedAct{g.act, g.act_limit, g.act_alpha, g.act_shift};
+  p.lin_act = EPI == 0 ? g.lin_act : NFK_LIN_NONE;
   p.groups = groups;
   p.group_n = group_n;
   p.group_k = g.group_k;
@@ -1448,7 +1424,7 @@ extern "C" int nfk_gemm_bf16(const nfk_gemm_params* g, cudaStream_t stream) {
       (g->epilogue != NFK_EPI_LINEAR || g->f32_col0 < 0 || g->f32_col0 % 8 != 0 || g->ld32 % 4 != 0 ||
        (reinterpret_cast<uintptr_t>(g->D32) & 15) != 0 || g->norm_w != nullptr))
     return NF_ERR_BAD_ARG;
-  if (g->act < NFK_ACT_SILU || g->act > NFK_ACT_GELU_TANH) return NF_ERR_BAD_ARG;
+  if (g->act < NFK_ACT_SILU || g->act > NFK_ACT_CAPPED || g->lin_act < NFK_LIN_NONE || g->lin_act > NFK_LIN_TANH) return NF_ERR_BAD_ARG;
   if (g->groups > 1 && (g->epilogue != NFK_EPI_LINEAR || g->N % (8 * g->groups) != 0 || g->group_k % 8 != 0 ||
                         g->group_k < 0 || g->gate_flags != nullptr))
     return NF_ERR_BAD_ARG;

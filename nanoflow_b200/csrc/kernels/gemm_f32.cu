@@ -2,18 +2,13 @@
 // the same products, epilogues and block-diagonal form as gemm.cu on fp32 operands. A 64 x 64 output tile
 // per 256-thread CTA, 4 x 4 outputs per thread, operands staged 16 k at a time in shared memory.
 #include "common.cuh"
+#include "gated_act.cuh"
 #include "kernels.h"
 
 namespace nf {
 namespace {
 
 constexpr int kT = 64, kKb = 16, kThr = 256;
-
-__device__ __forceinline__ float act_f32(float x, int act) {
-  if (act == NFK_ACT_RELU) return fmaxf(x, 0.f);
-  if (act == NFK_ACT_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-  return x / (1.0f + expf(-x));
-}
 
 template <bool GATED>
 __global__ void __launch_bounds__(kThr)
@@ -63,6 +58,7 @@ gemm_f32_kernel(nfk_gemm_params p, int groups, int group_n) {
   float* D32 = reinterpret_cast<float*>(p.D32);
   const float* C = reinterpret_cast<const float*>(p.C);
   const float* bias = reinterpret_cast<const float*>(p.bias);
+  const GatedAct act{p.act, p.act_limit, p.act_alpha, p.act_shift};
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int row = row0 + ty * 4 + i;
@@ -73,11 +69,12 @@ gemm_f32_kernel(nfk_gemm_params p, int groups, int group_n) {
       if (col >= col_end) continue;
       float v = acc[i][j];
       if (GATED) {
-        v = act_f32(v, p.act) * up[i][j];
+        v = gated_act_of<true>(v, up[i][j], act);
       } else {
         if (bias != nullptr) v += bias[col];
         if (C != nullptr) v += p.beta * C[static_cast<long long>(row) * p.ldc + col];
       }
+      if (!GATED && p.lin_act == NFK_LIN_TANH) v = tanhf(v);
       if (D32 != nullptr && col >= p.f32_col0) D32[static_cast<long long>(row) * p.ld32 + col - p.f32_col0] = v;
       else D[static_cast<long long>(row) * p.ldd + col] = v;
     }

@@ -14,7 +14,10 @@ extern "C" {
 // GEMM (gemm.cu)
 // ------------------------------------------------------------------------------------------------
 enum { NFK_EPI_LINEAR = 0, NFK_EPI_SWIGLU = 1, NFK_EPI_REDUCE_SCATTER = 2 };
-enum { NFK_ACT_SILU = 0, NFK_ACT_RELU = 1, NFK_ACT_GELU_TANH = 2 };   // activation of the gated epilogue
+// Gated epilogue: act(gate) * up, or for NFK_ACT_CAPPED g sigmoid(alpha g) (u + shift) with g = min(gate, limit) and
+// u = min(max(up, -limit), limit).
+enum { NFK_ACT_SILU = 0, NFK_ACT_RELU = 1, NFK_ACT_GELU_TANH = 2, NFK_ACT_CAPPED = 3 };
+enum { NFK_LIN_NONE = 0, NFK_LIN_TANH = 1 };                           // activation of the linear epilogue
 enum { NFK_BF16 = 0, NFK_F32 = 1 };                                    // storage type of activations and weights
 
 typedef struct nfk_gemm_params {
@@ -80,6 +83,8 @@ typedef struct nfk_gemm_params {
   // Block-diagonal product (linear epilogue): `groups` > 1 cuts the N columns (and B's rows) into equal
   // groups; group g reads A's columns [g * group_k, g * group_k + K). 0 or 1 = an ordinary product.
   int groups, group_k;
+  int lin_act;          // linear epilogue: NFK_LIN_*, applied to the finished columns
+  float act_limit, act_alpha, act_shift;   // constants of NFK_ACT_CAPPED
 } nfk_gemm_params;
 
 int nfk_gemm_bf16(const nfk_gemm_params* p, cudaStream_t stream);
@@ -203,6 +208,9 @@ typedef struct nfk_attn_params {
   int kv_ld, k_col, v_col;
   int q_rows;              // > 0 (one query head per KV head): rows of q, which is [q_rows][ld_q]
   int ld_q;                // 0 = q_heads * 128
+  // nfk_attn_decode and nfk_attn_prefill_ws (head_dim 64 or 128):
+  float softcap;           // > 0: score <- softcap tanh(score / softcap) before the softmax
+  int precise;             // 1: probabilities enter the second product as a bf16 pair (implied by the other extensions)
 } nfk_attn_params;
 int nfk_attn_decode(const nfk_attn_params* p, cudaStream_t stream);
 // The same with the pages copied by a TMA producer warp into a ring of decode_stages (2, 3 or 4) pages per
@@ -220,8 +228,8 @@ int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream);
 // Layer-list models: residual step, latent attention, mLSTM (residual_norm.cu, latent.cu, mlstm.cu)
 // ------------------------------------------------------------------------------------------------
 enum { NFK_NORM_NONE = 0, NFK_NORM_RMS = 1, NFK_NORM_LAYER = 2 };
-// x <- (table ? 0 : x) + norm_in(src) (+ add);  h = norm_out(x). Rows of x, y, table and h are padded to a
-// multiple of 4 elements; weight vectors are padded with zeros to that length.
+// x <- (table ? 0 : x) + norm_in(src_scale src) (+ y2_gate y2) (+ sum_k e_weight e_out[e_slot]) (+ add);  h = norm_out(x).
+// Rows of x, y, table and h are padded to a multiple of 4 elements; weight vectors are padded with zeros to that length.
 typedef struct nfk_residual_norm_params {
   float* x;                  // [*, ld_x] residual stream
   long long ld_x;
@@ -245,8 +253,17 @@ typedef struct nfk_residual_norm_params {
   int rows, cols;
   float eps;
   int in_kind, out_kind;     // NFK_NORM_*
-  int dtype;                 // NFK_BF16 / NFK_F32: y, table, h
+  int dtype;                 // NFK_BF16 / NFK_F32: y, table, h, y2, e_out
   unsigned int* status;
+  float src_scale;           // factor of the source row; 0 = 1
+  const void* y2;            // [*, ld_y2] a second sublayer output that joins the same sum, null: none
+  long long ld_y2;
+  const float* y2_gate;      // [*] factor per row of y2, null: 1
+  const void* e_out;         // [e_rows, ld_e] outputs of a mixture of experts, null: none
+  long long ld_e;
+  const int* e_slot;         // [*][e_top] rows of e_out of a token
+  const float* e_weight;     // [*][e_top]
+  int e_top, e_rows;
 } nfk_residual_norm_params;
 int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t stream);
 
@@ -365,6 +382,167 @@ typedef struct nfk_head_norm_gate_params {
   int dtype;
 } nfk_head_norm_gate_params;
 int nfk_head_norm_gate(const nfk_head_norm_gate_params* p, cudaStream_t stream);
+
+// ------------------------------------------------------------------------------------------------
+// Grouped-query attention without rotation (gqa.cu)
+// ------------------------------------------------------------------------------------------------
+// Pool of one layer as for nfk_attn_*: [pages][2 (K, V)][kv_heads][page_size][hd]; hd is the padded size of a head's
+// keys and values (padding columns are zero).
+// Per token: RMS norm of the whole query row and of the whole key row (all heads at once), keys and values to their
+// page slot. v_mode 1 also keeps the values in v_first; 2 mixes them, v <- (1 - lambda) v + lambda v_first.
+typedef struct nfk_gqa_append_params {
+  const void* src;           // [T, ld_src]: q at q_off, k at k_off, v at v_off, head h at column h * hd
+  long long ld_src;
+  int q_off, k_off, v_off;
+  void* q_out;               // [T, heads * hd]
+  const float* q_w;          // [heads * hd] norm weights, null: no norm
+  const float* k_w;          // [kv_heads * hd]
+  void* v_first;             // [T, kv_heads * hd]
+  int v_mode;
+  float v_lambda;
+  void* pool;
+  const int* positions;
+  const int* token_req;
+  const int* kv_indptr;
+  const int* kv_indices;
+  const int* kv_first;
+  int T, heads, kv_heads, hd, dim;    // dim: real size of a head's query and key
+  int page_size, num_pages;
+  float eps;
+  int dtype;
+  unsigned int* status;
+} nfk_gqa_append_params;
+int nfk_gqa_append(const nfk_gqa_append_params* p, cudaStream_t stream);
+
+// Attention of the tokens [token_begin, token_begin + n_tokens), any sizes, bf16 or fp32: one CTA per token and head.
+typedef struct nfk_gqa_attn_params {
+  const void* q;             // [T, heads * hd]
+  const void* pool;
+  void* out;                 // [T, heads * hd]
+  const int* positions;
+  const int* token_req;
+  const int* kv_indptr;
+  const int* kv_indices;
+  const int* kv_first;
+  const float* sinks;        // [heads], null: none
+  int token_begin, n_tokens, heads, kv_heads, hd, page_size, num_pages, window;
+  float scale, softcap;      // softcap 0: none
+  int dtype;
+  unsigned int* status;
+} nfk_gqa_attn_params;
+int nfk_gqa_attn(const nfk_gqa_attn_params* p, cudaStream_t stream);
+
+// ------------------------------------------------------------------------------------------------
+// Mixture of experts (moe.cu)
+// ------------------------------------------------------------------------------------------------
+// Scores s = sigmoid(logits); choice scores s + correction. Experts form `groups` equal runs of neighbours (1: no
+// grouping); a group counts by the sum of its two largest choice scores and only experts of the best `keep` groups
+// can be chosen. Weights: s of the `top` chosen ones over their sum, times scale. Ties go to the lower index.
+// Every chosen expert's counter is increased; what it was before is the token's rank among the expert's rows.
+typedef struct nfk_moe_route_params {
+  const float* logits;       // [T, ld]: experts at columns 0 .., the shared expert's gate at gate_col (< 0: none)
+  long long ld;
+  const float* correction;   // [experts], null: none
+  int* expert;               // [T][top]
+  float* weight;             // [T][top]
+  int* rank;                 // [T][top]
+  int* counts;               // [experts], zero before the launch
+  float* gate;               // [T] sigmoid of the gate column
+  int T, experts, top, groups, keep, gate_col;
+  float scale;
+} nfk_moe_route_params;
+int nfk_moe_route(const nfk_moe_route_params* p, cudaStream_t stream);
+
+// Rows of h in expert order: row rank + (rows of the experts before) of out for every chosen expert of a token.
+typedef struct nfk_moe_permute_params {
+  const void* h;             // [T, ld_h]
+  long long ld_h;
+  void* out;                 // [>= T * top, ld_out]
+  long long ld_out;
+  const int* expert;
+  const int* rank;
+  const int* counts;
+  int* slot;                 // [T][top]
+  int T, top, experts, cols; // cols: a multiple of 8
+  int dtype;
+} nfk_moe_permute_params;
+int nfk_moe_permute(const nfk_moe_permute_params* p, cudaStream_t stream);
+
+// One product per expert over its rows of A (rows in expert order, counts per expert on the device):
+// D = A B_e^T, or with B2 the gated epilogue of nfk_gemm_bf16. Matrices of the experts are stacked: B [experts * N, ldb].
+typedef struct nfk_moe_gemm_params {
+  const void* A;             // [rows, lda]
+  const void* B;
+  const void* B2;            // up matrices, null: linear
+  void* D;                   // [rows, ldd]
+  const int* counts;
+  long long lda, ldb, ldd;
+  int rows;                  // most rows (T * top)
+  int experts, N, K;         // N, K: multiples of 8
+  int act;
+  float act_limit, act_alpha, act_shift;
+  int dtype, num_ctas;
+  unsigned int* status;
+} nfk_moe_gemm_params;
+int nfk_moe_gemm(const nfk_moe_gemm_params* p, cudaStream_t stream);
+
+// ------------------------------------------------------------------------------------------------
+// WKV recurrence (wkv.cu)
+// ------------------------------------------------------------------------------------------------
+// out[t, s * ld_h + c] = h + (h' - h) mu[s][c] with h' the previous token's row: of the same request in this launch,
+// of the state (half ref & 1 is read, the other one receives the request's last row), or zero at position 0.
+typedef struct nfk_token_shift_params {
+  const void* h;             // [T, ld_h]
+  long long ld_h;
+  void* out;                 // [T, n_mix * ld_h]
+  const float* mu;           // [n_mix][ld_h]
+  void* state;               // [slots][2][ld_h]
+  const int* state_slot;     // [B] 2 * slot + half
+  const int* positions;
+  const int* token_req;
+  const int* qo_indptr;
+  int T, n_mix, num_slots;
+  int dtype;
+  unsigned int* status;
+} nfk_token_shift_params;
+int nfk_token_shift(const nfk_token_shift_params* p, cudaStream_t stream);
+
+// Per head, with w_t = exp(-exp(x_t)) per key channel:
+//   o_t = (S + diag(u) k_t v_t^T)^T r_t;  S <- diag(w_t) S + k_t v_t^T
+//   y_t = RMS norm of o_t (over the head's `dim_real` values) * norm * silu(g_t)
+// A request whose first token of the launch is at position 0 starts from a zero state.
+typedef struct nfk_wkv_params {
+  const void* rkvg;          // [T, ld]: r, k, v, g at their offsets, head h at column h * dim
+  long long ld;
+  int r_off, k_off, v_off, g_off;
+  const float* x;            // [T, ld_x] logarithm of the decay's negative logarithm
+  long long ld_x;
+  const float* u;            // [heads * dim]
+  const float* norm;         // [heads * dim]
+  float* S;                  // [slots][heads][dim][dim], key channel first
+  void* y;                   // [T, ld_y]
+  long long ld_y;
+  const int* positions;
+  const int* qo_indptr;
+  const int* state_slot;     // [B] 2 * slot (+ half, not used here)
+  int req_begin, req_count;  // decode: requests with one token each
+  int heads, dim, dim_real, num_slots;
+  float eps;
+  int dtype;
+  // prefill. Token by token: seq_reqs [num_seq] requests, o: fp32 [T, heads * dim] of scratch rows. In chunks of 64 tokens
+  // (bf16): items [num_items][4] (request, first token, tokens, chunk of the request's portion), a request's chunks one
+  // after the other, and scratch: num_items * heads * (dim * dim + dim) floats.
+  const int* seq_reqs;
+  int num_seq;
+  float* o;
+  const int* items;
+  int num_items;
+  float* scratch;
+  long long scratch_floats;
+  unsigned int* status;
+} nfk_wkv_params;
+int nfk_wkv_decode(const nfk_wkv_params* p, cudaStream_t stream);
+int nfk_wkv_prefill(const nfk_wkv_params* p, cudaStream_t stream);
 
 // ------------------------------------------------------------------------------------------------
 // KV offload (kv_offload.cu): gather / scatter whole pages between the pool and a staging buffer

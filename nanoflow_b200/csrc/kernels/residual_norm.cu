@@ -1,7 +1,7 @@
 // The step between two sublayers in one pass over the row: norm of the sublayer's output, residual sum in
 // fp32, an optional vector added to the stream, and the norm that the next sublayer reads.
 //
-//   x <- (table ? 0 : x) + norm_in(src) (+ add);   h = norm_out(x)
+//   x <- (table ? 0 : x) + norm_in(src) (+ second output) (+ weighted expert outputs) (+ add);   h = norm_out(x)
 //
 // `src` is the sublayer's output row, or the embedding row of the token (ids as in nfk_embedding, with the
 // previous iteration's tokens fed back on the device). Norms are RMS or layer norms with fp32 weights. The
@@ -21,6 +21,10 @@ __device__ __forceinline__ float cta_sum(float v, float* red) {
   if (lane == 0) red[warp] = v;
   __syncthreads();
   return warp_sum(lane < (kRnThreads >> 5) ? red[lane] : 0.f);
+}
+
+__device__ __forceinline__ void fma4(float4& a, float f, float4 b) {
+  a.x += f * b.x; a.y += f * b.y; a.z += f * b.z; a.w += f * b.w;
 }
 
 // In-place norm of the row held in v (elements at or past `cols` are zero and stay zero).
@@ -99,7 +103,38 @@ residual_norm_kernel(nfk_residual_norm_params p) {
       const int vi = threadIdx.x + i * kRnThreads;
       v[i] = (src != nullptr && vi < nvec) ? load4(src + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    if (src != nullptr && p.src_scale != 0.f) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        v[i].x *= p.src_scale; v[i].y *= p.src_scale; v[i].z *= p.src_scale; v[i].w *= p.src_scale;
+      }
+    }
     if (src != nullptr) norm_row<NV>(v, p.in_kind, p.in_w, p.in_b, p.cols, nvec, p.eps, red);
+    if (p.y2 != nullptr) {
+      const float f = p.y2_gate != nullptr ? p.y2_gate[src_row] : 1.f;
+      const T* y2 = reinterpret_cast<const T*>(p.y2) + static_cast<long long>(src_row) * p.ld_y2;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int vi = threadIdx.x + i * kRnThreads;
+        if (vi < nvec) fma4(v[i], f, load4(y2 + vi * 4));
+      }
+    }
+    if (p.e_out != nullptr) {
+      for (int k = 0; k < p.e_top; ++k) {
+        const int slot = p.e_slot[static_cast<long long>(src_row) * p.e_top + k];
+        const float f = p.e_weight[static_cast<long long>(src_row) * p.e_top + k];
+        if (slot < 0 || slot >= p.e_rows) {
+          if (threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
+          continue;
+        }
+        const T* e = reinterpret_cast<const T*>(p.e_out) + static_cast<long long>(slot) * p.ld_e;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int vi = threadIdx.x + i * kRnThreads;
+          if (vi < nvec) fma4(v[i], f, load4(e + vi * 4));
+        }
+      }
+    }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int vi = threadIdx.x + i * kRnThreads;
@@ -153,6 +188,8 @@ extern "C" int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t
   if (p->table && !p->host_ids && !(p->feedback_src && p->prev_tokens)) return NF_ERR_BAD_ARG;
   if ((p->y && p->ld_y % 4 != 0) || (p->h && p->ld_h % 4 != 0)) return NF_ERR_BAD_ARG;
   if (p->rows_idx && (p->in_rows <= 0 || !p->h)) return NF_ERR_BAD_ARG;
+  if (p->y2 && p->ld_y2 % 4 != 0) return NF_ERR_BAD_ARG;
+  if (p->e_out && (!p->e_slot || !p->e_weight || p->e_top <= 0 || p->e_rows <= 0 || p->ld_e % 4 != 0)) return NF_ERR_BAD_ARG;
   for (int kind : {p->in_kind, p->out_kind})
     if (kind != NFK_NORM_NONE && kind != NFK_NORM_RMS && kind != NFK_NORM_LAYER) return NF_ERR_BAD_ARG;
   if ((p->table || p->y) && p->in_kind != NFK_NORM_NONE && !p->in_w) return NF_ERR_BAD_ARG;

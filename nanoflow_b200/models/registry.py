@@ -18,6 +18,7 @@ class ModelFamily:
     random_weights: Callable[..., Any]       # (NanoflowConfig, rank, tp, device, seed) -> weights
     engine: Callable[..., Any]               # (NanoflowConfig, weights, **kw) -> engine
     cpu_engine: Callable[..., Any]           # (NanoflowConfig, list of per-rank weights, num_pages=) -> CPU engine
+    complete: Callable[..., Any] = None      # (config.json dict, checkpoint folder) -> the dict with sizes from the tensors
     listed_layers: bool = False              # the layers are listed one by one in config.json
     runs_float32: bool = False               # the engine can store and multiply in 32-bit
 
@@ -45,14 +46,14 @@ def _llama() -> ModelFamily:
                        load_folder, random, engine, cpu_engine)
 
 
-def _volarax() -> ModelFamily:
-    from . import volarax
+def _layer_list(name: str, design) -> ModelFamily:
+    """Family of a layer-list design: a module of ``models/`` with its keys, tensor names and random weights."""
 
     def load_folder(cfg, folder, device):
-        return volarax.load_weights(cfg.model, folder, device)
+        return design.load_weights(cfg.model, folder, device)
 
     def random(cfg, rank, tp, device, seed=0):
-        return volarax.random_weights(cfg.model, cfg.raw["model"], device, seed)
+        return design.random_weights(cfg.model, cfg.raw["model"], device, seed)
 
     def engine(cfg, weights, **kw):
         from ..runtime.layer_list import LayerListEngine
@@ -62,11 +63,21 @@ def _volarax() -> ModelFamily:
         from ..runtime.cpu_layer_list import CpuLayerListEngine
         return CpuLayerListEngine(cfg, shards[0], num_pages=num_pages)
 
-    return ModelFamily("volarax", (volarax.ARCHITECTURE,), volarax.parse_model, load_folder, random, engine, cpu_engine,
-                       listed_layers=True, runs_float32=True)
+    return ModelFamily(name, (design.ARCHITECTURE,), design.parse_model, load_folder, random, engine, cpu_engine,
+                       complete=getattr(design, "complete", None), listed_layers=True, runs_float32=True)
 
 
-_FAMILIES: Dict[str, Callable[[], ModelFamily]] = {"llama": _llama, "volarax": _volarax}
+def _volarax() -> ModelFamily:
+    from . import volarax
+    return _layer_list("volarax", volarax)
+
+
+def _zubedra() -> ModelFamily:
+    from . import zubedra
+    return _layer_list("zubedra", zubedra)
+
+
+_FAMILIES: Dict[str, Callable[[], ModelFamily]] = {"llama": _llama, "volarax": _volarax, "zubedra": _zubedra}
 _cache: Dict[str, ModelFamily] = {}
 
 

@@ -4,13 +4,23 @@ from __future__ import annotations
 
 import json
 import struct
-from typing import Dict
+from typing import Dict, Tuple
 
 import torch
 
 _DTYPES = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "F64": torch.float64,
            "I8": torch.int8, "I16": torch.int16, "I32": torch.int32, "I64": torch.int64, "U8": torch.uint8,
            "BOOL": torch.bool}
+
+
+def read_shapes(path: str) -> Dict[str, Tuple[int, ...]]:
+    """Names and shapes of the tensors of a file."""
+    with open(path, "rb") as f:
+        raw = f.read(8)
+        if len(raw) != 8:
+            raise ValueError(f"{path}: not a safetensors file")
+        header = json.loads(f.read(struct.unpack("<Q", raw)[0]))
+    return {name: tuple(info["shape"]) for name, info in header.items() if name != "__metadata__"}
 
 
 def read_safetensors(path: str) -> Dict[str, torch.Tensor]:
@@ -37,7 +47,7 @@ def write_safetensors(path: str, tensors: Dict[str, torch.Tensor]) -> None:
     names = {v: k for k, v in _DTYPES.items()}
     header, blobs, off = {}, [], 0
     for name, t in tensors.items():
-        b = t.detach().cpu().contiguous().view(torch.uint8).numpy().tobytes() if t.dim() else b""
+        b = t.detach().cpu().contiguous().reshape(-1).view(torch.uint8).numpy().tobytes()
         header[name] = {"dtype": names[t.dtype], "shape": list(t.shape), "data_offsets": [off, off + len(b)]}
         blobs.append(b)
         off += len(b)

@@ -13,7 +13,7 @@ from typing import Any, Callable, Dict, List, Tuple
 
 import torch
 
-from .layer_list import (LatentAttentionSpec, LayerListConfig, LayerListLayer, LayerListWeights, LayerSpec, MlpSpec,
+from .layer_list import (ActSpec, LatentAttentionSpec, LayerListConfig, LayerListLayer, LayerListWeights, LayerSpec, MlpSpec,
                          MlstmSpec, pack_latent_attention, pack_mlp, pack_mlstm, pack_norm, pad_to)
 from .safetensors_io import read_safetensors
 
@@ -40,7 +40,7 @@ def parse_model(raw: Dict[str, Any], *, tp: int = 1, run_layers: int = 0, name: 
         if mlp is not None and mlp.get("kind", "dense") != "dense":
             raise ValueError(f"layer {i}: unknown feed-forward '{mlp['kind']}'")
         layers.append(LayerSpec(_mixer(lay["type"], lay["mixer"], f"layer {i}"),
-                                None if mlp is None else MlpSpec(int(mlp["ff"]), "relu")))
+                                None if mlp is None else MlpSpec(int(mlp["ff"]), ActSpec("relu"))))
     loop = raw.get("loop")
     cfg = LayerListConfig(
         name=name or ARCHITECTURE, hidden_size=int(raw["width"]), vocab_size=int(raw["vocab"]), layers=layers,
@@ -105,8 +105,7 @@ def weights_from_tensors(cfg: LayerListConfig, get: Callable[[str], torch.Tensor
         out = LayerListLayer(mixer=mix, norm_in=norm(f"l{i}.norm1"), norm_out=norm(f"l{i}.norm1b"))
         if lay.mlp is not None:
             out.mlp_in, out.mlp_out = norm(f"l{i}.norm2"), norm(f"l{i}.norm2b")
-            out.w_gate, out.w_up, out.w_down = pack_mlp(cfg, lay.mlp.ff, get(f"l{i}.mlp.gate"), get(f"l{i}.mlp.up"),
-                                                        get(f"l{i}.mlp.down"), device)
+            out.mlp = pack_mlp(cfg, lay.mlp.ff, get(f"l{i}.mlp.gate"), get(f"l{i}.mlp.up"), get(f"l{i}.mlp.down"), device)
         w.layers.append(out)
     return w
 

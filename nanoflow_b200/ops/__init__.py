@@ -43,7 +43,8 @@ class GemmParams(Structure):
                 ("norm_w", c_void_p), ("norm_out", c_void_p), ("norm_ld", c_longlong), ("norm_eps", c_float),
                 ("rs_staged", c_int), ("gate_flags", c_void_p), ("gate_epoch", c_int), ("gate_nranks", c_int),
                 ("D32", c_void_p), ("ld32", c_longlong), ("f32_col0", c_int), ("act", c_int),
-                ("groups", c_int), ("group_k", c_int)]
+                ("groups", c_int), ("group_k", c_int), ("lin_act", c_int),
+                ("act_limit", c_float), ("act_alpha", c_float), ("act_shift", c_float)]
 
 
 class RopeAppendParams(Structure):
@@ -71,11 +72,12 @@ class AttnParams(Structure):
                 ("chunk_pages", c_int), ("workspace", c_void_p), ("max_chunks", c_int),
                 ("items", c_void_p), ("num_items", c_int), ("status", c_void_p), ("decode_stages", c_int),
                 ("window", c_int), ("sinks", c_void_p), ("kv_ld", c_int), ("k_col", c_int), ("v_col", c_int),
-                ("q_rows", c_int), ("ld_q", c_int)]
+                ("q_rows", c_int), ("ld_q", c_int), ("softcap", c_float), ("precise", c_int)]
 
 
 BF16, F32 = 0, 1                                        # storage type of a kernel's activations and weights
-ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 2}           # activation of the gated GEMM epilogue
+ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "capped": 3}   # activation of the gated GEMM epilogue
+LIN_ACTS = {None: 0, "tanh": 1}                         # activation of the linear GEMM epilogue
 NORMS = {None: 0, "rms": 1, "layer": 2}
 
 
@@ -93,7 +95,9 @@ class ResidualNormParams(Structure):
                 ("prev_tokens", c_void_p), ("vocab", c_int), ("in_w", c_void_p), ("in_b", c_void_p),
                 ("add", c_void_p), ("h", c_void_p), ("ld_h", c_longlong), ("out_w", c_void_p), ("out_b", c_void_p),
                 ("rows_idx", c_void_p), ("in_rows", c_int), ("rows", c_int), ("cols", c_int), ("eps", c_float),
-                ("in_kind", c_int), ("out_kind", c_int), ("dtype", c_int), ("status", c_void_p)]
+                ("in_kind", c_int), ("out_kind", c_int), ("dtype", c_int), ("status", c_void_p), ("src_scale", c_float),
+                ("y2", c_void_p), ("ld_y2", c_longlong), ("y2_gate", c_void_p), ("e_out", c_void_p), ("ld_e", c_longlong),
+                ("e_slot", c_void_p), ("e_weight", c_void_p), ("e_top", c_int), ("e_rows", c_int)]
 
 
 class LatentAppendParams(Structure):
@@ -132,6 +136,59 @@ class HeadNormGateParams(Structure):
     _fields_ = [("o", c_void_p), ("ld_o", c_longlong), ("g", c_void_p), ("ld_g", c_longlong), ("w", c_void_p),
                 ("out", c_void_p), ("ld_out", c_longlong), ("T", c_int), ("heads", c_int), ("vdim", c_int),
                 ("vdim_p", c_int), ("eps", c_float), ("dtype", c_int)]
+
+
+class GqaAppendParams(Structure):
+    _fields_ = [("src", c_void_p), ("ld_src", c_longlong), ("q_off", c_int), ("k_off", c_int), ("v_off", c_int),
+                ("q_out", c_void_p), ("q_w", c_void_p), ("k_w", c_void_p), ("v_first", c_void_p), ("v_mode", c_int),
+                ("v_lambda", c_float), ("pool", c_void_p), ("positions", c_void_p), ("token_req", c_void_p),
+                ("kv_indptr", c_void_p), ("kv_indices", c_void_p), ("kv_first", c_void_p), ("T", c_int), ("heads", c_int),
+                ("kv_heads", c_int), ("hd", c_int), ("dim", c_int), ("page_size", c_int), ("num_pages", c_int),
+                ("eps", c_float), ("dtype", c_int), ("status", c_void_p)]
+
+
+class GqaAttnParams(Structure):
+    _fields_ = [("q", c_void_p), ("pool", c_void_p), ("out", c_void_p), ("positions", c_void_p), ("token_req", c_void_p),
+                ("kv_indptr", c_void_p), ("kv_indices", c_void_p), ("kv_first", c_void_p), ("sinks", c_void_p),
+                ("token_begin", c_int), ("n_tokens", c_int), ("heads", c_int), ("kv_heads", c_int), ("hd", c_int),
+                ("page_size", c_int), ("num_pages", c_int), ("window", c_int), ("scale", c_float), ("softcap", c_float),
+                ("dtype", c_int), ("status", c_void_p)]
+
+
+class MoeRouteParams(Structure):
+    _fields_ = [("logits", c_void_p), ("ld", c_longlong), ("correction", c_void_p), ("expert", c_void_p),
+                ("weight", c_void_p), ("rank", c_void_p), ("counts", c_void_p), ("gate", c_void_p), ("T", c_int),
+                ("experts", c_int), ("top", c_int), ("groups", c_int), ("keep", c_int), ("gate_col", c_int),
+                ("scale", c_float)]
+
+
+class MoePermuteParams(Structure):
+    _fields_ = [("h", c_void_p), ("ld_h", c_longlong), ("out", c_void_p), ("ld_out", c_longlong), ("expert", c_void_p),
+                ("rank", c_void_p), ("counts", c_void_p), ("slot", c_void_p), ("T", c_int), ("top", c_int),
+                ("experts", c_int), ("cols", c_int), ("dtype", c_int)]
+
+
+class MoeGemmParams(Structure):
+    _fields_ = [("A", c_void_p), ("B", c_void_p), ("B2", c_void_p), ("D", c_void_p), ("counts", c_void_p),
+                ("lda", c_longlong), ("ldb", c_longlong), ("ldd", c_longlong), ("rows", c_int), ("experts", c_int),
+                ("N", c_int), ("K", c_int), ("act", c_int), ("act_limit", c_float), ("act_alpha", c_float),
+                ("act_shift", c_float), ("dtype", c_int), ("num_ctas", c_int), ("status", c_void_p)]
+
+
+class TokenShiftParams(Structure):
+    _fields_ = [("h", c_void_p), ("ld_h", c_longlong), ("out", c_void_p), ("mu", c_void_p), ("state", c_void_p),
+                ("state_slot", c_void_p), ("positions", c_void_p), ("token_req", c_void_p), ("qo_indptr", c_void_p),
+                ("T", c_int), ("n_mix", c_int), ("num_slots", c_int), ("dtype", c_int), ("status", c_void_p)]
+
+
+class WkvParams(Structure):
+    _fields_ = [("rkvg", c_void_p), ("ld", c_longlong), ("r_off", c_int), ("k_off", c_int), ("v_off", c_int),
+                ("g_off", c_int), ("x", c_void_p), ("ld_x", c_longlong), ("u", c_void_p), ("norm", c_void_p),
+                ("S", c_void_p), ("y", c_void_p), ("ld_y", c_longlong), ("positions", c_void_p), ("qo_indptr", c_void_p),
+                ("state_slot", c_void_p), ("req_begin", c_int), ("req_count", c_int), ("heads", c_int), ("dim", c_int),
+                ("dim_real", c_int), ("num_slots", c_int), ("eps", c_float), ("dtype", c_int), ("seq_reqs", c_void_p),
+                ("num_seq", c_int), ("o", c_void_p), ("items", c_void_p), ("num_items", c_int), ("scratch", c_void_p),
+                ("scratch_floats", c_longlong), ("status", c_void_p)]
 
 
 def library_path() -> Path:

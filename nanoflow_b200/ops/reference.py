@@ -133,13 +133,20 @@ def argmax(logits, col_offset=0):
 
 # ---- layer-list models ---------------------------------------------------------------------------------
 def layernorm(x, w, b, eps):
-    return torch.nn.functional.layer_norm(x.float(), (x.shape[-1],), w.float(), b.float(), eps)
+    return torch.nn.functional.layer_norm(x.float(), (x.shape[-1],), w.float(), None if b is None else b.float(), eps)
 
 
-def gated_mlp(h, w_gate, w_up, w_down, act: str):
+def gated_act(g, u, act: str, limit=0.0, alpha=1.0, shift=0.0):
+    if act == "capped":
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        return g * torch.sigmoid(alpha * g) * (u + shift)
     f = {"silu": torch.nn.functional.silu, "relu": torch.relu,
          "gelu_tanh": lambda z: torch.nn.functional.gelu(z, approximate="tanh")}[act]
-    return (f(h.float() @ w_gate.float().t()) * (h.float() @ w_up.float().t())) @ w_down.float().t()
+    return f(g) * u
+
+
+def gated_mlp(h, w_gate, w_up, w_down, act: str, **constants):
+    return gated_act(h.float() @ w_gate.float().t(), h.float() @ w_up.float().t(), act, **constants) @ w_down.float().t()
 
 
 def _pool_rows(positions, req, kv_indptr, kv_indices, kv_first, page_size):
@@ -205,3 +212,84 @@ def head_norm_gate(o, g, w, vdim, eps):
     """o, g [T, H, vd_padded], w [H, vd_padded]: RMS norm over each head's ``vdim`` values, weight, sigmoid gate."""
     inv = torch.rsqrt(o.float().pow(2).sum(-1, keepdim=True) / vdim + eps)
     return o.float() * inv * w.float() * torch.sigmoid(g.float())
+
+
+def gqa_append(q, k, v, q_w, k_w, pool, positions, token_req, kv_indptr, kv_indices, kv_first, *, heads, kv_heads, dim, eps):
+    """q [T, heads * hd], k, v [T, kv_heads * hd] (padding columns zero), norm weights or None: keys and values go to their
+    page slots of pool [pages, 2, kv_heads, page_size, hd] (in place). Returns the normed queries."""
+    def norm(x, w, n):
+        return x if w is None else x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / n + eps) * w
+    q, k = norm(q.float(), q_w, heads * dim), norm(k.float(), k_w, kv_heads * dim)
+    T, ps, hd = k.shape[0], pool.shape[3], pool.shape[4]
+    for t in range(T):
+        row = int(_pool_rows(torch.as_tensor([int(positions[t])]), int(token_req[t]), kv_indptr, kv_indices, kv_first, ps))
+        pool[row // ps, 0, :, row % ps] = k[t].reshape(kv_heads, hd).to(pool.dtype)
+        pool[row // ps, 1, :, row % ps] = v[t].reshape(kv_heads, hd).to(pool.dtype)
+    return q
+
+
+def gqa_attention(q, pool, positions, token_req, kv_indptr, kv_indices, kv_first, *, scale, softcap=0.0, window=0, sinks=None):
+    """q [T, H, hd] -> [T, H, hd] over the paged keys and values; capped scores, exp(sink) in the denominator."""
+    T, H, hd = q.shape
+    G, ps = pool.shape[2], pool.shape[3]
+    out = torch.zeros(T, H, hd)
+    for t in range(T):
+        pos = int(positions[t])
+        keys = torch.arange(max(0, pos - window + 1) if window else 0, pos + 1)
+        rows = _pool_rows(keys, int(token_req[t]), kv_indptr, kv_indices, kv_first, ps)
+        k, v = (pool[rows // ps, j, :, rows % ps].float() for j in (0, 1))          # [n, G, hd]
+        s = torch.einsum("gmd,ngd->gmn", q[t].float().reshape(G, H // G, hd), k).reshape(H, -1) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        if sinks is not None:
+            s = torch.cat([s, sinks.float()[:, None]], dim=1)
+        p = torch.softmax(s, dim=-1)[:, :keys.numel()].reshape(G, H // G, -1)
+        out[t] = torch.einsum("gmn,ngd->gmd", p, v).reshape(H, hd)
+    return out
+
+
+def token_shift(h, mu, state, positions, qo_indptr, state_ref):
+    """h [T, W], mu [n, W] -> [T, n, W]; ``state`` [slots, 2, W] holds each request's last row (half ``ref & 1`` is read,
+    the other written)."""
+    prev = torch.zeros_like(h)
+    prev[1:] = h[:-1]
+    for b in range(len(qo_indptr) - 1):
+        t0, t1, ref = int(qo_indptr[b]), int(qo_indptr[b + 1]), int(state_ref[b])
+        prev[t0] = state[ref >> 1, ref & 1] if int(positions[t0]) else 0.0
+        state[ref >> 1, (ref & 1) ^ 1] = h[t1 - 1]
+    return h[:, None] + (prev - h)[:, None] * mu[None]
+
+
+def wkv(r, k, v, x, u, state, positions, qo_indptr, state_ref):
+    """r, k, v, x [T, H, d] (x: log of the decay's negative log), u [H, d], state [slots, H, d, d], updated in place."""
+    out = torch.zeros(v.shape)
+    w = torch.exp(-torch.exp(x.float()))
+    for b in range(len(qo_indptr) - 1):
+        t0, t1, slot = int(qo_indptr[b]), int(qo_indptr[b + 1]), int(state_ref[b]) >> 1
+        S = state[slot].clone() if int(positions[t0]) else torch.zeros_like(state[slot])
+        for t in range(t0, t1):
+            kv = k[t].float()[:, :, None] * v[t].float()[:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S + u[:, :, None] * kv, r[t].float())
+            S = w[t][:, :, None] * S + kv
+        state[slot] = S
+    return out
+
+
+def head_norm_silu(o, g, w, dim, eps):
+    """o, g, w [.., H, d_padded]: RMS norm over each head's ``dim`` values, weight, SiLU gate."""
+    inv = torch.rsqrt(o.float().pow(2).sum(-1, keepdim=True) / dim + eps)
+    return o.float() * inv * w.float() * torch.nn.functional.silu(g.float())
+
+
+def moe_route(logits, correction, top, groups, keep, scale):
+    """(experts [T, top], weights [T, top]) from router logits [T, E]."""
+    s = torch.sigmoid(logits.float())
+    choice = s if correction is None else s + correction
+    if groups > 1:
+        c = choice.reshape(len(s), groups, -1)
+        best = c.topk(min(2, c.shape[-1]), dim=-1).values.sum(-1).topk(keep, dim=-1).indices
+        allowed = torch.zeros(len(s), groups, dtype=torch.bool).scatter_(1, best, True)
+        choice = c.masked_fill(~allowed[:, :, None], float("-inf")).reshape(len(s), -1)
+    idx = choice.topk(top, dim=-1).indices
+    w = s.gather(1, idx)
+    return idx, w / (w.sum(-1, keepdim=True) + 1e-20) * scale

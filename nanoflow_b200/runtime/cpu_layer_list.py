@@ -29,13 +29,16 @@ class CpuLayerListEngine:
         m = self.model
         self.num_slots = (self.eng.state_slots or self.eng.max_batch_size) if m.has_state else 0
         self.pools, self.state = [], []
+        n = self.num_slots
         for r in m.runs:
             s = m.layers[r.layer].mixer
-            latent = s.kind == "latent_attention"
-            self.pools.append(torch.zeros(num_pages, PAGE, m.latent_ld(s)) if latent else None)
-            d, v, n = round8(s.dim), round8(s.vdim), self.num_slots
-            self.state.append(None if latent else (torch.zeros(n, s.heads, d, v), torch.zeros(n, s.heads, 2, d),
-                                                   torch.zeros(n, s.heads, 2)))
+            d, v = round8(s.dim), round8(s.vdim)
+            self.pools.append(torch.zeros(num_pages, PAGE, m.latent_ld(s)) if s.kind == "latent_attention" else
+                              torch.zeros(num_pages, 2, s.kv_heads, PAGE, m.attn_hd(s)) if s.kind == "attention" else None)
+            self.state.append((torch.zeros(n, s.heads, d, v), torch.zeros(n, s.heads, 2, d), torch.zeros(n, s.heads, 2))
+                              if s.kind == "mlstm" else
+                              (torch.zeros(n, s.heads, d, d), torch.zeros(n, 2, m.width_p)) if s.kind == "wkv" else None)
+        self.v_first: Optional[torch.Tensor] = None
         self.sampled = torch.zeros(self.eng.max_sample_rows or self.eng.max_batch_size, dtype=torch.int32)
         self._staged: Optional[BatchPlan] = None
         self._inflight: List[np.ndarray] = []
@@ -45,7 +48,7 @@ class CpuLayerListEngine:
     # ---- one iteration --------------------------------------------------------------------------------
     def _norm(self, x, n):
         m = self.model
-        y = ref.layernorm(x, n.w[:m.hidden_size], n.b[:m.hidden_size], m.norm_eps) if m.norm_kind == "layer" else \
+        y = ref.layernorm(x, n.w[:m.hidden_size], None if n.b is None else n.b[:m.hidden_size], m.norm_eps) if m.norm_kind == "layer" else \
             ref.rmsnorm(x, n.w[:m.hidden_size], m.norm_eps)
         return torch.nn.functional.pad(y, (0, m.width_p - m.hidden_size))
 
@@ -71,6 +74,50 @@ class CpuLayerListEngine:
         return ref.head_norm_gate(o, g.reshape(T, H, v), lw.norm.reshape(H, v), s.vdim, self.model.norm_eps).reshape(T, -1) @ \
             lw.w_o.t()
 
+    def _attention(self, r, s, lw, h, plan):
+        m, T = self.model, h.shape[0]
+        H, G, hd = s.heads, s.kv_heads, m.attn_hd(s)
+        q, k, v = (h @ lw.w_in.t()).split([H * hd, G * hd, G * hd], dim=1)
+        if s.value_mix and r == m.first_value_run:
+            self.v_first = v
+        elif s.value_mix:
+            v = (1.0 - lw.value_lambda) * v + lw.value_lambda * self.v_first
+        pages = (plan.positions, plan.token_req, plan.kv_indptr, plan.kv_indices, plan.kv_first)
+        q = ref.gqa_append(q, k, v, lw.q_norm, lw.k_norm, self.pools[r], *pages, heads=H, kv_heads=G, dim=s.dim,
+                           eps=m.norm_eps)
+        o = ref.gqa_attention(q.reshape(T, H, hd), self.pools[r], *pages, scale=s.scale, softcap=s.softcap or 0.0,
+                              sinks=lw.sinks)
+        return o.reshape(T, -1) @ lw.w_o.t()
+
+    def _wkv(self, r, s, lw, h, plan):
+        m, T, H, d = self.model, h.shape[0], s.heads, round8(s.dim)
+        S, before = self.state[r]
+        mix = ref.token_shift(h, lw.mu, before, plan.positions, plan.qo_indptr, plan.state_ref)
+        proj = [(mix[:, j] @ w.t()).reshape(T, H, d) for j, w in enumerate(lw.w_in.chunk(4))]
+        x = torch.tanh(mix[:, 4] @ lw.w_down.t()) @ lw.w_up.t() + lw.w_bias
+        o = ref.wkv(proj[0], proj[1], proj[2], x.reshape(T, H, d), lw.u.reshape(H, d), S, plan.positions, plan.qo_indptr,
+                    plan.state_ref)
+        return ref.head_norm_silu(o, proj[3], lw.norm.reshape(H, d), s.dim, m.norm_eps).reshape(T, -1) @ lw.w_o.t()
+
+    # ---- feed-forwards ----------------------------------------------------------------------------------
+    def _dense(self, s, lw, h):
+        a = s.act
+        return ref.gated_mlp(h, lw.w_gate, lw.w_up, lw.w_down, a.name, limit=a.limit, alpha=a.alpha, shift=a.shift)
+
+    def _moe(self, s, lw, h):
+        logits = h @ lw.router.t()
+        idx, weight = ref.moe_route(logits[:, :s.experts], lw.correction, s.top, s.groups, s.keep, s.scale)
+        mats = [t.chunk(s.experts) for t in (lw.w_gate, lw.w_up, lw.w_down)]
+        a, out = s.expert.act, torch.zeros_like(h)
+        for e in range(s.experts):
+            t, k = (idx == e).nonzero(as_tuple=True)
+            if t.numel():
+                y = ref.gated_mlp(h[t], mats[0][e], mats[1][e], mats[2][e], a.name, limit=a.limit, alpha=a.alpha, shift=a.shift)
+                out.index_add_(0, t, y * weight[t, k][:, None])
+        if s.shared is not None:
+            out += torch.sigmoid(logits[:, s.experts:s.experts + 1]) * self._dense(s.shared, lw.shared, h)
+        return out
+
     def update(self, plan: BatchPlan) -> None:
         self._staged = plan
 
@@ -80,18 +127,23 @@ class CpuLayerListEngine:
         ids = torch.from_numpy(plan.host_ids).long().clone()
         fb = torch.from_numpy(plan.feedback_src).long()
         ids[fb >= 0] = self.sampled[fb[fb >= 0]].long()
-        x = self._norm(w.embed[ids][:, :m.hidden_size], w.embed_norm)
+        W = m.hidden_size
+        after = lambda y, n: y if n is None else self._norm(y[:, :W], n)
+        x = after(w.embed[ids] * m.embed_scale, w.embed_norm)
         for r, run in enumerate(m.runs):
             spec, lw = m.layers[run.layer], w.layers[run.layer]
             if run.step is not None:
                 x = x + w.loop_steps[run.step]
-            mix = self._latent_attention if spec.mixer.kind == "latent_attention" else self._mlstm
-            y = mix(r, spec.mixer, lw.mixer, self._norm(x[:, :m.hidden_size], lw.norm_in), plan)
-            x = x + self._norm(y[:, :m.hidden_size], lw.norm_out)
-            if spec.mlp is not None:
-                h = self._norm(x[:, :m.hidden_size], lw.mlp_in)
-                y = ref.gated_mlp(h, lw.w_gate, lw.w_up, lw.w_down, spec.mlp.act)
-                x = x + self._norm(y[:, :m.hidden_size], lw.mlp_out)
+            h = self._norm(x[:, :W], lw.norm_in)
+            y = MIXERS[spec.mixer.kind](self, r, spec.mixer, lw.mixer, h, plan)
+            if spec.mlp is None:
+                x = x + after(y, lw.norm_out)
+            elif m.parallel:
+                x = x + (y + FEED_FORWARDS[spec.mlp.kind](self, spec.mlp, lw.mlp, h))
+            else:
+                x = x + after(y, lw.norm_out)
+                h = self._norm(x[:, :W], lw.mlp_in)
+                x = x + after(FEED_FORWARDS[spec.mlp.kind](self, spec.mlp, lw.mlp, h), lw.mlp_out)
         rows = torch.from_numpy(plan.sample_rows).long()
         self._logits = (self._norm(x[rows][:, :m.hidden_size], w.final_norm) @ w.lm_head.t())[:, :m.vocab_size]
         toks = self._logits.argmax(dim=-1).int()
@@ -122,3 +174,8 @@ class CpuLayerListEngine:
 
     def finalize(self) -> None:
         self._inflight.clear()
+
+
+MIXERS = {"latent_attention": CpuLayerListEngine._latent_attention, "mlstm": CpuLayerListEngine._mlstm,
+          "attention": CpuLayerListEngine._attention, "wkv": CpuLayerListEngine._wkv}
+FEED_FORWARDS = {"dense": CpuLayerListEngine._dense, "moe": CpuLayerListEngine._moe}

@@ -87,6 +87,13 @@ LatentAttnParams = _ops.LatentAttnParams
 LatentGatherParams = _ops.LatentGatherParams
 MlstmParams = _ops.MlstmParams
 HeadNormGateParams = _ops.HeadNormGateParams
+GqaAppendParams = _ops.GqaAppendParams
+GqaAttnParams = _ops.GqaAttnParams
+MoeRouteParams = _ops.MoeRouteParams
+MoePermuteParams = _ops.MoePermuteParams
+MoeGemmParams = _ops.MoeGemmParams
+TokenShiftParams = _ops.TokenShiftParams
+WkvParams = _ops.WkvParams
 
 KERNEL_OF = {
     GemmParams: "nfk_gemm_bf16", RopeAppendParams: "nfk_rope_append", RopeTableParams: "nfk_rope_table",
@@ -95,6 +102,8 @@ KERNEL_OF = {
     ArgmaxCombineParams: "nfk_argmax_combine_p", CopyColsParams: "nfk_copy_cols_p",
     ResidualNormParams: "nfk_residual_norm", LatentAppendParams: "nfk_latent_append",
     LatentGatherParams: "nfk_latent_gather", LatentAttnParams: "nfk_latent_attn", HeadNormGateParams: "nfk_head_norm_gate",
+    GqaAppendParams: "nfk_gqa_append", GqaAttnParams: "nfk_gqa_attn", MoeRouteParams: "nfk_moe_route",
+    MoePermuteParams: "nfk_moe_permute", MoeGemmParams: "nfk_moe_gemm", TokenShiftParams: "nfk_token_shift",
     MemcpyParams: "nfk_memcpy_p", Memcpy2DParams: "nfk_memcpy2d_p", KvMoveParams: "nfk_kv_move_p", SleepParams: "nfk_sleep_p",
 }
 

@@ -11,11 +11,21 @@ one GPU, one stream. Per layer run:
   rows as keys and values at once, and a second block-diagonal GEMM applies the value matrices. Longer
   portions gather the latents they can see, expand them to keys and values of all heads with one GEMM, and
   run the tcgen05 prefill kernel over those;
+* grouped-query attention: queries and keys normed, values mixed, both appended to the paged pool; single tokens
+  on the split-KV decode kernel, portions on the tcgen05 prefill kernel (in 32-bit, and for head sizes those are
+  not built for, one simple kernel);
 * mLSTM: one kernel for requests with one token, one for longer portions, then head norm and output gate;
-* output projection, and one kernel for: norm of the sublayer's output, residual sum in fp32, the step
-  vector of a loop pass, and the norm the next sublayer reads.
+* WKV: every stream's mix with the previous token (kept per request), the four projections as one block-diagonal
+  product, the low-rank decay, one kernel for single tokens and one for portions (chunks, or token by token),
+  both with head norm and gate;
+* output projection;
+* feed-forward: gated, or a mixture of experts (router product, routing, rows in expert order, two products per
+  expert, the shared expert);
+* one kernel for: norm of the sublayer's output or the weighted sum of experts and shared expert, residual sum in
+  fp32, the step vector of a loop pass, and the norm the next sublayer reads.
 
-A new kind of mixer needs a spec and weights in ``models/layer_list.py`` and a builder in ``MIXERS``.
+A new kind of mixer needs a spec and weights in ``models/layer_list.py`` and a builder in ``MIXERS``, a new kind of
+feed-forward one in ``FEED_FORWARDS``.
 """
 from __future__ import annotations
 
@@ -26,13 +36,14 @@ import numpy as np
 import torch
 
 from .. import ops
-from ..models.layer_list import PREFILL_HEAD_DIM, LayerListConfig, NormWeights, round8
-from ..ops import ACTS, NORMS, dtype_code
+from ..models.layer_list import PREFILL_HEAD_DIM, WKV_CHUNK_DIM, ActSpec, LayerListConfig, NormWeights, round8
+from ..ops import ACTS, LIN_ACTS, NORMS, dtype_code
 from ..ops.layer_list import mlstm_scratch_floats
 from ..serving.scheduler import BatchPlan
-from .engine import GEMM_WS_BYTES, Engine, MetaLayout
-from .graph import (ArgmaxParams, AttnParams, GemmParams, HeadNormGateParams, LatentAppendParams,
-                    LatentAttnParams, LatentGatherParams, MemcpyParams, MlstmParams, OpGraph, ResidualNormParams)
+from .engine import DECODE_MAX_CHUNKS, DECODE_SPLIT_ROWS, GEMM_WS_BYTES, Engine, MetaLayout
+from .graph import (ArgmaxParams, AttnParams, GemmParams, GqaAppendParams, GqaAttnParams, HeadNormGateParams,
+                    LatentAppendParams, LatentAttnParams, LatentGatherParams, MemcpyParams, MlstmParams, MoeGemmParams,
+                    MoePermuteParams, MoeRouteParams, OpGraph, ResidualNormParams, TokenShiftParams, WkvParams)
 from .pipeline import _ptr
 
 PAGE = 16
@@ -40,6 +51,8 @@ QUERY_TILE = 128             # query tokens per work item of the prefill attenti
 MLSTM_CHUNK = 64             # tokens per chunk of the chunked mLSTM kernel
 MLSTM_COLS = 64              # columns of the state per CTA of that kernel
 SEGMENT_ITEMS = 48           # most segments that prompt portions are cut into for the mLSTM kernel
+WKV_CHUNK = 64               # tokens per chunk of the chunked WKV kernels
+WKV_SPARE_CHUNKS = 64        # chunks beyond whole ones that their scratch has room for; further portions go token by token
 
 
 class PathGroup:
@@ -73,6 +86,11 @@ class LayerListEngine(Engine):
             key = (s.window or 0, m.expands(s))
             if not any((g.window, g.expands) == key for g in self.groups):
                 self.groups.append(PathGroup(len(self.groups), *key))
+        # query heads per KV head of the attention layers on the tcgen05 prefill kernel: a work list for each
+        self.attn_groups = sorted({s.group for s in m.run_specs("attention") if m.attn_on_tensor_cores(s)})
+        self.wkv_cap = 0
+        if m.dtype == torch.bfloat16 and any(round8(s.dim) <= WKV_CHUNK_DIM for s in m.run_specs("wkv")):
+            self.wkv_cap = T // WKV_CHUNK + min(B, WKV_SPARE_CHUNKS)
         self.x_pages = self._expand_pages()
         self._alloc_state()
         self.num_pages = int(num_pages or e.num_pages or self._derive_num_pages(T, B))
@@ -81,8 +99,12 @@ class LayerListEngine(Engine):
             extra[g.name("abs")] = T
             if g.expands:
                 extra.update({g.name("xptr"): B + 1, g.name("xpage"): self.x_pages, g.name("xitem"): 3 * (T // QUERY_TILE + B + 1)})
-        if m.has_state:
+        for n in self.attn_groups:
+            extra[f"gitem{n}"] = 3 * (T // (QUERY_TILE // n) + B + 1)
+        if m.run_specs("mlstm"):
             extra["segs"] = 4 * max(B, SEGMENT_ITEMS)
+        if m.run_specs("wkv"):
+            extra.update(wkv_items=4 * max(1, self.wkv_cap), wkv_seq=B, wkv_all=B)
         self._make_metadata(MetaLayout(T, B, self.nano_sizes, self.num_pages, 0, self.S_cap, extra))
         self.meta = {n: self._meta_view(n) for n in self.layout.off}
         self._alloc_buffers()
@@ -104,20 +126,24 @@ class LayerListEngine(Engine):
 
     def _alloc_state(self) -> None:
         m, dev = self.model, self.device
-        self.state: List[Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]]] = []
+        self.state: List[Optional[Tuple[torch.Tensor, ...]]] = []
+        n = self.num_slots
+        z = lambda *shape, dtype=torch.float32: torch.zeros(*shape, dtype=dtype, device=dev)
         for r in m.runs:
             s = m.layers[r.layer].mixer
-            if s.kind != "mlstm":
+            d, v = round8(s.dim), round8(s.vdim)
+            if s.kind == "mlstm":
+                self.state.append((z(n, s.heads, d, v), z(n, s.heads, 2, d), z(n, s.heads, 2)))
+            elif s.kind == "wkv":
+                self.state.append((z(n, s.heads, d, d), z(n, 2, m.width_p, dtype=m.dtype)))
+            else:
                 self.state.append(None)
-                continue
-            d, v, n = round8(s.dim), round8(s.vdim), self.num_slots
-            z = lambda *shape: torch.zeros(*shape, dtype=torch.float32, device=dev)
-            self.state.append((z(n, s.heads, d, v), z(n, s.heads, 2, d), z(n, s.heads, 2)))
 
     def _widths(self) -> Dict[str, int]:
         """Columns of the shared activation buffers (the widest layer's)."""
         m = self.model
-        w = dict(proj=8, gates=8, attn=8, q_lat=0, o_lat=0, o_rec=8, act=8, kv=0, cg=0)
+        w = dict(proj=8, gates=8, attn=8, q_lat=0, o_lat=0, o_rec=8, act=8, kv=0, cg=0, qn=0, v_first=0, mix=0, lora=0,
+                 router=0, e_in=0, e_act=0, e_out=0, e_top=0)
         up = lambda k, n: w.__setitem__(k, max(w[k], n))
         for lay in m.layers:
             s = lay.mixer
@@ -130,14 +156,38 @@ class LayerListEngine(Engine):
                 if m.expands(s):
                     up("kv", s.heads * 2 * PREFILL_HEAD_DIM)
                     up("cg", ld)
+            elif s.kind == "attention":
+                hd = m.attn_hd(s)
+                up("proj", (s.heads + 2 * s.kv_heads) * hd)
+                up("qn", s.heads * hd)
+                up("attn", s.heads * hd)
+                if s.value_mix:
+                    up("v_first", s.kv_heads * hd)
+            elif s.kind == "wkv":
+                d = round8(s.dim)
+                up("mix", 5 * m.width_p)
+                up("proj", 4 * s.heads * d)
+                up("lora", round8(s.rank))
+                up("gates", s.heads * d)
+                up("o_rec", s.heads * d)
+                up("attn", s.heads * d)
             else:
                 d, v = round8(s.dim), round8(s.vdim)
                 up("proj", s.heads * 2 * (d + v))
                 up("gates", round8(2 * s.heads))
                 up("o_rec", s.heads * v)
                 up("attn", s.heads * v)
-            if lay.mlp is not None:
-                up("act", round8(lay.mlp.ff))
+            f = lay.mlp
+            if f is not None and f.kind == "dense":
+                up("act", round8(f.ff))
+            elif f is not None:
+                up("router", round8(f.router_cols))
+                up("e_in", f.top * m.width_p)
+                up("e_act", f.top * round8(f.expert.ff))
+                up("e_out", f.top * m.width_p)
+                up("e_top", f.top)
+                if f.shared is not None:
+                    up("act", round8(f.shared.ff))
         return w
 
     def _derive_num_pages(self, T: int, B: int) -> int:
@@ -145,15 +195,27 @@ class LayerListEngine(Engine):
         free, total = torch.cuda.mem_get_info(self.device)
         w = self._widths()
         es = m.elem_bytes
-        act = T * (4 * m.width_p + es * (2 * m.width_p + w["proj"] + w["attn"] + 2 * w["q_lat"] + w["act"]) +
-                   4 * (w["gates"] + w["o_rec"]))
+        act = T * (4 * m.width_p + es * (3 * m.width_p + w["proj"] + w["attn"] + 2 * w["q_lat"] + w["act"] + w["qn"] +
+                                         w["v_first"] + w["mix"] + w["lora"] + w["e_in"] + w["e_act"] + w["e_out"]) +
+                   4 * (w["gates"] + w["o_rec"] + w["router"] + 5 * w["e_top"]))
+        act += self._decode_ws_floats() * 4 + self._wkv_scratch_floats() * 4
         act += self.x_pages * PAGE * (w["kv"] + w["cg"]) * es + self.S_cap * (es * m.width_p + 4 * m.vocab_p)
         budget = free - total * (1.0 - e.gpu_mem_fraction) - act - (1 << 30)
         per_page = max(1, m.kv_bytes_per_token_local()) * PAGE
         n = int(min(budget // per_page, 1 << 22))
         if n < 64:
-            raise RuntimeError(f"not enough GPU memory for a latent pool ({free >> 20} MiB free)")
+            raise RuntimeError(f"not enough GPU memory for a page pool ({free >> 20} MiB free)")
         return n
+
+    def _decode_ws_floats(self) -> int:
+        """Partial results of split-KV decode attention."""
+        hd = max([self.model.attn_hd(s) for s in self.model.run_specs("attention") if self.model.attn_on_tensor_cores(s)],
+                 default=0)
+        return DECODE_SPLIT_ROWS * DECODE_MAX_CHUNKS * (hd + 2) if hd else 0
+
+    def _wkv_scratch_floats(self) -> int:
+        sizes = [(s.heads, round8(s.dim)) for s in self.model.run_specs("wkv")]
+        return max([self.wkv_cap * h * (d * d + d) for h, d in sizes if d <= WKV_CHUNK_DIM], default=0)
 
     def _alloc_buffers(self) -> None:
         m, T, dev = self.model, self.T, self.device
@@ -162,14 +224,27 @@ class LayerListEngine(Engine):
         self.x = P(T, m.width_p, f32, "x")
         self.h = P(T, m.width_p, dt, "h")
         self.y = P(T, m.width_p, dt, "y")
+        self.y2 = P(T, m.width_p, dt, "y2") if m.parallel or m.run_moes() else None
         flat = lambda k, dtype, rows=T: P(1, max(8, rows * w[k]), dtype, k).view(-1)
         self.flat = {"proj": flat("proj", dt), "attn": flat("attn", dt), "act": flat("act", dt), "gates": flat("gates", f32),
                      "o_rec": flat("o_rec", f32), "q_lat": flat("q_lat", dt), "o_lat": flat("q_lat", dt),
-                     "kv": flat("kv", dt, self.x_pages * PAGE), "cg": flat("cg", dt, self.x_pages * PAGE)}
+                     "kv": flat("kv", dt, self.x_pages * PAGE), "cg": flat("cg", dt, self.x_pages * PAGE),
+                     "router": flat("router", f32)}
+        self.flat.update({k: flat(k, dt) for k in ("qn", "v_first", "mix", "lora", "e_in", "e_act", "e_out")})
+        i32 = torch.int32
+        self.moe_ids = {k: flat("e_top", f32 if k == "weight" else i32) for k in ("expert", "rank", "slot", "weight")}
+        self.moe_gate = P(1, T, f32, "moe_gate").view(-1)
+        # one counter per expert and layer run, cleared from zeros at the start of an iteration
+        moes = [m.layers[r.layer].mlp for r in m.runs]
+        sizes = [f.experts if f is not None and f.kind == "moe" else 0 for f in moes]
+        self.moe_counts = torch.zeros(max(1, sum(sizes)), dtype=i32, device=dev)
+        self.moe_zeros = torch.zeros_like(self.moe_counts)
+        self.moe_counts_of = [c for c in self.moe_counts[:sum(sizes)].split(sizes)] if sum(sizes) else [None] * len(sizes)
+        self.decode_ws = torch.empty(max(8, self._decode_ws_floats()), dtype=f32, device=dev)
+        self.wkv_ws = torch.empty(max(8, self._wkv_scratch_floats()), dtype=f32, device=dev)
         self.h_s = P(self.S_cap, m.width_p, dt, "sample_h")
         self.logits = P(self.S_cap, m.vocab_p, f32, "logits")
-        self.pools = [torch.zeros(self.num_pages, PAGE, m.latent_ld(s.mixer), dtype=dt, device=dev)
-                      if s.mixer.kind == "latent_attention" else None for s in (m.layers[r.layer] for r in m.runs)]
+        self.pools = [self._pool(m.layers[r.layer].mixer) for r in m.runs]
         self.arange = torch.arange(self.x_pages + 1, dtype=torch.int32, device=dev)
         heads = max([s.heads * (m.latent_ld(s) + 2) for s in m.run_specs("latent_attention")], default=0)
         self.latent_ws = torch.empty(max(8, 160 * heads), dtype=f32, device=dev)
@@ -186,6 +261,12 @@ class LayerListEngine(Engine):
         self.bufs.sampled = self._plain(self.S_cap, dtype=torch.int32, name="sampled")
         self.bufs.status = torch.zeros(1, dtype=torch.int32, device=dev)
         self.bufs.logits = self.logits
+
+    def _pool(self, s) -> Optional[torch.Tensor]:
+        m, z = self.model, lambda *shape: torch.zeros(self.num_pages, *shape, dtype=self.model.dtype, device=self.device)
+        if s.kind == "latent_attention":
+            return z(PAGE, m.latent_ld(s))
+        return z(2, s.kv_heads, PAGE, m.attn_hd(s)) if s.kind == "attention" else None
 
     def view(self, name: str, cols: int, rows: Optional[int] = None) -> torch.Tensor:
         rows = rows or self.T
@@ -205,6 +286,9 @@ class LayerListEngine(Engine):
         self._op("kv_indices_h2d", MemcpyParams(dst=c_void_p(self.meta_dev.data_ptr() + 4 * lay.off["kv_indices"]),
                                                 src=c_void_p(0), elem_bytes=4, count=0),
                  dyn=[("src", g.symbol("kv_src")), ("count", g.symbol("kv_words"))])
+        if m.run_moes():
+            self._op("moe_counts", MemcpyParams(dst=_ptr(self.moe_counts), src=_ptr(self.moe_zeros), elem_bytes=4,
+                                                count=self.moe_counts.numel()))
         # the stream's step before each run, as (vector added, norm of its mixer's input)
         step = lambda r: None if m.runs[r].step is None else w.loop_steps[m.runs[r].step]
         self._residual("embedding", None, w.embed_norm, w.layers[m.runs[0].layer].norm_in, step(0), embed=True)
@@ -214,19 +298,20 @@ class LayerListEngine(Engine):
             nxt = None if last else w.layers[m.runs[r + 1].layer].norm_in
             add = None if last else step(r + 1)
             MIXERS[spec.mixer.kind](self, r, run.layer, spec.mixer, lw.mixer)
+            y, out, more = self.y, lw.norm_out, {}         # what joins the stream at the end of the layer
             if spec.mlp is not None:
-                self._residual(f"R{r}.mid", self.y, lw.norm_out, lw.mlp_in, None, layer=r)
-                act = self.view("act", round8(spec.mlp.ff))
-                self._gemm(f"R{r}.gate_up", self.h, lw.w_gate, act, rows=T, up=lw.w_up, act=spec.mlp.act,
-                           key=f"l{run.layer}.gate_up", layer=r)
-                self._gemm(f"R{r}.down", act, lw.w_down, self.y, rows=T, key=f"l{run.layer}.down", layer=r)
-            out = lw.mlp_out if spec.mlp is not None else lw.norm_out
+                if not m.parallel:
+                    self._residual(f"R{r}.mid", self.y, lw.norm_out, lw.mlp_in, None, layer=r)
+                    out = lw.mlp_out
+                more = FEED_FORWARDS[spec.mlp.kind](self, r, run.layer, spec.mlp, lw.mlp)
+                if not m.parallel:
+                    y = more.pop("y2", None) if "y2_gate" not in more else None
             if last and self.taps is None:
                 # only the sampled rows go on
-                self._residual("final", self.y, out, w.final_norm, None, sampled=True)
+                self._residual("final", y, out, w.final_norm, None, sampled=True, more=more)
             else:
                 tap_add = add if self.taps is None else None
-                self._residual(f"R{r}.out", self.y, out, None if (last or self.taps is not None) else nxt, tap_add, layer=r)
+                self._residual(f"R{r}.out", y, out, None if (last or self.taps is not None) else nxt, tap_add, layer=r, more=more)
                 if self.taps is not None:
                     self._op(f"R{r}.tap", MemcpyParams(dst=_ptr(self.taps[r]), src=_ptr(self.x), elem_bytes=4 * m.width_p,
                                                        count=0), dyn=[("count", T)], layer=r)
@@ -250,7 +335,9 @@ class LayerListEngine(Engine):
                                   kernel=kernel, layer=layer, nano=0)
 
     def _residual(self, name, y, norm_in: Optional[NormWeights], norm_out: Optional[NormWeights], add, *, embed=False,
-                  sampled=False, layer=-1) -> None:
+                  sampled=False, layer=-1, more: Optional[dict] = None) -> None:
+        """``more``: what a feed-forward adds to the sum besides ``y``: ``y2`` with ``y2_gate`` per row, and expert rows
+        (``e_out``, ``e_slot``, ``e_weight``, ``e_top``)."""
         m, kind = self.model, NORMS[self.model.norm_kind]
         p = ResidualNormParams()
         p.x, p.ld_x = _ptr(self.x), self.x.stride(0)
@@ -258,10 +345,17 @@ class LayerListEngine(Engine):
             p.table, p.ld_table, p.vocab = _ptr(self.w.embed), self.w.embed.stride(0), m.vocab_size
             p.host_ids, p.feedback_src = _ptr(self.meta["host_ids"]), _ptr(self.meta["feedback_src"])
             p.prev_tokens = _ptr(self.bufs.sampled)
+            p.src_scale = m.embed_scale
         elif y is not None:
             p.y, p.ld_y = _ptr(y), y.stride(0)
         if norm_in is not None:
             p.in_w, p.in_b, p.in_kind = _ptr(norm_in.w), _ptr(norm_in.b), kind
+        more = more or {}
+        if more.get("y2") is not None:
+            p.y2, p.ld_y2, p.y2_gate = _ptr(more["y2"]), more["y2"].stride(0), _ptr(more.get("y2_gate"))
+        if more.get("e_out") is not None:
+            p.e_out, p.ld_e, p.e_rows = _ptr(more["e_out"]), more["e_out"].stride(0), more["e_out"].shape[0]
+            p.e_slot, p.e_weight, p.e_top = _ptr(more["e_slot"]), _ptr(more["e_weight"]), more["e_top"]
         p.add = _ptr(add)
         if norm_out is not None:
             h = self.h_s if sampled else self.h
@@ -271,15 +365,16 @@ class LayerListEngine(Engine):
         p.cols, p.eps, p.dtype, p.status = m.hidden_size, m.norm_eps, self.code, _ptr(self.bufs.status)
         self._op(name, p, dyn=[("rows", "n_sample" if sampled else "T")], layer=layer)
 
-    def _gemm(self, name, a, wt, out, *, rows: str, up=None, act="silu", d32=None, f32_col0=0, groups=1, group_k=0, k=0,
-              key="", layer=-1) -> None:
+    def _gemm(self, name, a, wt, out, *, rows: str, up=None, act: ActSpec = ActSpec("silu"), lin_act=None, bias=None, d32=None,
+              f32_col0=0, groups=1, group_k=0, k=0, key="", layer=-1) -> None:
         """out[rows, N] = a @ wt^T. ``d32``: columns from ``f32_col0`` on leave as fp32; ``groups`` > 1:
         block-diagonal (each group of rows of ``wt`` sees ``k`` columns of ``a``, ``group_k`` apart)."""
         p = GemmParams()
         p.A, p.B, p.B2, p.D = _ptr(a), _ptr(wt), _ptr(up), _ptr(out)
         p.lda, p.ldb, p.ldd = a.stride(0), wt.stride(0), (out.stride(0) if out is not None else wt.shape[0])
         p.N, p.K = wt.shape[0], k or wt.shape[1]
-        p.epilogue, p.act = (1 if up is not None else 0), ACTS[act]
+        p.epilogue, p.lin_act, p.bias = (1 if up is not None else 0), LIN_ACTS[lin_act], _ptr(bias)
+        p.act, p.act_limit, p.act_alpha, p.act_shift = ACTS[act.name], act.limit, act.alpha, act.shift
         if d32 is not None:
             p.D32, p.ld32, p.f32_col0 = _ptr(d32), d32.stride(0), f32_col0
         p.groups, p.group_k = groups, group_k
@@ -373,6 +468,124 @@ class LayerListEngine(Engine):
         self._op(f"R{r}.head_norm", hp, dyn=[("T", T)], layer=r)
         self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
 
+    def _attention(self, r: int, layer: int, s, lw) -> None:
+        m, g, T, meta, st = self.model, self.g, "T", self.meta, _ptr(self.bufs.status)
+        H, G, hd, pool = s.heads, s.kv_heads, m.attn_hd(s), self.pools[r]
+        proj, qn, attn = self.view("proj", (H + 2 * G) * hd), self.view("qn", H * hd), self.view("attn", H * hd)
+        self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, key=f"l{layer}.in", layer=r)
+        mode = 0 if not s.value_mix else 1 if r == m.first_value_run else 2
+        ap = GqaAppendParams(src=_ptr(proj), ld_src=proj.stride(0), q_off=0, k_off=H * hd, v_off=(H + G) * hd, q_out=_ptr(qn),
+                             q_w=_ptr(lw.q_norm), k_w=_ptr(lw.k_norm), v_first=_ptr(self.flat["v_first"]), v_mode=mode,
+                             v_lambda=lw.value_lambda, pool=_ptr(pool), positions=_ptr(meta["positions"]),
+                             token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
+                             kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), T=0, heads=H, kv_heads=G,
+                             hd=hd, dim=s.dim, page_size=PAGE, num_pages=self.num_pages, eps=m.norm_eps, dtype=self.code,
+                             status=st)
+        self._op(f"R{r}.gqa_append", ap, dyn=[("T", T)], layer=r)
+        if m.attn_on_tensor_cores(s):
+            def params() -> AttnParams:
+                p = AttnParams()
+                p.q, p.out, p.kv_pool = _ptr(qn), _ptr(attn), _ptr(pool)
+                p.qo_indptr, p.kv_indptr = _ptr(meta["qo_indptr"]), _ptr(meta["kv_indptr"])
+                p.kv_indices, p.kv_last_page_len = _ptr(meta["kv_indices"]), _ptr(meta["kv_last_page_len"])
+                p.q_heads, p.kv_heads, p.head_dim, p.page_size, p.num_pages = H, G, hd, PAGE, self.num_pages
+                p.sm_scale, p.softcap, p.sinks, p.precise, p.status = s.scale, s.softcap or 0.0, _ptr(lw.sinks), 1, st
+                return p
+
+            d = params()
+            d.workspace, d.max_chunks = _ptr(self.decode_ws), 1
+            self._op(f"R{r}.attn_decode", d, kernel="nfk_attn_decode",
+                     dyn=[("req_count", "n_dec"), ("chunk_pages", g.symbol("dec_chunk_pages")),
+                          ("max_chunks", g.symbol("dec_max_chunks"))], layer=r)
+            p = params()
+            p.items = _ptr(meta[f"gitem{s.group}"])
+            self._op(f"R{r}.attn_prefill", p, kernel="nfk_attn_prefill_ws",
+                     dyn=[("num_items", g.symbol(f"n_gitems{s.group}"))], layer=r)
+        else:
+            gp = GqaAttnParams(q=_ptr(qn), pool=_ptr(pool), out=_ptr(attn), positions=_ptr(meta["positions"]),
+                               token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
+                               kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), sinks=_ptr(lw.sinks),
+                               token_begin=0, n_tokens=0, heads=H, kv_heads=G, hd=hd, page_size=PAGE,
+                               num_pages=self.num_pages, window=0, scale=s.scale, softcap=s.softcap or 0.0, dtype=self.code,
+                               status=st)
+            self._op(f"R{r}.attn", gp, dyn=[("n_tokens", T)], layer=r)
+        self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
+
+    def _wkv(self, r: int, layer: int, s, lw) -> None:
+        m, T, meta, st = self.model, "T", self.meta, _ptr(self.bufs.status)
+        H, d, wp = s.heads, round8(s.dim), m.width_p
+        S, before = self.state[r]
+        mix, proj, lora = self.view("mix", 5 * wp), self.view("proj", 4 * H * d), self.view("lora", round8(s.rank))
+        decay, attn = self.view("gates", H * d), self.view("attn", H * d)
+        ts = TokenShiftParams(h=_ptr(self.h), ld_h=wp, out=_ptr(mix), mu=_ptr(lw.mu), state=_ptr(before),
+                              state_slot=_ptr(meta["state_ref"]), positions=_ptr(meta["positions"]),
+                              token_req=_ptr(meta["token_req"]), qo_indptr=_ptr(meta["qo_indptr"]), T=0, n_mix=5,
+                              num_slots=self.num_slots, dtype=self.code, status=st)
+        self._op(f"R{r}.token_shift", ts, dyn=[("T", T)], layer=r)
+        self._gemm(f"R{r}.in", mix, lw.w_in, proj, rows=T, groups=4, group_k=wp, k=wp, key=f"l{layer}.in", layer=r)
+        self._gemm(f"R{r}.decay_down", mix[:, 4 * wp:], lw.w_down, lora, rows=T, lin_act="tanh", layer=r)
+        self._gemm(f"R{r}.decay_up", lora, lw.w_up, None, rows=T, d32=decay, bias=lw.w_bias, layer=r)
+
+        def params() -> WkvParams:
+            return WkvParams(rkvg=_ptr(proj), ld=proj.stride(0), r_off=0, k_off=H * d, v_off=2 * H * d, g_off=3 * H * d,
+                             x=_ptr(decay), ld_x=decay.stride(0), u=_ptr(lw.u), norm=_ptr(lw.norm), S=_ptr(S), y=_ptr(attn),
+                             ld_y=attn.stride(0), positions=_ptr(meta["positions"]), qo_indptr=_ptr(meta["qo_indptr"]),
+                             state_slot=_ptr(meta["state_ref"]), req_begin=0, req_count=0, heads=H, dim=d, dim_real=s.dim,
+                             num_slots=self.num_slots, eps=m.norm_eps, dtype=self.code, o=_ptr(self.flat["o_rec"]),
+                             items=_ptr(meta["wkv_items"]), scratch=_ptr(self.wkv_ws), scratch_floats=self.wkv_ws.numel(),
+                             status=st)
+
+        self._op(f"R{r}.wkv_decode", params(), kernel="nfk_wkv_decode", dyn=[("req_count", "n_dec")], layer=r)
+        chunked = self.wkv_cap > 0 and d <= WKV_CHUNK_DIM
+        p = params()
+        p.seq_reqs = _ptr(meta["wkv_seq" if chunked else "wkv_all"])
+        dyn = [("num_seq", self.g.symbol("n_wkv_seq" if chunked else "n_pre"))]
+        if chunked:
+            dyn.append(("num_items", self.g.symbol("n_wkv_items")))
+        self._op(f"R{r}.wkv_prefill", p, kernel="nfk_wkv_prefill", dyn=dyn, layer=r)
+        self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
+
+    # ---- feed-forwards: read self.h; return what joins the stream (see _residual) -------------------------
+    def _dense(self, r: int, layer: int, s, lw, key="") -> dict:
+        act = self.view("act", round8(s.ff))
+        out = self.y2 if self.y2 is not None else self.y
+        self._gemm(f"R{r}.{key}gate_up", self.h, lw.w_gate, act, rows="T", up=lw.w_up, act=s.act, key=f"l{layer}.{key}gate_up",
+                   layer=r)
+        self._gemm(f"R{r}.{key}down", act, lw.w_down, out, rows="T", key=f"l{layer}.{key}down", layer=r)
+        return {"y2": out}
+
+    def _moe(self, r: int, layer: int, s, lw) -> dict:
+        m, T, st, wp, ids = self.model, "T", _ptr(self.bufs.status), self.model.width_p, self.moe_ids
+        rows = self.g.symbol(f"e_rows{s.top}")                 # tokens x experts per token
+        logits, counts, cap = self.view("router", lw.router.shape[0]), self.moe_counts_of[r], self.T * s.top
+        flat = lambda k, cols: self.flat[k][:cap * cols].view(cap, cols)
+        e_in, e_act, e_out = flat("e_in", wp), flat("e_act", round8(s.expert.ff)), flat("e_out", wp)
+        self._gemm(f"R{r}.router", self.h, lw.router, None, rows=T, d32=logits, layer=r)
+        rp = MoeRouteParams(logits=_ptr(logits), ld=logits.stride(0), correction=_ptr(lw.correction), expert=_ptr(ids["expert"]),
+                            weight=_ptr(ids["weight"]), rank=_ptr(ids["rank"]), counts=_ptr(counts), gate=_ptr(self.moe_gate),
+                            T=0, experts=s.experts, top=s.top, groups=s.groups, keep=s.keep,
+                            gate_col=s.experts if s.shared is not None else -1, scale=s.scale)
+        self._op(f"R{r}.moe_route", rp, dyn=[("T", T)], layer=r)
+        pp = MoePermuteParams(h=_ptr(self.h), ld_h=wp, out=_ptr(e_in), ld_out=wp, expert=_ptr(ids["expert"]),
+                              rank=_ptr(ids["rank"]), counts=_ptr(counts), slot=_ptr(ids["slot"]), T=0, top=s.top,
+                              experts=s.experts, cols=wp, dtype=self.code)
+        self._op(f"R{r}.moe_permute", pp, dyn=[("T", T)], layer=r)
+
+        def product(name, a, b, b2, out, n) -> None:
+            act = s.expert.act
+            p = MoeGemmParams(A=_ptr(a), B=_ptr(b), B2=_ptr(b2), D=_ptr(out), counts=_ptr(counts), lda=a.stride(0),
+                              ldb=b.stride(0), ldd=out.stride(0), rows=0, experts=s.experts, N=n, K=b.shape[1],
+                              act=ACTS[act.name], act_limit=act.limit, act_alpha=act.alpha, act_shift=act.shift,
+                              dtype=self.code, num_ctas=0, status=st)
+            self._op(f"R{r}.{name}", p, dyn=[("rows", rows)], layer=r)
+
+        product("moe_gate_up", e_in, lw.w_gate, lw.w_up, e_act, round8(s.expert.ff))
+        product("moe_down", e_act, lw.w_down, None, e_out, wp)
+        out = dict(e_out=e_out, e_slot=ids["slot"], e_weight=ids["weight"], e_top=s.top)
+        if s.shared is not None:
+            out.update(self._dense(r, layer, s.shared, lw.shared, key="shared_"), y2_gate=self.moe_gate)
+        return out
+
     # ---- GEMM shapes ----------------------------------------------------------------------------------
     def _autotune(self) -> None:
         """Measured shapes for the dense products of every distinct layer at the full batch size."""
@@ -383,9 +596,12 @@ class LayerListEngine(Engine):
             self.flat[k].normal_()
         for i, lay in enumerate(m.layers):
             lw = self.w.layers[i]
-            specs = [("in", self.h, lw.mixer.w_in, None, self.flat["proj"]), ("o", None, lw.mixer.w_o, None, None)]
-            if lay.mlp is not None:
-                specs += [("gate_up", self.h, lw.w_gate, lw.w_up, self.flat["act"]), ("down", None, lw.w_down, None, None)]
+            specs = [("o", None, lw.mixer.w_o, None, None)]
+            if lay.mixer.kind != "wkv":          # (its input projection is block-diagonal: left to the cost model)
+                specs.append(("in", self.h, lw.mixer.w_in, None, self.flat["proj"]))
+            f, key = (lw.mlp, "") if lay.mlp is None or lay.mlp.kind == "dense" else (lw.mlp.shared, "shared_")
+            if f is not None:
+                specs += [(key + "gate_up", self.h, f.w_gate, f.w_up, self.flat["act"]), (key + "down", None, f.w_down, None, None)]
             for key, a, wt, up, out in specs:
                 name = f"l{i}.{key}"
                 if name in self.eng.gemm_shapes:
@@ -416,10 +632,24 @@ class LayerListEngine(Engine):
         put("state_ref", plan.state_ref)
         sym["n_dec"], sym["n_pre"] = D, P
         qo, span = plan.qo_indptr, np.diff(plan.qo_indptr)
-        if m.has_state:
+        if m.run_specs("mlstm"):
             segs = mlstm_segments(qo, D, self._segment_ctas(), ops.sm_count(self.device))
             put("segs", segs.reshape(-1))
             sym["n_segs"] = segs.shape[0]
+        if m.run_specs("wkv"):
+            items, seq = wkv_work(qo, D, self.wkv_cap)
+            put("wkv_items", items.reshape(-1))
+            put("wkv_seq", seq)
+            put("wkv_all", np.arange(D, D + P, dtype=np.int32))
+            sym["n_wkv_items"], sym["n_wkv_seq"] = items.shape[0], seq.size
+        for n in self.attn_groups:
+            items = query_items(qo, D, QUERY_TILE // n)
+            put(f"gitem{n}", items.reshape(-1))
+            sym[f"n_gitems{n}"] = items.shape[0]
+        if self.attn_groups:
+            sym["dec_chunk_pages"], sym["dec_max_chunks"] = self._attn_split(D, plan.max_kv_pages)
+        for top in {f.top for f in m.run_moes()}:
+            sym[f"e_rows{top}"] = plan.num_tokens * top
         for g in self.groups:
             work = route_attention(plan, g.window, g.expands, self.x_pages, self.eng.expand_min_tokens)
             put(g.name("abs"), work["abs"])
@@ -435,6 +665,16 @@ class LayerListEngine(Engine):
                 sym[g.name("n_xpages")] = int(work["xpage"].size)
                 sym[g.name("x_rows")] = int(work["xpage"].size) * PAGE
                 sym[g.name("n_xitems")] = int(work["items"].shape[0])
+
+    def _attn_split(self, n_dec: int, pages: int) -> Tuple[int, int]:
+        """(pages per key range, ranges) of decode attention, so that a few long contexts still occupy the SMs."""
+        specs = [s for s in self.model.run_specs("attention") if self.model.attn_on_tensor_cores(s)]
+        work = n_dec * min(s.kv_heads for s in specs)
+        target = 4 * ops.sm_count(self.device)
+        if work == 0 or work >= target or pages <= 16 or n_dec * max(s.heads for s in specs) > DECODE_SPLIT_ROWS:
+            return 0, 1
+        chunk = max(8, -(-pages // min(DECODE_MAX_CHUNKS, -(-target // work))))
+        return chunk, max(1, -(-pages // chunk))
 
     def _segment_ctas(self) -> int:
         """CTAs of the chunked mLSTM kernel per segment (of the layer with the fewest)."""
@@ -453,7 +693,9 @@ class LayerListEngine(Engine):
         return self.logits[:n, :self.model.vocab_size]
 
 
-MIXERS = {"latent_attention": LayerListEngine._latent_attention, "mlstm": LayerListEngine._mlstm}
+MIXERS = {"latent_attention": LayerListEngine._latent_attention, "mlstm": LayerListEngine._mlstm,
+          "attention": LayerListEngine._attention, "wkv": LayerListEngine._wkv}
+FEED_FORWARDS = {"dense": LayerListEngine._dense, "moe": LayerListEngine._moe}
 
 
 # --------------------------------------------------------------------------------------------------
@@ -478,6 +720,28 @@ def mlstm_segments(qo_indptr: np.ndarray, n_dec: int, ctas_per_segment: int, sms
         for k, t in enumerate(range(0, int(n), seg_len)):
             out.append((b, qo_indptr[b] + t, min(seg_len, n - t), k))
     return np.asarray(out, dtype=np.int32)
+
+
+def wkv_work(qo_indptr: np.ndarray, n_dec: int, chunk_cap: int) -> Tuple[np.ndarray, np.ndarray]:
+    """Rows (request, first token, tokens, chunk of the portion) for the chunked WKV kernels, and the requests whose
+    portions do not fit what is left of ``chunk_cap`` chunks: those go token by token."""
+    rows, seq = [], []
+    for b in range(n_dec, qo_indptr.size - 1):
+        t0, n = int(qo_indptr[b]), int(qo_indptr[b + 1] - qo_indptr[b])
+        if len(rows) + -(-n // WKV_CHUNK) > chunk_cap:
+            seq.append(b)
+            continue
+        rows += [(b, t0 + c, min(WKV_CHUNK, n - c), c // WKV_CHUNK) for c in range(0, n, WKV_CHUNK)]
+    return np.asarray(rows, dtype=np.int32).reshape(-1, 4), np.asarray(seq, dtype=np.int32)
+
+
+def query_items(qo_indptr: np.ndarray, n_dec: int, tile: int) -> np.ndarray:
+    """Rows (request, first token, tokens) of the prefill attention kernel."""
+    rows = []
+    for b in range(n_dec, qo_indptr.size - 1):
+        q0, q1 = int(qo_indptr[b]), int(qo_indptr[b + 1])
+        rows += [(b, t, min(tile, q1 - t)) for t in range(q0, q1, tile)]
+    return np.asarray(rows, dtype=np.int32).reshape(-1, 3)
 
 
 def route_attention(plan: BatchPlan, window: int, expands: bool, page_cap: int, min_tokens: int) -> dict:
