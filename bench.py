@@ -156,7 +156,8 @@ def main():
     ap.add_argument("--executor", default="auto", help="auto | native | graph (native executor, iterations "
                     "captured and launched as CUDA graphs) | python")
     ap.add_argument("--layer-list", default="", help="instead of the headline workload: prefill and decode throughput of the "
-                    "layer-list model (Volarax) beside the Llama of equal size, comma-separated sizes out of 2B, 8B")
+                    "layer-list model beside the Llama of equal size, comma-separated sizes out of 2B, 8B")
+    ap.add_argument("--layer-model", default="volarax", help="with --layer-list: volarax, zubedra, or both with a comma")
     ap.add_argument("--layer-list-only", default="", help="with --layer-list: only workloads whose name holds this text")
     ap.add_argument("--timeline", default="", help="after the timed regions, time every op of one iteration "
                     "with CUDA events and write the aggregate + Chrome trace to this file")
@@ -178,7 +179,8 @@ def main():
         sampler = ClockSampler(local_rank)
         sampler.start()
         t0 = time.perf_counter()
-        res = layer_bench.run(args.layer_list.split(","), args.steps, args.warmup, args.layer_list_only)
+        res = layer_bench.run(args.layer_list.split(","), args.steps, args.warmup, args.layer_list_only,
+                              args.layer_model)
         clocks = sampler.stop(t0, time.perf_counter())
         print(layer_bench.report(res), file=sys.stderr)
         print(json.dumps({"benchmark": "layer-list", "n_gpus": 1, "steps": args.steps, "dtype": "bf16",

@@ -23,6 +23,7 @@
 #include "kernels.h"
 #include "attn_decode_static.h"
 #include "attn_mma.cuh"
+#include "softcap.cuh"
 
 #include <atomic>
 #include <mutex>
@@ -85,10 +86,6 @@ __device__ __forceinline__ void pv_16tok_pair(float (&o)[HD / 8][4], const uint3
     mma_bf16(o[c], pl, b0, b1);
     mma_bf16(o[c + 1], pl, b2, b3);
   }
-}
-// tanh x = 1 - 2 / (e^(2x) + 1): within a few 1e-7 absolute everywhere, and +-1 at the far ends.
-__device__ __forceinline__ float tanh_by_exp(float x) {
-  return 1.f - __fdividef(2.f, fast_exp2(x * (2.f * kLog2e)) + 1.f);
 }
 
 // ================================================================================================

@@ -35,6 +35,7 @@
 // (gemv/include/attention/prefill.cuh:1066-1374, mma.sync m16n16k16 + ldmatrix on sm_80).
 #include "common.cuh"
 #include "kernels.h"
+#include "softcap.cuh"
 
 namespace nf {
 namespace {
@@ -68,10 +69,6 @@ __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
-}
-// tanh x = 1 - 2 / (e^(2x) + 1): within a few 1e-7 absolute everywhere, and +-1 at the far ends.
-__device__ __forceinline__ float tanh_by_exp(float x) {
-  return 1.f - __fdividef(2.f, fast_exp2(x * (2.f * kLog2e)) + 1.f);
 }
 __device__ __forceinline__ void st_shared_v4(uint32_t addr, uint32_t a, uint32_t b, uint32_t c, uint32_t d) {
   asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(a), "r"(b), "r"(c), "r"(d) : "memory");
@@ -345,10 +342,22 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld_32x32b_x32(t_lane + s * kTile + 32, r1);
         tmem_ld_wait();
         if (CAP) {
+          // a row whose scores are all well below the cap does without the special function unit
+          float top = 0.f;
 #pragma unroll
-          for (int j = 0; j < 32; ++j) {
-            r0[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r0[j]) * cap_in));
-            r1[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r1[j]) * cap_in));
+          for (int j = 0; j < 32; ++j) top = fmaxf(top, fmaxf(fabsf(__uint_as_float(r0[j])), fabsf(__uint_as_float(r1[j]))));
+          if (__all_sync(0xffffffffu, top * cap_in <= kTanhSmall)) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              r0[j] = __float_as_uint(cap_out * tanh_small(__uint_as_float(r0[j]) * cap_in));
+              r1[j] = __float_as_uint(cap_out * tanh_small(__uint_as_float(r1[j]) * cap_in));
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              r0[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r0[j]) * cap_in));
+              r1[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r1[j]) * cap_in));
+            }
           }
         }
         const int cbase = (it.t_first + t) * kTile;

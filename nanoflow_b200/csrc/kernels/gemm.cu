@@ -156,6 +156,7 @@ struct DevParams {
   float* D32;
   long long ld32;
   int f32_col0;
+  int d32_wide;                     // rows of D32 start on 32-byte boundaries
   GatedAct act;                     // gated epilogue
   int lin_act;                      // linear epilogue: NFK_LIN_*
   int groups, group_n, group_k;     // block-diagonal product (groups 1: an ordinary one)
@@ -192,7 +193,14 @@ __device__ __forceinline__ void store_cols8(const DevParams& p, int row, int col
     for (int j = 0; j < 8; ++j) v[j] = tanhf(v[j]);
   }
   if (p.D32 != nullptr && col >= p.f32_col0) {
-    float4* dst = reinterpret_cast<float4*>(p.D32 + static_cast<long long>(row) * p.ld32 + (col - p.f32_col0));
+    float* out = p.D32 + static_cast<long long>(row) * p.ld32 + (col - p.f32_col0);
+    if (p.d32_wide) {          // one store per 32-byte sector
+      asm volatile("st.global.v8.f32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(out), "f"(v[0]), "f"(v[1]), "f"(v[2]),
+                   "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7])
+                   : "memory");
+      return;
+    }
+    float4* dst = reinterpret_cast<float4*>(out);
     dst[0] = make_float4(v[0], v[1], v[2], v[3]);
     dst[1] = make_float4(v[4], v[5], v[6], v[7]);
     return;
@@ -1156,6 +1164,7 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
   p.D32 = reinterpret_cast<float*>(g.D32);
   p.ld32 = g.ld32;
   p.f32_col0 = g.f32_col0;
+  p.d32_wide = (reinterpret_cast<uintptr_t>(g.D32) & 31) == 0 && g.ld32 % 8 == 0;
   p.act = GatedAct{g.act, g.act_limit, g.act_alpha, g.act_shift};
   p.lin_act = EPI == 0 ? g.lin_act : NFK_LIN_NONE;
   p.groups = groups;

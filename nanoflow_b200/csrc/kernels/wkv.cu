@@ -1,6 +1,6 @@
 // WKV recurrence: a matrix state per head with a decay per key channel and token, and a bonus for the current
-// token (Peng et al., "RWKV"; see kernels.h for the equations). State, decays and everything derived from them
-// are fp32.
+// token (Peng et al., "Eagle and Finch: RWKV with Matrix-Valued States and Dynamic Recurrence"; see kernels.h for the
+// equations). State, decays and everything derived from them are fp32.
 //
 // nfk_token_shift   every stream's mix of a token's row with the previous token's row; the last row of a request
 //                   is kept for its next step.
@@ -12,10 +12,12 @@
 //                   2. a scan over the chunks, which leaves the state each chunk starts from (and the final one);
 //                   3. the outputs: read-out of the incoming state, plus A V with A_ti the decayed score of token
 //                      t and an earlier token i of the chunk.
-//                   A chunk is cut into four runs of 16 tokens. Sums of log decays are kept within a run, so every
-//                   weight is the exponential of a non-positive sum: between runs it factors at the end of the
-//                   earlier run (tensor cores), within a run it is formed pair by pair (fp32). Weighted rows, scores
-//                   and the state enter the products as bf16 pairs (high and low part), about 16 bits.
+//                   A chunk is cut into four runs of 16 tokens. Sums of log decays are kept within a run, and the
+//                   weight of a (query, key) pair factors at the end of the key's run: the key's factor is the
+//                   exponential of a non-positive sum, and so is the query's if it is in a later run. Inside a run the
+//                   query's factor grows, at most to 2^110: a run in which some channel decays by more than that
+//                   forms its weights pair by pair instead. Weighted rows, scores and the state enter the tensor-core
+//                   products as bf16 pairs (high and low part), about 16 bits.
 #include "attn_mma.cuh"
 #include "elem_io.cuh"
 
@@ -81,22 +83,34 @@ __device__ __forceinline__ float wkv_sum256(float v, float* red) {
   return warp_sum(lane < 8 ? red[lane] : 0.f);
 }
 __device__ __forceinline__ float silu_f(float g) { return g / (1.f + expf(-g)); }
+__device__ __forceinline__ float silu_fast(float g) { return __fdividef(g, 1.f + __expf(-g)); }   // for bf16 results
 
-// LC lanes share a row of S (four columns each, 4 * LC columns at a time), 256 / LC rows are in work at once.
-template <class T, int LC>
+// LC lanes share a row of S (four columns each, 4 * LC columns at a time), 256 / LC rows are in work at once. NR > 0: the
+// head fits into one pass of NR rows per thread, which are fetched before anything else.
+template <class T, int LC, int NR>
 __global__ void __launch_bounds__(256)
 wkv_decode_kernel(nfk_wkv_params p) {
   constexpr int R = 256 / LC;
   extern __shared__ float dsm[];                 // r | k | decay | o, [dim] each
   __shared__ float red[8];
-  __shared__ float4 part[R][LC];
+  __shared__ float4 part[8][LC];
   float *r_s = dsm, *k_s = r_s + p.dim, *w_s = k_s + p.dim, *o_s = w_s + p.dim;
   const int head = blockIdx.x % p.heads, req = p.req_begin + blockIdx.x / p.heads;
+  const int lc = threadIdx.x % LC, lr = threadIdx.x / LC;
   const WkvState st = wkv_state(p, req, head);
   if (!st.ok) return;
   const long long tok = p.qo_indptr[req];
   const int hc = head * p.dim;
   const T* row = reinterpret_cast<const T*>(p.rkvg) + tok * p.ld + hc;
+  float4 pre[NR > 0 ? NR : 1];
+  if (NR > 0) {
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int d = lr + i * R;
+      pre[i] = (st.fresh || d >= p.dim || lc * 4 >= p.dim) ? make_float4(0.f, 0.f, 0.f, 0.f)
+                                                           : load4(st.S + static_cast<long long>(d) * p.dim + lc * 4);
+    }
+  }
   float bonus = 0.f;
   for (int d = threadIdx.x; d < p.dim; d += 256) {
     const float r = to_f32(row[p.r_off + d]), k = to_f32(row[p.k_off + d]);
@@ -106,31 +120,45 @@ wkv_decode_kernel(nfk_wkv_params p) {
     bonus += r * p.u[hc + d] * k;
   }
   bonus = wkv_sum256(bonus, red);                // also orders r_s, k_s, w_s
-  const int lc = threadIdx.x % LC, lr = threadIdx.x / LC;
+  auto update = [&](float4 s, int d, float4 v, float4& acc, float* dst) {
+    const float rd = r_s[d], kd = k_s[d], wd = w_s[d];
+    acc.x += s.x * rd; acc.y += s.y * rd; acc.z += s.z * rd; acc.w += s.w * rd;
+    store4(dst, make_float4(wd * s.x + kd * v.x, wd * s.y + kd * v.y, wd * s.z + kd * v.z, wd * s.w + kd * v.w));
+  };
   for (int c0 = 0; c0 < p.dim; c0 += LC * 4) {
     const int col = c0 + lc * 4;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f), v = acc;
     if (col < p.dim) {
       v = load4(row + p.v_off + col);
       float* S = st.S + col;
+      if (NR > 0) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+          const int d = lr + i * R;
+          if (d < p.dim) update(pre[i], d, v, acc, S + static_cast<long long>(d) * p.dim);
+        }
+      } else {
 #pragma unroll 8
-      for (int d = lr; d < p.dim; d += R) {
-        float4* sp = reinterpret_cast<float4*>(S + static_cast<long long>(d) * p.dim);
-        float4 s = st.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *sp;
-        const float rd = r_s[d], kd = k_s[d], wd = w_s[d];
-        acc.x += s.x * rd; acc.y += s.y * rd; acc.z += s.z * rd; acc.w += s.w * rd;
-        s.x = wd * s.x + kd * v.x;
-        s.y = wd * s.y + kd * v.y;
-        s.z = wd * s.z + kd * v.z;
-        s.w = wd * s.w + kd * v.w;
-        *sp = s;
+        for (int d = lr; d < p.dim; d += R) {
+          float* sp = S + static_cast<long long>(d) * p.dim;
+          update(st.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(sp), d, v, acc, sp);
+        }
       }
     }
-    part[lr][lc] = acc;
+    // rows that share a warp are added up by shuffles, warps through shared memory
+#pragma unroll
+    for (int o = LC; o < 32; o <<= 1) {
+      acc.x += __shfl_xor_sync(0xffffffffu, acc.x, o);
+      acc.y += __shfl_xor_sync(0xffffffffu, acc.y, o);
+      acc.z += __shfl_xor_sync(0xffffffffu, acc.z, o);
+      acc.w += __shfl_xor_sync(0xffffffffu, acc.w, o);
+    }
+    const int warp = threadIdx.x >> 5;
+    if ((threadIdx.x & 31) < LC) part[warp][lc] = acc;
     __syncthreads();
     if (lr == 0 && col < p.dim) {
-#pragma unroll 8
-      for (int w = 1; w < R; ++w) {
+#pragma unroll
+      for (int w = 1; w < 8; ++w) {
         const float4 o = part[w][lc];
         acc.x += o.x; acc.y += o.y; acc.z += o.z; acc.w += o.w;
       }
@@ -230,6 +258,7 @@ wkv_seq_norm_kernel(nfk_wkv_params p) {
 
 // ---- prefill, chunks of 64 tokens -------------------------------------------------------------------------------
 constexpr int kChunk = 64, kRun = 16, kRuns = kChunk / kRun;
+constexpr float kMaxRunLog2 = 110.f;       // largest decay of a run (log2) whose weights are factored inside the run
 
 __host__ __device__ __forceinline__ long long wkv_item_floats(int dim) { return static_cast<long long>(dim) * dim + dim; }
 
@@ -241,10 +270,10 @@ struct WkvCfg {
   static constexpr int ROWS_BYTES = kChunk * BLD * 2;    // r, k or v
   static constexpr int CE_BYTES = kChunk * FLD * 4;
   static constexpr int TOT_BYTES = kRuns * DP * 4;
-  static constexpr int S_BYTES = DP * FLD * 4;
+  static constexpr int S_BYTES = DP * BLD * 2;           // one part
   static constexpr int A_BYTES = kChunk * ALD * 2;       // one part
   static constexpr int STATE_SMEM = 2 * ROWS_BYTES + CE_BYTES + TOT_BYTES;
-  static constexpr int OUT_SMEM = 3 * ROWS_BYTES + CE_BYTES + TOT_BYTES + S_BYTES + 2 * A_BYTES + DP * 4 + 2 * kChunk * 4;
+  static constexpr int OUT_SMEM = 5 * ROWS_BYTES + CE_BYTES + TOT_BYTES + 2 * S_BYTES + 2 * A_BYTES + DP * 4 + 3 * kChunk * 4 + 16;
 };
 
 // 64 rows of a head's columns of rkvg into [64][BLD]; rows past `n` and columns past the head's are zero.
@@ -261,7 +290,8 @@ __device__ __forceinline__ void load_rows(__nv_bfloat16* dst, const nfk_wkv_para
 }
 // ce[t][d]: sum of the log2 decays of the tokens of t's run before t; tot[run][d]: sum over the run.
 template <int DP>
-__device__ __forceinline__ void load_decays(float* ce, float* tot, const nfk_wkv_params& p, long long tok0, int n, int hc) {
+__device__ __forceinline__ void load_decays(float* ce, float* tot, const nfk_wkv_params& p, long long tok0, int n, int hc,
+                                            int* slow = nullptr) {
   constexpr int CH = DP / 4, FLD = WkvCfg<DP>::FLD;
   for (int i = threadIdx.x; i < kChunk * CH; i += 256) {
     const int r = i / CH, c = (i % CH) * 4;
@@ -275,15 +305,16 @@ __device__ __forceinline__ void load_decays(float* ce, float* tot, const nfk_wkv
   __syncthreads();
   for (int i = threadIdx.x; i < kRuns * DP; i += 256) {
     const int run = i / DP, d = i % DP;
-    float s = 0.f;
+    float l[kRun], s = 0.f;
+#pragma unroll
+    for (int j = 0; j < kRun; ++j) l[j] = ce[(run * kRun + j) * FLD + d];
 #pragma unroll
     for (int j = 0; j < kRun; ++j) {
-      float* e = ce + (run * kRun + j) * FLD + d;
-      const float l = *e;
-      *e = s;
-      s += l;
+      ce[(run * kRun + j) * FLD + d] = s;
+      s += l[j];
     }
     tot[i] = s;
+    if (slow != nullptr && s < -kMaxRunLog2) slow[run] = 1;
   }
   __syncthreads();
 }
@@ -417,13 +448,18 @@ wkv_chunk_out_kernel(nfk_wkv_params p) {
   __nv_bfloat16* r_s = reinterpret_cast<__nv_bfloat16*>(smem);
   __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem + C::ROWS_BYTES);
   __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(smem + 2 * C::ROWS_BYTES);
-  float* ce = reinterpret_cast<float*>(smem + 3 * C::ROWS_BYTES);
-  float* tot = reinterpret_cast<float*>(smem + 3 * C::ROWS_BYTES + C::CE_BYTES);
-  float* S_s = tot + kRuns * DP;
-  __nv_bfloat16* ah_s = reinterpret_cast<__nv_bfloat16*>(S_s + DP * C::FLD);
+  __nv_bfloat16* kh_s = reinterpret_cast<__nv_bfloat16*>(smem + 3 * C::ROWS_BYTES);      // decayed keys, two parts
+  __nv_bfloat16* kl_s = reinterpret_cast<__nv_bfloat16*>(smem + 4 * C::ROWS_BYTES);
+  float* ce = reinterpret_cast<float*>(smem + 5 * C::ROWS_BYTES);
+  float* tot = reinterpret_cast<float*>(smem + 5 * C::ROWS_BYTES + C::CE_BYTES);
+  __nv_bfloat16* sh_s = reinterpret_cast<__nv_bfloat16*>(tot + kRuns * DP);              // incoming state, two parts
+  __nv_bfloat16* sl_s = sh_s + DP * C::BLD;
+  __nv_bfloat16* ah_s = sl_s + DP * C::BLD;                                             // scores, two parts
   __nv_bfloat16* al_s = ah_s + kChunk * C::ALD;
   float* u_s = reinterpret_cast<float*>(al_s + kChunk * C::ALD);
-  float* ss_s = u_s + DP;                                  // [2][64]
+  float* bonus_s = u_s + DP;                               // [64]
+  float* ss_s = bonus_s + kChunk;                          // [2][64]
+  int* slow_s = reinterpret_cast<int*>(ss_s + 2 * kChunk);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.x % p.heads, item = blockIdx.x / p.heads;
   const int n = p.items[item * 4 + 2], hc = head * p.dim;
@@ -434,68 +470,156 @@ wkv_chunk_out_kernel(nfk_wkv_params p) {
   const float* S = p.scratch + (static_cast<long long>(item) * p.heads + head) * wkv_item_floats(p.dim);
   for (int i = threadIdx.x; i < DP * (DP / 4); i += 256) {
     const int d = i / (DP / 4), c = (i % (DP / 4)) * 4;
-    store4(S_s + d * C::FLD + c, (d < p.dim && c < p.dim) ? load4(S + d * p.dim + c) : make_float4(0.f, 0.f, 0.f, 0.f));
+    const float4 x = (d < p.dim && c < p.dim) ? load4(S + d * p.dim + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    uint2 hi, lo;
+    split_pair(x.x, x.y, hi.x, lo.x);
+    split_pair(x.z, x.w, hi.y, lo.y);
+    *reinterpret_cast<uint2*>(sh_s + d * C::BLD + c) = hi;
+    *reinterpret_cast<uint2*>(sl_s + d * C::BLD + c) = lo;
   }
   for (int d = threadIdx.x; d < DP; d += 256) u_s[d] = d < p.dim ? p.u[hc + d] : 0.f;
-  load_decays<DP>(ce, tot, p, tok0, n, hc);
+  if (threadIdx.x < kRuns) slow_s[threadIdx.x] = 0;
+  load_decays<DP>(ce, tot, p, tok0, n, hc, slow_s);
 
-  // ---- scores between runs: warps 0-5, one 16 x 16 block (run a of queries, earlier run b of keys) each ----
-  if (warp < 6) {
-    const int a = warp == 0 ? 1 : warp < 3 ? 2 : 3;
-    const int b = warp == 0 ? 0 : warp < 3 ? warp - 1 : warp - 3;
-    float acc[2][4];
+  // ---- keys decayed to the end of their run, and every token's own score ----
+  for (int i = threadIdx.x; i < kChunk * (DP / 2); i += 256) {
+    const int t = i / (DP / 2), d = (i % (DP / 2)) * 2;
+    const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + t * C::BLD + d));
+    const float2 e = *reinterpret_cast<const float2*>(tot + (t / kRun) * DP + d);
+    const float2 c = (t & (kRun - 1)) == kRun - 1 ? e : *reinterpret_cast<const float2*>(ce + (t + 1) * C::FLD + d);
+    uint32_t hi, lo;
+    split_pair(k.x * fast_exp2(e.x - c.x), k.y * fast_exp2(e.y - c.y), hi, lo);
+    *reinterpret_cast<uint32_t*>(kh_s + t * C::BLD + d) = hi;
+    *reinterpret_cast<uint32_t*>(kl_s + t * C::BLD + d) = lo;
+  }
+  {
+    const int t = threadIdx.x >> 2;
+    float b = 0.f;
 #pragma unroll
-    for (int j = 0; j < 2; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
-    const int t0 = a * kRun + (lane >> 2);
-#pragma unroll 2
-    for (int ks = 0; ks < DP / 16; ++ks) {
-      uint32_t rh[4], rl[4];
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int d = ks * 16 + half * 8 + (lane & 3) * 2;
-        float2 mid = make_float2(0.f, 0.f);                // runs between b and a
-        for (int j = b + 1; j < a; ++j) {
-          mid.x += tot[j * DP + d];
-          mid.y += tot[j * DP + d + 1];
-        }
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const int t = t0 + h * 8;
-          const float2 r = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_s + t * C::BLD + d));
-          const float2 c = *reinterpret_cast<const float2*>(ce + t * C::FLD + d);
-          split_pair(r.x * fast_exp2(c.x + mid.x), r.y * fast_exp2(c.y + mid.y), rh[half * 2 + h], rl[half * 2 + h]);
-        }
-      }
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        uint32_t kh[2], kl[2];
-        const int jj = j * 8 + (lane >> 2), t = b * kRun + jj;          // key token
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int d = ks * 16 + half * 8 + (lane & 3) * 2;
-          const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + t * C::BLD + d));
-          const float2 e = *reinterpret_cast<const float2*>(tot + b * DP + d);
-          const float2 c = jj == kRun - 1 ? e : *reinterpret_cast<const float2*>(ce + (t + 1) * C::FLD + d);
-          split_pair(k.x * fast_exp2(e.x - c.x), k.y * fast_exp2(e.y - c.y), kh[half], kl[half]);
-        }
-        mma_bf16(acc[j], rh, kh[0], kh[1]);
-        mma_bf16(acc[j], rh, kl[0], kl[1]);
-        mma_bf16(acc[j], rl, kh[0], kh[1]);
-      }
+    for (int d = (threadIdx.x & 3) * 2; d < DP; d += 8) {
+      const float2 r = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_s + t * C::BLD + d));
+      const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + t * C::BLD + d));
+      b += r.x * k.x * u_s[d] + r.y * k.y * u_s[d + 1];
     }
+    b = quad_sum(b);
+    if ((threadIdx.x & 3) == 0) bonus_s[t] = b;
+  }
+  __syncthreads();
+
+  // ---- scores and read-out of the incoming state. A warp takes a run `a` of queries; one of the run's two warps has
+  // the key runs 0 and 2 and the first half of the columns, the other one key runs 1 and 3 and the second half ----
+  constexpr int NT = DP / 16;
+  const int half = warp >> 2, a = half == 0 ? warp & 3 : 3 - (warp & 3), n0 = half * NT;
+  const int t0 = a * kRun + (lane >> 2);
+  const int mm = lane >> 3, rr = lane & 7;
+  const uint32_t khb = smem_u32(kh_s), klb = smem_u32(kl_s), shb = smem_u32(sh_s), slb = smem_u32(sl_s);
+  float acc[NT][4], sc[2][2][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) sc[i][j][0] = sc[i][j][1] = sc[i][j][2] = sc[i][j][3] = 0.f;
+  const bool has[2] = {half <= a && !(half == a && slow_s[a] != 0), half + 2 <= a && !(half + 2 == a && slow_s[a] != 0)};
+#pragma unroll 1
+  for (int ks = 0; ks < DP / 16; ++ks) {
+    // queries decayed to the start of their run
+    float2 f[2][2], pre[2], own[2], cum[2][2];
+#pragma unroll
+    for (int dh = 0; dh < 2; ++dh) {
+      const int d = ks * 16 + dh * 8 + (lane & 3) * 2;
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const float2 r = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_s + (t0 + h * 8) * C::BLD + d));
+        const float2 c = *reinterpret_cast<const float2*>(ce + (t0 + h * 8) * C::FLD + d);
+        f[dh][h] = make_float2(r.x * fast_exp2(c.x), r.y * fast_exp2(c.y));
+      }
+      // log decays of the runs before `a`, and of those between each of this warp's key runs and `a` (within a run: what
+      // takes the query back from the run's end)
+      pre[dh] = make_float2(0.f, 0.f);
+      cum[0][dh] = cum[1][dh] = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int j = 0; j < kRuns; ++j) {
+        const float2 x = *reinterpret_cast<const float2*>(tot + j * DP + d);
+        if (j == a) own[dh] = x;
+        if (j < a) {
+          pre[dh].x += x.x;
+          pre[dh].y += x.y;
+          if (j > half) {
+            cum[0][dh].x += x.x;
+            cum[0][dh].y += x.y;
+          }
+          if (j > half + 2) {
+            cum[1][dh].x += x.x;
+            cum[1][dh].y += x.y;
+          }
+        }
+      }
+#pragma unroll
+      for (int s = 0; s < 2; ++s)
+        if (half + 2 * s == a) cum[s][dh] = make_float2(-own[dh].x, -own[dh].y);
+    }
+    uint32_t qh[4], ql[4];
+    auto weighted = [&](const float2 (&e)[2]) {
+#pragma unroll
+      for (int dh = 0; dh < 2; ++dh) {
+        const float ex = fast_exp2(e[dh].x), ey = fast_exp2(e[dh].y);
+#pragma unroll
+        for (int h = 0; h < 2; ++h) split_pair(f[dh][h].x * ex, f[dh][h].y * ey, qh[dh * 2 + h], ql[dh * 2 + h]);
+      }
+    };
+#pragma unroll
+    for (int s = 0; s < 2; ++s) {
+      if (!has[s]) continue;
+      weighted(cum[s]);
+      const uint32_t o = (((half + 2 * s) * kRun + (mm >> 1) * 8 + rr) * C::BLD + (2 * ks + (mm & 1)) * 8) * 2;
+      uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+      ldsm_x4(khb + o, h0, h1, h2, h3);
+      ldsm_x4(klb + o, l0, l1, l2, l3);
+      mma_bf16(sc[s][0], qh, h0, h1);
+      mma_bf16(sc[s][1], qh, h2, h3);
+      mma_bf16(sc[s][0], qh, l0, l1);
+      mma_bf16(sc[s][1], qh, l2, l3);
+      mma_bf16(sc[s][0], ql, h0, h1);
+      mma_bf16(sc[s][1], ql, h2, h3);
+    }
+    weighted(pre);
+#pragma unroll
+    for (int i = 0; i < NT; i += 2) {
+      const uint32_t o = ((ks * 16 + (mm & 1) * 8 + rr) * C::BLD + (n0 + i + (mm >> 1)) * 8) * 2;
+      uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+      ldsm_x4_trans(shb + o, h0, h1, h2, h3);
+      ldsm_x4_trans(slb + o, l0, l1, l2, l3);
+      mma_bf16(acc[i], qh, h0, h1);
+      mma_bf16(acc[i + 1], qh, h2, h3);
+      mma_bf16(acc[i], qh, l0, l1);
+      mma_bf16(acc[i + 1], qh, l2, l3);
+      mma_bf16(acc[i], ql, h0, h1);
+      mma_bf16(acc[i + 1], ql, h2, h3);
+    }
+  }
+#pragma unroll
+  for (int s = 0; s < 2; ++s) {
+    if (!has[s]) continue;
+    const int b = half + 2 * s;
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
+        const int t = t0 + h * 8, i = b * kRun + j * 8 + (lane & 3) * 2;
+        float x = sc[s][j][2 * h], y = sc[s][j][2 * h + 1];
+        if (b == a) {                       // the token itself with its bonus, later ones not at all
+          x = i < t ? x : i == t ? bonus_s[t] : 0.f;
+          y = i + 1 < t ? y : i + 1 == t ? bonus_s[t] : 0.f;
+        }
         uint32_t hi, lo;
-        split_pair(acc[j][2 * h], acc[j][2 * h + 1], hi, lo);
-        const int o = (t0 + h * 8) * C::ALD + b * kRun + j * 8 + (lane & 3) * 2;
-        *reinterpret_cast<uint32_t*>(ah_s + o) = hi;
-        *reinterpret_cast<uint32_t*>(al_s + o) = lo;
+        split_pair(x, y, hi, lo);
+        *reinterpret_cast<uint32_t*>(ah_s + t * C::ALD + i) = hi;
+        *reinterpret_cast<uint32_t*>(al_s + t * C::ALD + i) = lo;
       }
   }
-  // ---- scores within a run: 64 threads per run, 2 x 2 (query, key) pairs each ----
-  {
+  // ---- runs that decay too much for factored weights: 64 threads per run, 2 x 2 (query, key) pairs each ----
+  if (slow_s[threadIdx.x >> 6] != 0) {
     const int run = threadIdx.x >> 6, ti = (threadIdx.x >> 3) & 7, ii = threadIdx.x & 7;
     const int t = run * kRun + ti * 2, i = run * kRun + ii * 2;
     float a00 = 0.f, a10 = 0.f, a11 = 0.f, a01 = 0.f;      // a[query][key]
@@ -516,15 +640,12 @@ wkv_chunk_out_kernel(nfk_wkv_params p) {
         a11 += r1.x * k1.x * fast_exp2(q1.x - c1.x) + r1.y * k1.y * fast_exp2(q1.y - c1.y);
       }
     } else if (ii == ti) {
-      for (int d = 0; d < DP; d += 2) {
-        const float2 r0 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_s + t * C::BLD + d));
+      a00 = bonus_s[t];
+      a11 = bonus_s[t + 1];
+      for (int d = 0; d < DP; d += 2) {                    // the token right before: not decayed yet
         const float2 r1 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_s + (t + 1) * C::BLD + d));
         const float2 k0 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + i * C::BLD + d));
-        const float2 k1 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + (i + 1) * C::BLD + d));
-        const float2 u = *reinterpret_cast<const float2*>(u_s + d);
-        a00 += r0.x * k0.x * u.x + r0.y * k0.y * u.y;      // the token itself: bonus, no decay
-        a11 += r1.x * k1.x * u.x + r1.y * k1.y * u.y;
-        a10 += r1.x * k0.x + r1.y * k0.y;                  // the token right before: not decayed yet
+        a10 += r1.x * k0.x + r1.y * k0.y;
       }
     }
     uint32_t hi, lo;
@@ -537,44 +658,7 @@ wkv_chunk_out_kernel(nfk_wkv_params p) {
   }
   __syncthreads();
 
-  // ---- outputs: 16 tokens x half of the columns per warp ----
-  constexpr int NT = DP / 16;
-  const int a = warp & 3, n0 = (warp >> 2) * NT;
-  float acc[NT][4];
-#pragma unroll
-  for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-  const int t0 = a * kRun + (lane >> 2);
-#pragma unroll 2
-  for (int ks = 0; ks < DP / 16; ++ks) {
-    uint32_t rh[4], rl[4];
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int d = ks * 16 + half * 8 + (lane & 3) * 2;
-      float2 pre = make_float2(0.f, 0.f);
-      for (int j = 0; j < a; ++j) {
-        pre.x += tot[j * DP + d];
-        pre.y += tot[j * DP + d + 1];
-      }
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int t = t0 + h * 8;
-        const float2 r = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_s + t * C::BLD + d));
-        const float2 c = *reinterpret_cast<const float2*>(ce + t * C::FLD + d);
-        split_pair(r.x * fast_exp2(c.x + pre.x), r.y * fast_exp2(c.y + pre.y), rh[half * 2 + h], rl[half * 2 + h]);
-      }
-    }
-    const float* s0 = S_s + (ks * 16 + (lane & 3) * 2) * C::FLD + n0 * 8 + (lane >> 2);
-#pragma unroll
-    for (int i = 0; i < NT; ++i) {
-      uint32_t h0, l0, h1, l1;
-      split_pair(s0[i * 8], s0[C::FLD + i * 8], h0, l0);
-      split_pair(s0[8 * C::FLD + i * 8], s0[9 * C::FLD + i * 8], h1, l1);
-      mma_bf16(acc[i], rh, h0, h1);
-      mma_bf16(acc[i], rh, l0, l1);
-      mma_bf16(acc[i], rl, h0, h1);
-    }
-  }
-  const int mm = lane >> 3, rr = lane & 7;
+  // ---- scores times values ----
   const uint32_t vb = smem_u32(v_s), ahb = smem_u32(ah_s), alb = smem_u32(al_s);
 #pragma unroll
   for (int ks = 0; ks < kRuns; ++ks) {
@@ -594,32 +678,39 @@ wkv_chunk_out_kernel(nfk_wkv_params p) {
     }
   }
   // ---- head norm over both column halves, weight, gate ----
+  const __nv_bfloat16* rkvg = reinterpret_cast<const __nv_bfloat16*>(p.rkvg);
+  uint32_t gate[2][NT];
+#pragma unroll
+  for (int h = 0; h < 2; ++h)
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int t = t0 + h * 8, v = (n0 + i) * 8 + (lane & 3) * 2;
+      gate[h][i] = (t < n && v < p.dim) ? *reinterpret_cast<const uint32_t*>(rkvg + (tok0 + t) * p.ld + p.g_off + hc + v) : 0u;
+    }
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NT; ++i) ss += acc[i][2 * h] * acc[i][2 * h] + acc[i][2 * h + 1] * acc[i][2 * h + 1];
     ss = quad_sum(ss);
-    if ((lane & 3) == 0) ss_s[(warp >> 2) * kChunk + t0 + h * 8] = ss;
+    if ((lane & 3) == 0) ss_s[half * kChunk + t0 + h * 8] = ss;
   }
   __syncthreads();
-  const __nv_bfloat16* rkvg = reinterpret_cast<const __nv_bfloat16*>(p.rkvg);
   __nv_bfloat16* y = reinterpret_cast<__nv_bfloat16*>(p.y);
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int t = t0 + h * 8;
     if (t >= n) continue;
     const float inv = rsqrtf((ss_s[t] + ss_s[kChunk + t]) / static_cast<float>(p.dim_real) + p.eps);
-    const __nv_bfloat16* g = rkvg + (tok0 + t) * p.ld + p.g_off + hc;
     __nv_bfloat16* dst = y + (tok0 + t) * p.ld_y + hc;
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
       const int v = (n0 + i) * 8 + (lane & 3) * 2;
       if (v >= p.dim) continue;
-      const float2 gg = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(g + v));
+      const float2 gg = unpack_bf16x2(gate[h][i]);
       const float2 w = *reinterpret_cast<const float2*>(p.norm + hc + v);
       *reinterpret_cast<uint32_t*>(dst + v) =
-          pack_bf16x2(acc[i][2 * h] * inv * w.x * silu_f(gg.x), acc[i][2 * h + 1] * inv * w.y * silu_f(gg.y));
+          pack_bf16x2(acc[i][2 * h] * inv * w.x * silu_fast(gg.x), acc[i][2 * h + 1] * inv * w.y * silu_fast(gg.y));
     }
   }
 }
@@ -686,9 +777,10 @@ int launch_wkv_decode(const nfk_wkv_params& p, cudaStream_t stream) {
   const size_t sm = static_cast<size_t>(p.dim) * 16;
   if (grid > 0x7fffffffll || sm > 40 * 1024) return NF_ERR_BAD_ARG;
   const int g = static_cast<int>(grid);
-  if (p.dim <= 32) wkv_decode_kernel<T, 8><<<g, 256, sm, stream>>>(p);
-  else if (p.dim <= 64) wkv_decode_kernel<T, 16><<<g, 256, sm, stream>>>(p);
-  else wkv_decode_kernel<T, 32><<<g, 256, sm, stream>>>(p);
+  if (p.dim <= 32) wkv_decode_kernel<T, 8, 1><<<g, 256, sm, stream>>>(p);
+  else if (p.dim <= 64) wkv_decode_kernel<T, 16, 4><<<g, 256, sm, stream>>>(p);
+  else if (p.dim <= 128) wkv_decode_kernel<T, 32, 16><<<g, 256, sm, stream>>>(p);
+  else wkv_decode_kernel<T, 32, 0><<<g, 256, sm, stream>>>(p);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 

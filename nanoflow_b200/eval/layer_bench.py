@@ -1,9 +1,10 @@
 """Prefill and decode throughput of a layer-list model beside the Llama model of equal size, layer by layer.
 
     python bench.py --layer-list 8B            (or 2B, or both: 2B,8B)
+    python bench.py --layer-list 8B --layer-model zubedra
 
-Both models get the same width, feed-forward, head count and number of layers, random weights, and the same
-batches: whole prompts in one iteration, and single-token decoding over a given context. Engines, kernels
+Both models get the same width, feed-forward (of a mixture of experts: what a token uses), head count and number of
+layers, random weights, and the same batches: whole prompts in one iteration, and single-token decoding over a given context. Engines, kernels
 and step function are those of serving; each workload has an engine of its own batch size, so that both models'
 GEMM shapes are the tuned ones. Time: CUDA events around repeated iterations (CUDA graphs, weights far larger than
 L2), then one iteration with an event pair around every op for the per-kernel table. Each kernel is set against
@@ -19,10 +20,14 @@ import numpy as np
 import torch
 
 SIZES = {
-    # name: (width, ff, heads, kv heads of the Llama, vocab, latent rank, window, mLSTM heads, dim, vdim)
-    "8B": dict(width=4096, ff=14336, heads=32, kv=8, vocab=128256, rank=512, window=1024, mh=8, md=256, mv=512),
-    "2B": dict(width=2048, ff=8192, heads=16, kv=4, vocab=32000, rank=256, window=512, mh=4, md=256, mv=512),
+    # name: (width, ff, heads, kv heads of the Llama, vocab, latent rank, window, mLSTM heads, dim, vdim,
+    #        WKV decay rank, ff of an expert and of the shared one: 6 experts per token and the shared one make up ff)
+    "8B": dict(width=4096, ff=14336, heads=32, kv=8, vocab=128256, rank=512, window=1024, mh=8, md=256, mv=512, decay=128,
+               eff=2048, sff=2048),
+    "2B": dict(width=2048, ff=8192, heads=16, kv=4, vocab=32000, rank=256, window=512, mh=4, md=256, mv=512, decay=64,
+               eff=1024, sff=2048),
 }
+EXPERTS, TOP, GROUPS, KEEP = 64, 6, 8, 4
 WORKLOADS = [("prefill 4 x 1024", [(0, 1024)] * 4), ("prefill 1 x 4096", [(0, 4096)]),
              ("decode 256 at 1280", [(1280, 1)] * 256), ("decode 32 at 4096", [(4096, 1)] * 32)]
 LAYERS = 4
@@ -39,10 +44,14 @@ def peaks() -> Tuple[float, float]:
 
 def model_dict(kind: str, s: Dict[str, int]) -> Dict[str, Any]:
     from ..config import _hf
-    from ..models.volarax import builtin
+    from ..models import volarax, zubedra
     if kind == "llama":
         return _hf(s["width"], s["ff"], LAYERS, s["heads"], s["kv"], s["vocab"], 500000.0)
-    return builtin(s["width"], s["vocab"], "am" * (LAYERS // 2), heads=s["heads"], dim=128, vdim=128, kv_rank=s["rank"],
+    if kind == "zubedra":
+        return zubedra.builtin(s["width"], s["vocab"], "aw" * (LAYERS // 2), heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128,
+                               softcap=50.0, w_heads=s["width"] // 64, w_dim=64, rank=s["decay"], experts=EXPERTS, top=TOP,
+                               ff=s["eff"], groups=GROUPS, keep=KEEP, shared_ff=s["sff"])
+    return volarax.builtin(s["width"], s["vocab"], "am" * (LAYERS // 2), heads=s["heads"], dim=128, vdim=128, kv_rank=s["rank"],
                    window=s["window"], m_heads=s["mh"], m_dim=s["md"], m_vdim=s["mv"], ff=s["ff"], m_ff=s["ff"])
 
 
@@ -72,7 +81,7 @@ def make_plan(engine, spans, pages: int):
         if window:
             kv.trim(ctx - window + 1)
         kv.allocate_tokens(n)
-        parts.append(Portion(kv, np.random.default_rng(0).integers(0, m.vocab_size, n), [n - 1]))
+        parts.append(Portion(kv, np.random.default_rng(len(parts)).integers(0, m.vocab_size, n), [n - 1]))
     return plan_portions(parts, tile_tokens=max(1, 128 // m.group_size))
 
 
@@ -114,7 +123,28 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
         return T * p.heads * (chunk * (p.dim + p.vdim) + 4.0 * p.dim * p.vdim), (2 if dec else 1) * state + io
     if isinstance(p, G.ResidualNormParams):
         rows = T if not p.rows_idx else len(spans)
-        return 0.0, rows * p.cols * (8 + 2 * es)
+        more = (1 if p.y2 else 0) + (p.e_top if p.e_out else 0)
+        return 0.0, rows * p.cols * (8 + (2 + more) * es)
+    if isinstance(p, G.GqaAppendParams):
+        return 0.0, T * 2 * (p.heads + 2 * p.kv_heads) * p.hd * es
+    if isinstance(p, G.TokenShiftParams):
+        return 0.0, T * (1 + p.n_mix) * p.ld_h * es
+    if isinstance(p, G.WkvParams):
+        dec = "decode" in op.kernel
+        if (spans[0][1] == 1) != dec:
+            return 0.0, 0.0
+        state = len(spans) * p.heads * p.dim * p.dim * 4
+        io = T * p.heads * p.dim * (5 * es + 4)
+        chunk = 0 if dec else 64
+        return T * p.heads * (2.0 * chunk * p.dim + 4.0 * p.dim * p.dim), 2 * state + io
+    if isinstance(p, G.MoeRouteParams):
+        return 0.0, T * 4 * (p.experts + 3 * p.top)
+    if isinstance(p, G.MoePermuteParams):
+        return 0.0, T * (1 + p.top) * p.cols * es
+    if isinstance(p, G.MoeGemmParams):
+        rows, mats = engine._last_sym.get(dict(op.dyn)["rows"], 0), 2 if p.B2 else 1
+        used = min(p.experts, engine._experts_used)
+        return 2.0 * rows * p.N * p.K * mats, es * (mats * used * p.N * p.K + rows * (p.K + p.N))
     if isinstance(p, G.HeadNormGateParams):
         return 0.0, T * p.heads * p.vdim * (4 + 2 * es)
     if isinstance(p, G.LatentAppendParams):
@@ -145,6 +175,9 @@ def measure(engine, plan, spans, steps: int, warmup: int) -> Dict[str, Any]:
     torch.cuda.synchronize()
     ms = e0.elapsed_time(e1) / steps
     engine.check_status()
+    # experts that got rows in the last iteration (fewest of all layers): their weights have to be read
+    counts = [c for c in getattr(engine, "moe_counts_of", []) if c is not None]
+    engine._experts_used = min((int((c > 0).sum()) for c in counts), default=0)
     # one op at a time, best of three iterations
     best: Dict[int, float] = {}
     for _ in range(3):
@@ -172,7 +205,7 @@ def measure(engine, plan, spans, steps: int, warmup: int) -> Dict[str, Any]:
             "ops": {k: {"us": round(us / n, 1), "of_roofline": round(roof / us, 3)} for k, (n, us, roof) in table.items()}}
 
 
-def run(sizes: List[str], steps: int, warmup: int, only: str = "") -> Dict[str, Any]:
+def run(sizes: List[str], steps: int, warmup: int, only: str = "", model: str = "volarax") -> Dict[str, Any]:
     device = torch.device("cuda", torch.cuda.current_device())
     out: Dict[str, Any] = {}
     for size in sizes:
@@ -180,7 +213,7 @@ def run(sizes: List[str], steps: int, warmup: int, only: str = "") -> Dict[str, 
             if only and only not in label:
                 continue
             pages = sum((c + n + 15) // 16 for c, n in spans) + 8
-            for kind in ("llama", "volarax"):
+            for kind in ["llama"] + model.split(","):
                 engine = make_engine(kind, SIZES[size], spans, device, pages)
                 res = measure(engine, make_plan(engine, spans, pages), spans, steps, warmup)
                 engine.finalize()

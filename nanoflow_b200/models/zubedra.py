@@ -192,7 +192,7 @@ def random_weights(cfg: LayerListConfig, raw: Dict[str, Any], device="cpu", seed
 
 def builtin(width: int, vocab: int, pattern: str, *, heads: int, kv_heads: int, dim: int, vdim: int, softcap: float,
             w_heads: int, w_dim: int, rank: int, experts: int, top: int, ff: int, groups: int, keep: int, shared_ff: int,
-            limit: float = 7.0, router_scale: float = 2.5, eps: float = 1e-5) -> Dict[str, Any]:
+            limit: float = 7.0, router_scale: float = 2.0, eps: float = 1e-5) -> Dict[str, Any]:
     """A ``config.json`` dictionary from a layer pattern ("a": attention, "w": WKV; both with the mixture of experts)."""
     mlp = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "shared": {"ff": shared_ff, "limit": limit},
            "router": {"experts": experts, "top": top, "scale": router_scale, "groups": {"count": groups, "keep": keep}}}

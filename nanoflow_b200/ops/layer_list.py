@@ -1,4 +1,5 @@
-"""Python entry points for the layer-list kernels (residual step, latent attention, mLSTM, general GEMM forms).
+"""Python entry points for the layer-list kernels (residual step, attention, recurrences, mixture of experts, general
+GEMM forms).
 
 Like the functions of :mod:`nanoflow_b200.ops` they take torch CUDA tensors, check what the C ABI cannot and
 launch on the current stream; engines do not call them but put the same parameter blocks into their op graph.
@@ -10,8 +11,9 @@ from typing import Optional
 
 import torch
 
-from . import (ACTS, NORMS, AttnParams, GemmParams, HeadNormGateParams, LatentAppendParams, LatentAttnParams, MlstmParams,
-               ResidualNormParams, LatentGatherParams, _check, _i32, _p, _stream, dtype_code, lib)
+from . import (ACTS, LIN_ACTS, NORMS, AttnParams, GemmParams, GqaAppendParams, GqaAttnParams, HeadNormGateParams,
+               LatentAppendParams, LatentAttnParams, LatentGatherParams, MlstmParams, MoeGemmParams, MoePermuteParams,
+               MoeRouteParams, ResidualNormParams, TokenShiftParams, WkvParams, _check, _i32, _p, _stream, dtype_code, lib)
 
 
 def _f32(t: Optional[torch.Tensor], name: str) -> None:
@@ -21,9 +23,11 @@ def _f32(t: Optional[torch.Tensor], name: str) -> None:
 
 def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None, up: Optional[torch.Tensor] = None,
          act: str = "silu", out32: Optional[torch.Tensor] = None, f32_col0: int = 0, groups: int = 1, group_k: int = 0,
-         k: int = 0, workspace: Optional[torch.Tensor] = None, status=None, **shape) -> Optional[torch.Tensor]:
+         k: int = 0, lin_act: Optional[str] = None, bias=None, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0,
+         workspace: Optional[torch.Tensor] = None, status=None, **shape) -> Optional[torch.Tensor]:
     """a @ w^T in the storage type of the operands (bf16: tensor cores, fp32: FMA). ``up``: act(a @ w^T) * (a @ up^T).
-    ``out32``: columns from ``f32_col0`` on are written there as fp32. ``groups``: block-diagonal product."""
+    ``out32``: columns from ``f32_col0`` on are written there as fp32. ``groups``: block-diagonal product. ``lin_act``:
+    activation of the finished columns; ``limit``, ``alpha``, ``shift``: constants of the "capped" gated form."""
     M, N, p = a.shape[0], w.shape[0], GemmParams()
     if a.dtype != w.dtype or a.stride(1) != 1 or w.stride(1) != 1:
         raise RuntimeError("gemm: operands of one type with unit inner stride expected")
@@ -34,6 +38,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
     p.lda, p.ldb, p.ldd = a.stride(0), w.stride(0), out.stride(0) if out is not None else N
     p.M, p.N, p.K = M, N, k or w.shape[1]
     p.epilogue, p.act, p.groups, p.group_k = (1 if up is not None else 0), ACTS[act], groups, group_k
+    p.lin_act, p.bias, p.act_limit, p.act_alpha, p.act_shift = LIN_ACTS[lin_act], _p(bias), limit, alpha, shift
     if out32 is not None:
         p.D32, p.ld32, p.f32_col0 = _p(out32), out32.stride(0), f32_col0
     if workspace is not None:
@@ -47,13 +52,23 @@ def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
 
 
 def residual_norm(x: torch.Tensor, *, y=None, table=None, ids=None, feedback_src=None, prev_tokens=None, norm_in=None,
-                  add=None, h=None, norm_out=None, rows_idx=None, cols: int, eps: float, rows: Optional[int] = None,
-                  status=None) -> None:
-    """x <- (table ? 0 : x) + norm_in(y or table[ids]) (+ add); h <- norm_out(x). Norms: (kind, weight, bias)."""
+                  add=None, h=None, norm_out=None, rows_idx=None, src_scale: float = 1.0, y2=None, y2_gate=None, experts=None,
+                  cols: int, eps: float, rows: Optional[int] = None, status=None) -> None:
+    """x <- (table ? 0 : x) + norm_in(src_scale * (y or table[ids])) (+ y2_gate y2) (+ weighted rows of ``experts``:
+    outputs, slots, weights) (+ add); h <- norm_out(x). Norms: (kind, weight, bias)."""
     p = ResidualNormParams()
     _f32(x, "x")
     p.x, p.ld_x = _p(x), x.stride(0)
-    typed = next(t for t in (y, table, h) if t is not None)
+    typed = next(t for t in (y, table, h, y2) if t is not None)
+    p.src_scale = src_scale
+    if y2 is not None:
+        _f32(y2_gate, "y2_gate")
+        p.y2, p.ld_y2, p.y2_gate = _p(y2), y2.stride(0), _p(y2_gate)
+    if experts is not None:
+        out, slot, weight = experts
+        _i32(slot, "slots"); _f32(weight, "weights")
+        p.e_out, p.ld_e, p.e_rows = _p(out), out.stride(0), out.shape[0]
+        p.e_slot, p.e_weight, p.e_top = _p(slot), _p(weight), slot.shape[1]
     p.dtype = dtype_code(typed.dtype)
     if y is not None:
         p.y, p.ld_y = _p(y), y.stride(0)
@@ -176,3 +191,123 @@ def head_norm_gate(o, g, w, out, *, heads: int, vdim: int, eps: float) -> None:
     p = HeadNormGateParams(o=_p(o), ld_o=o.stride(0), g=_p(g), ld_g=g.stride(0), w=_p(w), out=_p(out), ld_out=out.stride(0),
                            T=o.shape[0], heads=heads, vdim=vdim, vdim_p=w.numel() // heads, eps=eps, dtype=dtype_code(out.dtype))
     _check(lib().nfk_head_norm_gate(byref(p), _stream()), "nfk_head_norm_gate")
+
+
+def gqa_append(src, q_out, pool, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, heads: int, dim: int,
+               q_w=None, k_w=None, v_first=None, v_mode: int = 0, v_lambda: float = 0.0, eps: float, status=None) -> None:
+    """src rows are q | k | v (heads padded to the pool's head size); normed keys and the values go to ``pool`` [pages, 2,
+    kv_heads, page size, head size], normed queries to ``q_out``."""
+    for t, nm in ((q_w, "q_w"), (k_w, "k_w")):
+        _f32(t, nm)
+    n, _, G, ps, hd = pool.shape
+    p = GqaAppendParams(src=_p(src), ld_src=src.stride(0), q_off=0, k_off=heads * hd, v_off=(heads + G) * hd, q_out=_p(q_out),
+                        q_w=_p(q_w), k_w=_p(k_w), v_first=_p(v_first), v_mode=v_mode, v_lambda=v_lambda, pool=_p(pool),
+                        positions=_p(positions), token_req=_p(token_req), kv_indptr=_p(kv_indptr), kv_indices=_p(kv_indices),
+                        kv_first=_p(kv_first), T=src.shape[0], heads=heads, kv_heads=G, hd=hd, dim=dim, page_size=ps,
+                        num_pages=n, eps=eps, dtype=dtype_code(pool.dtype), status=_p(status))
+    _check(lib().nfk_gqa_append(byref(p), _stream()), "nfk_gqa_append")
+
+
+def gqa_attention(q, pool, out, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, heads: int, scale: float,
+                  softcap: float = 0.0, window: int = 0, sinks=None, token_begin: int = 0, n_tokens: Optional[int] = None,
+                  status=None) -> None:
+    """The simple kernel: any head size, bf16 or fp32; q, out [T, heads * head size]."""
+    _f32(sinks, "sinks")
+    n, _, G, ps, hd = pool.shape
+    p = GqaAttnParams(q=_p(q), pool=_p(pool), out=_p(out), positions=_p(positions), token_req=_p(token_req),
+                      kv_indptr=_p(kv_indptr), kv_indices=_p(kv_indices), kv_first=_p(kv_first), sinks=_p(sinks),
+                      token_begin=token_begin, n_tokens=q.shape[0] - token_begin if n_tokens is None else n_tokens, heads=heads,
+                      kv_heads=G, hd=hd, page_size=ps, num_pages=n, window=window, scale=scale, softcap=softcap,
+                      dtype=dtype_code(pool.dtype), status=_p(status))
+    _check(lib().nfk_gqa_attn(byref(p), _stream()), "nfk_gqa_attn")
+
+
+def paged_attention(q, pool, out, qo_indptr, kv_indptr, kv_indices, kv_last_page_len, *, heads: int, scale: float,
+                    softcap: float = 0.0, sinks=None, items=None, req_count: int = 0, chunk_pages: int = 0,
+                    max_chunks: int = 1, workspace=None, status=None) -> None:
+    """The tensor-core kernels with capped scores, sinks and probabilities in two parts: portions (``items`` [n, 3]: request,
+    first token, tokens) on the prefill kernel, else single tokens of the first ``req_count`` requests."""
+    _f32(sinks, "sinks")
+    p = AttnParams()
+    p.q, p.out, p.kv_pool = _p(q), _p(out), _p(pool)
+    p.qo_indptr, p.kv_indptr, p.kv_indices = _p(qo_indptr), _p(kv_indptr), _p(kv_indices)
+    p.kv_last_page_len, p.q_heads, p.kv_heads = _p(kv_last_page_len), heads, pool.shape[2]
+    p.head_dim, p.page_size, p.num_pages, p.sm_scale = pool.shape[4], pool.shape[3], pool.shape[0], scale
+    p.softcap, p.sinks, p.precise, p.status = softcap, _p(sinks), 1, _p(status)
+    if items is not None:
+        p.items, p.num_items = _p(items), items.shape[0]
+        _check(lib().nfk_attn_prefill_ws(byref(p), _stream()), "nfk_attn_prefill_ws")
+        return
+    p.req_count, p.chunk_pages, p.max_chunks, p.workspace = req_count, chunk_pages, max_chunks, _p(workspace)
+    _check(lib().nfk_attn_decode(byref(p), _stream()), "nfk_attn_decode")
+
+
+def moe_route(logits, correction, counts, *, top: int, experts: int, groups: int = 1, keep: int = 1, scale: float,
+              gate_col: int = -1):
+    """(experts [T, top], weights, ranks, gate [T]); ``counts`` [experts] is increased."""
+    _f32(logits, "logits"); _f32(correction, "correction"); _i32(counts, "counts")
+    T, dev = logits.shape[0], logits.device
+    idx, rank = (torch.zeros(T, top, dtype=torch.int32, device=dev) for _ in range(2))
+    weight, gate = torch.zeros(T, top, device=dev), torch.zeros(T, device=dev)
+    p = MoeRouteParams(logits=_p(logits), ld=logits.stride(0), correction=_p(correction), expert=_p(idx), weight=_p(weight),
+                       rank=_p(rank), counts=_p(counts), gate=_p(gate), T=T, experts=experts, top=top, groups=groups, keep=keep,
+                       gate_col=gate_col, scale=scale)
+    _check(lib().nfk_moe_route(byref(p), _stream()), "nfk_moe_route")
+    return idx, weight, rank, gate
+
+
+def moe_permute(h, expert, rank, counts):
+    """(rows of h in expert order [T * top, cols], slots [T, top])."""
+    T, top = expert.shape
+    out = torch.zeros(T * top, h.shape[1], dtype=h.dtype, device=h.device)
+    slot = torch.zeros(T, top, dtype=torch.int32, device=h.device)
+    p = MoePermuteParams(h=_p(h), ld_h=h.stride(0), out=_p(out), ld_out=out.stride(0), expert=_p(expert), rank=_p(rank),
+                         counts=_p(counts), slot=_p(slot), T=T, top=top, experts=counts.numel(), cols=h.shape[1],
+                         dtype=dtype_code(h.dtype))
+    _check(lib().nfk_moe_permute(byref(p), _stream()), "nfk_moe_permute")
+    return out, slot
+
+
+def moe_gemm(a, w, counts, *, up=None, act: str = "silu", limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0,
+             status=None) -> torch.Tensor:
+    """Rows of ``a`` in expert order times their expert's matrix; w (and up) [experts * N, K]."""
+    _i32(counts, "counts")
+    E = counts.numel()
+    n = w.shape[0] // E
+    out = torch.zeros(a.shape[0], n, dtype=a.dtype, device=a.device)
+    p = MoeGemmParams(A=_p(a), B=_p(w), B2=_p(up), D=_p(out), counts=_p(counts), lda=a.stride(0), ldb=w.stride(0),
+                      ldd=out.stride(0), rows=a.shape[0], experts=E, N=n, K=w.shape[1], act=ACTS[act], act_limit=limit,
+                      act_alpha=alpha, act_shift=shift, dtype=dtype_code(a.dtype), num_ctas=0, status=_p(status))
+    _check(lib().nfk_moe_gemm(byref(p), _stream()), "nfk_moe_gemm")
+    return out
+
+
+def token_shift(h, mu, state, state_ref, positions, token_req, qo_indptr, status=None) -> torch.Tensor:
+    """[T, n_mix * width]: every stream's mix of a row with the previous token's; ``state`` [slots, 2, width]."""
+    _f32(mu, "mu")
+    out = torch.zeros(h.shape[0], mu.shape[0] * h.shape[1], dtype=h.dtype, device=h.device)
+    p = TokenShiftParams(h=_p(h), ld_h=h.stride(0), out=_p(out), mu=_p(mu), state=_p(state), state_slot=_p(state_ref),
+                         positions=_p(positions), token_req=_p(token_req), qo_indptr=_p(qo_indptr), T=h.shape[0],
+                         n_mix=mu.shape[0], num_slots=state.shape[0], dtype=dtype_code(h.dtype), status=_p(status))
+    _check(lib().nfk_token_shift(byref(p), _stream()), "nfk_token_shift")
+    return out
+
+
+def wkv(rkvg, x, u, norm, state, y, positions, qo_indptr, state_ref, *, dim_real: int, eps: float, decode: int = 0,
+        items=None, seq=None, status=None) -> None:
+    """rkvg rows are r | k | v | g of all heads, x [T, heads * dim]; ``state`` [slots, heads, dim, dim] in place. ``decode``: the
+    first so many requests have one token each; else ``items`` [n, 4] in chunks and the requests ``seq`` token by token."""
+    for t, nm in ((x, "x"), (u, "u"), (norm, "norm"), (state, "state")):
+        _f32(t, nm)
+    _, heads, dim, _ = state.shape
+    o = torch.zeros(rkvg.shape[0], heads * dim, device=rkvg.device)
+    n = 0 if items is None else items.shape[0]
+    ws = torch.zeros(max(1, n) * heads * (dim * dim + dim), device=rkvg.device)
+    p = WkvParams(rkvg=_p(rkvg), ld=rkvg.stride(0), r_off=0, k_off=heads * dim, v_off=2 * heads * dim, g_off=3 * heads * dim,
+                  x=_p(x), ld_x=x.stride(0), u=_p(u), norm=_p(norm), S=_p(state), y=_p(y), ld_y=y.stride(0),
+                  positions=_p(positions), qo_indptr=_p(qo_indptr), state_slot=_p(state_ref), req_begin=0, req_count=decode,
+                  heads=heads, dim=dim, dim_real=dim_real, num_slots=state.shape[0], eps=eps, dtype=dtype_code(rkvg.dtype),
+                  seq_reqs=_p(seq), num_seq=0 if seq is None else seq.numel(), o=_p(o), items=_p(items), num_items=n,
+                  scratch=_p(ws), scratch_floats=ws.numel(), status=_p(status))
+    name = "nfk_wkv_decode" if decode else "nfk_wkv_prefill"
+    _check(getattr(lib(), name)(byref(p), _stream()), name)

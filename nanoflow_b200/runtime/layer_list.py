@@ -523,8 +523,8 @@ class LayerListEngine(Engine):
                               num_slots=self.num_slots, dtype=self.code, status=st)
         self._op(f"R{r}.token_shift", ts, dyn=[("T", T)], layer=r)
         self._gemm(f"R{r}.in", mix, lw.w_in, proj, rows=T, groups=4, group_k=wp, k=wp, key=f"l{layer}.in", layer=r)
-        self._gemm(f"R{r}.decay_down", mix[:, 4 * wp:], lw.w_down, lora, rows=T, lin_act="tanh", layer=r)
-        self._gemm(f"R{r}.decay_up", lora, lw.w_up, None, rows=T, d32=decay, bias=lw.w_bias, layer=r)
+        self._gemm(f"R{r}.decay_down", mix[:, 4 * wp:], lw.w_down, lora, rows=T, lin_act="tanh", key=f"l{layer}.decay_down", layer=r)
+        self._gemm(f"R{r}.decay_up", lora, lw.w_up, None, rows=T, d32=decay, bias=lw.w_bias, key=f"l{layer}.decay_up", layer=r)
 
         def params() -> WkvParams:
             return WkvParams(rkvg=_ptr(proj), ld=proj.stride(0), r_off=0, k_off=H * d, v_off=2 * H * d, g_off=3 * H * d,
@@ -560,7 +560,7 @@ class LayerListEngine(Engine):
         logits, counts, cap = self.view("router", lw.router.shape[0]), self.moe_counts_of[r], self.T * s.top
         flat = lambda k, cols: self.flat[k][:cap * cols].view(cap, cols)
         e_in, e_act, e_out = flat("e_in", wp), flat("e_act", round8(s.expert.ff)), flat("e_out", wp)
-        self._gemm(f"R{r}.router", self.h, lw.router, None, rows=T, d32=logits, layer=r)
+        self._gemm(f"R{r}.router", self.h, lw.router, None, rows=T, d32=logits, key=f"l{layer}.router", layer=r)
         rp = MoeRouteParams(logits=_ptr(logits), ld=logits.stride(0), correction=_ptr(lw.correction), expert=_ptr(ids["expert"]),
                             weight=_ptr(ids["weight"]), rank=_ptr(ids["rank"]), counts=_ptr(counts), gate=_ptr(self.moe_gate),
                             T=0, experts=s.experts, top=s.top, groups=s.groups, keep=s.keep,
@@ -592,13 +592,19 @@ class LayerListEngine(Engine):
         from ..ops import autotune
         m, T, done = self.model, self.T, {}
         self.h.normal_()
-        for k in ("attn", "act"):
+        for k in ("attn", "act", "lora"):
             self.flat[k].normal_()
         for i, lay in enumerate(m.layers):
             lw = self.w.layers[i]
             specs = [("o", None, lw.mixer.w_o, None, None)]
-            if lay.mixer.kind != "wkv":          # (its input projection is block-diagonal: left to the cost model)
+            if lay.mixer.kind == "wkv":          # (its input projection is block-diagonal: left to the cost model)
+                lora = self.view("lora", lw.mixer.w_down.shape[0])
+                specs += [("decay_down", self.h, lw.mixer.w_down, None, self.flat["proj"]),
+                          ("decay_up", lora, lw.mixer.w_up, None, self.flat["proj"])]
+            else:
                 specs.append(("in", self.h, lw.mixer.w_in, None, self.flat["proj"]))
+            if lay.mlp is not None and lay.mlp.kind == "moe":
+                specs.append(("router", self.h, lw.mlp.router, None, self.flat["proj"]))
             f, key = (lw.mlp, "") if lay.mlp is None or lay.mlp.kind == "dense" else (lw.mlp.shared, "shared_")
             if f is not None:
                 specs += [(key + "gate_up", self.h, f.w_gate, f.w_up, self.flat["act"]), (key + "down", None, f.w_down, None, None)]
