@@ -342,22 +342,10 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld_32x32b_x32(t_lane + s * kTile + 32, r1);
         tmem_ld_wait();
         if (CAP) {
-          // a row whose scores are all well below the cap does without the special function unit
-          float top = 0.f;
 #pragma unroll
-          for (int j = 0; j < 32; ++j) top = fmaxf(top, fmaxf(fabsf(__uint_as_float(r0[j])), fabsf(__uint_as_float(r1[j]))));
-          if (__all_sync(0xffffffffu, top * cap_in <= kTanhSmall)) {
-#pragma unroll
-            for (int j = 0; j < 32; ++j) {
-              r0[j] = __float_as_uint(cap_out * tanh_small(__uint_as_float(r0[j]) * cap_in));
-              r1[j] = __float_as_uint(cap_out * tanh_small(__uint_as_float(r1[j]) * cap_in));
-            }
-          } else {
-#pragma unroll
-            for (int j = 0; j < 32; ++j) {
-              r0[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r0[j]) * cap_in));
-              r1[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r1[j]) * cap_in));
-            }
+          for (int j = 0; j < 32; ++j) {
+            r0[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r0[j]) * cap_in));
+            r1[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r1[j]) * cap_in));
           }
         }
         const int cbase = (it.t_first + t) * kTile;

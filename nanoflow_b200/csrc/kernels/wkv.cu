@@ -276,48 +276,63 @@ struct WkvCfg {
   static constexpr int OUT_SMEM = 5 * ROWS_BYTES + CE_BYTES + TOT_BYTES + 2 * S_BYTES + 2 * A_BYTES + DP * 4 + 3 * kChunk * 4 + 16;
 };
 
+// A chunk's operands are all requested before any of them is waited for: rows of r, k, v by asynchronous copies, logs
+// of the decays (and the incoming state) into registers.
+__device__ __forceinline__ void cp_async16_or_zero(void* smem_dst, const void* src, bool ok) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
 // 64 rows of a head's columns of rkvg into [64][BLD]; rows past `n` and columns past the head's are zero.
 template <int DP>
 __device__ __forceinline__ void load_rows(__nv_bfloat16* dst, const nfk_wkv_params& p, long long tok0, int n, int col0) {
   constexpr int CH = DP / 8;
   const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.rkvg);
-  for (int i = threadIdx.x; i < kChunk * CH; i += 256) {
-    const int r = i / CH, c = (i % CH) * 8;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < n && c < p.dim) v = *reinterpret_cast<const uint4*>(src + (tok0 + r) * p.ld + col0 + c);
-    *reinterpret_cast<uint4*>(dst + r * WkvCfg<DP>::BLD + c) = v;
+#pragma unroll
+  for (int j = 0; j < kChunk * CH / 256; ++j) {
+    const int i = threadIdx.x + j * 256, r = i / CH, c = (i % CH) * 8;
+    const bool ok = r < n && c < p.dim;
+    cp_async16_or_zero(dst + r * WkvCfg<DP>::BLD + c, src + (ok ? (tok0 + r) * p.ld + col0 + c : 0), ok);
   }
 }
-// ce[t][d]: sum of the log2 decays of the tokens of t's run before t; tot[run][d]: sum over the run.
 template <int DP>
-__device__ __forceinline__ void load_decays(float* ce, float* tot, const nfk_wkv_params& p, long long tok0, int n, int hc,
-                                            int* slow = nullptr) {
-  constexpr int CH = DP / 4, FLD = WkvCfg<DP>::FLD;
-  for (int i = threadIdx.x; i < kChunk * CH; i += 256) {
-    const int r = i / CH, c = (i % CH) * 4;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < n && c < p.dim) {
-      v = load4(p.x + (tok0 + r) * p.ld_x + hc + c);
-      v = make_float4(decay_log2(v.x), decay_log2(v.y), decay_log2(v.z), decay_log2(v.w));
-    }
-    store4(ce + r * FLD + c, v);
-  }
-  __syncthreads();
-  for (int i = threadIdx.x; i < kRuns * DP; i += 256) {
-    const int run = i / DP, d = i % DP;
-    float l[kRun], s = 0.f;
+struct DecayRegs {
+  static constexpr int N = kChunk * (DP / 4) / 256;
+  float4 v[N];
+  __device__ __forceinline__ void fetch(const nfk_wkv_params& p, long long tok0, int n, int hc) {
 #pragma unroll
-    for (int j = 0; j < kRun; ++j) l[j] = ce[(run * kRun + j) * FLD + d];
-#pragma unroll
-    for (int j = 0; j < kRun; ++j) {
-      ce[(run * kRun + j) * FLD + d] = s;
-      s += l[j];
+    for (int j = 0; j < N; ++j) {
+      const int i = threadIdx.x + j * 256, r = i / (DP / 4), c = (i % (DP / 4)) * 4;
+      // no decay past the last token: the chunk's total is that of its tokens
+      v[j] = (r < n && c < p.dim) ? load4(p.x + (tok0 + r) * p.ld_x + hc + c) : make_float4(-INFINITY, -INFINITY, -INFINITY, -INFINITY);
     }
-    tot[i] = s;
-    if (slow != nullptr && s < -kMaxRunLog2) slow[run] = 1;
   }
-  __syncthreads();
-}
+  // ce[t][d]: sum of the log2 decays of the tokens of t's run before t; tot[run][d]: sum over the run. Also waits for the
+  // rows.
+  __device__ __forceinline__ void finish(float* ce, float* tot, int* slow) const {
+    constexpr int FLD = WkvCfg<DP>::FLD;
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+      const int i = threadIdx.x + j * 256, r = i / (DP / 4), c = (i % (DP / 4)) * 4;
+      store4(ce + r * FLD + c, make_float4(decay_log2(v[j].x), decay_log2(v[j].y), decay_log2(v[j].z), decay_log2(v[j].w)));
+    }
+    cp_async_commit();
+    cp_async_wait<0>();
+    __syncthreads();
+    for (int i = threadIdx.x; i < kRuns * DP; i += 256) {
+      const int run = i / DP, d = i % DP;
+      float l[kRun], s = 0.f;
+#pragma unroll
+      for (int j = 0; j < kRun; ++j) l[j] = ce[(run * kRun + j) * FLD + d];
+#pragma unroll
+      for (int j = 0; j < kRun; ++j) {
+        ce[(run * kRun + j) * FLD + d] = s;
+        s += l[j];
+      }
+      tot[i] = s;
+      if (slow != nullptr && s < -kMaxRunLog2) slow[run] = 1;
+    }
+    __syncthreads();
+  }
+};
 __device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(x, y);
   const float2 h = unpack_bf16x2(hi);
@@ -340,7 +355,9 @@ wkv_chunk_state_kernel(nfk_wkv_params p) {
   const long long tok0 = p.items[item * 4 + 1];
   load_rows<DP>(k_s, p, tok0, n, p.k_off + hc);
   load_rows<DP>(v_s, p, tok0, n, p.v_off + hc);
-  load_decays<DP>(ce, tot, p, tok0, n, hc);
+  DecayRegs<DP> dec;
+  dec.fetch(p, tok0, n, hc);
+  dec.finish(ce, tot, nullptr);
   float* L = p.scratch + (static_cast<long long>(item) * p.heads + head) * wkv_item_floats(p.dim);
   for (int d = threadIdx.x; d < p.dim; d += 256)
     L[p.dim * p.dim + d] = fast_exp2((tot[d] + tot[DP + d]) + (tot[2 * DP + d] + tot[3 * DP + d]));
@@ -467,19 +484,28 @@ wkv_chunk_out_kernel(nfk_wkv_params p) {
   load_rows<DP>(r_s, p, tok0, n, p.r_off + hc);
   load_rows<DP>(k_s, p, tok0, n, p.k_off + hc);
   load_rows<DP>(v_s, p, tok0, n, p.v_off + hc);
+  DecayRegs<DP> dec;
+  dec.fetch(p, tok0, n, hc);
   const float* S = p.scratch + (static_cast<long long>(item) * p.heads + head) * wkv_item_floats(p.dim);
-  for (int i = threadIdx.x; i < DP * (DP / 4); i += 256) {
-    const int d = i / (DP / 4), c = (i % (DP / 4)) * 4;
-    const float4 x = (d < p.dim && c < p.dim) ? load4(S + d * p.dim + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-    uint2 hi, lo;
-    split_pair(x.x, x.y, hi.x, lo.x);
-    split_pair(x.z, x.w, hi.y, lo.y);
-    *reinterpret_cast<uint2*>(sh_s + d * C::BLD + c) = hi;
-    *reinterpret_cast<uint2*>(sl_s + d * C::BLD + c) = lo;
+  constexpr int SN = DP * (DP / 4) / 256;
+  float4 s_in[SN];
+#pragma unroll
+  for (int j = 0; j < SN; ++j) {
+    const int i = threadIdx.x + j * 256, d = i / (DP / 4), c = (i % (DP / 4)) * 4;
+    s_in[j] = (d < p.dim && c < p.dim) ? load4(S + d * p.dim + c) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   for (int d = threadIdx.x; d < DP; d += 256) u_s[d] = d < p.dim ? p.u[hc + d] : 0.f;
   if (threadIdx.x < kRuns) slow_s[threadIdx.x] = 0;
-  load_decays<DP>(ce, tot, p, tok0, n, hc, slow_s);
+#pragma unroll
+  for (int j = 0; j < SN; ++j) {
+    const int i = threadIdx.x + j * 256, d = i / (DP / 4), c = (i % (DP / 4)) * 4;
+    uint2 hi, lo;
+    split_pair(s_in[j].x, s_in[j].y, hi.x, lo.x);
+    split_pair(s_in[j].z, s_in[j].w, hi.y, lo.y);
+    *reinterpret_cast<uint2*>(sh_s + d * C::BLD + c) = hi;
+    *reinterpret_cast<uint2*>(sl_s + d * C::BLD + c) = lo;
+  }
+  dec.finish(ce, tot, slow_s);
 
   // ---- keys decayed to the end of their run, and every token's own score ----
   for (int i = threadIdx.x; i < kChunk * (DP / 2); i += 256) {
