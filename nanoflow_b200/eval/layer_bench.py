@@ -99,7 +99,8 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
             return 0.0, 0.0
         gated = 2 if p.epilogue == 1 else 1
         groups = max(1, p.groups)
-        return 2.0 * M * p.N * p.K * gated, es * (gated * p.N * p.K + M * (p.K * groups + p.N))
+        wide = p.N - p.f32_col0 if p.D32 else 0          # columns that leave as fp32
+        return 2.0 * M * p.N * p.K * gated, es * (gated * p.N * p.K + M * (p.K * groups + p.N)) + (4 - es) * M * wide
     if isinstance(p, G.AttnParams):
         pre = "prefill" in op.kernel
         if (spans[0][1] == 1) == pre:
