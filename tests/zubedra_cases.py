@@ -1,5 +1,4 @@
 """Small Zubedra configurations and tensors for the tests, made from their own sizes and seeds."""
-import numpy as np
 import torch
 
 from nanoflow_b200.config import parse_config
