@@ -348,6 +348,11 @@ def _zubedra(*a, **kw):
     return builtin(*a, **kw)
 
 
+def _gupizen(*a, **kw):
+    from .models.gupizen import builtin
+    return builtin(*a, **kw)
+
+
 _LLAMA31_SCALING = {"factor": 8.0, "low_freq_factor": 1.0, "high_freq_factor": 4.0,
                     "original_max_position_embeddings": 8192, "rope_type": "llama3"}
 
@@ -383,6 +388,15 @@ MODEL_ARCHS: Dict[str, Dict[str, Any]] = {
                            w_dim=64, rank=128, experts=64, top=6, ff=2048, groups=8, keep=4, shared_ff=2048),
     "zubedra-2B": _zubedra(2048, 32000, "aw" * 12, heads=16, kv_heads=4, dim=128, vdim=128, softcap=50.0, w_heads=32,
                            w_dim=64, rank=64, experts=64, top=6, ff=1024, groups=8, keep=4, shared_ff=2048),
+    "gupizen-tiny": _gupizen(200, 1000, "pdpd", heads=6, kv_heads=2, dim=40, vdim=24, window=37, rot_dims=20, rec_width=144,
+                             rec_blocks=3, d_heads=6, d_kv_heads=3, d_dim=24, d_vdim=40, rank=12, experts=12, top=3, ff=40,
+                             conv=3, loop=(1, 3, 2)),
+    "gupizen-8B": _gupizen(4096, 128256, "pd" * 16, heads=32, kv_heads=8, dim=128, vdim=128, window=1024, rec_width=4096,
+                           rec_blocks=16, d_heads=32, d_kv_heads=32, d_dim=128, d_vdim=128, rank=128, experts=64, top=6,
+                           ff=3584),
+    "gupizen-2B": _gupizen(2048, 32000, "pd" * 12, heads=16, kv_heads=4, dim=128, vdim=128, window=512, rec_width=2048,
+                           rec_blocks=16, d_heads=16, d_kv_heads=16, d_dim=128, d_vdim=128, rank=128, experts=64, top=6,
+                           ff=2048),
 }
 
 MODEL_IDS = {
@@ -392,6 +406,7 @@ MODEL_IDS = {
     "deepseek-67B": "deepseek-ai/deepseek-llm-67b-chat", "mixtral-8-7B": "mistralai/Mixtral-8x7B-Instruct-v0.1",
     "tiny": "nanoflow/tiny-llama-test", "tiny8": "nanoflow/tiny8-llama-test",
     "volarax-tiny": "nanoflow/volarax-tiny-test", "zubedra-tiny": "nanoflow/zubedra-tiny-test",
+    "gupizen-tiny": "nanoflow/gupizen-tiny-test",
 }
 
 

@@ -1,4 +1,4 @@
-// Activation of the gated GEMM epilogues (NFK_ACT_*), shared by the dense and the grouped products.
+// Activations of the GEMM epilogues (NFK_ACT_*, NFK_LIN_*), shared by the dense and the grouped products.
 #pragma once
 #include "kernels.h"
 
@@ -22,5 +22,11 @@ __device__ __forceinline__ float gated_act_of(float g, float u, const GatedAct& 
   return g / (1.f + (PRECISE ? expf(-g) : __expf(-g))) * u;
 }
 __device__ __forceinline__ float gated_act(float g, float u, const GatedAct& a) { return gated_act_of<false>(g, u, a); }
+
+__device__ __forceinline__ float lin_act_of(float v, int kind) {
+  if (kind == NFK_LIN_TANH) return tanhf(v);
+  if (kind == NFK_LIN_GELU) return 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
+  return v;
+}
 
 }  // namespace nf

@@ -188,9 +188,9 @@ __device__ __forceinline__ NBlock n_block(const DevParams& p, int n_blk, int out
 
 // Eight finished columns of one row: bf16 to D, or fp32 to D32 from f32_col0 on (a multiple of 8).
 __device__ __forceinline__ void store_cols8(const DevParams& p, int row, int col, float* v) {
-  if (p.lin_act == NFK_LIN_TANH) {
+  if (p.lin_act != NFK_LIN_NONE) {
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] = tanhf(v[j]);
+    for (int j = 0; j < 8; ++j) v[j] = lin_act_of(v[j], p.lin_act);
   }
   if (p.D32 != nullptr && col >= p.f32_col0) {
     float* out = p.D32 + static_cast<long long>(row) * p.ld32 + (col - p.f32_col0);
@@ -1433,7 +1433,7 @@ extern "C" int nfk_gemm_bf16(const nfk_gemm_params* g, cudaStream_t stream) {
       (g->epilogue != NFK_EPI_LINEAR || g->f32_col0 < 0 || g->f32_col0 % 8 != 0 || g->ld32 % 4 != 0 ||
        (reinterpret_cast<uintptr_t>(g->D32) & 15) != 0 || g->norm_w != nullptr))
     return NF_ERR_BAD_ARG;
-  if (g->act < NFK_ACT_SILU || g->act > NFK_ACT_CAPPED || g->lin_act < NFK_LIN_NONE || g->lin_act > NFK_LIN_TANH) return NF_ERR_BAD_ARG;
+  if (g->act < NFK_ACT_SILU || g->act > NFK_ACT_CAPPED || g->lin_act < NFK_LIN_NONE || g->lin_act > NFK_LIN_GELU) return NF_ERR_BAD_ARG;
   if (g->groups > 1 && (g->epilogue != NFK_EPI_LINEAR || g->N % (8 * g->groups) != 0 || g->group_k % 8 != 0 ||
                         g->group_k < 0 || g->gate_flags != nullptr))
     return NF_ERR_BAD_ARG;

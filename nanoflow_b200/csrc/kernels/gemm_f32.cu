@@ -74,7 +74,7 @@ gemm_f32_kernel(nfk_gemm_params p, int groups, int group_n) {
         if (bias != nullptr) v += bias[col];
         if (C != nullptr) v += p.beta * C[static_cast<long long>(row) * p.ldc + col];
       }
-      if (!GATED && p.lin_act == NFK_LIN_TANH) v = tanhf(v);
+      if (!GATED) v = lin_act_of(v, p.lin_act);
       if (D32 != nullptr && col >= p.f32_col0) D32[static_cast<long long>(row) * p.ld32 + col - p.f32_col0] = v;
       else D[static_cast<long long>(row) * p.ldd + col] = v;
     }

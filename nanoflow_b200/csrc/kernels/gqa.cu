@@ -1,7 +1,7 @@
-// Grouped-query attention whose queries and keys are normed and not rotated (see kernels.h for the pool layout).
+// Grouped-query attention with options (see kernels.h for the pool layout).
 //
-// nfk_gqa_append   per token: RMS norm over the whole query row and the whole key row (all heads at once), keys and
-//                  values to their page slot, values optionally mixed with those of an earlier layer.
+// nfk_gqa_append   per token: RMS norm over the whole query row and the whole key row (all heads at once), rotation,
+//                  keys and values to their page slot, values optionally mixed with those of an earlier layer.
 // nfk_gqa_attn     attention for any head size, bf16 or fp32, with window, sink and capped scores: one CTA per token
 //                  and query head. 32-bit engines use it for everything, bf16 engines for heads that the tensor-core
 //                  kernels (nfk_attn_decode, nfk_attn_prefill_ws) are not built for.
@@ -19,6 +19,15 @@ __device__ __forceinline__ float ap_sum(float v, float* red) {
   if (lane == 0) red[warp] = v;
   __syncthreads();
   return warp_sum(lane < (kApThreads >> 5) ? red[lane] : 0.f);
+}
+
+// Two neighbouring pairs from column `col` of a head, turned by the token's angles.
+__device__ __forceinline__ float4 turn4(float4 x, int col, const float* table, int pairs) {
+  const int i = col >> 1;
+  if (i >= pairs) return x;
+  const float2 a = *reinterpret_cast<const float2*>(table + 2 * i);
+  const float2 b = i + 1 < pairs ? *reinterpret_cast<const float2*>(table + 2 * i + 2) : make_float2(1.f, 0.f);
+  return make_float4(x.x * a.x - x.y * a.y, x.y * a.x + x.x * a.y, x.z * b.x - x.w * b.y, x.w * b.x + x.z * b.y);
 }
 
 template <class T>
@@ -48,6 +57,8 @@ gqa_append_kernel(nfk_gqa_append_params p) {
       qi = rsqrtf(ap_sum(sq, red) / static_cast<float>(p.heads * p.dim) + p.eps);
       ki = rsqrtf(ap_sum(sk, red) / static_cast<float>(p.kv_heads * p.dim) + p.eps);
     }
+    const float* rot = p.rot != nullptr ? p.rot + static_cast<long long>(t) * p.rot_ld * 2 : nullptr;
+    const float* v_rot = p.v_rot != nullptr ? p.v_rot + static_cast<long long>(t) * p.v_ld * 2 : nullptr;
     T* qo = reinterpret_cast<T*>(p.q_out) + static_cast<long long>(t) * nq;
     for (int c = threadIdx.x * 4; c < nq; c += kApThreads * 4) {
       float4 x = load4(q + c);
@@ -55,6 +66,7 @@ gqa_append_kernel(nfk_gqa_append_params p) {
         const float4 w = load4(p.q_w + c);
         x = make_float4(x.x * qi * w.x, x.y * qi * w.y, x.z * qi * w.z, x.w * qi * w.w);
       }
+      if (rot != nullptr) x = turn4(x, c % p.hd, rot, p.rot_pairs);
       store4(qo + c, x);
     }
     T* vf = p.v_mode != 0 ? reinterpret_cast<T*>(p.v_first) + static_cast<long long>(t) * nkv : nullptr;
@@ -74,6 +86,8 @@ gqa_append_kernel(nfk_gqa_append_params p) {
       }
       if (page < 0) continue;
       const int head = c / p.hd, col = c - head * p.hd;
+      if (rot != nullptr) x = turn4(x, col, rot, p.rot_pairs);
+      if (v_rot != nullptr) y = turn4(y, col, v_rot, p.v_pairs);
       T* kp = pool + ((static_cast<long long>(page) * 2 * p.kv_heads + head) * p.page_size + pos % p.page_size) * p.hd + col;
       store4(kp, x);
       store4(kp + static_cast<long long>(p.kv_heads) * p.page_size * p.hd, y);
@@ -168,6 +182,9 @@ extern "C" int nfk_gqa_append(const nfk_gqa_append_params* p, cudaStream_t strea
     return NF_ERR_BAD_ARG;
   if (p->ld_src % 8 != 0 || p->q_off % 8 != 0 || p->k_off % 8 != 0 || p->v_off % 8 != 0) return NF_ERR_BAD_ARG;
   if ((p->q_w == nullptr) != (p->k_w == nullptr) || p->v_mode < 0 || p->v_mode > 2 || (p->v_mode != 0 && !p->v_first))
+    return NF_ERR_BAD_ARG;
+  if ((p->rot && (p->rot_pairs < 0 || p->rot_pairs > p->hd / 2 || p->rot_ld < p->rot_pairs || p->rot_ld % 2 != 0)) ||
+      (p->v_rot && (p->v_pairs < 0 || p->v_pairs > p->hd / 2 || p->v_ld < p->v_pairs || p->v_ld % 2 != 0)))
     return NF_ERR_BAD_ARG;
   int grid = 8 * device_sm_count();
   if (grid > p->T) grid = p->T;

@@ -17,7 +17,7 @@ enum { NFK_EPI_LINEAR = 0, NFK_EPI_SWIGLU = 1, NFK_EPI_REDUCE_SCATTER = 2 };
 // Gated epilogue: act(gate) * up, or for NFK_ACT_CAPPED g sigmoid(alpha g) (u + shift) with g = min(gate, limit) and
 // u = min(max(up, -limit), limit).
 enum { NFK_ACT_SILU = 0, NFK_ACT_RELU = 1, NFK_ACT_GELU_TANH = 2, NFK_ACT_CAPPED = 3 };
-enum { NFK_LIN_NONE = 0, NFK_LIN_TANH = 1 };                           // activation of the linear epilogue
+enum { NFK_LIN_NONE = 0, NFK_LIN_TANH = 1, NFK_LIN_GELU = 2 };         // activation of the linear epilogue (GELU: by erf)
 enum { NFK_BF16 = 0, NFK_F32 = 1 };                                    // storage type of activations and weights
 
 typedef struct nfk_gemm_params {
@@ -229,6 +229,8 @@ int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream);
 // ------------------------------------------------------------------------------------------------
 enum { NFK_NORM_NONE = 0, NFK_NORM_RMS = 1, NFK_NORM_LAYER = 2 };
 // x <- (table ? 0 : x) + norm_in(src_scale src) (+ y2_gate y2) (+ sum_k e_weight e_out[e_slot]) (+ add);  h = norm_out(x).
+// norm_sum: norm_in takes in y2 and the experts' rows too. pair_w: the source is half the sum of RMS norms of y (times
+// pair_w) and y2 (times pair_w2). table_add: x <- x + ... + src_scale (embedding row), which is then not a source.
 // Rows of x, y, table and h are padded to a multiple of 4 elements; weight vectors are padded with zeros to that length.
 typedef struct nfk_residual_norm_params {
   float* x;                  // [*, ld_x] residual stream
@@ -264,6 +266,10 @@ typedef struct nfk_residual_norm_params {
   const int* e_slot;         // [*][e_top] rows of e_out of a token
   const float* e_weight;     // [*][e_top]
   int e_top, e_rows;
+  int norm_sum;
+  const float* pair_w;       // [cols] padded, null: none
+  const float* pair_w2;
+  int table_add;
 } nfk_residual_norm_params;
 int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t stream);
 
@@ -384,12 +390,14 @@ typedef struct nfk_head_norm_gate_params {
 int nfk_head_norm_gate(const nfk_head_norm_gate_params* p, cudaStream_t stream);
 
 // ------------------------------------------------------------------------------------------------
-// Grouped-query attention without rotation (gqa.cu)
+// Grouped-query attention with options (gqa.cu)
 // ------------------------------------------------------------------------------------------------
 // Pool of one layer as for nfk_attn_*: [pages][2 (K, V)][kv_heads][page_size][hd]; hd is the padded size of a head's
 // keys and values (padding columns are zero).
 // Per token: RMS norm of the whole query row and of the whole key row (all heads at once), keys and values to their
 // page slot. v_mode 1 also keeps the values in v_first; 2 mixes them, v <- (1 - lambda) v + lambda v_first.
+// rot: neighbouring columns 2i, 2i + 1 (i < rot_pairs) of every query and key head turn by the token's angles, table
+// [T][rot_ld][2] of (cos, sin) as nfk_rope_table makes it; v_rot the same for the values.
 typedef struct nfk_gqa_append_params {
   const void* src;           // [T, ld_src]: q at q_off, k at k_off, v at v_off, head h at column h * hd
   long long ld_src;
@@ -411,6 +419,9 @@ typedef struct nfk_gqa_append_params {
   float eps;
   int dtype;
   unsigned int* status;
+  const float* rot;          // null: none
+  const float* v_rot;
+  int rot_pairs, rot_ld, v_pairs, v_ld;
 } nfk_gqa_append_params;
 int nfk_gqa_append(const nfk_gqa_append_params* p, cudaStream_t stream);
 
@@ -433,8 +444,133 @@ typedef struct nfk_gqa_attn_params {
 int nfk_gqa_attn(const nfk_gqa_attn_params* p, cudaStream_t stream);
 
 // ------------------------------------------------------------------------------------------------
+// Attention with mixed heads (talk.cu)
+// ------------------------------------------------------------------------------------------------
+// Softmax weights w_g(i, j) of every head (window and sink as for nfk_gqa_attn), then
+// out_h(i) = sum_j (sum_g talk[h][g] w_g(i, j)) v(j) with the values of h's own key/value head. v_rot: the output's
+// neighbouring columns turn back by the token's angles (table [T][v_ld][2] of (cos, sin), v_pairs pairs per head).
+// Pool as for nfk_gqa_append.
+typedef struct nfk_talk_attn_params {
+  const void* q;             // [T, heads * hd]
+  const void* pool;
+  void* out;                 // [T, heads * hd]
+  const int* positions;
+  const int* token_req;
+  const int* kv_indptr;
+  const int* kv_indices;
+  const int* kv_first;
+  const float* sinks;        // [heads], null: none
+  const float* talk;         // [heads][heads]
+  const float* v_rot;        // null: none
+  int v_pairs, v_ld;
+  int token_begin, n_tokens; // simple kernel
+  int heads, kv_heads, hd, page_size, num_pages, window;   // window 0: none
+  float scale;
+  int dtype;
+  unsigned int* status;
+} nfk_talk_attn_params;
+// Any sizes (shared memory for a few rows of all heads permitting), bf16 or fp32: one CTA per token.
+int nfk_talk_attn(const nfk_talk_attn_params* p, cudaStream_t stream);
+
+// ------------------------------------------------------------------------------------------------
+// Short convolution over time (short_conv.cu)
+// ------------------------------------------------------------------------------------------------
+// Per channel: y_t = act(sum_j w[j] x_(t - taps + 1 + j) (+ bias)) (+ x_t if residual), zeros before the sequence's start.
+// The last taps - 1 inputs of a request are kept in its state: half ref & 1 is read, the other one written.
+enum { NFK_CONV_NONE = 0, NFK_CONV_SILU = 1 };
+typedef struct nfk_short_conv_params {
+  const void* x;             // [T, ld_x]
+  long long ld_x;
+  void* out;                 // [T, ld_out], not x
+  long long ld_out;
+  const float* w;            // [taps][cols]
+  const float* bias;         // [cols], null: none
+  void* state;               // [slots][2][max(1, taps - 1)][cols], stored as x
+  const int* state_slot;     // [B] 2 * slot + half
+  const int* positions;
+  const int* token_req;
+  const int* qo_indptr;
+  int row_begin, T;          // rows row_begin .. T - 1 (whole requests)
+  int cols, taps, act, residual, num_slots, dtype;
+  unsigned int* status;
+} nfk_short_conv_params;
+int nfk_short_conv(const nfk_short_conv_params* p, cudaStream_t stream);
+
+// ------------------------------------------------------------------------------------------------
+// Real-gated linear recurrent unit (rglru.cu)
+// ------------------------------------------------------------------------------------------------
+// Per channel: log a = log_a sigmoid(r + r_b), S <- a S + sqrt(1 - a^2) sigmoid(i + i_b) u; out = S gelu_tanh(y).
+// Channels come in blocks of `block`: the gates' pre-activations of a block are its r columns, then its i columns.
+// A request whose first token of the launch is at position 0 starts from zero.
+typedef struct nfk_rglru_params {
+  const void* u;             // [T, ld_u]
+  long long ld_u;
+  const void* y;             // [T, ld_y]
+  long long ld_y;
+  const float* gates;        // [T, ld_g]
+  long long ld_g;
+  const float* r_b;          // [cols]
+  const float* i_b;
+  const float* log_a;
+  float* S;                  // [slots][cols]
+  void* out;                 // [T, ld_out]
+  long long ld_out;
+  const int* positions;
+  const int* qo_indptr;
+  const int* state_slot;     // [B] 2 * slot (+ half, not used here)
+  int req_begin, req_count, cols, block, num_slots;
+  int dtype;
+  unsigned int* status;
+} nfk_rglru_params;
+int nfk_rglru_decode(const nfk_rglru_params* p, cudaStream_t stream);    // one token per request
+int nfk_rglru_prefill(const nfk_rglru_params* p, cudaStream_t stream);   // any number of tokens per request
+
+// ------------------------------------------------------------------------------------------------
+// Delta-rule recurrence (delta.cu)
+// ------------------------------------------------------------------------------------------------
+// Per head, q and k of head h being those of q/k head h / (heads / kv_heads) as unit vectors (x / sqrt(sum x^2 + unit_eps)),
+// q times q_scale, with w = exp(-rate softplus(x + dt_bias)) per key channel and beta = sigmoid(b):
+//   S <- diag(w) S;  S <- S + k (beta (v - S^T k))^T;  o = S^T q
+//   y = RMS norm of o (over the head's vdim_real values) * norm * sigmoid(g)
+// A request whose first token of the launch is at position 0 starts from a zero state.
+typedef struct nfk_delta_params {
+  const void* qkv;           // [T, ld]: q at q_off + head * dim, k at k_off, v at v_off + head * vdim
+  long long ld;
+  int q_off, k_off, v_off;
+  const float* x;            // [T, ld_x], head h at column h * dim
+  long long ld_x;
+  const float* beta;         // [T, ld_b], head h at column h
+  long long ld_b;
+  const void* g;             // [T, ld_g], head h at column h * vdim
+  long long ld_g;
+  const float* rate;         // [heads]
+  const float* dt_bias;      // [heads * dim]
+  const float* norm;         // [vdim]
+  float* S;                  // [slots][heads][dim][vdim]
+  void* y;                   // [T, ld_y]
+  long long ld_y;
+  const int* positions;
+  const int* qo_indptr;
+  const int* state_slot;     // [B] 2 * slot (+ half, not used here)
+  int req_begin, req_count;  // decode: requests with one token each
+  int heads, kv_heads, dim, vdim, vdim_real, num_slots;    // dim, vdim: padded to multiples of 8 (padding columns are zero)
+  float q_scale, unit_eps, eps;
+  int dtype;
+  // prefill, token by token: seq_reqs [num_seq] requests, o: fp32 [T, heads * vdim] of scratch rows
+  const int* seq_reqs;
+  int num_seq;
+  float* o;
+  unsigned int* status;
+} nfk_delta_params;
+int nfk_delta_decode(const nfk_delta_params* p, cudaStream_t stream);
+int nfk_delta_prefill(const nfk_delta_params* p, cudaStream_t stream);
+
+// ------------------------------------------------------------------------------------------------
 // Mixture of experts (moe.cu)
 // ------------------------------------------------------------------------------------------------
+enum { NFK_SCORE_SIGMOID = 0, NFK_SCORE_SOFTMAX = 1 };
+// NFK_SCORE_SOFTMAX: the experts are chosen by logits + correction and weighted by the softmax of those sums over the
+// chosen ones, times scale (groups as below). NFK_SCORE_SIGMOID:
 // Scores s = sigmoid(logits); choice scores s + correction. Experts form `groups` equal runs of neighbours (1: no
 // grouping); a group counts by the sum of its two largest choice scores and only experts of the best `keep` groups
 // can be chosen. Weights: s of the `top` chosen ones over their sum, times scale. Ties go to the lower index.
@@ -450,6 +586,7 @@ typedef struct nfk_moe_route_params {
   float* gate;               // [T] sigmoid of the gate column
   int T, experts, top, groups, keep, gate_col;
   float scale;
+  int score;                 // NFK_SCORE_*
 } nfk_moe_route_params;
 int nfk_moe_route(const nfk_moe_route_params* p, cudaStream_t stream);
 
@@ -469,7 +606,7 @@ typedef struct nfk_moe_permute_params {
 int nfk_moe_permute(const nfk_moe_permute_params* p, cudaStream_t stream);
 
 // One product per expert over its rows of A (rows in expert order, counts per expert on the device):
-// D = A B_e^T, or with B2 the gated epilogue of nfk_gemm_bf16. Matrices of the experts are stacked: B [experts * N, ldb].
+// D = A B_e^T with lin_act, or with B2 the gated epilogue of nfk_gemm_bf16. Matrices of the experts are stacked: B [experts * N, ldb].
 typedef struct nfk_moe_gemm_params {
   const void* A;             // [rows, lda]
   const void* B;
@@ -483,6 +620,7 @@ typedef struct nfk_moe_gemm_params {
   float act_limit, act_alpha, act_shift;
   int dtype, num_ctas;
   unsigned int* status;
+  int lin_act;               // NFK_LIN_*
 } nfk_moe_gemm_params;
 int nfk_moe_gemm(const nfk_moe_gemm_params* p, cudaStream_t stream);
 

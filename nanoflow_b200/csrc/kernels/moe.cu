@@ -40,12 +40,14 @@ moe_route_kernel(nfk_moe_route_params p) {
   float* s_s = rsm + warp * (2 * E + p.groups);
   float* c_s = s_s + E;
   float* g_s = c_s + E;
+  const bool softmax = p.score == NFK_SCORE_SOFTMAX;
   for (int t = blockIdx.x * kRouteWarps + warp; t < p.T; t += gridDim.x * kRouteWarps) {
     const float* z = p.logits + t * p.ld;
     for (int e = lane; e < E; e += 32) {
-      const float s = 1.f / (1.f + expf(-z[e]));
+      const float corr = p.correction != nullptr ? p.correction[e] : 0.f;
+      const float s = softmax ? z[e] + corr : 1.f / (1.f + expf(-z[e]));
       s_s[e] = s;
-      c_s[e] = s + (p.correction != nullptr ? p.correction[e] : 0.f);
+      c_s[e] = softmax ? s : s + corr;
     }
     if (lane == 0 && p.gate_col >= 0) p.gate[t] = 1.f / (1.f + expf(-z[p.gate_col]));
     __syncwarp();
@@ -92,10 +94,18 @@ moe_route_kernel(nfk_moe_route_params p) {
       if (lane == 0) c_s[i] = -INFINITY;
       __syncwarp();
     }
+    float share = mine >= 0 ? s_s[mine] : 0.f;
+    if (softmax) {
+      const float top = __shfl_sync(0xffffffffu, share, 0);        // the first one chosen has the largest logit
+      share = mine >= 0 ? expf(share - top) : 0.f;
+      share /= warp_sum(share);
+    } else {
+      share /= sum + 1e-20f;
+    }
     if (lane < p.top) {
       const long long o = static_cast<long long>(t) * p.top + lane;
       p.expert[o] = mine;
-      p.weight[o] = s_s[mine] / (sum + 1e-20f) * p.scale;
+      p.weight[o] = share * p.scale;
       p.rank[o] = atomicAdd(p.counts + mine, 1);
     }
     __syncwarp();
@@ -353,6 +363,10 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
 #pragma unroll
           for (int j = 0; j < 32; ++j)
             v[j] = GATED ? gated_act(__uint_as_float(r[j]), __uint_as_float(u[j]), act) : __uint_as_float(r[j]);
+          if (!GATED && p.lin_act != NFK_LIN_NONE) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = lin_act_of(v[j], p.lin_act);
+          }
           if (row_ok) {
 #pragma unroll
             for (int g = 0; g < 4; ++g) {
@@ -444,7 +458,7 @@ moe_gemm_f32_kernel(nfk_moe_gemm_params p) {
       const int col = col0 + tx * 4 + j;
       if (col < p.N)
         reinterpret_cast<float*>(p.D)[static_cast<long long>(row) * p.ldd + col] =
-            GATED ? gated_act_of<true>(acc[i][j], up[i][j], act) : acc[i][j];
+            GATED ? gated_act_of<true>(acc[i][j], up[i][j], act) : lin_act_of(acc[i][j], p.lin_act);
     }
   }
 }
@@ -486,7 +500,8 @@ extern "C" int nfk_moe_route(const nfk_moe_route_params* p, cudaStream_t stream)
   if (p->T == 0) return NF_OK;
   if (!p->logits || !p->expert || !p->weight || !p->rank || !p->counts || p->T < 0 || p->experts <= 0 ||
       p->experts > kMaxExperts || p->groups <= 0 || p->experts % p->groups != 0 || p->keep <= 0 || p->keep > p->groups ||
-      p->top <= 0 || p->top > 32 || p->top > p->keep * (p->experts / p->groups) || (p->gate_col >= 0 && !p->gate))
+      p->top <= 0 || p->top > 32 || p->top > p->keep * (p->experts / p->groups) || (p->gate_col >= 0 && !p->gate) ||
+      p->score < NFK_SCORE_SIGMOID || p->score > NFK_SCORE_SOFTMAX)
     return NF_ERR_BAD_ARG;
   const size_t sm = static_cast<size_t>(kRouteWarps) * (2 * p->experts + p->groups) * 4;
   if (sm > 48 * 1024) return NF_ERR_UNSUPPORTED;
@@ -516,7 +531,7 @@ extern "C" int nfk_moe_gemm(const nfk_moe_gemm_params* p, cudaStream_t stream) {
   if (p->rows == 0) return NF_OK;
   if (!p->A || !p->B || !p->D || !p->counts || p->rows < 0 || p->experts <= 0 || p->experts > kMaxExperts || p->N <= 0 ||
       p->K <= 0 || p->N % 8 != 0 || p->K % 8 != 0 || p->lda % 8 != 0 || p->ldb % 8 != 0 || p->ldd % 8 != 0 ||
-      p->act < NFK_ACT_SILU || p->act > NFK_ACT_CAPPED || (reinterpret_cast<uintptr_t>(p->D) & 15) != 0)
+      p->act < NFK_ACT_SILU || p->act > NFK_ACT_CAPPED || p->lin_act < NFK_LIN_NONE || p->lin_act > NFK_LIN_GELU || (reinterpret_cast<uintptr_t>(p->D) & 15) != 0)
     return NF_ERR_BAD_ARG;
   if (p->dtype == NFK_F32) {
     const long long m_tiles = p->rows / kFt + (p->rows < p->experts ? p->rows : p->experts);

@@ -3,6 +3,8 @@
 //
 //   x <- (table ? 0 : x) + norm_in(src) (+ second output) (+ weighted expert outputs) (+ add);   h = norm_out(x)
 //
+// The norm can also be taken of the whole sum, the source can be the mean of two normed outputs, and the embedding row
+// can join a stream that goes on (see kernels.h).
 // `src` is the sublayer's output row, or the embedding row of the token (ids as in nfk_embedding, with the
 // previous iteration's tokens fed back on the device). Norms are RMS or layer norms with fp32 weights. The
 // stream x is fp32; src and h are bf16 or fp32. One CTA per row, the row stays in registers.
@@ -81,7 +83,7 @@ residual_norm_kernel(nfk_residual_norm_params p) {
         src_row = 0;
       }
     }
-    const T* src = nullptr;
+    const T *src = nullptr, *again = nullptr;
     if (p.table != nullptr) {
       int id = p.host_ids != nullptr ? p.host_ids[row] : 0;
       if (p.feedback_src != nullptr && p.prev_tokens != nullptr) {
@@ -92,8 +94,9 @@ residual_norm_kernel(nfk_residual_norm_params p) {
         if (threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
         id = 0;
       }
-      src = reinterpret_cast<const T*>(p.table) + static_cast<long long>(id) * p.ld_table;
-    } else if (p.y != nullptr) {
+      (p.table_add != 0 ? again : src) = reinterpret_cast<const T*>(p.table) + static_cast<long long>(id) * p.ld_table;
+    }
+    if (p.y != nullptr && (p.table == nullptr || p.table_add != 0)) {
       src = reinterpret_cast<const T*>(p.y) + static_cast<long long>(src_row) * p.ld_y;
     }
     float* xr = p.x + static_cast<long long>(src_row) * p.ld_x;
@@ -103,14 +106,28 @@ residual_norm_kernel(nfk_residual_norm_params p) {
       const int vi = threadIdx.x + i * kRnThreads;
       v[i] = (src != nullptr && vi < nvec) ? load4(src + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    if (src != nullptr && p.src_scale != 0.f) {
+    if (src != nullptr && again == nullptr && p.src_scale != 0.f) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         v[i].x *= p.src_scale; v[i].y *= p.src_scale; v[i].z *= p.src_scale; v[i].w *= p.src_scale;
       }
     }
-    if (src != nullptr) norm_row<NV>(v, p.in_kind, p.in_w, p.in_b, p.cols, nvec, p.eps, red);
-    if (p.y2 != nullptr) {
+    if (p.pair_w != nullptr) {
+      const T* y2 = reinterpret_cast<const T*>(p.y2) + static_cast<long long>(src_row) * p.ld_y2;
+      float4 o[NV];
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int vi = threadIdx.x + i * kRnThreads;
+        o[i] = vi < nvec ? load4(y2 + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+      norm_row<NV>(v, NFK_NORM_RMS, p.pair_w, nullptr, p.cols, nvec, p.eps, red);
+      norm_row<NV>(o, NFK_NORM_RMS, p.pair_w2, nullptr, p.cols, nvec, p.eps, red);
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        v[i] = make_float4(0.5f * (v[i].x + o[i].x), 0.5f * (v[i].y + o[i].y), 0.5f * (v[i].z + o[i].z), 0.5f * (v[i].w + o[i].w));
+    }
+    if (src != nullptr && p.norm_sum == 0) norm_row<NV>(v, p.in_kind, p.in_w, p.in_b, p.cols, nvec, p.eps, red);
+    if (p.y2 != nullptr && p.pair_w == nullptr) {
       const float f = p.y2_gate != nullptr ? p.y2_gate[src_row] : 1.f;
       const T* y2 = reinterpret_cast<const T*>(p.y2) + static_cast<long long>(src_row) * p.ld_y2;
 #pragma unroll
@@ -135,11 +152,19 @@ residual_norm_kernel(nfk_residual_norm_params p) {
         }
       }
     }
+    if (p.norm_sum != 0) norm_row<NV>(v, p.in_kind, p.in_w, p.in_b, p.cols, nvec, p.eps, red);
+    if (again != nullptr) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int vi = threadIdx.x + i * kRnThreads;
+        if (vi < nvec) fma4(v[i], p.src_scale != 0.f ? p.src_scale : 1.f, load4(again + vi * 4));
+      }
+    }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int vi = threadIdx.x + i * kRnThreads;
       if (vi < nvec) {
-        if (p.table == nullptr) {
+        if (p.table == nullptr || p.table_add != 0) {
           const float4 x = load4(xr + vi * 4);
           v[i].x += x.x; v[i].y += x.y; v[i].z += x.z; v[i].w += x.w;
         }
@@ -190,6 +215,8 @@ extern "C" int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t
   if (p->rows_idx && (p->in_rows <= 0 || !p->h)) return NF_ERR_BAD_ARG;
   if (p->y2 && p->ld_y2 % 4 != 0) return NF_ERR_BAD_ARG;
   if (p->e_out && (!p->e_slot || !p->e_weight || p->e_top <= 0 || p->e_rows <= 0 || p->ld_e % 4 != 0)) return NF_ERR_BAD_ARG;
+  if (p->pair_w && (!p->pair_w2 || !p->y || !p->y2)) return NF_ERR_BAD_ARG;
+  if (p->norm_sum && p->in_kind != NFK_NORM_NONE && !p->in_w) return NF_ERR_BAD_ARG;
   for (int kind : {p->in_kind, p->out_kind})
     if (kind != NFK_NORM_NONE && kind != NFK_NORM_RMS && kind != NFK_NORM_LAYER) return NF_ERR_BAD_ARG;
   if ((p->table || p->y) && p->in_kind != NFK_NORM_NONE && !p->in_w) return NF_ERR_BAD_ARG;

@@ -1,10 +1,11 @@
 """Models described as an explicit list of layers: configuration, weights in kernel layout, random weights.
 
-A layer is a mixer (one of the registered kinds below, with its own sizes) and optionally a feed-forward
-(gated, or a mixture of gated experts), one after the other or side by side on one normed input; a contiguous range of layers may run several times in a row with the same weights, each
-pass with a cache or state of its own. :class:`LayerListConfig` plays the part :class:`~..config.ModelConfig`
-plays for the Llama family; :class:`LayerListWeights` that of ``RankWeights``. Designs map their
-``config.json`` and tensor names onto these (``models/volarax.py``, ``models/zubedra.py``).
+A layer is a mixer (one of the registered kinds below, with its own sizes, or two of them side by side) and optionally
+a feed-forward (gated, or a mixture of experts), one after the other or side by side on one normed input; what a
+sublayer reads may first pass a short convolution over time. A contiguous range of layers may run several times in a row
+with the same weights, each pass with a cache or state of its own. :class:`LayerListConfig` plays the part
+:class:`~..config.ModelConfig` plays for the Llama family; :class:`LayerListWeights` that of ``RankWeights``. Designs map
+their ``config.json`` and tensor names onto these (``models/volarax.py``, ``models/zubedra.py``, ``models/gupizen.py``).
 
 Kernel layout of the weights: every matrix ``[N, K]`` with both sizes padded with zeros to multiples of 8
 (per head where a matrix is per head), projections of one input packed into one matrix, norm weights,
@@ -13,6 +14,7 @@ activations, so no kernel needs to know about them.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional, Tuple
 
@@ -22,7 +24,10 @@ PREFILL_HEAD_DIM = 128        # head size of the tcgen05 prefill attention kerne
 ATTN_HEAD_DIMS = (64, 128)    # head sizes of the tensor-core attention kernels over pages of keys and values
 ATTN_MAX_GROUP = 16           # query heads per KV head that the decode kernel takes
 WKV_CHUNK_DIM = 128           # largest head size of the chunked WKV kernels
+PAGE = 16                     # tokens per cache page
 MOE_MAX_EXPERTS, MOE_MAX_TOP = 1024, 32
+LINEAR_ACTS = ("gelu",)       # activations of products without a gate
+CONV_MAX_TAPS = 8             # taps of the short convolution kernel
 LATENT_LDS = (64, 128, 192, 256, 384, 512)   # row sizes the tensor-core latent attention kernel is built for
 
 
@@ -59,9 +64,46 @@ class LatentAttentionSpec:
 
 
 @dataclass(frozen=True)
+class RotaryScaling:
+    """Rotations with a wavelength above ``original / low`` are slowed by ``factor``, those below ``original / high`` are
+    kept, with a ramp in between (the scaling of Llama 3.1)."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on the first ``dims`` dimensions of queries and keys, neighbours 2i and 2i + 1 in a pair.
+    ``values``: the values turn with their position too (all dimensions, unscaled), and every output turns back by the
+    query's, so that it depends on distances only."""
+    dims: int
+    base: float
+    scaling: Optional[RotaryScaling] = None
+    values: bool = False
+
+    def frequencies(self, n: int, scaled: bool) -> List[float]:
+        """Radians per position of the n / 2 pairs."""
+        out, s = [], self.scaling if scaled else None
+        for i in range(n // 2):
+            f = self.base ** (-2.0 * i / n)
+            if s is not None:
+                length = 2.0 * math.pi / f
+                if length > s.original / s.low:
+                    f /= s.factor
+                elif length >= s.original / s.high:
+                    ramp = (s.original / length - s.low) / (s.high - s.low)
+                    f = (1.0 - ramp) * f / s.factor + ramp * f
+            out.append(f)
+        return out
+
+
+@dataclass(frozen=True)
 class AttentionSpec:
-    """Grouped-query attention without positions: RMS norm over whole query and key rows, optionally capped scores
-    and a sink per head. ``value_mix``: values are mixed with those of the first layer that has it set."""
+    """Grouped-query attention, with options: RMS norm over whole query and key rows, rotary positions, a sliding window,
+    capped scores, a sink per head. ``value_mix``: values are mixed with those of the first layer that has it set.
+    ``talk``: the heads' softmax weights are mixed by a matrix before they meet the values."""
     heads: int
     kv_heads: int
     dim: int
@@ -70,6 +112,10 @@ class AttentionSpec:
     softcap: Optional[float] = None
     sink: bool = True
     value_mix: bool = False
+    qk_norm: bool = True
+    rotary: Optional[RotarySpec] = None
+    window: Optional[int] = None
+    talk: bool = False
     kind = "attention"
 
     @property
@@ -80,8 +126,21 @@ class AttentionSpec:
         _positive(where, heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, scale=self.scale)
         if self.softcap is not None:
             _positive(where, softcap=self.softcap)
+        if self.window is not None:
+            _positive(where, window=self.window)
         if self.heads % self.kv_heads:
             raise ValueError(f"{where}: {self.heads} query heads do not share {self.kv_heads} key/value heads evenly")
+        if self.rotary is not None:
+            _positive(where, rotary_base=self.rotary.base)
+            if self.rotary.dims < 0 or self.rotary.dims % 2 or self.rotary.dims > self.dim:
+                raise ValueError(f"{where}: {self.rotary.dims} rotated dimensions do not fit heads of {self.dim}")
+            if self.rotary.values and self.vdim % 2:
+                raise ValueError(f"{where}: rotated values need an even size, not {self.vdim}")
+            if self.rotary.scaling is not None:
+                s = self.rotary.scaling
+                _positive(where, factor=s.factor, low=s.low, original=s.original, high_over_low=s.high - s.low)
+        if self.talk and (self.softcap is not None or self.value_mix):
+            raise ValueError(f"{where}: capped scores and mixed values are not built for mixed heads")
 
     def matrix_params(self, w: int) -> int:
         return w * (self.heads * (self.dim + self.vdim) + self.kv_heads * (self.dim + self.vdim))
@@ -124,8 +183,92 @@ class WkvSpec:
 
 
 @dataclass(frozen=True)
+class RgLruSpec:
+    """Real-gated linear recurrent unit (one number of state per channel) behind a short convolution, times a GELU branch;
+    the gates are block-diagonal projections of the convolution's output."""
+    width: int
+    blocks: int
+    conv: int
+    kind = "rglru"
+
+    @property
+    def block_p(self) -> int:
+        """Columns per block."""
+        return round8(self.width // self.blocks)
+
+    @property
+    def cols(self) -> int:
+        return self.blocks * self.block_p
+
+    def check(self, where: str) -> None:
+        _positive(where, width=self.width, blocks=self.blocks, conv=self.conv)
+        if self.width % self.blocks:
+            raise ValueError(f"{where}: a width of {self.width} does not form {self.blocks} blocks")
+        if self.conv > CONV_MAX_TAPS:
+            raise ValueError(f"{where}: at most {CONV_MAX_TAPS} taps are built, not {self.conv}")
+
+    def matrix_params(self, w: int) -> int:
+        return 3 * w * self.width + 2 * self.width * (self.width // self.blocks)
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """Delta-rule recurrence: a matrix state per head with a decay per key channel and token, from which what the key
+    recalls is replaced by the value; short convolutions on queries, keys and values. ``decay_rank``, ``gate_rank``: of
+    the low-rank projections of decays and output gates."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    decay_rank: int
+    gate_rank: int
+    kind = "delta"
+
+    @property
+    def rank_p(self) -> int:
+        return round8(max(self.decay_rank, self.gate_rank))
+
+    def check(self, where: str) -> None:
+        _positive(where, heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, conv=self.conv,
+                  decay_rank=self.decay_rank, gate_rank=self.gate_rank)
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{where}: {self.heads} heads do not share {self.kv_heads} query/key heads evenly")
+        if self.conv > CONV_MAX_TAPS:
+            raise ValueError(f"{where}: at most {CONV_MAX_TAPS} taps are built, not {self.conv}")
+
+    def matrix_params(self, w: int) -> int:
+        return w * (2 * self.kv_heads * self.dim + 2 * self.heads * self.vdim + self.heads + self.decay_rank + self.gate_rank) + \
+            self.heads * (self.decay_rank * self.dim + self.gate_rank * self.vdim)
+
+
+@dataclass(frozen=True)
+class PairSpec:
+    """An attention and a linear recurrent unit side by side on one input: half the sum of their RMS-normed outputs."""
+    left: AttentionSpec
+    right: RgLruSpec
+    kind = "pair"
+
+    def check(self, where: str) -> None:
+        if self.left.kind != "attention" or self.right.kind != "rglru":
+            raise ValueError(f"{where}: a pair of {self.left.kind} and {self.right.kind} is not built")
+        if self.left.value_mix:
+            raise ValueError(f"{where}: mixed values are not built inside a pair")
+        self.left.check(where + " (left)")
+        self.right.check(where + " (right)")
+
+    def matrix_params(self, w: int) -> int:
+        return self.left.matrix_params(w) + self.right.matrix_params(w)
+
+
+def parts_of(spec) -> Tuple[Any, ...]:
+    """The mixers a layer's mixer consists of."""
+    return (spec.left, spec.right) if spec.kind == "pair" else (spec,)
+
+
+@dataclass(frozen=True)
 class ActSpec:
-    """Activation of a gated feed-forward with its constants (those of "capped", see the GEMM epilogue)."""
+    """Activation of a feed-forward with its constants (those of "capped", see the GEMM epilogue)."""
     name: str
     limit: float = 0.0
     alpha: float = 1.0
@@ -134,24 +277,27 @@ class ActSpec:
 
 @dataclass(frozen=True)
 class MlpSpec:
+    """``gated``: act(gate) * up; else act(up)."""
     ff: int
     act: ActSpec
+    gated: bool = True
     kind = "dense"
 
     def check(self, where: str) -> None:
         _positive(where, ff=self.ff)
 
     def matrix_params(self, w: int) -> int:
-        return 3 * w * self.ff
+        return (3 if self.gated else 2) * w * self.ff
 
     active_params = matrix_params
 
 
 @dataclass(frozen=True)
 class MoeSpec:
-    """Mixture of gated experts: sigmoid scores, a correction added for the choice, experts in ``groups`` of which
-    only the best ``keep`` can be chosen, the ``top`` chosen scores normed and times ``scale``. ``shared``: an
-    expert that runs for every token, times a sigmoid gate of its own."""
+    """Mixture of experts, of which a token uses ``top``. ``score`` "sigmoid": sigmoid scores, a correction added for the
+    choice, the chosen scores normed and times ``scale``; "softmax": softmax over the chosen logits times ``scale``.
+    Experts in ``groups`` of which only the best ``keep`` can be chosen. ``shared``: an expert that runs for every token,
+    times a sigmoid gate of its own."""
     expert: MlpSpec
     experts: int
     top: int
@@ -159,6 +305,7 @@ class MoeSpec:
     groups: int = 1
     keep: int = 1
     shared: Optional[MlpSpec] = None
+    score: str = "sigmoid"
     kind = "moe"
 
     def check(self, where: str) -> None:
@@ -170,6 +317,12 @@ class MoeSpec:
             raise ValueError(f"{where}: {self.experts} experts do not form {self.groups} groups of which {self.keep} are kept")
         if self.top > self.keep * (self.experts // self.groups):
             raise ValueError(f"{where}: {self.top} experts per token cannot be chosen from {self.keep} groups")
+        if self.score not in ("sigmoid", "softmax"):
+            raise ValueError(f"{where}: unknown router score '{self.score}'")
+        if self.expert.gated == (self.expert.act.name in LINEAR_ACTS):
+            raise ValueError(f"{where}: activation '{self.expert.act.name}' is not built for this kind of expert")
+        if self.shared is not None and not self.shared.gated:
+            raise ValueError(f"{where}: a shared expert without a gate product is not built")
         if self.experts > MOE_MAX_EXPERTS or self.top > MOE_MAX_TOP:
             raise ValueError(f"{where}: at most {MOE_MAX_EXPERTS} experts and {MOE_MAX_TOP} per token are built")
 
@@ -194,7 +347,8 @@ class LayerSpec:
 
 @dataclass(frozen=True)
 class LayerRun:
-    """One execution of a layer: ``step`` is the pass whose step vector joins the stream right before it."""
+    """One execution of a layer: ``step`` is the pass whose step vector (or the embedding output, see ``loop_add``) joins
+    the stream right before it."""
     layer: int
     step: Optional[int] = None
 
@@ -212,7 +366,11 @@ class LayerListConfig:
     parallel: bool = False              # mixer and feed-forward read one normed input and join the stream together
     embed_scale: float = 1.0
     logit_scale: float = 1.0            # folded into the final norm's weight
+    input_conv: int = 0                 # taps of the convolution over time that a sublayer's input passes (0: none)
+    tied_head: bool = False             # the embedding table is the output matrix
     loop: Optional[Tuple[int, int, int]] = None      # (start, stop, times)
+    loop_add: str = "steps"             # what joins the stream ahead of a pass: a vector per pass, or "embedding": what the
+                                        # layers started from, ahead of every pass but the first
     eos_token_id: int = -1
     bos_token_id: int = -1
     dtype: torch.dtype = torch.bfloat16              # storage of weights, activations and caches
@@ -231,12 +389,20 @@ class LayerListConfig:
                 raise ValueError(f"loop {self.loop} does not fit {len(self.layers)} layers")
         if self.parallel and self.output_norms:
             raise ValueError("norms of sublayer outputs are not built for parallel layers")
+        if self.loop_add not in ("steps", "embedding"):
+            raise ValueError(f"unknown loop addition '{self.loop_add}'")
+        if self.loop_add == "embedding" and self.embed_norm and self.loop is not None:
+            raise ValueError("a normed embedding output that joins every pass of a loop is not built")
+        if not 0 <= self.input_conv <= CONV_MAX_TAPS:
+            raise ValueError(f"at most {CONV_MAX_TAPS} taps of the input convolution are built, not {self.input_conv}")
+        if self.input_conv and self.parallel:
+            raise ValueError("input convolutions are not built for parallel layers")
         for i, lay in enumerate(self.layers):
             lay.mixer.check(f"layer {i}")
+            if lay.mixer.kind == "pair" and (self.parallel or not self.output_norms or self.norm_kind != "rms"):
+                raise ValueError(f"layer {i}: mixers side by side need RMS norms of sublayer outputs")
             if lay.mlp is not None:
                 lay.mlp.check(f"layer {i}")
-                if lay.mlp.kind == "moe" and self.output_norms:
-                    raise ValueError(f"layer {i}: norms of sublayer outputs are not built for a mixture of experts")
         mixed = {(l.mixer.kv_heads, l.mixer.vdim) for l in self.layers if getattr(l.mixer, "value_mix", False)}
         if len(mixed) > 1:
             raise ValueError(f"layers that mix values need the same key/value heads and value size, not {sorted(mixed)}")
@@ -246,7 +412,8 @@ class LayerListConfig:
                 self.runs.append(LayerRun(i))
             elif i == self.loop[0]:
                 for t in range(self.loop[2]):
-                    self.runs += [LayerRun(j, t if j == i else None) for j in range(*self.loop[:2])]
+                    joins = self.loop_add == "steps" or t > 0
+                    self.runs += [LayerRun(j, t if j == i and joins else None) for j in range(*self.loop[:2])]
 
     # ---- what the scheduler, the page pool and the benchmarks ask for --------------------------------
     @property
@@ -262,8 +429,9 @@ class LayerListConfig:
 
     @property
     def head_dim(self) -> int:
-        return max([l.mixer.kv_rank for l in self.layers if l.mixer.kind == "latent_attention"] +
-                   [max(l.mixer.dim, l.mixer.vdim) for l in self.layers if l.mixer.kind == "attention"], default=0)
+        mixers = [s for l in self.layers for s in parts_of(l.mixer)]
+        return max([s.kv_rank for s in mixers if s.kind == "latent_attention"] +
+                   [max(s.dim, s.vdim) for s in mixers if s.kind == "attention"], default=0)
 
     @property
     def width_p(self) -> int:
@@ -274,7 +442,7 @@ class LayerListConfig:
         return round8(self.vocab_size)
 
     def run_specs(self, kind: str) -> List[Any]:
-        return [self.layers[r.layer].mixer for r in self.runs if self.layers[r.layer].mixer.kind == kind]
+        return [s for r in self.runs for s in parts_of(self.layers[r.layer].mixer) if s.kind == kind]
 
     def run_moes(self) -> List[MoeSpec]:
         mlps = [self.layers[r.layer].mlp for r in self.runs]
@@ -283,14 +451,14 @@ class LayerListConfig:
     @property
     def kv_window(self) -> int:
         """Positions back that any token sees at most (itself included); 0 = no bound."""
-        specs = self.run_specs("latent_attention")
-        if not specs or self.run_specs("attention") or any(s.window is None for s in specs):
+        specs = self.run_specs("latent_attention") + self.run_specs("attention")
+        if not specs or any(s.window is None for s in specs):
             return 0
         return max(s.window for s in specs)
 
     @property
     def has_state(self) -> bool:
-        return bool(self.run_specs("mlstm") or self.run_specs("wkv"))
+        return any(self.run_specs(kind) for kind in ("mlstm", "wkv", "rglru", "delta")) or self.input_conv > 1
 
     @property
     def first_value_run(self) -> int:
@@ -330,26 +498,56 @@ class LayerListConfig:
         return round8(n)
 
     def attn_on_tensor_cores(self, spec: AttentionSpec) -> bool:
-        return self.dtype == torch.bfloat16 and self.attn_hd(spec) in ATTN_HEAD_DIMS and spec.group <= ATTN_MAX_GROUP
+        return self.dtype == torch.bfloat16 and self.attn_hd(spec) in ATTN_HEAD_DIMS and spec.group <= ATTN_MAX_GROUP and \
+            spec.window is None and not spec.talk and spec.rotary is None
 
     def kv_bytes_per_token_local(self, dtype_bytes: int = 0) -> int:
         elems = sum(self.latent_ld(s) for s in self.run_specs("latent_attention")) + \
             sum(2 * s.kv_heads * self.attn_hd(s) for s in self.run_specs("attention"))
         return elems * (dtype_bytes or self.elem_bytes)
 
+    def pool_shape(self, spec) -> Optional[Tuple[int, ...]]:
+        """Shape of one page of a mixer's cache (None: it keeps none)."""
+        if spec.kind == "latent_attention":
+            return (PAGE, self.latent_ld(spec))
+        return (2, spec.kv_heads, PAGE, self.attn_hd(spec)) if spec.kind == "attention" else None
+
+    def state_shapes(self, spec) -> List[Tuple[Tuple[int, ...], torch.dtype]]:
+        """What a request keeps of a recurrent mixer, as (shape, type) without the leading slots. Small vectors come in two
+        halves, of which a step reads one and writes the other (see ``DistKVCache.state_ref``)."""
+        f32 = torch.float32
+        if spec.kind == "mlstm":
+            d, v = round8(spec.dim), round8(spec.vdim)
+            return [((spec.heads, d, v), f32), ((spec.heads, 2, d), f32), ((spec.heads, 2), f32)]
+        if spec.kind == "wkv":
+            d = round8(spec.dim)
+            return [((spec.heads, d, d), f32), ((2, self.width_p), self.dtype)]
+        if spec.kind == "rglru":
+            return [((spec.cols,), f32), ((2, max(1, spec.conv - 1), spec.cols), self.dtype)]
+        if spec.kind == "delta":
+            d, v = round8(spec.dim), round8(spec.vdim)
+            return [((spec.heads, d, v), f32),
+                    ((2, max(1, spec.conv - 1), 2 * spec.kv_heads * d + spec.heads * v), self.dtype)]
+        return []
+
+    def conv_state_shape(self) -> Tuple[int, ...]:
+        """The last inputs of a sublayer's input convolution, in two halves."""
+        return (2, max(1, self.input_conv - 1), self.width_p)
+
     def state_bytes_per_slot(self) -> int:
         n = 0
-        for s in self.run_specs("wkv"):
-            n += s.heads * round8(s.dim) ** 2 * 4 + 2 * self.width_p * self.elem_bytes
-        for s in self.run_specs("mlstm"):
-            d, v = round8(s.dim), round8(s.vdim)
-            n += s.heads * (d * v + 2 * d + 2) * 4
+        for r in self.runs:
+            lay = self.layers[r.layer]
+            for s in parts_of(lay.mixer):
+                n += sum(math.prod(shape) * (4 if dt == torch.float32 else 2) for shape, dt in self.state_shapes(s))
+            if self.input_conv:
+                n += (1 if lay.mlp is None else 2) * math.prod(self.conv_state_shape()) * self.elem_bytes
         return n
 
     def param_count(self) -> int:
         w = self.hidden_size
         return sum(l.mixer.matrix_params(w) + (l.mlp.matrix_params(w) if l.mlp is not None else 0) for l in self.layers) + \
-            2 * self.vocab_size * w
+            (1 if self.tied_head else 2) * self.vocab_size * w
 
     def matmul_flops_per_token(self) -> float:
         w = self.hidden_size
@@ -389,11 +587,12 @@ class MlstmWeights:
 @dataclass
 class AttentionWeights:
     w_in: torch.Tensor                   # queries | keys | values, per head padded
-    q_norm: torch.Tensor                 # fp32 [heads * hd]
-    k_norm: torch.Tensor                 # fp32 [kv_heads * hd]
+    q_norm: Optional[torch.Tensor]       # fp32 [heads * hd]
+    k_norm: Optional[torch.Tensor]       # fp32 [kv_heads * hd]
     w_o: torch.Tensor
     sinks: Optional[torch.Tensor]        # fp32 [heads]
     value_lambda: float
+    talk: Optional[torch.Tensor] = None  # fp32 [heads, heads]
 
 
 @dataclass
@@ -409,6 +608,41 @@ class WkvWeights:
 
 
 @dataclass
+class RgLruWeights:
+    w_in: torch.Tensor                   # GELU branch | convolved branch, [2 cols, width_p]
+    b_in: torch.Tensor                   # [2 cols]
+    conv: torch.Tensor                   # fp32 [taps, cols]
+    conv_b: torch.Tensor                 # fp32 [cols]
+    w_gates: torch.Tensor                # per block: recurrence gate | input gate, [blocks * 2 block_p, block_p]
+    r_b: torch.Tensor                    # fp32 [cols]
+    i_b: torch.Tensor                    # fp32 [cols]
+    log_a: torch.Tensor                  # fp32 [cols]: log of the decay at a recurrence gate of one
+    w_o: torch.Tensor
+
+
+@dataclass
+class DeltaWeights:
+    w_in: torch.Tensor                   # q | k | v | decay down | gate down | beta
+    conv: torch.Tensor                   # fp32 [taps, q | k | v]
+    w_decay: torch.Tensor                # [heads * dim_p, rank_p]
+    w_gate: torch.Tensor                 # [heads * vdim_p, rank_p]
+    dt_bias: torch.Tensor                # fp32 [heads * dim_p]
+    rate: torch.Tensor                   # fp32 [heads]: exp(A_log)
+    norm: torch.Tensor                   # fp32 [vdim_p]
+    w_o: torch.Tensor
+
+
+@dataclass
+class PairWeights:
+    w_in: torch.Tensor                   # input projections of both mixers
+    b_in: torch.Tensor
+    left: Any
+    right: Any
+    left_norm: torch.Tensor              # fp32 [width_p]
+    right_norm: torch.Tensor
+
+
+@dataclass
 class MlpWeights:
     w_gate: torch.Tensor
     w_up: torch.Tensor
@@ -418,8 +652,8 @@ class MlpWeights:
 @dataclass
 class MoeWeights:
     router: torch.Tensor                 # experts | gate of the shared expert, rows padded to a multiple of 8
-    correction: Optional[torch.Tensor]   # fp32 [experts]
-    w_gate: torch.Tensor                 # [experts * ff_p, width_p]
+    correction: Optional[torch.Tensor]   # fp32 [experts]: added for the choice, or to the logits of a softmax router
+    w_gate: Optional[torch.Tensor]       # [experts * ff_p, width_p], None in experts without a gate product
     w_up: torch.Tensor
     w_down: torch.Tensor                 # [experts * width_p, ff_p]
     shared: Optional[MlpWeights]
@@ -433,6 +667,8 @@ class LayerListLayer:
     mlp_in: Optional[NormWeights] = None         # not in parallel layers
     mlp_out: Optional[NormWeights] = None
     mlp: Any = None
+    conv_in: Optional[torch.Tensor] = None       # fp32 [taps, width_p]: input convolutions of the two sublayers
+    conv_mlp: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -447,11 +683,13 @@ class LayerListWeights:
     tp: int = 1
 
     def nbytes(self) -> int:
-        total, stack = 0, [self]
+        total, stack, seen = 0, [self], set()
         while stack:
             o = stack.pop()
             if isinstance(o, torch.Tensor):
-                total += o.numel() * o.element_size()
+                if o.untyped_storage().data_ptr() not in seen:       # parts of one matrix, tied tables
+                    seen.add(o.untyped_storage().data_ptr())
+                    total += o.untyped_storage().nbytes()
             elif isinstance(o, list):
                 stack += o
             elif hasattr(o, "__dataclass_fields__"):
@@ -505,15 +743,17 @@ def pack_mlstm(cfg: LayerListConfig, spec: MlstmSpec, q, k, v, g, i, f, i_b, f_b
 
 
 def pack_attention(cfg: LayerListConfig, spec: AttentionSpec, q, k, v, q_norm, k_norm, sink, o, value_lambda: float,
-                   device) -> AttentionWeights:
+                   device, talk=None) -> AttentionWeights:
     H, G, wp, hd = spec.heads, spec.kv_heads, cfg.width_p, cfg.attn_hd(spec)
     mv = lambda t: t.to(device=device, dtype=cfg.dtype).contiguous()
     f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
     w_in = torch.cat([pad_heads(q, H, spec.dim, hd), pad_heads(k, G, spec.dim, hd), pad_heads(v, G, spec.vdim, hd)])
     w_o = pad_to(o.reshape(-1, H, spec.vdim), wp, H, hd).reshape(wp, H * hd)
-    return AttentionWeights(w_in=mv(pad_to(w_in, w_in.shape[0], wp)), q_norm=f32(pad_heads(q_norm, H, spec.dim, hd)),
-                            k_norm=f32(pad_heads(k_norm, G, spec.dim, hd)), w_o=mv(w_o),
-                            sinks=None if sink is None else f32(sink), value_lambda=float(value_lambda))
+    return AttentionWeights(w_in=mv(pad_to(w_in, w_in.shape[0], wp)),
+                            q_norm=None if q_norm is None else f32(pad_heads(q_norm, H, spec.dim, hd)),
+                            k_norm=None if k_norm is None else f32(pad_heads(k_norm, G, spec.dim, hd)), w_o=mv(w_o),
+                            sinks=None if sink is None else f32(sink), value_lambda=float(value_lambda),
+                            talk=None if talk is None else f32(talk))
 
 
 def pack_wkv(cfg: LayerListConfig, spec: WkvSpec, mu, r, k, v, g, w1, w2, w0, u, norm, o, device) -> WkvWeights:
@@ -529,6 +769,53 @@ def pack_wkv(cfg: LayerListConfig, spec: WkvSpec, mu, r, k, v, g, w1, w2, w0, u,
                       u=f32(heads(u.reshape(-1))), norm=f32(heads(norm)), w_o=mv(w_o))
 
 
+def pack_conv(cfg: LayerListConfig, w, cols: int, device) -> torch.Tensor:
+    """[channels, taps] -> fp32 [taps, cols]."""
+    return pad_to(w.to(device=device, dtype=torch.float32).t(), w.shape[1], cols).contiguous()
+
+
+def pack_rglru(cfg: LayerListConfig, spec: RgLruSpec, y, y_b, x, x_b, conv, conv_b, ra, ra_b, ri, ri_b, lam, o,
+               device) -> RgLruWeights:
+    """``lam``: the recurrence decays by exp(-8 softplus(lam)) per token at a gate of one."""
+    n, b, bp, wp = spec.blocks, spec.width // spec.blocks, spec.block_p, cfg.width_p
+    mv = lambda t: t.to(device=device, dtype=cfg.dtype).contiguous()
+    f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+    ch = lambda t: pad_heads(t, n, b, bp)
+    w_in = torch.cat([ch(y), ch(x)])
+    gates = torch.cat([pad_to(ra, n, bp, bp), pad_to(ri, n, bp, bp)], dim=1).reshape(n * 2 * bp, bp)
+    w_o = pad_to(o.reshape(-1, n, b), wp, n, bp).reshape(wp, n * bp)
+    log_a = -8.0 * torch.nn.functional.softplus(lam.double())
+    return RgLruWeights(w_in=mv(pad_to(w_in, w_in.shape[0], wp)), b_in=mv(torch.cat([ch(y_b), ch(x_b)])),
+                        conv=pack_conv(cfg, ch(conv), spec.cols, device), conv_b=f32(ch(conv_b)), w_gates=mv(gates),
+                        r_b=f32(ch(ra_b.reshape(-1))), i_b=f32(ch(ri_b.reshape(-1))), log_a=f32(ch(log_a)), w_o=mv(w_o))
+
+
+def pack_delta(cfg: LayerListConfig, spec: DeltaSpec, q, k, v, q_conv, k_conv, v_conv, beta, a_log, a1, a2, dt_bias, g1, g2,
+               norm, o, device) -> DeltaWeights:
+    H, G, wp, d, vd, rp = spec.heads, spec.kv_heads, cfg.width_p, round8(spec.dim), round8(spec.vdim), spec.rank_p
+    mv = lambda t: t.to(device=device, dtype=cfg.dtype).contiguous()
+    f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+    qk, vh = (lambda t: pad_heads(t, G, spec.dim, d)), (lambda t: pad_heads(t, H, spec.vdim, vd))
+    w_in = torch.cat([qk(q), qk(k), vh(v), pad_to(a1, rp, a1.shape[1]), pad_to(g1, rp, g1.shape[1]),
+                      pad_to(beta, round8(H), beta.shape[1])])
+    conv = torch.cat([qk(q_conv), qk(k_conv), vh(v_conv)])
+    w_o = pad_to(o.reshape(-1, H, spec.vdim), wp, H, vd).reshape(wp, H * vd)
+    return DeltaWeights(w_in=mv(pad_to(w_in, w_in.shape[0], wp)), conv=pack_conv(cfg, conv, conv.shape[0], device),
+                        w_decay=mv(pad_to(pad_heads(a2, H, spec.dim, d), H * d, rp)),
+                        w_gate=mv(pad_to(vh(g2), H * vd, rp)), dt_bias=f32(pad_heads(dt_bias, H, spec.dim, d)),
+                        rate=f32(torch.exp(a_log.double())), norm=f32(pad_to(norm, vd)), w_o=mv(w_o))
+
+
+def pack_pair(cfg: LayerListConfig, spec: PairSpec, left: AttentionWeights, right: RgLruWeights, left_norm, right_norm,
+              device) -> PairWeights:
+    """One matrix for both mixers' input projections, of which theirs become parts."""
+    w_in, n = torch.cat([left.w_in, right.w_in]), left.w_in.shape[0]
+    b_in = torch.cat([torch.zeros(n, dtype=right.b_in.dtype, device=right.b_in.device), right.b_in])
+    left.w_in, right.w_in, right.b_in = w_in[:n], w_in[n:], b_in[n:]
+    f32 = lambda t: pad_to(t.to(device=device, dtype=torch.float32), cfg.width_p).contiguous()
+    return PairWeights(w_in=w_in, b_in=b_in, left=left, right=right, left_norm=f32(left_norm), right_norm=f32(right_norm))
+
+
 def pack_mlp(cfg: LayerListConfig, ff: int, gate, up, down, device) -> MlpWeights:
     fp, wp = round8(ff), cfg.width_p
     mv = lambda t: t.to(device=device, dtype=cfg.dtype).contiguous()
@@ -536,7 +823,7 @@ def pack_mlp(cfg: LayerListConfig, ff: int, gate, up, down, device) -> MlpWeight
 
 
 def pack_moe(cfg: LayerListConfig, spec: MoeSpec, router, correction, expert, shared, shared_gate, device) -> MoeWeights:
-    """``expert(e, part)``: a matrix of expert ``e`` (part "gate", "up" or "down"); ``shared``: the shared expert's three
+    """``expert(e, part)``: a matrix of expert ``e`` (part "gate" if it has one, "up" or "down"); ``shared``: the shared expert's three
     matrices, or None; ``shared_gate`` [1, width]."""
     fp, wp = round8(spec.expert.ff), cfg.width_p
 
@@ -551,7 +838,7 @@ def pack_moe(cfg: LayerListConfig, spec: MoeSpec, router, correction, expert, sh
     return MoeWeights(
         router=pad_to(torch.cat(rows), round8(spec.router_cols), wp).to(device=device, dtype=cfg.dtype).contiguous(),
         correction=None if correction is None else correction.to(device=device, dtype=torch.float32).contiguous(),
-        w_gate=stack("gate", fp, wp), w_up=stack("up", fp, wp), w_down=stack("down", wp, fp),
+        w_gate=stack("gate", fp, wp) if spec.expert.gated else None, w_up=stack("up", fp, wp), w_down=stack("down", wp, fp),
         shared=None if spec.shared is None else pack_mlp(cfg, spec.shared.ff, *shared, device))
 
 

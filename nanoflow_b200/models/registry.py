@@ -77,7 +77,13 @@ def _zubedra() -> ModelFamily:
     return _layer_list("zubedra", zubedra)
 
 
-_FAMILIES: Dict[str, Callable[[], ModelFamily]] = {"llama": _llama, "volarax": _volarax, "zubedra": _zubedra}
+def _gupizen() -> ModelFamily:
+    from . import gupizen
+    return _layer_list("gupizen", gupizen)
+
+
+_FAMILIES: Dict[str, Callable[[], ModelFamily]] = {"llama": _llama, "volarax": _volarax, "zubedra": _zubedra,
+                                                    "gupizen": _gupizen}
 _cache: Dict[str, ModelFamily] = {}
 
 

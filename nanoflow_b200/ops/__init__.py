@@ -77,7 +77,9 @@ class AttnParams(Structure):
 
 BF16, F32 = 0, 1                                        # storage type of a kernel's activations and weights
 ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "capped": 3}   # activation of the gated GEMM epilogue
-LIN_ACTS = {None: 0, "tanh": 1}                         # activation of the linear GEMM epilogue
+LIN_ACTS = {None: 0, "tanh": 1, "gelu": 2}              # activation of the linear GEMM epilogue
+CONV_ACTS = {None: 0, "silu": 1}                        # activation of the short convolution
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
 NORMS = {None: 0, "rms": 1, "layer": 2}
 
 
@@ -97,7 +99,8 @@ class ResidualNormParams(Structure):
                 ("rows_idx", c_void_p), ("in_rows", c_int), ("rows", c_int), ("cols", c_int), ("eps", c_float),
                 ("in_kind", c_int), ("out_kind", c_int), ("dtype", c_int), ("status", c_void_p), ("src_scale", c_float),
                 ("y2", c_void_p), ("ld_y2", c_longlong), ("y2_gate", c_void_p), ("e_out", c_void_p), ("ld_e", c_longlong),
-                ("e_slot", c_void_p), ("e_weight", c_void_p), ("e_top", c_int), ("e_rows", c_int)]
+                ("e_slot", c_void_p), ("e_weight", c_void_p), ("e_top", c_int), ("e_rows", c_int), ("norm_sum", c_int),
+                ("pair_w", c_void_p), ("pair_w2", c_void_p), ("table_add", c_int)]
 
 
 class LatentAppendParams(Structure):
@@ -144,7 +147,43 @@ class GqaAppendParams(Structure):
                 ("v_lambda", c_float), ("pool", c_void_p), ("positions", c_void_p), ("token_req", c_void_p),
                 ("kv_indptr", c_void_p), ("kv_indices", c_void_p), ("kv_first", c_void_p), ("T", c_int), ("heads", c_int),
                 ("kv_heads", c_int), ("hd", c_int), ("dim", c_int), ("page_size", c_int), ("num_pages", c_int),
-                ("eps", c_float), ("dtype", c_int), ("status", c_void_p)]
+                ("eps", c_float), ("dtype", c_int), ("status", c_void_p), ("rot", c_void_p), ("v_rot", c_void_p),
+                ("rot_pairs", c_int), ("rot_ld", c_int), ("v_pairs", c_int), ("v_ld", c_int)]
+
+
+class TalkAttnParams(Structure):
+    _fields_ = [("q", c_void_p), ("pool", c_void_p), ("out", c_void_p), ("positions", c_void_p), ("token_req", c_void_p),
+                ("kv_indptr", c_void_p), ("kv_indices", c_void_p), ("kv_first", c_void_p), ("sinks", c_void_p),
+                ("talk", c_void_p), ("v_rot", c_void_p), ("v_pairs", c_int), ("v_ld", c_int), ("token_begin", c_int),
+                ("n_tokens", c_int), ("heads", c_int), ("kv_heads", c_int), ("hd", c_int), ("page_size", c_int),
+                ("num_pages", c_int), ("window", c_int), ("scale", c_float), ("dtype", c_int), ("status", c_void_p)]
+
+
+class ShortConvParams(Structure):
+    _fields_ = [("x", c_void_p), ("ld_x", c_longlong), ("out", c_void_p), ("ld_out", c_longlong), ("w", c_void_p),
+                ("bias", c_void_p), ("state", c_void_p), ("state_slot", c_void_p), ("positions", c_void_p),
+                ("token_req", c_void_p), ("qo_indptr", c_void_p), ("row_begin", c_int), ("T", c_int), ("cols", c_int),
+                ("taps", c_int), ("act", c_int), ("residual", c_int), ("num_slots", c_int), ("dtype", c_int),
+                ("status", c_void_p)]
+
+
+class RgLruParams(Structure):
+    _fields_ = [("u", c_void_p), ("ld_u", c_longlong), ("y", c_void_p), ("ld_y", c_longlong), ("gates", c_void_p),
+                ("ld_g", c_longlong), ("r_b", c_void_p), ("i_b", c_void_p), ("log_a", c_void_p), ("S", c_void_p),
+                ("out", c_void_p), ("ld_out", c_longlong), ("positions", c_void_p), ("qo_indptr", c_void_p),
+                ("state_slot", c_void_p), ("req_begin", c_int), ("req_count", c_int), ("cols", c_int), ("block", c_int),
+                ("num_slots", c_int), ("dtype", c_int), ("status", c_void_p)]
+
+
+class DeltaParams(Structure):
+    _fields_ = [("qkv", c_void_p), ("ld", c_longlong), ("q_off", c_int), ("k_off", c_int), ("v_off", c_int), ("x", c_void_p),
+                ("ld_x", c_longlong), ("beta", c_void_p), ("ld_b", c_longlong), ("g", c_void_p), ("ld_g", c_longlong),
+                ("rate", c_void_p), ("dt_bias", c_void_p), ("norm", c_void_p), ("S", c_void_p), ("y", c_void_p),
+                ("ld_y", c_longlong), ("positions", c_void_p), ("qo_indptr", c_void_p), ("state_slot", c_void_p),
+                ("req_begin", c_int), ("req_count", c_int), ("heads", c_int), ("kv_heads", c_int), ("dim", c_int),
+                ("vdim", c_int), ("vdim_real", c_int), ("num_slots", c_int), ("q_scale", c_float), ("unit_eps", c_float),
+                ("eps", c_float), ("dtype", c_int), ("seq_reqs", c_void_p), ("num_seq", c_int), ("o", c_void_p),
+                ("status", c_void_p)]
 
 
 class GqaAttnParams(Structure):
@@ -159,7 +198,7 @@ class MoeRouteParams(Structure):
     _fields_ = [("logits", c_void_p), ("ld", c_longlong), ("correction", c_void_p), ("expert", c_void_p),
                 ("weight", c_void_p), ("rank", c_void_p), ("counts", c_void_p), ("gate", c_void_p), ("T", c_int),
                 ("experts", c_int), ("top", c_int), ("groups", c_int), ("keep", c_int), ("gate_col", c_int),
-                ("scale", c_float)]
+                ("scale", c_float), ("score", c_int)]
 
 
 class MoePermuteParams(Structure):
@@ -172,7 +211,7 @@ class MoeGemmParams(Structure):
     _fields_ = [("A", c_void_p), ("B", c_void_p), ("B2", c_void_p), ("D", c_void_p), ("counts", c_void_p),
                 ("lda", c_longlong), ("ldb", c_longlong), ("ldd", c_longlong), ("rows", c_int), ("experts", c_int),
                 ("N", c_int), ("K", c_int), ("act", c_int), ("act_limit", c_float), ("act_alpha", c_float),
-                ("act_shift", c_float), ("dtype", c_int), ("num_ctas", c_int), ("status", c_void_p)]
+                ("act_shift", c_float), ("dtype", c_int), ("num_ctas", c_int), ("status", c_void_p), ("lin_act", c_int)]
 
 
 class TokenShiftParams(Structure):

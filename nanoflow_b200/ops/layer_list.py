@@ -11,9 +11,9 @@ from typing import Optional
 
 import torch
 
-from . import (ACTS, LIN_ACTS, NORMS, AttnParams, GemmParams, GqaAppendParams, GqaAttnParams, HeadNormGateParams,
+from . import (ACTS, CONV_ACTS, LIN_ACTS, NORMS, ROUTER_SCORES, AttnParams, DeltaParams, GemmParams, GqaAppendParams, GqaAttnParams, HeadNormGateParams,
                LatentAppendParams, LatentAttnParams, LatentGatherParams, MlstmParams, MoeGemmParams, MoePermuteParams,
-               MoeRouteParams, ResidualNormParams, TokenShiftParams, WkvParams, _check, _i32, _p, _stream, dtype_code, lib)
+               MoeRouteParams, ResidualNormParams, RgLruParams, ShortConvParams, TalkAttnParams, TokenShiftParams, WkvParams, _check, _i32, _p, _stream, dtype_code, lib)
 
 
 def _f32(t: Optional[torch.Tensor], name: str) -> None:
@@ -53,10 +53,17 @@ def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
 
 def residual_norm(x: torch.Tensor, *, y=None, table=None, ids=None, feedback_src=None, prev_tokens=None, norm_in=None,
                   add=None, h=None, norm_out=None, rows_idx=None, src_scale: float = 1.0, y2=None, y2_gate=None, experts=None,
-                  cols: int, eps: float, rows: Optional[int] = None, status=None) -> None:
+                  cols: int, eps: float, rows: Optional[int] = None, norm_sum: bool = False, pair=None, table_add: bool = False,
+                  status=None) -> None:
     """x <- (table ? 0 : x) + norm_in(src_scale * (y or table[ids])) (+ y2_gate y2) (+ weighted rows of ``experts``:
-    outputs, slots, weights) (+ add); h <- norm_out(x). Norms: (kind, weight, bias)."""
+    outputs, slots, weights) (+ add); h <- norm_out(x). Norms: (kind, weight, bias). ``norm_sum``: norm_in of the whole
+    sum; ``pair``: two RMS weights, the source is the mean of the normed y and y2; ``table_add``: the embedding row joins
+    the stream instead of being the source."""
     p = ResidualNormParams()
+    p.norm_sum, p.table_add = int(norm_sum), int(table_add)
+    if pair is not None:
+        _f32(pair[0], "pair"); _f32(pair[1], "pair")
+        p.pair_w, p.pair_w2 = _p(pair[0]), _p(pair[1])
     _f32(x, "x")
     p.x, p.ld_x = _p(x), x.stride(0)
     typed = next(t for t in (y, table, h, y2) if t is not None)
@@ -194,10 +201,12 @@ def head_norm_gate(o, g, w, out, *, heads: int, vdim: int, eps: float) -> None:
 
 
 def gqa_append(src, q_out, pool, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, heads: int, dim: int,
-               q_w=None, k_w=None, v_first=None, v_mode: int = 0, v_lambda: float = 0.0, eps: float, status=None) -> None:
+               q_w=None, k_w=None, v_first=None, v_mode: int = 0, v_lambda: float = 0.0, eps: float, rot=None, v_rot=None,
+               status=None) -> None:
     """src rows are q | k | v (heads padded to the pool's head size); normed keys and the values go to ``pool`` [pages, 2,
-    kv_heads, page size, head size], normed queries to ``q_out``."""
-    for t, nm in ((q_w, "q_w"), (k_w, "k_w")):
+    kv_heads, page size, head size], normed queries to ``q_out``. ``rot``, ``v_rot``: (table of angles [T, n, 2], pairs per
+    head) for queries and keys, and for values."""
+    for t, nm in ((q_w, "q_w"), (k_w, "k_w"), (rot and rot[0], "rot"), (v_rot and v_rot[0], "v_rot")):
         _f32(t, nm)
     n, _, G, ps, hd = pool.shape
     p = GqaAppendParams(src=_p(src), ld_src=src.stride(0), q_off=0, k_off=heads * hd, v_off=(heads + G) * hd, q_out=_p(q_out),
@@ -205,6 +214,10 @@ def gqa_append(src, q_out, pool, positions, token_req, kv_indptr, kv_indices, kv
                         positions=_p(positions), token_req=_p(token_req), kv_indptr=_p(kv_indptr), kv_indices=_p(kv_indices),
                         kv_first=_p(kv_first), T=src.shape[0], heads=heads, kv_heads=G, hd=hd, dim=dim, page_size=ps,
                         num_pages=n, eps=eps, dtype=dtype_code(pool.dtype), status=_p(status))
+    if rot is not None:
+        p.rot, p.rot_ld, p.rot_pairs = _p(rot[0]), rot[0].shape[1], rot[1]
+    if v_rot is not None:
+        p.v_rot, p.v_ld, p.v_pairs = _p(v_rot[0]), v_rot[0].shape[1], v_rot[1]
     _check(lib().nfk_gqa_append(byref(p), _stream()), "nfk_gqa_append")
 
 
@@ -242,8 +255,75 @@ def paged_attention(q, pool, out, qo_indptr, kv_indptr, kv_indices, kv_last_page
     _check(lib().nfk_attn_decode(byref(p), _stream()), "nfk_attn_decode")
 
 
+def talk_attention(q, pool, out, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, heads: int, scale: float, talk,
+                   window: int = 0, sinks=None, v_rot=None, token_begin: int = 0, n_tokens: Optional[int] = None,
+                   status=None) -> None:
+    """Attention whose heads' weights are mixed by ``talk`` [heads, heads]; any head size, bf16 or fp32; q, out [T, heads *
+    head size]. ``v_rot``: (table of angles [T, n, 2], pairs per head) by which outputs turn back."""
+    _f32(sinks, "sinks"); _f32(talk, "talk")
+    n, _, G, ps, hd = pool.shape
+    p = TalkAttnParams(q=_p(q), pool=_p(pool), out=_p(out), positions=_p(positions), token_req=_p(token_req),
+                       kv_indptr=_p(kv_indptr), kv_indices=_p(kv_indices), kv_first=_p(kv_first), sinks=_p(sinks),
+                       talk=_p(talk), token_begin=token_begin, n_tokens=q.shape[0] - token_begin if n_tokens is None else n_tokens,
+                       heads=heads, kv_heads=G, hd=hd, page_size=ps, num_pages=n, window=window, scale=scale,
+                       dtype=dtype_code(pool.dtype), status=_p(status))
+    if v_rot is not None:
+        _f32(v_rot[0], "v_rot")
+        p.v_rot, p.v_ld, p.v_pairs = _p(v_rot[0]), v_rot[0].shape[1], v_rot[1]
+    _check(lib().nfk_talk_attn(byref(p), _stream()), "nfk_talk_attn")
+
+
+def short_conv(x, w, state, state_ref, positions, token_req, qo_indptr, *, bias=None, act: Optional[str] = None,
+               residual: bool = False, row_begin: int = 0, status=None) -> torch.Tensor:
+    """x [T, cols], w [taps, cols]; ``state`` [slots, 2, max(1, taps - 1), cols] in place (one half is read, the other
+    written)."""
+    _f32(w, "w"); _f32(bias, "bias")
+    out = torch.zeros(x.shape[0], w.shape[1], dtype=x.dtype, device=x.device)
+    p = ShortConvParams(x=_p(x), ld_x=x.stride(0), out=_p(out), ld_out=out.stride(0), w=_p(w), bias=_p(bias), state=_p(state),
+                        state_slot=_p(state_ref), positions=_p(positions), token_req=_p(token_req), qo_indptr=_p(qo_indptr),
+                        row_begin=row_begin, T=x.shape[0], cols=w.shape[1], taps=w.shape[0], act=CONV_ACTS[act],
+                        residual=int(residual), num_slots=state.shape[0], dtype=dtype_code(x.dtype), status=_p(status))
+    _check(lib().nfk_short_conv(byref(p), _stream()), "nfk_short_conv")
+    return out
+
+
+def rglru(u, y, gates, r_b, i_b, log_a, state, out, positions, qo_indptr, state_ref, *, block: int, req_begin: int = 0,
+          req_count: Optional[int] = None, decode: bool = False, status=None) -> None:
+    """u, y, out [T, cols], gates [T, 2 cols] (per block of channels: recurrence gates, input gates), ``state`` [slots, cols] in
+    place. ``decode``: every request has one token."""
+    for t, nm in ((gates, "gates"), (r_b, "r_b"), (i_b, "i_b"), (log_a, "log_a"), (state, "state")):
+        _f32(t, nm)
+    p = RgLruParams(u=_p(u), ld_u=u.stride(0), y=_p(y), ld_y=y.stride(0), gates=_p(gates), ld_g=gates.stride(0), r_b=_p(r_b),
+                    i_b=_p(i_b), log_a=_p(log_a), S=_p(state), out=_p(out), ld_out=out.stride(0), positions=_p(positions),
+                    qo_indptr=_p(qo_indptr), state_slot=_p(state_ref), req_begin=req_begin,
+                    req_count=qo_indptr.numel() - 1 - req_begin if req_count is None else req_count, cols=state.shape[1],
+                    block=block, num_slots=state.shape[0], dtype=dtype_code(u.dtype), status=_p(status))
+    name = "nfk_rglru_decode" if decode else "nfk_rglru_prefill"
+    _check(getattr(lib(), name)(byref(p), _stream()), name)
+
+
+def delta(qkv, x, beta, g, rate, dt_bias, norm, state, y, positions, qo_indptr, state_ref, *, kv_heads: int, vdim_real: int,
+          q_scale: float, eps: float, unit_eps: float = 1e-6, decode: int = 0, seq=None, status=None) -> None:
+    """qkv rows are q | k (kv_heads each) | v, x [T, heads * dim], beta [T, >= heads], g [T, heads * vdim]; ``state`` [slots,
+    heads, dim, vdim] in place. ``decode``: the first so many requests have one token each; else the requests ``seq`` token
+    by token."""
+    for t, nm in ((x, "x"), (beta, "beta"), (rate, "rate"), (dt_bias, "dt_bias"), (norm, "norm"), (state, "state")):
+        _f32(t, nm)
+    slots, heads, dim, vdim = state.shape
+    o = torch.zeros(qkv.shape[0], heads * vdim, device=qkv.device)
+    p = DeltaParams(qkv=_p(qkv), ld=qkv.stride(0), q_off=0, k_off=kv_heads * dim, v_off=2 * kv_heads * dim, x=_p(x),
+                    ld_x=x.stride(0), beta=_p(beta), ld_b=beta.stride(0), g=_p(g), ld_g=g.stride(0), rate=_p(rate),
+                    dt_bias=_p(dt_bias), norm=_p(norm), S=_p(state), y=_p(y), ld_y=y.stride(0), positions=_p(positions),
+                    qo_indptr=_p(qo_indptr), state_slot=_p(state_ref), req_begin=0, req_count=decode, heads=heads,
+                    kv_heads=kv_heads, dim=dim, vdim=vdim, vdim_real=vdim_real, num_slots=slots, q_scale=q_scale,
+                    unit_eps=unit_eps, eps=eps, dtype=dtype_code(qkv.dtype), seq_reqs=_p(seq),
+                    num_seq=0 if seq is None else seq.numel(), o=_p(o), status=_p(status))
+    name = "nfk_delta_decode" if decode else "nfk_delta_prefill"
+    _check(getattr(lib(), name)(byref(p), _stream()), name)
+
+
 def moe_route(logits, correction, counts, *, top: int, experts: int, groups: int = 1, keep: int = 1, scale: float,
-              gate_col: int = -1):
+              gate_col: int = -1, score: str = "sigmoid"):
     """(experts [T, top], weights, ranks, gate [T]); ``counts`` [experts] is increased."""
     _f32(logits, "logits"); _f32(correction, "correction"); _i32(counts, "counts")
     T, dev = logits.shape[0], logits.device
@@ -251,7 +331,7 @@ def moe_route(logits, correction, counts, *, top: int, experts: int, groups: int
     weight, gate = torch.zeros(T, top, device=dev), torch.zeros(T, device=dev)
     p = MoeRouteParams(logits=_p(logits), ld=logits.stride(0), correction=_p(correction), expert=_p(idx), weight=_p(weight),
                        rank=_p(rank), counts=_p(counts), gate=_p(gate), T=T, experts=experts, top=top, groups=groups, keep=keep,
-                       gate_col=gate_col, scale=scale)
+                       gate_col=gate_col, scale=scale, score=ROUTER_SCORES[score])
     _check(lib().nfk_moe_route(byref(p), _stream()), "nfk_moe_route")
     return idx, weight, rank, gate
 
@@ -269,15 +349,17 @@ def moe_permute(h, expert, rank, counts):
 
 
 def moe_gemm(a, w, counts, *, up=None, act: str = "silu", limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0,
-             status=None) -> torch.Tensor:
-    """Rows of ``a`` in expert order times their expert's matrix; w (and up) [experts * N, K]."""
+             lin_act: Optional[str] = None, status=None) -> torch.Tensor:
+    """Rows of ``a`` in expert order times their expert's matrix; w (and up) [experts * N, K]. ``lin_act``: activation
+    without ``up``."""
     _i32(counts, "counts")
     E = counts.numel()
     n = w.shape[0] // E
     out = torch.zeros(a.shape[0], n, dtype=a.dtype, device=a.device)
     p = MoeGemmParams(A=_p(a), B=_p(w), B2=_p(up), D=_p(out), counts=_p(counts), lda=a.stride(0), ldb=w.stride(0),
                       ldd=out.stride(0), rows=a.shape[0], experts=E, N=n, K=w.shape[1], act=ACTS[act], act_limit=limit,
-                      act_alpha=alpha, act_shift=shift, dtype=dtype_code(a.dtype), num_ctas=0, status=_p(status))
+                      act_alpha=alpha, act_shift=shift, dtype=dtype_code(a.dtype), num_ctas=0, status=_p(status),
+                      lin_act=LIN_ACTS[lin_act])
     _check(lib().nfk_moe_gemm(byref(p), _stream()), "nfk_moe_gemm")
     return out
 

@@ -214,6 +214,86 @@ def head_norm_gate(o, g, w, vdim, eps):
     return o.float() * inv * w.float() * torch.sigmoid(g.float())
 
 
+def turn_pairs(x, positions, freqs, sign=1.0):
+    """x [T, heads, n]: neighbouring columns 2i, 2i + 1 turn by sign * position * freqs[i]."""
+    n = len(freqs)
+    a = sign * torch.as_tensor(positions, dtype=torch.float32)[:, None] * torch.tensor(freqs, dtype=torch.float32)
+    c, s = torch.cos(a)[:, None], torch.sin(a)[:, None]
+    u, v, out = x[..., 0:2 * n:2], x[..., 1:2 * n:2], x.clone()
+    out[..., 0:2 * n:2], out[..., 1:2 * n:2] = u * c - v * s, v * c + u * s
+    return out
+
+
+def talk_attention(q, pool, positions, token_req, kv_indptr, kv_indices, kv_first, *, scale, talk, window=0, sinks=None):
+    """q [T, H, hd] -> [T, H, hd]: the heads' softmax weights (exp(sink) in the denominator) are mixed by talk [H, H] before
+    they meet the values."""
+    T, H, hd = q.shape
+    G, ps = pool.shape[2], pool.shape[3]
+    out = torch.zeros(T, H, hd)
+    for t in range(T):
+        pos = int(positions[t])
+        keys = torch.arange(max(0, pos - window + 1) if window else 0, pos + 1)
+        rows = _pool_rows(keys, int(token_req[t]), kv_indptr, kv_indices, kv_first, ps)
+        k, v = (pool[rows // ps, j, :, rows % ps].float() for j in (0, 1))          # [n, G, hd]
+        s = torch.einsum("gmd,ngd->gmn", q[t].float().reshape(G, H // G, hd), k).reshape(H, -1) * scale
+        if sinks is not None:
+            s = torch.cat([s, sinks.float()[:, None]], dim=1)
+        p = (talk.float() @ torch.softmax(s, dim=-1)[:, :keys.numel()]).reshape(G, H // G, -1)
+        out[t] = torch.einsum("gmn,ngd->gmd", p, v).reshape(H, hd)
+    return out
+
+
+def short_conv(x, w, state, positions, qo_indptr, state_ref, bias=None, act=None, residual=False):
+    """x [T, C], w [taps, C], ``state`` [slots, 2, max(1, taps - 1), C] holds each request's last inputs (half ``ref & 1`` is
+    read, the other written)."""
+    H, out = w.shape[0] - 1, torch.zeros_like(x, dtype=torch.float32)
+    for b in range(len(qo_indptr) - 1):
+        t0, t1, ref = int(qo_indptr[b]), int(qo_indptr[b + 1]), int(state_ref[b])
+        before = state[ref >> 1, ref & 1, :H].float() if int(positions[t0]) else torch.zeros(H, x.shape[1])
+        xs = torch.cat([before, x[t0:t1].float()])
+        y = sum(w[j].float() * xs[j:j + t1 - t0] for j in range(H + 1))
+        y = y if bias is None else y + bias
+        y = torch.nn.functional.silu(y) if act == "silu" else y
+        out[t0:t1] = y + x[t0:t1] if residual else y
+        if H:
+            state[ref >> 1, (ref & 1) ^ 1, :H] = xs[xs.shape[0] - H:].to(state.dtype)
+    return out
+
+
+def rglru(u, y, r, i, log_a, state, positions, qo_indptr, state_ref):
+    """u, y (before the GELU), gate pre-activations r, i (biases included) [T, C], state [slots, C], updated in place."""
+    la = log_a * torch.sigmoid(r)
+    a, x = torch.exp(la), torch.sqrt(-torch.expm1(2.0 * la)) * torch.sigmoid(i) * u
+    out = torch.zeros_like(x)
+    for b in range(len(qo_indptr) - 1):
+        t0, t1, slot = int(qo_indptr[b]), int(qo_indptr[b + 1]), int(state_ref[b]) >> 1
+        S = state[slot].clone() if int(positions[t0]) else torch.zeros_like(state[slot])
+        for t in range(t0, t1):
+            S = a[t] * S + x[t]
+            out[t] = S
+        state[slot] = S
+    return out * torch.nn.functional.gelu(y, approximate="tanh")
+
+
+def delta(q, k, v, x, rate, beta, state, positions, qo_indptr, state_ref, *, q_scale, eps):
+    """q, k [T, G, d], v [T, H, dv], x [T, H, d] (decay pre-activation, bias included), rate [H], beta [T, H]
+    (pre-activation), state [slots, H, d, dv], updated in place."""
+    H = v.shape[1]
+    unit = lambda t: (t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + eps)).repeat_interleave(H // t.shape[1], dim=1)
+    q, k, out = unit(q.float()) * q_scale, unit(k.float()), torch.zeros(v.shape)
+    w, beta = torch.exp(-rate[:, None] * torch.nn.functional.softplus(x.float())), torch.sigmoid(beta.float())
+    for b in range(len(qo_indptr) - 1):
+        t0, t1, slot = int(qo_indptr[b]), int(qo_indptr[b + 1]), int(state_ref[b]) >> 1
+        S = state[slot].clone() if int(positions[t0]) else torch.zeros_like(state[slot])
+        for t in range(t0, t1):
+            S = w[t][:, :, None] * S
+            u = beta[t][:, None] * (v[t].float() - torch.einsum("hdv,hd->hv", S, k[t]))
+            S = S + k[t][:, :, None] * u[:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        state[slot] = S
+    return out
+
+
 def gqa_append(q, k, v, q_w, k_w, pool, positions, token_req, kv_indptr, kv_indices, kv_first, *, heads, kv_heads, dim, eps):
     """q [T, heads * hd], k, v [T, kv_heads * hd] (padding columns zero), norm weights or None: keys and values go to their
     page slots of pool [pages, 2, kv_heads, page_size, hd] (in place). Returns the normed queries."""
@@ -281,15 +361,19 @@ def head_norm_silu(o, g, w, dim, eps):
     return o.float() * inv * w.float() * torch.nn.functional.silu(g.float())
 
 
-def moe_route(logits, correction, top, groups, keep, scale):
-    """(experts [T, top], weights [T, top]) from router logits [T, E]."""
-    s = torch.sigmoid(logits.float())
+def moe_route(logits, correction, top, groups, keep, scale, score="sigmoid"):
+    """(experts [T, top], weights [T, top]) from router logits [T, E]. ``score`` "softmax": of the chosen logits, the
+    correction included."""
+    s = torch.sigmoid(logits.float()) if score == "sigmoid" else logits.float()
     choice = s if correction is None else s + correction
+    z = choice
     if groups > 1:
         c = choice.reshape(len(s), groups, -1)
         best = c.topk(min(2, c.shape[-1]), dim=-1).values.sum(-1).topk(keep, dim=-1).indices
         allowed = torch.zeros(len(s), groups, dtype=torch.bool).scatter_(1, best, True)
         choice = c.masked_fill(~allowed[:, :, None], float("-inf")).reshape(len(s), -1)
     idx = choice.topk(top, dim=-1).indices
+    if score == "softmax":
+        return idx, torch.softmax(z.gather(1, idx), dim=-1) * scale
     w = s.gather(1, idx)
     return idx, w / (w.sum(-1, keepdim=True) + 1e-20) * scale

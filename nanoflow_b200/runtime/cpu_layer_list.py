@@ -13,10 +13,10 @@ import numpy as np
 import torch
 
 from ..config import NanoflowConfig
-from ..models.layer_list import LayerListConfig, LayerListWeights, round8
+from ..models.layer_list import LayerListConfig, LayerListWeights, parts_of, round8
 from ..ops import reference as ref
 from ..serving.scheduler import BatchPlan
-from .layer_list import PAGE
+from .layer_list import DELTA_UNIT_EPS, rotations
 
 
 class CpuLayerListEngine:
@@ -28,16 +28,14 @@ class CpuLayerListEngine:
         self.w, self.num_pages = weights, num_pages
         m = self.model
         self.num_slots = (self.eng.state_slots or self.eng.max_batch_size) if m.has_state else 0
-        self.pools, self.state = [], []
+        self.pools, self.state, self.conv_state = [], [], []
         n = self.num_slots
         for r in m.runs:
-            s = m.layers[r.layer].mixer
-            d, v = round8(s.dim), round8(s.vdim)
-            self.pools.append(torch.zeros(num_pages, PAGE, m.latent_ld(s)) if s.kind == "latent_attention" else
-                              torch.zeros(num_pages, 2, s.kv_heads, PAGE, m.attn_hd(s)) if s.kind == "attention" else None)
-            self.state.append((torch.zeros(n, s.heads, d, v), torch.zeros(n, s.heads, 2, d), torch.zeros(n, s.heads, 2))
-                              if s.kind == "mlstm" else
-                              (torch.zeros(n, s.heads, d, d), torch.zeros(n, 2, m.width_p)) if s.kind == "wkv" else None)
+            parts = parts_of(m.layers[r.layer].mixer)
+            shapes = [m.pool_shape(s) for s in parts if m.pool_shape(s) is not None]
+            self.pools.append(torch.zeros(num_pages, *shapes[0]) if shapes else None)
+            self.state.append(tuple(torch.zeros(n, *shape) for s in parts for shape, _ in m.state_shapes(s)))
+            self.conv_state.append([torch.zeros(n, *m.conv_state_shape()) for _ in range(2)] if m.input_conv else None)
         self.v_first: Optional[torch.Tensor] = None
         self.sampled = torch.zeros(self.eng.max_sample_rows or self.eng.max_batch_size, dtype=torch.int32)
         self._staged: Optional[BatchPlan] = None
@@ -51,6 +49,10 @@ class CpuLayerListEngine:
         y = ref.layernorm(x, n.w[:m.hidden_size], None if n.b is None else n.b[:m.hidden_size], m.norm_eps) if m.norm_kind == "layer" else \
             ref.rmsnorm(x, n.w[:m.hidden_size], m.norm_eps)
         return torch.nn.functional.pad(y, (0, m.width_p - m.hidden_size))
+
+    def _input_conv(self, r, sublayer, h, w, plan):
+        return h if w is None else ref.short_conv(h, w, self.conv_state[r][sublayer], plan.positions, plan.qo_indptr,
+                                                  plan.state_ref, residual=True)
 
     def _latent_attention(self, r, s, lw, h, plan):
         m = self.model
@@ -83,10 +85,19 @@ class CpuLayerListEngine:
         elif s.value_mix:
             v = (1.0 - lw.value_lambda) * v + lw.value_lambda * self.v_first
         pages = (plan.positions, plan.token_req, plan.kv_indptr, plan.kv_indices, plan.kv_first)
+        turns = rotations(s)
+        turn = lambda x, n, i, sign=1.0: x if len(turns) <= i else \
+            ref.turn_pairs(x.reshape(T, n, hd), plan.positions, turns[i], sign).reshape(T, -1)
+        q, k, v = turn(q, H, 0), turn(k, G, 0), turn(v, G, 1)
         q = ref.gqa_append(q, k, v, lw.q_norm, lw.k_norm, self.pools[r], *pages, heads=H, kv_heads=G, dim=s.dim,
                            eps=m.norm_eps)
-        o = ref.gqa_attention(q.reshape(T, H, hd), self.pools[r], *pages, scale=s.scale, softcap=s.softcap or 0.0,
-                              sinks=lw.sinks)
+        if s.talk:
+            o = ref.talk_attention(q.reshape(T, H, hd), self.pools[r], *pages, scale=s.scale, talk=lw.talk, window=s.window or 0,
+                                   sinks=lw.sinks)
+        else:
+            o = ref.gqa_attention(q.reshape(T, H, hd), self.pools[r], *pages, scale=s.scale, softcap=s.softcap or 0.0,
+                                  window=s.window or 0, sinks=lw.sinks)
+        o = turn(o, H, 1, -1.0)
         return o.reshape(T, -1) @ lw.w_o.t()
 
     def _wkv(self, r, s, lw, h, plan):
@@ -99,6 +110,35 @@ class CpuLayerListEngine:
                     plan.state_ref)
         return ref.head_norm_silu(o, proj[3], lw.norm.reshape(H, d), s.dim, m.norm_eps).reshape(T, -1) @ lw.w_o.t()
 
+    def _rglru(self, r, s, lw, h, plan):
+        T, n, bp = h.shape[0], s.cols, s.block_p
+        S, before = self.state[r]
+        step = (plan.positions, plan.qo_indptr, plan.state_ref)
+        y, x = (h @ lw.w_in.t() + lw.b_in).split([n, n], dim=1)
+        u = ref.short_conv(x, lw.conv, before, *step, bias=lw.conv_b)
+        gates = torch.einsum("tbk,bok->tbo", u.reshape(T, s.blocks, bp), lw.w_gates.reshape(s.blocks, 2 * bp, bp))
+        o = ref.rglru(u, y, gates[:, :, :bp].reshape(T, n) + lw.r_b, gates[:, :, bp:].reshape(T, n) + lw.i_b, lw.log_a, S, *step)
+        return o @ lw.w_o.t()
+
+    def _pair(self, r, s, lw, h, plan):
+        m = self.model
+        rms = lambda y, w: ref.rmsnorm(y[:, :m.hidden_size], w[:m.hidden_size], m.norm_eps)
+        y = 0.5 * (rms(self._attention(r, s.left, lw.left, h, plan), lw.left_norm) +
+                   rms(self._rglru(r, s.right, lw.right, h, plan), lw.right_norm))
+        return torch.nn.functional.pad(y, (0, m.width_p - m.hidden_size))
+
+    def _delta(self, r, s, lw, h, plan):
+        T, H, G, d, v, rp = h.shape[0], s.heads, s.kv_heads, round8(s.dim), round8(s.vdim), s.rank_p
+        S, before = self.state[r]
+        step = (plan.positions, plan.qo_indptr, plan.state_ref)
+        qkv, down, gate, beta = (h @ lw.w_in.t()).split([2 * G * d + H * v, rp, rp, round8(H)], dim=1)
+        q, k, vv = ref.short_conv(qkv, lw.conv, before, *step, act="silu").split([G * d, G * d, H * v], dim=1)
+        x = down @ lw.w_decay.t() + lw.dt_bias
+        o = ref.delta(q.reshape(T, G, d), k.reshape(T, G, d), vv.reshape(T, H, v), x.reshape(T, H, d), lw.rate, beta[:, :H], S,
+                      *step, q_scale=s.dim ** -0.5, eps=DELTA_UNIT_EPS)
+        o = ref.head_norm_gate(o, (gate @ lw.w_gate.t()).reshape(T, H, v), lw.norm.expand(H, v), s.vdim, self.model.norm_eps)
+        return o.reshape(T, -1) @ lw.w_o.t()
+
     # ---- feed-forwards ----------------------------------------------------------------------------------
     def _dense(self, s, lw, h):
         a = s.act
@@ -106,13 +146,14 @@ class CpuLayerListEngine:
 
     def _moe(self, s, lw, h):
         logits = h @ lw.router.t()
-        idx, weight = ref.moe_route(logits[:, :s.experts], lw.correction, s.top, s.groups, s.keep, s.scale)
-        mats = [t.chunk(s.experts) for t in (lw.w_gate, lw.w_up, lw.w_down)]
+        idx, weight = ref.moe_route(logits[:, :s.experts], lw.correction, s.top, s.groups, s.keep, s.scale, s.score)
+        mats = [None if t is None else t.chunk(s.experts) for t in (lw.w_gate, lw.w_up, lw.w_down)]
         a, out = s.expert.act, torch.zeros_like(h)
         for e in range(s.experts):
             t, k = (idx == e).nonzero(as_tuple=True)
             if t.numel():
-                y = ref.gated_mlp(h[t], mats[0][e], mats[1][e], mats[2][e], a.name, limit=a.limit, alpha=a.alpha, shift=a.shift)
+                y = torch.nn.functional.gelu(h[t] @ mats[1][e].t()) @ mats[2][e].t() if not s.expert.gated else \
+                    ref.gated_mlp(h[t], mats[0][e], mats[1][e], mats[2][e], a.name, limit=a.limit, alpha=a.alpha, shift=a.shift)
                 out.index_add_(0, t, y * weight[t, k][:, None])
         if s.shared is not None:
             out += torch.sigmoid(logits[:, s.experts:s.experts + 1]) * self._dense(s.shared, lw.shared, h)
@@ -129,12 +170,12 @@ class CpuLayerListEngine:
         ids[fb >= 0] = self.sampled[fb[fb >= 0]].long()
         W = m.hidden_size
         after = lambda y, n: y if n is None else self._norm(y[:, :W], n)
-        x = after(w.embed[ids] * m.embed_scale, w.embed_norm)
+        x = start = after(w.embed[ids] * m.embed_scale, w.embed_norm)
         for r, run in enumerate(m.runs):
             spec, lw = m.layers[run.layer], w.layers[run.layer]
             if run.step is not None:
-                x = x + w.loop_steps[run.step]
-            h = self._norm(x[:, :W], lw.norm_in)
+                x = x + (start if m.loop_add == "embedding" else w.loop_steps[run.step])
+            h = self._input_conv(r, 0, self._norm(x[:, :W], lw.norm_in), lw.conv_in, plan)
             y = MIXERS[spec.mixer.kind](self, r, spec.mixer, lw.mixer, h, plan)
             if spec.mlp is None:
                 x = x + after(y, lw.norm_out)
@@ -142,7 +183,7 @@ class CpuLayerListEngine:
                 x = x + (y + FEED_FORWARDS[spec.mlp.kind](self, spec.mlp, lw.mlp, h))
             else:
                 x = x + after(y, lw.norm_out)
-                h = self._norm(x[:, :W], lw.mlp_in)
+                h = self._input_conv(r, 1, self._norm(x[:, :W], lw.mlp_in), lw.conv_mlp, plan)
                 x = x + after(FEED_FORWARDS[spec.mlp.kind](self, spec.mlp, lw.mlp, h), lw.mlp_out)
         rows = torch.from_numpy(plan.sample_rows).long()
         self._logits = (self._norm(x[rows][:, :m.hidden_size], w.final_norm) @ w.lm_head.t())[:, :m.vocab_size]
@@ -177,5 +218,6 @@ class CpuLayerListEngine:
 
 
 MIXERS = {"latent_attention": CpuLayerListEngine._latent_attention, "mlstm": CpuLayerListEngine._mlstm,
-          "attention": CpuLayerListEngine._attention, "wkv": CpuLayerListEngine._wkv}
+          "attention": CpuLayerListEngine._attention, "wkv": CpuLayerListEngine._wkv,
+          "rglru": CpuLayerListEngine._rglru, "delta": CpuLayerListEngine._delta, "pair": CpuLayerListEngine._pair}
 FEED_FORWARDS = {"dense": CpuLayerListEngine._dense, "moe": CpuLayerListEngine._moe}

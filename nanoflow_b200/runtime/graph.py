@@ -94,6 +94,10 @@ MoePermuteParams = _ops.MoePermuteParams
 MoeGemmParams = _ops.MoeGemmParams
 TokenShiftParams = _ops.TokenShiftParams
 WkvParams = _ops.WkvParams
+TalkAttnParams = _ops.TalkAttnParams
+ShortConvParams = _ops.ShortConvParams
+RgLruParams = _ops.RgLruParams
+DeltaParams = _ops.DeltaParams
 
 KERNEL_OF = {
     GemmParams: "nfk_gemm_bf16", RopeAppendParams: "nfk_rope_append", RopeTableParams: "nfk_rope_table",
@@ -104,6 +108,7 @@ KERNEL_OF = {
     LatentGatherParams: "nfk_latent_gather", LatentAttnParams: "nfk_latent_attn", HeadNormGateParams: "nfk_head_norm_gate",
     GqaAppendParams: "nfk_gqa_append", GqaAttnParams: "nfk_gqa_attn", MoeRouteParams: "nfk_moe_route",
     MoePermuteParams: "nfk_moe_permute", MoeGemmParams: "nfk_moe_gemm", TokenShiftParams: "nfk_token_shift",
+    TalkAttnParams: "nfk_talk_attn", ShortConvParams: "nfk_short_conv",
     MemcpyParams: "nfk_memcpy_p", Memcpy2DParams: "nfk_memcpy2d_p", KvMoveParams: "nfk_kv_move_p", SleepParams: "nfk_sleep_p",
 }
 

@@ -11,18 +11,24 @@ one GPU, one stream. Per layer run:
   rows as keys and values at once, and a second block-diagonal GEMM applies the value matrices. Longer
   portions gather the latents they can see, expand them to keys and values of all heads with one GEMM, and
   run the tcgen05 prefill kernel over those;
-* grouped-query attention: queries and keys normed, values mixed, both appended to the paged pool; single tokens
-  on the split-KV decode kernel, portions on the tcgen05 prefill kernel (in 32-bit, and for head sizes those are
-  not built for, one simple kernel);
+* grouped-query attention: queries and keys normed or rotated, values mixed or rotated, both appended to the paged
+  pool; single tokens on the split-KV decode kernel, portions on the tcgen05 prefill kernel (in 32-bit, and for head
+  sizes and options those are not built for, one simple kernel); attention with mixed heads on kernels of its own;
 * mLSTM: one kernel for requests with one token, one for longer portions, then head norm and output gate;
 * WKV: every stream's mix with the previous token (kept per request), the four projections as one block-diagonal
   product, the low-rank decay, one kernel for single tokens and one for portions (chunks, or token by token),
   both with head norm and gate;
+* real-gated linear recurrent unit: short convolution, both gates as one block-diagonal product, one kernel for the
+  recurrence and the product with the GELU branch;
+* delta rule: short convolutions of queries, keys and values as one, low-rank decays and gates, one kernel for single
+  tokens and one for portions, both with head norm and gate;
+* two mixers side by side: one input projection for both;
 * output projection;
 * feed-forward: gated, or a mixture of experts (router product, routing, rows in expert order, two products per
   expert, the shared expert);
-* one kernel for: norm of the sublayer's output or the weighted sum of experts and shared expert, residual sum in
-  fp32, the step vector of a loop pass, and the norm the next sublayer reads.
+* one kernel for: norm of the sublayer's output, of a pair's outputs, or of the weighted sum of experts and shared
+  expert, residual sum in fp32, the step vector of a loop pass or the embedding row, and the norm the next sublayer
+  reads; a convolution over time after it where the model has one.
 
 A new kind of mixer needs a spec and weights in ``models/layer_list.py`` and a builder in ``MIXERS``, a new kind of
 feed-forward one in ``FEED_FORWARDS``.
@@ -36,23 +42,27 @@ import numpy as np
 import torch
 
 from .. import ops
-from ..models.layer_list import PREFILL_HEAD_DIM, WKV_CHUNK_DIM, ActSpec, LayerListConfig, NormWeights, round8
-from ..ops import ACTS, LIN_ACTS, NORMS, dtype_code
+from ..models.layer_list import (PAGE, PREFILL_HEAD_DIM, WKV_CHUNK_DIM, ActSpec, LayerListConfig, NormWeights, parts_of,
+                                 round8)
+from ..ops import ACTS, CONV_ACTS, LIN_ACTS, NORMS, ROUTER_SCORES, dtype_code
 from ..ops.layer_list import mlstm_scratch_floats
 from ..serving.scheduler import BatchPlan
 from .engine import DECODE_MAX_CHUNKS, DECODE_SPLIT_ROWS, GEMM_WS_BYTES, Engine, MetaLayout
-from .graph import (ArgmaxParams, AttnParams, GemmParams, GqaAppendParams, GqaAttnParams, HeadNormGateParams,
+from .graph import (ArgmaxParams, AttnParams, DeltaParams, GemmParams, GqaAppendParams, GqaAttnParams, HeadNormGateParams,
                     LatentAppendParams, LatentAttnParams, LatentGatherParams, MemcpyParams, MlstmParams, MoeGemmParams,
-                    MoePermuteParams, MoeRouteParams, OpGraph, ResidualNormParams, TokenShiftParams, WkvParams)
+                    MoePermuteParams, MoeRouteParams, OpGraph, ResidualNormParams, RgLruParams, RopeTableParams,
+                    ShortConvParams, TalkAttnParams, TokenShiftParams, WkvParams)
 from .pipeline import _ptr
 
-PAGE = 16
 QUERY_TILE = 128             # query tokens per work item of the prefill attention kernel
 MLSTM_CHUNK = 64             # tokens per chunk of the chunked mLSTM kernel
 MLSTM_COLS = 64              # columns of the state per CTA of that kernel
 SEGMENT_ITEMS = 48           # most segments that prompt portions are cut into for the mLSTM kernel
 WKV_CHUNK = 64               # tokens per chunk of the chunked WKV kernels
 WKV_SPARE_CHUNKS = 64        # chunks beyond whole ones that their scratch has room for; further portions go token by token
+
+
+DELTA_UNIT_EPS = 1e-6        # of the unit vectors of the delta rule
 
 
 class PathGroup:
@@ -104,7 +114,9 @@ class LayerListEngine(Engine):
         if m.run_specs("mlstm"):
             extra["segs"] = 4 * max(B, SEGMENT_ITEMS)
         if m.run_specs("wkv"):
-            extra.update(wkv_items=4 * max(1, self.wkv_cap), wkv_seq=B, wkv_all=B)
+            extra.update(wkv_items=4 * max(1, self.wkv_cap), wkv_seq=B)
+        if m.run_specs("wkv") or m.run_specs("delta"):
+            extra["pre_reqs"] = B
         self._make_metadata(MetaLayout(T, B, self.nano_sizes, self.num_pages, 0, self.S_cap, extra))
         self.meta = {n: self._meta_view(n) for n in self.layout.off}
         self._alloc_buffers()
@@ -126,28 +138,49 @@ class LayerListEngine(Engine):
 
     def _alloc_state(self) -> None:
         m, dev = self.model, self.device
-        self.state: List[Optional[Tuple[torch.Tensor, ...]]] = []
         n = self.num_slots
         z = lambda *shape, dtype=torch.float32: torch.zeros(*shape, dtype=dtype, device=dev)
+        # per run: the state of its recurrent mixer, and the last inputs of the two sublayers' input convolutions
+        self.state: List[Tuple[torch.Tensor, ...]] = []
+        self.conv_state: List[Tuple[Optional[torch.Tensor], ...]] = []
         for r in m.runs:
-            s = m.layers[r.layer].mixer
-            d, v = round8(s.dim), round8(s.vdim)
-            if s.kind == "mlstm":
-                self.state.append((z(n, s.heads, d, v), z(n, s.heads, 2, d), z(n, s.heads, 2)))
-            elif s.kind == "wkv":
-                self.state.append((z(n, s.heads, d, d), z(n, 2, m.width_p, dtype=m.dtype)))
-            else:
-                self.state.append(None)
+            lay = m.layers[r.layer]
+            self.state.append(tuple(z(n, *shape, dtype=dt) for s in parts_of(lay.mixer) for shape, dt in m.state_shapes(s)))
+            conv = lambda used: z(n, *m.conv_state_shape(), dtype=m.dtype) if m.input_conv and used else None
+            self.conv_state.append((conv(True), conv(lay.mlp is not None)))
 
     def _widths(self) -> Dict[str, int]:
         """Columns of the shared activation buffers (the widest layer's)."""
         m = self.model
         w = dict(proj=8, gates=8, attn=8, q_lat=0, o_lat=0, o_rec=8, act=8, kv=0, cg=0, qn=0, v_first=0, mix=0, lora=0,
-                 router=0, e_in=0, e_act=0, e_out=0, e_top=0)
+                 router=0, e_in=0, e_act=0, e_out=0, e_top=0, conv=0, aux=0, beta=0)
         up = lambda k, n: w.__setitem__(k, max(w[k], n))
         for lay in m.layers:
             s = lay.mixer
-            if s.kind == "latent_attention":
+            if s.kind == "pair":
+                a, b, hd = s.left, s.right, m.attn_hd(s.left)
+                up("proj", (a.heads + 2 * a.kv_heads) * hd + 2 * b.cols)
+                up("qn", a.heads * hd)
+                up("attn", a.heads * hd)
+                up("conv", b.cols)
+                up("gates", 2 * b.cols)
+                up("aux", b.cols)
+            elif s.kind == "rglru":
+                up("proj", 2 * s.cols)
+                up("conv", s.cols)
+                up("gates", 2 * s.cols)
+                up("attn", s.cols)
+            elif s.kind == "delta":
+                d, v = round8(s.dim), round8(s.vdim)
+                qkv = 2 * s.kv_heads * d + s.heads * v
+                up("proj", qkv + 2 * s.rank_p)
+                up("conv", qkv)
+                up("beta", round8(s.heads))
+                up("gates", s.heads * d)
+                up("aux", s.heads * v)
+                up("o_rec", s.heads * v)
+                up("attn", s.heads * v)
+            elif s.kind == "latent_attention":
                 dq, dv = m.head_pads(s)
                 ld = m.latent_ld(s)
                 up("proj", s.heads * dq + round8(s.kv_rank))
@@ -196,8 +229,9 @@ class LayerListEngine(Engine):
         w = self._widths()
         es = m.elem_bytes
         act = T * (4 * m.width_p + es * (3 * m.width_p + w["proj"] + w["attn"] + 2 * w["q_lat"] + w["act"] + w["qn"] +
-                                         w["v_first"] + w["mix"] + w["lora"] + w["e_in"] + w["e_act"] + w["e_out"]) +
-                   4 * (w["gates"] + w["o_rec"] + w["router"] + 5 * w["e_top"]))
+                                         w["v_first"] + w["mix"] + w["lora"] + w["e_in"] + w["e_act"] + w["e_out"] + w["conv"] +
+                                         w["aux"] + 2 * m.width_p) +
+                   4 * (w["gates"] + w["o_rec"] + w["router"] + w["beta"] + 5 * w["e_top"] + 2 * sum((len(k) + 7) // 8 * 8 for k in self._rotations())))
         act += self._decode_ws_floats() * 4 + self._wkv_scratch_floats() * 4
         act += self.x_pages * PAGE * (w["kv"] + w["cg"]) * es + self.S_cap * (es * m.width_p + 4 * m.vocab_p)
         budget = free - total * (1.0 - e.gpu_mem_fraction) - act - (1 << 30)
@@ -206,6 +240,10 @@ class LayerListEngine(Engine):
         if n < 64:
             raise RuntimeError(f"not enough GPU memory for a page pool ({free >> 20} MiB free)")
         return n
+
+    def _rotations(self) -> List[tuple]:
+        """The distinct lists of frequencies of the model."""
+        return sorted({key for s in self.model.run_specs("attention") for key in rotations(s)})
 
     def _decode_ws_floats(self) -> int:
         """Partial results of split-KV decode attention."""
@@ -224,13 +262,21 @@ class LayerListEngine(Engine):
         self.x = P(T, m.width_p, f32, "x")
         self.h = P(T, m.width_p, dt, "h")
         self.y = P(T, m.width_p, dt, "y")
-        self.y2 = P(T, m.width_p, dt, "y2") if m.parallel or m.run_moes() else None
+        self.h_raw = P(T, m.width_p, dt, "h_raw") if m.input_conv else None      # before the input convolution
+        pairs = any(lay.mixer.kind == "pair" for lay in m.layers)
+        self.y2 = P(T, m.width_p, dt, "y2") if m.parallel or m.run_moes() or pairs else None
         flat = lambda k, dtype, rows=T: P(1, max(8, rows * w[k]), dtype, k).view(-1)
         self.flat = {"proj": flat("proj", dt), "attn": flat("attn", dt), "act": flat("act", dt), "gates": flat("gates", f32),
                      "o_rec": flat("o_rec", f32), "q_lat": flat("q_lat", dt), "o_lat": flat("q_lat", dt),
                      "kv": flat("kv", dt, self.x_pages * PAGE), "cg": flat("cg", dt, self.x_pages * PAGE),
-                     "router": flat("router", f32)}
-        self.flat.update({k: flat(k, dt) for k in ("qn", "v_first", "mix", "lora", "e_in", "e_act", "e_out")})
+                     "router": flat("router", f32), "beta": flat("beta", f32)}
+        self.flat.update({k: flat(k, dt) for k in ("qn", "v_first", "mix", "lora", "e_in", "e_act", "e_out", "conv", "aux")})
+        # (cos, sin) of every token's angles, one table per distinct list of frequencies
+        self.angles: Dict[tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
+        for key in self._rotations():
+            f = torch.zeros(max(8, (len(key) + 7) // 8 * 8), dtype=f32, device=dev)
+            f[:len(key)] = torch.tensor(key, dtype=torch.float64)
+            self.angles[key] = (f, torch.zeros(T, f.numel(), 2, dtype=f32, device=dev))
         i32 = torch.int32
         self.moe_ids = {k: flat("e_top", f32 if k == "weight" else i32) for k in ("expert", "rank", "slot", "weight")}
         self.moe_gate = P(1, T, f32, "moe_gate").view(-1)
@@ -244,7 +290,8 @@ class LayerListEngine(Engine):
         self.wkv_ws = torch.empty(max(8, self._wkv_scratch_floats()), dtype=f32, device=dev)
         self.h_s = P(self.S_cap, m.width_p, dt, "sample_h")
         self.logits = P(self.S_cap, m.vocab_p, f32, "logits")
-        self.pools = [self._pool(m.layers[r.layer].mixer) for r in m.runs]
+        self.pools = [next((p for s in parts_of(m.layers[r.layer].mixer) for p in [self._pool(s)] if p is not None), None)
+                      for r in m.runs]
         self.arange = torch.arange(self.x_pages + 1, dtype=torch.int32, device=dev)
         heads = max([s.heads * (m.latent_ld(s) + 2) for s in m.run_specs("latent_attention")], default=0)
         self.latent_ws = torch.empty(max(8, 160 * heads), dtype=f32, device=dev)
@@ -263,10 +310,8 @@ class LayerListEngine(Engine):
         self.bufs.logits = self.logits
 
     def _pool(self, s) -> Optional[torch.Tensor]:
-        m, z = self.model, lambda *shape: torch.zeros(self.num_pages, *shape, dtype=self.model.dtype, device=self.device)
-        if s.kind == "latent_attention":
-            return z(PAGE, m.latent_ld(s))
-        return z(2, s.kv_heads, PAGE, m.attn_hd(s)) if s.kind == "attention" else None
+        shape = self.model.pool_shape(s)
+        return None if shape is None else torch.zeros(self.num_pages, *shape, dtype=self.model.dtype, device=self.device)
 
     def view(self, name: str, cols: int, rows: Optional[int] = None) -> torch.Tensor:
         rows = rows or self.T
@@ -289,19 +334,25 @@ class LayerListEngine(Engine):
         if m.run_moes():
             self._op("moe_counts", MemcpyParams(dst=_ptr(self.moe_counts), src=_ptr(self.moe_zeros), elem_bytes=4,
                                                 count=self.moe_counts.numel()))
-        # the stream's step before each run, as (vector added, norm of its mixer's input)
-        step = lambda r: None if m.runs[r].step is None else w.loop_steps[m.runs[r].step]
+        for i, (freq, table) in enumerate(self.angles.values()):
+            self._op(f"angles{i}", RopeTableParams(cos_sin=_ptr(table), inv_freq=_ptr(freq), positions=_ptr(self.meta["positions"]),
+                                                   T=0, half=freq.numel()), dyn=[("T", T)])
+        # what joins the stream before each run: a step vector, or the embedding row
+        step = lambda r: None if m.runs[r].step is None else "embedding" if m.loop_add == "embedding" else \
+            w.loop_steps[m.runs[r].step]
         self._residual("embedding", None, w.embed_norm, w.layers[m.runs[0].layer].norm_in, step(0), embed=True)
+        self._input_conv(0, 0)
         for r, run in enumerate(m.runs):
             spec, lw = m.layers[run.layer], w.layers[run.layer]
             last = r + 1 == len(m.runs)
             nxt = None if last else w.layers[m.runs[r + 1].layer].norm_in
             add = None if last else step(r + 1)
-            MIXERS[spec.mixer.kind](self, r, run.layer, spec.mixer, lw.mixer)
-            y, out, more = self.y, lw.norm_out, {}         # what joins the stream at the end of the layer
+            more = MIXERS[spec.mixer.kind](self, r, run.layer, spec.mixer, lw.mixer) or {}
+            y, out = self.y, lw.norm_out                   # what joins the stream at the end of the layer
             if spec.mlp is not None:
                 if not m.parallel:
-                    self._residual(f"R{r}.mid", self.y, lw.norm_out, lw.mlp_in, None, layer=r)
+                    self._residual(f"R{r}.mid", self.y, lw.norm_out, lw.mlp_in, None, layer=r, more=more)
+                    self._input_conv(r, 1)
                     out = lw.mlp_out
                 more = FEED_FORWARDS[spec.mlp.kind](self, r, run.layer, spec.mlp, lw.mlp)
                 if not m.parallel:
@@ -312,6 +363,8 @@ class LayerListEngine(Engine):
             else:
                 tap_add = add if self.taps is None else None
                 self._residual(f"R{r}.out", y, out, None if (last or self.taps is not None) else nxt, tap_add, layer=r, more=more)
+                if not last and self.taps is None:
+                    self._input_conv(r + 1, 0)
                 if self.taps is not None:
                     self._op(f"R{r}.tap", MemcpyParams(dst=_ptr(self.taps[r]), src=_ptr(self.x), elem_bytes=4 * m.width_p,
                                                        count=0), dyn=[("count", T)], layer=r)
@@ -319,6 +372,7 @@ class LayerListEngine(Engine):
                         self._residual("final", None, None, w.final_norm, None, sampled=True)
                     else:
                         self._residual(f"R{r}.next", None, None, nxt, add, layer=r)
+                        self._input_conv(r + 1, 0)
         S = g.symbol("n_sample")
         self._gemm("lm_head", self.h_s, w.lm_head, None, rows=S, d32=self.logits)
         self._op("argmax", ArgmaxParams(idx_out=_ptr(self.bufs.sampled), val_out=c_void_p(0), logits=_ptr(self.logits),
@@ -336,17 +390,20 @@ class LayerListEngine(Engine):
 
     def _residual(self, name, y, norm_in: Optional[NormWeights], norm_out: Optional[NormWeights], add, *, embed=False,
                   sampled=False, layer=-1, more: Optional[dict] = None) -> None:
-        """``more``: what a feed-forward adds to the sum besides ``y``: ``y2`` with ``y2_gate`` per row, and expert rows
-        (``e_out``, ``e_slot``, ``e_weight``, ``e_top``)."""
+        """``more``: what a sublayer adds to the sum besides ``y``: ``y2`` with ``y2_gate`` per row, and expert rows
+        (``e_out``, ``e_slot``, ``e_weight``, ``e_top``), under the same norm; or ``pair``: the norms of ``y`` and ``y2``
+        whose mean is the output. ``add``: a vector, or "embedding"."""
         m, kind = self.model, NORMS[self.model.norm_kind]
         p = ResidualNormParams()
         p.x, p.ld_x = _ptr(self.x), self.x.stride(0)
-        if embed:
+        again = isinstance(add, str)
+        if embed or again:
+            p.table_add = int(again)
             p.table, p.ld_table, p.vocab = _ptr(self.w.embed), self.w.embed.stride(0), m.vocab_size
             p.host_ids, p.feedback_src = _ptr(self.meta["host_ids"]), _ptr(self.meta["feedback_src"])
             p.prev_tokens = _ptr(self.bufs.sampled)
             p.src_scale = m.embed_scale
-        elif y is not None:
+        if y is not None and not embed:
             p.y, p.ld_y = _ptr(y), y.stride(0)
         if norm_in is not None:
             p.in_w, p.in_b, p.in_kind = _ptr(norm_in.w), _ptr(norm_in.b), kind
@@ -356,14 +413,35 @@ class LayerListEngine(Engine):
         if more.get("e_out") is not None:
             p.e_out, p.ld_e, p.e_rows = _ptr(more["e_out"]), more["e_out"].stride(0), more["e_out"].shape[0]
             p.e_slot, p.e_weight, p.e_top = _ptr(more["e_slot"]), _ptr(more["e_weight"]), more["e_top"]
-        p.add = _ptr(add)
+        if more.get("pair") is not None:
+            p.pair_w, p.pair_w2 = _ptr(more["pair"][0]), _ptr(more["pair"][1])
+        elif norm_in is not None and (p.y2 or p.e_out):
+            p.norm_sum = 1
+        p.add = None if again else _ptr(add)
         if norm_out is not None:
-            h = self.h_s if sampled else self.h
+            h = self.h_s if sampled else self.h if self.h_raw is None else self.h_raw
             p.h, p.ld_h, p.out_w, p.out_b, p.out_kind = _ptr(h), h.stride(0), _ptr(norm_out.w), _ptr(norm_out.b), kind
         if sampled:
             p.rows_idx, p.in_rows = _ptr(self.meta["sample_rows"]), self.T
         p.cols, p.eps, p.dtype, p.status = m.hidden_size, m.norm_eps, self.code, _ptr(self.bufs.status)
         self._op(name, p, dyn=[("rows", "n_sample" if sampled else "T")], layer=layer)
+
+    def _short_conv(self, name, x, out, w, state, *, bias=None, act=None, residual=False, layer=-1) -> None:
+        meta, m = self.meta, self.model
+        p = ShortConvParams(x=_ptr(x), ld_x=x.stride(0), out=_ptr(out), ld_out=out.stride(0), w=_ptr(w), bias=_ptr(bias),
+                            state=_ptr(state), state_slot=_ptr(meta["state_ref"]), positions=_ptr(meta["positions"]),
+                            token_req=_ptr(meta["token_req"]), qo_indptr=_ptr(meta["qo_indptr"]), row_begin=0, T=0,
+                            cols=w.shape[1], taps=w.shape[0], act=CONV_ACTS[act], residual=int(residual),
+                            num_slots=self.num_slots, dtype=self.code, status=_ptr(self.bufs.status))
+        self._op(name, p, dyn=[("T", "T")], layer=layer)
+
+    def _input_conv(self, r: int, sublayer: int) -> None:
+        """h = h_raw + its convolution, ahead of run ``r``'s mixer (0) or feed-forward (1)."""
+        lw = self.w.layers[self.model.runs[r].layer]
+        w = lw.conv_mlp if sublayer else lw.conv_in
+        if w is not None:
+            self._short_conv(f"R{r}.input_conv{sublayer}", self.h_raw, self.h, w, self.conv_state[r][sublayer], residual=True,
+                             layer=r)
 
     def _gemm(self, name, a, wt, out, *, rows: str, up=None, act: ActSpec = ActSpec("silu"), lin_act=None, bias=None, d32=None,
               f32_col0=0, groups=1, group_k=0, k=0, key="", layer=-1) -> None:
@@ -468,11 +546,14 @@ class LayerListEngine(Engine):
         self._op(f"R{r}.head_norm", hp, dyn=[("T", T)], layer=r)
         self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
 
-    def _attention(self, r: int, layer: int, s, lw) -> None:
+    def _attention(self, r: int, layer: int, s, lw, proj=None) -> None:
+        """``proj``: the projected queries, keys and values, if they are there already."""
         m, g, T, meta, st = self.model, self.g, "T", self.meta, _ptr(self.bufs.status)
         H, G, hd, pool = s.heads, s.kv_heads, m.attn_hd(s), self.pools[r]
-        proj, qn, attn = self.view("proj", (H + 2 * G) * hd), self.view("qn", H * hd), self.view("attn", H * hd)
-        self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, key=f"l{layer}.in", layer=r)
+        qn, attn = self.view("qn", H * hd), self.view("attn", H * hd)
+        if proj is None:
+            proj = self.view("proj", (H + 2 * G) * hd)
+            self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, key=f"l{layer}.in", layer=r)
         mode = 0 if not s.value_mix else 1 if r == m.first_value_run else 2
         ap = GqaAppendParams(src=_ptr(proj), ld_src=proj.stride(0), q_off=0, k_off=H * hd, v_off=(H + G) * hd, q_out=_ptr(qn),
                              q_w=_ptr(lw.q_norm), k_w=_ptr(lw.k_norm), v_first=_ptr(self.flat["v_first"]), v_mode=mode,
@@ -481,8 +562,24 @@ class LayerListEngine(Engine):
                              kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), T=0, heads=H, kv_heads=G,
                              hd=hd, dim=s.dim, page_size=PAGE, num_pages=self.num_pages, eps=m.norm_eps, dtype=self.code,
                              status=st)
+        turns = rotations(s)
+        if turns:
+            ap.rot, ap.rot_pairs, ap.rot_ld = _ptr(self.angles[turns[0]][1]), len(turns[0]), self.angles[turns[0]][0].numel()
+        if len(turns) > 1:
+            v_rot, v_pairs, v_ld = _ptr(self.angles[turns[1]][1]), len(turns[1]), self.angles[turns[1]][0].numel()
+            ap.v_rot, ap.v_pairs, ap.v_ld = v_rot, v_pairs, v_ld
+        else:
+            v_rot, v_pairs, v_ld = None, 0, 0
         self._op(f"R{r}.gqa_append", ap, dyn=[("T", T)], layer=r)
-        if m.attn_on_tensor_cores(s):
+        if s.talk:
+            tp = TalkAttnParams(q=_ptr(qn), pool=_ptr(pool), out=_ptr(attn), positions=_ptr(meta["positions"]),
+                                token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
+                                kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), sinks=_ptr(lw.sinks),
+                                talk=_ptr(lw.talk), v_rot=v_rot, v_pairs=v_pairs, v_ld=v_ld, token_begin=0, n_tokens=0, heads=H,
+                                kv_heads=G, hd=hd, page_size=PAGE, num_pages=self.num_pages, window=s.window or 0, scale=s.scale,
+                                dtype=self.code, status=st)
+            self._op(f"R{r}.talk_attn", tp, dyn=[("n_tokens", T)], layer=r)
+        elif m.attn_on_tensor_cores(s):
             def params() -> AttnParams:
                 p = AttnParams()
                 p.q, p.out, p.kv_pool = _ptr(qn), _ptr(attn), _ptr(pool)
@@ -506,7 +603,7 @@ class LayerListEngine(Engine):
                                token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
                                kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), sinks=_ptr(lw.sinks),
                                token_begin=0, n_tokens=0, heads=H, kv_heads=G, hd=hd, page_size=PAGE,
-                               num_pages=self.num_pages, window=0, scale=s.scale, softcap=s.softcap or 0.0, dtype=self.code,
+                               num_pages=self.num_pages, window=s.window or 0, scale=s.scale, softcap=s.softcap or 0.0, dtype=self.code,
                                status=st)
             self._op(f"R{r}.attn", gp, dyn=[("n_tokens", T)], layer=r)
         self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
@@ -538,11 +635,70 @@ class LayerListEngine(Engine):
         self._op(f"R{r}.wkv_decode", params(), kernel="nfk_wkv_decode", dyn=[("req_count", "n_dec")], layer=r)
         chunked = self.wkv_cap > 0 and d <= WKV_CHUNK_DIM
         p = params()
-        p.seq_reqs = _ptr(meta["wkv_seq" if chunked else "wkv_all"])
+        p.seq_reqs = _ptr(meta["wkv_seq" if chunked else "pre_reqs"])
         dyn = [("num_seq", self.g.symbol("n_wkv_seq" if chunked else "n_pre"))]
         if chunked:
             dyn.append(("num_items", self.g.symbol("n_wkv_items")))
         self._op(f"R{r}.wkv_prefill", p, kernel="nfk_wkv_prefill", dyn=dyn, layer=r)
+        self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
+
+    def _rglru(self, r: int, layer: int, s, lw, proj=None, act=None, out=None) -> None:
+        """``proj``: the two projected branches, if they are there already; ``act``, ``out``: where the recurrence's result
+        and its output projection go."""
+        T, meta, n, bp = "T", self.meta, s.cols, s.block_p
+        S, before = self.state[r]
+        if proj is None:
+            proj = self.view("proj", 2 * n)
+            self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, bias=lw.b_in, key=f"l{layer}.in", layer=r)
+        act = self.view("attn", n) if act is None else act
+        u, gates = self.view("conv", n), self.view("gates", 2 * n)
+        self._short_conv(f"R{r}.rec_conv", proj[:, n:], u, lw.conv, before, bias=lw.conv_b, layer=r)
+        self._gemm(f"R{r}.rec_gates", u, lw.w_gates, None, rows=T, d32=gates, groups=s.blocks, group_k=bp, k=bp, layer=r)
+
+        def params() -> RgLruParams:
+            return RgLruParams(u=_ptr(u), ld_u=u.stride(0), y=_ptr(proj), ld_y=proj.stride(0), gates=_ptr(gates),
+                               ld_g=gates.stride(0), r_b=_ptr(lw.r_b), i_b=_ptr(lw.i_b), log_a=_ptr(lw.log_a), S=_ptr(S),
+                               out=_ptr(act), ld_out=act.stride(0), positions=_ptr(meta["positions"]),
+                               qo_indptr=_ptr(meta["qo_indptr"]), state_slot=_ptr(meta["state_ref"]), req_begin=0, req_count=0,
+                               cols=n, block=bp, num_slots=self.num_slots, dtype=self.code, status=_ptr(self.bufs.status))
+
+        self._op(f"R{r}.rglru_decode", params(), kernel="nfk_rglru_decode", dyn=[("req_count", "n_dec")], layer=r)
+        self._op(f"R{r}.rglru_prefill", params(), kernel="nfk_rglru_prefill",
+                 dyn=[("req_begin", "n_dec"), ("req_count", "n_pre")], layer=r)
+        self._gemm(f"R{r}.rec_o", act, lw.w_o, self.y if out is None else out, rows=T, key=f"l{layer}.rec_o", layer=r)
+
+    def _pair(self, r: int, layer: int, s, lw) -> dict:
+        n = lw.left.w_in.shape[0]
+        proj = self.view("proj", lw.w_in.shape[0])
+        self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows="T", bias=lw.b_in, key=f"l{layer}.in", layer=r)
+        self._attention(r, layer, s.left, lw.left, proj[:, :n])
+        self._rglru(r, layer, s.right, lw.right, proj[:, n:], self.view("aux", s.right.cols), self.y2)
+        return {"y2": self.y2, "pair": (lw.left_norm, lw.right_norm)}
+
+    def _delta(self, r: int, layer: int, s, lw) -> None:
+        T, meta, st = "T", self.meta, _ptr(self.bufs.status)
+        H, G, d, v, rp = s.heads, s.kv_heads, round8(s.dim), round8(s.vdim), s.rank_p
+        S, before = self.state[r]
+        qkv = 2 * G * d + H * v
+        proj, conv, beta = self.view("proj", qkv + 2 * rp), self.view("conv", qkv), self.view("beta", round8(H))
+        decay, gate, attn = self.view("gates", H * d), self.view("aux", H * v), self.view("attn", H * v)
+        self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, d32=beta, f32_col0=qkv + 2 * rp, key=f"l{layer}.in", layer=r)
+        self._short_conv(f"R{r}.qkv_conv", proj, conv, lw.conv, before, act="silu", layer=r)
+        self._gemm(f"R{r}.decay_up", proj[:, qkv:qkv + rp], lw.w_decay, None, rows=T, d32=decay, key=f"l{layer}.decay_up", layer=r)
+        self._gemm(f"R{r}.gate_up2", proj[:, qkv + rp:], lw.w_gate, gate, rows=T, key=f"l{layer}.gate_up2", layer=r)
+
+        def params() -> DeltaParams:
+            return DeltaParams(qkv=_ptr(conv), ld=conv.stride(0), q_off=0, k_off=G * d, v_off=2 * G * d, x=_ptr(decay),
+                               ld_x=decay.stride(0), beta=_ptr(beta), ld_b=beta.stride(0), g=_ptr(gate), ld_g=gate.stride(0),
+                               rate=_ptr(lw.rate), dt_bias=_ptr(lw.dt_bias), norm=_ptr(lw.norm), S=_ptr(S), y=_ptr(attn),
+                               ld_y=attn.stride(0), positions=_ptr(meta["positions"]), qo_indptr=_ptr(meta["qo_indptr"]),
+                               state_slot=_ptr(meta["state_ref"]), req_begin=0, req_count=0, heads=H, kv_heads=G, dim=d, vdim=v,
+                               vdim_real=s.vdim, num_slots=self.num_slots, q_scale=s.dim ** -0.5, unit_eps=DELTA_UNIT_EPS,
+                               eps=self.model.norm_eps, dtype=self.code, seq_reqs=_ptr(meta["pre_reqs"]), num_seq=0,
+                               o=_ptr(self.flat["o_rec"]), status=st)
+
+        self._op(f"R{r}.delta_decode", params(), kernel="nfk_delta_decode", dyn=[("req_count", "n_dec")], layer=r)
+        self._op(f"R{r}.delta_prefill", params(), kernel="nfk_delta_prefill", dyn=[("num_seq", "n_pre")], layer=r)
         self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
 
     # ---- feed-forwards: read self.h; return what joins the stream (see _residual) -------------------------
@@ -564,22 +720,25 @@ class LayerListEngine(Engine):
         rp = MoeRouteParams(logits=_ptr(logits), ld=logits.stride(0), correction=_ptr(lw.correction), expert=_ptr(ids["expert"]),
                             weight=_ptr(ids["weight"]), rank=_ptr(ids["rank"]), counts=_ptr(counts), gate=_ptr(self.moe_gate),
                             T=0, experts=s.experts, top=s.top, groups=s.groups, keep=s.keep,
-                            gate_col=s.experts if s.shared is not None else -1, scale=s.scale)
+                            gate_col=s.experts if s.shared is not None else -1, scale=s.scale, score=ROUTER_SCORES[s.score])
         self._op(f"R{r}.moe_route", rp, dyn=[("T", T)], layer=r)
         pp = MoePermuteParams(h=_ptr(self.h), ld_h=wp, out=_ptr(e_in), ld_out=wp, expert=_ptr(ids["expert"]),
                               rank=_ptr(ids["rank"]), counts=_ptr(counts), slot=_ptr(ids["slot"]), T=0, top=s.top,
                               experts=s.experts, cols=wp, dtype=self.code)
         self._op(f"R{r}.moe_permute", pp, dyn=[("T", T)], layer=r)
 
-        def product(name, a, b, b2, out, n) -> None:
+        def product(name, a, b, b2, out, n, lin_act=None) -> None:
             act = s.expert.act
             p = MoeGemmParams(A=_ptr(a), B=_ptr(b), B2=_ptr(b2), D=_ptr(out), counts=_ptr(counts), lda=a.stride(0),
                               ldb=b.stride(0), ldd=out.stride(0), rows=0, experts=s.experts, N=n, K=b.shape[1],
-                              act=ACTS[act.name], act_limit=act.limit, act_alpha=act.alpha, act_shift=act.shift,
-                              dtype=self.code, num_ctas=0, status=st)
+                              act=ACTS.get(act.name, 0), act_limit=act.limit, act_alpha=act.alpha, act_shift=act.shift,
+                              dtype=self.code, num_ctas=0, status=st, lin_act=LIN_ACTS[lin_act])
             self._op(f"R{r}.{name}", p, dyn=[("rows", rows)], layer=r)
 
-        product("moe_gate_up", e_in, lw.w_gate, lw.w_up, e_act, round8(s.expert.ff))
+        if s.expert.gated:
+            product("moe_gate_up", e_in, lw.w_gate, lw.w_up, e_act, round8(s.expert.ff))
+        else:
+            product("moe_up", e_in, lw.w_up, None, e_act, round8(s.expert.ff), s.expert.act.name)
         product("moe_down", e_act, lw.w_down, None, e_out, wp)
         out = dict(e_out=e_out, e_slot=ids["slot"], e_weight=ids["weight"], e_top=s.top)
         if s.shared is not None:
@@ -592,12 +751,21 @@ class LayerListEngine(Engine):
         from ..ops import autotune
         m, T, done = self.model, self.T, {}
         self.h.normal_()
-        for k in ("attn", "act", "lora"):
+        for k in ("attn", "act", "lora", "aux"):
             self.flat[k].normal_()
         for i, lay in enumerate(m.layers):
             lw = self.w.layers[i]
-            specs = [("o", None, lw.mixer.w_o, None, None)]
-            if lay.mixer.kind == "wkv":          # (its input projection is block-diagonal: left to the cost model)
+            mixer = lw.mixer.left if lay.mixer.kind == "pair" else lw.mixer
+            specs = [("o", None, mixer.w_o, None, None)]
+            if lay.mixer.kind == "pair":
+                rec = lw.mixer.right.w_o
+                specs += [("in", self.h, lw.mixer.w_in, None, self.flat["proj"]),
+                          ("rec_o", self.view("aux", rec.shape[1]), rec, None, None)]
+            elif lay.mixer.kind == "delta":
+                specs += [("in", self.h, lw.mixer.w_in, None, self.flat["proj"]),
+                          ("decay_up", self.h[:, :lay.mixer.rank_p], lw.mixer.w_decay, None, self.flat["proj"]),
+                          ("gate_up2", self.h[:, :lay.mixer.rank_p], lw.mixer.w_gate, None, self.flat["proj"])]
+            elif lay.mixer.kind == "wkv":          # (its input projection is block-diagonal: left to the cost model)
                 lora = self.view("lora", lw.mixer.w_down.shape[0])
                 specs += [("decay_down", self.h, lw.mixer.w_down, None, self.flat["proj"]),
                           ("decay_up", lora, lw.mixer.w_up, None, self.flat["proj"])]
@@ -646,8 +814,9 @@ class LayerListEngine(Engine):
             items, seq = wkv_work(qo, D, self.wkv_cap)
             put("wkv_items", items.reshape(-1))
             put("wkv_seq", seq)
-            put("wkv_all", np.arange(D, D + P, dtype=np.int32))
             sym["n_wkv_items"], sym["n_wkv_seq"] = items.shape[0], seq.size
+        if "pre_reqs" in self.meta:
+            put("pre_reqs", np.arange(D, D + P, dtype=np.int32))
         for n in self.attn_groups:
             items = query_items(qo, D, QUERY_TILE // n)
             put(f"gitem{n}", items.reshape(-1))
@@ -700,8 +869,17 @@ class LayerListEngine(Engine):
 
 
 MIXERS = {"latent_attention": LayerListEngine._latent_attention, "mlstm": LayerListEngine._mlstm,
-          "attention": LayerListEngine._attention, "wkv": LayerListEngine._wkv}
+          "attention": LayerListEngine._attention, "wkv": LayerListEngine._wkv, "rglru": LayerListEngine._rglru,
+          "delta": LayerListEngine._delta, "pair": LayerListEngine._pair}
 FEED_FORWARDS = {"dense": LayerListEngine._dense, "moe": LayerListEngine._moe}
+
+
+def rotations(s) -> List[tuple]:
+    """Frequencies by which an attention layer turns queries and keys, and if it does, values."""
+    if s.rotary is None:
+        return []
+    keys = tuple(s.rotary.frequencies(s.rotary.dims, True))
+    return [keys, tuple(s.rotary.frequencies(s.vdim, False))] if s.rotary.values else [keys]
 
 
 # --------------------------------------------------------------------------------------------------
