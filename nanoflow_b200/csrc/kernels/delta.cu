@@ -4,7 +4,20 @@
 //
 // nfk_delta_decode   one token per request: a CTA per request and head streams S through registers (recall, read-out and
 //                    update in one pass: o = S'^T q = (diag(w) S)^T q + (q . k) u), then head norm, weight and gate.
-// nfk_delta_prefill  token by token (any size, bf16 or fp32), S in shared memory.
+// nfk_delta_prefill  token by token (any size, bf16 or fp32), S in shared memory; or in chunks of 64 tokens on tensor cores
+//                    (bf16). With c_t the sum of log decays from the chunk's start through token t, the values written are
+//                        u_t = beta_t (v_t - S0^T (e^c_t k_t) - sum_{s<t} <k_t, k_s>_ts u_s),  <x, y>_ts = sum_d x y e^(c_t - c_s),
+//                    a lower-triangular system with the same matrix for all columns. Three kernels:
+//                    1. per chunk: the decayed scores <k, k> and <q, k>, the inverse M = (1 + diag(beta) <k, k>)^-1 diag(beta)
+//                       (forward substitution in fp32, by blocks of 16), then M V and W = M (e^c k);
+//                    2. along the chunks, 32 columns of S per CTA, S in registers: u = M V - W S0, the outputs
+//                       (e^c q) S0 + <q, k> u, and S = e^c_end S0 + (e^(c_end - c) k)^T u;
+//                    3. head norm, weight and gate.
+//                    Decayed rows, scores, W, u and S enter the products as bf16 pairs (high and low part, about 16 bits).
+//                    Weights of scores factor at the ends of runs of 16 tokens: the key's factor is the exponential of a
+//                    non-positive sum, and so is the query's in a later run; inside a run the query's factor grows, at most to
+//                    2^110, and a run in which some channel decays by more forms its scores pair by pair.
+#include "attn_mma.cuh"
 #include "elem_io.cuh"
 
 namespace nf {
@@ -234,14 +247,16 @@ delta_seq_kernel(nfk_delta_params p, int v_slices) {
     if (col_ok) S[static_cast<long long>(d) * p.vdim] = S_s[d * kSeqCols + lane];
 }
 
-// Head norm, weight and gate of the rows that delta_seq_kernel left in p.o: one warp per (token, head).
-template <class T>
+// Head norm, weight and gate of the rows left in p.o: one warp per (token, head). Row y of the grid is a request's
+// portion, or with CHUNKS a chunk.
+template <class T, bool CHUNKS>
 __global__ void __launch_bounds__(256)
-delta_seq_norm_kernel(nfk_delta_params p) {
+delta_norm_kernel(nfk_delta_params p) {
   const int lane = threadIdx.x & 31;
-  const int req = p.seq_reqs[blockIdx.y];
-  const int t0 = p.qo_indptr[req];
-  const long long total = static_cast<long long>(p.qo_indptr[req + 1] - t0) * p.heads;
+  const int req = CHUNKS ? 0 : p.seq_reqs[blockIdx.y];
+  const int t0 = CHUNKS ? p.items[blockIdx.y * 4 + 1] : p.qo_indptr[req];
+  const int n = CHUNKS ? p.items[blockIdx.y * 4 + 2] : p.qo_indptr[req + 1] - t0;
+  const long long total = static_cast<long long>(n) * p.heads;
   for (long long i = blockIdx.x * 8ll + (threadIdx.x >> 5); i < total; i += gridDim.x * 8ll) {
     const long long t = t0 + i / p.heads;
     const int head = static_cast<int>(i % p.heads);
@@ -259,6 +274,575 @@ delta_seq_norm_kernel(nfk_delta_params p) {
       store4(y + c, make_float4(v.x * inv * w.x * sigmoid_f(gg.x), v.y * inv * w.y * sigmoid_f(gg.y),
                                 v.z * inv * w.z * sigmoid_f(gg.z), v.w * inv * w.w * sigmoid_f(gg.w)));
     }
+  }
+}
+
+// ---- prefill, chunks of 64 tokens -------------------------------------------------------------------------------
+constexpr int kChunk = 64, kRun = 16, kRuns = kChunk / kRun, kDcThreads = 512, kDsThreads = 256;
+constexpr int kSlice = 32;                 // columns of S per CTA of the second kernel
+constexpr float kMaxRunLog2 = 110.f;       // largest decay of a run (log2) whose weights are factored inside the run
+constexpr float kMaxDecayLog2 = 150.f;     // a stronger decay is zero in fp32 anyway
+
+// Scratch of a chunk and head: W, decayed keys, decayed queries [64][dim] and scores [64][64] as bf16 pairs (high parts,
+// then low parts), M V [64][vdim] fp32, the chunk's decay [dim].
+struct DeltaItem {
+  __nv_bfloat16 *w, *k, *q, *a;
+  float *u, *decay;
+};
+__host__ __device__ __forceinline__ long long delta_item_floats(int dim, int vdim) {
+  return 3ll * kChunk * dim + kChunk * kChunk + static_cast<long long>(kChunk) * vdim + dim;
+}
+__device__ __forceinline__ DeltaItem delta_item(const nfk_delta_params& p, int item, int head) {
+  float* f = p.scratch + (static_cast<long long>(item) * p.heads + head) * delta_item_floats(p.dim, p.vdim);
+  DeltaItem d;
+  d.w = reinterpret_cast<__nv_bfloat16*>(f);
+  d.k = d.w + 2 * kChunk * p.dim;
+  d.q = d.k + 2 * kChunk * p.dim;
+  d.a = d.q + 2 * kChunk * p.dim;
+  d.u = f + 3 * kChunk * p.dim + kChunk * kChunk;
+  d.decay = d.u + kChunk * p.vdim;
+  return d;
+}
+__device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(x, y);
+  const float2 h = unpack_bf16x2(hi);
+  lo = pack_bf16x2(x - h.x, y - h.y);
+}
+__device__ __forceinline__ void cp_async16_or_zero(void* smem_dst, const void* src, bool ok) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+
+template <int P>
+struct DeltaChunkCfg {
+  static constexpr int BLD = P + 8;                      // bf16 row stride: conflict-free ldmatrix
+  static constexpr int FLD = P + 4;                      // fp32 row stride
+  static constexpr int MLD = kChunk + 8, XLD = kChunk + 1;
+  static constexpr int ROWS = kChunk * BLD * 2;
+  static constexpr int CE = kChunk * FLD * 4, TOT = kRuns * P * 4, M = kChunk * MLD * 2, X = kChunk * XLD * 4;
+  // q | k | v | decayed keys (pair) | log decays | their sums | N | X | Y | M (pair) | factors
+  static constexpr int SMEM = 5 * ROWS + CE + TOT + 2 * X + 16 * kChunk * 4 + 2 * M + 3 * kChunk * 4 + 16;
+};
+
+template <int P>
+__global__ void __launch_bounds__(kDcThreads, 1)
+delta_chunk_kernel(nfk_delta_params p) {
+  using C = DeltaChunkCfg<P>;
+  extern __shared__ __align__(16) uint8_t smem[];
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
+  __nv_bfloat16* k_s = q_s + kChunk * C::BLD;
+  __nv_bfloat16* v_s = k_s + kChunk * C::BLD;
+  __nv_bfloat16* kh_s = v_s + kChunk * C::BLD;
+  __nv_bfloat16* kl_s = kh_s + kChunk * C::BLD;
+  float* ce = reinterpret_cast<float*>(kl_s + kChunk * C::BLD);     // log2 decays through a token, from its run's start
+  float* tot = ce + kChunk * C::FLD;                                 // ... of whole runs
+  float* n_s = tot + kRuns * P;                                      // diag(beta) <k, k>, strictly lower
+  float* x_s = n_s + kChunk * C::XLD;                                // its (1 + N)^-1
+  float* y_s = x_s + kChunk * C::XLD;                                // [16][64]
+  __nv_bfloat16* mh_s = reinterpret_cast<__nv_bfloat16*>(y_s + 16 * kChunk);
+  __nv_bfloat16* ml_s = mh_s + kChunk * C::MLD;
+  float* qn_s = reinterpret_cast<float*>(ml_s + kChunk * C::MLD);    // factors that make queries and keys unit vectors
+  float* kn_s = qn_s + kChunk;
+  float* beta_s = kn_s + kChunk;
+  int* slow_s = reinterpret_cast<int*>(beta_s + kChunk);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int head = blockIdx.x % p.heads, item = blockIdx.x / p.heads, kvh = head / (p.heads / p.kv_heads);
+  const int n = p.items[item * 4 + 2];
+  const long long tok0 = p.items[item * 4 + 1];
+  const DeltaItem out = delta_item(p, item, head);
+
+  // ---- operands: all requested before any of them is waited for ----
+  {
+    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.qkv);
+    constexpr int CH = P / 8;
+    const int off[3] = {p.q_off + kvh * p.dim, p.k_off + kvh * p.dim, p.v_off + head * p.vdim};
+#pragma unroll
+    for (int a = 0; a < 3; ++a)
+#pragma unroll
+      for (int i = threadIdx.x; i < kChunk * CH; i += kDcThreads) {
+        const int r = i / CH, c = (i % CH) * 8;
+        const bool ok = r < n && c < (a == 2 ? p.vdim : p.dim);
+        cp_async16_or_zero(q_s + a * kChunk * C::BLD + r * C::BLD + c, src + (ok ? (tok0 + r) * p.ld + off[a] + c : 0), ok);
+      }
+    cp_async_commit();
+  }
+  const float rate = p.rate[head] * kLog2e;
+  for (int i = threadIdx.x; i < kChunk * (P / 4); i += kDcThreads) {
+    const int r = i / (P / 4), c = (i % (P / 4)) * 4;
+    float4 l = make_float4(0.f, 0.f, 0.f, 0.f);           // no decay past the last token: the chunk's is that of its tokens
+    if (r < n && c < p.dim) {
+      const float4 x = load4(p.x + (tok0 + r) * p.ld_x + head * p.dim + c), b = load4(p.dt_bias + head * p.dim + c);
+      l = make_float4(-fminf(rate * softplus_f(x.x + b.x), kMaxDecayLog2), -fminf(rate * softplus_f(x.y + b.y), kMaxDecayLog2),
+                      -fminf(rate * softplus_f(x.z + b.z), kMaxDecayLog2), -fminf(rate * softplus_f(x.w + b.w), kMaxDecayLog2));
+    }
+    store4(ce + r * C::FLD + c, l);
+  }
+  for (int i = threadIdx.x; i < kChunk * C::XLD; i += kDcThreads) x_s[i] = n_s[i] = 0.f;
+  if (threadIdx.x < kRuns) slow_s[threadIdx.x] = 0;
+  cp_async_wait<0>();
+  __syncthreads();
+
+  // ---- sums of log decays, norms, step sizes ----
+  for (int i = threadIdx.x; i < kRuns * P; i += kDcThreads) {
+    const int run = i / P, d = i % P;
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < kRun; ++j) {
+      s += ce[(run * kRun + j) * C::FLD + d];
+      ce[(run * kRun + j) * C::FLD + d] = s;
+    }
+    tot[i] = s;
+    if (s < -kMaxRunLog2) slow_s[run] = 1;
+  }
+#pragma unroll
+  for (int j = 0; j < kChunk / 16; ++j) {
+    const int t = warp * (kChunk / 16) + j;
+    float sq = 0.f, sk = 0.f;
+    for (int d = lane * 2; d < P; d += 64) {
+      const float2 a = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(q_s + t * C::BLD + d));
+      const float2 b = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + t * C::BLD + d));
+      sq += a.x * a.x + a.y * a.y;
+      sk += b.x * b.x + b.y * b.y;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) {
+      qn_s[t] = rsqrtf(sq + p.unit_eps) * p.q_scale;
+      kn_s[t] = rsqrtf(sk + p.unit_eps);
+      beta_s[t] = t < n ? sigmoid_f(p.beta[(tok0 + t) * p.ld_b + head]) : 0.f;
+    }
+  }
+  __syncthreads();
+
+  // ---- keys decayed to the end of their run ----
+  for (int i = threadIdx.x; i < kChunk * (P / 2); i += kDcThreads) {
+    const int t = i / (P / 2), d = (i % (P / 2)) * 2;
+    const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + t * C::BLD + d));
+    const float2 e = *reinterpret_cast<const float2*>(tot + (t / kRun) * P + d);
+    const float2 c = *reinterpret_cast<const float2*>(ce + t * C::FLD + d);
+    const float f = kn_s[t];
+    uint32_t hi, lo;
+    split_pair(k.x * f * fast_exp2(e.x - c.x), k.y * f * fast_exp2(e.y - c.y), hi, lo);
+    *reinterpret_cast<uint32_t*>(kh_s + t * C::BLD + d) = hi;
+    *reinterpret_cast<uint32_t*>(kl_s + t * C::BLD + d) = lo;
+  }
+  __syncthreads();
+
+  // ---- scores of (row run a, key run b <= a), rows of queries and rows of keys ----
+  const int mm = lane >> 3, rr = lane & 7;
+  const uint32_t khb = smem_u32(kh_s), klb = smem_u32(kl_s);
+  for (int task = warp; task < kRuns * (kRuns + 1); task += kDcThreads / 32) {
+    const bool keys = (task & 1) != 0;
+    int b = task >> 1, a = 0;                              // the pair's number -> (a, b)
+    while (b > a) {
+      ++a;
+      b -= a;
+    }
+    const __nv_bfloat16* rows = keys ? k_s : q_s;
+    const float* norm = keys ? kn_s : qn_s;
+    const int t0 = a * kRun + (lane >> 2), t1 = t0 + 8;
+    const float f0 = norm[t0], f1 = norm[t1];
+    float sc[2][4];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+    if (a == b && slow_s[a] != 0) {
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int t = e < 2 ? t0 : t1, s = b * kRun + j * 8 + (lane & 3) * 2 + (e & 1);
+          if (s > t) continue;
+          float x = 0.f;
+          for (int d = 0; d < P; ++d)
+            x += to_f32(rows[t * C::BLD + d]) * to_f32(k_s[s * C::BLD + d]) * fast_exp2(ce[t * C::FLD + d] - ce[s * C::FLD + d]);
+          sc[j][e] = x * (e < 2 ? f0 : f1) * kn_s[s];
+        }
+    } else {
+#pragma unroll 2
+      for (int ks = 0; ks < P / 16; ++ks) {
+        uint32_t rh[4], rl[4];
+#pragma unroll
+        for (int dh = 0; dh < 2; ++dh) {
+          const int d = ks * 16 + dh * 8 + (lane & 3) * 2;
+          // log decays of the runs between; within a run: what takes the row back from the run's end
+          float2 cum = make_float2(0.f, 0.f);
+          if (a == b) {
+            const float2 x = *reinterpret_cast<const float2*>(tot + a * P + d);
+            cum = make_float2(-x.x, -x.y);
+          }
+          for (int j = b + 1; j < a; ++j) {
+            const float2 x = *reinterpret_cast<const float2*>(tot + j * P + d);
+            cum.x += x.x;
+            cum.y += x.y;
+          }
+          const float2 r0 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(rows + t0 * C::BLD + d));
+          const float2 r1 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(rows + t1 * C::BLD + d));
+          const float2 c0 = *reinterpret_cast<const float2*>(ce + t0 * C::FLD + d);
+          const float2 c1 = *reinterpret_cast<const float2*>(ce + t1 * C::FLD + d);
+          split_pair(r0.x * f0 * fast_exp2(c0.x + cum.x), r0.y * f0 * fast_exp2(c0.y + cum.y), rh[dh * 2], rl[dh * 2]);
+          split_pair(r1.x * f1 * fast_exp2(c1.x + cum.x), r1.y * f1 * fast_exp2(c1.y + cum.y), rh[dh * 2 + 1], rl[dh * 2 + 1]);
+        }
+        const uint32_t o = ((b * kRun + (mm >> 1) * 8 + rr) * C::BLD + (2 * ks + (mm & 1)) * 8) * 2;
+        uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+        ldsm_x4(khb + o, h0, h1, h2, h3);
+        ldsm_x4(klb + o, l0, l1, l2, l3);
+        mma_bf16(sc[0], rh, h0, h1);
+        mma_bf16(sc[1], rh, h2, h3);
+        mma_bf16(sc[0], rh, l0, l1);
+        mma_bf16(sc[1], rh, l2, l3);
+        mma_bf16(sc[0], rl, h0, h1);
+        mma_bf16(sc[1], rl, h2, h3);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int t = h == 0 ? t0 : t1, s = b * kRun + j * 8 + (lane & 3) * 2;
+        const float x = sc[j][2 * h], y = sc[j][2 * h + 1];
+        if (keys) {
+          n_s[t * C::XLD + s] = s < t ? beta_s[t] * x : 0.f;
+          n_s[t * C::XLD + s + 1] = s + 1 < t ? beta_s[t] * y : 0.f;
+        } else {
+          uint32_t hi, lo;
+          split_pair(s <= t ? x : 0.f, s + 1 <= t ? y : 0.f, hi, lo);
+          *reinterpret_cast<uint32_t*>(out.a + t * kChunk + s) = hi;
+          *reinterpret_cast<uint32_t*>(out.a + kChunk * kChunk + t * kChunk + s) = lo;
+        }
+      }
+  }
+  __syncthreads();
+
+  // ---- X = (1 + N)^-1: blocks on the diagonal column by column, then the rows of blocks below ----
+  if (threadIdx.x < kChunk) {
+    const int b0 = (threadIdx.x / kRun) * kRun, c = threadIdx.x % kRun;
+    float x[kRun];
+#pragma unroll
+    for (int i = 0; i < kRun; ++i) {
+      float s = i == c ? 1.f : 0.f;
+#pragma unroll
+      for (int j = 0; j < i; ++j) s -= n_s[(b0 + i) * C::XLD + b0 + j] * x[j];
+      x[i] = i < c ? 0.f : s;
+      x_s[(b0 + i) * C::XLD + b0 + c] = x[i];
+    }
+  }
+  __syncthreads();
+  for (int a = 1; a < kRuns; ++a) {
+    const int w = a * kRun;
+    for (int i = threadIdx.x; i < kRun * w; i += kDcThreads) {
+      const int r = i / w, c = i % w;
+      float s = 0.f;
+      for (int j = c / kRun * kRun; j < w; ++j) s += n_s[(w + r) * C::XLD + j] * x_s[j * C::XLD + c];
+      y_s[r * kChunk + c] = s;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < kRun * w; i += kDcThreads) {
+      const int r = i / w, c = i % w;
+      float s = 0.f;
+      for (int j = 0; j <= r; ++j) s -= x_s[(w + r) * C::XLD + w + j] * y_s[j * kChunk + c];
+      x_s[(w + r) * C::XLD + c] = s;
+    }
+    __syncthreads();
+  }
+
+  // ---- M, and what the second kernel reads: keys decayed to the chunk's end, queries decayed from its start; keys
+  // decayed from its start take the place of those above ----
+  for (int i = threadIdx.x; i < kChunk * kChunk / 2; i += kDcThreads) {
+    const int t = i / (kChunk / 2), s = (i % (kChunk / 2)) * 2;
+    uint32_t hi, lo;
+    split_pair(x_s[t * C::XLD + s] * beta_s[s], x_s[t * C::XLD + s + 1] * beta_s[s + 1], hi, lo);
+    *reinterpret_cast<uint32_t*>(mh_s + t * C::MLD + s) = hi;
+    *reinterpret_cast<uint32_t*>(ml_s + t * C::MLD + s) = lo;
+  }
+  for (int i = threadIdx.x; i < kChunk * (P / 2); i += kDcThreads) {
+    const int t = i / (P / 2), d = (i % (P / 2)) * 2, run = t / kRun;
+    const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + t * C::BLD + d));
+    const float2 q = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(q_s + t * C::BLD + d));
+    float2 c = *reinterpret_cast<const float2*>(ce + t * C::FLD + d), after = make_float2(-c.x, -c.y);
+#pragma unroll
+    for (int j = 0; j < kRuns; ++j) {
+      const float2 x = *reinterpret_cast<const float2*>(tot + j * P + d);
+      if (j < run) {
+        c.x += x.x;
+        c.y += x.y;
+      } else {
+        after.x += x.x;
+        after.y += x.y;
+      }
+    }
+    const float kf = kn_s[t], qf = qn_s[t], ex = fast_exp2(c.x), ey = fast_exp2(c.y);
+    uint32_t hi, lo;
+    split_pair(k.x * kf * ex, k.y * kf * ey, hi, lo);
+    *reinterpret_cast<uint32_t*>(kh_s + t * C::BLD + d) = hi;
+    *reinterpret_cast<uint32_t*>(kl_s + t * C::BLD + d) = lo;
+    if (d < p.dim) {
+      const int o = t * p.dim + d, low = kChunk * p.dim;
+      split_pair(q.x * qf * ex, q.y * qf * ey, hi, lo);
+      *reinterpret_cast<uint32_t*>(out.q + o) = hi;
+      *reinterpret_cast<uint32_t*>(out.q + low + o) = lo;
+      split_pair(k.x * kf * fast_exp2(after.x), k.y * kf * fast_exp2(after.y), hi, lo);
+      *reinterpret_cast<uint32_t*>(out.k + o) = hi;
+      *reinterpret_cast<uint32_t*>(out.k + low + o) = lo;
+    }
+  }
+  for (int d = threadIdx.x; d < p.dim; d += kDcThreads)
+    out.decay[d] = fast_exp2((tot[d] + tot[P + d]) + (tot[2 * P + d] + tot[3 * P + d]));
+  __syncthreads();
+
+  // ---- M V and W = M (decayed keys): a warp takes a run of rows and a quarter of the columns ----
+  constexpr int NT = P / 8 / 4;
+  const int a = warp & 3, n0 = (warp >> 2) * NT;
+  float u[NT][4], w[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    u[i][0] = u[i][1] = u[i][2] = u[i][3] = 0.f;
+    w[i][0] = w[i][1] = w[i][2] = w[i][3] = 0.f;
+  }
+  const uint32_t vb = smem_u32(v_s), mhb = smem_u32(mh_s), mlb = smem_u32(ml_s);
+  for (int ks = 0; ks <= a; ++ks) {
+    uint32_t mh[4], ml[4];
+    const uint32_t mo = ((a * kRun + (lane & 15)) * C::MLD + ks * 16 + (lane >> 4) * 8) * 2;
+    ldsm_x4(mhb + mo, mh[0], mh[1], mh[2], mh[3]);
+    ldsm_x4(mlb + mo, ml[0], ml[1], ml[2], ml[3]);
+#pragma unroll
+    for (int i = 0; i < NT; i += 2) {
+      const uint32_t o = ((ks * 16 + (mm & 1) * 8 + rr) * C::BLD + (n0 + i + (mm >> 1)) * 8) * 2;
+      uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+      ldsm_x4_trans(vb + o, h0, h1, h2, h3);
+      mma_bf16(u[i], mh, h0, h1);
+      mma_bf16(u[i + 1], mh, h2, h3);
+      mma_bf16(u[i], ml, h0, h1);
+      mma_bf16(u[i + 1], ml, h2, h3);
+      ldsm_x4_trans(khb + o, h0, h1, h2, h3);
+      ldsm_x4_trans(klb + o, l0, l1, l2, l3);
+      mma_bf16(w[i], mh, h0, h1);
+      mma_bf16(w[i + 1], mh, h2, h3);
+      mma_bf16(w[i], mh, l0, l1);
+      mma_bf16(w[i + 1], mh, l2, l3);
+      mma_bf16(w[i], ml, h0, h1);
+      mma_bf16(w[i + 1], ml, h2, h3);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int t = a * kRun + (lane >> 2) + h * 8, c = (n0 + i) * 8 + (lane & 3) * 2;
+      if (c < p.vdim) *reinterpret_cast<float2*>(out.u + t * p.vdim + c) = make_float2(u[i][2 * h], u[i][2 * h + 1]);
+      if (c < p.dim) {
+        uint32_t hi, lo;
+        split_pair(w[i][2 * h], w[i][2 * h + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(out.w + t * p.dim + c) = hi;
+        *reinterpret_cast<uint32_t*>(out.w + kChunk * p.dim + t * p.dim + c) = lo;
+      }
+    }
+}
+
+template <int P>
+struct DeltaScanCfg {
+  static constexpr int BLD = P + 8, MLD = kChunk + 8, SLD = kSlice + 8, ULD = kSlice + 4;
+  static constexpr int ROWS = kChunk * BLD * 2, A = kChunk * MLD * 2, S = P * SLD * 2, U = kChunk * SLD * 2;
+  // W, K, Q (pairs) | A (pair) | M V | S (pair) | u (pair) | decay
+  static constexpr int SMEM = 6 * ROWS + 2 * A + kChunk * ULD * 4 + 2 * S + 2 * U + P * 4;
+};
+
+template <int P>
+__global__ void __launch_bounds__(kDsThreads, 1)
+delta_scan_kernel(nfk_delta_params p, int slices) {
+  using C = DeltaScanCfg<P>;
+  extern __shared__ __align__(16) uint8_t smem[];
+  __nv_bfloat16* w_s = reinterpret_cast<__nv_bfloat16*>(smem);
+  __nv_bfloat16* k_s = w_s + 2 * kChunk * C::BLD;
+  __nv_bfloat16* q_s = k_s + 2 * kChunk * C::BLD;
+  __nv_bfloat16* a_s = q_s + 2 * kChunk * C::BLD;
+  float* mv_s = reinterpret_cast<float*>(a_s + 2 * kChunk * C::MLD);
+  __nv_bfloat16* s_s = reinterpret_cast<__nv_bfloat16*>(mv_s + kChunk * C::ULD);
+  __nv_bfloat16* u_s = s_s + 2 * P * C::SLD;
+  float* decay_s = reinterpret_cast<float*>(u_s + 2 * kChunk * C::SLD);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int v0 = (blockIdx.x % slices) * kSlice, head = (blockIdx.x / slices) % p.heads, item0 = blockIdx.x / (slices * p.heads);
+  if (p.items[item0 * 4 + 3] != 0) return;                 // not the first chunk of a portion
+  const int req = p.items[item0 * 4];
+  const DeltaState st = delta_state(p, req, head);
+  if (!st.ok) return;
+  const int n_tok = p.qo_indptr[req + 1] - p.qo_indptr[req];
+  const int chunks = min((n_tok + kChunk - 1) / kChunk, p.num_items - item0);
+  const long long tok0 = p.qo_indptr[req];
+
+  // rows of `cols` elements as 16-byte pieces; columns past `have` become zeros
+  auto copy = [&](void* dst, int dst_row_bytes, const void* src, int src_row_bytes, int rows, int row_bytes, int have_bytes) {
+    const int per = row_bytes / 16;
+    for (int i = threadIdx.x; i < rows * per; i += kDsThreads) {
+      const int r = i / per, b = (i % per) * 16;
+      const bool ok = b < have_bytes;
+      cp_async16_or_zero(static_cast<char*>(dst) + r * dst_row_bytes + b,
+                         static_cast<const char*>(src) + static_cast<long long>(r) * src_row_bytes + (ok ? b : 0), ok);
+    }
+  };
+  auto fetch_first = [&](int c) {                          // what the values written need
+    const DeltaItem d = delta_item(p, item0 + c, head);
+    copy(w_s, C::BLD * 2, d.w, p.dim * 2, 2 * kChunk, P * 2, p.dim * 2);
+    copy(mv_s, C::ULD * 4, d.u + v0, p.vdim * 4, kChunk, kSlice * 4, (p.vdim - v0) * 4);
+    cp_async_commit();
+  };
+  auto fetch_rest = [&](int c) {
+    const DeltaItem d = delta_item(p, item0 + c, head);
+    copy(k_s, C::BLD * 2, d.k, p.dim * 2, 2 * kChunk, P * 2, p.dim * 2);
+    copy(q_s, C::BLD * 2, d.q, p.dim * 2, 2 * kChunk, P * 2, p.dim * 2);
+    copy(a_s, C::MLD * 2, d.a, kChunk * 2, 2 * kChunk, kChunk * 2, kChunk * 2);
+    copy(decay_s, P * 4, d.decay, p.dim * 4, 1, P * 4, p.dim * 4);
+    cp_async_commit();
+  };
+  fetch_first(0);
+  fetch_rest(0);
+
+  // ---- S: warps over 16-row tiles of the key channels and, for the small size, halves of the columns ----
+  constexpr int MT = P / 16, SN = kSlice / 8 * MT / 8;     // row tiles; column blocks per warp
+  const int sm0 = (warp % MT) * 16, sn0 = (warp / MT) * SN;
+  const int d0 = sm0 + (lane >> 2), d1 = d0 + 8;
+  float S[SN][4];
+#pragma unroll
+  for (int i = 0; i < SN; ++i) {
+    const int c = (sn0 + i) * 8 + (lane & 3) * 2;
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int d = h == 0 ? d0 : d1;
+      const bool ok = !st.fresh && d < p.dim && v0 + c < p.vdim;
+      const float2 x = ok ? *reinterpret_cast<const float2*>(st.S + static_cast<long long>(d) * p.vdim + v0 + c) : make_float2(0.f, 0.f);
+      S[i][2 * h] = x.x;
+      S[i][2 * h + 1] = x.y;
+    }
+  }
+  auto publish = [&]() {
+#pragma unroll
+    for (int i = 0; i < SN; ++i)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int o = (h == 0 ? d0 : d1) * C::SLD + (sn0 + i) * 8 + (lane & 3) * 2;
+        uint32_t hi, lo;
+        split_pair(S[i][2 * h], S[i][2 * h + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(s_s + o) = hi;
+        *reinterpret_cast<uint32_t*>(s_s + P * C::SLD + o) = lo;
+      }
+  };
+  publish();
+
+  const int mm = lane >> 3, rr = lane & 7;
+  const int a = warp & 3, c0 = (warp >> 2) * 16;           // this warp's run of rows and half of the columns
+  const int t0 = a * kRun + (lane >> 2);
+  const uint32_t wb = smem_u32(w_s), kb = smem_u32(k_s), qb = smem_u32(q_s), ab = smem_u32(a_s), sb = smem_u32(s_s), ub = smem_u32(u_s);
+  constexpr uint32_t R_LO = kChunk * C::BLD * 2, A_LO = kChunk * C::MLD * 2, S_LO = P * C::SLD * 2, U_LO = kChunk * C::SLD * 2;
+  // acc += rows (pair, of this warp's run) x S (pair, this warp's half of the columns)
+  auto rows_times_s = [&](float (&acc)[2][4], uint32_t base) {
+#pragma unroll
+    for (int ks = 0; ks < P / 16; ++ks) {
+      uint32_t rh[4], rl[4], h0, h1, h2, h3, l0, l1, l2, l3;
+      const uint32_t ro = ((a * kRun + (lane & 15)) * C::BLD + ks * 16 + (lane >> 4) * 8) * 2;
+      ldsm_x4(base + ro, rh[0], rh[1], rh[2], rh[3]);
+      ldsm_x4(base + R_LO + ro, rl[0], rl[1], rl[2], rl[3]);
+      const uint32_t so = ((ks * 16 + (mm & 1) * 8 + rr) * C::SLD + c0 + (mm >> 1) * 8) * 2;
+      ldsm_x4_trans(sb + so, h0, h1, h2, h3);
+      ldsm_x4_trans(sb + S_LO + so, l0, l1, l2, l3);
+      mma_bf16(acc[0], rh, h0, h1);
+      mma_bf16(acc[1], rh, h2, h3);
+      mma_bf16(acc[0], rh, l0, l1);
+      mma_bf16(acc[1], rh, l2, l3);
+      mma_bf16(acc[0], rl, h0, h1);
+      mma_bf16(acc[1], rl, h2, h3);
+    }
+  };
+
+  for (int c = 0; c < chunks; ++c) {
+    cp_async_wait<1>();
+    __syncthreads();                                       // W and M V are there, S is published
+    float acc[2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    rows_times_s(acc, wb);
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int t = t0 + h * 8, col = c0 + i * 8 + (lane & 3) * 2;
+        const float2 m = *reinterpret_cast<const float2*>(mv_s + t * C::ULD + col);
+        uint32_t hi, lo;
+        split_pair(m.x - acc[i][2 * h], m.y - acc[i][2 * h + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(u_s + t * C::SLD + col) = hi;
+        *reinterpret_cast<uint32_t*>(u_s + kChunk * C::SLD + t * C::SLD + col) = lo;
+      }
+    cp_async_wait<0>();
+    __syncthreads();                                       // the rest is there, u is written, W and M V are read
+    if (c + 1 < chunks) fetch_first(c + 1);
+    else cp_async_commit();
+    // ---- outputs ----
+#pragma unroll
+    for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    rows_times_s(acc, qb);
+#pragma unroll
+    for (int ks = 0; ks < kRuns; ++ks) {
+      if (ks > a) continue;
+      uint32_t ah[4], al[4], h0, h1, h2, h3, l0, l1, l2, l3;
+      const uint32_t ao = ((a * kRun + (lane & 15)) * C::MLD + ks * 16 + (lane >> 4) * 8) * 2;
+      ldsm_x4(ab + ao, ah[0], ah[1], ah[2], ah[3]);
+      ldsm_x4(ab + A_LO + ao, al[0], al[1], al[2], al[3]);
+      const uint32_t uo = ((ks * 16 + (mm & 1) * 8 + rr) * C::SLD + c0 + (mm >> 1) * 8) * 2;
+      ldsm_x4_trans(ub + uo, h0, h1, h2, h3);
+      ldsm_x4_trans(ub + U_LO + uo, l0, l1, l2, l3);
+      mma_bf16(acc[0], ah, h0, h1);
+      mma_bf16(acc[1], ah, h2, h3);
+      mma_bf16(acc[0], ah, l0, l1);
+      mma_bf16(acc[1], ah, l2, l3);
+      mma_bf16(acc[0], al, h0, h1);
+      mma_bf16(acc[1], al, h2, h3);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int t = c * kChunk + t0 + h * 8, col = v0 + c0 + i * 8 + (lane & 3) * 2;
+        if (t < n_tok && col < p.vdim)
+          *reinterpret_cast<float2*>(p.o + ((tok0 + t) * p.heads + head) * p.vdim + col) = make_float2(acc[i][2 * h], acc[i][2 * h + 1]);
+      }
+    // ---- the next state ----
+    const float e0 = decay_s[d0], e1 = decay_s[d1];
+#pragma unroll
+    for (int i = 0; i < SN; ++i) {
+      S[i][0] *= e0;
+      S[i][1] *= e0;
+      S[i][2] *= e1;
+      S[i][3] *= e1;
+    }
+#pragma unroll
+    for (int ks = 0; ks < kRuns; ++ks) {
+      uint32_t kh[4], kl[4];                               // transposed: rows are key channels
+      const uint32_t ko = ((ks * 16 + (mm >> 1) * 8 + rr) * C::BLD + sm0 + (mm & 1) * 8) * 2;
+      ldsm_x4_trans(kb + ko, kh[0], kh[1], kh[2], kh[3]);
+      ldsm_x4_trans(kb + R_LO + ko, kl[0], kl[1], kl[2], kl[3]);
+#pragma unroll
+      for (int i = 0; i < SN; i += 2) {
+        uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+        const uint32_t uo = ((ks * 16 + (mm & 1) * 8 + rr) * C::SLD + (sn0 + i + (mm >> 1)) * 8) * 2;
+        ldsm_x4_trans(ub + uo, h0, h1, h2, h3);
+        ldsm_x4_trans(ub + U_LO + uo, l0, l1, l2, l3);
+        mma_bf16(S[i], kh, h0, h1);
+        mma_bf16(S[i + 1], kh, h2, h3);
+        mma_bf16(S[i], kh, l0, l1);
+        mma_bf16(S[i + 1], kh, l2, l3);
+        mma_bf16(S[i], kl, h0, h1);
+        mma_bf16(S[i + 1], kl, h2, h3);
+      }
+    }
+    __syncthreads();                                       // S, u and the copies are read
+    publish();
+    if (c + 1 < chunks) fetch_rest(c + 1);
+    else cp_async_commit();
+  }
+  cp_async_wait<0>();
+#pragma unroll
+  for (int i = 0; i < SN; ++i) {
+    const int c = v0 + (sn0 + i) * 8 + (lane & 3) * 2;
+    if (c >= p.vdim) continue;
+    if (d0 < p.dim) *reinterpret_cast<float2*>(st.S + static_cast<long long>(d0) * p.vdim + c) = make_float2(S[i][0], S[i][1]);
+    if (d1 < p.dim) *reinterpret_cast<float2*>(st.S + static_cast<long long>(d1) * p.vdim + c) = make_float2(S[i][2], S[i][3]);
   }
 }
 
@@ -295,7 +879,27 @@ int launch_delta_seq(const nfk_delta_params& p, cudaStream_t stream) {
   if (rc != NF_OK) return rc;
   delta_seq_kernel<T><<<static_cast<int>(grid), 256, sm, stream>>>(p, v_slices);
   if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
-  delta_seq_norm_kernel<T><<<dim3(64, p.num_seq), 256, 0, stream>>>(p);
+  delta_norm_kernel<T, false><<<dim3(64, p.num_seq), 256, 0, stream>>>(p);
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+template <int P>
+int launch_delta_chunks(const nfk_delta_params& p, cudaStream_t stream) {
+  static bool attr_dev[kMaxDevices] = {false};
+  bool& attr = attr_dev[device_slot()];
+  if (!attr) {
+    int rc = set_smem(delta_chunk_kernel<P>, DeltaChunkCfg<P>::SMEM);
+    if (rc == NF_OK) rc = set_smem(delta_scan_kernel<P>, DeltaScanCfg<P>::SMEM);
+    if (rc != NF_OK) return rc;
+    attr = true;
+  }
+  const int grid = p.num_items * p.heads, slices = (p.vdim + kSlice - 1) / kSlice;
+  delta_chunk_kernel<P><<<grid, kDcThreads, DeltaChunkCfg<P>::SMEM, stream>>>(p);
+  if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
+  delta_scan_kernel<P><<<grid * slices, kDsThreads, DeltaScanCfg<P>::SMEM, stream>>>(p, slices);
+  if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
+  const int per = kChunk * p.heads / 8;
+  delta_norm_kernel<__nv_bfloat16, true><<<dim3(per < 64 ? (per > 0 ? per : 1) : 64, p.num_items), 256, 0, stream>>>(p);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 
@@ -327,7 +931,19 @@ extern "C" int nfk_delta_prefill(const nfk_delta_params* p, cudaStream_t stream)
   using namespace nf;
   const int rc = check_delta(p);
   if (rc != NF_OK) return rc;
-  if (p->num_seq < 0 || (p->num_seq > 0 && (!p->seq_reqs || !p->o))) return NF_ERR_BAD_ARG;
+  if (p->num_seq < 0 || p->num_items < 0 || p->num_items > 65535 || (p->num_seq > 0 && !p->seq_reqs) ||
+      (p->num_items > 0 && !p->items) || (p->num_seq + p->num_items > 0 && !p->o))
+    return NF_ERR_BAD_ARG;
+  if (p->num_items > 0) {
+    if (p->dtype != NFK_BF16 || p->dim > 128 || p->vdim > 128) return NF_ERR_UNSUPPORTED;
+    if (p->scratch == nullptr || (reinterpret_cast<uintptr_t>(p->scratch) & 15) != 0 ||
+        p->num_items * static_cast<long long>(p->heads) * delta_item_floats(p->dim, p->vdim) > p->scratch_floats)
+      return NF_ERR_BAD_ARG;
+    const int rc2 = p->dim <= 64 && p->vdim <= 64 ? launch_delta_chunks<64>(*p, stream) : launch_delta_chunks<128>(*p, stream);
+    if (rc2 != NF_OK) return rc2;
+  }
   if (p->num_seq == 0) return NF_OK;
   return p->dtype == NFK_F32 ? launch_delta_seq<float>(*p, stream) : launch_delta_seq<__nv_bfloat16>(*p, stream);
 }
+
+extern "C" long long nfk_delta_item_floats(int dim, int vdim) { return nf::delta_item_floats(dim, vdim); }

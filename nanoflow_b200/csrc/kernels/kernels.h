@@ -463,14 +463,24 @@ typedef struct nfk_talk_attn_params {
   const float* talk;         // [heads][heads]
   const float* v_rot;        // null: none
   int v_pairs, v_ld;
-  int token_begin, n_tokens; // simple kernel
+  int token_begin, n_tokens;
   int heads, kv_heads, hd, page_size, num_pages, window;   // window 0: none
   float scale;
   int dtype;
   unsigned int* status;
+  int max_keys;              // decode: most keys that a token sees
+  const int* items;          // prefill: [num_items][3] (request, first token, tokens: at most 16)
+  int num_items;
 } nfk_talk_attn_params;
-// Any sizes (shared memory for a few rows of all heads permitting), bf16 or fp32: one CTA per token.
+// Tokens [token_begin, token_begin + n_tokens), any sizes (shared memory for a few rows of all heads permitting), bf16 or
+// fp32: one CTA per token.
 int nfk_talk_attn(const nfk_talk_attn_params* p, cudaStream_t stream);
+// bf16, hd 64 or 128, at most 64 heads. Tokens [token_begin, token_begin + n_tokens), a cluster of CTAs each:
+int nfk_talk_attn_decode(const nfk_talk_attn_params* p, cudaStream_t stream);
+// ... and portions on tensor cores; `talk` enters the products in bf16.
+int nfk_talk_attn_prefill(const nfk_talk_attn_params* p, cudaStream_t stream);
+// Which of the two take these sizes: 1 = prefill, 2 = decode (for max_keys keys), added up.
+int nfk_talk_attn_fits(int heads, int kv_heads, int hd, int max_keys);
 
 // ------------------------------------------------------------------------------------------------
 // Short convolution over time (short_conv.cu)
@@ -556,12 +566,19 @@ typedef struct nfk_delta_params {
   int heads, kv_heads, dim, vdim, vdim_real, num_slots;    // dim, vdim: padded to multiples of 8 (padding columns are zero)
   float q_scale, unit_eps, eps;
   int dtype;
-  // prefill, token by token: seq_reqs [num_seq] requests, o: fp32 [T, heads * vdim] of scratch rows
+  // prefill. o: fp32 [T, heads * vdim] of scratch rows. Token by token: seq_reqs [num_seq] requests. In chunks of 64 tokens
+  // (bf16, dim and vdim up to 128): items [num_items][4] (request, first token, tokens, chunk of the request's portion), a
+  // request's chunks one after the other, and scratch: num_items * heads * nfk_delta_item_floats(dim, vdim) floats.
   const int* seq_reqs;
   int num_seq;
   float* o;
+  const int* items;
+  int num_items;
+  float* scratch;
+  long long scratch_floats;
   unsigned int* status;
 } nfk_delta_params;
+long long nfk_delta_item_floats(int dim, int vdim);
 int nfk_delta_decode(const nfk_delta_params* p, cudaStream_t stream);
 int nfk_delta_prefill(const nfk_delta_params* p, cudaStream_t stream);
 

@@ -2,9 +2,22 @@
 // denominator) the weights of all heads are mixed by a matrix before they meet the values (Shazeer et al., "Talking-Heads
 // Attention"; see kernels.h). Scores, weights, mixing and the turn of the outputs are fp32.
 //
-// nfk_talk_attn   any sizes, bf16 or fp32: one CTA per token, all heads. Two passes over the keys, because the mixing
-//                 needs every head's normalised weights: maxima and sums first, then weights, mixing and values.
+// The mixing needs every head's normalised weights, so maxima and sums come first, then weights, mixing and values.
+//
+// nfk_talk_attn          any sizes, bf16 or fp32: one CTA per token, all heads, two passes over the keys.
+// nfk_talk_attn_decode   one token per request (bf16): a cluster of CTAs shares the token's keys. Scores stay in shared
+//                        memory, keys and values are read once, straight into registers; maxima, sums and the partial
+//                        outputs are exchanged through distributed shared memory.
+// nfk_talk_attn_prefill  portions (bf16): a cluster takes 16 tokens, each of its CTAs 16 heads, one per warp. First loop
+//                        over the keys: maxima and sums; second loop: every CTA's weights go to all CTAs of the cluster,
+//                        each mixes them for its own heads (a product with the mixing matrix on tensor cores) and applies
+//                        them to the values. Weights enter the products as bf16 pairs (high and low part, about 16 bits).
+#include <cooperative_groups.h>
+
+#include "attn_mma.cuh"
 #include "elem_io.cuh"
+
+namespace cg = cooperative_groups;
 
 namespace nf {
 namespace {
@@ -119,6 +132,540 @@ talk_attn_kernel(nfk_talk_attn_params p) {
   }
 }
 
+// ---- decode ---------------------------------------------------------------------------------------------------
+constexpr int kTdThreads = 256, kTdWarps = kTdThreads / 32, kTdKeys = 32;      // keys of a warp's work item
+constexpr int kTdMaxCluster = 8;
+
+// Shared memory: rows [keys] | scores [H][keys + 4] (later weights, [keys][H4]) | (max, sum) [H] | partial outputs [H][hd].
+struct TalkDecodeLayout {
+  int keys, s_ld, h4, rows, scores, stat, out, bytes;
+};
+__host__ __device__ inline TalkDecodeLayout talk_decode_layout(int heads, int hd, int keys) {
+  TalkDecodeLayout l;
+  l.keys = (keys + kTdKeys - 1) / kTdKeys * kTdKeys;
+  l.s_ld = l.keys + 4;
+  l.h4 = (heads + 3) / 4 * 4;
+  l.rows = 0;
+  l.scores = l.rows + l.keys * 4;
+  const int s_bytes = heads * l.s_ld * 4, w_bytes = l.keys * l.h4 * 4;
+  l.stat = l.scores + s_bytes + w_bytes;
+  l.out = l.stat + (heads * 8 + 15) / 16 * 16;
+  l.bytes = l.out + heads * hd * 4;
+  return l;
+}
+
+// GV: a thread's heads per pass over the values (heads of one KV head).
+template <int HD, int GV>
+__global__ void __launch_bounds__(kTdThreads)
+talk_decode_kernel(nfk_talk_attn_params p, TalkDecodeLayout lay) {
+  extern __shared__ __align__(16) uint8_t tds[];
+  int* row_s = reinterpret_cast<int*>(tds + lay.rows);
+  float* s_s = reinterpret_cast<float*>(tds + lay.scores);
+  float* w_s = s_s + p.heads * lay.s_ld;
+  float2* stat_s = reinterpret_cast<float2*>(tds + lay.stat);
+  float* o_s = reinterpret_cast<float*>(tds + lay.out);
+  cg::cluster_group cluster = cg::this_cluster();
+  const int C = static_cast<int>(cluster.num_blocks()), rank = static_cast<int>(cluster.block_rank());
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int H = p.heads, G = p.kv_heads, group = H / G;
+  const int tok = p.token_begin + blockIdx.x / C;
+  const int pos = p.positions[tok], req = p.token_req[tok];
+  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int total = pos + 1 - lo, per = ((total + C - 1) / C + kTdKeys - 1) / kTdKeys * kTdKeys;
+  const int k0 = lo + rank * per;
+  int n = min(per, pos + 1 - k0);
+  n = n < 0 ? 0 : n;
+  if (n > lay.keys) {                            // more keys than the launcher was told
+    if (threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
+    n = lay.keys;
+  }
+  const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
+  const long long head_step = static_cast<long long>(p.page_size) * HD, v_step = G * head_step;
+  for (int k = threadIdx.x; k < lay.keys; k += kTdThreads) {
+    int r = -1;
+    if (k < n) {
+      const int page = page_of(k0 + k, req, p.page_size, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
+      if (page >= 0) r = page * 2 * G * p.page_size + (k0 + k) % p.page_size;
+    }
+    row_s[k] = r;
+  }
+  __syncthreads();
+  // ---- scores: a warp takes 32 keys of a KV head. Rows of the tiles: the KV head's query heads, 16 at a time ----
+  const int blocks = (n + kTdKeys - 1) / kTdKeys;
+  const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + static_cast<long long>(tok) * H * HD;
+  for (int item = warp; item < blocks * G; item += kTdWarps) {
+    const int kvh = item / blocks, kb = (item - kvh * blocks) * kTdKeys;
+    // a lane brings eight neighbouring columns of a key at a time, for two steps of the product: the columns of a step
+    // are those {c, c + 1, c + 2, c + 3} of every lane's eight, in queries and keys alike
+    uint4 kr[kTdKeys / 8][HD / 32];
+#pragma unroll
+    for (int t = 0; t < kTdKeys / 8; ++t) {
+      const int r = row_s[kb + t * 8 + (lane >> 2)];
+      const __nv_bfloat16* src = pool + static_cast<long long>(r < 0 ? 0 : r) * HD + kvh * head_step + (lane & 3) * 8;
+#pragma unroll
+      for (int b = 0; b < HD / 32; ++b) kr[t][b] = r < 0 ? make_uint4(0, 0, 0, 0) : *reinterpret_cast<const uint4*>(src + b * 32);
+    }
+    for (int m0 = 0; m0 < group; m0 += 16) {
+      float acc[kTdKeys / 8][4];
+#pragma unroll
+      for (int t = 0; t < kTdKeys / 8; ++t) acc[t][0] = acc[t][1] = acc[t][2] = acc[t][3] = 0.f;
+      const int r0 = m0 + (lane >> 2), r1 = r0 + 8;
+      const __nv_bfloat16* q0 = q + (kvh * group + r0) * HD + (lane & 3) * 8;
+#pragma unroll
+      for (int b = 0; b < HD / 32; ++b) {
+        const uint4 x0 = r0 < group ? *reinterpret_cast<const uint4*>(q0 + b * 32) : make_uint4(0, 0, 0, 0);
+        const uint4 x1 = r1 < group ? *reinterpret_cast<const uint4*>(q0 + 8 * HD + b * 32) : make_uint4(0, 0, 0, 0);
+        const uint32_t a0[4] = {x0.x, x1.x, x0.y, x1.y}, a1[4] = {x0.z, x1.z, x0.w, x1.w};
+#pragma unroll
+        for (int t = 0; t < kTdKeys / 8; ++t) {
+          mma_bf16(acc[t], a0, kr[t][b].x, kr[t][b].y);
+          mma_bf16(acc[t], a1, kr[t][b].z, kr[t][b].w);
+        }
+      }
+#pragma unroll
+      for (int t = 0; t < kTdKeys / 8; ++t) {
+        const int k = kb + t * 8 + (lane & 3) * 2;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const bool ok = row_s[k + e] >= 0;
+          if (r0 < group) s_s[(kvh * group + r0) * lay.s_ld + k + e] = ok ? acc[t][e] * p.scale : -INFINITY;
+          if (r1 < group) s_s[(kvh * group + r1) * lay.s_ld + k + e] = ok ? acc[t][2 + e] * p.scale : -INFINITY;
+        }
+      }
+    }
+  }
+  __syncthreads();
+  // ---- maxima and sums, of this CTA's keys and then of the token's ----
+  const int nk = blocks * kTdKeys;
+  for (int h = warp; h < H; h += kTdWarps) {
+    const float* s = s_s + h * lay.s_ld;
+    float m = -INFINITY, l = 0.f;
+    for (int k = lane; k < nk; k += 32) m = fmaxf(m, s[k]);
+    m = warp_max(m);
+    if (m != -INFINITY)
+      for (int k = lane; k < nk; k += 32) l += expf(s[k] - m);
+    l = warp_sum(l);
+    if (lane == 0) stat_s[h] = make_float2(m, l);
+  }
+  cluster.sync();
+  for (int h = warp; h < H; h += kTdWarps) {
+    const float2 st = lane < C ? *cluster.map_shared_rank(stat_s + h, lane) : make_float2(-INFINITY, 0.f);
+    const float sink = p.sinks != nullptr ? p.sinks[h] : -INFINITY;
+    const float m = fmaxf(warp_max(st.x), sink);
+    float l = st.x == -INFINITY ? 0.f : st.y * expf(st.x - m);
+    l = warp_sum(l) + (sink == -INFINITY ? 0.f : expf(sink - m));
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float* s = s_s + h * lay.s_ld;
+    for (int k = lane; k < nk; k += 32) s[k] = s[k] == -INFINITY ? 0.f : expf(s[k] - m) * inv;
+  }
+  __syncthreads();
+  // ---- mixing: a thread takes a key and four heads at a time; the result lies key by key ----
+  for (int k = threadIdx.x; k < nk; k += kTdThreads) {
+    for (int h = 0; h < lay.h4; h += 4) {
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      const float* t = p.talk + h * H;
+      const int left = H - h;
+      for (int g = 0; g < H; ++g) {
+        const float w = s_s[g * lay.s_ld + k];
+        a.x += __ldg(t + g) * w;
+        if (left > 1) a.y += __ldg(t + H + g) * w;
+        if (left > 2) a.z += __ldg(t + 2 * H + g) * w;
+        if (left > 3) a.w += __ldg(t + 3 * H + g) * w;
+      }
+      *reinterpret_cast<float4*>(w_s + k * lay.h4 + h) = a;
+    }
+  }
+  for (int c = threadIdx.x; c < H * HD; c += kTdThreads) o_s[c] = 0.f;
+  __syncthreads();
+  // ---- values: a thread takes four columns of a KV head for up to GV of its query heads; what threads are left over
+  // split the keys ----
+  const int quads = G * (HD / 4), parts = max(1, kTdThreads / quads);
+  for (int unit = threadIdx.x; unit < quads * parts; unit += kTdThreads) {
+    const int part = unit / quads, qd = unit - part * quads, kvh = qd / (HD / 4), col = (qd - kvh * (HD / 4)) * 4;
+    const __nv_bfloat16* v = pool + v_step + kvh * head_step + col;
+    for (int m0 = 0; m0 < group; m0 += GV) {
+      const int nh = min(GV, group - m0), h0 = kvh * group + m0;
+      float4 acc[GV];
+#pragma unroll
+      for (int i = 0; i < GV; ++i) acc[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      constexpr int U = 8;
+      for (int kb = part * U; kb < nk; kb += parts * U) {
+        uint2 x[U];
+#pragma unroll
+        for (int j = 0; j < U; ++j) {
+          const int r = row_s[kb + j];
+          x[j] = r < 0 ? make_uint2(0, 0) : *reinterpret_cast<const uint2*>(v + static_cast<long long>(r) * HD);
+        }
+#pragma unroll
+        for (int j = 0; j < U; ++j) {
+          const float2 a = unpack_bf16x2(x[j].x), b = unpack_bf16x2(x[j].y);
+          const float* w = w_s + (kb + j) * lay.h4 + h0;
+#pragma unroll
+          for (int i = 0; i < GV; ++i) {
+            const float f = i < nh ? w[i] : 0.f;
+            acc[i].x += f * a.x; acc[i].y += f * a.y; acc[i].z += f * b.x; acc[i].w += f * b.y;
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < GV; ++i)
+        if (i < nh) {
+          float* o = o_s + (h0 + i) * HD + col;
+          if (parts == 1) {
+            store4(o, acc[i]);
+          } else {
+            atomicAdd(o, acc[i].x); atomicAdd(o + 1, acc[i].y); atomicAdd(o + 2, acc[i].z); atomicAdd(o + 3, acc[i].w);
+          }
+        }
+    }
+  }
+  cluster.sync();
+  // ---- outputs: the CTAs of the cluster share the pairs of columns ----
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(tok) * H * HD;
+  const float* rot = p.v_rot != nullptr ? p.v_rot + static_cast<long long>(tok) * p.v_ld * 2 : nullptr;
+  for (int c = (rank * kTdThreads + threadIdx.x) * 2; c < H * HD; c += C * kTdThreads * 2) {
+    float a = 0.f, b = 0.f;
+    for (int r = 0; r < C; ++r) {
+      const float2 x = *reinterpret_cast<const float2*>(cluster.map_shared_rank(o_s + c, r));
+      a += x.x;
+      b += x.y;
+    }
+    const int i = (c % HD) / 2;
+    if (rot != nullptr && i < p.v_pairs) {
+      const float cs = rot[2 * i], sn = rot[2 * i + 1], x = a;
+      a = x * cs + b * sn;
+      b = b * cs - x * sn;
+    }
+    *reinterpret_cast<uint32_t*>(out + c) = pack_bf16x2(a, b);
+  }
+  cluster.sync();                                // nobody leaves while its shared memory is read
+}
+
+template <int HD>
+int launch_talk_decode(const nfk_talk_attn_params& p, cudaStream_t stream) {
+  // few tokens: more CTAs per token; many keys: enough CTAs for their scores to fit, two CTAs per SM if they can
+  const int sms = device_sm_count();
+  int C = 1;
+  while (C < kTdMaxCluster && (p.n_tokens * C * 2 <= 2 * sms || talk_decode_layout(p.heads, HD, (p.max_keys + C - 1) / C).bytes > 110 * 1024)) C *= 2;
+  while (C > 1 && (p.max_keys + C - 1) / C < kTdKeys) C /= 2;
+  const TalkDecodeLayout lay = talk_decode_layout(p.heads, HD, (p.max_keys + C - 1) / C);
+  if (lay.bytes > 220 * 1024) return NF_ERR_UNSUPPORTED;
+  const int group = p.heads / p.kv_heads;
+  auto kernel = group == 1 ? talk_decode_kernel<HD, 1> : group == 2 ? talk_decode_kernel<HD, 2> : talk_decode_kernel<HD, 4>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess) return NF_ERR_CUDA;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(static_cast<unsigned>(p.n_tokens) * C);
+  cfg.blockDim = dim3(kTdThreads);
+  cfg.dynamicSmemBytes = lay.bytes;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = C;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  return cudaLaunchKernelEx(&cfg, kernel, p, lay) == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+// ---- prefill --------------------------------------------------------------------------------------------------
+constexpr int kTpQ = 16, kTpHeads = 16, kTpThreads = kTpHeads * 32;
+constexpr int kTpMaxHeads = 64;
+
+template <int HD, int KT>
+struct TalkCfg {
+  static constexpr int KLD = HD + 8;                     // row strides in elements: conflict-free ldmatrix
+  static constexpr int XLD = KT + 8;                     // mixed weights [head][query][key]
+  static constexpr int PLD = kTpQ * KT + 8;              // weights [head][query * KT + key]
+  static constexpr int ROWS = KT * KLD * 2;              // keys or values of a KV head
+  static constexpr int X_BYTES = kTpHeads * kTpQ * XLD * 2;
+  __host__ __device__ static constexpr int p_bytes(int hp) { return hp * PLD * 2; }
+  __host__ __device__ static constexpr int smem(int hp, int kvs) { return 2 * kvs * ROWS + 2 * p_bytes(hp) + 2 * X_BYTES + KT * 8; }
+};
+
+__device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(x, y);
+  const float2 h = unpack_bf16x2(hi);
+  lo = pack_bf16x2(x - h.x, y - h.y);
+}
+
+// hp: heads padded to a multiple of 16; kvs: KV heads that 16 query heads can touch.
+template <int HD, int KT>
+__global__ void __launch_bounds__(kTpThreads, 1)
+talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
+  using Cfg = TalkCfg<HD, KT>;
+  constexpr int NT = KT / 8;                             // key blocks of a tile
+  extern __shared__ __align__(16) uint8_t tps[];
+  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(tps);
+  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(tps + kvs * Cfg::ROWS);
+  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(tps + 2 * kvs * Cfg::ROWS);          // high parts, then low parts
+  __nv_bfloat16* x_s = reinterpret_cast<__nv_bfloat16*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp));
+  long long* row_s = reinterpret_cast<long long*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp) + 2 * Cfg::X_BYTES);
+  cg::cluster_group cluster = cg::this_cluster();
+  const int C = hp / kTpHeads, rank = static_cast<int>(cluster.block_rank());
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int H = p.heads, G = p.kv_heads, group = H / G;
+  const int* item = p.items + (blockIdx.x / C) * 3;
+  const int req = item[0], tok0 = item[1], cnt = item[2];
+  const int pos0 = p.positions[tok0];
+  const int head0 = rank * kTpHeads, head = head0 + warp;
+  const bool live = head < H;
+  const int kv0 = head0 / group, kvn = (min(H, head0 + kTpHeads) - 1) / group - kv0 + 1;
+  const int kvl = live ? head / group - kv0 : 0;         // this warp's KV head among the CTA's
+  const int lo = (p.window > 0 ? max(0, pos0 - p.window + 1) : 0) / KT * KT;
+  const int tiles = (pos0 + cnt - 1 - lo) / KT + 1;
+  const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
+  const long long head_step = static_cast<long long>(p.page_size) * HD, v_step = G * head_step;
+
+  // rows of a tile's keys (KV head kv0) into dst; keys that are not there become zeros
+  auto find_rows = [&](int t) {
+    if (threadIdx.x < KT) {
+      const int j = lo + t * KT + threadIdx.x;
+      long long r = -1;
+      const int first = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+      if (j >= first && j <= pos0 + cnt - 1) {
+        const int page = page_of(j, req, p.page_size, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
+        if (page >= 0) r = (static_cast<long long>(page) * 2 * G * p.page_size + j % p.page_size) * HD + kv0 * head_step;
+      }
+      row_s[threadIdx.x] = r;
+    }
+  };
+  auto fetch = [&](__nv_bfloat16* dst, long long off) {
+    constexpr int CH = HD / 8;
+    for (int i = threadIdx.x; i < kvn * KT * CH; i += kTpThreads) {
+      const int kv = i / (KT * CH), k = i / CH % KT, c = (i % CH) * 8;
+      const bool ok = row_s[k] >= 0;
+      const __nv_bfloat16* src = ok ? pool + row_s[k] + off + kv * head_step + c : pool;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + (kv * KT + k) * Cfg::KLD + c)), "l"(src),
+                   "r"(ok ? 16 : 0) : "memory");
+    }
+    cp_async_commit();
+  };
+
+  uint32_t qa[HD / 16][4];
+  {
+    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + static_cast<long long>(tok0) * H * HD + head * HD;
+    load_q_frags<HD>(qa, [&](int r) -> const __nv_bfloat16* { return live && r < cnt ? q + static_cast<long long>(r) * H * HD : nullptr; });
+  }
+  const int mm = lane >> 3, rr = lane & 7;
+  const float scale = p.scale * kLog2e;
+  const int i0 = pos0 + (lane >> 2), i1 = i0 + 8;        // positions of this lane's two queries
+  const bool q0_ok = live && (lane >> 2) < cnt, q1_ok = live && (lane >> 2) + 8 < cnt;
+  const uint32_t kb = smem_u32(k_s) + kvl * Cfg::ROWS, vb = smem_u32(v_s) + kvl * Cfg::ROWS;
+  auto seen = [&](int i, int j) { return j <= i && j >= 0 && (p.window <= 0 || i - j < p.window); };
+  // scores of this warp's head times log2 e, -inf where the query does not see the key
+  auto scores = [&](float (&s)[NT][4], int t) {
+#pragma unroll
+    for (int b = 0; b < NT; ++b) s[b][0] = s[b][1] = s[b][2] = s[b][3] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < HD / 16; ++ks)
+#pragma unroll
+      for (int b = 0; b < NT; b += 2) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4(kb + ((b * 8 + (mm >> 1) * 8 + rr) * Cfg::KLD + ks * 16 + (mm & 1) * 8) * 2, b0, b1, b2, b3);
+        mma_bf16(s[b], qa[ks], b0, b1);
+        mma_bf16(s[b + 1], qa[ks], b2, b3);
+      }
+#pragma unroll
+    for (int b = 0; b < NT; ++b)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int j = lo + t * KT + b * 8 + (lane & 3) * 2 + e;
+        s[b][e] = q0_ok && seen(i0, j) ? s[b][e] * scale : -INFINITY;
+        s[b][2 + e] = q1_ok && seen(i1, j) ? s[b][2 + e] * scale : -INFINITY;
+      }
+  };
+
+  // ---- first loop: maxima and sums ----
+  const float sink = p.sinks != nullptr && live ? p.sinks[head] * kLog2e : -INFINITY;
+  float m0 = sink, m1 = sink, l0 = 0.f, l1 = 0.f;        // sums of this lane's keys
+  find_rows(0);
+  __syncthreads();
+  fetch(k_s, 0);
+  for (int t = 0; t < tiles; ++t) {
+    cp_async_wait<0>();
+    __syncthreads();
+    float s[NT][4];
+    scores(s, t);
+    if (t + 1 < tiles) find_rows(t + 1);
+    else find_rows(0);                                   // for the second loop
+    __syncthreads();
+    fetch(k_s, 0);
+    float x0 = m0, x1 = m1;
+#pragma unroll
+    for (int b = 0; b < NT; ++b) {
+      x0 = fmaxf(x0, fmaxf(s[b][0], s[b][1]));
+      x1 = fmaxf(x1, fmaxf(s[b][2], s[b][3]));
+    }
+    x0 = quad_max(x0);
+    x1 = quad_max(x1);
+    const float z0 = x0 == -INFINITY ? 0.f : x0, z1 = x1 == -INFINITY ? 0.f : x1;
+    l0 *= fast_exp2(m0 - z0);
+    l1 *= fast_exp2(m1 - z1);
+    m0 = x0;
+    m1 = x1;
+#pragma unroll
+    for (int b = 0; b < NT; ++b) {
+      l0 += fast_exp2(s[b][0] - z0) + fast_exp2(s[b][1] - z0);
+      l1 += fast_exp2(s[b][2] - z1) + fast_exp2(s[b][3] - z1);
+    }
+  }
+  l0 = quad_sum(l0);
+  l1 = quad_sum(l1);
+  if (m0 == -INFINITY) m0 = 0.f;
+  if (m1 == -INFINITY) m1 = 0.f;
+  l0 += sink == -INFINITY ? 0.f : fast_exp2(sink - m0);
+  l1 += sink == -INFINITY ? 0.f : fast_exp2(sink - m1);
+  const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+
+  // ---- second loop: weights, mixing, values ----
+  float acc[HD / 8][4];
+#pragma unroll
+  for (int b = 0; b < HD / 8; ++b) acc[b][0] = acc[b][1] = acc[b][2] = acc[b][3] = 0.f;
+  const uint32_t pb = smem_u32(p_s), xb = smem_u32(x_s);
+  const uint32_t p_lo = static_cast<uint32_t>(Cfg::p_bytes(hp)), x_lo = Cfg::X_BYTES;
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  for (int t = 0; t < tiles; ++t) {
+    cp_async_wait<0>();
+    __syncthreads();                                     // keys are there; everyone is done with the last values
+    fetch(v_s, v_step);
+    {
+      float s[NT][4];
+      scores(s, t);
+      asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");      // all have started, and mixed the last weights
+#pragma unroll
+      for (int b = 0; b < NT; ++b) {
+        uint32_t h0, l0_, h1, l1_;
+        split_bf16x2(fast_exp2(s[b][0] - m0) * inv0, fast_exp2(s[b][1] - m0) * inv0, h0, l0_);
+        split_bf16x2(fast_exp2(s[b][2] - m1) * inv1, fast_exp2(s[b][3] - m1) * inv1, h1, l1_);
+        const int o = head * Cfg::PLD + (lane >> 2) * KT + b * 8 + (lane & 3) * 2;
+        for (int r = 0; r < C; ++r) {
+          __nv_bfloat16* dst = cluster.map_shared_rank(p_s, r) + o;
+          *reinterpret_cast<uint32_t*>(dst) = h0;
+          *reinterpret_cast<uint32_t*>(dst + 8 * KT) = h1;
+          *reinterpret_cast<uint32_t*>(dst + hp * Cfg::PLD) = l0_;
+          *reinterpret_cast<uint32_t*>(dst + hp * Cfg::PLD + 8 * KT) = l1_;
+        }
+      }
+    }
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    // rows for the next keys; the copies of this tile's values have been started
+    if (t + 1 < tiles) find_rows(t + 1);
+    __syncthreads();
+    if (t + 1 < tiles) fetch(k_s, 0);
+    else cp_async_commit();
+    // mixed weights of the CTA's 16 heads: [16 x H] times [H x (query, key)], columns over the warps
+#pragma unroll
+    for (int c = 0; c < kTpQ * KT / 8 / kTpHeads; c += 2) {
+      const int col = (warp * (kTpQ * KT / 8 / kTpHeads) + c) * 8;
+      float x[2][4];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) x[e][0] = x[e][1] = x[e][2] = x[e][3] = 0.f;
+      for (int g = 0; g < hp; g += 16) {
+        const int hr0 = head0 + (lane >> 2), hr1 = hr0 + 8, gc = g + (lane & 3) * 2;
+        auto talk2 = [&](int h, int gg) {
+          const float a = h < H && gg < H ? __ldg(p.talk + h * H + gg) : 0.f, b = h < H && gg + 1 < H ? __ldg(p.talk + h * H + gg + 1) : 0.f;
+          return pack_bf16x2(a, b);
+        };
+        const uint32_t a[4] = {talk2(hr0, gc), talk2(hr1, gc), talk2(hr0, gc + 8), talk2(hr1, gc + 8)};
+        const uint32_t o = ((g + (mm & 1) * 8 + rr) * Cfg::PLD + col + (mm >> 1) * 8) * 2;
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4_trans(pb + o, b0, b1, b2, b3);
+        mma_bf16(x[0], a, b0, b1);
+        mma_bf16(x[1], a, b2, b3);
+        ldsm_x4_trans(pb + p_lo + o, b0, b1, b2, b3);
+        mma_bf16(x[0], a, b0, b1);
+        mma_bf16(x[1], a, b2, b3);
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int cc = col + e * 8 + (lane & 3) * 2, qq = cc / KT, kk = cc % KT;
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          uint32_t hi, lo_;
+          split_bf16x2(x[e][2 * h], x[e][2 * h + 1], hi, lo_);
+          __nv_bfloat16* dst = x_s + (((lane >> 2) + h * 8) * kTpQ + qq) * Cfg::XLD + kk;
+          *reinterpret_cast<uint32_t*>(dst) = hi;
+          *reinterpret_cast<uint32_t*>(dst + Cfg::X_BYTES / 2) = lo_;
+        }
+      }
+    }
+    if (t + 1 < tiles) asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    cp_async_wait<1>();                                  // values
+    __syncthreads();
+#pragma unroll
+    for (int ks = 0; ks < KT / 16; ++ks) {
+      uint32_t ah[4], al[4];
+      const uint32_t o = ((warp * kTpQ + (lane & 15)) * Cfg::XLD + ks * 16 + (lane >> 4) * 8) * 2;
+      ldsm_x4(xb + o, ah[0], ah[1], ah[2], ah[3]);
+      ldsm_x4(xb + x_lo + o, al[0], al[1], al[2], al[3]);
+#pragma unroll
+      for (int b = 0; b < HD / 8; b += 2) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4_trans(vb + ((ks * 16 + (mm & 1) * 8 + rr) * Cfg::KLD + (b + (mm >> 1)) * 8) * 2, b0, b1, b2, b3);
+        mma_bf16(acc[b], ah, b0, b1);
+        mma_bf16(acc[b + 1], ah, b2, b3);
+        mma_bf16(acc[b], al, b0, b1);
+        mma_bf16(acc[b + 1], al, b2, b3);
+      }
+    }
+  }
+  // ---- outputs turn back by their query's angles ----
+  if (live) {
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = (lane >> 2) + h * 8;
+      if (r >= cnt) continue;
+      const long long tok = tok0 + r;
+      const float2* rot = p.v_rot != nullptr ? reinterpret_cast<const float2*>(p.v_rot) + tok * p.v_ld : nullptr;
+#pragma unroll
+      for (int b = 0; b < HD / 8; ++b) {
+        const int i = b * 4 + (lane & 3);
+        float x = acc[b][2 * h], y = acc[b][2 * h + 1];
+        if (rot != nullptr && i < p.v_pairs) {
+          const float2 a = rot[i];
+          const float z = x;
+          x = z * a.x + y * a.y;
+          y = y * a.x - z * a.y;
+        }
+        *reinterpret_cast<uint32_t*>(out + tok * H * HD + head * HD + i * 2) = pack_bf16x2(x, y);
+      }
+    }
+  }
+  // a CTA may only leave when nobody writes to its shared memory any more: every write comes before the last
+  // cluster barrier, which all have passed
+}
+
+template <int HD, int KT>
+int launch_talk_prefill(const nfk_talk_attn_params& p, int hp, int kvs, cudaStream_t stream) {
+  const int C = hp / kTpHeads, sm = TalkCfg<HD, KT>::smem(hp, kvs);
+  auto kernel = talk_prefill_kernel<HD, KT>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, sm) != cudaSuccess) return NF_ERR_CUDA;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(static_cast<unsigned>(p.num_items) * C);
+  cfg.blockDim = dim3(kTpThreads);
+  cfg.dynamicSmemBytes = sm;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = C;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  return cudaLaunchKernelEx(&cfg, kernel, p, hp, kvs) == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+// KV heads that 16 neighbouring query heads (from a multiple of 16) can touch.
+int kv_heads_of_16(int heads, int group) {
+  int most = 1;
+  for (int h0 = 0; h0 < heads; h0 += kTpHeads) {
+    const int last = (heads < h0 + kTpHeads ? heads : h0 + kTpHeads) - 1, n = last / group - h0 / group + 1;
+    if (n > most) most = n;
+  }
+  return most;
+}
+
 int check_talk(const nfk_talk_attn_params* p) {
   if (p == nullptr) return NF_ERR_BAD_ARG;
   if (!p->q || !p->pool || !p->out || !p->positions || !p->token_req || !p->kv_indptr || !p->kv_indices || !p->talk ||
@@ -148,4 +695,40 @@ extern "C" int nfk_talk_attn(const nfk_talk_attn_params* p, cudaStream_t stream)
   const int rc = check_talk(p);
   if (rc != NF_OK || p->n_tokens == 0) return rc;
   return p->dtype == NFK_F32 ? launch_talk_simple<float>(*p, stream) : launch_talk_simple<__nv_bfloat16>(*p, stream);
+}
+
+extern "C" int nfk_talk_attn_decode(const nfk_talk_attn_params* p, cudaStream_t stream) {
+  using namespace nf;
+  const int rc = check_talk(p);
+  if (rc != NF_OK || p->n_tokens == 0) return rc;
+  if (p->dtype != NFK_BF16 || (p->hd != 64 && p->hd != 128)) return NF_ERR_UNSUPPORTED;
+  if (p->max_keys <= 0 || static_cast<long long>(p->num_pages) * 2 * p->kv_heads * p->page_size > 0x7fffffffll) return NF_ERR_BAD_ARG;
+  return p->hd == 64 ? launch_talk_decode<64>(*p, stream) : launch_talk_decode<128>(*p, stream);
+}
+
+extern "C" int nfk_talk_attn_prefill(const nfk_talk_attn_params* p, cudaStream_t stream) {
+  using namespace nf;
+  const int rc = check_talk(p);
+  if (rc != NF_OK || p->num_items == 0) return rc;
+  if (p->num_items < 0 || !p->items) return NF_ERR_BAD_ARG;
+  if (p->dtype != NFK_BF16 || (p->hd != 64 && p->hd != 128) || p->heads > kTpMaxHeads) return NF_ERR_UNSUPPORTED;
+  const int hp = (p->heads + kTpHeads - 1) / kTpHeads * kTpHeads, kvs = kv_heads_of_16(p->heads, p->heads / p->kv_heads);
+  constexpr int kMost = 227 * 1024;
+  if (p->hd == 64) {
+    if (TalkCfg<64, 32>::smem(hp, kvs) <= kMost) return launch_talk_prefill<64, 32>(*p, hp, kvs, stream);
+    if (TalkCfg<64, 16>::smem(hp, kvs) <= kMost) return launch_talk_prefill<64, 16>(*p, hp, kvs, stream);
+  } else {
+    if (TalkCfg<128, 32>::smem(hp, kvs) <= kMost) return launch_talk_prefill<128, 32>(*p, hp, kvs, stream);
+    if (TalkCfg<128, 16>::smem(hp, kvs) <= kMost) return launch_talk_prefill<128, 16>(*p, hp, kvs, stream);
+  }
+  return NF_ERR_UNSUPPORTED;
+}
+
+extern "C" int nfk_talk_attn_fits(int heads, int kv_heads, int hd, int max_keys) {
+  using namespace nf;
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || heads > kTpMaxHeads || (hd != 64 && hd != 128) || max_keys <= 0) return 0;
+  const int hp = (heads + kTpHeads - 1) / kTpHeads * kTpHeads, kvs = kv_heads_of_16(heads, heads / kv_heads);
+  const int pre = hd == 64 ? TalkCfg<64, 16>::smem(hp, kvs) : TalkCfg<128, 16>::smem(hp, kvs);
+  const int dec = talk_decode_layout(heads, hd, (max_keys + kTdMaxCluster - 1) / kTdMaxCluster).bytes;
+  return (pre <= 227 * 1024 ? 1 : 0) + (dec <= 220 * 1024 ? 2 : 0);
 }

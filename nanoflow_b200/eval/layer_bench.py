@@ -21,11 +21,12 @@ import torch
 
 SIZES = {
     # name: (width, ff, heads, kv heads of the Llama, vocab, latent rank, window, mLSTM heads, dim, vdim,
-    #        WKV decay rank, ff of an expert and of the shared one: 6 experts per token and the shared one make up ff)
+    #        WKV decay rank, ff of an expert and of the shared one: 6 experts per token and the shared one make up ff,
+    #        blocks of the linear recurrent unit, ff of an expert without a gate: 6 of them have as many weights as ff)
     "8B": dict(width=4096, ff=14336, heads=32, kv=8, vocab=128256, rank=512, window=1024, mh=8, md=256, mv=512, decay=128,
-               eff=2048, sff=2048),
+               eff=2048, sff=2048, blocks=16, uff=3584),
     "2B": dict(width=2048, ff=8192, heads=16, kv=4, vocab=32000, rank=256, window=512, mh=4, md=256, mv=512, decay=64,
-               eff=1024, sff=2048),
+               eff=1024, sff=2048, blocks=16, uff=2048),
 }
 EXPERTS, TOP, GROUPS, KEEP = 64, 6, 8, 4
 WORKLOADS = [("prefill 4 x 1024", [(0, 1024)] * 4), ("prefill 1 x 4096", [(0, 4096)]),
@@ -44,13 +45,17 @@ def peaks() -> Tuple[float, float]:
 
 def model_dict(kind: str, s: Dict[str, int]) -> Dict[str, Any]:
     from ..config import _hf
-    from ..models import volarax, zubedra
+    from ..models import gupizen, volarax, zubedra
     if kind == "llama":
         return _hf(s["width"], s["ff"], LAYERS, s["heads"], s["kv"], s["vocab"], 500000.0)
     if kind == "zubedra":
         return zubedra.builtin(s["width"], s["vocab"], "aw" * (LAYERS // 2), heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128,
                                softcap=50.0, w_heads=s["width"] // 64, w_dim=64, rank=s["decay"], experts=EXPERTS, top=TOP,
                                ff=s["eff"], groups=GROUPS, keep=KEEP, shared_ff=s["sff"])
+    if kind == "gupizen":
+        return gupizen.builtin(s["width"], s["vocab"], "pd" * (LAYERS // 2), heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128,
+                               window=s["window"], rec_width=s["width"], rec_blocks=s["blocks"], d_heads=s["heads"],
+                               d_kv_heads=s["heads"], d_dim=128, d_vdim=128, rank=128, experts=EXPERTS, top=TOP, ff=s["uff"])
     return volarax.builtin(s["width"], s["vocab"], "am" * (LAYERS // 2), heads=s["heads"], dim=128, vdim=128, kv_rank=s["rank"],
                    window=s["window"], m_heads=s["mh"], m_dim=s["md"], m_vdim=s["mv"], ff=s["ff"], m_ff=s["ff"])
 
@@ -128,6 +133,26 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
         return 0.0, rows * p.cols * (8 + (2 + more) * es)
     if isinstance(p, G.GqaAppendParams):
         return 0.0, T * 2 * (p.heads + 2 * p.kv_heads) * p.hd * es
+    if isinstance(p, G.TalkAttnParams):
+        if (spans[0][1] == 1) != (dict(op.dyn).get("n_tokens") == "n_dec"):
+            return 0.0, 0.0
+        pairs = sees(p.window)
+        keys = sum(min(c + n, (p.window + n - 1) if p.window else c + n) for c, n in spans)
+        return pairs * p.heads * (4.0 * p.hd + 2.0 * p.heads), es * (2 * keys * p.kv_heads * p.hd + 2 * T * p.heads * p.hd)
+    if isinstance(p, G.ShortConvParams):
+        return 0.0, T * 2 * p.cols * es
+    if isinstance(p, G.RgLruParams):
+        if (spans[0][1] == 1) != ("decode" in op.kernel):
+            return 0.0, 0.0
+        return 0.0, T * p.cols * (3 * es + 8) + 2 * len(spans) * p.cols * 4
+    if isinstance(p, G.DeltaParams):
+        dec = "decode" in op.kernel
+        if (spans[0][1] == 1) != dec:
+            return 0.0, 0.0
+        state = len(spans) * p.heads * p.dim * p.vdim * 4
+        io = T * ((2 * p.kv_heads * p.dim + 3 * p.heads * p.vdim) * es + p.heads * p.dim * 4)
+        chunk = 0 if dec else 64
+        return T * p.heads * (2.0 * chunk * (p.dim + p.vdim) + 6.0 * p.dim * p.vdim), 2 * state + io
     if isinstance(p, G.TokenShiftParams):
         return 0.0, T * (1 + p.n_mix) * p.ld_h * es
     if isinstance(p, G.WkvParams):

@@ -24,6 +24,7 @@ PREFILL_HEAD_DIM = 128        # head size of the tcgen05 prefill attention kerne
 ATTN_HEAD_DIMS = (64, 128)    # head sizes of the tensor-core attention kernels over pages of keys and values
 ATTN_MAX_GROUP = 16           # query heads per KV head that the decode kernel takes
 WKV_CHUNK_DIM = 128           # largest head size of the chunked WKV kernels
+DELTA_CHUNK_DIM = 128         # ... and of the chunked delta-rule kernels
 PAGE = 16                     # tokens per cache page
 MOE_MAX_EXPERTS, MOE_MAX_TOP = 1024, 32
 LINEAR_ACTS = ("gelu",)       # activations of products without a gate

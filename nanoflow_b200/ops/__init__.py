@@ -156,7 +156,8 @@ class TalkAttnParams(Structure):
                 ("kv_indptr", c_void_p), ("kv_indices", c_void_p), ("kv_first", c_void_p), ("sinks", c_void_p),
                 ("talk", c_void_p), ("v_rot", c_void_p), ("v_pairs", c_int), ("v_ld", c_int), ("token_begin", c_int),
                 ("n_tokens", c_int), ("heads", c_int), ("kv_heads", c_int), ("hd", c_int), ("page_size", c_int),
-                ("num_pages", c_int), ("window", c_int), ("scale", c_float), ("dtype", c_int), ("status", c_void_p)]
+                ("num_pages", c_int), ("window", c_int), ("scale", c_float), ("dtype", c_int), ("status", c_void_p),
+                ("max_keys", c_int), ("items", c_void_p), ("num_items", c_int)]
 
 
 class ShortConvParams(Structure):
@@ -183,6 +184,7 @@ class DeltaParams(Structure):
                 ("req_begin", c_int), ("req_count", c_int), ("heads", c_int), ("kv_heads", c_int), ("dim", c_int),
                 ("vdim", c_int), ("vdim_real", c_int), ("num_slots", c_int), ("q_scale", c_float), ("unit_eps", c_float),
                 ("eps", c_float), ("dtype", c_int), ("seq_reqs", c_void_p), ("num_seq", c_int), ("o", c_void_p),
+                ("items", c_void_p), ("num_items", c_int), ("scratch", c_void_p), ("scratch_floats", c_longlong),
                 ("status", c_void_p)]
 
 

@@ -6,7 +6,7 @@ launch on the current stream; engines do not call them but put the same paramete
 """
 from __future__ import annotations
 
-from ctypes import byref
+from ctypes import byref, c_longlong
 from typing import Optional
 
 import torch
@@ -257,9 +257,10 @@ def paged_attention(q, pool, out, qo_indptr, kv_indptr, kv_indices, kv_last_page
 
 def talk_attention(q, pool, out, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, heads: int, scale: float, talk,
                    window: int = 0, sinks=None, v_rot=None, token_begin: int = 0, n_tokens: Optional[int] = None,
-                   status=None) -> None:
-    """Attention whose heads' weights are mixed by ``talk`` [heads, heads]; any head size, bf16 or fp32; q, out [T, heads *
-    head size]. ``v_rot``: (table of angles [T, n, 2], pairs per head) by which outputs turn back."""
+                   items=None, max_keys: int = 0, status=None) -> None:
+    """Attention whose heads' weights are mixed by ``talk`` [heads, heads]; q, out [T, heads * head size]. ``v_rot``: (table
+    of angles [T, n, 2], pairs per head) by which outputs turn back. ``items`` [n, 3] (request, first token, at most 16
+    tokens): the prefill kernel; ``max_keys``: the decode kernel; else the simple one (any head size, bf16 or fp32)."""
     _f32(sinks, "sinks"); _f32(talk, "talk")
     n, _, G, ps, hd = pool.shape
     p = TalkAttnParams(q=_p(q), pool=_p(pool), out=_p(out), positions=_p(positions), token_req=_p(token_req),
@@ -270,7 +271,13 @@ def talk_attention(q, pool, out, positions, token_req, kv_indptr, kv_indices, kv
     if v_rot is not None:
         _f32(v_rot[0], "v_rot")
         p.v_rot, p.v_ld, p.v_pairs = _p(v_rot[0]), v_rot[0].shape[1], v_rot[1]
-    _check(lib().nfk_talk_attn(byref(p), _stream()), "nfk_talk_attn")
+    name = "nfk_talk_attn"
+    if items is not None:
+        _i32(items, "items")
+        p.items, p.num_items, name = _p(items), items.shape[0], "nfk_talk_attn_prefill"
+    elif max_keys:
+        p.max_keys, name = max_keys, "nfk_talk_attn_decode"
+    _check(getattr(lib(), name)(byref(p), _stream()), name)
 
 
 def short_conv(x, w, state, state_ref, positions, token_req, qo_indptr, *, bias=None, act: Optional[str] = None,
@@ -303,21 +310,25 @@ def rglru(u, y, gates, r_b, i_b, log_a, state, out, positions, qo_indptr, state_
 
 
 def delta(qkv, x, beta, g, rate, dt_bias, norm, state, y, positions, qo_indptr, state_ref, *, kv_heads: int, vdim_real: int,
-          q_scale: float, eps: float, unit_eps: float = 1e-6, decode: int = 0, seq=None, status=None) -> None:
+          q_scale: float, eps: float, unit_eps: float = 1e-6, decode: int = 0, items=None, seq=None, status=None) -> None:
     """qkv rows are q | k (kv_heads each) | v, x [T, heads * dim], beta [T, >= heads], g [T, heads * vdim]; ``state`` [slots,
-    heads, dim, vdim] in place. ``decode``: the first so many requests have one token each; else the requests ``seq`` token
-    by token."""
+    heads, dim, vdim] in place. ``decode``: the first so many requests have one token each; else ``items`` [n, 4] in chunks
+    and the requests ``seq`` token by token."""
     for t, nm in ((x, "x"), (beta, "beta"), (rate, "rate"), (dt_bias, "dt_bias"), (norm, "norm"), (state, "state")):
         _f32(t, nm)
     slots, heads, dim, vdim = state.shape
     o = torch.zeros(qkv.shape[0], heads * vdim, device=qkv.device)
+    n = 0 if items is None else items.shape[0]
+    lib().nfk_delta_item_floats.restype = c_longlong
+    ws = torch.zeros(max(1, n) * heads * lib().nfk_delta_item_floats(dim, vdim), device=qkv.device)
     p = DeltaParams(qkv=_p(qkv), ld=qkv.stride(0), q_off=0, k_off=kv_heads * dim, v_off=2 * kv_heads * dim, x=_p(x),
                     ld_x=x.stride(0), beta=_p(beta), ld_b=beta.stride(0), g=_p(g), ld_g=g.stride(0), rate=_p(rate),
                     dt_bias=_p(dt_bias), norm=_p(norm), S=_p(state), y=_p(y), ld_y=y.stride(0), positions=_p(positions),
                     qo_indptr=_p(qo_indptr), state_slot=_p(state_ref), req_begin=0, req_count=decode, heads=heads,
                     kv_heads=kv_heads, dim=dim, vdim=vdim, vdim_real=vdim_real, num_slots=slots, q_scale=q_scale,
                     unit_eps=unit_eps, eps=eps, dtype=dtype_code(qkv.dtype), seq_reqs=_p(seq),
-                    num_seq=0 if seq is None else seq.numel(), o=_p(o), status=_p(status))
+                    num_seq=0 if seq is None else seq.numel(), o=_p(o), items=_p(items), num_items=n, scratch=_p(ws),
+                    scratch_floats=ws.numel(), status=_p(status))
     name = "nfk_delta_decode" if decode else "nfk_delta_prefill"
     _check(getattr(lib(), name)(byref(p), _stream()), name)
 

@@ -42,7 +42,7 @@ import numpy as np
 import torch
 
 from .. import ops
-from ..models.layer_list import (PAGE, PREFILL_HEAD_DIM, WKV_CHUNK_DIM, ActSpec, LayerListConfig, NormWeights, parts_of,
+from ..models.layer_list import (DELTA_CHUNK_DIM, PAGE, PREFILL_HEAD_DIM, WKV_CHUNK_DIM, ActSpec, LayerListConfig, NormWeights, parts_of,
                                  round8)
 from ..ops import ACTS, CONV_ACTS, LIN_ACTS, NORMS, ROUTER_SCORES, dtype_code
 from ..ops.layer_list import mlstm_scratch_floats
@@ -58,10 +58,11 @@ QUERY_TILE = 128             # query tokens per work item of the prefill attenti
 MLSTM_CHUNK = 64             # tokens per chunk of the chunked mLSTM kernel
 MLSTM_COLS = 64              # columns of the state per CTA of that kernel
 SEGMENT_ITEMS = 48           # most segments that prompt portions are cut into for the mLSTM kernel
-WKV_CHUNK = 64               # tokens per chunk of the chunked WKV kernels
-WKV_SPARE_CHUNKS = 64        # chunks beyond whole ones that their scratch has room for; further portions go token by token
+CHUNK = 64                   # tokens per chunk of the chunked WKV and delta-rule kernels
+SPARE_CHUNKS = 64        # chunks beyond whole ones that their scratch has room for; further portions go token by token
 
 
+TALK_TILE = 16               # query tokens per work item of the prefill kernel for mixed heads
 DELTA_UNIT_EPS = 1e-6        # of the unit vectors of the delta rule
 
 
@@ -98,9 +99,10 @@ class LayerListEngine(Engine):
                 self.groups.append(PathGroup(len(self.groups), *key))
         # query heads per KV head of the attention layers on the tcgen05 prefill kernel: a work list for each
         self.attn_groups = sorted({s.group for s in m.run_specs("attention") if m.attn_on_tensor_cores(s)})
-        self.wkv_cap = 0
-        if m.dtype == torch.bfloat16 and any(round8(s.dim) <= WKV_CHUNK_DIM for s in m.run_specs("wkv")):
-            self.wkv_cap = T // WKV_CHUNK + min(B, WKV_SPARE_CHUNKS)
+        self.chunk_cap = 0
+        if m.dtype == torch.bfloat16 and (any(round8(s.dim) <= WKV_CHUNK_DIM for s in m.run_specs("wkv")) or
+                                          any(self._delta_in_chunks(s) for s in m.run_specs("delta"))):
+            self.chunk_cap = T // CHUNK + min(B, SPARE_CHUNKS)
         self.x_pages = self._expand_pages()
         self._alloc_state()
         self.num_pages = int(num_pages or e.num_pages or self._derive_num_pages(T, B))
@@ -113,8 +115,10 @@ class LayerListEngine(Engine):
             extra[f"gitem{n}"] = 3 * (T // (QUERY_TILE // n) + B + 1)
         if m.run_specs("mlstm"):
             extra["segs"] = 4 * max(B, SEGMENT_ITEMS)
-        if m.run_specs("wkv"):
-            extra.update(wkv_items=4 * max(1, self.wkv_cap), wkv_seq=B)
+        if any(s.talk for s in m.run_specs("attention")):
+            extra["titem"] = 3 * (T // TALK_TILE + B + 1)
+        if m.run_specs("wkv") or m.run_specs("delta"):
+            extra.update(chunk_items=4 * max(1, self.chunk_cap), chunk_seq=B)
         if m.run_specs("wkv") or m.run_specs("delta"):
             extra["pre_reqs"] = B
         self._make_metadata(MetaLayout(T, B, self.nano_sizes, self.num_pages, 0, self.S_cap, extra))
@@ -232,7 +236,7 @@ class LayerListEngine(Engine):
                                          w["v_first"] + w["mix"] + w["lora"] + w["e_in"] + w["e_act"] + w["e_out"] + w["conv"] +
                                          w["aux"] + 2 * m.width_p) +
                    4 * (w["gates"] + w["o_rec"] + w["router"] + w["beta"] + 5 * w["e_top"] + 2 * sum((len(k) + 7) // 8 * 8 for k in self._rotations())))
-        act += self._decode_ws_floats() * 4 + self._wkv_scratch_floats() * 4
+        act += self._decode_ws_floats() * 4 + self._chunk_scratch_floats() * 4
         act += self.x_pages * PAGE * (w["kv"] + w["cg"]) * es + self.S_cap * (es * m.width_p + 4 * m.vocab_p)
         budget = free - total * (1.0 - e.gpu_mem_fraction) - act - (1 << 30)
         per_page = max(1, m.kv_bytes_per_token_local()) * PAGE
@@ -251,9 +255,23 @@ class LayerListEngine(Engine):
                  default=0)
         return DECODE_SPLIT_ROWS * DECODE_MAX_CHUNKS * (hd + 2) if hd else 0
 
-    def _wkv_scratch_floats(self) -> int:
+    def _chunk_scratch_floats(self) -> int:
         sizes = [(s.heads, round8(s.dim)) for s in self.model.run_specs("wkv")]
-        return max([self.wkv_cap * h * (d * d + d) for h, d in sizes if d <= WKV_CHUNK_DIM], default=0)
+        floats = [h * (d * d + d) for h, d in sizes if d <= WKV_CHUNK_DIM]
+        floats += [s.heads * delta_item_floats(s) for s in self.model.run_specs("delta") if self._delta_in_chunks(s)]
+        return self.chunk_cap * max(floats, default=0)
+
+    def _delta_in_chunks(self, s) -> bool:
+        return self.model.dtype == torch.bfloat16 and max(round8(s.dim), round8(s.vdim)) <= DELTA_CHUNK_DIM
+
+    def _talk_kernels(self, s, talk: torch.Tensor) -> Tuple[bool, bool]:
+        """Whether single tokens and portions of an attention layer with mixed heads run on the kernels made for them."""
+        if self.model.dtype != torch.bfloat16:
+            return False, False
+        keys = min(s.window or self.num_pages * PAGE, self.num_pages * PAGE)
+        fits = ops.lib().nfk_talk_attn_fits(s.heads, s.kv_heads, self.model.attn_hd(s), keys)
+        exact = torch.equal(talk.to(torch.bfloat16).float(), talk)      # it enters the prefill kernel's products in bf16
+        return bool(fits & 2), bool(fits & 1) and exact
 
     def _alloc_buffers(self) -> None:
         m, T, dev = self.model, self.T, self.device
@@ -287,7 +305,7 @@ class LayerListEngine(Engine):
         self.moe_zeros = torch.zeros_like(self.moe_counts)
         self.moe_counts_of = [c for c in self.moe_counts[:sum(sizes)].split(sizes)] if sum(sizes) else [None] * len(sizes)
         self.decode_ws = torch.empty(max(8, self._decode_ws_floats()), dtype=f32, device=dev)
-        self.wkv_ws = torch.empty(max(8, self._wkv_scratch_floats()), dtype=f32, device=dev)
+        self.chunk_ws = torch.empty(max(8, self._chunk_scratch_floats()), dtype=f32, device=dev)
         self.h_s = P(self.S_cap, m.width_p, dt, "sample_h")
         self.logits = P(self.S_cap, m.vocab_p, f32, "logits")
         self.pools = [next((p for s in parts_of(m.layers[r.layer].mixer) for p in [self._pool(s)] if p is not None), None)
@@ -572,13 +590,23 @@ class LayerListEngine(Engine):
             v_rot, v_pairs, v_ld = None, 0, 0
         self._op(f"R{r}.gqa_append", ap, dyn=[("T", T)], layer=r)
         if s.talk:
-            tp = TalkAttnParams(q=_ptr(qn), pool=_ptr(pool), out=_ptr(attn), positions=_ptr(meta["positions"]),
-                                token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
-                                kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), sinks=_ptr(lw.sinks),
-                                talk=_ptr(lw.talk), v_rot=v_rot, v_pairs=v_pairs, v_ld=v_ld, token_begin=0, n_tokens=0, heads=H,
-                                kv_heads=G, hd=hd, page_size=PAGE, num_pages=self.num_pages, window=s.window or 0, scale=s.scale,
-                                dtype=self.code, status=st)
-            self._op(f"R{r}.talk_attn", tp, dyn=[("n_tokens", T)], layer=r)
+            def params() -> TalkAttnParams:
+                return TalkAttnParams(
+                    q=_ptr(qn), pool=_ptr(pool), out=_ptr(attn), positions=_ptr(meta["positions"]),
+                    token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]), kv_indices=_ptr(meta["kv_indices"]),
+                    kv_first=_ptr(meta["kv_first"]), sinks=_ptr(lw.sinks), talk=_ptr(lw.talk), v_rot=v_rot, v_pairs=v_pairs,
+                    v_ld=v_ld, token_begin=0, n_tokens=0, heads=H, kv_heads=G, hd=hd, page_size=PAGE, num_pages=self.num_pages,
+                    window=s.window or 0, scale=s.scale, dtype=self.code, status=st, items=_ptr(meta["titem"]))
+
+            dec, pre = self._talk_kernels(s, lw.talk)
+            self._op(f"R{r}.talk_decode", params(), kernel="nfk_talk_attn_decode" if dec else "nfk_talk_attn",
+                     dyn=[("n_tokens", "n_dec")] + ([("max_keys", g.symbol(f"keys{s.window or 0}"))] if dec else []), layer=r)
+            if pre:
+                self._op(f"R{r}.talk_prefill", params(), kernel="nfk_talk_attn_prefill",
+                         dyn=[("num_items", g.symbol("n_titems"))], layer=r)
+            else:
+                self._op(f"R{r}.talk_prefill", params(), kernel="nfk_talk_attn",
+                         dyn=[("token_begin", "n_dec"), ("n_tokens", g.symbol("pre_tokens"))], layer=r)
         elif m.attn_on_tensor_cores(s):
             def params() -> AttnParams:
                 p = AttnParams()
@@ -629,16 +657,16 @@ class LayerListEngine(Engine):
                              ld_y=attn.stride(0), positions=_ptr(meta["positions"]), qo_indptr=_ptr(meta["qo_indptr"]),
                              state_slot=_ptr(meta["state_ref"]), req_begin=0, req_count=0, heads=H, dim=d, dim_real=s.dim,
                              num_slots=self.num_slots, eps=m.norm_eps, dtype=self.code, o=_ptr(self.flat["o_rec"]),
-                             items=_ptr(meta["wkv_items"]), scratch=_ptr(self.wkv_ws), scratch_floats=self.wkv_ws.numel(),
+                             items=_ptr(meta["chunk_items"]), scratch=_ptr(self.chunk_ws), scratch_floats=self.chunk_ws.numel(),
                              status=st)
 
         self._op(f"R{r}.wkv_decode", params(), kernel="nfk_wkv_decode", dyn=[("req_count", "n_dec")], layer=r)
-        chunked = self.wkv_cap > 0 and d <= WKV_CHUNK_DIM
+        chunked = self.chunk_cap > 0 and d <= WKV_CHUNK_DIM
         p = params()
-        p.seq_reqs = _ptr(meta["wkv_seq" if chunked else "pre_reqs"])
-        dyn = [("num_seq", self.g.symbol("n_wkv_seq" if chunked else "n_pre"))]
+        p.seq_reqs = _ptr(meta["chunk_seq" if chunked else "pre_reqs"])
+        dyn = [("num_seq", self.g.symbol("n_chunk_seq" if chunked else "n_pre"))]
         if chunked:
-            dyn.append(("num_items", self.g.symbol("n_wkv_items")))
+            dyn.append(("num_items", self.g.symbol("n_chunks")))
         self._op(f"R{r}.wkv_prefill", p, kernel="nfk_wkv_prefill", dyn=dyn, layer=r)
         self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
 
@@ -695,10 +723,15 @@ class LayerListEngine(Engine):
                                state_slot=_ptr(meta["state_ref"]), req_begin=0, req_count=0, heads=H, kv_heads=G, dim=d, vdim=v,
                                vdim_real=s.vdim, num_slots=self.num_slots, q_scale=s.dim ** -0.5, unit_eps=DELTA_UNIT_EPS,
                                eps=self.model.norm_eps, dtype=self.code, seq_reqs=_ptr(meta["pre_reqs"]), num_seq=0,
-                               o=_ptr(self.flat["o_rec"]), status=st)
+                               o=_ptr(self.flat["o_rec"]), items=_ptr(meta["chunk_items"]), scratch=_ptr(self.chunk_ws),
+                               scratch_floats=self.chunk_ws.numel(), status=st)
 
         self._op(f"R{r}.delta_decode", params(), kernel="nfk_delta_decode", dyn=[("req_count", "n_dec")], layer=r)
-        self._op(f"R{r}.delta_prefill", params(), kernel="nfk_delta_prefill", dyn=[("num_seq", "n_pre")], layer=r)
+        p, dyn = params(), [("num_seq", "n_pre")]
+        if self._delta_in_chunks(s):
+            p.seq_reqs = _ptr(meta["chunk_seq"])
+            dyn = [("num_seq", self.g.symbol("n_chunk_seq")), ("num_items", self.g.symbol("n_chunks"))]
+        self._op(f"R{r}.delta_prefill", p, kernel="nfk_delta_prefill", dyn=dyn, layer=r)
         self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
 
     # ---- feed-forwards: read self.h; return what joins the stream (see _residual) -------------------------
@@ -810,11 +843,18 @@ class LayerListEngine(Engine):
             segs = mlstm_segments(qo, D, self._segment_ctas(), ops.sm_count(self.device))
             put("segs", segs.reshape(-1))
             sym["n_segs"] = segs.shape[0]
-        if m.run_specs("wkv"):
-            items, seq = wkv_work(qo, D, self.wkv_cap)
-            put("wkv_items", items.reshape(-1))
-            put("wkv_seq", seq)
-            sym["n_wkv_items"], sym["n_wkv_seq"] = items.shape[0], seq.size
+        if "chunk_items" in self.meta:
+            items, seq = chunk_work(qo, D, self.chunk_cap)
+            put("chunk_items", items.reshape(-1))
+            put("chunk_seq", seq)
+            sym["n_chunks"], sym["n_chunk_seq"] = items.shape[0], seq.size
+        if "titem" in self.meta:
+            items = query_items(qo, D, TALK_TILE)
+            put("titem", items.reshape(-1))
+            sym["n_titems"], sym["pre_tokens"] = items.shape[0], plan.num_tokens - int(qo[D])
+            seen = int(plan.positions[:D].max()) + 1 if D else 1
+            for w in {s.window or 0 for s in m.run_specs("attention")}:
+                sym[f"keys{w}"] = min(w or seen, seen)
         if "pre_reqs" in self.meta:
             put("pre_reqs", np.arange(D, D + P, dtype=np.int32))
         for n in self.attn_groups:
@@ -874,6 +914,12 @@ MIXERS = {"latent_attention": LayerListEngine._latent_attention, "mlstm": LayerL
 FEED_FORWARDS = {"dense": LayerListEngine._dense, "moe": LayerListEngine._moe}
 
 
+def delta_item_floats(s) -> int:
+    """Scratch of a chunk and head of the chunked delta-rule kernels (nfk_delta_item_floats)."""
+    d, v = round8(s.dim), round8(s.vdim)
+    return 3 * CHUNK * d + CHUNK * CHUNK + CHUNK * v + d
+
+
 def rotations(s) -> List[tuple]:
     """Frequencies by which an attention layer turns queries and keys, and if it does, values."""
     if s.rotary is None:
@@ -906,16 +952,16 @@ def mlstm_segments(qo_indptr: np.ndarray, n_dec: int, ctas_per_segment: int, sms
     return np.asarray(out, dtype=np.int32)
 
 
-def wkv_work(qo_indptr: np.ndarray, n_dec: int, chunk_cap: int) -> Tuple[np.ndarray, np.ndarray]:
-    """Rows (request, first token, tokens, chunk of the portion) for the chunked WKV kernels, and the requests whose
+def chunk_work(qo_indptr: np.ndarray, n_dec: int, chunk_cap: int) -> Tuple[np.ndarray, np.ndarray]:
+    """Rows (request, first token, tokens, chunk of the portion) for the chunked WKV and delta-rule kernels, and the requests whose
     portions do not fit what is left of ``chunk_cap`` chunks: those go token by token."""
     rows, seq = [], []
     for b in range(n_dec, qo_indptr.size - 1):
         t0, n = int(qo_indptr[b]), int(qo_indptr[b + 1] - qo_indptr[b])
-        if len(rows) + -(-n // WKV_CHUNK) > chunk_cap:
+        if len(rows) + -(-n // CHUNK) > chunk_cap:
             seq.append(b)
             continue
-        rows += [(b, t0 + c, min(WKV_CHUNK, n - c), c // WKV_CHUNK) for c in range(0, n, WKV_CHUNK)]
+        rows += [(b, t0 + c, min(CHUNK, n - c), c // CHUNK) for c in range(0, n, CHUNK)]
     return np.asarray(rows, dtype=np.int32).reshape(-1, 4), np.asarray(seq, dtype=np.int32)
 
 

@@ -15,7 +15,7 @@ from nanoflow_b200.models.safetensors_io import read_safetensors, write_safetens
 from nanoflow_b200.ops import reference as ref
 from nanoflow_b200.replay import TraceReplay
 from nanoflow_b200.runtime.cpu_layer_list import CpuLayerListEngine
-from nanoflow_b200.runtime.layer_list import query_items, wkv_work
+from nanoflow_b200.runtime.layer_list import chunk_work, query_items
 from nanoflow_b200.serving import DistKVPool, RequestManager, Scheduler, StateSlotPool
 from nanoflow_b200.serving.loop import ServingLoop
 from volarax_cases import prompt, row_errors
@@ -126,12 +126,12 @@ def test_groups_left_out_lose_even_to_negative_choice_scores():
 # ---- work lists ---------------------------------------------------------------------------------------------------
 def test_wkv_chunks_cover_portions_in_order_and_the_rest_goes_token_by_token():
     qo = np.asarray([0, 1, 2, 132, 134, 198, 300], dtype=np.int32)      # two single tokens, portions of 130, 2, 64, 102
-    items, seq = wkv_work(qo, 2, 100)
+    items, seq = chunk_work(qo, 2, 100)
     assert seq.size == 0 and items.tolist() == [[2, 2, 64, 0], [2, 66, 64, 1], [2, 130, 2, 2], [3, 132, 2, 0], [4, 134, 64, 0],
                                                 [5, 198, 64, 0], [5, 262, 38, 1]]
-    items, seq = wkv_work(qo, 2, 5)
+    items, seq = chunk_work(qo, 2, 5)
     assert seq.tolist() == [5] and items.shape == (5, 4)
-    items, seq = wkv_work(qo, 2, 0)
+    items, seq = chunk_work(qo, 2, 0)
     assert seq.tolist() == [2, 3, 4, 5] and items.shape == (0, 4)
     assert query_items(qo, 2, 42).tolist() == [[2, 2, 42], [2, 44, 42], [2, 86, 42], [2, 128, 4], [3, 132, 2], [4, 134, 42],
                                                [4, 176, 22], [5, 198, 42], [5, 240, 42], [5, 282, 18]]

@@ -14,7 +14,7 @@ from nanoflow_b200.models import zubedra
 from nanoflow_b200.models.registry import family
 from nanoflow_b200.ops import layer_list as K
 from nanoflow_b200.replay import TraceReplay
-from nanoflow_b200.runtime.layer_list import query_items, wkv_work
+from nanoflow_b200.runtime.layer_list import query_items, chunk_work
 from nanoflow_b200.serving import DistKVPool, RequestManager, Scheduler, StateSlotPool
 from nanoflow_b200.serving.loop import ServingLoop
 from volarax_cases import prompt, row_errors
@@ -286,7 +286,7 @@ class WkvCase:
         if how == "decode":
             kw["decode"] = len(tokens)
         else:
-            items, seq = wkv_work(qo, 0, {"chunks": 1 << 20, "seq": 0, "both": 4}[how])
+            items, seq = chunk_work(qo, 0, {"chunks": 1 << 20, "seq": 0, "both": 4}[how])
             kw = dict(items=i32(items) if items.size else None, seq=i32(seq) if seq.size else None)
         K.wkv(rkvg, self.pad(self.x[sel]), self.pad(self.u[None])[0], self.pad(self.norm[None])[0], self.state, y, i32(pos), i32(qo),
               i32([2 * (b + 1) + self.at[b] % 2 for b in tokens]), dim_real=self.dim, eps=1e-4, status=st, **kw)
