@@ -10,7 +10,7 @@
 //                    a lower-triangular system with the same matrix for all columns. Three kernels:
 //                    1. per chunk: the decayed scores <k, k> and <q, k>, the inverse M = (1 + diag(beta) <k, k>)^-1 diag(beta)
 //                       (forward substitution in fp32, by blocks of 16), then M V and W = M (e^c k);
-//                    2. along the chunks, 32 columns of S per CTA, S in registers: u = M V - W S0, the outputs
+//                    2. along the chunks, 64 columns of S per CTA, S in registers: u = M V - W S0, the outputs
 //                       (e^c q) S0 + <q, k> u, and S = e^c_end S0 + (e^(c_end - c) k)^T u;
 //                    3. head norm, weight and gate.
 //                    Decayed rows, scores, W, u and S enter the products as bf16 pairs (high and low part, about 16 bits).
@@ -26,6 +26,13 @@ namespace {
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float delta_decay(float x, float bias, float rate) { return expf(-rate * softplus_f(x + bias)); }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+// With the special-function unit's exponential and logarithm; small values by their series, which keeps them exact to a
+// few units in the last place.
+__device__ __forceinline__ float softplus_fast(float x) {
+  const float e = __expf(x);
+  return x > 20.f ? x : e < 0.015625f ? e * (1.f - e * (0.5f - e * (0.33333333f - 0.25f * e))) : __logf(1.f + e);
+}
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 
 struct DeltaState {
   float* S;
@@ -256,10 +263,11 @@ delta_norm_kernel(nfk_delta_params p) {
   const int req = CHUNKS ? 0 : p.seq_reqs[blockIdx.y];
   const int t0 = CHUNKS ? p.items[blockIdx.y * 4 + 1] : p.qo_indptr[req];
   const int n = CHUNKS ? p.items[blockIdx.y * 4 + 2] : p.qo_indptr[req + 1] - t0;
-  const long long total = static_cast<long long>(n) * p.heads;
-  for (long long i = blockIdx.x * 8ll + (threadIdx.x >> 5); i < total; i += gridDim.x * 8ll) {
-    const long long t = t0 + i / p.heads;
-    const int head = static_cast<int>(i % p.heads);
+  const unsigned total = static_cast<unsigned>(n) * p.heads;
+  for (unsigned i = blockIdx.x * 8u + (threadIdx.x >> 5); i < total; i += gridDim.x * 8u) {
+    const unsigned row = i / static_cast<unsigned>(p.heads);
+    const long long t = t0 + static_cast<long long>(row);
+    const int head = static_cast<int>(i - row * p.heads);
     const float* o = p.o + (t * p.heads + head) * p.vdim;
     float ss = 0.f;
     for (int c = lane * 4; c < p.vdim; c += 128) {
@@ -271,42 +279,57 @@ delta_norm_kernel(nfk_delta_params p) {
     T* y = reinterpret_cast<T*>(p.y) + t * p.ld_y + head * p.vdim;
     for (int c = lane * 4; c < p.vdim; c += 128) {
       const float4 v = load4(o + c), w = load4(p.norm + c), gg = load4(g + c);
-      store4(y + c, make_float4(v.x * inv * w.x * sigmoid_f(gg.x), v.y * inv * w.y * sigmoid_f(gg.y),
-                                v.z * inv * w.z * sigmoid_f(gg.z), v.w * inv * w.w * sigmoid_f(gg.w)));
+      if (CHUNKS)
+        store4(y + c, make_float4(v.x * inv * w.x * sigmoid_fast(gg.x), v.y * inv * w.y * sigmoid_fast(gg.y),
+                                  v.z * inv * w.z * sigmoid_fast(gg.z), v.w * inv * w.w * sigmoid_fast(gg.w)));
+      else
+        store4(y + c, make_float4(v.x * inv * w.x * sigmoid_f(gg.x), v.y * inv * w.y * sigmoid_f(gg.y),
+                                  v.z * inv * w.z * sigmoid_f(gg.z), v.w * inv * w.w * sigmoid_f(gg.w)));
     }
   }
 }
 
 // ---- prefill, chunks of 64 tokens -------------------------------------------------------------------------------
-constexpr int kChunk = 64, kRun = 16, kRuns = kChunk / kRun, kDcThreads = 512, kDsThreads = 256;
-constexpr int kSlice = 32;                 // columns of S per CTA of the second kernel
+constexpr int kChunk = 64, kRun = 16, kRuns = kChunk / kRun, kDcThreads = 1024, kDsThreads = 512;
+constexpr int kDcWarps = kDcThreads / 32;
+constexpr int kSlice = 64;                 // columns of S per CTA of the second kernel
 constexpr float kMaxRunLog2 = 110.f;       // largest decay of a run (log2) whose weights are factored inside the run
 constexpr float kMaxDecayLog2 = 150.f;     // a stronger decay is zero in fp32 anyway
 
-// Scratch of a chunk and head: W, decayed keys, decayed queries [64][dim] and scores [64][64] as bf16 pairs (high parts,
-// then low parts), M V [64][vdim] fp32, the chunk's decay [dim].
+// Scratch of a chunk and head, laid out as the second kernel keeps it in shared memory (padded rows), so that a few bulk
+// copies bring it in: W [2 parts][64][P + 8] | decayed keys, decayed queries alike | scores [2][64][72] | the chunk's decay
+// [P] fp32 | M V [P / 64 slices][64][68] fp32. P: the head's size rounded up to 64 or 128, columns past it are zero.
+template <int P>
 struct DeltaItem {
+  static constexpr int BLD = P + 8, MLD = kChunk + 8, ULD = kSlice + 4;
+  static constexpr int PAIR = 2 * kChunk * BLD * 2, A = 2 * kChunk * MLD * 2, U = kChunk * ULD * 4;      // bytes
+  static constexpr int REST = 2 * PAIR + A + P * 4;
+  static constexpr int BYTES = PAIR + REST + P / kSlice * U;
   __nv_bfloat16 *w, *k, *q, *a;
-  float *u, *decay;
+  float *decay, *u;
+  __device__ __forceinline__ DeltaItem(const nfk_delta_params& p, int item, int head) {
+    char* b = reinterpret_cast<char*>(p.scratch) + (static_cast<long long>(item) * p.heads + head) * BYTES;
+    w = reinterpret_cast<__nv_bfloat16*>(b);
+    k = reinterpret_cast<__nv_bfloat16*>(b + PAIR);
+    q = reinterpret_cast<__nv_bfloat16*>(b + 2 * PAIR);
+    a = reinterpret_cast<__nv_bfloat16*>(b + 3 * PAIR);
+    decay = reinterpret_cast<float*>(b + 3 * PAIR + A);
+    u = reinterpret_cast<float*>(b + PAIR + REST);
+  }
 };
 __host__ __device__ __forceinline__ long long delta_item_floats(int dim, int vdim) {
-  return 3ll * kChunk * dim + kChunk * kChunk + static_cast<long long>(kChunk) * vdim + dim;
-}
-__device__ __forceinline__ DeltaItem delta_item(const nfk_delta_params& p, int item, int head) {
-  float* f = p.scratch + (static_cast<long long>(item) * p.heads + head) * delta_item_floats(p.dim, p.vdim);
-  DeltaItem d;
-  d.w = reinterpret_cast<__nv_bfloat16*>(f);
-  d.k = d.w + 2 * kChunk * p.dim;
-  d.q = d.k + 2 * kChunk * p.dim;
-  d.a = d.q + 2 * kChunk * p.dim;
-  d.u = f + 3 * kChunk * p.dim + kChunk * kChunk;
-  d.decay = d.u + kChunk * p.vdim;
-  return d;
+  return (dim <= 64 && vdim <= 64 ? DeltaItem<64>::BYTES : DeltaItem<128>::BYTES) / 4;
 }
 __device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(x, y);
   const float2 h = unpack_bf16x2(hi);
   lo = pack_bf16x2(x - h.x, y - h.y);
+}
+// Untiled bulk copy global -> shared, counted by an mbarrier.
+__device__ __forceinline__ void bulk_load(void* smem_dst, const void* src, int bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(smem_dst)),
+               "l"(src), "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
 }
 __device__ __forceinline__ void cp_async16_or_zero(void* smem_dst, const void* src, bool ok) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
@@ -348,7 +371,7 @@ delta_chunk_kernel(nfk_delta_params p) {
   const int head = blockIdx.x % p.heads, item = blockIdx.x / p.heads, kvh = head / (p.heads / p.kv_heads);
   const int n = p.items[item * 4 + 2];
   const long long tok0 = p.items[item * 4 + 1];
-  const DeltaItem out = delta_item(p, item, head);
+  const DeltaItem<P> out(p, item, head);
 
   // ---- operands: all requested before any of them is waited for ----
   {
@@ -371,8 +394,8 @@ delta_chunk_kernel(nfk_delta_params p) {
     float4 l = make_float4(0.f, 0.f, 0.f, 0.f);           // no decay past the last token: the chunk's is that of its tokens
     if (r < n && c < p.dim) {
       const float4 x = load4(p.x + (tok0 + r) * p.ld_x + head * p.dim + c), b = load4(p.dt_bias + head * p.dim + c);
-      l = make_float4(-fminf(rate * softplus_f(x.x + b.x), kMaxDecayLog2), -fminf(rate * softplus_f(x.y + b.y), kMaxDecayLog2),
-                      -fminf(rate * softplus_f(x.z + b.z), kMaxDecayLog2), -fminf(rate * softplus_f(x.w + b.w), kMaxDecayLog2));
+      l = make_float4(-fminf(rate * softplus_fast(x.x + b.x), kMaxDecayLog2), -fminf(rate * softplus_fast(x.y + b.y), kMaxDecayLog2),
+                      -fminf(rate * softplus_fast(x.z + b.z), kMaxDecayLog2), -fminf(rate * softplus_fast(x.w + b.w), kMaxDecayLog2));
     }
     store4(ce + r * C::FLD + c, l);
   }
@@ -394,8 +417,8 @@ delta_chunk_kernel(nfk_delta_params p) {
     if (s < -kMaxRunLog2) slow_s[run] = 1;
   }
 #pragma unroll
-  for (int j = 0; j < kChunk / 16; ++j) {
-    const int t = warp * (kChunk / 16) + j;
+  for (int j = 0; j < kChunk / kDcWarps; ++j) {
+    const int t = warp * (kChunk / kDcWarps) + j;
     float sq = 0.f, sk = 0.f;
     for (int d = lane * 2; d < P; d += 64) {
       const float2 a = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(q_s + t * C::BLD + d));
@@ -505,8 +528,8 @@ delta_chunk_kernel(nfk_delta_params p) {
         } else {
           uint32_t hi, lo;
           split_pair(s <= t ? x : 0.f, s + 1 <= t ? y : 0.f, hi, lo);
-          *reinterpret_cast<uint32_t*>(out.a + t * kChunk + s) = hi;
-          *reinterpret_cast<uint32_t*>(out.a + kChunk * kChunk + t * kChunk + s) = lo;
+          *reinterpret_cast<uint32_t*>(out.a + t * C::MLD + s) = hi;
+          *reinterpret_cast<uint32_t*>(out.a + kChunk * C::MLD + t * C::MLD + s) = lo;
         }
       }
   }
@@ -574,22 +597,20 @@ delta_chunk_kernel(nfk_delta_params p) {
     split_pair(k.x * kf * ex, k.y * kf * ey, hi, lo);
     *reinterpret_cast<uint32_t*>(kh_s + t * C::BLD + d) = hi;
     *reinterpret_cast<uint32_t*>(kl_s + t * C::BLD + d) = lo;
-    if (d < p.dim) {
-      const int o = t * p.dim + d, low = kChunk * p.dim;
-      split_pair(q.x * qf * ex, q.y * qf * ey, hi, lo);
-      *reinterpret_cast<uint32_t*>(out.q + o) = hi;
-      *reinterpret_cast<uint32_t*>(out.q + low + o) = lo;
-      split_pair(k.x * kf * fast_exp2(after.x), k.y * kf * fast_exp2(after.y), hi, lo);
-      *reinterpret_cast<uint32_t*>(out.k + o) = hi;
-      *reinterpret_cast<uint32_t*>(out.k + low + o) = lo;
-    }
+    const int o = t * C::BLD + d, low = kChunk * C::BLD;
+    split_pair(q.x * qf * ex, q.y * qf * ey, hi, lo);
+    *reinterpret_cast<uint32_t*>(out.q + o) = hi;
+    *reinterpret_cast<uint32_t*>(out.q + low + o) = lo;
+    split_pair(k.x * kf * fast_exp2(after.x), k.y * kf * fast_exp2(after.y), hi, lo);
+    *reinterpret_cast<uint32_t*>(out.k + o) = hi;
+    *reinterpret_cast<uint32_t*>(out.k + low + o) = lo;
   }
-  for (int d = threadIdx.x; d < p.dim; d += kDcThreads)
+  for (int d = threadIdx.x; d < P; d += kDcThreads)
     out.decay[d] = fast_exp2((tot[d] + tot[P + d]) + (tot[2 * P + d] + tot[3 * P + d]));
   __syncthreads();
 
-  // ---- M V and W = M (decayed keys): a warp takes a run of rows and a quarter of the columns ----
-  constexpr int NT = P / 8 / 4;
+  // ---- M V and W = M (decayed keys): a warp takes a run of rows and an eighth of the columns ----
+  constexpr int NT = P / 8 / (kDcWarps / 4);
   const int a = warp & 3, n0 = (warp >> 2) * NT;
   float u[NT][4], w[NT][4];
 #pragma unroll
@@ -603,23 +624,28 @@ delta_chunk_kernel(nfk_delta_params p) {
     const uint32_t mo = ((a * kRun + (lane & 15)) * C::MLD + ks * 16 + (lane >> 4) * 8) * 2;
     ldsm_x4(mhb + mo, mh[0], mh[1], mh[2], mh[3]);
     ldsm_x4(mlb + mo, ml[0], ml[1], ml[2], ml[3]);
+    // two blocks of columns per load; a warp with one block (the small size) loads its neighbour's too
 #pragma unroll
     for (int i = 0; i < NT; i += 2) {
-      const uint32_t o = ((ks * 16 + (mm & 1) * 8 + rr) * C::BLD + (n0 + i + (mm >> 1)) * 8) * 2;
+      const uint32_t o = ((ks * 16 + (mm & 1) * 8 + rr) * C::BLD + (NT == 1 ? n0 : n0 + i + (mm >> 1)) * 8) * 2;
       uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
       ldsm_x4_trans(vb + o, h0, h1, h2, h3);
       mma_bf16(u[i], mh, h0, h1);
-      mma_bf16(u[i + 1], mh, h2, h3);
       mma_bf16(u[i], ml, h0, h1);
-      mma_bf16(u[i + 1], ml, h2, h3);
+      if (NT > 1) {
+        mma_bf16(u[i + 1 < NT ? i + 1 : i], mh, h2, h3);
+        mma_bf16(u[i + 1 < NT ? i + 1 : i], ml, h2, h3);
+      }
       ldsm_x4_trans(khb + o, h0, h1, h2, h3);
       ldsm_x4_trans(klb + o, l0, l1, l2, l3);
       mma_bf16(w[i], mh, h0, h1);
-      mma_bf16(w[i + 1], mh, h2, h3);
       mma_bf16(w[i], mh, l0, l1);
-      mma_bf16(w[i + 1], mh, l2, l3);
       mma_bf16(w[i], ml, h0, h1);
-      mma_bf16(w[i + 1], ml, h2, h3);
+      if (NT > 1) {
+        mma_bf16(w[i + 1 < NT ? i + 1 : i], mh, h2, h3);
+        mma_bf16(w[i + 1 < NT ? i + 1 : i], mh, l2, l3);
+        mma_bf16(w[i + 1 < NT ? i + 1 : i], ml, h2, h3);
+      }
     }
   }
 #pragma unroll
@@ -627,37 +653,36 @@ delta_chunk_kernel(nfk_delta_params p) {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int t = a * kRun + (lane >> 2) + h * 8, c = (n0 + i) * 8 + (lane & 3) * 2;
-      if (c < p.vdim) *reinterpret_cast<float2*>(out.u + t * p.vdim + c) = make_float2(u[i][2 * h], u[i][2 * h + 1]);
-      if (c < p.dim) {
-        uint32_t hi, lo;
-        split_pair(w[i][2 * h], w[i][2 * h + 1], hi, lo);
-        *reinterpret_cast<uint32_t*>(out.w + t * p.dim + c) = hi;
-        *reinterpret_cast<uint32_t*>(out.w + kChunk * p.dim + t * p.dim + c) = lo;
-      }
+      *reinterpret_cast<float2*>(out.u + c / kSlice * (DeltaItem<P>::U / 4) + t * DeltaItem<P>::ULD + c % kSlice) =
+          make_float2(u[i][2 * h], u[i][2 * h + 1]);
+      uint32_t hi, lo;
+      split_pair(w[i][2 * h], w[i][2 * h + 1], hi, lo);
+      *reinterpret_cast<uint32_t*>(out.w + t * C::BLD + c) = hi;
+      *reinterpret_cast<uint32_t*>(out.w + kChunk * C::BLD + t * C::BLD + c) = lo;
     }
 }
 
 template <int P>
 struct DeltaScanCfg {
-  static constexpr int BLD = P + 8, MLD = kChunk + 8, SLD = kSlice + 8, ULD = kSlice + 4;
-  static constexpr int ROWS = kChunk * BLD * 2, A = kChunk * MLD * 2, S = P * SLD * 2, U = kChunk * SLD * 2;
-  // W, K, Q (pairs) | A (pair) | M V | S (pair) | u (pair) | decay
-  static constexpr int SMEM = 6 * ROWS + 2 * A + kChunk * ULD * 4 + 2 * S + 2 * U + P * 4;
+  using I = DeltaItem<P>;
+  static constexpr int BLD = I::BLD, MLD = I::MLD, SLD = kSlice + 8, ULD = I::ULD;
+  static constexpr int S = P * SLD * 2, U = kChunk * SLD * 2;            // one part
+  // W | M V | the rest of a chunk's scratch | S (pair) | u (pair) | barriers
+  static constexpr int SMEM = I::PAIR + I::U + I::REST + 2 * S + 2 * U + 64;
 };
 
 template <int P>
 __global__ void __launch_bounds__(kDsThreads, 1)
 delta_scan_kernel(nfk_delta_params p, int slices) {
   using C = DeltaScanCfg<P>;
+  using I = DeltaItem<P>;
   extern __shared__ __align__(16) uint8_t smem[];
-  __nv_bfloat16* w_s = reinterpret_cast<__nv_bfloat16*>(smem);
-  __nv_bfloat16* k_s = w_s + 2 * kChunk * C::BLD;
-  __nv_bfloat16* q_s = k_s + 2 * kChunk * C::BLD;
-  __nv_bfloat16* a_s = q_s + 2 * kChunk * C::BLD;
-  float* mv_s = reinterpret_cast<float*>(a_s + 2 * kChunk * C::MLD);
-  __nv_bfloat16* s_s = reinterpret_cast<__nv_bfloat16*>(mv_s + kChunk * C::ULD);
+  uint8_t *w_b = smem, *mv_b = w_b + I::PAIR, *rest_b = mv_b + I::U;
+  float* mv_s = reinterpret_cast<float*>(mv_b);
+  float* decay_s = reinterpret_cast<float*>(rest_b + 2 * I::PAIR + I::A);
+  __nv_bfloat16* s_s = reinterpret_cast<__nv_bfloat16*>(rest_b + I::REST);
   __nv_bfloat16* u_s = s_s + 2 * P * C::SLD;
-  float* decay_s = reinterpret_cast<float*>(u_s + 2 * kChunk * C::SLD);
+  uint64_t* bar = reinterpret_cast<uint64_t*>(reinterpret_cast<uint8_t*>(u_s) + 2 * C::U);       // first part, rest
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int v0 = (blockIdx.x % slices) * kSlice, head = (blockIdx.x / slices) % p.heads, item0 = blockIdx.x / (slices * p.heads);
   if (p.items[item0 * 4 + 3] != 0) return;                 // not the first chunk of a portion
@@ -668,35 +693,27 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
   const int chunks = min((n_tok + kChunk - 1) / kChunk, p.num_items - item0);
   const long long tok0 = p.qo_indptr[req];
 
-  // rows of `cols` elements as 16-byte pieces; columns past `have` become zeros
-  auto copy = [&](void* dst, int dst_row_bytes, const void* src, int src_row_bytes, int rows, int row_bytes, int have_bytes) {
-    const int per = row_bytes / 16;
-    for (int i = threadIdx.x; i < rows * per; i += kDsThreads) {
-      const int r = i / per, b = (i % per) * 16;
-      const bool ok = b < have_bytes;
-      cp_async16_or_zero(static_cast<char*>(dst) + r * dst_row_bytes + b,
-                         static_cast<const char*>(src) + static_cast<long long>(r) * src_row_bytes + (ok ? b : 0), ok);
-    }
-  };
-  auto fetch_first = [&](int c) {                          // what the values written need
-    const DeltaItem d = delta_item(p, item0 + c, head);
-    copy(w_s, C::BLD * 2, d.w, p.dim * 2, 2 * kChunk, P * 2, p.dim * 2);
-    copy(mv_s, C::ULD * 4, d.u + v0, p.vdim * 4, kChunk, kSlice * 4, (p.vdim - v0) * 4);
-    cp_async_commit();
+  auto fetch_first = [&](int c) {                          // what the values written need; one thread
+    const I d(p, item0 + c, head);
+    mbar_expect_tx(&bar[0], I::PAIR + I::U);
+    bulk_load(w_b, d.w, I::PAIR, &bar[0]);
+    bulk_load(mv_b, d.u + v0 / kSlice * (I::U / 4), I::U, &bar[0]);
   };
   auto fetch_rest = [&](int c) {
-    const DeltaItem d = delta_item(p, item0 + c, head);
-    copy(k_s, C::BLD * 2, d.k, p.dim * 2, 2 * kChunk, P * 2, p.dim * 2);
-    copy(q_s, C::BLD * 2, d.q, p.dim * 2, 2 * kChunk, P * 2, p.dim * 2);
-    copy(a_s, C::MLD * 2, d.a, kChunk * 2, 2 * kChunk, kChunk * 2, kChunk * 2);
-    copy(decay_s, P * 4, d.decay, p.dim * 4, 1, P * 4, p.dim * 4);
-    cp_async_commit();
+    const I d(p, item0 + c, head);
+    mbar_expect_tx(&bar[1], I::REST);
+    bulk_load(rest_b, d.k, I::REST, &bar[1]);
   };
-  fetch_first(0);
-  fetch_rest(0);
+  if (threadIdx.x == 0) {
+    mbar_init(&bar[0], 1);
+    mbar_init(&bar[1], 1);
+    mbar_fence_init();
+    fetch_first(0);
+    fetch_rest(0);
+  }
 
-  // ---- S: warps over 16-row tiles of the key channels and, for the small size, halves of the columns ----
-  constexpr int MT = P / 16, SN = kSlice / 8 * MT / 8;     // row tiles; column blocks per warp
+  // ---- S: warps over 16-row tiles of the key channels and parts of the columns ----
+  constexpr int MT = P / 16, SN = kSlice / 8 * MT / (kDsThreads / 32);     // row tiles; column blocks per warp
   const int sm0 = (warp % MT) * 16, sn0 = (warp / MT) * SN;
   const int d0 = sm0 + (lane >> 2), d1 = d0 + 8;
   float S[SN][4];
@@ -725,13 +742,14 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
       }
   };
   publish();
+  __syncthreads();                                         // also: the barriers are set up
 
   const int mm = lane >> 3, rr = lane & 7;
-  const int a = warp & 3, c0 = (warp >> 2) * 16;           // this warp's run of rows and half of the columns
+  const int a = warp & 3, c0 = (warp >> 2) * 16;           // this warp's run of rows and its columns
   const int t0 = a * kRun + (lane >> 2);
-  const uint32_t wb = smem_u32(w_s), kb = smem_u32(k_s), qb = smem_u32(q_s), ab = smem_u32(a_s), sb = smem_u32(s_s), ub = smem_u32(u_s);
-  constexpr uint32_t R_LO = kChunk * C::BLD * 2, A_LO = kChunk * C::MLD * 2, S_LO = P * C::SLD * 2, U_LO = kChunk * C::SLD * 2;
-  // acc += rows (pair, of this warp's run) x S (pair, this warp's half of the columns)
+  const uint32_t wb = smem_u32(w_b), kb = smem_u32(rest_b), qb = kb + I::PAIR, ab = qb + I::PAIR, sb = smem_u32(s_s), ub = smem_u32(u_s);
+  constexpr uint32_t R_LO = I::PAIR / 2, A_LO = kChunk * C::MLD * 2, S_LO = P * C::SLD * 2, U_LO = kChunk * C::SLD * 2;
+  // acc += rows (pair, of this warp's run) x S (pair, this warp's columns)
   auto rows_times_s = [&](float (&acc)[2][4], uint32_t base) {
 #pragma unroll
     for (int ks = 0; ks < P / 16; ++ks) {
@@ -752,7 +770,8 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
   };
 
   for (int c = 0; c < chunks; ++c) {
-    cp_async_wait<1>();
+    // a wait that runs out is reported; the warps go on in step, so that they meet at their barriers
+    if (!mbar_wait(&bar[0], c & 1)) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
     __syncthreads();                                       // W and M V are there, S is published
     float acc[2][4];
 #pragma unroll
@@ -769,10 +788,9 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
         *reinterpret_cast<uint32_t*>(u_s + t * C::SLD + col) = hi;
         *reinterpret_cast<uint32_t*>(u_s + kChunk * C::SLD + t * C::SLD + col) = lo;
       }
-    cp_async_wait<0>();
+    if (!mbar_wait(&bar[1], c & 1)) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
     __syncthreads();                                       // the rest is there, u is written, W and M V are read
-    if (c + 1 < chunks) fetch_first(c + 1);
-    else cp_async_commit();
+    if (threadIdx.x == 0 && c + 1 < chunks) fetch_first(c + 1);
     // ---- outputs ----
 #pragma unroll
     for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
@@ -832,11 +850,9 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
       }
     }
     __syncthreads();                                       // S, u and the copies are read
+    if (threadIdx.x == 0 && c + 1 < chunks) fetch_rest(c + 1);
     publish();
-    if (c + 1 < chunks) fetch_rest(c + 1);
-    else cp_async_commit();
   }
-  cp_async_wait<0>();
 #pragma unroll
   for (int i = 0; i < SN; ++i) {
     const int c = v0 + (sn0 + i) * 8 + (lane & 3) * 2;

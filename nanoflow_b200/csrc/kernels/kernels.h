@@ -270,6 +270,14 @@ typedef struct nfk_residual_norm_params {
   const float* pair_w;       // [cols] padded, null: none
   const float* pair_w2;
   int table_add;
+  // Input convolution of the next sublayer (see nfk_short_conv, residual form) for the first conv_rows rows, each the only
+  // token of the request of the same number: the result goes to conv_out instead of h's row.
+  const float* conv_w;       // [conv_taps][conv_ld], null: none
+  void* conv_out;            // [*, conv_ld]
+  void* conv_state;          // [slots][2][max(1, conv_taps - 1)][conv_ld]
+  const int* state_slot;
+  const int* positions;
+  int conv_taps, conv_rows, conv_ld, num_slots;
 } nfk_residual_norm_params;
 int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t stream);
 

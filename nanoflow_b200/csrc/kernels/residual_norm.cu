@@ -4,7 +4,8 @@
 //   x <- (table ? 0 : x) + norm_in(src) (+ second output) (+ weighted expert outputs) (+ add);   h = norm_out(x)
 //
 // The norm can also be taken of the whole sum, the source can be the mean of two normed outputs, and the embedding row
-// can join a stream that goes on (see kernels.h).
+// can join a stream that goes on (see kernels.h). Where the next sublayer reads its input through a convolution over time,
+// rows that are the only token of their request get it here, from the request's state.
 // `src` is the sublayer's output row, or the embedding row of the token (ids as in nfk_embedding, with the
 // previous iteration's tokens fed back on the device). Norms are RMS or layer norms with fp32 weights. The
 // stream x is fp32; src and h are bf16 or fp32. One CTA per row, the row stays in registers.
@@ -66,6 +67,38 @@ __device__ __forceinline__ void norm_row(float4 (&v)[NV], int kind, const float*
       v[i].z = v[i].z * inv * ww.z + bb.z;
       v[i].w = v[i].w * inv * ww.w + bb.w;
     }
+  }
+}
+
+__device__ __forceinline__ float4 rounded(float4 v, float) { return v; }
+__device__ __forceinline__ float4 rounded(float4 v, __nv_bfloat16) {
+  const float2 a = unpack_bf16x2(pack_bf16x2(v.x, v.y)), b = unpack_bf16x2(pack_bf16x2(v.z, v.w));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+// The normed row v of a request's only token plus its convolution with the inputs kept in the request's state.
+template <class T, int NV>
+__device__ __forceinline__ void input_conv(const float4 (&v)[NV], const nfk_residual_norm_params& p, int row, int nvec) {
+  const int ref = p.state_slot[row], before = p.conv_taps - 1;
+  const bool ok = ref >= 0 && (ref >> 1) < p.num_slots, older = ok && p.positions[row] > 0;
+  if (!ok && threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
+  const long long half = static_cast<long long>(before > 0 ? before : 1) * p.conv_ld;
+  const T* st = reinterpret_cast<const T*>(p.conv_state) + (ok ? ref : 0) * half;
+  T* keep = reinterpret_cast<T*>(p.conv_state) + (ok ? ref ^ 1 : 0) * half;
+  T* out = reinterpret_cast<T*>(p.conv_out) + static_cast<long long>(row) * p.conv_ld;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int vi = threadIdx.x + i * kRnThreads;
+    if (vi >= nvec) continue;
+    const float4 x = rounded(v[i], T(0.f)), w = load4(p.conv_w + static_cast<long long>(before) * p.conv_ld + vi * 4);
+    float4 y = make_float4(x.x + w.x * x.x, x.y + w.y * x.y, x.z + w.z * x.z, x.w + w.w * x.w);
+    for (int j = 0; j < before; ++j) {
+      const float4 s = older ? load4(st + static_cast<long long>(j) * p.conv_ld + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 f = load4(p.conv_w + static_cast<long long>(j) * p.conv_ld + vi * 4);
+      y.x += f.x * s.x; y.y += f.y * s.y; y.z += f.z * s.z; y.w += f.w * s.w;
+      if (ok && j > 0) store4(keep + static_cast<long long>(j - 1) * p.conv_ld + vi * 4, s);
+    }
+    if (ok && before > 0) store4(keep + static_cast<long long>(before - 1) * p.conv_ld + vi * 4, x);
+    store4(out + vi * 4, y);
   }
 }
 
@@ -177,6 +210,10 @@ residual_norm_kernel(nfk_residual_norm_params p) {
     }
     if (p.h != nullptr) {
       norm_row<NV>(v, p.out_kind, p.out_w, p.out_b, p.cols, nvec, p.eps, red);
+      if (p.conv_w != nullptr && row < p.conv_rows) {
+        input_conv<T, NV>(v, p, row, nvec);
+        continue;
+      }
       T* hr = reinterpret_cast<T*>(p.h) + static_cast<long long>(row) * p.ld_h;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
@@ -215,6 +252,9 @@ extern "C" int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t
   if (p->rows_idx && (p->in_rows <= 0 || !p->h)) return NF_ERR_BAD_ARG;
   if (p->y2 && p->ld_y2 % 4 != 0) return NF_ERR_BAD_ARG;
   if (p->e_out && (!p->e_slot || !p->e_weight || p->e_top <= 0 || p->e_rows <= 0 || p->ld_e % 4 != 0)) return NF_ERR_BAD_ARG;
+  if (p->conv_w && (!p->conv_out || !p->conv_state || !p->state_slot || !p->positions || !p->h || p->conv_taps <= 0 ||
+                    p->conv_rows < 0 || p->conv_ld < p->cols || p->conv_ld % 4 != 0 || p->num_slots <= 0 || p->rows_idx))
+    return NF_ERR_BAD_ARG;
   if (p->pair_w && (!p->pair_w2 || !p->y || !p->y2)) return NF_ERR_BAD_ARG;
   if (p->norm_sum && p->in_kind != NFK_NORM_NONE && !p->in_w) return NF_ERR_BAD_ARG;
   for (int kind : {p->in_kind, p->out_kind})

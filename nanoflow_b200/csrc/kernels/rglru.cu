@@ -2,9 +2,9 @@
 // Language Models"; see kernels.h for the equations). State, gates, decays and their logarithms are fp32.
 //
 // nfk_rglru_decode   one token per request: a thread per channel.
-// nfk_rglru_prefill  a CTA takes 32 channels of a request and walks its tokens 256 at a time: each of 32 warps reduces
-//                    eight tokens to (decay, end state from zero), one warp chains those, and every warp then runs its
-//                    tokens again from the state it starts with, out of registers. Inputs are read once.
+// nfk_rglru_prefill  a CTA takes 32 channels of a request and walks its tokens 128 at a time: each of 16 warps reduces
+//                    eight tokens to (decay, end state from zero), all chain those, and every warp then runs its tokens
+//                    again from the state it starts with, out of registers. Inputs are read once, a step ahead.
 #include "elem_io.cuh"
 
 namespace nf {
@@ -13,17 +13,36 @@ namespace {
 struct RgStep {
   float a, b;      // S <- a S + b
 };
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+// FAST (bf16 results): exponentials, reciprocals and square roots of the special-function unit, a few units in the last
+// place of fp32; 1 - a^2 of slow decays by the exponential's series, so that it does not cancel.
+template <bool FAST>
+__device__ __forceinline__ float sigmoid_f(float z) {
+  return FAST ? __fdividef(1.f, 1.f + __expf(-z)) : 1.f / (1.f + expf(-z));
+}
+template <bool FAST>
 __device__ __forceinline__ RgStep rg_step(float r, float i, float u, float r_b, float i_b, float log_a) {
-  const float la = log_a * sigmoid_f(r + r_b);
+  const float la = log_a * sigmoid_f<FAST>(r + r_b);
   RgStep s;
-  s.a = expf(la);
-  s.b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(i + i_b) * u;
+  float rest;      // sqrt(1 - a^2)
+  if (FAST) {
+    const float x = -2.f * la;
+    s.a = __expf(la);
+    const float d = x < 0.03125f ? x * (1.f - x * (0.5f - x * (0.16666667f - x * 0.041666667f))) : 1.f - s.a * s.a;
+    asm("sqrt.approx.f32 %0, %1;" : "=f"(rest) : "f"(d));
+  } else {
+    s.a = expf(la);
+    rest = sqrtf(-expm1f(2.f * la));
+  }
+  s.b = rest * sigmoid_f<FAST>(i + i_b) * u;
   return s;
 }
+template <bool FAST>
 __device__ __forceinline__ float gelu_tanh_f(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  const float w = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return FAST ? z * sigmoid_f<true>(2.f * w) : 0.5f * z * (1.f + tanhf(w));
 }
+template <class T>
+constexpr bool kFast = sizeof(T) == 2;
 // Column of a channel's recurrence gate; its input gate is `block` columns on.
 __device__ __forceinline__ int gate_col(int c, int block) { return c / block * 2 * block + c % block; }
 
@@ -41,18 +60,25 @@ rglru_decode_kernel(nfk_rglru_params p) {
   const long long t = p.qo_indptr[req];
   float* S = p.S + static_cast<long long>(ref >> 1) * p.cols + c;
   const float* g = p.gates + t * p.ld_g + gate_col(c, p.block);
-  const RgStep s = rg_step(g[0], g[p.block], to_f32(reinterpret_cast<const T*>(p.u)[t * p.ld_u + c]), p.r_b[c], p.i_b[c], p.log_a[c]);
+  const RgStep s = rg_step<kFast<T>>(g[0], g[p.block], to_f32(reinterpret_cast<const T*>(p.u)[t * p.ld_u + c]), p.r_b[c], p.i_b[c], p.log_a[c]);
   const float x = s.a * (p.positions[t] == 0 ? 0.f : *S) + s.b;
   *S = x;
-  put(reinterpret_cast<T*>(p.out) + t * p.ld_out + c, x * gelu_tanh_f(to_f32(reinterpret_cast<const T*>(p.y)[t * p.ld_y + c])));
+  put(reinterpret_cast<T*>(p.out) + t * p.ld_out + c, x * gelu_tanh_f<kFast<T>>(to_f32(reinterpret_cast<const T*>(p.y)[t * p.ld_y + c])));
 }
 
-constexpr int kRgWarps = 32, kRgRun = 8;
+constexpr int kRgWarps = 16, kRgRun = 8, kRgBlock = kRgWarps * kRgRun;
+
+// What a thread reads of its run of tokens.
+template <class T>
+struct RgInputs {
+  float r[kRgRun], i[kRgRun];
+  T u[kRgRun], y[kRgRun];
+};
 
 template <class T>
 __global__ void __launch_bounds__(kRgWarps * 32)
 rglru_prefill_kernel(nfk_rglru_params p) {
-  __shared__ float a_s[kRgWarps][32], b_s[kRgWarps][32], carry_s[32];
+  __shared__ float a_s[2][kRgWarps][32], b_s[2][kRgWarps][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int c = blockIdx.x * 32 + lane;
   const int req = p.req_begin + blockIdx.y;
@@ -64,54 +90,57 @@ rglru_prefill_kernel(nfk_rglru_params p) {
   const bool ok = c < p.cols;
   const int t0 = p.qo_indptr[req], t1 = p.qo_indptr[req + 1];
   float* S = p.S + static_cast<long long>(ref >> 1) * p.cols + c;
-  const int gc = ok ? gate_col(c, p.block) : 0;
   const float r_b = ok ? p.r_b[c] : 0.f, i_b = ok ? p.i_b[c] : 0.f, log_a = ok ? p.log_a[c] : 0.f;
-  if (warp == 0) carry_s[lane] = (ok && p.positions[t0] != 0) ? *S : 0.f;
-  const T* u = reinterpret_cast<const T*>(p.u) + c;
-  const T* y = reinterpret_cast<const T*>(p.y) + c;
+  const T* u = reinterpret_cast<const T*>(p.u) + (ok ? c : 0);
+  const T* y = reinterpret_cast<const T*>(p.y) + (ok ? c : 0);
+  const float* g = p.gates + (ok ? gate_col(c, p.block) : 0);
   T* out = reinterpret_cast<T*>(p.out) + c;
-  for (int base = t0; base < t1; base += kRgWarps * kRgRun) {
-    const int begin = base + warp * kRgRun;
-    RgStep s[kRgRun];
-    float yy[kRgRun];
-    float a = 1.f, b = 0.f;
+  auto fetch = [&](RgInputs<T>& in, int begin) {
 #pragma unroll
     for (int j = 0; j < kRgRun; ++j) {
-      const long long t = begin + j;
+      const long long t = begin + j < t1 ? begin + j : t1 - 1;       // past the end: not used
+      in.r[j] = g[t * p.ld_g];
+      in.i[j] = g[t * p.ld_g + p.block];
+      in.u[j] = u[t * p.ld_u];
+      in.y[j] = y[t * p.ld_y];
+    }
+  };
+  float carry = (ok && p.positions[t0] != 0) ? *S : 0.f;             // every warp keeps it
+  RgInputs<T> in;
+  fetch(in, t0 + warp * kRgRun);
+  int buf = 0;
+  for (int base = t0; base < t1; base += kRgBlock, buf ^= 1) {
+    const int begin = base + warp * kRgRun;
+    RgStep s[kRgRun];
+    float yy[kRgRun], a = 1.f, b = 0.f;
+#pragma unroll
+    for (int j = 0; j < kRgRun; ++j) {
       s[j].a = 1.f;
       s[j].b = yy[j] = 0.f;
-      if (t < t1 && ok) {
-        const float* g = p.gates + t * p.ld_g + gc;
-        s[j] = rg_step(g[0], g[p.block], to_f32(u[t * p.ld_u]), r_b, i_b, log_a);
-        yy[j] = to_f32(y[t * p.ld_y]);
+      if (begin + j < t1) {
+        s[j] = rg_step<kFast<T>>(in.r[j], in.i[j], to_f32(in.u[j]), r_b, i_b, log_a);
+        yy[j] = gelu_tanh_f<kFast<T>>(to_f32(in.y[j]));
       }
       a *= s[j].a;
       b = s[j].a * b + s[j].b;
     }
-    a_s[warp][lane] = a;
-    b_s[warp][lane] = b;
+    if (base + kRgBlock < t1) fetch(in, begin + kRgBlock);           // while the warps wait for one another
+    a_s[buf][warp][lane] = a;
+    b_s[buf][warp][lane] = b;
     __syncthreads();
-    if (warp == 0) {
-      float x = carry_s[lane];
+    float x = carry;
 #pragma unroll
-      for (int k = 0; k < kRgWarps; ++k) {
-        const float next = a_s[k][lane] * x + b_s[k][lane];
-        b_s[k][lane] = x;                        // what warp k starts from
-        x = next;
-      }
-      carry_s[lane] = x;
+    for (int k = 0; k < kRgWarps; ++k) {
+      if (k == warp) x = carry;                                      // what this warp's run starts from
+      carry = a_s[buf][k][lane] * carry + b_s[buf][k][lane];
     }
-    __syncthreads();
-    float x = b_s[warp][lane];
 #pragma unroll
     for (int j = 0; j < kRgRun; ++j) {
-      const long long t = begin + j;
       x = s[j].a * x + s[j].b;
-      if (t < t1 && ok) put(out + t * p.ld_out, x * gelu_tanh_f(yy[j]));
+      if (begin + j < t1 && ok) put(out + static_cast<long long>(begin + j) * p.ld_out, x * yy[j]);
     }
-    __syncthreads();
   }
-  if (warp == 0 && ok) *S = carry_s[lane];
+  if (warp == 0 && ok) *S = carry;
 }
 
 int check_rglru(const nfk_rglru_params* p) {

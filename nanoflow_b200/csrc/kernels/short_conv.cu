@@ -9,26 +9,47 @@ namespace {
 
 constexpr int kScRun = 8, kScThreads = 128;
 
-template <class T, int TAPS>
+__device__ __forceinline__ uint2 load_raw(const __nv_bfloat16* p) { return *reinterpret_cast<const uint2*>(p); }
+__device__ __forceinline__ float4 load_raw(const float* p) { return load4(p); }
+__device__ __forceinline__ float4 as_f32(float4 v) { return v; }
+__device__ __forceinline__ float4 as_f32(uint2 u) {
+  const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <bool FAST>
+__device__ __forceinline__ float silu_f(float y) { return FAST ? __fdividef(y, 1.f + __expf(-y)) : y / (1.f + expf(-y)); }
+
+// RUN: tokens per thread.
+template <class T, int TAPS, int RUN>
 __global__ void __launch_bounds__(kScThreads)
 short_conv_kernel(nfk_short_conv_params p, int groups) {
   constexpr int H = TAPS - 1;                    // inputs before the current one
-  const long long id = blockIdx.x * static_cast<long long>(kScThreads) + threadIdx.x;
-  const int c = static_cast<int>(id % groups) * 4;
-  const int begin = p.row_begin + static_cast<int>(id / groups) * kScRun, end = min(begin + kScRun, p.T);
+  constexpr bool FAST = sizeof(T) == 2;
+  using Raw = decltype(load_raw(static_cast<const T*>(nullptr)));
+  const unsigned id = blockIdx.x * kScThreads + threadIdx.x;
+  const unsigned run = id / static_cast<unsigned>(groups);
+  const int c = static_cast<int>(id - run * groups) * 4;
+  const int begin = p.row_begin + static_cast<int>(run) * RUN, end = min(begin + RUN, p.T);
   if (begin >= end) return;
+  const T* x = reinterpret_cast<const T*>(p.x) + c;
+  Raw raw[RUN];                                  // all rows are requested before any of them is used
+#pragma unroll
+  for (int i = 0; i < RUN; ++i)
+    if (begin + i < end) raw[i] = load_raw(x + (begin + i) * p.ld_x);
   float4 w[TAPS];
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) w[j] = load4(p.w + static_cast<long long>(j) * p.cols + c);
   const float4 b = p.bias != nullptr ? load4(p.bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-  const T* x = reinterpret_cast<const T*>(p.x) + c;
   T* out = reinterpret_cast<T*>(p.out) + c;
   T* state = reinterpret_cast<T*>(p.state) + c;
   float4 hist[H > 0 ? H : 1];
   int t1 = begin;                                // end of the current request
   int ref = -1;
-  for (int t = begin; t < end; ++t) {
-    if (t == t1 || t == begin) {
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    const int t = begin + i;
+    if (t >= end) break;
+    if (t == t1 || i == 0) {
       const int req = p.token_req[t];
       const int t0 = p.qo_indptr[req];
       t1 = p.qo_indptr[req + 1];
@@ -37,7 +58,7 @@ short_conv_kernel(nfk_short_conv_params p, int groups) {
         if (c == 0) report_status(p.status, NF_ST_BAD_INDEX);
         ref = -1;
       }
-      const bool older = ref >= 0 && p.positions[t0] > 0;
+      const bool older = ref >= 0 && t - H < t0 && p.positions[t0] > 0;
       const T* st = state + static_cast<long long>(ref >= 0 ? ref : 0) * (H > 0 ? H : 1) * p.cols;
 #pragma unroll
       for (int j = 0; j < H; ++j) {
@@ -47,17 +68,14 @@ short_conv_kernel(nfk_short_conv_params p, int groups) {
         else if (older) hist[j] = load4(st + static_cast<long long>(s - t0 + H) * p.cols);
       }
     }
-    const float4 v = load4(x + t * p.ld_x);
+    const float4 v = as_f32(raw[i]);
     float4 y = b;
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
       const float4 s = j < H ? hist[j < H ? j : 0] : v;
       y.x += w[j].x * s.x; y.y += w[j].y * s.y; y.z += w[j].z * s.z; y.w += w[j].w * s.w;
     }
-    if (p.act == NFK_CONV_SILU) {
-      y.x = y.x / (1.f + expf(-y.x)); y.y = y.y / (1.f + expf(-y.y));
-      y.z = y.z / (1.f + expf(-y.z)); y.w = y.w / (1.f + expf(-y.w));
-    }
+    if (p.act == NFK_CONV_SILU) y = make_float4(silu_f<FAST>(y.x), silu_f<FAST>(y.y), silu_f<FAST>(y.z), silu_f<FAST>(y.w));
     if (p.residual != 0) {
       y.x += v.x; y.y += v.y; y.z += v.z; y.w += v.w;
     }
@@ -73,25 +91,31 @@ short_conv_kernel(nfk_short_conv_params p, int groups) {
   }
 }
 
+template <class T, int TAPS>
+int launch_taps(const nfk_short_conv_params& p, cudaStream_t stream) {
+  const int groups = p.cols / 4, rows = p.T - p.row_begin;
+  const int run = rows <= 1024 ? 1 : kScRun;     // few rows: one thread each, also for single tokens of many requests
+  const long long threads = static_cast<long long>((rows + run - 1) / run) * groups;
+  if (threads > 0x7fffffffll) return NF_ERR_BAD_ARG;
+  const int g = static_cast<int>((threads + kScThreads - 1) / kScThreads);
+  if (run == 1) short_conv_kernel<T, TAPS, 1><<<g, kScThreads, 0, stream>>>(p, groups);
+  else short_conv_kernel<T, TAPS, kScRun><<<g, kScThreads, 0, stream>>>(p, groups);
+  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
 template <class T>
 int launch_short_conv(const nfk_short_conv_params& p, cudaStream_t stream) {
-  const int groups = p.cols / 4;
-  const long long threads = static_cast<long long>((p.T - p.row_begin + kScRun - 1) / kScRun) * groups;
-  const long long grid = (threads + kScThreads - 1) / kScThreads;
-  if (grid > 0x7fffffffll) return NF_ERR_BAD_ARG;
-  const int g = static_cast<int>(grid);
   switch (p.taps) {
-    case 1: short_conv_kernel<T, 1><<<g, kScThreads, 0, stream>>>(p, groups); break;
-    case 2: short_conv_kernel<T, 2><<<g, kScThreads, 0, stream>>>(p, groups); break;
-    case 3: short_conv_kernel<T, 3><<<g, kScThreads, 0, stream>>>(p, groups); break;
-    case 4: short_conv_kernel<T, 4><<<g, kScThreads, 0, stream>>>(p, groups); break;
-    case 5: short_conv_kernel<T, 5><<<g, kScThreads, 0, stream>>>(p, groups); break;
-    case 6: short_conv_kernel<T, 6><<<g, kScThreads, 0, stream>>>(p, groups); break;
-    case 7: short_conv_kernel<T, 7><<<g, kScThreads, 0, stream>>>(p, groups); break;
-    case 8: short_conv_kernel<T, 8><<<g, kScThreads, 0, stream>>>(p, groups); break;
+    case 1: return launch_taps<T, 1>(p, stream);
+    case 2: return launch_taps<T, 2>(p, stream);
+    case 3: return launch_taps<T, 3>(p, stream);
+    case 4: return launch_taps<T, 4>(p, stream);
+    case 5: return launch_taps<T, 5>(p, stream);
+    case 6: return launch_taps<T, 6>(p, stream);
+    case 7: return launch_taps<T, 7>(p, stream);
+    case 8: return launch_taps<T, 8>(p, stream);
     default: return NF_ERR_UNSUPPORTED;
   }
-  return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 
 }  // namespace

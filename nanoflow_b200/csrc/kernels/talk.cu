@@ -370,22 +370,36 @@ int launch_talk_decode(const nfk_talk_attn_params& p, cudaStream_t stream) {
 // ---- prefill --------------------------------------------------------------------------------------------------
 constexpr int kTpQ = 16, kTpHeads = 16, kTpThreads = kTpHeads * 32;
 constexpr int kTpMaxHeads = 64;
+constexpr int kTpPages = 1024;             // page ids kept in shared memory; later ones are looked up in memory
 
 template <int HD, int KT>
 struct TalkCfg {
   static constexpr int KLD = HD + 8;                     // row strides in elements: conflict-free ldmatrix
   static constexpr int XLD = KT + 8;                     // mixed weights [head][query][key]
-  static constexpr int PLD = kTpQ * KT + 8;              // weights [head][query * KT + key]
+  static constexpr int XHD = kTpQ * XLD + 8;             // ... from head to head
+  static constexpr int PLD = kTpQ * KT + 8;              // weights [head][query * KT + key], see p_col
   static constexpr int ROWS = KT * KLD * 2;              // keys or values of a KV head
-  static constexpr int X_BYTES = kTpHeads * kTpQ * XLD * 2;
+  static constexpr int X_BYTES = kTpHeads * XHD * 2;
   __host__ __device__ static constexpr int p_bytes(int hp) { return hp * PLD * 2; }
-  __host__ __device__ static constexpr int smem(int hp, int kvs) { return 2 * kvs * ROWS + 2 * p_bytes(hp) + 2 * X_BYTES + KT * 8; }
+  // keys | values | weights (pair) | mixed weights (pair, two buffers) | mixing matrix in fragments | page ids
+  __host__ __device__ static constexpr int smem(int hp, int kvs) {
+    return 2 * kvs * ROWS + 2 * p_bytes(hp) + 4 * X_BYTES + hp / 16 * 512 + kTpPages * 4;
+  }
 };
+// Column of a query's block of eight keys: neighbouring queries' blocks lie in different banks.
+template <int KT>
+__device__ __forceinline__ int p_col(int q, int block) {
+  return KT == 32 ? q * 32 + ((block ^ (q >> 1)) & 3) * 8 : q * 16 + ((block ^ (q >> 2)) & 1) * 8;
+}
 
 __device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(x, y);
   const float2 h = unpack_bf16x2(hi);
   lo = pack_bf16x2(x - h.x, y - h.y);
+}
+__device__ __forceinline__ void stsm_x4(uint32_t addr, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
+  asm volatile("stmatrix.sync.aligned.m8n8.x4.shared.b16 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(r0), "r"(r1), "r"(r2), "r"(r3)
+               : "memory");
 }
 
 // hp: heads padded to a multiple of 16; kvs: KV heads that 16 query heads can touch.
@@ -399,45 +413,56 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(tps + kvs * Cfg::ROWS);
   __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(tps + 2 * kvs * Cfg::ROWS);          // high parts, then low parts
   __nv_bfloat16* x_s = reinterpret_cast<__nv_bfloat16*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp));
-  long long* row_s = reinterpret_cast<long long*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp) + 2 * Cfg::X_BYTES);
+  uint4* t_s = reinterpret_cast<uint4*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp) + 4 * Cfg::X_BYTES);
+  int* page_s = reinterpret_cast<int*>(t_s + hp / 16 * 32);
   cg::cluster_group cluster = cg::this_cluster();
   const int C = hp / kTpHeads, rank = static_cast<int>(cluster.block_rank());
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int H = p.heads, G = p.kv_heads, group = H / G;
-  const int* item = p.items + (blockIdx.x / C) * 3;
-  const int req = item[0], tok0 = item[1], cnt = item[2];
+  // the last items of a portion see most keys: they start first
+  const int* item = p.items + (p.num_items - 1 - static_cast<int>(blockIdx.x) / C) * 3;
+  const int req = item[0], tok0 = item[1], cnt = min(item[2], kTpQ);
   const int pos0 = p.positions[tok0];
   const int head0 = rank * kTpHeads, head = head0 + warp;
   const bool live = head < H;
   const int kv0 = head0 / group, kvn = (min(H, head0 + kTpHeads) - 1) / group - kv0 + 1;
   const int kvl = live ? head / group - kv0 : 0;         // this warp's KV head among the CTA's
-  const int lo = (p.window > 0 ? max(0, pos0 - p.window + 1) : 0) / KT * KT;
-  const int tiles = (pos0 + cnt - 1 - lo) / KT + 1;
+  const int first = p.window > 0 ? max(0, pos0 - p.window + 1) : 0, last = pos0 + cnt - 1;
+  const int lo = first / KT * KT, tiles = (last - lo) / KT + 1;
   const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
-  const long long head_step = static_cast<long long>(p.page_size) * HD, v_step = G * head_step;
+  const long long head_step = kPage * HD, v_step = G * head_step;
 
-  // rows of a tile's keys (KV head kv0) into dst; keys that are not there become zeros
-  auto find_rows = [&](int t) {
-    if (threadIdx.x < KT) {
-      const int j = lo + t * KT + threadIdx.x;
-      long long r = -1;
-      const int first = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-      if (j >= first && j <= pos0 + cnt - 1) {
-        const int page = page_of(j, req, p.page_size, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
-        if (page >= 0) r = (static_cast<long long>(page) * 2 * G * p.page_size + j % p.page_size) * HD + kv0 * head_step;
-      }
-      row_s[threadIdx.x] = r;
+  const int slot0 = first / kPage;
+  for (int i = threadIdx.x; i < kTpPages && slot0 + i <= last / kPage; i += kTpThreads)
+    page_s[i] = page_of((slot0 + i) * kPage, req, kPage, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
+  for (int i = threadIdx.x; i < hp / 16 * 32; i += kTpThreads) {
+    const int g = i / 32 * 16 + (i & 3) * 2, h = head0 + ((i >> 2) & 7);
+    auto talk2 = [&](int hh, int gg) {
+      return pack_bf16x2(hh < H && gg < H ? p.talk[hh * H + gg] : 0.f, hh < H && gg + 1 < H ? p.talk[hh * H + gg + 1] : 0.f);
+    };
+    t_s[i] = make_uint4(talk2(h, g), talk2(h + 8, g), talk2(h, g + 8), talk2(h + 8, g + 8));
+  }
+  __syncthreads();
+
+  // keys or values of a tile (from KV head kv0) into dst; keys that are not there become zeros. A thread brings the same
+  // 16 bytes of a key for one KV head after the other.
+  constexpr int CH = HD / 8, UNIT = KT * CH;
+  const int my_key = threadIdx.x % UNIT / CH, my_col = (threadIdx.x % CH) * 8;
+  auto fetch = [&](__nv_bfloat16* dst, int t, long long off) {
+    const int j = lo + t * KT + my_key;
+    int page = -1;
+    if (j >= first && j <= last) {
+      const int slot = j / kPage - slot0;
+      page = slot < kTpPages ? page_s[slot]
+                             : page_of(j, req, kPage, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
     }
-  };
-  auto fetch = [&](__nv_bfloat16* dst, long long off) {
-    constexpr int CH = HD / 8;
-    for (int i = threadIdx.x; i < kvn * KT * CH; i += kTpThreads) {
-      const int kv = i / (KT * CH), k = i / CH % KT, c = (i % CH) * 8;
-      const bool ok = row_s[k] >= 0;
-      const __nv_bfloat16* src = ok ? pool + row_s[k] + off + kv * head_step + c : pool;
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + (kv * KT + k) * Cfg::KLD + c)), "l"(src),
+    const bool ok = page >= 0;
+    const __nv_bfloat16* src = pool + off + my_col;
+    if (ok) src += (static_cast<long long>(page) * 2 * G * kPage + j % kPage) * HD + kv0 * head_step;
+    const uint32_t d = smem_u32(dst + my_key * Cfg::KLD + my_col);
+    for (int kv = threadIdx.x / UNIT; kv < kvn; kv += kTpThreads / UNIT)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d + kv * Cfg::ROWS), "l"(ok ? src + kv * head_step : pool),
                    "r"(ok ? 16 : 0) : "memory");
-    }
     cp_async_commit();
   };
 
@@ -449,11 +474,11 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   const int mm = lane >> 3, rr = lane & 7;
   const float scale = p.scale * kLog2e;
   const int i0 = pos0 + (lane >> 2), i1 = i0 + 8;        // positions of this lane's two queries
-  const bool q0_ok = live && (lane >> 2) < cnt, q1_ok = live && (lane >> 2) + 8 < cnt;
-  const uint32_t kb = smem_u32(k_s) + kvl * Cfg::ROWS, vb = smem_u32(v_s) + kvl * Cfg::ROWS;
+  const uint32_t vb = smem_u32(v_s) + kvl * Cfg::ROWS;
   auto seen = [&](int i, int j) { return j <= i && j >= 0 && (p.window <= 0 || i - j < p.window); };
-  // scores of this warp's head times log2 e, -inf where the query does not see the key
-  auto scores = [&](float (&s)[NT][4], int t) {
+  // scores of this warp's head, -inf where the query does not see the key
+  auto scores = [&](float (&s)[NT][4], const __nv_bfloat16* keys, int t) {
+    const uint32_t kb = smem_u32(keys) + kvl * Cfg::ROWS;
 #pragma unroll
     for (int b = 0; b < NT; ++b) s[b][0] = s[b][1] = s[b][2] = s[b][3] = 0.f;
 #pragma unroll
@@ -465,39 +490,37 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
         mma_bf16(s[b], qa[ks], b0, b1);
         mma_bf16(s[b + 1], qa[ks], b2, b3);
       }
+    const int j0 = lo + t * KT;
+    if (j0 + KT - 1 > pos0 || (p.window > 0 && pos0 + kTpQ - 1 - j0 >= p.window)) {      // not seen by all 16 queries
 #pragma unroll
-    for (int b = 0; b < NT; ++b)
+      for (int b = 0; b < NT; ++b)
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int j = lo + t * KT + b * 8 + (lane & 3) * 2 + e;
-        s[b][e] = q0_ok && seen(i0, j) ? s[b][e] * scale : -INFINITY;
-        s[b][2 + e] = q1_ok && seen(i1, j) ? s[b][2 + e] * scale : -INFINITY;
-      }
+        for (int e = 0; e < 2; ++e) {
+          const int j = j0 + b * 8 + (lane & 3) * 2 + e;
+          if (!seen(i0, j)) s[b][e] = -INFINITY;
+          if (!seen(i1, j)) s[b][2 + e] = -INFINITY;
+        }
+    }
   };
 
-  // ---- first loop: maxima and sums ----
+  // ---- first loop: maxima and sums, keys in the two buffers by turns ----
   const float sink = p.sinks != nullptr && live ? p.sinks[head] * kLog2e : -INFINITY;
-  float m0 = sink, m1 = sink, l0 = 0.f, l1 = 0.f;        // sums of this lane's keys
-  find_rows(0);
-  __syncthreads();
-  fetch(k_s, 0);
+  float m0 = sink, m1 = sink, l0 = 0.f, l1 = 0.f;        // of scores times log2 e; sums of this lane's keys
+  fetch(k_s, 0, 0);
   for (int t = 0; t < tiles; ++t) {
     cp_async_wait<0>();
     __syncthreads();
+    if (t + 1 < tiles) fetch((t & 1) != 0 ? k_s : v_s, t + 1, 0);
     float s[NT][4];
-    scores(s, t);
-    if (t + 1 < tiles) find_rows(t + 1);
-    else find_rows(0);                                   // for the second loop
-    __syncthreads();
-    fetch(k_s, 0);
-    float x0 = m0, x1 = m1;
+    scores(s, (t & 1) != 0 ? v_s : k_s, t);
+    float x0 = s[0][0], x1 = s[0][2];
 #pragma unroll
     for (int b = 0; b < NT; ++b) {
       x0 = fmaxf(x0, fmaxf(s[b][0], s[b][1]));
       x1 = fmaxf(x1, fmaxf(s[b][2], s[b][3]));
     }
-    x0 = quad_max(x0);
-    x1 = quad_max(x1);
+    x0 = fmaxf(m0, quad_max(x0) * scale);
+    x1 = fmaxf(m1, quad_max(x1) * scale);
     const float z0 = x0 == -INFINITY ? 0.f : x0, z1 = x1 == -INFINITY ? 0.f : x1;
     l0 *= fast_exp2(m0 - z0);
     l1 *= fast_exp2(m1 - z1);
@@ -505,17 +528,21 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
     m1 = x1;
 #pragma unroll
     for (int b = 0; b < NT; ++b) {
-      l0 += fast_exp2(s[b][0] - z0) + fast_exp2(s[b][1] - z0);
-      l1 += fast_exp2(s[b][2] - z1) + fast_exp2(s[b][3] - z1);
+      l0 += fast_exp2(fmaf(s[b][0], scale, -z0)) + fast_exp2(fmaf(s[b][1], scale, -z0));
+      l1 += fast_exp2(fmaf(s[b][2], scale, -z1)) + fast_exp2(fmaf(s[b][3], scale, -z1));
     }
   }
+  __syncthreads();
+  fetch(k_s, 0, 0);
+  // weight = 2^(score - m - log2(sum)); rows of the tile that are no queries get none
   l0 = quad_sum(l0);
   l1 = quad_sum(l1);
-  if (m0 == -INFINITY) m0 = 0.f;
-  if (m1 == -INFINITY) m1 = 0.f;
+  m0 = m0 == -INFINITY ? 0.f : m0;
+  m1 = m1 == -INFINITY ? 0.f : m1;
   l0 += sink == -INFINITY ? 0.f : fast_exp2(sink - m0);
   l1 += sink == -INFINITY ? 0.f : fast_exp2(sink - m1);
-  const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+  m0 = live && (lane >> 2) < cnt && l0 > 0.f ? m0 + log2f(l0) : INFINITY;
+  m1 = live && (lane >> 2) + 8 < cnt && l1 > 0.f ? m1 + log2f(l1) : INFINITY;
 
   // ---- second loop: weights, mixing, values ----
   float acc[HD / 8][4];
@@ -523,82 +550,15 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   for (int b = 0; b < HD / 8; ++b) acc[b][0] = acc[b][1] = acc[b][2] = acc[b][3] = 0.f;
   const uint32_t pb = smem_u32(p_s), xb = smem_u32(x_s);
   const uint32_t p_lo = static_cast<uint32_t>(Cfg::p_bytes(hp)), x_lo = Cfg::X_BYTES;
-  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-  for (int t = 0; t < tiles; ++t) {
-    cp_async_wait<0>();
-    __syncthreads();                                     // keys are there; everyone is done with the last values
-    fetch(v_s, v_step);
-    {
-      float s[NT][4];
-      scores(s, t);
-      asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");      // all have started, and mixed the last weights
-#pragma unroll
-      for (int b = 0; b < NT; ++b) {
-        uint32_t h0, l0_, h1, l1_;
-        split_bf16x2(fast_exp2(s[b][0] - m0) * inv0, fast_exp2(s[b][1] - m0) * inv0, h0, l0_);
-        split_bf16x2(fast_exp2(s[b][2] - m1) * inv1, fast_exp2(s[b][3] - m1) * inv1, h1, l1_);
-        const int o = head * Cfg::PLD + (lane >> 2) * KT + b * 8 + (lane & 3) * 2;
-        for (int r = 0; r < C; ++r) {
-          __nv_bfloat16* dst = cluster.map_shared_rank(p_s, r) + o;
-          *reinterpret_cast<uint32_t*>(dst) = h0;
-          *reinterpret_cast<uint32_t*>(dst + 8 * KT) = h1;
-          *reinterpret_cast<uint32_t*>(dst + hp * Cfg::PLD) = l0_;
-          *reinterpret_cast<uint32_t*>(dst + hp * Cfg::PLD + 8 * KT) = l1_;
-        }
-      }
-    }
-    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-    // rows for the next keys; the copies of this tile's values have been started
-    if (t + 1 < tiles) find_rows(t + 1);
-    __syncthreads();
-    if (t + 1 < tiles) fetch(k_s, 0);
-    else cp_async_commit();
-    // mixed weights of the CTA's 16 heads: [16 x H] times [H x (query, key)], columns over the warps
-#pragma unroll
-    for (int c = 0; c < kTpQ * KT / 8 / kTpHeads; c += 2) {
-      const int col = (warp * (kTpQ * KT / 8 / kTpHeads) + c) * 8;
-      float x[2][4];
-#pragma unroll
-      for (int e = 0; e < 2; ++e) x[e][0] = x[e][1] = x[e][2] = x[e][3] = 0.f;
-      for (int g = 0; g < hp; g += 16) {
-        const int hr0 = head0 + (lane >> 2), hr1 = hr0 + 8, gc = g + (lane & 3) * 2;
-        auto talk2 = [&](int h, int gg) {
-          const float a = h < H && gg < H ? __ldg(p.talk + h * H + gg) : 0.f, b = h < H && gg + 1 < H ? __ldg(p.talk + h * H + gg + 1) : 0.f;
-          return pack_bf16x2(a, b);
-        };
-        const uint32_t a[4] = {talk2(hr0, gc), talk2(hr1, gc), talk2(hr0, gc + 8), talk2(hr1, gc + 8)};
-        const uint32_t o = ((g + (mm & 1) * 8 + rr) * Cfg::PLD + col + (mm >> 1) * 8) * 2;
-        uint32_t b0, b1, b2, b3;
-        ldsm_x4_trans(pb + o, b0, b1, b2, b3);
-        mma_bf16(x[0], a, b0, b1);
-        mma_bf16(x[1], a, b2, b3);
-        ldsm_x4_trans(pb + p_lo + o, b0, b1, b2, b3);
-        mma_bf16(x[0], a, b0, b1);
-        mma_bf16(x[1], a, b2, b3);
-      }
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int cc = col + e * 8 + (lane & 3) * 2, qq = cc / KT, kk = cc % KT;
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          uint32_t hi, lo_;
-          split_bf16x2(x[e][2 * h], x[e][2 * h + 1], hi, lo_);
-          __nv_bfloat16* dst = x_s + (((lane >> 2) + h * 8) * kTpQ + qq) * Cfg::XLD + kk;
-          *reinterpret_cast<uint32_t*>(dst) = hi;
-          *reinterpret_cast<uint32_t*>(dst + Cfg::X_BYTES / 2) = lo_;
-        }
-      }
-    }
-    if (t + 1 < tiles) asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-    cp_async_wait<1>();                                  // values
-    __syncthreads();
+  // mixed weights of tile t times its values
+  auto values = [&](int t) {
+    const uint32_t base = xb + ((t & 1) != 0 ? 2 * x_lo : 0);
 #pragma unroll
     for (int ks = 0; ks < KT / 16; ++ks) {
       uint32_t ah[4], al[4];
-      const uint32_t o = ((warp * kTpQ + (lane & 15)) * Cfg::XLD + ks * 16 + (lane >> 4) * 8) * 2;
-      ldsm_x4(xb + o, ah[0], ah[1], ah[2], ah[3]);
-      ldsm_x4(xb + x_lo + o, al[0], al[1], al[2], al[3]);
+      const uint32_t o = (warp * Cfg::XHD + (lane & 15) * Cfg::XLD + ks * 16 + (lane >> 4) * 8) * 2;
+      ldsm_x4(base + o, ah[0], ah[1], ah[2], ah[3]);
+      ldsm_x4(base + x_lo + o, al[0], al[1], al[2], al[3]);
 #pragma unroll
       for (int b = 0; b < HD / 8; b += 2) {
         uint32_t b0, b1, b2, b3;
@@ -609,7 +569,89 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
         mma_bf16(acc[b + 1], al, b2, b3);
       }
     }
+  };
+  // Products with values lag by one tile: they run while the weights travel to the other CTAs.
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  cp_async_wait<0>();
+  __syncthreads();
+  for (int t = 0; t < tiles; ++t) {
+    {
+      float s[NT][4];
+      scores(s, k_s, t);
+      uint32_t hi[NT][2], lw[NT][2];
+#pragma unroll
+      for (int b = 0; b < NT; ++b) {
+        split_bf16x2(fast_exp2(fmaf(s[b][0], scale, -m0)), fast_exp2(fmaf(s[b][1], scale, -m0)), hi[b][0], lw[b][0]);
+        split_bf16x2(fast_exp2(fmaf(s[b][2], scale, -m1)), fast_exp2(fmaf(s[b][3], scale, -m1)), hi[b][1], lw[b][1]);
+      }
+      asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");      // all have started, and mixed the last weights
+#pragma unroll
+      for (int b = 0; b < NT; b += 2) {
+        // matrices: queries 0-7 and 8-15 of key blocks b and b + 1
+        const uint32_t o = (head * Cfg::PLD + p_col<KT>((mm & 1) * 8 + rr, b + (mm >> 1))) * 2;
+        stsm_x4(pb + o, hi[b][0], hi[b][1], hi[b + 1][0], hi[b + 1][1]);
+        stsm_x4(pb + p_lo + o, lw[b][0], lw[b][1], lw[b + 1][0], lw[b + 1][1]);
+      }
+      if (C > 1) {                                       // the head's weights to the other CTAs of the cluster
+        __syncwarp();
+        constexpr int N16 = kTpQ * KT / 8;               // 16-byte pieces of a part
+        const uint4* src = reinterpret_cast<const uint4*>(p_s + head * Cfg::PLD);
+        const int part = static_cast<int>(p_lo / 16);
+        for (int r = 1; r < C; ++r) {
+          uint4* dst = cluster.map_shared_rank(const_cast<uint4*>(src), rank + r < C ? rank + r : rank + r - C);
+#pragma unroll
+          for (int i = 0; i < N16 / 32; ++i) {
+            dst[i * 32 + lane] = src[i * 32 + lane];
+            dst[part + i * 32 + lane] = src[part + i * 32 + lane];
+          }
+        }
+      }
+    }
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    cp_async_wait<0>();
+    __syncthreads();                                     // the last tile's values are there
+    if (t > 0) values(t - 1);
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    if (t + 1 < tiles) fetch(k_s, t + 1, 0);             // everyone is done with these keys
+    // mixed weights of the CTA's 16 heads: [16 x H] times [H x (query, key)], columns over the warps: one query per warp
+#pragma unroll
+    for (int b = 0; b < NT; b += 2) {
+      float x[2][4];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) x[e][0] = x[e][1] = x[e][2] = x[e][3] = 0.f;
+      const uint32_t col = p_col<KT>(warp, b + (mm >> 1));
+      for (int g = 0; g < hp; g += 16) {
+        const uint4 tf = t_s[g * 2 + lane];
+        const uint32_t a[4] = {tf.x, tf.y, tf.z, tf.w};
+        const uint32_t o = ((g + (mm & 1) * 8 + rr) * Cfg::PLD + col) * 2;
+        uint32_t b0, b1, b2, b3, c0, c1, c2, c3;
+        ldsm_x4_trans(pb + o, b0, b1, b2, b3);
+        ldsm_x4_trans(pb + p_lo + o, c0, c1, c2, c3);
+        mma_bf16(x[0], a, b0, b1);
+        mma_bf16(x[1], a, b2, b3);
+        mma_bf16(x[0], a, c0, c1);
+        mma_bf16(x[1], a, c2, c3);
+      }
+      uint32_t hi[4], lw[4];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        split_bf16x2(x[e][0], x[e][1], hi[e * 2], lw[e * 2]);
+        split_bf16x2(x[e][2], x[e][3], hi[e * 2 + 1], lw[e * 2 + 1]);
+      }
+      // matrices: heads 0-7 and 8-15 of key blocks b and b + 1
+      const uint32_t o = (((mm & 1) * 8 + rr) * Cfg::XHD + warp * Cfg::XLD + (b + (mm >> 1)) * 8) * 2;
+      const uint32_t base = xb + ((t & 1) != 0 ? 2 * x_lo : 0);
+      stsm_x4(base + o, hi[0], hi[1], hi[2], hi[3]);
+      stsm_x4(base + x_lo + o, lw[0], lw[1], lw[2], lw[3]);
+    }
+    if (t + 1 < tiles) asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    cp_async_wait<0>();
+    __syncthreads();                                     // mixed weights and the next keys are there, the last values are read
+    fetch(v_s, t, v_step);
   }
+  cp_async_wait<0>();
+  __syncthreads();
+  values(tiles - 1);
   // ---- outputs turn back by their query's angles ----
   if (live) {
     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out);
@@ -711,7 +753,8 @@ extern "C" int nfk_talk_attn_prefill(const nfk_talk_attn_params* p, cudaStream_t
   const int rc = check_talk(p);
   if (rc != NF_OK || p->num_items == 0) return rc;
   if (p->num_items < 0 || !p->items) return NF_ERR_BAD_ARG;
-  if (p->dtype != NFK_BF16 || (p->hd != 64 && p->hd != 128) || p->heads > kTpMaxHeads) return NF_ERR_UNSUPPORTED;
+  if (p->dtype != NFK_BF16 || (p->hd != 64 && p->hd != 128) || p->heads > kTpMaxHeads || p->page_size != kPage)
+    return NF_ERR_UNSUPPORTED;
   const int hp = (p->heads + kTpHeads - 1) / kTpHeads * kTpHeads, kvs = kv_heads_of_16(p->heads, p->heads / p->kv_heads);
   constexpr int kMost = 227 * 1024;
   if (p->hd == 64) {

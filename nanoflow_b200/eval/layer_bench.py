@@ -140,6 +140,8 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
         keys = sum(min(c + n, (p.window + n - 1) if p.window else c + n) for c, n in spans)
         return pairs * p.heads * (4.0 * p.hd + 2.0 * p.heads), es * (2 * keys * p.kv_heads * p.hd + 2 * T * p.heads * p.hd)
     if isinstance(p, G.ShortConvParams):
+        if spans[0][1] == 1 and ("row_begin", "n_dec") in op.dyn:
+            return 0.0, 0.0                             # single tokens go through it in the residual step
         return 0.0, T * 2 * p.cols * es
     if isinstance(p, G.RgLruParams):
         if (spans[0][1] == 1) != ("decode" in op.kernel):

@@ -100,7 +100,9 @@ class ResidualNormParams(Structure):
                 ("in_kind", c_int), ("out_kind", c_int), ("dtype", c_int), ("status", c_void_p), ("src_scale", c_float),
                 ("y2", c_void_p), ("ld_y2", c_longlong), ("y2_gate", c_void_p), ("e_out", c_void_p), ("ld_e", c_longlong),
                 ("e_slot", c_void_p), ("e_weight", c_void_p), ("e_top", c_int), ("e_rows", c_int), ("norm_sum", c_int),
-                ("pair_w", c_void_p), ("pair_w2", c_void_p), ("table_add", c_int)]
+                ("pair_w", c_void_p), ("pair_w2", c_void_p), ("table_add", c_int), ("conv_w", c_void_p), ("conv_out", c_void_p),
+                ("conv_state", c_void_p), ("state_slot", c_void_p), ("positions", c_void_p), ("conv_taps", c_int),
+                ("conv_rows", c_int), ("conv_ld", c_int), ("num_slots", c_int)]
 
 
 class LatentAppendParams(Structure):

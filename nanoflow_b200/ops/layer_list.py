@@ -54,12 +54,18 @@ def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
 def residual_norm(x: torch.Tensor, *, y=None, table=None, ids=None, feedback_src=None, prev_tokens=None, norm_in=None,
                   add=None, h=None, norm_out=None, rows_idx=None, src_scale: float = 1.0, y2=None, y2_gate=None, experts=None,
                   cols: int, eps: float, rows: Optional[int] = None, norm_sum: bool = False, pair=None, table_add: bool = False,
-                  status=None) -> None:
+                  conv=None, status=None) -> None:
     """x <- (table ? 0 : x) + norm_in(src_scale * (y or table[ids])) (+ y2_gate y2) (+ weighted rows of ``experts``:
     outputs, slots, weights) (+ add); h <- norm_out(x). Norms: (kind, weight, bias). ``norm_sum``: norm_in of the whole
     sum; ``pair``: two RMS weights, the source is the mean of the normed y and y2; ``table_add``: the embedding row joins
-    the stream instead of being the source."""
+    the stream instead of being the source; ``conv``: (weights [taps, ld], output, state, state references, positions,
+    rows): the input convolution of the first rows."""
     p = ResidualNormParams()
+    if conv is not None:
+        w, out, state, ref, pos, n = conv
+        _f32(w, "conv"); _i32(ref, "state references"); _i32(pos, "positions")
+        p.conv_w, p.conv_out, p.conv_state, p.state_slot, p.positions = _p(w), _p(out), _p(state), _p(ref), _p(pos)
+        p.conv_taps, p.conv_rows, p.conv_ld, p.num_slots = w.shape[0], n, w.shape[1], state.shape[0]
     p.norm_sum, p.table_add = int(norm_sum), int(table_add)
     if pair is not None:
         _f32(pair[0], "pair"); _f32(pair[1], "pair")

@@ -358,8 +358,7 @@ class LayerListEngine(Engine):
         # what joins the stream before each run: a step vector, or the embedding row
         step = lambda r: None if m.runs[r].step is None else "embedding" if m.loop_add == "embedding" else \
             w.loop_steps[m.runs[r].step]
-        self._residual("embedding", None, w.embed_norm, w.layers[m.runs[0].layer].norm_in, step(0), embed=True)
-        self._input_conv(0, 0)
+        self._residual("embedding", None, w.embed_norm, w.layers[m.runs[0].layer].norm_in, step(0), embed=True, feeds=(0, 0))
         for r, run in enumerate(m.runs):
             spec, lw = m.layers[run.layer], w.layers[run.layer]
             last = r + 1 == len(m.runs)
@@ -369,8 +368,7 @@ class LayerListEngine(Engine):
             y, out = self.y, lw.norm_out                   # what joins the stream at the end of the layer
             if spec.mlp is not None:
                 if not m.parallel:
-                    self._residual(f"R{r}.mid", self.y, lw.norm_out, lw.mlp_in, None, layer=r, more=more)
-                    self._input_conv(r, 1)
+                    self._residual(f"R{r}.mid", self.y, lw.norm_out, lw.mlp_in, None, layer=r, more=more, feeds=(r, 1))
                     out = lw.mlp_out
                 more = FEED_FORWARDS[spec.mlp.kind](self, r, run.layer, spec.mlp, lw.mlp)
                 if not m.parallel:
@@ -380,17 +378,16 @@ class LayerListEngine(Engine):
                 self._residual("final", y, out, w.final_norm, None, sampled=True, more=more)
             else:
                 tap_add = add if self.taps is None else None
-                self._residual(f"R{r}.out", y, out, None if (last or self.taps is not None) else nxt, tap_add, layer=r, more=more)
-                if not last and self.taps is None:
-                    self._input_conv(r + 1, 0)
+                go_on = not last and self.taps is None
+                self._residual(f"R{r}.out", y, out, nxt if go_on else None, tap_add, layer=r, more=more,
+                               feeds=(r + 1, 0) if go_on else None)
                 if self.taps is not None:
                     self._op(f"R{r}.tap", MemcpyParams(dst=_ptr(self.taps[r]), src=_ptr(self.x), elem_bytes=4 * m.width_p,
                                                        count=0), dyn=[("count", T)], layer=r)
                     if last:
                         self._residual("final", None, None, w.final_norm, None, sampled=True)
                     else:
-                        self._residual(f"R{r}.next", None, None, nxt, add, layer=r)
-                        self._input_conv(r + 1, 0)
+                        self._residual(f"R{r}.next", None, None, nxt, add, layer=r, feeds=(r + 1, 0))
         S = g.symbol("n_sample")
         self._gemm("lm_head", self.h_s, w.lm_head, None, rows=S, d32=self.logits)
         self._op("argmax", ArgmaxParams(idx_out=_ptr(self.bufs.sampled), val_out=c_void_p(0), logits=_ptr(self.logits),
@@ -407,10 +404,12 @@ class LayerListEngine(Engine):
                                   kernel=kernel, layer=layer, nano=0)
 
     def _residual(self, name, y, norm_in: Optional[NormWeights], norm_out: Optional[NormWeights], add, *, embed=False,
-                  sampled=False, layer=-1, more: Optional[dict] = None) -> None:
+                  sampled=False, layer=-1, more: Optional[dict] = None, feeds: Optional[Tuple[int, int]] = None) -> None:
         """``more``: what a sublayer adds to the sum besides ``y``: ``y2`` with ``y2_gate`` per row, and expert rows
         (``e_out``, ``e_slot``, ``e_weight``, ``e_top``), under the same norm; or ``pair``: the norms of ``y`` and ``y2``
-        whose mean is the output. ``add``: a vector, or "embedding"."""
+        whose mean is the output. ``add``: a vector, or "embedding". ``feeds``: the run and sublayer (mixer 0, feed-forward
+        1) that reads the normed stream, through its input convolution if it has one: single tokens get it here, portions
+        by an op of its own."""
         m, kind = self.model, NORMS[self.model.norm_kind]
         p = ResidualNormParams()
         p.x, p.ld_x = _ptr(self.x), self.x.stride(0)
@@ -442,24 +441,31 @@ class LayerListEngine(Engine):
         if sampled:
             p.rows_idx, p.in_rows = _ptr(self.meta["sample_rows"]), self.T
         p.cols, p.eps, p.dtype, p.status = m.hidden_size, m.norm_eps, self.code, _ptr(self.bufs.status)
-        self._op(name, p, dyn=[("rows", "n_sample" if sampled else "T")], layer=layer)
+        dyn = [("rows", "n_sample" if sampled else "T")]
+        w = None
+        if feeds is not None:
+            lw = self.w.layers[m.runs[feeds[0]].layer]
+            w, state = (lw.conv_mlp if feeds[1] else lw.conv_in), self.conv_state[feeds[0]][feeds[1]]
+        if w is not None:
+            p.conv_w, p.conv_out, p.conv_state = _ptr(w), _ptr(self.h), _ptr(state)
+            p.state_slot, p.positions = _ptr(self.meta["state_ref"]), _ptr(self.meta["positions"])
+            p.conv_taps, p.conv_ld, p.num_slots = w.shape[0], w.shape[1], self.num_slots
+            dyn.append(("conv_rows", "n_dec"))
+        self._op(name, p, dyn=dyn, layer=layer)
+        if w is not None:
+            self._short_conv(f"R{feeds[0]}.input_conv{feeds[1]}", self.h_raw, self.h, w, state, residual=True, portions=True,
+                             layer=feeds[0])
 
-    def _short_conv(self, name, x, out, w, state, *, bias=None, act=None, residual=False, layer=-1) -> None:
+    def _short_conv(self, name, x, out, w, state, *, bias=None, act=None, residual=False, portions=False,
+                    layer=-1) -> None:
+        """``portions``: only the rows behind the single tokens."""
         meta, m = self.meta, self.model
         p = ShortConvParams(x=_ptr(x), ld_x=x.stride(0), out=_ptr(out), ld_out=out.stride(0), w=_ptr(w), bias=_ptr(bias),
                             state=_ptr(state), state_slot=_ptr(meta["state_ref"]), positions=_ptr(meta["positions"]),
                             token_req=_ptr(meta["token_req"]), qo_indptr=_ptr(meta["qo_indptr"]), row_begin=0, T=0,
                             cols=w.shape[1], taps=w.shape[0], act=CONV_ACTS[act], residual=int(residual),
                             num_slots=self.num_slots, dtype=self.code, status=_ptr(self.bufs.status))
-        self._op(name, p, dyn=[("T", "T")], layer=layer)
-
-    def _input_conv(self, r: int, sublayer: int) -> None:
-        """h = h_raw + its convolution, ahead of run ``r``'s mixer (0) or feed-forward (1)."""
-        lw = self.w.layers[self.model.runs[r].layer]
-        w = lw.conv_mlp if sublayer else lw.conv_in
-        if w is not None:
-            self._short_conv(f"R{r}.input_conv{sublayer}", self.h_raw, self.h, w, self.conv_state[r][sublayer], residual=True,
-                             layer=r)
+        self._op(name, p, dyn=[("T", "T")] + ([("row_begin", "n_dec")] if portions else []), layer=layer)
 
     def _gemm(self, name, a, wt, out, *, rows: str, up=None, act: ActSpec = ActSpec("silu"), lin_act=None, bias=None, d32=None,
               f32_col0=0, groups=1, group_k=0, k=0, key="", layer=-1) -> None:
@@ -916,8 +922,8 @@ FEED_FORWARDS = {"dense": LayerListEngine._dense, "moe": LayerListEngine._moe}
 
 def delta_item_floats(s) -> int:
     """Scratch of a chunk and head of the chunked delta-rule kernels (nfk_delta_item_floats)."""
-    d, v = round8(s.dim), round8(s.vdim)
-    return 3 * CHUNK * d + CHUNK * CHUNK + CHUNK * v + d
+    n = 64 if max(round8(s.dim), round8(s.vdim)) <= 64 else 128
+    return (6 * CHUNK * (n + 8) + 2 * CHUNK * (CHUNK + 8)) // 2 + n + n // 64 * CHUNK * 68
 
 
 def rotations(s) -> List[tuple]:

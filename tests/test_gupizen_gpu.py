@@ -131,6 +131,35 @@ def test_short_convolution_over_portions(dtype, taps, cols, form):
     assert torch.equal(state[0], before[0]) and torch.equal(state[4], before[4])    # nobody else's slot
 
 
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("taps,cols", [(1, 5), (2, 56), (4, 104), (4, 4096), (8, 40)])
+def test_input_convolution_of_single_tokens_in_the_residual_step(dtype, taps, cols):
+    """The same state, token by token in the residual step and in portions in the kernel of its own."""
+    ld, n, eps = pad8(cols), 14, 1e-3
+    pad = lambda t: torch.nn.functional.pad(t, (0, ld - cols)).contiguous()
+    x, w, wn = pad(rnd(2 * n, cols, seed=1)), pad(rnd(taps, cols, seed=2)), pad(rnd(1, cols, seed=3))[0]
+    state = pad(rnd(4, 2, max(1, taps - 1), cols, seed=4, dtype=dtype))
+    got, s = torch.zeros(2 * n, ld, device="cuda"), Steps([n, n])
+    hs = torch.zeros(2 * n, ld, device="cuda")
+    for tokens in ({0: 1}, {1: 1, 0: 1}, {0: 1, 1: 1}, {0: 1, 1: 4}, {1: 1, 0: 3}, {0: 1, 1: 1}, {0: 1, 1: 2}, {1: 1, 0: 1}):
+        rows, pos, req, qo, ref = s.next(tokens)
+        dec = sum(k == 1 for k in tokens.values())                   # single tokens come first
+        h, out = (torch.zeros(len(rows), ld, dtype=dtype, device="cuda") for _ in range(2))
+        st = ops.new_status()
+        K.residual_norm(x[rows].contiguous(), h=h, norm_out=("rms", wn, None), cols=cols, eps=eps, conv=(w, out, state, ref, pos, dec),
+                        status=st)
+        if dec < len(rows):
+            out[dec:] = K.short_conv(h, w, state, ref, pos, req, i32(qo), residual=True, row_begin=dec, status=st)[dec:]
+        ops.check_status(st)
+        got[rows] = out.float()
+        hs[rows] = pad(oracle.rms_norm(x[rows].double()[:, :cols], eps, wn.double()[:cols]).to(dtype).float())
+    for b in range(2):
+        z = slice(s.off[b], s.off[b] + s.at[b])
+        h = hs[z, :cols].double().cpu()
+        want = h + oracle.causal_conv(h, w[:, :cols].double().cpu().T)
+        assert off(got[z, :cols], want) < ROUNDED[dtype] * (4 if dtype == torch.float32 else 2)
+
+
 # ---- attention -----------------------------------------------------------------------------------------------------
 class PagedKv:
     """Sequences of keys and values in a paged pool, pages handed out in a shuffled order; pages that have left ``window``
