@@ -10,7 +10,7 @@
 //                    a lower-triangular system with the same matrix for all columns. Three kernels:
 //                    1. per chunk: the decayed scores <k, k> and <q, k>, the inverse M = (1 + diag(beta) <k, k>)^-1 diag(beta)
 //                       (forward substitution in fp32, by blocks of 16), then M V and W = M (e^c k);
-//                    2. along the chunks, 64 columns of S per CTA, S in registers: u = M V - W S0, the outputs
+//                    2. along the chunks, 32 columns of S per CTA, S in registers: u = M V - W S0, the outputs
 //                       (e^c q) S0 + <q, k> u, and S = e^c_end S0 + (e^(c_end - c) k)^T u;
 //                    3. head norm, weight and gate.
 //                    Decayed rows, scores, W, u and S enter the products as bf16 pairs (high and low part, about 16 bits).
@@ -290,15 +290,15 @@ delta_norm_kernel(nfk_delta_params p) {
 }
 
 // ---- prefill, chunks of 64 tokens -------------------------------------------------------------------------------
-constexpr int kChunk = 64, kRun = 16, kRuns = kChunk / kRun, kDcThreads = 1024, kDsThreads = 512;
+constexpr int kChunk = 64, kRun = 16, kRuns = kChunk / kRun, kDcThreads = 1024, kDsThreads = 256;
 constexpr int kDcWarps = kDcThreads / 32;
-constexpr int kSlice = 64;                 // columns of S per CTA of the second kernel
+constexpr int kSlice = 32;                 // columns of S per CTA of the second kernel
 constexpr float kMaxRunLog2 = 110.f;       // largest decay of a run (log2) whose weights are factored inside the run
 constexpr float kMaxDecayLog2 = 150.f;     // a stronger decay is zero in fp32 anyway
 
 // Scratch of a chunk and head, laid out as the second kernel keeps it in shared memory (padded rows), so that a few bulk
 // copies bring it in: W [2 parts][64][P + 8] | decayed keys, decayed queries alike | scores [2][64][72] | the chunk's decay
-// [P] fp32 | M V [P / 64 slices][64][68] fp32. P: the head's size rounded up to 64 or 128, columns past it are zero.
+// [P] fp32 | M V [P / 32 slices][64][36] fp32. P: the head's size rounded up to 64 or 128, columns past it are zero.
 template <int P>
 struct DeltaItem {
   static constexpr int BLD = P + 8, MLD = kChunk + 8, ULD = kSlice + 4;

@@ -483,9 +483,10 @@ typedef struct nfk_talk_attn_params {
 // Tokens [token_begin, token_begin + n_tokens), any sizes (shared memory for a few rows of all heads permitting), bf16 or
 // fp32: one CTA per token.
 int nfk_talk_attn(const nfk_talk_attn_params* p, cudaStream_t stream);
-// bf16, hd 64 or 128, at most 64 heads. Tokens [token_begin, token_begin + n_tokens), a cluster of CTAs each:
+// bf16, hd 64 or 128, at most 64 heads, `talk` enters the products in bf16. Tokens [token_begin, token_begin + n_tokens), a
+// cluster of CTAs each:
 int nfk_talk_attn_decode(const nfk_talk_attn_params* p, cudaStream_t stream);
-// ... and portions on tensor cores; `talk` enters the products in bf16.
+// ... and portions:
 int nfk_talk_attn_prefill(const nfk_talk_attn_params* p, cudaStream_t stream);
 // Which of the two take these sizes: 1 = prefill, 2 = decode (for max_keys keys), added up.
 int nfk_talk_attn_fits(int heads, int kv_heads, int hd, int max_keys);

@@ -6,8 +6,8 @@
 //
 // nfk_talk_attn          any sizes, bf16 or fp32: one CTA per token, all heads, two passes over the keys.
 // nfk_talk_attn_decode   one token per request (bf16): a cluster of CTAs shares the token's keys. Scores stay in shared
-//                        memory, keys and values are read once, straight into registers; maxima, sums and the partial
-//                        outputs are exchanged through distributed shared memory.
+//                        memory, keys and values are read once, straight into registers (a product with the mixing
+//                        matrix on tensor cores lies between); maxima, sums and the partial outputs are exchanged through distributed shared memory.
 // nfk_talk_attn_prefill  portions (bf16): a cluster takes 16 tokens, each of its CTAs 16 heads, one per warp. First loop
 //                        over the keys: maxima and sums; second loop: every CTA's weights go to all CTAs of the cluster,
 //                        each mixes them for its own heads (a product with the mixing matrix on tensor cores) and applies
@@ -134,34 +134,66 @@ talk_attn_kernel(nfk_talk_attn_params p) {
 
 // ---- decode ---------------------------------------------------------------------------------------------------
 constexpr int kTdThreads = 256, kTdWarps = kTdThreads / 32, kTdKeys = 32;      // keys of a warp's work item
-constexpr int kTdMaxCluster = 8;
+constexpr int kTdMaxCluster = 8, kTpMaxHeads = 64;
 
-// Shared memory: rows [keys] | scores [H][keys + 4] (later weights, [keys][H4]) | (max, sum) [H] | partial outputs [H][hd].
+// Shared memory: rows [keys] | scores, then weights [H][s_ld] | mixed weights [keys][w_ld] | mixing matrix in fragments |
+// (max, sum) [H] | partial outputs [H][hd]. Row strides that spread the fragments' accesses over the banks.
 struct TalkDecodeLayout {
-  int keys, s_ld, h4, rows, scores, stat, out, bytes;
+  int keys, s_ld, w_ld, scores, mixed, talk, stat, out, bytes;
 };
 __host__ __device__ inline TalkDecodeLayout talk_decode_layout(int heads, int hd, int keys) {
   TalkDecodeLayout l;
+  const int hp = (heads + 15) / 16;
   l.keys = (keys + kTdKeys - 1) / kTdKeys * kTdKeys;
   l.s_ld = l.keys + 4;
-  l.h4 = (heads + 3) / 4 * 4;
-  l.rows = 0;
-  l.scores = l.rows + l.keys * 4;
-  const int s_bytes = heads * l.s_ld * 4, w_bytes = l.keys * l.h4 * 4;
-  l.stat = l.scores + s_bytes + w_bytes;
+  l.w_ld = hp * 16 + 4;
+  l.scores = l.keys * 4;
+  l.mixed = l.scores + hp * 16 * l.s_ld * 4;
+  l.talk = l.mixed + l.keys * l.w_ld * 4;
+  l.stat = l.talk + hp * hp * 512;
   l.out = l.stat + (heads * 8 + 15) / 16 * 16;
   l.bytes = l.out + heads * hd * 4;
   return l;
 }
 
+__device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(x, y);
+  const float2 h = unpack_bf16x2(hi);
+  lo = pack_bf16x2(x - h.x, y - h.y);
+}
+// Two fp32 products and sums at once.
+__device__ __forceinline__ uint64_t pair_f32(float x, float y) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ void fma2(uint64_t& acc, uint64_t a, uint64_t b) {
+  asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(acc) : "l"(a), "l"(b));
+}
+__device__ __forceinline__ float2 unpair_f32(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+// Fragments of the mixing matrix (16 x 16 tiles, bf16): piece i of [row tile][column tile][lane].
+__device__ __forceinline__ uint4 talk_fragment(const nfk_talk_attn_params& p, int row0, int col0, int lane) {
+  const int h = row0 + (lane >> 2), g = col0 + (lane & 3) * 2;
+  auto two = [&](int hh, int gg) {
+    return pack_bf16x2(hh < p.heads && gg < p.heads ? p.talk[hh * p.heads + gg] : 0.f,
+                       hh < p.heads && gg + 1 < p.heads ? p.talk[hh * p.heads + gg + 1] : 0.f);
+  };
+  return make_uint4(two(h, g), two(h + 8, g), two(h, g + 8), two(h + 8, g + 8));
+}
+
 // GV: a thread's heads per pass over the values (heads of one KV head).
 template <int HD, int GV>
-__global__ void __launch_bounds__(kTdThreads)
+__global__ void __launch_bounds__(kTdThreads, 2)
 talk_decode_kernel(nfk_talk_attn_params p, TalkDecodeLayout lay) {
   extern __shared__ __align__(16) uint8_t tds[];
-  int* row_s = reinterpret_cast<int*>(tds + lay.rows);
+  int* row_s = reinterpret_cast<int*>(tds);
   float* s_s = reinterpret_cast<float*>(tds + lay.scores);
-  float* w_s = s_s + p.heads * lay.s_ld;
+  float* w_s = reinterpret_cast<float*>(tds + lay.mixed);
+  uint4* t_s = reinterpret_cast<uint4*>(tds + lay.talk);
   float2* stat_s = reinterpret_cast<float2*>(tds + lay.stat);
   float* o_s = reinterpret_cast<float*>(tds + lay.out);
   cg::cluster_group cluster = cg::this_cluster();
@@ -181,14 +213,18 @@ talk_decode_kernel(nfk_talk_attn_params p, TalkDecodeLayout lay) {
   }
   const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
   const long long head_step = static_cast<long long>(p.page_size) * HD, v_step = G * head_step;
+  // rows of the keys; past the last one its row again, with no weight
   for (int k = threadIdx.x; k < lay.keys; k += kTdThreads) {
-    int r = -1;
-    if (k < n) {
-      const int page = page_of(k0 + k, req, p.page_size, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
-      if (page >= 0) r = page * 2 * G * p.page_size + (k0 + k) % p.page_size;
+    int r = 0;
+    if (n > 0) {
+      const int j = k0 + min(k, n - 1), page = page_of(j, req, p.page_size, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
+      if (page >= 0) r = page * 2 * G * p.page_size + j % p.page_size;
     }
     row_s[k] = r;
   }
+  const int hp = (H + 15) / 16;
+  for (int i = threadIdx.x; i < hp * hp * 32; i += kTdThreads) t_s[i] = talk_fragment(p, i / (hp * 32) * 16, i / 32 % hp * 16, i & 31);
+  for (int i = threadIdx.x; i < (hp * 16 - H) * lay.s_ld; i += kTdThreads) s_s[H * lay.s_ld + i] = 0.f;      // heads that are not there
   __syncthreads();
   // ---- scores: a warp takes 32 keys of a KV head. Rows of the tiles: the KV head's query heads, 16 at a time ----
   const int blocks = (n + kTdKeys - 1) / kTdKeys;
@@ -201,9 +237,9 @@ talk_decode_kernel(nfk_talk_attn_params p, TalkDecodeLayout lay) {
 #pragma unroll
     for (int t = 0; t < kTdKeys / 8; ++t) {
       const int r = row_s[kb + t * 8 + (lane >> 2)];
-      const __nv_bfloat16* src = pool + static_cast<long long>(r < 0 ? 0 : r) * HD + kvh * head_step + (lane & 3) * 8;
+      const __nv_bfloat16* src = pool + static_cast<long long>(r) * HD + kvh * head_step + (lane & 3) * 8;
 #pragma unroll
-      for (int b = 0; b < HD / 32; ++b) kr[t][b] = r < 0 ? make_uint4(0, 0, 0, 0) : *reinterpret_cast<const uint4*>(src + b * 32);
+      for (int b = 0; b < HD / 32; ++b) kr[t][b] = *reinterpret_cast<const uint4*>(src + b * 32);
     }
     for (int m0 = 0; m0 < group; m0 += 16) {
       float acc[kTdKeys / 8][4];
@@ -227,7 +263,7 @@ talk_decode_kernel(nfk_talk_attn_params p, TalkDecodeLayout lay) {
         const int k = kb + t * 8 + (lane & 3) * 2;
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const bool ok = row_s[k + e] >= 0;
+          const bool ok = k + e < n;
           if (r0 < group) s_s[(kvh * group + r0) * lay.s_ld + k + e] = ok ? acc[t][e] * p.scale : -INFINITY;
           if (r1 < group) s_s[(kvh * group + r1) * lay.s_ld + k + e] = ok ? acc[t][2 + e] * p.scale : -INFINITY;
         }
@@ -259,62 +295,100 @@ talk_decode_kernel(nfk_talk_attn_params p, TalkDecodeLayout lay) {
     for (int k = lane; k < nk; k += 32) s[k] = s[k] == -INFINITY ? 0.f : expf(s[k] - m) * inv;
   }
   __syncthreads();
-  // ---- mixing: a thread takes a key and four heads at a time; the result lies key by key ----
-  for (int k = threadIdx.x; k < nk; k += kTdThreads) {
-    for (int h = 0; h < lay.h4; h += 4) {
-      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-      const float* t = p.talk + h * H;
-      const int left = H - h;
-      for (int g = 0; g < H; ++g) {
-        const float w = s_s[g * lay.s_ld + k];
-        a.x += __ldg(t + g) * w;
-        if (left > 1) a.y += __ldg(t + H + g) * w;
-        if (left > 2) a.z += __ldg(t + 2 * H + g) * w;
-        if (left > 3) a.w += __ldg(t + 3 * H + g) * w;
+  // ---- mixing: [H x H] times [H x keys] on tensor cores, eight keys per warp and step, weights as bf16 pairs; the result
+  // lies key by key ----
+  for (int kb = warp * 8; kb < nk; kb += kTdWarps * 8) {
+    constexpr int kTiles = kTpMaxHeads / 16;
+    uint32_t bh[kTiles][2], bl[kTiles][2];
+#pragma unroll
+    for (int g = 0; g < kTiles; ++g)
+      if (g < hp) {
+        const float* w = s_s + (g * 16 + (lane & 3) * 2) * lay.s_ld + kb + (lane >> 2);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) split_bf16x2(w[e * 8 * lay.s_ld], w[(e * 8 + 1) * lay.s_ld], bh[g][e], bl[g][e]);
       }
-      *reinterpret_cast<float4*>(w_s + k * lay.h4 + h) = a;
+    for (int h = 0; h < hp; ++h) {
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int g = 0; g < kTiles; ++g)
+        if (g < hp) {
+          const uint4 tf = t_s[(h * hp + g) * 32 + lane];
+          const uint32_t a[4] = {tf.x, tf.y, tf.z, tf.w};
+          mma_bf16(x, a, bh[g][0], bh[g][1]);
+          mma_bf16(x, a, bl[g][0], bl[g][1]);
+        }
+      float* dst = w_s + (kb + (lane & 3) * 2) * lay.w_ld + h * 16 + (lane >> 2);
+      dst[0] = x[0];
+      dst[lay.w_ld] = x[1];
+      dst[8] = x[2];
+      dst[lay.w_ld + 8] = x[3];
     }
   }
   for (int c = threadIdx.x; c < H * HD; c += kTdThreads) o_s[c] = 0.f;
   __syncthreads();
   // ---- values: a thread takes four columns of a KV head for up to GV of its query heads; what threads are left over
-  // split the keys ----
+  // split the keys. The next keys' values are on their way while these are worked on ----
   const int quads = G * (HD / 4), parts = max(1, kTdThreads / quads);
   for (int unit = threadIdx.x; unit < quads * parts; unit += kTdThreads) {
     const int part = unit / quads, qd = unit - part * quads, kvh = qd / (HD / 4), col = (qd - kvh * (HD / 4)) * 4;
     const __nv_bfloat16* v = pool + v_step + kvh * head_step + col;
+    constexpr int U = 8;
+    auto fetch = [&](uint2 (&x)[U], int kb) {
+#pragma unroll
+      for (int j = 0; j < U; j += 4) {
+        const int4 r = *reinterpret_cast<const int4*>(row_s + min(kb, nk - U) + j);      // past the end: not used
+        const int rr[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) x[j + i] = *reinterpret_cast<const uint2*>(v + static_cast<long long>(rr[i]) * HD);
+      }
+    };
     for (int m0 = 0; m0 < group; m0 += GV) {
       const int nh = min(GV, group - m0), h0 = kvh * group + m0;
-      float4 acc[GV];
+      uint64_t acc[GV][2];
 #pragma unroll
-      for (int i = 0; i < GV; ++i) acc[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-      constexpr int U = 8;
-      for (int kb = part * U; kb < nk; kb += parts * U) {
-        uint2 x[U];
+      for (int i = 0; i < GV; ++i) acc[i][0] = acc[i][1] = 0;
+      auto add = [&](const uint2 (&x)[U], int kb) {
+        const float* w = w_s + kb * lay.w_ld + h0;
 #pragma unroll
-        for (int j = 0; j < U; ++j) {
-          const int r = row_s[kb + j];
-          x[j] = r < 0 ? make_uint2(0, 0) : *reinterpret_cast<const uint2*>(v + static_cast<long long>(r) * HD);
-        }
-#pragma unroll
-        for (int j = 0; j < U; ++j) {
+        for (int j = 0; j < U; ++j, w += lay.w_ld) {
           const float2 a = unpack_bf16x2(x[j].x), b = unpack_bf16x2(x[j].y);
-          const float* w = w_s + (kb + j) * lay.h4 + h0;
+          const uint64_t ab = pair_f32(a.x, a.y), cd = pair_f32(b.x, b.y);
+          float f[GV];
+          if (GV == 4 && (h0 & 3) == 0 && nh == 4) {
+            const float4 q4 = *reinterpret_cast<const float4*>(w);
+            f[0] = q4.x; f[GV > 1 ? 1 : 0] = q4.y; f[GV > 2 ? 2 : 0] = q4.z; f[GV > 3 ? 3 : 0] = q4.w;
+          } else {
+#pragma unroll
+            for (int i = 0; i < GV; ++i) f[i] = i < nh ? w[i] : 0.f;
+          }
 #pragma unroll
           for (int i = 0; i < GV; ++i) {
-            const float f = i < nh ? w[i] : 0.f;
-            acc[i].x += f * a.x; acc[i].y += f * a.y; acc[i].z += f * b.x; acc[i].w += f * b.y;
+            const uint64_t ff = pair_f32(f[i], f[i]);
+            fma2(acc[i][0], ff, ab);
+            fma2(acc[i][1], ff, cd);
           }
+        }
+      };
+      uint2 x[U], y[U];
+      const int step = parts * U;
+      if (part * U < nk) fetch(x, part * U);
+      for (int kb = part * U; kb < nk; kb += 2 * step) {
+        fetch(y, kb + step);
+        add(x, kb);
+        if (kb + step < nk) {
+          fetch(x, kb + 2 * step);
+          add(y, kb + step);
         }
       }
 #pragma unroll
       for (int i = 0; i < GV; ++i)
         if (i < nh) {
+          const float2 a = unpair_f32(acc[i][0]), b = unpair_f32(acc[i][1]);
           float* o = o_s + (h0 + i) * HD + col;
           if (parts == 1) {
-            store4(o, acc[i]);
+            store4(o, make_float4(a.x, a.y, b.x, b.y));
           } else {
-            atomicAdd(o, acc[i].x); atomicAdd(o + 1, acc[i].y); atomicAdd(o + 2, acc[i].z); atomicAdd(o + 3, acc[i].w);
+            atomicAdd(o, a.x); atomicAdd(o + 1, a.y); atomicAdd(o + 2, b.x); atomicAdd(o + 3, b.y);
           }
         }
     }
@@ -369,7 +443,6 @@ int launch_talk_decode(const nfk_talk_attn_params& p, cudaStream_t stream) {
 
 // ---- prefill --------------------------------------------------------------------------------------------------
 constexpr int kTpQ = 16, kTpHeads = 16, kTpThreads = kTpHeads * 32;
-constexpr int kTpMaxHeads = 64;
 constexpr int kTpPages = 1024;             // page ids kept in shared memory; later ones are looked up in memory
 
 template <int HD, int KT>
@@ -381,9 +454,9 @@ struct TalkCfg {
   static constexpr int ROWS = KT * KLD * 2;              // keys or values of a KV head
   static constexpr int X_BYTES = kTpHeads * XHD * 2;
   __host__ __device__ static constexpr int p_bytes(int hp) { return hp * PLD * 2; }
-  // keys | values | weights (pair) | mixed weights (pair, two buffers) | mixing matrix in fragments | page ids
+  // keys | values | weights (pair) | mixed weights (pair, two buffers) | mixing matrix in fragments | page ids | barriers
   __host__ __device__ static constexpr int smem(int hp, int kvs) {
-    return 2 * kvs * ROWS + 2 * p_bytes(hp) + 4 * X_BYTES + hp / 16 * 512 + kTpPages * 4;
+    return 2 * kvs * ROWS + 2 * p_bytes(hp) + 4 * X_BYTES + hp / 16 * 512 + kTpPages * 4 + 32;
   }
 };
 // Column of a query's block of eight keys: neighbouring queries' blocks lie in different banks.
@@ -392,14 +465,34 @@ __device__ __forceinline__ int p_col(int q, int block) {
   return KT == 32 ? q * 32 + ((block ^ (q >> 1)) & 3) * 8 : q * 16 + ((block ^ (q >> 2)) & 1) * 8;
 }
 
-__device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(x, y);
-  const float2 h = unpack_bf16x2(hi);
-  lo = pack_bf16x2(x - h.x, y - h.y);
-}
 __device__ __forceinline__ void stsm_x4(uint32_t addr, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
   asm volatile("stmatrix.sync.aligned.m8n8.x4.shared.b16 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(r0), "r"(r1), "r"(r2), "r"(r3)
                : "memory");
+}
+
+// Barriers of a cluster: a warp's arrival at CTA `rank`'s copy, ordered behind the warp's writes to that CTA, and the wait
+// for all of them (bounded: false when the bound ran out).
+__device__ __forceinline__ void cluster_arrive(uint64_t* bar, int rank) {
+  asm volatile(
+      "{\n\t.reg .b32 a;\n\t"
+      "mapa.shared::cluster.u32 a, %0, %1;\n\t"
+      "mbarrier.arrive.release.cluster.shared::cluster.b64 _, [a];\n\t}" ::"r"(smem_u32(bar)), "r"(rank)
+      : "memory");
+}
+__device__ __forceinline__ bool cluster_wait(uint64_t* bar, uint32_t parity) {
+  const uint32_t addr = smem_u32(bar);
+  for (uint32_t it = 0; it < kMbarSpinLimit; ++it) {
+    uint32_t ok;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "mbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(ok)
+        : "r"(addr), "r"(parity)
+        : "memory");
+    if (ok) return true;
+  }
+  return false;
 }
 
 // hp: heads padded to a multiple of 16; kvs: KV heads that 16 query heads can touch.
@@ -415,6 +508,9 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   __nv_bfloat16* x_s = reinterpret_cast<__nv_bfloat16*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp));
   uint4* t_s = reinterpret_cast<uint4*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp) + 4 * Cfg::X_BYTES);
   int* page_s = reinterpret_cast<int*>(t_s + hp / 16 * 32);
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(page_s + kTpPages);       // all weights of a tile are here
+  uint64_t* empty_bar = full_bar + 1;                                        // everyone has mixed a tile's weights
+  uint64_t* v_bar = full_bar + 2;                                            // values have arrived
   cg::cluster_group cluster = cg::this_cluster();
   const int C = hp / kTpHeads, rank = static_cast<int>(cluster.block_rank());
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -432,17 +528,17 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
   const long long head_step = kPage * HD, v_step = G * head_step;
 
+  if (threadIdx.x == 0) {
+    mbar_init(full_bar, C * kTpHeads);
+    mbar_init(empty_bar, C * kTpHeads);
+    mbar_init(v_bar, kTpThreads);
+    mbar_fence_init();
+  }
   const int slot0 = first / kPage;
   for (int i = threadIdx.x; i < kTpPages && slot0 + i <= last / kPage; i += kTpThreads)
     page_s[i] = page_of((slot0 + i) * kPage, req, kPage, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
-  for (int i = threadIdx.x; i < hp / 16 * 32; i += kTpThreads) {
-    const int g = i / 32 * 16 + (i & 3) * 2, h = head0 + ((i >> 2) & 7);
-    auto talk2 = [&](int hh, int gg) {
-      return pack_bf16x2(hh < H && gg < H ? p.talk[hh * H + gg] : 0.f, hh < H && gg + 1 < H ? p.talk[hh * H + gg + 1] : 0.f);
-    };
-    t_s[i] = make_uint4(talk2(h, g), talk2(h + 8, g), talk2(h, g + 8), talk2(h + 8, g + 8));
-  }
-  __syncthreads();
+  for (int i = threadIdx.x; i < hp / 16 * 32; i += kTpThreads) t_s[i] = talk_fragment(p, head0, i / 32 * 16, i & 31);
+  cluster.sync();                                        // barriers are set up everywhere
 
   // keys or values of a tile (from KV head kv0) into dst; keys that are not there become zeros. A thread brings the same
   // 16 bytes of a key for one KV head after the other.
@@ -463,7 +559,6 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
     for (int kv = threadIdx.x / UNIT; kv < kvn; kv += kTpThreads / UNIT)
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d + kv * Cfg::ROWS), "l"(ok ? src + kv * head_step : pool),
                    "r"(ok ? 16 : 0) : "memory");
-    cp_async_commit();
   };
 
   uint32_t qa[HD / 16][4];
@@ -507,10 +602,12 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   const float sink = p.sinks != nullptr && live ? p.sinks[head] * kLog2e : -INFINITY;
   float m0 = sink, m1 = sink, l0 = 0.f, l1 = 0.f;        // of scores times log2 e; sums of this lane's keys
   fetch(k_s, 0, 0);
+  cp_async_commit();
   for (int t = 0; t < tiles; ++t) {
     cp_async_wait<0>();
     __syncthreads();
     if (t + 1 < tiles) fetch((t & 1) != 0 ? k_s : v_s, t + 1, 0);
+    cp_async_commit();
     float s[NT][4];
     scores(s, (t & 1) != 0 ? v_s : k_s, t);
     float x0 = s[0][0], x1 = s[0][2];
@@ -534,6 +631,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   }
   __syncthreads();
   fetch(k_s, 0, 0);
+  cp_async_commit();
   // weight = 2^(score - m - log2(sum)); rows of the tile that are no queries get none
   l0 = quad_sum(l0);
   l1 = quad_sum(l1);
@@ -570,8 +668,11 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
       }
     }
   };
-  // Products with values lag by one tile: they run while the weights travel to the other CTAs.
-  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  // Products with values lag by one tile: they run while the weights travel to the other CTAs. A wait that runs out is
+  // reported; the warps go on in step, so that they meet at their barriers.
+  auto check = [&](bool ok) {
+    if (!ok) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
+  };
   cp_async_wait<0>();
   __syncthreads();
   for (int t = 0; t < tiles; ++t) {
@@ -584,7 +685,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
         split_bf16x2(fast_exp2(fmaf(s[b][0], scale, -m0)), fast_exp2(fmaf(s[b][1], scale, -m0)), hi[b][0], lw[b][0]);
         split_bf16x2(fast_exp2(fmaf(s[b][2], scale, -m1)), fast_exp2(fmaf(s[b][3], scale, -m1)), hi[b][1], lw[b][1]);
       }
-      asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");      // all have started, and mixed the last weights
+      if (t > 0) check(cluster_wait(empty_bar, (t - 1) & 1));
 #pragma unroll
       for (int b = 0; b < NT; b += 2) {
         // matrices: queries 0-7 and 8-15 of key blocks b and b + 1
@@ -607,50 +708,59 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
         }
       }
     }
-    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-    cp_async_wait<0>();
-    __syncthreads();                                     // the last tile's values are there
-    if (t > 0) values(t - 1);
-    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    __syncwarp();
+    if (lane < C) cluster_arrive(full_bar, lane);
+    if (t > 0) {
+      check(mbar_wait(v_bar, (t - 1) & 1));
+      values(t - 1);
+    }
+    check(cluster_wait(full_bar, t & 1));
     if (t + 1 < tiles) fetch(k_s, t + 1, 0);             // everyone is done with these keys
+    cp_async_commit();
     // mixed weights of the CTA's 16 heads: [16 x H] times [H x (query, key)], columns over the warps: one query per warp
+    {
+      float x[NT][4];
 #pragma unroll
-    for (int b = 0; b < NT; b += 2) {
-      float x[2][4];
-#pragma unroll
-      for (int e = 0; e < 2; ++e) x[e][0] = x[e][1] = x[e][2] = x[e][3] = 0.f;
-      const uint32_t col = p_col<KT>(warp, b + (mm >> 1));
+      for (int b = 0; b < NT; ++b) x[b][0] = x[b][1] = x[b][2] = x[b][3] = 0.f;
       for (int g = 0; g < hp; g += 16) {
         const uint4 tf = t_s[g * 2 + lane];
         const uint32_t a[4] = {tf.x, tf.y, tf.z, tf.w};
-        const uint32_t o = ((g + (mm & 1) * 8 + rr) * Cfg::PLD + col) * 2;
-        uint32_t b0, b1, b2, b3, c0, c1, c2, c3;
-        ldsm_x4_trans(pb + o, b0, b1, b2, b3);
-        ldsm_x4_trans(pb + p_lo + o, c0, c1, c2, c3);
-        mma_bf16(x[0], a, b0, b1);
-        mma_bf16(x[1], a, b2, b3);
-        mma_bf16(x[0], a, c0, c1);
-        mma_bf16(x[1], a, c2, c3);
-      }
-      uint32_t hi[4], lw[4];
+        const uint32_t row = (g + (mm & 1) * 8 + rr) * Cfg::PLD;
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        split_bf16x2(x[e][0], x[e][1], hi[e * 2], lw[e * 2]);
-        split_bf16x2(x[e][2], x[e][3], hi[e * 2 + 1], lw[e * 2 + 1]);
+        for (int b = 0; b < NT; b += 2) {
+          const uint32_t o = (row + p_col<KT>(warp, b + (mm >> 1))) * 2;
+          uint32_t b0, b1, b2, b3, c0, c1, c2, c3;
+          ldsm_x4_trans(pb + o, b0, b1, b2, b3);
+          ldsm_x4_trans(pb + p_lo + o, c0, c1, c2, c3);
+          mma_bf16(x[b], a, b0, b1);
+          mma_bf16(x[b + 1], a, b2, b3);
+          mma_bf16(x[b], a, c0, c1);
+          mma_bf16(x[b + 1], a, c2, c3);
+        }
       }
-      // matrices: heads 0-7 and 8-15 of key blocks b and b + 1
-      const uint32_t o = (((mm & 1) * 8 + rr) * Cfg::XHD + warp * Cfg::XLD + (b + (mm >> 1)) * 8) * 2;
+      __syncwarp();
+      if (t + 1 < tiles && lane < C) cluster_arrive(empty_bar, lane);
       const uint32_t base = xb + ((t & 1) != 0 ? 2 * x_lo : 0);
-      stsm_x4(base + o, hi[0], hi[1], hi[2], hi[3]);
-      stsm_x4(base + x_lo + o, lw[0], lw[1], lw[2], lw[3]);
+#pragma unroll
+      for (int b = 0; b < NT; b += 2) {
+        uint32_t hi[4], lw[4];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          split_bf16x2(x[b + e][0], x[b + e][1], hi[e * 2], lw[e * 2]);
+          split_bf16x2(x[b + e][2], x[b + e][3], hi[e * 2 + 1], lw[e * 2 + 1]);
+        }
+        // matrices: heads 0-7 and 8-15 of key blocks b and b + 1
+        const uint32_t o = (((mm & 1) * 8 + rr) * Cfg::XHD + warp * Cfg::XLD + (b + (mm >> 1)) * 8) * 2;
+        stsm_x4(base + o, hi[0], hi[1], hi[2], hi[3]);
+        stsm_x4(base + x_lo + o, lw[0], lw[1], lw[2], lw[3]);
+      }
     }
-    if (t + 1 < tiles) asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
     cp_async_wait<0>();
     __syncthreads();                                     // mixed weights and the next keys are there, the last values are read
     fetch(v_s, t, v_step);
+    asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];" ::"r"(smem_u32(v_bar)) : "memory");
   }
-  cp_async_wait<0>();
-  __syncthreads();
+  check(mbar_wait(v_bar, (tiles - 1) & 1));
   values(tiles - 1);
   // ---- outputs turn back by their query's angles ----
   if (live) {
@@ -675,8 +785,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
       }
     }
   }
-  // a CTA may only leave when nobody writes to its shared memory any more: every write comes before the last
-  // cluster barrier, which all have passed
+  cluster.sync();                                        // nobody leaves while others still arrive at its barriers
 }
 
 template <int HD, int KT>
@@ -743,7 +852,7 @@ extern "C" int nfk_talk_attn_decode(const nfk_talk_attn_params* p, cudaStream_t 
   using namespace nf;
   const int rc = check_talk(p);
   if (rc != NF_OK || p->n_tokens == 0) return rc;
-  if (p->dtype != NFK_BF16 || (p->hd != 64 && p->hd != 128)) return NF_ERR_UNSUPPORTED;
+  if (p->dtype != NFK_BF16 || (p->hd != 64 && p->hd != 128) || p->heads > kTpMaxHeads) return NF_ERR_UNSUPPORTED;
   if (p->max_keys <= 0 || static_cast<long long>(p->num_pages) * 2 * p->kv_heads * p->page_size > 0x7fffffffll) return NF_ERR_BAD_ARG;
   return p->hd == 64 ? launch_talk_decode<64>(*p, stream) : launch_talk_decode<128>(*p, stream);
 }

@@ -270,8 +270,8 @@ class LayerListEngine(Engine):
             return False, False
         keys = min(s.window or self.num_pages * PAGE, self.num_pages * PAGE)
         fits = ops.lib().nfk_talk_attn_fits(s.heads, s.kv_heads, self.model.attn_hd(s), keys)
-        exact = torch.equal(talk.to(torch.bfloat16).float(), talk)      # it enters the prefill kernel's products in bf16
-        return bool(fits & 2), bool(fits & 1) and exact
+        exact = torch.equal(talk.to(torch.bfloat16).float(), talk)      # it enters their products in bf16
+        return bool(fits & 2) and exact, bool(fits & 1) and exact
 
     def _alloc_buffers(self) -> None:
         m, T, dev = self.model, self.T, self.device
@@ -923,7 +923,7 @@ FEED_FORWARDS = {"dense": LayerListEngine._dense, "moe": LayerListEngine._moe}
 def delta_item_floats(s) -> int:
     """Scratch of a chunk and head of the chunked delta-rule kernels (nfk_delta_item_floats)."""
     n = 64 if max(round8(s.dim), round8(s.vdim)) <= 64 else 128
-    return (6 * CHUNK * (n + 8) + 2 * CHUNK * (CHUNK + 8)) // 2 + n + n // 64 * CHUNK * 68
+    return (6 * CHUNK * (n + 8) + 2 * CHUNK * (CHUNK + 8)) // 2 + n + n // 32 * CHUNK * 36
 
 
 def rotations(s) -> List[tuple]:
