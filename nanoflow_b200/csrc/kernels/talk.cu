@@ -454,9 +454,9 @@ struct TalkCfg {
   static constexpr int ROWS = KT * KLD * 2;              // keys or values of a KV head
   static constexpr int X_BYTES = kTpHeads * XHD * 2;
   __host__ __device__ static constexpr int p_bytes(int hp) { return hp * PLD * 2; }
-  // keys | values | weights (pair) | mixed weights (pair, two buffers) | mixing matrix in fragments | page ids | barriers
+  // keys | values | weights (pair) | mixed weights (pair, two buffers) | mixing matrix in fragments | page ids
   __host__ __device__ static constexpr int smem(int hp, int kvs) {
-    return 2 * kvs * ROWS + 2 * p_bytes(hp) + 4 * X_BYTES + hp / 16 * 512 + kTpPages * 4 + 32;
+    return 2 * kvs * ROWS + 2 * p_bytes(hp) + 4 * X_BYTES + hp / 16 * 512 + kTpPages * 4;
   }
 };
 // Column of a query's block of eight keys: neighbouring queries' blocks lie in different banks.
@@ -470,30 +470,9 @@ __device__ __forceinline__ void stsm_x4(uint32_t addr, uint32_t r0, uint32_t r1,
                : "memory");
 }
 
-// Barriers of a cluster: a warp's arrival at CTA `rank`'s copy, ordered behind the warp's writes to that CTA, and the wait
-// for all of them (bounded: false when the bound ran out).
-__device__ __forceinline__ void cluster_arrive(uint64_t* bar, int rank) {
-  asm volatile(
-      "{\n\t.reg .b32 a;\n\t"
-      "mapa.shared::cluster.u32 a, %0, %1;\n\t"
-      "mbarrier.arrive.release.cluster.shared::cluster.b64 _, [a];\n\t}" ::"r"(smem_u32(bar)), "r"(rank)
-      : "memory");
-}
-__device__ __forceinline__ bool cluster_wait(uint64_t* bar, uint32_t parity) {
-  const uint32_t addr = smem_u32(bar);
-  for (uint32_t it = 0; it < kMbarSpinLimit; ++it) {
-    uint32_t ok;
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(ok)
-        : "r"(addr), "r"(parity)
-        : "memory");
-    if (ok) return true;
-  }
-  return false;
-}
+// The cluster's barrier in two halves, so that work fits in between.
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
 
 // hp: heads padded to a multiple of 16; kvs: KV heads that 16 query heads can touch.
 template <int HD, int KT>
@@ -508,9 +487,6 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   __nv_bfloat16* x_s = reinterpret_cast<__nv_bfloat16*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp));
   uint4* t_s = reinterpret_cast<uint4*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp) + 4 * Cfg::X_BYTES);
   int* page_s = reinterpret_cast<int*>(t_s + hp / 16 * 32);
-  uint64_t* full_bar = reinterpret_cast<uint64_t*>(page_s + kTpPages);       // all weights of a tile are here
-  uint64_t* empty_bar = full_bar + 1;                                        // everyone has mixed a tile's weights
-  uint64_t* v_bar = full_bar + 2;                                            // values have arrived
   cg::cluster_group cluster = cg::this_cluster();
   const int C = hp / kTpHeads, rank = static_cast<int>(cluster.block_rank());
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -528,17 +504,11 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
   const long long head_step = kPage * HD, v_step = G * head_step;
 
-  if (threadIdx.x == 0) {
-    mbar_init(full_bar, C * kTpHeads);
-    mbar_init(empty_bar, C * kTpHeads);
-    mbar_init(v_bar, kTpThreads);
-    mbar_fence_init();
-  }
   const int slot0 = first / kPage;
   for (int i = threadIdx.x; i < kTpPages && slot0 + i <= last / kPage; i += kTpThreads)
     page_s[i] = page_of((slot0 + i) * kPage, req, kPage, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
   for (int i = threadIdx.x; i < hp / 16 * 32; i += kTpThreads) t_s[i] = talk_fragment(p, head0, i / 32 * 16, i & 31);
-  cluster.sync();                                        // barriers are set up everywhere
+  __syncthreads();
 
   // keys or values of a tile (from KV head kv0) into dst; keys that are not there become zeros. A thread brings the same
   // 16 bytes of a key for one KV head after the other.
@@ -668,11 +638,8 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
       }
     }
   };
-  // Products with values lag by one tile: they run while the weights travel to the other CTAs. A wait that runs out is
-  // reported; the warps go on in step, so that they meet at their barriers.
-  auto check = [&](bool ok) {
-    if (!ok) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
-  };
+  // Products with values lag by one tile: they run while the weights travel to the other CTAs.
+  if (C > 1) cluster_arrive();
   cp_async_wait<0>();
   __syncthreads();
   for (int t = 0; t < tiles; ++t) {
@@ -685,7 +652,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
         split_bf16x2(fast_exp2(fmaf(s[b][0], scale, -m0)), fast_exp2(fmaf(s[b][1], scale, -m0)), hi[b][0], lw[b][0]);
         split_bf16x2(fast_exp2(fmaf(s[b][2], scale, -m1)), fast_exp2(fmaf(s[b][3], scale, -m1)), hi[b][1], lw[b][1]);
       }
-      if (t > 0) check(cluster_wait(empty_bar, (t - 1) & 1));
+      if (C > 1) cluster_wait();                         // all have started, and mixed the last weights
 #pragma unroll
       for (int b = 0; b < NT; b += 2) {
         // matrices: queries 0-7 and 8-15 of key blocks b and b + 1
@@ -708,13 +675,11 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
         }
       }
     }
-    __syncwarp();
-    if (lane < C) cluster_arrive(full_bar, lane);
-    if (t > 0) {
-      check(mbar_wait(v_bar, (t - 1) & 1));
-      values(t - 1);
-    }
-    check(cluster_wait(full_bar, t & 1));
+    if (C > 1) cluster_arrive();
+    cp_async_wait<0>();
+    __syncthreads();                                     // this CTA's weights and the last tile's values are there
+    if (t > 0) values(t - 1);
+    if (C > 1) cluster_wait();
     if (t + 1 < tiles) fetch(k_s, t + 1, 0);             // everyone is done with these keys
     cp_async_commit();
     // mixed weights of the CTA's 16 heads: [16 x H] times [H x (query, key)], columns over the warps: one query per warp
@@ -738,8 +703,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
           mma_bf16(x[b + 1], a, c2, c3);
         }
       }
-      __syncwarp();
-      if (t + 1 < tiles && lane < C) cluster_arrive(empty_bar, lane);
+      if (C > 1 && t + 1 < tiles) cluster_arrive();
       const uint32_t base = xb + ((t & 1) != 0 ? 2 * x_lo : 0);
 #pragma unroll
       for (int b = 0; b < NT; b += 2) {
@@ -758,9 +722,10 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
     cp_async_wait<0>();
     __syncthreads();                                     // mixed weights and the next keys are there, the last values are read
     fetch(v_s, t, v_step);
-    asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];" ::"r"(smem_u32(v_bar)) : "memory");
+    cp_async_commit();
   }
-  check(mbar_wait(v_bar, (tiles - 1) & 1));
+  cp_async_wait<0>();
+  __syncthreads();
   values(tiles - 1);
   // ---- outputs turn back by their query's angles ----
   if (live) {
@@ -785,7 +750,8 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
       }
     }
   }
-  cluster.sync();                                        // nobody leaves while others still arrive at its barriers
+  // a CTA may only leave when nobody writes to its shared memory any more: every write comes before the last cluster
+  // barrier, which all have passed
 }
 
 template <int HD, int KT>
