@@ -91,18 +91,29 @@ __device__ __forceinline__ void input_conv(const float4 (&v)[NV], const nfk_resi
     if (vi >= nvec) continue;
     const float4 x = rounded(v[i], T(0.f)), w = load4(p.conv_w + static_cast<long long>(before) * p.conv_ld + vi * 4);
     float4 y = make_float4(x.x + w.x * x.x, x.y + w.y * x.y, x.z + w.z * x.z, x.w + w.w * x.w);
-    for (int j = 0; j < before; ++j) {
-      const float4 s = older ? load4(st + static_cast<long long>(j) * p.conv_ld + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
-      const float4 f = load4(p.conv_w + static_cast<long long>(j) * p.conv_ld + vi * 4);
-      y.x += f.x * s.x; y.y += f.y * s.y; y.z += f.z * s.z; y.w += f.w * s.w;
-      if (ok && j > 0) store4(keep + static_cast<long long>(j - 1) * p.conv_ld + vi * 4, s);
+    for (int j0 = 0; j0 < before; j0 += 3) {             // three taps are requested at once
+      float4 s[3], f[3];
+#pragma unroll
+      for (int k = 0; k < 3; ++k) {
+        const int j = j0 + k < before ? j0 + k : 0;
+        s[k] = older ? load4(st + static_cast<long long>(j) * p.conv_ld + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+        f[k] = load4(p.conv_w + static_cast<long long>(j) * p.conv_ld + vi * 4);
+      }
+#pragma unroll
+      for (int k = 0; k < 3; ++k) {
+        const int j = j0 + k;
+        if (j >= before) break;
+        y.x += f[k].x * s[k].x; y.y += f[k].y * s[k].y; y.z += f[k].z * s[k].z; y.w += f[k].w * s[k].w;
+        if (ok && j > 0) store4(keep + static_cast<long long>(j - 1) * p.conv_ld + vi * 4, s[k]);
+      }
     }
     if (ok && before > 0) store4(keep + static_cast<long long>(before - 1) * p.conv_ld + vi * 4, x);
     store4(out + vi * 4, y);
   }
 }
 
-template <class T, int NV>
+// CONV: some rows go through the input convolution.
+template <class T, int NV, bool CONV>
 __global__ void __launch_bounds__(kRnThreads)
 residual_norm_kernel(nfk_residual_norm_params p) {
   __shared__ float red[kRnThreads / 32];
@@ -210,7 +221,7 @@ residual_norm_kernel(nfk_residual_norm_params p) {
     }
     if (p.h != nullptr) {
       norm_row<NV>(v, p.out_kind, p.out_w, p.out_b, p.cols, nvec, p.eps, red);
-      if (p.conv_w != nullptr && row < p.conv_rows) {
+      if (CONV && row < p.conv_rows) {
         input_conv<T, NV>(v, p, row, nvec);
         continue;
       }
@@ -224,16 +235,16 @@ residual_norm_kernel(nfk_residual_norm_params p) {
   }
 }
 
-template <class T>
+template <class T, bool CONV>
 int launch_rn(const nfk_residual_norm_params& p, cudaStream_t stream) {
   const int nvec = (p.cols + 3) / 4, per = (nvec + kRnThreads - 1) / kRnThreads;
   const int cap = device_sm_count() * 16;
   const int grid = p.rows < cap ? p.rows : cap;
-  if (per <= 1) residual_norm_kernel<T, 1><<<grid, kRnThreads, 0, stream>>>(p);
-  else if (per <= 2) residual_norm_kernel<T, 2><<<grid, kRnThreads, 0, stream>>>(p);
-  else if (per <= 4) residual_norm_kernel<T, 4><<<grid, kRnThreads, 0, stream>>>(p);
-  else if (per <= 8) residual_norm_kernel<T, 8><<<grid, kRnThreads, 0, stream>>>(p);
-  else if (per <= 16) residual_norm_kernel<T, 16><<<grid, kRnThreads, 0, stream>>>(p);
+  if (per <= 1) residual_norm_kernel<T, 1, CONV><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 2) residual_norm_kernel<T, 2, CONV><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 4) residual_norm_kernel<T, 4, CONV><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 8) residual_norm_kernel<T, 8, CONV><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 16) residual_norm_kernel<T, 16, CONV><<<grid, kRnThreads, 0, stream>>>(p);
   else return NF_ERR_UNSUPPORTED;
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
@@ -261,5 +272,7 @@ extern "C" int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t
     if (kind != NFK_NORM_NONE && kind != NFK_NORM_RMS && kind != NFK_NORM_LAYER) return NF_ERR_BAD_ARG;
   if ((p->table || p->y) && p->in_kind != NFK_NORM_NONE && !p->in_w) return NF_ERR_BAD_ARG;
   if (p->h && p->out_kind != NFK_NORM_NONE && !p->out_w) return NF_ERR_BAD_ARG;
-  return p->dtype == NFK_F32 ? launch_rn<float>(*p, stream) : launch_rn<__nv_bfloat16>(*p, stream);
+  if (p->conv_w && p->conv_rows > 0)
+    return p->dtype == NFK_F32 ? launch_rn<float, true>(*p, stream) : launch_rn<__nv_bfloat16, true>(*p, stream);
+  return p->dtype == NFK_F32 ? launch_rn<float, false>(*p, stream) : launch_rn<__nv_bfloat16, false>(*p, stream);
 }
