@@ -264,11 +264,26 @@ delta_norm_kernel(nfk_delta_params p) {
   const int t0 = CHUNKS ? p.items[blockIdx.y * 4 + 1] : p.qo_indptr[req];
   const int n = CHUNKS ? p.items[blockIdx.y * 4 + 2] : p.qo_indptr[req + 1] - t0;
   const unsigned total = static_cast<unsigned>(n) * p.heads;
+#pragma unroll 2
   for (unsigned i = blockIdx.x * 8u + (threadIdx.x >> 5); i < total; i += gridDim.x * 8u) {
     const unsigned row = i / static_cast<unsigned>(p.heads);
     const long long t = t0 + static_cast<long long>(row);
     const int head = static_cast<int>(i - row * p.heads);
     const float* o = p.o + (t * p.heads + head) * p.vdim;
+    if (CHUNKS) {                                          // one round: at most 128 values
+      const int c = lane * 4;
+      const bool ok = c < p.vdim;
+      const float4 v = ok ? load4(o + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 gg = ok ? load4(reinterpret_cast<const T*>(p.g) + t * p.ld_g + head * p.vdim + c) : v;
+      const float inv = rsqrtf(warp_sum((v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w)) / static_cast<float>(p.vdim_real) + p.eps);
+      if (ok) {
+        const float4 w = load4(p.norm + c);
+        store4(reinterpret_cast<T*>(p.y) + t * p.ld_y + head * p.vdim + c,
+               make_float4(v.x * inv * w.x * sigmoid_fast(gg.x), v.y * inv * w.y * sigmoid_fast(gg.y),
+                           v.z * inv * w.z * sigmoid_fast(gg.z), v.w * inv * w.w * sigmoid_fast(gg.w)));
+      }
+      continue;
+    }
     float ss = 0.f;
     for (int c = lane * 4; c < p.vdim; c += 128) {
       const float4 v = load4(o + c);
@@ -279,12 +294,8 @@ delta_norm_kernel(nfk_delta_params p) {
     T* y = reinterpret_cast<T*>(p.y) + t * p.ld_y + head * p.vdim;
     for (int c = lane * 4; c < p.vdim; c += 128) {
       const float4 v = load4(o + c), w = load4(p.norm + c), gg = load4(g + c);
-      if (CHUNKS)
-        store4(y + c, make_float4(v.x * inv * w.x * sigmoid_fast(gg.x), v.y * inv * w.y * sigmoid_fast(gg.y),
-                                  v.z * inv * w.z * sigmoid_fast(gg.z), v.w * inv * w.w * sigmoid_fast(gg.w)));
-      else
-        store4(y + c, make_float4(v.x * inv * w.x * sigmoid_f(gg.x), v.y * inv * w.y * sigmoid_f(gg.y),
-                                  v.z * inv * w.z * sigmoid_f(gg.z), v.w * inv * w.w * sigmoid_f(gg.w)));
+      store4(y + c, make_float4(v.x * inv * w.x * sigmoid_f(gg.x), v.y * inv * w.y * sigmoid_f(gg.y),
+                                v.z * inv * w.z * sigmoid_f(gg.z), v.w * inv * w.w * sigmoid_f(gg.w)));
     }
   }
 }
@@ -339,11 +350,11 @@ template <int P>
 struct DeltaChunkCfg {
   static constexpr int BLD = P + 8;                      // bf16 row stride: conflict-free ldmatrix
   static constexpr int FLD = P + 4;                      // fp32 row stride
-  static constexpr int MLD = kChunk + 8, XLD = kChunk + 1;
+  static constexpr int MLD = kChunk + 8, XLD = kChunk + 4;
   static constexpr int ROWS = kChunk * BLD * 2;
   static constexpr int CE = kChunk * FLD * 4, TOT = kRuns * P * 4, M = kChunk * MLD * 2, X = kChunk * XLD * 4;
-  // q | k | v | decayed keys (pair) | log decays | their sums | N | X | Y | M (pair) | factors
-  static constexpr int SMEM = 5 * ROWS + CE + TOT + 2 * X + 16 * kChunk * 4 + 2 * M + 3 * kChunk * 4 + 16;
+  // q | k | v | decayed keys (pair) | log decays | sums of runs, of those before, of those after | N | X | Y | M (pair) | factors
+  static constexpr int SMEM = 5 * ROWS + CE + 3 * TOT + 2 * X + 16 * kChunk * 4 + 2 * M + 3 * kChunk * 4 + 16;
 };
 
 template <int P>
@@ -358,7 +369,9 @@ delta_chunk_kernel(nfk_delta_params p) {
   __nv_bfloat16* kl_s = kh_s + kChunk * C::BLD;
   float* ce = reinterpret_cast<float*>(kl_s + kChunk * C::BLD);     // log2 decays through a token, from its run's start
   float* tot = ce + kChunk * C::FLD;                                 // ... of whole runs
-  float* n_s = tot + kRuns * P;                                      // diag(beta) <k, k>, strictly lower
+  float* pre = tot + kRuns * P;                                      // ... of the runs before, and of those after
+  float* post = pre + kRuns * P;
+  float* n_s = post + kRuns * P;                                     // diag(beta) <k, k>, strictly lower
   float* x_s = n_s + kChunk * C::XLD;                                // its (1 + N)^-1
   float* y_s = x_s + kChunk * C::XLD;                                // [16][64]
   __nv_bfloat16* mh_s = reinterpret_cast<__nv_bfloat16*>(y_s + 16 * kChunk);
@@ -399,7 +412,6 @@ delta_chunk_kernel(nfk_delta_params p) {
     }
     store4(ce + r * C::FLD + c, l);
   }
-  for (int i = threadIdx.x; i < kChunk * C::XLD; i += kDcThreads) x_s[i] = n_s[i] = 0.f;
   if (threadIdx.x < kRuns) slow_s[threadIdx.x] = 0;
   cp_async_wait<0>();
   __syncthreads();
@@ -436,37 +448,49 @@ delta_chunk_kernel(nfk_delta_params p) {
   }
   __syncthreads();
 
-  // ---- keys decayed to the end of their run ----
-  for (int i = threadIdx.x; i < kChunk * (P / 2); i += kDcThreads) {
-    const int t = i / (P / 2), d = (i % (P / 2)) * 2;
-    const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + t * C::BLD + d));
-    const float2 e = *reinterpret_cast<const float2*>(tot + (t / kRun) * P + d);
-    const float2 c = *reinterpret_cast<const float2*>(ce + t * C::FLD + d);
+  // ---- keys decayed to the end of their run; sums over runs ----
+  for (int i = threadIdx.x; i < kChunk * (P / 4); i += kDcThreads) {
+    const int t = i / (P / 4), d = (i % (P / 4)) * 4;
+    const float4 k = load4(k_s + t * C::BLD + d), e = load4(tot + (t / kRun) * P + d), c = load4(ce + t * C::FLD + d);
     const float f = kn_s[t];
-    uint32_t hi, lo;
-    split_pair(k.x * f * fast_exp2(e.x - c.x), k.y * f * fast_exp2(e.y - c.y), hi, lo);
-    *reinterpret_cast<uint32_t*>(kh_s + t * C::BLD + d) = hi;
-    *reinterpret_cast<uint32_t*>(kl_s + t * C::BLD + d) = lo;
+    uint2 hi, lo;
+    split_pair(k.x * f * fast_exp2(e.x - c.x), k.y * f * fast_exp2(e.y - c.y), hi.x, lo.x);
+    split_pair(k.z * f * fast_exp2(e.z - c.z), k.w * f * fast_exp2(e.w - c.w), hi.y, lo.y);
+    *reinterpret_cast<uint2*>(kh_s + t * C::BLD + d) = hi;
+    *reinterpret_cast<uint2*>(kl_s + t * C::BLD + d) = lo;
+  }
+  if (threadIdx.x < P) {
+    const int d = threadIdx.x;
+    float x = 0.f, y = 0.f;
+#pragma unroll
+    for (int j = 0; j < kRuns; ++j) {
+      pre[j * P + d] = x;
+      x += tot[j * P + d];
+      post[(kRuns - 1 - j) * P + d] = y;
+      y += tot[(kRuns - 1 - j) * P + d];
+    }
+    out.decay[d] = fast_exp2(x);
   }
   __syncthreads();
 
-  // ---- scores of (row run a, key run b <= a), rows of queries and rows of keys ----
+  // ---- scores of (row run a, key run b <= a), rows of queries and rows of keys with the same weights. Two warps share a
+  // pair of runs, half of the key channels each ----
   const int mm = lane >> 3, rr = lane & 7;
   const uint32_t khb = smem_u32(kh_s), klb = smem_u32(kl_s);
-  for (int task = warp; task < kRuns * (kRuns + 1); task += kDcThreads / 32) {
-    const bool keys = (task & 1) != 0;
-    int b = task >> 1, a = 0;                              // the pair's number -> (a, b)
+  if (warp < kRuns * (kRuns + 1)) {
+    const int half = warp & 1;
+    int b = warp >> 1, a = 0;                              // the pair's number -> (a, b)
     while (b > a) {
       ++a;
       b -= a;
     }
-    const __nv_bfloat16* rows = keys ? k_s : q_s;
-    const float* norm = keys ? kn_s : qn_s;
     const int t0 = a * kRun + (lane >> 2), t1 = t0 + 8;
-    const float f0 = norm[t0], f1 = norm[t1];
-    float sc[2][4];
+    const float q0 = qn_s[t0], q1 = qn_s[t1], f0 = kn_s[t0], f1 = kn_s[t1];
+    float sc[2][2][4];                                     // [queries, keys][block of keys]
 #pragma unroll
-    for (int j = 0; j < 2; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+    for (int r = 0; r < 2; ++r)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) sc[r][j][0] = sc[r][j][1] = sc[r][j][2] = sc[r][j][3] = 0.f;
     if (a == b && slow_s[a] != 0) {
 #pragma unroll
       for (int j = 0; j < 2; ++j)
@@ -474,15 +498,19 @@ delta_chunk_kernel(nfk_delta_params p) {
         for (int e = 0; e < 4; ++e) {
           const int t = e < 2 ? t0 : t1, s = b * kRun + j * 8 + (lane & 3) * 2 + (e & 1);
           if (s > t) continue;
-          float x = 0.f;
-          for (int d = 0; d < P; ++d)
-            x += to_f32(rows[t * C::BLD + d]) * to_f32(k_s[s * C::BLD + d]) * fast_exp2(ce[t * C::FLD + d] - ce[s * C::FLD + d]);
-          sc[j][e] = x * (e < 2 ? f0 : f1) * kn_s[s];
+          float x = 0.f, y = 0.f;
+          for (int d = half * (P / 2); d < (half + 1) * (P / 2); ++d) {
+            const float w = to_f32(k_s[s * C::BLD + d]) * fast_exp2(ce[t * C::FLD + d] - ce[s * C::FLD + d]);
+            x += to_f32(q_s[t * C::BLD + d]) * w;
+            y += to_f32(k_s[t * C::BLD + d]) * w;
+          }
+          sc[0][j][e] = x * (e < 2 ? q0 : q1) * kn_s[s];
+          sc[1][j][e] = y * (e < 2 ? f0 : f1) * kn_s[s];
         }
     } else {
 #pragma unroll 2
-      for (int ks = 0; ks < P / 16; ++ks) {
-        uint32_t rh[4], rl[4];
+      for (int ks = half * (P / 32); ks < (half + 1) * (P / 32); ++ks) {
+        uint32_t rh[2][4], rl[2][4];
 #pragma unroll
         for (int dh = 0; dh < 2; ++dh) {
           const int d = ks * 16 + dh * 8 + (lane & 3) * 2;
@@ -497,34 +525,56 @@ delta_chunk_kernel(nfk_delta_params p) {
             cum.x += x.x;
             cum.y += x.y;
           }
-          const float2 r0 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(rows + t0 * C::BLD + d));
-          const float2 r1 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(rows + t1 * C::BLD + d));
           const float2 c0 = *reinterpret_cast<const float2*>(ce + t0 * C::FLD + d);
           const float2 c1 = *reinterpret_cast<const float2*>(ce + t1 * C::FLD + d);
-          split_pair(r0.x * f0 * fast_exp2(c0.x + cum.x), r0.y * f0 * fast_exp2(c0.y + cum.y), rh[dh * 2], rl[dh * 2]);
-          split_pair(r1.x * f1 * fast_exp2(c1.x + cum.x), r1.y * f1 * fast_exp2(c1.y + cum.y), rh[dh * 2 + 1], rl[dh * 2 + 1]);
+          const float2 w0 = make_float2(fast_exp2(c0.x + cum.x), fast_exp2(c0.y + cum.y));
+          const float2 w1 = make_float2(fast_exp2(c1.x + cum.x), fast_exp2(c1.y + cum.y));
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const __nv_bfloat16* rows = r == 0 ? q_s : k_s;
+            const float g0 = r == 0 ? q0 : f0, g1 = r == 0 ? q1 : f1;
+            const float2 r0 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(rows + t0 * C::BLD + d));
+            const float2 r1 = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(rows + t1 * C::BLD + d));
+            split_pair(r0.x * g0 * w0.x, r0.y * g0 * w0.y, rh[r][dh * 2], rl[r][dh * 2]);
+            split_pair(r1.x * g1 * w1.x, r1.y * g1 * w1.y, rh[r][dh * 2 + 1], rl[r][dh * 2 + 1]);
+          }
         }
         const uint32_t o = ((b * kRun + (mm >> 1) * 8 + rr) * C::BLD + (2 * ks + (mm & 1)) * 8) * 2;
         uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
         ldsm_x4(khb + o, h0, h1, h2, h3);
         ldsm_x4(klb + o, l0, l1, l2, l3);
-        mma_bf16(sc[0], rh, h0, h1);
-        mma_bf16(sc[1], rh, h2, h3);
-        mma_bf16(sc[0], rh, l0, l1);
-        mma_bf16(sc[1], rh, l2, l3);
-        mma_bf16(sc[0], rl, h0, h1);
-        mma_bf16(sc[1], rl, h2, h3);
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          mma_bf16(sc[r][0], rh[r], h0, h1);
+          mma_bf16(sc[r][1], rh[r], h2, h3);
+          mma_bf16(sc[r][0], rh[r], l0, l1);
+          mma_bf16(sc[r][1], rh[r], l2, l3);
+          mma_bf16(sc[r][0], rl[r], h0, h1);
+          mma_bf16(sc[r][1], rl[r], h2, h3);
+        }
       }
     }
+    // each warp of the pair finishes one kind of rows: it gives the other kind's sums away (through the place of Y and M)
+    float4* swap = reinterpret_cast<float4*>(y_s) + (warp >> 1) * 128 + half * 64 + lane;
 #pragma unroll
-    for (int j = 0; j < 2; ++j)
+    for (int j = 0; j < 2; ++j) {
+      const float(&g)[4] = half == 0 ? sc[1][j] : sc[0][j];
+      swap[j * 32] = make_float4(g[0], g[1], g[2], g[3]);
+    }
+    asm volatile("bar.sync %0, 64;" ::"r"((warp >> 1) + 1) : "memory");
+    swap += half == 0 ? 64 : -64;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const float4 other = swap[j * 32];
+      const float z[4] = {other.x, other.y, other.z, other.w};
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         const int t = h == 0 ? t0 : t1, s = b * kRun + j * 8 + (lane & 3) * 2;
-        const float x = sc[j][2 * h], y = sc[j][2 * h + 1];
-        if (keys) {
-          n_s[t * C::XLD + s] = s < t ? beta_s[t] * x : 0.f;
-          n_s[t * C::XLD + s + 1] = s + 1 < t ? beta_s[t] * y : 0.f;
+        const float x = (half == 0 ? sc[0][j][2 * h] : sc[1][j][2 * h]) + z[2 * h];
+        const float y = (half == 0 ? sc[0][j][2 * h + 1] : sc[1][j][2 * h + 1]) + z[2 * h + 1];
+        if (half == 1) {
+          const float bt = beta_s[t];
+          *reinterpret_cast<float2*>(n_s + t * C::XLD + s) = make_float2(s < t ? bt * x : 0.f, s + 1 < t ? bt * y : 0.f);
         } else {
           uint32_t hi, lo;
           split_pair(s <= t ? x : 0.f, s + 1 <= t ? y : 0.f, hi, lo);
@@ -532,6 +582,7 @@ delta_chunk_kernel(nfk_delta_params p) {
           *reinterpret_cast<uint32_t*>(out.a + kChunk * C::MLD + t * C::MLD + s) = lo;
         }
       }
+    }
   }
   __syncthreads();
 
@@ -550,63 +601,58 @@ delta_chunk_kernel(nfk_delta_params p) {
   }
   __syncthreads();
   for (int a = 1; a < kRuns; ++a) {
-    const int w = a * kRun;
-    for (int i = threadIdx.x; i < kRun * w; i += kDcThreads) {
-      const int r = i / w, c = i % w;
-      float s = 0.f;
-      for (int j = c / kRun * kRun; j < w; ++j) s += n_s[(w + r) * C::XLD + j] * x_s[j * C::XLD + c];
-      y_s[r * kChunk + c] = s;
+    const int w = a * kRun, groups = w / 4;                // four columns per thread
+    const int r = threadIdx.x / groups, c = (threadIdx.x % groups) * 4;
+    if (r < kRun) {
+      float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+      for (int j = c / kRun * kRun; j < w; ++j) fma4(y, n_s[(w + r) * C::XLD + j], load4(x_s + j * C::XLD + c));
+      store4(y_s + r * kChunk + c, y);
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < kRun * w; i += kDcThreads) {
-      const int r = i / w, c = i % w;
-      float s = 0.f;
-      for (int j = 0; j <= r; ++j) s -= x_s[(w + r) * C::XLD + w + j] * y_s[j * kChunk + c];
-      x_s[(w + r) * C::XLD + c] = s;
+    if (r < kRun) {
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+      for (int j = 0; j <= r; ++j) fma4(x, -x_s[(w + r) * C::XLD + w + j], load4(y_s + j * kChunk + c));
+      store4(x_s + (w + r) * C::XLD + c, x);
     }
     __syncthreads();
   }
 
   // ---- M, and what the second kernel reads: keys decayed to the chunk's end, queries decayed from its start; keys
   // decayed from its start take the place of those above ----
-  for (int i = threadIdx.x; i < kChunk * kChunk / 2; i += kDcThreads) {
-    const int t = i / (kChunk / 2), s = (i % (kChunk / 2)) * 2;
-    uint32_t hi, lo;
-    split_pair(x_s[t * C::XLD + s] * beta_s[s], x_s[t * C::XLD + s + 1] * beta_s[s + 1], hi, lo);
-    *reinterpret_cast<uint32_t*>(mh_s + t * C::MLD + s) = hi;
-    *reinterpret_cast<uint32_t*>(ml_s + t * C::MLD + s) = lo;
+  for (int i = threadIdx.x; i < kChunk * kChunk / 4; i += kDcThreads) {
+    const int t = i / (kChunk / 4), s = (i % (kChunk / 4)) * 4;
+    const bool low = s <= t;                               // (blocks above the diagonal were never written)
+    const float4 x = load4(x_s + t * C::XLD + s), bt = load4(beta_s + s);
+    uint2 hi, lo;
+    split_pair(low ? x.x * bt.x : 0.f, s + 1 <= t ? x.y * bt.y : 0.f, hi.x, lo.x);
+    split_pair(s + 2 <= t ? x.z * bt.z : 0.f, s + 3 <= t ? x.w * bt.w : 0.f, hi.y, lo.y);
+    *reinterpret_cast<uint2*>(mh_s + t * C::MLD + s) = hi;
+    *reinterpret_cast<uint2*>(ml_s + t * C::MLD + s) = lo;
   }
-  for (int i = threadIdx.x; i < kChunk * (P / 2); i += kDcThreads) {
-    const int t = i / (P / 2), d = (i % (P / 2)) * 2, run = t / kRun;
-    const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_s + t * C::BLD + d));
-    const float2 q = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(q_s + t * C::BLD + d));
-    float2 c = *reinterpret_cast<const float2*>(ce + t * C::FLD + d), after = make_float2(-c.x, -c.y);
-#pragma unroll
-    for (int j = 0; j < kRuns; ++j) {
-      const float2 x = *reinterpret_cast<const float2*>(tot + j * P + d);
-      if (j < run) {
-        c.x += x.x;
-        c.y += x.y;
-      } else {
-        after.x += x.x;
-        after.y += x.y;
-      }
-    }
-    const float kf = kn_s[t], qf = qn_s[t], ex = fast_exp2(c.x), ey = fast_exp2(c.y);
-    uint32_t hi, lo;
-    split_pair(k.x * kf * ex, k.y * kf * ey, hi, lo);
-    *reinterpret_cast<uint32_t*>(kh_s + t * C::BLD + d) = hi;
-    *reinterpret_cast<uint32_t*>(kl_s + t * C::BLD + d) = lo;
+  for (int i = threadIdx.x; i < kChunk * (P / 4); i += kDcThreads) {
+    const int t = i / (P / 4), d = (i % (P / 4)) * 4, run = t / kRun;
+    const float4 k = load4(k_s + t * C::BLD + d), q = load4(q_s + t * C::BLD + d), c = load4(ce + t * C::FLD + d);
+    const float4 from = load4(pre + run * P + d), to = load4(post + run * P + d), own = load4(tot + run * P + d);
+    const float kf = kn_s[t], qf = qn_s[t];
+    const float4 e = make_float4(fast_exp2(from.x + c.x), fast_exp2(from.y + c.y), fast_exp2(from.z + c.z), fast_exp2(from.w + c.w));
+    const float4 kk = make_float4(k.x * kf, k.y * kf, k.z * kf, k.w * kf);
     const int o = t * C::BLD + d, low = kChunk * C::BLD;
-    split_pair(q.x * qf * ex, q.y * qf * ey, hi, lo);
-    *reinterpret_cast<uint32_t*>(out.q + o) = hi;
-    *reinterpret_cast<uint32_t*>(out.q + low + o) = lo;
-    split_pair(k.x * kf * fast_exp2(after.x), k.y * kf * fast_exp2(after.y), hi, lo);
-    *reinterpret_cast<uint32_t*>(out.k + o) = hi;
-    *reinterpret_cast<uint32_t*>(out.k + low + o) = lo;
+    uint2 hi, lo;
+    split_pair(kk.x * e.x, kk.y * e.y, hi.x, lo.x);
+    split_pair(kk.z * e.z, kk.w * e.w, hi.y, lo.y);
+    *reinterpret_cast<uint2*>(kh_s + o) = hi;
+    *reinterpret_cast<uint2*>(kl_s + o) = lo;
+    split_pair(q.x * qf * e.x, q.y * qf * e.y, hi.x, lo.x);
+    split_pair(q.z * qf * e.z, q.w * qf * e.w, hi.y, lo.y);
+    *reinterpret_cast<uint2*>(out.q + o) = hi;
+    *reinterpret_cast<uint2*>(out.q + low + o) = lo;
+    split_pair(kk.x * fast_exp2((own.x - c.x) + to.x), kk.y * fast_exp2((own.y - c.y) + to.y), hi.x, lo.x);
+    split_pair(kk.z * fast_exp2((own.z - c.z) + to.z), kk.w * fast_exp2((own.w - c.w) + to.w), hi.y, lo.y);
+    *reinterpret_cast<uint2*>(out.k + o) = hi;
+    *reinterpret_cast<uint2*>(out.k + low + o) = lo;
   }
-  for (int d = threadIdx.x; d < P; d += kDcThreads)
-    out.decay[d] = fast_exp2((tot[d] + tot[P + d]) + (tot[2 * P + d] + tot[3 * P + d]));
   __syncthreads();
 
   // ---- M V and W = M (decayed keys): a warp takes a run of rows and an eighth of the columns ----
@@ -684,8 +730,17 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
   __nv_bfloat16* u_s = s_s + 2 * P * C::SLD;
   uint64_t* bar = reinterpret_cast<uint64_t*>(reinterpret_cast<uint8_t*>(u_s) + 2 * C::U);       // first part, rest
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int v0 = (blockIdx.x % slices) * kSlice, head = (blockIdx.x / slices) % p.heads, item0 = blockIdx.x / (slices * p.heads);
-  if (p.items[item0 * 4 + 3] != 0) return;                 // not the first chunk of a portion
+  const int v0 = (blockIdx.x % slices) * kSlice, head = (blockIdx.x / slices) % p.heads, portion = blockIdx.x / (slices * p.heads);
+  int item0 = -1;                                          // first chunk of the portion
+  for (int base = 0, before = 0; base < p.num_items; base += 32) {
+    const unsigned firsts = __ballot_sync(0xffffffffu, base + lane < p.num_items && p.items[(base + lane) * 4 + 3] == 0);
+    if (portion < before + __popc(firsts)) {
+      item0 = base + static_cast<int>(__fns(firsts, 0, portion - before + 1));
+      break;
+    }
+    before += __popc(firsts);
+  }
+  if (item0 < 0) return;
   const int req = p.items[item0 * 4];
   const DeltaState st = delta_state(p, req, head);
   if (!st.ok) return;
@@ -910,9 +965,10 @@ int launch_delta_chunks(const nfk_delta_params& p, cudaStream_t stream) {
     attr = true;
   }
   const int grid = p.num_items * p.heads, slices = (p.vdim + kSlice - 1) / kSlice;
+  const int portions = p.num_portions > 0 && p.num_portions < p.num_items ? p.num_portions : p.num_items;
   delta_chunk_kernel<P><<<grid, kDcThreads, DeltaChunkCfg<P>::SMEM, stream>>>(p);
   if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
-  delta_scan_kernel<P><<<grid * slices, kDsThreads, DeltaScanCfg<P>::SMEM, stream>>>(p, slices);
+  delta_scan_kernel<P><<<portions * p.heads * slices, kDsThreads, DeltaScanCfg<P>::SMEM, stream>>>(p, slices);
   if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
   const int per = kChunk * p.heads / 8;
   delta_norm_kernel<__nv_bfloat16, true><<<dim3(per < 64 ? (per > 0 ? per : 1) : 64, p.num_items), 256, 0, stream>>>(p);

@@ -577,7 +577,8 @@ typedef struct nfk_delta_params {
   int dtype;
   // prefill. o: fp32 [T, heads * vdim] of scratch rows. Token by token: seq_reqs [num_seq] requests. In chunks of 64 tokens
   // (bf16, dim and vdim up to 128): items [num_items][4] (request, first token, tokens, chunk of the request's portion), a
-  // request's chunks one after the other, and scratch: num_items * heads * nfk_delta_item_floats(dim, vdim) floats.
+  // request's chunks one after the other, of num_portions requests (0: not said), and scratch: num_items * heads *
+  // nfk_delta_item_floats(dim, vdim) floats.
   const int* seq_reqs;
   int num_seq;
   float* o;
@@ -586,6 +587,7 @@ typedef struct nfk_delta_params {
   float* scratch;
   long long scratch_floats;
   unsigned int* status;
+  int num_portions;          // requests whose chunks are listed; 0: not said
 } nfk_delta_params;
 long long nfk_delta_item_floats(int dim, int vdim);
 int nfk_delta_decode(const nfk_delta_params* p, cudaStream_t stream);

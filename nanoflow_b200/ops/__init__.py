@@ -187,7 +187,7 @@ class DeltaParams(Structure):
                 ("vdim", c_int), ("vdim_real", c_int), ("num_slots", c_int), ("q_scale", c_float), ("unit_eps", c_float),
                 ("eps", c_float), ("dtype", c_int), ("seq_reqs", c_void_p), ("num_seq", c_int), ("o", c_void_p),
                 ("items", c_void_p), ("num_items", c_int), ("scratch", c_void_p), ("scratch_floats", c_longlong),
-                ("status", c_void_p)]
+                ("status", c_void_p), ("num_portions", c_int)]
 
 
 class GqaAttnParams(Structure):

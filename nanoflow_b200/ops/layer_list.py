@@ -334,7 +334,8 @@ def delta(qkv, x, beta, g, rate, dt_bias, norm, state, y, positions, qo_indptr, 
                     kv_heads=kv_heads, dim=dim, vdim=vdim, vdim_real=vdim_real, num_slots=slots, q_scale=q_scale,
                     unit_eps=unit_eps, eps=eps, dtype=dtype_code(qkv.dtype), seq_reqs=_p(seq),
                     num_seq=0 if seq is None else seq.numel(), o=_p(o), items=_p(items), num_items=n, scratch=_p(ws),
-                    scratch_floats=ws.numel(), status=_p(status))
+                    scratch_floats=ws.numel(), status=_p(status),
+                    num_portions=0 if items is None else int((items[:, 3] == 0).sum()))
     name = "nfk_delta_decode" if decode else "nfk_delta_prefill"
     _check(getattr(lib(), name)(byref(p), _stream()), name)
 

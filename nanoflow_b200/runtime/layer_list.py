@@ -736,7 +736,8 @@ class LayerListEngine(Engine):
         p, dyn = params(), [("num_seq", "n_pre")]
         if self._delta_in_chunks(s):
             p.seq_reqs = _ptr(meta["chunk_seq"])
-            dyn = [("num_seq", self.g.symbol("n_chunk_seq")), ("num_items", self.g.symbol("n_chunks"))]
+            dyn = [("num_seq", self.g.symbol("n_chunk_seq")), ("num_items", self.g.symbol("n_chunks")),
+                   ("num_portions", self.g.symbol("n_chunk_reqs"))]
         self._op(f"R{r}.delta_prefill", p, kernel="nfk_delta_prefill", dyn=dyn, layer=r)
         self._gemm(f"R{r}.o", attn, lw.w_o, self.y, rows=T, key=f"l{layer}.o", layer=r)
 
@@ -853,7 +854,7 @@ class LayerListEngine(Engine):
             items, seq = chunk_work(qo, D, self.chunk_cap)
             put("chunk_items", items.reshape(-1))
             put("chunk_seq", seq)
-            sym["n_chunks"], sym["n_chunk_seq"] = items.shape[0], seq.size
+            sym["n_chunks"], sym["n_chunk_seq"], sym["n_chunk_reqs"] = items.shape[0], seq.size, P - seq.size
         if "titem" in self.meta:
             items = query_items(qo, D, TALK_TILE)
             put("titem", items.reshape(-1))
