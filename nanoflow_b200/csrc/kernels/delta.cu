@@ -301,31 +301,31 @@ delta_norm_kernel(nfk_delta_params p) {
 }
 
 // ---- prefill, chunks of 64 tokens -------------------------------------------------------------------------------
-constexpr int kChunk = 64, kRun = 16, kRuns = kChunk / kRun, kDcThreads = 1024, kDsThreads = 256;
+constexpr int kChunk = 64, kRun = 16, kRuns = kChunk / kRun, kDcThreads = 1024, kDsThreads = 512, kDsGroup = kDsThreads / 2;
 constexpr int kDcWarps = kDcThreads / 32;
 constexpr int kSlice = 32;                 // columns of S per CTA of the second kernel
 constexpr float kMaxRunLog2 = 110.f;       // largest decay of a run (log2) whose weights are factored inside the run
 constexpr float kMaxDecayLog2 = 150.f;     // a stronger decay is zero in fp32 anyway
 
 // Scratch of a chunk and head, laid out as the second kernel keeps it in shared memory (padded rows), so that a few bulk
-// copies bring it in: W [2 parts][64][P + 8] | decayed keys, decayed queries alike | scores [2][64][72] | the chunk's decay
-// [P] fp32 | M V [P / 32 slices][64][36] fp32. P: the head's size rounded up to 64 or 128, columns past it are zero.
+// copies bring it in: W [2 parts][64][P + 8] | decayed keys alike | the chunk's decay [P] fp32 | decayed queries as W | scores
+// [2][64][72] | M V [P / 32 slices][64][36] fp32. P: the head's size rounded up to 64 or 128, columns past it are zero.
 template <int P>
 struct DeltaItem {
   static constexpr int BLD = P + 8, MLD = kChunk + 8, ULD = kSlice + 4;
   static constexpr int PAIR = 2 * kChunk * BLD * 2, A = 2 * kChunk * MLD * 2, U = kChunk * ULD * 4;      // bytes
-  static constexpr int REST = 2 * PAIR + A + P * 4;
-  static constexpr int BYTES = PAIR + REST + P / kSlice * U;
+  static constexpr int KEYS = PAIR + P * 4, READ = PAIR + A;             // what S is updated with, what outputs need
+  static constexpr int BYTES = PAIR + KEYS + READ + P / kSlice * U;
   __nv_bfloat16 *w, *k, *q, *a;
   float *decay, *u;
   __device__ __forceinline__ DeltaItem(const nfk_delta_params& p, int item, int head) {
     char* b = reinterpret_cast<char*>(p.scratch) + (static_cast<long long>(item) * p.heads + head) * BYTES;
     w = reinterpret_cast<__nv_bfloat16*>(b);
     k = reinterpret_cast<__nv_bfloat16*>(b + PAIR);
-    q = reinterpret_cast<__nv_bfloat16*>(b + 2 * PAIR);
-    a = reinterpret_cast<__nv_bfloat16*>(b + 3 * PAIR);
-    decay = reinterpret_cast<float*>(b + 3 * PAIR + A);
-    u = reinterpret_cast<float*>(b + PAIR + REST);
+    decay = reinterpret_cast<float*>(b + 2 * PAIR);
+    q = reinterpret_cast<__nv_bfloat16*>(b + PAIR + KEYS);
+    a = reinterpret_cast<__nv_bfloat16*>(b + 2 * PAIR + KEYS);
+    u = reinterpret_cast<float*>(b + PAIR + KEYS + READ);
   }
 };
 __host__ __device__ __forceinline__ long long delta_item_floats(int dim, int vdim) {
@@ -712,23 +712,27 @@ template <int P>
 struct DeltaScanCfg {
   using I = DeltaItem<P>;
   static constexpr int BLD = I::BLD, MLD = I::MLD, SLD = kSlice + 8, ULD = I::ULD;
-  static constexpr int S = P * SLD * 2, U = kChunk * SLD * 2;            // one part
-  // W | M V | the rest of a chunk's scratch | S (pair) | u (pair) | barriers
-  static constexpr int SMEM = I::PAIR + I::U + I::REST + 2 * S + 2 * U + 64;
+  static constexpr int S = 2 * P * SLD * 2, U = 2 * kChunk * SLD * 2;    // pairs
+  // W | M V | keys, decay | queries, scores | S (two buffers) | u (two buffers) | barriers
+  static constexpr int SMEM = I::PAIR + I::U + I::KEYS + I::READ + 2 * S + 2 * U + 64;
 };
+__device__ __forceinline__ void named_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+__device__ __forceinline__ void named_arrive(int id, int threads) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 
+// Two groups of eight warps. The first follows the chain from chunk to chunk (values written, next state); the second forms
+// the outputs of a chunk from the state and the values that the first one left for it, one chunk behind at most.
 template <int P>
 __global__ void __launch_bounds__(kDsThreads, 1)
 delta_scan_kernel(nfk_delta_params p, int slices) {
   using C = DeltaScanCfg<P>;
   using I = DeltaItem<P>;
+  enum { kBarChain = 1, kBarOut = 2, kBarFull = 3, kBarFree = 5 };       // the last two: one per buffer
   extern __shared__ __align__(16) uint8_t smem[];
-  uint8_t *w_b = smem, *mv_b = w_b + I::PAIR, *rest_b = mv_b + I::U;
+  uint8_t *w_b = smem, *mv_b = w_b + I::PAIR, *keys_b = mv_b + I::U, *read_b = keys_b + I::KEYS;
   float* mv_s = reinterpret_cast<float*>(mv_b);
-  float* decay_s = reinterpret_cast<float*>(rest_b + 2 * I::PAIR + I::A);
-  __nv_bfloat16* s_s = reinterpret_cast<__nv_bfloat16*>(rest_b + I::REST);
-  __nv_bfloat16* u_s = s_s + 2 * P * C::SLD;
-  uint64_t* bar = reinterpret_cast<uint64_t*>(reinterpret_cast<uint8_t*>(u_s) + 2 * C::U);       // first part, rest
+  float* decay_s = reinterpret_cast<float*>(keys_b + I::PAIR);
+  uint8_t *s_b = read_b + I::READ, *u_b = s_b + 2 * C::S;
+  uint64_t* bar = reinterpret_cast<uint64_t*>(u_b + 2 * C::U);           // W and M V, keys, queries
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int v0 = (blockIdx.x % slices) * kSlice, head = (blockIdx.x / slices) % p.heads, portion = blockIdx.x / (slices * p.heads);
   int item0 = -1;                                          // first chunk of the portion
@@ -748,64 +752,41 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
   const int chunks = min((n_tok + kChunk - 1) / kChunk, p.num_items - item0);
   const long long tok0 = p.qo_indptr[req];
 
-  auto fetch_first = [&](int c) {                          // what the values written need; one thread
+  auto fetch_w = [&](int c) {                              // one thread
     const I d(p, item0 + c, head);
     mbar_expect_tx(&bar[0], I::PAIR + I::U);
     bulk_load(w_b, d.w, I::PAIR, &bar[0]);
     bulk_load(mv_b, d.u + v0 / kSlice * (I::U / 4), I::U, &bar[0]);
   };
-  auto fetch_rest = [&](int c) {
+  auto fetch_keys = [&](int c) {
     const I d(p, item0 + c, head);
-    mbar_expect_tx(&bar[1], I::REST);
-    bulk_load(rest_b, d.k, I::REST, &bar[1]);
+    mbar_expect_tx(&bar[1], I::KEYS);
+    bulk_load(keys_b, d.k, I::KEYS, &bar[1]);
+  };
+  auto fetch_read = [&](int c) {
+    const I d(p, item0 + c, head);
+    mbar_expect_tx(&bar[2], I::READ);
+    bulk_load(read_b, d.q, I::READ, &bar[2]);
   };
   if (threadIdx.x == 0) {
-    mbar_init(&bar[0], 1);
-    mbar_init(&bar[1], 1);
+    for (int i = 0; i < 3; ++i) mbar_init(&bar[i], 1);
     mbar_fence_init();
-    fetch_first(0);
-    fetch_rest(0);
+    fetch_w(0);
+    fetch_keys(0);
+    fetch_read(0);
   }
-
-  // ---- S: warps over 16-row tiles of the key channels and parts of the columns ----
-  constexpr int MT = P / 16, SN = kSlice / 8 * MT / (kDsThreads / 32);     // row tiles; column blocks per warp
-  const int sm0 = (warp % MT) * 16, sn0 = (warp / MT) * SN;
-  const int d0 = sm0 + (lane >> 2), d1 = d0 + 8;
-  float S[SN][4];
-#pragma unroll
-  for (int i = 0; i < SN; ++i) {
-    const int c = (sn0 + i) * 8 + (lane & 3) * 2;
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int d = h == 0 ? d0 : d1;
-      const bool ok = !st.fresh && d < p.dim && v0 + c < p.vdim;
-      const float2 x = ok ? *reinterpret_cast<const float2*>(st.S + static_cast<long long>(d) * p.vdim + v0 + c) : make_float2(0.f, 0.f);
-      S[i][2 * h] = x.x;
-      S[i][2 * h + 1] = x.y;
-    }
-  }
-  auto publish = [&]() {
-#pragma unroll
-    for (int i = 0; i < SN; ++i)
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int o = (h == 0 ? d0 : d1) * C::SLD + (sn0 + i) * 8 + (lane & 3) * 2;
-        uint32_t hi, lo;
-        split_pair(S[i][2 * h], S[i][2 * h + 1], hi, lo);
-        *reinterpret_cast<uint32_t*>(s_s + o) = hi;
-        *reinterpret_cast<uint32_t*>(s_s + P * C::SLD + o) = lo;
-      }
+  __syncthreads();
+  // a wait that runs out is reported; the warps go on in step, so that they meet at their barriers
+  auto arrived = [&](int i, int c) {
+    if (!mbar_wait(&bar[i], c & 1)) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
   };
-  publish();
-  __syncthreads();                                         // also: the barriers are set up
-
   const int mm = lane >> 3, rr = lane & 7;
-  const int a = warp & 3, c0 = (warp >> 2) * 16;           // this warp's run of rows and its columns
+  const int a = warp & 3, c0 = ((warp >> 2) & 1) * 16;     // a warp's run of rows and its columns
   const int t0 = a * kRun + (lane >> 2);
-  const uint32_t wb = smem_u32(w_b), kb = smem_u32(rest_b), qb = kb + I::PAIR, ab = qb + I::PAIR, sb = smem_u32(s_s), ub = smem_u32(u_s);
-  constexpr uint32_t R_LO = I::PAIR / 2, A_LO = kChunk * C::MLD * 2, S_LO = P * C::SLD * 2, U_LO = kChunk * C::SLD * 2;
+  const uint32_t wb = smem_u32(w_b), kb = smem_u32(keys_b), qb = smem_u32(read_b), ab = qb + I::PAIR;
+  constexpr uint32_t R_LO = I::PAIR / 2, A_LO = I::A / 2, S_LO = C::S / 2, U_LO = C::U / 2;
   // acc += rows (pair, of this warp's run) x S (pair, this warp's columns)
-  auto rows_times_s = [&](float (&acc)[2][4], uint32_t base) {
+  auto rows_times_s = [&](float (&acc)[2][4], uint32_t base, uint32_t sb) {
 #pragma unroll
     for (int ks = 0; ks < P / 16; ++ks) {
       uint32_t rh[4], rl[4], h0, h1, h2, h3, l0, l1, l2, l3;
@@ -824,14 +805,88 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
     }
   };
 
+  if (warp >= kDsGroup / 32) {
+    // ---- outputs ----
+    for (int c = 0; c < chunks; ++c) {
+      named_sync(kBarFull + (c & 1), kDsThreads);
+      arrived(2, c);
+      const uint32_t sb = smem_u32(s_b + (c & 1) * C::S), ub = smem_u32(u_b + (c & 1) * C::U);
+      float acc[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+      rows_times_s(acc, qb, sb);
+#pragma unroll
+      for (int ks = 0; ks < kRuns; ++ks) {
+        if (ks > a) continue;
+        uint32_t ah[4], al[4], h0, h1, h2, h3, l0, l1, l2, l3;
+        const uint32_t ao = ((a * kRun + (lane & 15)) * C::MLD + ks * 16 + (lane >> 4) * 8) * 2;
+        ldsm_x4(ab + ao, ah[0], ah[1], ah[2], ah[3]);
+        ldsm_x4(ab + A_LO + ao, al[0], al[1], al[2], al[3]);
+        const uint32_t uo = ((ks * 16 + (mm & 1) * 8 + rr) * C::SLD + c0 + (mm >> 1) * 8) * 2;
+        ldsm_x4_trans(ub + uo, h0, h1, h2, h3);
+        ldsm_x4_trans(ub + U_LO + uo, l0, l1, l2, l3);
+        mma_bf16(acc[0], ah, h0, h1);
+        mma_bf16(acc[1], ah, h2, h3);
+        mma_bf16(acc[0], ah, l0, l1);
+        mma_bf16(acc[1], ah, l2, l3);
+        mma_bf16(acc[0], al, h0, h1);
+        mma_bf16(acc[1], al, h2, h3);
+      }
+      named_sync(kBarOut, kDsGroup);                       // queries and scores are read
+      if (threadIdx.x == kDsGroup && c + 1 < chunks) fetch_read(c + 1);
+      if (c + 2 < chunks) named_arrive(kBarFree + (c & 1), kDsThreads);      // (waited for when chunk c + 2 gets its state)
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int t = c * kChunk + t0 + h * 8, col = v0 + c0 + i * 8 + (lane & 3) * 2;
+          if (t < n_tok && col < p.vdim)
+            *reinterpret_cast<float2*>(p.o + ((tok0 + t) * p.heads + head) * p.vdim + col) = make_float2(acc[i][2 * h], acc[i][2 * h + 1]);
+        }
+    }
+    return;
+  }
+
+  // ---- S: warps over 16-row tiles of the key channels and parts of the columns ----
+  constexpr int MT = P / 16, SN = kSlice / 8 * MT / (kDsGroup / 32);     // row tiles; column blocks per warp
+  const int sm0 = (warp % MT) * 16, sn0 = (warp / MT) * SN;
+  const int d0 = sm0 + (lane >> 2), d1 = d0 + 8;
+  float S[SN][4];
+#pragma unroll
+  for (int i = 0; i < SN; ++i) {
+    const int c = (sn0 + i) * 8 + (lane & 3) * 2;
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int d = h == 0 ? d0 : d1;
+      const bool ok = !st.fresh && d < p.dim && v0 + c < p.vdim;
+      const float2 x = ok ? *reinterpret_cast<const float2*>(st.S + static_cast<long long>(d) * p.vdim + v0 + c) : make_float2(0.f, 0.f);
+      S[i][2 * h] = x.x;
+      S[i][2 * h + 1] = x.y;
+    }
+  }
+  auto publish = [&](int buf) {
+    __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(s_b + buf * C::S);
+#pragma unroll
+    for (int i = 0; i < SN; ++i)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int o = (h == 0 ? d0 : d1) * C::SLD + (sn0 + i) * 8 + (lane & 3) * 2;
+        uint32_t hi, lo;
+        split_pair(S[i][2 * h], S[i][2 * h + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(dst + o) = hi;
+        *reinterpret_cast<uint32_t*>(dst + P * C::SLD + o) = lo;
+      }
+  };
+  publish(0);
+  named_sync(kBarChain, kDsGroup);
   for (int c = 0; c < chunks; ++c) {
-    // a wait that runs out is reported; the warps go on in step, so that they meet at their barriers
-    if (!mbar_wait(&bar[0], c & 1)) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
-    __syncthreads();                                       // W and M V are there, S is published
+    // ---- values written: u = M V - W S ----
+    arrived(0, c);
     float acc[2][4];
 #pragma unroll
     for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    rows_times_s(acc, wb);
+    rows_times_s(acc, wb, smem_u32(s_b + (c & 1) * C::S));
+    __nv_bfloat16* u_s = reinterpret_cast<__nv_bfloat16*>(u_b + (c & 1) * C::U);       // the outputs are done with it
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -843,39 +898,12 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
         *reinterpret_cast<uint32_t*>(u_s + t * C::SLD + col) = hi;
         *reinterpret_cast<uint32_t*>(u_s + kChunk * C::SLD + t * C::SLD + col) = lo;
       }
-    if (!mbar_wait(&bar[1], c & 1)) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
-    __syncthreads();                                       // the rest is there, u is written, W and M V are read
-    if (threadIdx.x == 0 && c + 1 < chunks) fetch_first(c + 1);
-    // ---- outputs ----
-#pragma unroll
-    for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    rows_times_s(acc, qb);
-#pragma unroll
-    for (int ks = 0; ks < kRuns; ++ks) {
-      if (ks > a) continue;
-      uint32_t ah[4], al[4], h0, h1, h2, h3, l0, l1, l2, l3;
-      const uint32_t ao = ((a * kRun + (lane & 15)) * C::MLD + ks * 16 + (lane >> 4) * 8) * 2;
-      ldsm_x4(ab + ao, ah[0], ah[1], ah[2], ah[3]);
-      ldsm_x4(ab + A_LO + ao, al[0], al[1], al[2], al[3]);
-      const uint32_t uo = ((ks * 16 + (mm & 1) * 8 + rr) * C::SLD + c0 + (mm >> 1) * 8) * 2;
-      ldsm_x4_trans(ub + uo, h0, h1, h2, h3);
-      ldsm_x4_trans(ub + U_LO + uo, l0, l1, l2, l3);
-      mma_bf16(acc[0], ah, h0, h1);
-      mma_bf16(acc[1], ah, h2, h3);
-      mma_bf16(acc[0], ah, l0, l1);
-      mma_bf16(acc[1], ah, l2, l3);
-      mma_bf16(acc[0], al, h0, h1);
-      mma_bf16(acc[1], al, h2, h3);
-    }
-#pragma unroll
-    for (int i = 0; i < 2; ++i)
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int t = c * kChunk + t0 + h * 8, col = v0 + c0 + i * 8 + (lane & 3) * 2;
-        if (t < n_tok && col < p.vdim)
-          *reinterpret_cast<float2*>(p.o + ((tok0 + t) * p.heads + head) * p.vdim + col) = make_float2(acc[i][2 * h], acc[i][2 * h + 1]);
-      }
+    named_sync(kBarChain, kDsGroup);                       // u is written, W and M V are read
+    if (threadIdx.x == 0 && c + 1 < chunks) fetch_w(c + 1);
+    named_arrive(kBarFull + (c & 1), kDsThreads);
     // ---- the next state ----
+    arrived(1, c);
+    const uint32_t ub = smem_u32(u_s);
     const float e0 = decay_s[d0], e1 = decay_s[d1];
 #pragma unroll
     for (int i = 0; i < SN; ++i) {
@@ -904,9 +932,11 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
         mma_bf16(S[i + 1], kl, h2, h3);
       }
     }
-    __syncthreads();                                       // S, u and the copies are read
-    if (threadIdx.x == 0 && c + 1 < chunks) fetch_rest(c + 1);
-    publish();
+    if (c + 1 == chunks) break;
+    if (c > 0) named_sync(kBarFree + ((c - 1) & 1), kDsThreads);         // the outputs are done with the other buffers
+    publish((c + 1) & 1);
+    named_sync(kBarChain, kDsGroup);                       // the state is published, keys are read
+    if (threadIdx.x == 0) fetch_keys(c + 1);
   }
 #pragma unroll
   for (int i = 0; i < SN; ++i) {
