@@ -443,20 +443,21 @@ int launch_talk_decode(const nfk_talk_attn_params& p, cudaStream_t stream) {
 
 // ---- prefill --------------------------------------------------------------------------------------------------
 constexpr int kTpQ = 16, kTpHeads = 16, kTpThreads = kTpHeads * 32;
-constexpr int kTpPages = 1024;             // page ids kept in shared memory; later ones are looked up in memory
+constexpr int kTpPages = 1024;             // pages that the keys of a work item may lie in
 
 template <int HD, int KT>
 struct TalkCfg {
-  static constexpr int KLD = HD + 8;                     // row strides in elements: conflict-free ldmatrix
-  static constexpr int XLD = KT + 8;                     // mixed weights [head][query][key]
+  static constexpr int XLD = KT + 8;                     // mixed weights [head][query][key]; strides without bank conflicts
   static constexpr int XHD = kTpQ * XLD + 8;             // ... from head to head
   static constexpr int PLD = kTpQ * KT + 8;              // weights [head][query * KT + key], see p_col
-  static constexpr int ROWS = KT * KLD * 2;              // keys or values of a KV head
+  static constexpr int BOX = kPage * 128;                // 64 columns of a page's keys or values, 128-byte swizzle
+  static constexpr int PAGE_BYTES = HD / 64 * BOX;
+  static constexpr int ROWS = KT / kPage * PAGE_BYTES;   // keys or values of a KV head
   static constexpr int X_BYTES = kTpHeads * XHD * 2;
   __host__ __device__ static constexpr int p_bytes(int hp) { return hp * PLD * 2; }
-  // keys | values | weights (pair) | mixed weights (pair, two buffers) | mixing matrix in fragments | page ids
+  // keys | values | weights (pair) | mixed weights (pair, two buffers) | mixing matrix in fragments | page ids | barriers
   __host__ __device__ static constexpr int smem(int hp, int kvs) {
-    return 2 * kvs * ROWS + 2 * p_bytes(hp) + 4 * X_BYTES + hp / 16 * 512 + kTpPages * 4;
+    return 1024 + 2 * kvs * ROWS + 2 * p_bytes(hp) + 4 * X_BYTES + hp / 16 * 512 + kTpPages * 4 + 16;
   }
 };
 // Column of a query's block of eight keys: neighbouring queries' blocks lie in different banks.
@@ -470,6 +471,12 @@ __device__ __forceinline__ void stsm_x4(uint32_t addr, uint32_t r0, uint32_t r1,
                : "memory");
 }
 
+// x ^ bits, computed where it stands (kept in registers across a loop, the variants of an address cost spills).
+__device__ __forceinline__ uint32_t flip(uint32_t x, uint32_t bits) {
+  uint32_t r;
+  asm volatile("xor.b32 %0, %1, %2;" : "=r"(r) : "r"(x), "r"(bits));
+  return r;
+}
 // The cluster's barrier in two halves, so that work fits in between.
 __device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
 __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
@@ -477,16 +484,17 @@ __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.w
 // hp: heads padded to a multiple of 16; kvs: KV heads that 16 query heads can touch.
 template <int HD, int KT>
 __global__ void __launch_bounds__(kTpThreads, 1)
-talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
+talk_prefill_kernel(const __grid_constant__ CUtensorMap tm, nfk_talk_attn_params p, int hp, int kvs) {
   using Cfg = TalkCfg<HD, KT>;
   constexpr int NT = KT / 8;                             // key blocks of a tile
-  extern __shared__ __align__(16) uint8_t tps[];
-  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(tps);
-  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(tps + kvs * Cfg::ROWS);
+  extern __shared__ __align__(16) uint8_t tps_raw[];
+  uint8_t* tps = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tps_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  uint8_t *k_s = tps, *v_s = tps + kvs * Cfg::ROWS;
   __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(tps + 2 * kvs * Cfg::ROWS);          // high parts, then low parts
   __nv_bfloat16* x_s = reinterpret_cast<__nv_bfloat16*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp));
   uint4* t_s = reinterpret_cast<uint4*>(tps + 2 * kvs * Cfg::ROWS + 2 * Cfg::p_bytes(hp) + 4 * Cfg::X_BYTES);
   int* page_s = reinterpret_cast<int*>(t_s + hp / 16 * 32);
+  uint64_t* bar = reinterpret_cast<uint64_t*>(page_s + kTpPages);            // copies into k_s and v_s
   cg::cluster_group cluster = cg::this_cluster();
   const int C = hp / kTpHeads, rank = static_cast<int>(cluster.block_rank());
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -501,35 +509,39 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   const int kvl = live ? head / group - kv0 : 0;         // this warp's KV head among the CTA's
   const int first = p.window > 0 ? max(0, pos0 - p.window + 1) : 0, last = pos0 + cnt - 1;
   const int lo = first / KT * KT, tiles = (last - lo) / KT + 1;
-  const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
-  const long long head_step = kPage * HD, v_step = G * head_step;
-
-  const int slot0 = first / kPage;
-  for (int i = threadIdx.x; i < kTpPages && slot0 + i <= last / kPage; i += kTpThreads)
-    page_s[i] = page_of((slot0 + i) * kPage, req, kPage, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
+  const int slot0 = first / kPage, slot1 = last / kPage;
+  if (threadIdx.x == 0) {
+    mbar_init(&bar[0], 1);
+    mbar_init(&bar[1], 1);
+    mbar_fence_init();
+    tma_prefetch_desc(&tm);
+  }
+  if (slot1 - slot0 >= kTpPages && threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
+  for (int i = threadIdx.x; i < kTpPages && slot0 + i <= slot1; i += kTpThreads)
+    page_s[i] = max(page_of((slot0 + i) * kPage, req, kPage, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status), 0) * 2 * G * kPage;
   for (int i = threadIdx.x; i < hp / 16 * 32; i += kTpThreads) t_s[i] = talk_fragment(p, head0, i / 32 * 16, i & 31);
   __syncthreads();
 
-  // keys or values of a tile (from KV head kv0) into dst; keys that are not there become zeros. A thread brings the same
-  // 16 bytes of a key for one KV head after the other.
-  constexpr int CH = HD / 8, UNIT = KT * CH;
-  const int my_key = threadIdx.x % UNIT / CH, my_col = (threadIdx.x % CH) * 8;
-  auto fetch = [&](__nv_bfloat16* dst, int t, long long off) {
-    const int j = lo + t * KT + my_key;
-    int page = -1;
-    if (j >= first && j <= last) {
-      const int slot = j / kPage - slot0;
-      page = slot < kTpPages ? page_s[slot]
-                             : page_of(j, req, kPage, p.kv_indptr, p.kv_indices, p.kv_first, p.num_pages, p.status);
+  // Copies of a tile's pages, the CTA's KV heads one after the other, by the first warp. kind: 0 keys, 1 values. Past the
+  // first and last page that one again: all keys outside the range get no weight.
+  const int pages = min(slot1 - slot0, kTpPages - 1), page0 = lo / kPage - slot0;
+  auto fetch = [&](int buf, int t, int kind) {
+    if (warp != 0) return;
+    if (lane == 0) mbar_expect_tx(&bar[buf], kvn * Cfg::ROWS);
+    __syncwarp();
+    constexpr int HB = HD / 64, PG = KT / kPage;
+    const int row0 = (kind * G + kv0) * kPage;
+#pragma unroll 1
+    for (int i = lane; i < kvn * PG * HB; i += 32) {
+      const int half = i % HB, pg = i / HB % PG, kv = i / (HB * PG);
+      const int page = page_s[min(max(page0 + t * PG + pg, 0), pages)];
+      tma_load_2d((buf == 0 ? k_s : v_s) + kv * Cfg::ROWS + pg * Cfg::PAGE_BYTES + half * Cfg::BOX, &tm, &bar[buf], half * 64,
+                  page + row0 + kv * kPage);
     }
-    const bool ok = page >= 0;
-    const __nv_bfloat16* src = pool + off + my_col;
-    if (ok) src += (static_cast<long long>(page) * 2 * G * kPage + j % kPage) * HD + kv0 * head_step;
-    const uint32_t d = smem_u32(dst + my_key * Cfg::KLD + my_col);
-    for (int kv = threadIdx.x / UNIT; kv < kvn; kv += kTpThreads / UNIT)
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d + kv * Cfg::ROWS), "l"(ok ? src + kv * head_step : pool),
-                   "r"(ok ? 16 : 0) : "memory");
   };
+  // a wait that runs out is reported at the end; the warps go on in step, so that they meet at their barriers
+  bool late = false;
+  auto arrived = [&](int buf, int n) { late |= !mbar_wait(&bar[buf], n & 1); };      // the n-th copy into a buffer
 
   uint32_t qa[HD / 16][4];
   {
@@ -539,11 +551,13 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   const int mm = lane >> 3, rr = lane & 7;
   const float scale = p.scale * kLog2e;
   const int i0 = pos0 + (lane >> 2), i1 = i0 + 8;        // positions of this lane's two queries
-  const uint32_t vb = smem_u32(v_s) + kvl * Cfg::ROWS;
+  // 16-byte pieces of a row lie at their number xor the row's: this lane's row and first piece, later ones by an xor
+  const uint32_t k_lane = ((mm >> 1) * 8 + rr) * 128 + (((mm & 1) ^ rr) << 4), v_lane = ((mm & 1) * 8 + rr) * 128 + (((mm >> 1) ^ rr) << 4);
+  const uint32_t vb = smem_u32(v_s) + kvl * Cfg::ROWS + v_lane;
   auto seen = [&](int i, int j) { return j <= i && j >= 0 && (p.window <= 0 || i - j < p.window); };
   // scores of this warp's head, -inf where the query does not see the key
-  auto scores = [&](float (&s)[NT][4], const __nv_bfloat16* keys, int t) {
-    const uint32_t kb = smem_u32(keys) + kvl * Cfg::ROWS;
+  auto scores = [&](float (&s)[NT][4], const uint8_t* keys, int t) {
+    const uint32_t kb = smem_u32(keys) + kvl * Cfg::ROWS + k_lane;
 #pragma unroll
     for (int b = 0; b < NT; ++b) s[b][0] = s[b][1] = s[b][2] = s[b][3] = 0.f;
 #pragma unroll
@@ -551,7 +565,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
 #pragma unroll
       for (int b = 0; b < NT; b += 2) {
         uint32_t b0, b1, b2, b3;
-        ldsm_x4(kb + ((b * 8 + (mm >> 1) * 8 + rr) * Cfg::KLD + ks * 16 + (mm & 1) * 8) * 2, b0, b1, b2, b3);
+        ldsm_x4(flip(kb, (ks & 3) << 5) + b / 2 * Cfg::PAGE_BYTES + ks / 4 * Cfg::BOX, b0, b1, b2, b3);
         mma_bf16(s[b], qa[ks], b0, b1);
         mma_bf16(s[b + 1], qa[ks], b2, b3);
       }
@@ -571,13 +585,11 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   // ---- first loop: maxima and sums, keys in the two buffers by turns ----
   const float sink = p.sinks != nullptr && live ? p.sinks[head] * kLog2e : -INFINITY;
   float m0 = sink, m1 = sink, l0 = 0.f, l1 = 0.f;        // of scores times log2 e; sums of this lane's keys
-  fetch(k_s, 0, 0);
-  cp_async_commit();
+  fetch(0, 0, 0);
   for (int t = 0; t < tiles; ++t) {
-    cp_async_wait<0>();
-    __syncthreads();
-    if (t + 1 < tiles) fetch((t & 1) != 0 ? k_s : v_s, t + 1, 0);
-    cp_async_commit();
+    arrived(t & 1, t >> 1);
+    __syncthreads();                                     // everyone is done with the other buffer
+    if (t + 1 < tiles) fetch((t + 1) & 1, t + 1, 0);
     float s[NT][4];
     scores(s, (t & 1) != 0 ? v_s : k_s, t);
     float x0 = s[0][0], x1 = s[0][2];
@@ -600,8 +612,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
     }
   }
   __syncthreads();
-  fetch(k_s, 0, 0);
-  cp_async_commit();
+  fetch(0, 0, 0);
   // weight = 2^(score - m - log2(sum)); rows of the tile that are no queries get none
   l0 = quad_sum(l0);
   l1 = quad_sum(l1);
@@ -621,8 +632,8 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   // mixed weights of tile t times its values
   auto values = [&](int t) {
     const uint32_t base = xb + ((t & 1) != 0 ? 2 * x_lo : 0);
-#pragma unroll
-    for (int ks = 0; ks < KT / 16; ++ks) {
+#pragma unroll 1
+    for (int ks = 0; ks < KT / 16; ++ks) {               // (registers: what unrolling would hoist has no room)
       uint32_t ah[4], al[4];
       const uint32_t o = (warp * Cfg::XHD + (lane & 15) * Cfg::XLD + ks * 16 + (lane >> 4) * 8) * 2;
       ldsm_x4(base + o, ah[0], ah[1], ah[2], ah[3]);
@@ -630,7 +641,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
 #pragma unroll
       for (int b = 0; b < HD / 8; b += 2) {
         uint32_t b0, b1, b2, b3;
-        ldsm_x4_trans(vb + ((ks * 16 + (mm & 1) * 8 + rr) * Cfg::KLD + (b + (mm >> 1)) * 8) * 2, b0, b1, b2, b3);
+        ldsm_x4_trans(flip(vb, (b / 2 & 3) << 5) + ks * Cfg::PAGE_BYTES + b / 8 * Cfg::BOX, b0, b1, b2, b3);
         mma_bf16(acc[b], ah, b0, b1);
         mma_bf16(acc[b + 1], ah, b2, b3);
         mma_bf16(acc[b], al, b0, b1);
@@ -640,11 +651,10 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
   };
   // Products with values lag by one tile: they run while the weights travel to the other CTAs.
   if (C > 1) cluster_arrive();
-  cp_async_wait<0>();
-  __syncthreads();
   for (int t = 0; t < tiles; ++t) {
     {
       float s[NT][4];
+      arrived(0, (tiles + 1) / 2 + t);
       scores(s, k_s, t);
       uint32_t hi[NT][2], lw[NT][2];
 #pragma unroll
@@ -665,6 +675,7 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
         constexpr int N16 = kTpQ * KT / 8;               // 16-byte pieces of a part
         const uint4* src = reinterpret_cast<const uint4*>(p_s + head * Cfg::PLD);
         const int part = static_cast<int>(p_lo / 16);
+#pragma unroll 1
         for (int r = 1; r < C; ++r) {
           uint4* dst = cluster.map_shared_rank(const_cast<uint4*>(src), rank + r < C ? rank + r : rank + r - C);
 #pragma unroll
@@ -676,17 +687,19 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
       }
     }
     if (C > 1) cluster_arrive();
-    cp_async_wait<0>();
-    __syncthreads();                                     // this CTA's weights and the last tile's values are there
-    if (t > 0) values(t - 1);
+    else __syncthreads();                                // the weights are there
+    if (t > 0) {
+      arrived(1, tiles / 2 + t - 1);
+      values(t - 1);
+    }
     if (C > 1) cluster_wait();
-    if (t + 1 < tiles) fetch(k_s, t + 1, 0);             // everyone is done with these keys
-    cp_async_commit();
+    if (t + 1 < tiles) fetch(0, t + 1, 0);               // everyone is done with these keys
     // mixed weights of the CTA's 16 heads: [16 x H] times [H x (query, key)], columns over the warps: one query per warp
     {
       float x[NT][4];
 #pragma unroll
       for (int b = 0; b < NT; ++b) x[b][0] = x[b][1] = x[b][2] = x[b][3] = 0.f;
+#pragma unroll 1
       for (int g = 0; g < hp; g += 16) {
         const uint4 tf = t_s[g * 2 + lane];
         const uint32_t a[4] = {tf.x, tf.y, tf.z, tf.w};
@@ -719,14 +732,12 @@ talk_prefill_kernel(nfk_talk_attn_params p, int hp, int kvs) {
         stsm_x4(base + x_lo + o, lw[0], lw[1], lw[2], lw[3]);
       }
     }
-    cp_async_wait<0>();
-    __syncthreads();                                     // mixed weights and the next keys are there, the last values are read
-    fetch(v_s, t, v_step);
-    cp_async_commit();
+    __syncthreads();                                     // mixed weights are there, the last values are read
+    fetch(1, t, 1);
   }
-  cp_async_wait<0>();
-  __syncthreads();
+  arrived(1, tiles / 2 + tiles - 1);
   values(tiles - 1);
+  if (late) report_status(p.status, NF_ST_TIMEOUT_SMEM_FULL);
   // ---- outputs turn back by their query's angles ----
   if (live) {
     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out);
@@ -758,6 +769,9 @@ template <int HD, int KT>
 int launch_talk_prefill(const nfk_talk_attn_params& p, int hp, int kvs, cudaStream_t stream) {
   const int C = hp / kTpHeads, sm = TalkCfg<HD, KT>::smem(hp, kvs);
   auto kernel = talk_prefill_kernel<HD, KT>;
+  CUtensorMap tm;
+  const int rc = make_tmap_bf16_2d(&tm, p.pool, static_cast<uint64_t>(p.num_pages) * 2 * p.kv_heads * kPage, HD, HD, kPage, 64);
+  if (rc != NF_OK) return rc;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, sm) != cudaSuccess) return NF_ERR_CUDA;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(static_cast<unsigned>(p.num_items) * C);
@@ -770,7 +784,7 @@ int launch_talk_prefill(const nfk_talk_attn_params& p, int hp, int kvs, cudaStre
   attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
   cfg.attrs = attr;
   cfg.numAttrs = 1;
-  return cudaLaunchKernelEx(&cfg, kernel, p, hp, kvs) == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+  return cudaLaunchKernelEx(&cfg, kernel, tm, p, hp, kvs) == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 
 // KV heads that 16 neighbouring query heads (from a multiple of 16) can touch.
@@ -848,5 +862,5 @@ extern "C" int nfk_talk_attn_fits(int heads, int kv_heads, int hd, int max_keys)
   const int hp = (heads + kTpHeads - 1) / kTpHeads * kTpHeads, kvs = kv_heads_of_16(heads, heads / kv_heads);
   const int pre = hd == 64 ? TalkCfg<64, 16>::smem(hp, kvs) : TalkCfg<128, 16>::smem(hp, kvs);
   const int dec = talk_decode_layout(heads, hd, (max_keys + kTdMaxCluster - 1) / kTdMaxCluster).bytes;
-  return (pre <= 227 * 1024 ? 1 : 0) + (dec <= 220 * 1024 ? 2 : 0);
+  return (pre <= 227 * 1024 && max_keys <= (kTpPages - 3) * kPage ? 1 : 0) + (dec <= 220 * 1024 ? 2 : 0);
 }
