@@ -254,36 +254,18 @@ delta_seq_kernel(nfk_delta_params p, int v_slices) {
     if (col_ok) S[static_cast<long long>(d) * p.vdim] = S_s[d * kSeqCols + lane];
 }
 
-// Head norm, weight and gate of the rows left in p.o: one warp per (token, head). Row y of the grid is a request's
-// portion, or with CHUNKS a chunk.
-template <class T, bool CHUNKS>
+// Head norm, weight and gate of the rows that delta_seq_kernel left in p.o: one warp per (token, head).
+template <class T>
 __global__ void __launch_bounds__(256)
-delta_norm_kernel(nfk_delta_params p) {
+delta_seq_norm_kernel(nfk_delta_params p) {
   const int lane = threadIdx.x & 31;
-  const int req = CHUNKS ? 0 : p.seq_reqs[blockIdx.y];
-  const int t0 = CHUNKS ? p.items[blockIdx.y * 4 + 1] : p.qo_indptr[req];
-  const int n = CHUNKS ? p.items[blockIdx.y * 4 + 2] : p.qo_indptr[req + 1] - t0;
-  const unsigned total = static_cast<unsigned>(n) * p.heads;
-#pragma unroll 2
+  const int req = p.seq_reqs[blockIdx.y], t0 = p.qo_indptr[req];
+  const unsigned total = static_cast<unsigned>(p.qo_indptr[req + 1] - t0) * p.heads;
   for (unsigned i = blockIdx.x * 8u + (threadIdx.x >> 5); i < total; i += gridDim.x * 8u) {
     const unsigned row = i / static_cast<unsigned>(p.heads);
     const long long t = t0 + static_cast<long long>(row);
     const int head = static_cast<int>(i - row * p.heads);
     const float* o = p.o + (t * p.heads + head) * p.vdim;
-    if (CHUNKS) {                                          // one round: at most 128 values
-      const int c = lane * 4;
-      const bool ok = c < p.vdim;
-      const float4 v = ok ? load4(o + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-      const float4 gg = ok ? load4(reinterpret_cast<const T*>(p.g) + t * p.ld_g + head * p.vdim + c) : v;
-      const float inv = rsqrtf(warp_sum((v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w)) / static_cast<float>(p.vdim_real) + p.eps);
-      if (ok) {
-        const float4 w = load4(p.norm + c);
-        store4(reinterpret_cast<T*>(p.y) + t * p.ld_y + head * p.vdim + c,
-               make_float4(v.x * inv * w.x * sigmoid_fast(gg.x), v.y * inv * w.y * sigmoid_fast(gg.y),
-                           v.z * inv * w.z * sigmoid_fast(gg.z), v.w * inv * w.w * sigmoid_fast(gg.w)));
-      }
-      continue;
-    }
     float ss = 0.f;
     for (int c = lane * 4; c < p.vdim; c += 128) {
       const float4 v = load4(o + c);
@@ -947,6 +929,32 @@ delta_scan_kernel(nfk_delta_params p, int slices) {
   }
 }
 
+// Head norm, weight and gate of a chunk (row y of the grid): a block takes a head, its warps a token each in turn. At most
+// 128 values per head, four per lane.
+__global__ void __launch_bounds__(256)
+delta_chunk_norm_kernel(nfk_delta_params p) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, head = blockIdx.x, c = lane * 4;
+  const int n = p.items[blockIdx.y * 4 + 2];
+  const long long t0 = p.items[blockIdx.y * 4 + 1];
+  const bool ok = c < p.vdim;
+  const int col = head * p.vdim + (ok ? c : 0);
+  const float* o = p.o + t0 * p.heads * p.vdim + col;
+  const __nv_bfloat16* g = reinterpret_cast<const __nv_bfloat16*>(p.g) + t0 * p.ld_g + col;
+  __nv_bfloat16* y = reinterpret_cast<__nv_bfloat16*>(p.y) + t0 * p.ld_y + col;
+  const float4 w = load4(p.norm + (ok ? c : 0));
+  const float inv_n = 1.f / static_cast<float>(p.vdim_real);
+#pragma unroll 4
+  for (int t = warp; t < n; t += 8) {
+    const float4 gg = load4(g + t * p.ld_g);
+    float4 v = load4(o + static_cast<long long>(t) * p.heads * p.vdim);
+    if (!ok) v = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float inv = rsqrtf(warp_sum((v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w)) * inv_n + p.eps);
+    if (ok)
+      store4(y + t * p.ld_y, make_float4(v.x * inv * w.x * sigmoid_fast(gg.x), v.y * inv * w.y * sigmoid_fast(gg.y),
+                                         v.z * inv * w.z * sigmoid_fast(gg.z), v.w * inv * w.w * sigmoid_fast(gg.w)));
+  }
+}
+
 template <class K>
 int set_smem(K kernel, size_t bytes) {
   if (bytes > 227 * 1024) return NF_ERR_UNSUPPORTED;
@@ -980,7 +988,7 @@ int launch_delta_seq(const nfk_delta_params& p, cudaStream_t stream) {
   if (rc != NF_OK) return rc;
   delta_seq_kernel<T><<<static_cast<int>(grid), 256, sm, stream>>>(p, v_slices);
   if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
-  delta_norm_kernel<T, false><<<dim3(64, p.num_seq), 256, 0, stream>>>(p);
+  delta_seq_norm_kernel<T><<<dim3(64, p.num_seq), 256, 0, stream>>>(p);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 
@@ -1000,8 +1008,7 @@ int launch_delta_chunks(const nfk_delta_params& p, cudaStream_t stream) {
   if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
   delta_scan_kernel<P><<<portions * p.heads * slices, kDsThreads, DeltaScanCfg<P>::SMEM, stream>>>(p, slices);
   if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
-  const int per = kChunk * p.heads / 8;
-  delta_norm_kernel<__nv_bfloat16, true><<<dim3(per < 64 ? (per > 0 ? per : 1) : 64, p.num_items), 256, 0, stream>>>(p);
+  delta_chunk_norm_kernel<<<dim3(p.heads, p.num_items), 256, 0, stream>>>(p);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 

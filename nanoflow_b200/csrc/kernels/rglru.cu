@@ -2,9 +2,9 @@
 // Language Models"; see kernels.h for the equations). State, gates, decays and their logarithms are fp32.
 //
 // nfk_rglru_decode   one token per request: a thread per channel.
-// nfk_rglru_prefill  a CTA takes 32 channels of a request and walks its tokens 128 at a time: each of 16 warps reduces
-//                    eight tokens to (decay, end state from zero), all chain those, and every warp then runs its tokens
-//                    again from the state it starts with, out of registers. Inputs are read once, a step ahead.
+// nfk_rglru_prefill  a CTA takes 32 (or 16) channels of a request and walks its tokens 128 (256) at a time, in runs of eight:
+//                    each run is reduced to (decay, end state from zero), all chain those, and every run then goes through
+//                    its tokens again from the state it starts with, out of registers. Inputs are read once, a step ahead.
 #include "elem_io.cuh"
 
 namespace nf {
@@ -66,7 +66,7 @@ rglru_decode_kernel(nfk_rglru_params p) {
   put(reinterpret_cast<T*>(p.out) + t * p.ld_out + c, x * gelu_tanh_f<kFast<T>>(to_f32(reinterpret_cast<const T*>(p.y)[t * p.ld_y + c])));
 }
 
-constexpr int kRgWarps = 16, kRgRun = 8, kRgBlock = kRgWarps * kRgRun;
+constexpr int kRgWarps = 16, kRgRun = 8;
 
 // What a thread reads of its run of tokens.
 template <class T>
@@ -75,12 +75,14 @@ struct RgInputs {
   T u[kRgRun], y[kRgRun];
 };
 
-template <class T>
+// CW: channels per CTA, 32 or (when there are few CTAs) 16; 32 / CW runs of tokens share a warp.
+template <class T, int CW>
 __global__ void __launch_bounds__(kRgWarps * 32)
 rglru_prefill_kernel(nfk_rglru_params p) {
-  __shared__ float a_s[2][kRgWarps][32], b_s[2][kRgWarps][32];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int c = blockIdx.x * 32 + lane;
+  constexpr int kRuns = kRgWarps * 32 / CW, kBlock = kRuns * kRgRun;
+  __shared__ float a_s[2][kRuns][CW], b_s[2][kRuns][CW];
+  const int run = threadIdx.x / CW, lane = threadIdx.x % CW;
+  const int c = blockIdx.x * CW + lane;
   const int req = p.req_begin + blockIdx.y;
   const int ref = p.state_slot[req];
   if (ref < 0 || (ref >> 1) >= p.num_slots) {
@@ -105,12 +107,12 @@ rglru_prefill_kernel(nfk_rglru_params p) {
       in.y[j] = y[t * p.ld_y];
     }
   };
-  float carry = (ok && p.positions[t0] != 0) ? *S : 0.f;             // every warp keeps it
+  float carry = (ok && p.positions[t0] != 0) ? *S : 0.f;             // every run keeps it
   RgInputs<T> in;
-  fetch(in, t0 + warp * kRgRun);
+  fetch(in, t0 + run * kRgRun);
   int buf = 0;
-  for (int base = t0; base < t1; base += kRgBlock, buf ^= 1) {
-    const int begin = base + warp * kRgRun;
+  for (int base = t0; base < t1; base += kBlock, buf ^= 1) {
+    const int begin = base + run * kRgRun;
     RgStep s[kRgRun];
     float yy[kRgRun], a = 1.f, b = 0.f;
 #pragma unroll
@@ -124,14 +126,14 @@ rglru_prefill_kernel(nfk_rglru_params p) {
       a *= s[j].a;
       b = s[j].a * b + s[j].b;
     }
-    if (base + kRgBlock < t1) fetch(in, begin + kRgBlock);           // while the warps wait for one another
-    a_s[buf][warp][lane] = a;
-    b_s[buf][warp][lane] = b;
+    if (base + kBlock < t1) fetch(in, begin + kBlock);               // while the warps wait for one another
+    a_s[buf][run][lane] = a;
+    b_s[buf][run][lane] = b;
     __syncthreads();
     float x = carry;
 #pragma unroll
-    for (int k = 0; k < kRgWarps; ++k) {
-      if (k == warp) x = carry;                                      // what this warp's run starts from
+    for (int k = 0; k < kRuns; ++k) {
+      if (k == run) x = carry;                                       // what this run starts from
       carry = a_s[buf][k][lane] * carry + b_s[buf][k][lane];
     }
 #pragma unroll
@@ -140,7 +142,16 @@ rglru_prefill_kernel(nfk_rglru_params p) {
       if (begin + j < t1 && ok) put(out + static_cast<long long>(begin + j) * p.ld_out, x * yy[j]);
     }
   }
-  if (warp == 0 && ok) *S = carry;
+  if (run == 0 && ok) *S = carry;
+}
+
+template <class T>
+void launch_rglru_prefill(const nfk_rglru_params& p, cudaStream_t stream) {
+  const int wide = (p.cols + 31) / 32;
+  if (wide * p.req_count < device_sm_count())
+    rglru_prefill_kernel<T, 16><<<dim3((p.cols + 15) / 16, p.req_count), kRgWarps * 32, 0, stream>>>(p);
+  else
+    rglru_prefill_kernel<T, 32><<<dim3(wide, p.req_count), kRgWarps * 32, 0, stream>>>(p);
 }
 
 int check_rglru(const nfk_rglru_params* p) {
@@ -169,8 +180,7 @@ extern "C" int nfk_rglru_prefill(const nfk_rglru_params* p, cudaStream_t stream)
   using namespace nf;
   const int rc = check_rglru(p);
   if (rc != NF_OK || p->req_count == 0) return rc;
-  const dim3 grid((p->cols + 31) / 32, p->req_count);
-  if (p->dtype == NFK_F32) rglru_prefill_kernel<float><<<grid, kRgWarps * 32, 0, stream>>>(*p);
-  else rglru_prefill_kernel<__nv_bfloat16><<<grid, kRgWarps * 32, 0, stream>>>(*p);
+  if (p->dtype == NFK_F32) launch_rglru_prefill<float>(*p, stream);
+  else launch_rglru_prefill<__nv_bfloat16>(*p, stream);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
