@@ -113,7 +113,21 @@ struct DecCfg {
 constexpr int kDecodeCounterSlots = 64;
 __device__ unsigned int g_decode_counters[kDecodeCounterSlots][2];
 
-// EXT: sink in the denominator, capped scores, probabilities as a bf16 pair (in an instantiation of its own).
+// What the token at the end of a request sees: its position, the page slot that the page list starts with, and how many
+// pages of the list lie before the token's chunk.
+struct DecodeRange {
+  int pos, first, skip;
+};
+__device__ __forceinline__ DecodeRange decode_range(const nfk_attn_params& p, int req, int np, int last_len) {
+  DecodeRange r;
+  r.first = p.kv_first != nullptr ? p.kv_first[req] : 0;
+  r.pos = (r.first + np - 1) * kPage + last_len - 1;
+  r.skip = p.chunk > 0 && np > 0 ? max(0, r.pos / p.chunk * p.chunk / kPage - r.first) : 0;
+  return r;
+}
+
+// EXT: sink in the denominator, capped scores, distance bias, chunks, page lists that start inside the sequence, queries in
+// wider rows, probabilities as a bf16 pair (in an instantiation of its own).
 template <int HD, int ST, bool EXT>
 __global__ void __launch_bounds__(kDecThreads, EXT ? 2 : 3)
 attn_decode_kernel(nfk_attn_params p, int slot) {
@@ -145,21 +159,28 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
     const int pg0 = p.kv_indptr[req];
     const int np = p.kv_indptr[req + 1] - pg0;
     const int last_len = p.kv_last_page_len[req];
-    int c_begin = 0, c_end = np, n_chunks = 1;
+    const DecodeRange rg = EXT ? decode_range(p, req, np, last_len) : DecodeRange{0, 0, 0};
+    int c_begin = rg.skip, c_end = np, n_chunks = 1;
     if (p.chunk_pages > 0) {
       // A context longer than chunk_pages * max_chunks pages still has only max_chunks work items:
       // the last one takes all remaining pages, and the merge below counts the same number of chunks.
-      c_begin = chunk * p.chunk_pages;
+      c_begin = rg.skip + chunk * p.chunk_pages;
       c_end = (chunk == max_chunks - 1) ? np : min(np, c_begin + p.chunk_pages);
-      n_chunks = min(max_chunks, (np + p.chunk_pages - 1) / p.chunk_pages);
+      n_chunks = min(max_chunks, (np - rg.skip + p.chunk_pages - 1) / p.chunk_pages);
     }
     if (c_begin >= c_end) break;  // uniform across the CTA: on to the next item
     const int tok = p.qo_indptr[req];
+    const long long ld_q = EXT && p.ld_q > 0 ? p.ld_q : p.q_heads * HD;
+    float2 far0 = make_float2(0.f, 0.f), far1 = far0;        // distance bias of this lane's two rows
+    if (EXT && p.dist != nullptr) {
+      const float2* dist = reinterpret_cast<const float2*>(p.dist) + kvh * group;
+      if ((lane >> 2) < group) far0 = dist[lane >> 2];
+      if ((lane >> 2) + 8 < group) far1 = dist[(lane >> 2) + 8];
+    }
 
     uint32_t qa[HD / 16][4];
     load_q_frags<HD>(qa, [&](int r) -> const __nv_bfloat16* {
-      return r < group ? qbase + (static_cast<long long>(tok) * p.q_heads + kvh * group + r) * HD
-                       : nullptr;
+      return r < group ? qbase + tok * ld_q + (kvh * group + r) * HD : nullptr;
     });
 
     float o[HD / 8][4];
@@ -215,6 +236,24 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
       for (int e = 0; e < 4; ++e) {
         s0[e] = (c0 + (e & 1) < valid) ? s0[e] * scale : -INFINITY;
         s1[e] = (8 + c0 + (e & 1) < valid) ? s1[e] * scale : -INFINITY;
+      }
+      if (EXT && p.dist != nullptr) {                        // masked entries stay at minus infinity
+        const float d0 = static_cast<float>(rg.pos - (rg.first + pslot) * kPage - c0);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = e < 2 ? far0 : far1;
+          const float d = fmaxf(d0 - (e & 1), 0.f), d8 = fmaxf(d0 - (e & 1) - 8.f, 0.f);
+          s0[e] -= f.x * __log2f(fmaf(f.y, d, 1.f));
+          s1[e] -= f.x * __log2f(fmaf(f.y, d8, 1.f));
+        }
+      }
+      if (EXT && pslot == rg.skip && p.chunk > 0) {          // the page that the chunk starts in
+        const int lo = rg.pos / p.chunk * p.chunk - (rg.first + pslot) * kPage;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          if (c0 + (e & 1) < lo) s0[e] = -INFINITY;
+          if (8 + c0 + (e & 1) < lo) s1[e] = -INFINITY;
+        }
       }
       const float mx0 = quad_max(fmaxf(fmaxf(s0[0], s0[1]), fmaxf(s1[0], s1[1])));
       const float mx1 = quad_max(fmaxf(fmaxf(s0[2], s0[3]), fmaxf(s1[2], s1[3])));
@@ -327,7 +366,8 @@ __global__ void attn_decode_merge_kernel(nfk_attn_params p) {
   const int bl = blockIdx.x / p.q_heads, head = blockIdx.x % p.q_heads;
   const int req = p.req_begin + bl;
   const int np = p.kv_indptr[req + 1] - p.kv_indptr[req];
-  const int n_chunks = min(p.max_chunks, (np + p.chunk_pages - 1) / p.chunk_pages);   // as in the decode kernel
+  const int seen = np - decode_range(p, req, np, p.kv_last_page_len[req]).skip;
+  const int n_chunks = min(p.max_chunks, (seen + p.chunk_pages - 1) / p.chunk_pages);   // as in the decode kernel
   if (n_chunks <= 1) return;  // the decode kernel already wrote the final rows
   const float* ws = p.workspace + (static_cast<long long>(bl) * p.q_heads + head) * p.max_chunks * (HD + 2);
   float mm = -INFINITY;
@@ -519,6 +559,8 @@ attn_prefill_kernel(nfk_attn_params p) {
 inline int sm_count_attn() { return device_sm_count(); }
 
 bool decode_ext(const nfk_attn_params& p) { return p.sinks != nullptr || p.softcap > 0.f || p.precise != 0; }
+// What only the extended kernels know.
+bool ext_only(const nfk_attn_params& p) { return p.kv_first != nullptr || p.dist != nullptr || p.chunk != 0 || p.ld_q != 0; }
 
 int check_common(const nfk_attn_params* p, bool decode = false) {
   if (p == nullptr) return NF_ERR_BAD_ARG;
@@ -531,6 +573,8 @@ int check_common(const nfk_attn_params* p, bool decode = false) {
   if (group > 16 || ((16 % group) != 0 && !(decode && decode_ext(*p)))) return NF_ERR_UNSUPPORTED;
   if (p->page_size != kPage || p->softcap < 0.f || (!decode && (p->sinks != nullptr || p->softcap > 0.f))) return NF_ERR_UNSUPPORTED;
   if (p->head_dim != 128 && p->head_dim != 64) return NF_ERR_UNSUPPORTED;
+  if (p->chunk < 0 || p->ld_q % 8 != 0 || (p->ld_q > 0 && p->ld_q < p->q_heads * p->head_dim)) return NF_ERR_BAD_ARG;
+  if (ext_only(*p) && !(decode && p->precise != 0)) return NF_ERR_UNSUPPORTED;
   return NF_OK;
 }
 

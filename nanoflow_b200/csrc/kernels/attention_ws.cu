@@ -29,7 +29,9 @@
 // the first row's window are never loaded), a sink in the softmax denominator, K / V as columns of plain
 // rows instead of pool pages (keys expanded from a latent cache), and probabilities that enter the second
 // product as a bf16 pair: the high parts over the first half of the S accumulator, the low parts over the
-// second half. CAP adds capped scores (cap tanh(score / cap)); with either, head_dim 64 is built as well.
+// second half; also chunks (a position sees its own chunk only), and page lists that start inside the sequence.
+// CAP adds capped scores (cap tanh(score / cap)), DIST scores that lose a ln(1 + b distance) with two numbers per head;
+// with any of these, head_dim 64 is built as well.
 //
 // Takes the place of the reference's FlashInfer BatchPrefillWithPagedKVCacheKernel
 // (gemv/include/attention/prefill.cuh:1066-1374, mma.sync m16n16k16 + ldmatrix on sm_80).
@@ -89,7 +91,8 @@ constexpr uint32_t kIdescBMnMajor = 1u << 16;
 
 struct Item {
   int req, tok0, ntok, kvh, pg0, np, kv_len, q_end, n_tiles;
-  int t_first;      // first key tile (EXT: the one the first row's window starts in)
+  int t_first;      // first key tile (EXT: the one the first row's window or chunk starts in)
+  int pg_first;     // page slot of the sequence that the page list starts with
   bool valid;
 };
 template <bool EXT>
@@ -102,7 +105,8 @@ __device__ __forceinline__ Item read_item(const nfk_attn_params& p, long long w)
   it.ntok = p.items[item * 3 + 2];
   it.pg0 = p.kv_indptr[it.req];
   it.np = p.kv_indptr[it.req + 1] - it.pg0;
-  it.kv_len = (it.np - 1) * kPage + p.kv_last_page_len[it.req];
+  it.pg_first = EXT && p.kv_first != nullptr ? p.kv_first[it.req] : 0;
+  it.kv_len = (it.pg_first + it.np - 1) * kPage + p.kv_last_page_len[it.req];
   it.q_end = p.qo_indptr[it.req + 1];
   // absolute position of global token t of this request: kv_len - (q_end - t)
   const int kv_hi = it.kv_len - (it.q_end - (it.tok0 + it.ntok - 1)) + 1;   // keys visible to the last row
@@ -113,11 +117,14 @@ __device__ __forceinline__ Item read_item(const nfk_attn_params& p, long long w)
     const int lo = it.kv_len - (it.q_end - it.tok0) - p.window + 1;     // first key of the first row
     if (lo > 0) it.t_first = lo / kTile;
     it.n_tiles -= it.t_first;
+  } else if (EXT && p.chunk > 0 && it.valid) {
+    it.t_first = (it.kv_len - (it.q_end - it.tok0)) / p.chunk * p.chunk / kTile;
+    it.n_tiles -= it.t_first;
   }
   return it;
 }
 
-template <int HD, bool EXT, bool CAP>
+template <int HD, bool EXT, bool CAP, bool DIST>
 __global__ void __launch_bounds__(kThreads, 2)
 attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                        nfk_attn_params p) {
@@ -187,7 +194,8 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         } else {
         mbar_expect_tx(&bars[Q_FULL], static_cast<uint32_t>(it.ntok * group) * HD * 2);
         for (int tl = 0; tl < it.ntok; ++tl) {
-          const int grow = (it.tok0 + tl) * p.q_heads + it.kvh * group;     // row of the [T*q_heads][128] view
+          // row of the [T * heads per row][HD] view
+          const int grow = (it.tok0 + tl) * (EXT && p.ld_q > 0 ? p.ld_q / HD : p.q_heads) + it.kvh * group;
 #pragma unroll
           for (int h = 0; h < NH; ++h)
             tma_load_2d(smem + Q_OFF + h * 16384 + tl * group * 128, &tmQ, &bars[Q_FULL], h * 64, grow);
@@ -199,8 +207,9 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         auto fetch_pages = [&](int t) {
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
-            int pslot = (it.t_first + t) * (kTile / kPage) + j;
-            if (pslot >= it.np) pslot = 0;      // past the sequence: a valid page, masked by position
+            int pslot = (it.t_first + t) * (kTile / kPage) + j - it.pg_first;
+            // past the sequence, or given back since nobody sees it: a valid page, masked by position
+            if (pslot < 0 || pslot >= it.np) pslot = 0;
             int page = p.kv_indices[it.pg0 + pslot];
             if (page < 0 || page >= p.num_pages) {
               report_status(p.status, NF_ST_BAD_INDEX);
@@ -321,7 +330,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const uint32_t t_lane = tmem + (static_cast<uint32_t>(warp * 32) << 16);
     __nv_bfloat16* outp = reinterpret_cast<__nv_bfloat16*>(p.out);
     // CAP: capped scores carry the scale themselves
-    const float scale = CAP ? 1.f : p.sm_scale * kLog2e;
+    const float scale = CAP || DIST ? 1.f : p.sm_scale * kLog2e;
     const float cap_in = CAP ? p.sm_scale / p.softcap : 0.f, cap_out = CAP ? p.softcap * kLog2e : 0.f;
     uint32_t g = 0, n_item = 0;
     bool ok = true;
@@ -331,6 +340,9 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       const int tl = row / group, hh = row % group;
       const bool row_valid = tl < it.ntok;
       const int pos = row_valid ? it.kv_len - (it.q_end - (it.tok0 + tl)) : -1;
+      const int chunk_lo = EXT && p.chunk > 0 && row_valid ? pos / p.chunk * p.chunk : 0;
+      float2 far = make_float2(0.f, 0.f);
+      if (DIST && row_valid) far = reinterpret_cast<const float2*>(p.dist)[it.kvh * group + hh];
       float m_ref = -INFINITY, l = 0.f;
       for (int t = 0; t < it.n_tiles; ++t) {
         const uint32_t gt = g + t;
@@ -349,6 +361,15 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           }
         }
         const int cbase = (it.t_first + t) * kTile;
+        if (DIST) {
+          const float in = p.sm_scale * kLog2e, d0 = static_cast<float>(pos - cbase);
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {                      // (keys behind the row are masked below)
+            const float a = __log2f(fmaf(far.y, d0 - j, 1.f)), b = __log2f(fmaf(far.y, d0 - (32 + j), 1.f));
+            r0[j] = __float_as_uint(fmaf(__uint_as_float(r0[j]), in, -far.x * a));
+            r1[j] = __float_as_uint(fmaf(__uint_as_float(r1[j]), in, -far.x * b));
+          }
+        }
         if (cbase + kTile - 1 > pos) {                        // only tiles on the diagonal need the mask
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
@@ -362,6 +383,13 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           for (int j = 0; j < 32; ++j) {
             if (cbase + j < lo) r0[j] = 0xff800000u;
             if (cbase + 32 + j < lo) r1[j] = 0xff800000u;
+          }
+        }
+        if (EXT && cbase < chunk_lo) {                          // tiles that start before the row's chunk
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            if (cbase + j < chunk_lo) r0[j] = 0xff800000u;
+            if (cbase + 32 + j < chunk_lo) r1[j] = 0xff800000u;
           }
         }
         float mxp = -INFINITY;
@@ -467,13 +495,13 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   }
 }
 
-template <int HD, bool EXT, bool CAP>
+template <int HD, bool EXT, bool CAP, bool DIST = false>
 int launch_ws(const nfk_attn_params& p, const CUtensorMap& tmQ, const CUtensorMap& tmKV, cudaStream_t stream) {
   constexpr int bytes = WsCfg<HD>::kSmemBytes;
   static bool attr_dev[kMaxDevices] = {false};   // the attribute is per device
   bool& attr = attr_dev[device_slot()];
   if (!attr) {
-    if (cudaFuncSetAttribute(attn_prefill_ws_kernel<HD, EXT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) !=
+    if (cudaFuncSetAttribute(attn_prefill_ws_kernel<HD, EXT, CAP, DIST>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) !=
         cudaSuccess)
       return NF_ERR_CUDA;
     attr = true;
@@ -481,7 +509,7 @@ int launch_ws(const nfk_attn_params& p, const CUtensorMap& tmQ, const CUtensorMa
   const long long total = static_cast<long long>(p.num_items) * p.kv_heads;
   long long ctas = p.num_ctas > 0 ? p.num_ctas : 2LL * device_sm_count();   // two resident CTAs per SM
   if (ctas > total) ctas = total;
-  attn_prefill_ws_kernel<HD, EXT, CAP><<<static_cast<int>(ctas), kThreads, bytes, stream>>>(tmQ, tmKV, p);
+  attn_prefill_ws_kernel<HD, EXT, CAP, DIST><<<static_cast<int>(ctas), kThreads, bytes, stream>>>(tmQ, tmKV, p);
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
 }
 
@@ -496,9 +524,11 @@ extern "C" int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream
   if (p->kv_heads <= 0 || p->q_heads % p->kv_heads != 0 || p->num_pages <= 0) return NF_ERR_BAD_ARG;
   const int group = p->q_heads / p->kv_heads;
   // `precise` and the extensions run in the EXT instantiations, capped scores and head_dim 64 in one of their own
-  const bool cap = p->softcap > 0.f;
+  const bool cap = p->softcap > 0.f, dist = p->dist != nullptr;
   const bool ext = p->window > 0 || p->sinks != nullptr || p->kv_ld > 0 || p->q_rows > 0 || cap || p->precise != 0;
-  if (p->page_size != kPage || p->softcap < 0.f) return NF_ERR_UNSUPPORTED;
+  if (p->page_size != kPage || p->softcap < 0.f || (cap && dist)) return NF_ERR_UNSUPPORTED;
+  if (p->chunk < 0 || (p->chunk > 0 && p->window > 0)) return NF_ERR_BAD_ARG;
+  if ((dist || p->chunk > 0 || p->kv_first != nullptr) && p->precise == 0) return NF_ERR_UNSUPPORTED;
   if (p->head_dim != 128 && !(p->head_dim == 64 && ext)) return NF_ERR_UNSUPPORTED;
   if (ext ? group > 128 : (group > 16 || (16 % group) != 0)) return NF_ERR_UNSUPPORTED;
   const uint64_t HD = static_cast<uint64_t>(p->head_dim);
@@ -510,6 +540,8 @@ extern "C" int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream
   // With q_rows the queries are [q_rows][q_heads * 128] and a box is 128 tokens of one head; with kv_ld the
   // keys and values are columns of [num_pages * 16][kv_ld] rows.
   if (p->window < 0 || (p->q_rows > 0 && group != 1)) return NF_ERR_BAD_ARG;
+  if (p->q_rows == 0 && p->ld_q != 0 && (p->precise == 0 || p->ld_q % p->head_dim != 0 || p->ld_q < p->q_heads * p->head_dim))
+    return NF_ERR_BAD_ARG;
   if (p->kv_ld > 0 && (p->kv_ld % 8 != 0 || p->k_col < 0 || p->v_col < 0 || p->k_col % 8 != 0 || p->v_col % 8 != 0))
     return NF_ERR_BAD_ARG;
   CUtensorMap tmQ, tmKV;
@@ -520,6 +552,7 @@ extern "C" int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream
   rc = p->kv_ld > 0 ? make_tmap_bf16_2d(&tmKV, p->kv_pool, static_cast<uint64_t>(p->num_pages) * kPage, p->kv_ld, p->kv_ld, kPage, 64)
                     : make_tmap_bf16_2d(&tmKV, p->kv_pool, static_cast<uint64_t>(p->num_pages) * 2 * p->kv_heads * kPage, HD, HD, kPage, 64);
   if (rc != NF_OK) return rc;
+  if (dist) return p->head_dim == 64 ? launch_ws<64, true, false, true>(*p, tmQ, tmKV, stream) : launch_ws<128, true, false, true>(*p, tmQ, tmKV, stream);
   if (p->head_dim == 64) return cap ? launch_ws<64, true, true>(*p, tmQ, tmKV, stream) : launch_ws<64, true, false>(*p, tmQ, tmKV, stream);
   if (cap) return launch_ws<128, true, true>(*p, tmQ, tmKV, stream);
   return ext ? launch_ws<128, true, false>(*p, tmQ, tmKV, stream) : launch_ws<128, false, false>(*p, tmQ, tmKV, stream);

@@ -26,6 +26,10 @@ __device__ __forceinline__ float gated_act(float g, float u, const GatedAct& a) 
 __device__ __forceinline__ float lin_act_of(float v, int kind) {
   if (kind == NFK_LIN_TANH) return tanhf(v);
   if (kind == NFK_LIN_GELU) return 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
+  if (kind == NFK_LIN_RELU2) {
+    const float r = fmaxf(v, 0.f);
+    return r * r;
+  }
   return v;
 }
 

@@ -129,6 +129,7 @@ struct DevParams {
   __nv_bfloat16* D;
   const __nv_bfloat16* C;
   const __nv_bfloat16* bias;
+  const __nv_bfloat16* bias2;       // of the up half (gated epilogue)
   float* partial;   // split-K: fp32 [split_k][M][N] partial sums (second pass reduces them)
   long long ldd, ldc;
   float beta;
@@ -184,6 +185,18 @@ __device__ __forceinline__ NBlock n_block(const DevParams& p, int n_blk, int out
     b.col_end = min((g + 1) * p.group_n, b.col0 + out_bn);
   }
   return b;
+}
+
+// v += the bias of eight columns.
+__device__ __forceinline__ void add_bias8(float* v, const __nv_bfloat16* bias) {
+  const uint4 bv = *reinterpret_cast<const uint4*>(bias);
+  const uint32_t bw[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 f = unpack_bf16x2(bw[j]);
+    v[2 * j] += f.x;
+    v[2 * j + 1] += f.y;
+  }
 }
 
 // Eight finished columns of one row: bf16 to D, or fp32 to D32 from f32_col0 on (a multiple of 8).
@@ -629,6 +642,16 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 }
                 continue;
               }
+              if (p.bias != nullptr) {
+#pragma unroll
+                for (int g8 = 0; g8 < 4; ++g8) {
+                  const int col = nb.col0 + c * 32 + g8 * 8;
+                  if (col < tile_col_end) {
+                    add_bias8(gsum + g8 * 8, p.bias + col);
+                    add_bias8(usum + g8 * 8, p.bias2 + col);
+                  }
+                }
+              }
 #pragma unroll
               for (int j = 0; j < 32; ++j) v[j] = gated_act(gsum[j], usum[j], p.act);
             } else {
@@ -729,16 +752,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 if (col < tile_col_end) {  // N is a multiple of 8
                   float* vv = v + g8 * 8;
                   if (EPI == 0) {
-                    if (p.bias != nullptr) {
-                      const uint4 bv = *reinterpret_cast<const uint4*>(p.bias + col);
-                      const uint32_t bw[4] = {bv.x, bv.y, bv.z, bv.w};
-#pragma unroll
-                      for (int j = 0; j < 4; ++j) {
-                        const float2 f = unpack_bf16x2(bw[j]);
-                        vv[2 * j] += f.x;
-                        vv[2 * j + 1] += f.y;
-                      }
-                    }
+                    if (p.bias != nullptr) add_bias8(vv, p.bias + col);
                     if (crow != nullptr) {
                       const uint4 cv = *reinterpret_cast<const uint4*>(crow + col);
                       const uint32_t cw[4] = {cv.x, cv.y, cv.z, cv.w};
@@ -829,16 +843,7 @@ splitk_reduce_kernel(DevParams p) {
       v[0] += a.x; v[1] += a.y; v[2] += a.z; v[3] += a.w;
       v[4] += b.x; v[5] += b.y; v[6] += b.z; v[7] += b.w;
     }
-    if (p.bias != nullptr) {
-      const uint4 bv = *reinterpret_cast<const uint4*>(p.bias + col);
-      const uint32_t bw[4] = {bv.x, bv.y, bv.z, bv.w};
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float2 f = unpack_bf16x2(bw[j]);
-        v[2 * j] += f.x;
-        v[2 * j + 1] += f.y;
-      }
-    }
+    if (p.bias != nullptr) add_bias8(v, p.bias + col);
     if (p.C != nullptr) {
       const uint4 cv = *reinterpret_cast<const uint4*>(p.C + static_cast<long long>(row) * p.ldc + col);
       const uint32_t cw[4] = {cv.x, cv.y, cv.z, cv.w};
@@ -878,16 +883,7 @@ splitk_reduce_norm_kernel(DevParams p) {
           v[i][0] += a.x; v[i][1] += a.y; v[i][2] += a.z; v[i][3] += a.w;
           v[i][4] += b.x; v[i][5] += b.y; v[i][6] += b.z; v[i][7] += b.w;
         }
-        if (p.bias != nullptr) {
-          const uint4 bv = *reinterpret_cast<const uint4*>(p.bias + col);
-          const uint32_t bw[4] = {bv.x, bv.y, bv.z, bv.w};
-#pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const float2 f = unpack_bf16x2(bw[j]);
-            v[i][2 * j] += f.x;
-            v[i][2 * j + 1] += f.y;
-          }
-        }
+        if (p.bias != nullptr) add_bias8(v[i], p.bias + col);
         if (p.C != nullptr) {
           const uint4 cv = *reinterpret_cast<const uint4*>(p.C + static_cast<long long>(row) * p.ldc + col);
           const uint32_t cw[4] = {cv.x, cv.y, cv.z, cv.w};
@@ -992,19 +988,14 @@ sk_fixup_kernel(DevParams p, FixupGeom f) {
       }
     }
     if (EPI == 1) {
+      if (p.bias != nullptr) {
+        add_bias8(a, p.bias + col);
+        add_bias8(u, p.bias2 + col);
+      }
 #pragma unroll
       for (int j = 0; j < 8; ++j) a[j] = gated_act(a[j], u[j], p.act);
     } else {
-      if (p.bias != nullptr) {
-        const uint4 bv = *reinterpret_cast<const uint4*>(p.bias + col);
-        const uint32_t bw[4] = {bv.x, bv.y, bv.z, bv.w};
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const float2 fl = unpack_bf16x2(bw[j]);
-          a[2 * j] += fl.x;
-          a[2 * j + 1] += fl.y;
-        }
-      }
+      if (p.bias != nullptr) add_bias8(a, p.bias + col);
       if (p.C != nullptr) {
         const uint4 cv = *reinterpret_cast<const uint4*>(p.C + static_cast<long long>(row) * p.ldc + col);
         const uint32_t cw[4] = {cv.x, cv.y, cv.z, cv.w};
@@ -1133,6 +1124,7 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
   p.D = reinterpret_cast<__nv_bfloat16*>(g.D);
   p.C = reinterpret_cast<const __nv_bfloat16*>(g.C);
   p.bias = reinterpret_cast<const __nv_bfloat16*>(g.bias);
+  p.bias2 = reinterpret_cast<const __nv_bfloat16*>(g.bias2);
   p.partial = split_k > 1 ? reinterpret_cast<float*>(g.workspace) : nullptr;
   p.sk_partial = sk.q > 0 ? reinterpret_cast<float*>(g.workspace) : nullptr;
   p.sk_tiles_dp = sk.tiles_dp;
@@ -1433,7 +1425,7 @@ extern "C" int nfk_gemm_bf16(const nfk_gemm_params* g, cudaStream_t stream) {
       (g->epilogue != NFK_EPI_LINEAR || g->f32_col0 < 0 || g->f32_col0 % 8 != 0 || g->ld32 % 4 != 0 ||
        (reinterpret_cast<uintptr_t>(g->D32) & 15) != 0 || g->norm_w != nullptr))
     return NF_ERR_BAD_ARG;
-  if (g->act < NFK_ACT_SILU || g->act > NFK_ACT_CAPPED || g->lin_act < NFK_LIN_NONE || g->lin_act > NFK_LIN_GELU) return NF_ERR_BAD_ARG;
+  if (g->act < NFK_ACT_SILU || g->act > NFK_ACT_CAPPED || g->lin_act < NFK_LIN_NONE || g->lin_act > NFK_LIN_RELU2) return NF_ERR_BAD_ARG;
   if (g->groups > 1 && (g->epilogue != NFK_EPI_LINEAR || g->N % (8 * g->groups) != 0 || g->group_k % 8 != 0 ||
                         g->group_k < 0 || g->gate_flags != nullptr))
     return NF_ERR_BAD_ARG;
@@ -1445,7 +1437,7 @@ extern "C" int nfk_gemm_bf16(const nfk_gemm_params* g, cudaStream_t stream) {
     return NF_ERR_BAD_ARG;
   if (g->workspace != nullptr && (reinterpret_cast<uintptr_t>(g->workspace) & 15) != 0) return NF_ERR_BAD_ARG;
   const bool swiglu = g->epilogue == NFK_EPI_SWIGLU;
-  if (swiglu && g->B2 == nullptr) return NF_ERR_BAD_ARG;
+  if (swiglu && (g->B2 == nullptr || (g->bias == nullptr) != (g->bias2 == nullptr))) return NF_ERR_BAD_ARG;
   const bool rs = g->epilogue == NFK_EPI_REDUCE_SCATTER;
   if (g->gate_flags != nullptr &&
       (rs || g->gate_nranks < 1 || g->gate_nranks > 8 || (reinterpret_cast<uintptr_t>(g->gate_flags) & 3) != 0))

@@ -58,6 +58,7 @@ gemm_f32_kernel(nfk_gemm_params p, int groups, int group_n) {
   float* D32 = reinterpret_cast<float*>(p.D32);
   const float* C = reinterpret_cast<const float*>(p.C);
   const float* bias = reinterpret_cast<const float*>(p.bias);
+  const float* bias2 = reinterpret_cast<const float*>(p.bias2);
   const GatedAct act{p.act, p.act_limit, p.act_alpha, p.act_shift};
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -69,7 +70,8 @@ gemm_f32_kernel(nfk_gemm_params p, int groups, int group_n) {
       if (col >= col_end) continue;
       float v = acc[i][j];
       if (GATED) {
-        v = gated_act_of<true>(v, up[i][j], act);
+        const float u = up[i][j];
+        v = bias != nullptr ? gated_act_of<true>(v + bias[col], u + bias2[col], act) : gated_act_of<true>(v, u, act);
       } else {
         if (bias != nullptr) v += bias[col];
         if (C != nullptr) v += p.beta * C[static_cast<long long>(row) * p.ldc + col];
@@ -91,7 +93,7 @@ extern "C" int nfk_gemm_f32(const nfk_gemm_params* p, cudaStream_t stream) {
   const int groups = p->groups > 1 ? p->groups : 1;
   if (!p->A || !p->B || p->M < 0 || p->N < 0 || p->K <= 0 || p->N % groups != 0 || p->group_k < 0) return NF_ERR_BAD_ARG;
   if (!p->D && !(p->D32 && p->f32_col0 == 0)) return NF_ERR_BAD_ARG;
-  if (p->epilogue == NFK_EPI_SWIGLU && (!p->B2 || groups > 1 || p->D32)) return NF_ERR_BAD_ARG;
+  if (p->epilogue == NFK_EPI_SWIGLU && (!p->B2 || groups > 1 || p->D32 || (p->bias == nullptr) != (p->bias2 == nullptr))) return NF_ERR_BAD_ARG;
   if (p->epilogue != NFK_EPI_LINEAR && p->epilogue != NFK_EPI_SWIGLU) return NF_ERR_UNSUPPORTED;
   if (p->norm_w || p->gate_flags) return NF_ERR_UNSUPPORTED;
   const int group_n = p->N / groups;

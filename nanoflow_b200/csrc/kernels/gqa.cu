@@ -2,8 +2,8 @@
 //
 // nfk_gqa_append   per token: RMS norm over the whole query row and the whole key row (all heads at once), rotation,
 //                  keys and values to their page slot, values optionally mixed with those of an earlier layer.
-// nfk_gqa_attn     attention for any head size, bf16 or fp32, with window, sink and capped scores: one CTA per token
-//                  and query head. 32-bit engines use it for everything, bf16 engines for heads that the tensor-core
+// nfk_gqa_attn     attention for any head size, bf16 or fp32, with window, chunks, distance bias, sink and capped
+//                  scores: one CTA per token and query head. 32-bit engines use it for everything, bf16 engines for heads that the tensor-core
 //                  kernels (nfk_attn_decode, nfk_attn_prefill_ws) are not built for.
 #include "elem_io.cuh"
 
@@ -59,8 +59,8 @@ gqa_append_kernel(nfk_gqa_append_params p) {
     }
     const float* rot = p.rot != nullptr ? p.rot + static_cast<long long>(t) * p.rot_ld * 2 : nullptr;
     const float* v_rot = p.v_rot != nullptr ? p.v_rot + static_cast<long long>(t) * p.v_ld * 2 : nullptr;
-    T* qo = reinterpret_cast<T*>(p.q_out) + static_cast<long long>(t) * nq;
-    for (int c = threadIdx.x * 4; c < nq; c += kApThreads * 4) {
+    T* qo = p.q_out != nullptr ? reinterpret_cast<T*>(p.q_out) + static_cast<long long>(t) * nq : nullptr;
+    for (int c = threadIdx.x * 4; c < nq && qo != nullptr; c += kApThreads * 4) {
       float4 x = load4(q + c);
       if (p.q_w != nullptr) {
         const float4 w = load4(p.q_w + c);
@@ -110,13 +110,14 @@ gqa_attn_kernel(nfk_gqa_attn_params p) {
   const int pos = p.positions[tok], req = p.token_req[tok];
   const T* pool = reinterpret_cast<const T*>(p.pool);
   const long long v_step = static_cast<long long>(p.kv_heads) * p.page_size * hd;
-  const T* q = reinterpret_cast<const T*>(p.q) + (static_cast<long long>(tok) * p.heads + head) * hd;
+  const T* q = reinterpret_cast<const T*>(p.q) + static_cast<long long>(tok) * (p.ld_q > 0 ? p.ld_q : p.heads * hd) + head * hd;
+  const float far_a = p.dist != nullptr ? p.dist[2 * head] : 0.f, far_b = p.dist != nullptr ? p.dist[2 * head + 1] : 0.f;
   for (int c = threadIdx.x; c < hd; c += kGaThreads) q_s[c] = to_f32(q[c]);
   float acc[kGaCols];
 #pragma unroll
   for (int i = 0; i < kGaCols; ++i) acc[i] = 0.f;
   float m = p.sinks != nullptr ? p.sinks[head] : -INFINITY, l = p.sinks != nullptr ? 1.f : 0.f;
-  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int lo = max(p.window > 0 ? max(0, pos - p.window + 1) : 0, p.chunk > 0 ? pos / p.chunk * p.chunk : 0);
   for (int j0 = lo; j0 <= pos; j0 += kGaTile) {
     const int n = min(kGaTile, pos + 1 - j0);
     __syncthreads();
@@ -137,6 +138,7 @@ gqa_attn_kernel(nfk_gqa_attn_params p) {
       }
       d = warp_sum(d) * p.scale;
       if (p.softcap > 0.f) d = p.softcap * tanhf(d / p.softcap);
+      if (p.dist != nullptr) d -= far_a * logf(fmaf(far_b, static_cast<float>(pos - j0 - k), 1.f));
       if (lane == 0) s_s[k] = row_s[k] >= 0 ? d : -INFINITY;
     }
     __syncthreads();
@@ -176,11 +178,12 @@ extern "C" int nfk_gqa_append(const nfk_gqa_append_params* p, cudaStream_t strea
   using namespace nf;
   if (p == nullptr) return NF_ERR_BAD_ARG;
   if (p->T == 0) return NF_OK;
-  if (!p->src || !p->q_out || !p->pool || !p->positions || !p->token_req || !p->kv_indptr || !p->kv_indices || p->T < 0 ||
+  if (!p->src || !p->pool || !p->positions || !p->token_req || !p->kv_indptr || !p->kv_indices || p->T < 0 ||
       p->heads <= 0 || p->kv_heads <= 0 || p->hd <= 0 || p->hd % 8 != 0 || p->dim <= 0 || p->dim > p->hd ||
       p->page_size <= 0 || p->num_pages <= 0)
     return NF_ERR_BAD_ARG;
   if (p->ld_src % 8 != 0 || p->q_off % 8 != 0 || p->k_off % 8 != 0 || p->v_off % 8 != 0) return NF_ERR_BAD_ARG;
+  if (!p->q_out && (p->q_w || p->rot)) return NF_ERR_BAD_ARG;
   if ((p->q_w == nullptr) != (p->k_w == nullptr) || p->v_mode < 0 || p->v_mode > 2 || (p->v_mode != 0 && !p->v_first))
     return NF_ERR_BAD_ARG;
   if ((p->rot && (p->rot_pairs < 0 || p->rot_pairs > p->hd / 2 || p->rot_ld < p->rot_pairs || p->rot_ld % 2 != 0)) ||
@@ -199,7 +202,8 @@ extern "C" int nfk_gqa_attn(const nfk_gqa_attn_params* p, cudaStream_t stream) {
   if (p->n_tokens == 0) return NF_OK;
   if (!p->q || !p->pool || !p->out || !p->positions || !p->token_req || !p->kv_indptr || !p->kv_indices || p->n_tokens < 0 ||
       p->token_begin < 0 || p->heads <= 0 || p->kv_heads <= 0 || p->heads % p->kv_heads != 0 || p->hd <= 0 || p->hd % 8 != 0 ||
-      p->page_size <= 0 || p->num_pages <= 0 || p->window < 0)
+      p->page_size <= 0 || p->num_pages <= 0 || p->window < 0 || p->chunk < 0 ||
+      (p->ld_q > 0 && (p->ld_q % 4 != 0 || p->ld_q < p->heads * p->hd)))
     return NF_ERR_BAD_ARG;
   if (p->hd > kGaThreads * kGaCols) return NF_ERR_UNSUPPORTED;
   const long long grid = static_cast<long long>(p->n_tokens) * p->heads;

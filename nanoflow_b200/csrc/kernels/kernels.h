@@ -17,7 +17,8 @@ enum { NFK_EPI_LINEAR = 0, NFK_EPI_SWIGLU = 1, NFK_EPI_REDUCE_SCATTER = 2 };
 // Gated epilogue: act(gate) * up, or for NFK_ACT_CAPPED g sigmoid(alpha g) (u + shift) with g = min(gate, limit) and
 // u = min(max(up, -limit), limit).
 enum { NFK_ACT_SILU = 0, NFK_ACT_RELU = 1, NFK_ACT_GELU_TANH = 2, NFK_ACT_CAPPED = 3 };
-enum { NFK_LIN_NONE = 0, NFK_LIN_TANH = 1, NFK_LIN_GELU = 2 };         // activation of the linear epilogue (GELU: by erf)
+// activation of the linear epilogue (GELU: by erf; RELU2: the square of relu)
+enum { NFK_LIN_NONE = 0, NFK_LIN_TANH = 1, NFK_LIN_GELU = 2, NFK_LIN_RELU2 = 3 };
 enum { NFK_BF16 = 0, NFK_F32 = 1 };                                    // storage type of activations and weights
 
 typedef struct nfk_gemm_params {
@@ -85,6 +86,7 @@ typedef struct nfk_gemm_params {
   int groups, group_k;
   int lin_act;          // linear epilogue: NFK_LIN_*, applied to the finished columns
   float act_limit, act_alpha, act_shift;   // constants of NFK_ACT_CAPPED
+  const void* bias2;    // gated epilogue: [N] bf16 bias of the up half (`bias` is the gate half's), null = none
 } nfk_gemm_params;
 
 int nfk_gemm_bf16(const nfk_gemm_params* p, cudaStream_t stream);
@@ -211,6 +213,11 @@ typedef struct nfk_attn_params {
   // nfk_attn_decode and nfk_attn_prefill_ws (head_dim 64 or 128):
   float softcap;           // > 0: score <- softcap tanh(score / softcap) before the softmax
   int precise;             // 1: probabilities enter the second product as a bf16 pair (implied by the other extensions)
+  // nfk_attn_decode and nfk_attn_prefill_ws, together with `precise`. ld_q (elements from token to token of q, a multiple of
+  // head_dim) also holds for these.
+  const int* kv_first;     // [B] page slot of the sequence that a request's page list starts with; null = 0
+  const float* dist;       // [q_heads][2] (a, b): score <- score - a ln(1 + b (i - j)); null = none
+  int chunk;               // > 0: position i sees j only if i / chunk = j / chunk
 } nfk_attn_params;
 int nfk_attn_decode(const nfk_attn_params* p, cudaStream_t stream);
 // The same with the pages copied by a TMA producer warp into a ring of decode_stages (2, 3 or 4) pages per
@@ -227,10 +234,13 @@ int nfk_attn_prefill_ws(const nfk_attn_params* p, cudaStream_t stream);
 // ------------------------------------------------------------------------------------------------
 // Layer-list models: residual step, latent attention, mLSTM (residual_norm.cu, latent.cu, mlstm.cu)
 // ------------------------------------------------------------------------------------------------
-enum { NFK_NORM_NONE = 0, NFK_NORM_RMS = 1, NFK_NORM_LAYER = 2 };
+enum { NFK_NORM_NONE = 0, NFK_NORM_RMS = 1, NFK_NORM_LAYER = 2, NFK_NORM_SCALE = 3 };   // SCALE: only times the weights
 // x <- (table ? 0 : x) + norm_in(src_scale src) (+ y2_gate y2) (+ sum_k e_weight e_out[e_slot]) (+ add);  h = norm_out(x).
 // norm_sum: norm_in takes in y2 and the experts' rows too. pair_w: the source is half the sum of RMS norms of y (times
 // pair_w) and y2 (times pair_w2). table_add: x <- x + ... + src_scale (embedding row), which is then not a source.
+// pos_freq: a sinusoidal position vector joins the embedding row, entry 2i sin(p f_i), entry 2i + 1 cos(p f_i).
+// hist: earlier versions of the stream. The sum goes to hist_out; with hist_w, x <- hist_w[hist_n] (sum) + sum_j hist_w[j]
+// hist[j] is what goes on.
 // Rows of x, y, table and h are padded to a multiple of 4 elements; weight vectors are padded with zeros to that length.
 typedef struct nfk_residual_norm_params {
   float* x;                  // [*, ld_x] residual stream
@@ -263,7 +273,7 @@ typedef struct nfk_residual_norm_params {
   const float* y2_gate;      // [*] factor per row of y2, null: 1
   const void* e_out;         // [e_rows, ld_e] outputs of a mixture of experts, null: none
   long long ld_e;
-  const int* e_slot;         // [*][e_top] rows of e_out of a token
+  const int* e_slot;         // [*][e_top] rows of e_out of a token, -1: none
   const float* e_weight;     // [*][e_top]
   int e_top, e_rows;
   int norm_sum;
@@ -278,6 +288,12 @@ typedef struct nfk_residual_norm_params {
   const int* state_slot;
   const int* positions;
   int conv_taps, conv_rows, conv_ld, num_slots;
+  const float* pos_freq;     // [(cols + 1) / 2][2]: f_i as the sum of two floats, null: none; needs positions
+  const float* hist;         // [hist_n][*, ld_x], hist_stride elements apart
+  const float* hist_w;       // [hist_n + 1], null: none
+  float* hist_out;           // [*, ld_x], null: none
+  long long hist_stride;
+  int hist_n;
 } nfk_residual_norm_params;
 int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t stream);
 
@@ -410,7 +426,7 @@ typedef struct nfk_gqa_append_params {
   const void* src;           // [T, ld_src]: q at q_off, k at k_off, v at v_off, head h at column h * hd
   long long ld_src;
   int q_off, k_off, v_off;
-  void* q_out;               // [T, heads * hd]
+  void* q_out;               // [T, heads * hd], null: queries are left where they are (no norm, no rotation)
   const float* q_w;          // [heads * hd] norm weights, null: no norm
   const float* k_w;          // [kv_heads * hd]
   void* v_first;             // [T, kv_heads * hd]
@@ -448,6 +464,9 @@ typedef struct nfk_gqa_attn_params {
   float scale, softcap;      // softcap 0: none
   int dtype;
   unsigned int* status;
+  const float* dist;         // as in nfk_attn_params
+  int chunk;
+  int ld_q;                  // elements from token to token of q; 0 = heads * hd
 } nfk_gqa_attn_params;
 int nfk_gqa_attn(const nfk_gqa_attn_params* p, cudaStream_t stream);
 
@@ -596,7 +615,11 @@ int nfk_delta_prefill(const nfk_delta_params* p, cudaStream_t stream);
 // ------------------------------------------------------------------------------------------------
 // Mixture of experts (moe.cu)
 // ------------------------------------------------------------------------------------------------
-enum { NFK_SCORE_SIGMOID = 0, NFK_SCORE_SOFTMAX = 1 };
+enum { NFK_SCORE_SIGMOID = 0, NFK_SCORE_SOFTMAX = 1, NFK_SCORE_SOFTMAX_ALL = 2 };
+// NFK_SCORE_SOFTMAX_ALL: scores s = softmax(logits) over all outputs, choice scores s + correction, weights s times scale (not
+// normed). `identity`: so many outputs behind the experts stand for the input itself: they take part in scores, groups and
+// choice, but get no row; the sum of a token's weights of such choices goes to gate. group_max: a group counts by its
+// largest choice score instead of the sum of the two largest.
 // NFK_SCORE_SOFTMAX: the experts are chosen by logits + correction and weighted by the softmax of those sums over the
 // chosen ones, times scale (groups as below). NFK_SCORE_SIGMOID:
 // Scores s = sigmoid(logits); choice scores s + correction. Experts form `groups` equal runs of neighbours (1: no
@@ -615,10 +638,12 @@ typedef struct nfk_moe_route_params {
   int T, experts, top, groups, keep, gate_col;
   float scale;
   int score;                 // NFK_SCORE_*
+  int identity, group_max;   // identity > 0: no gate column
 } nfk_moe_route_params;
 int nfk_moe_route(const nfk_moe_route_params* p, cudaStream_t stream);
 
-// Rows of h in expert order: row rank + (rows of the experts before) of out for every chosen expert of a token.
+// Rows of h in expert order: row rank + (rows of the experts before) of out for every chosen expert of a token. Choices past the
+// experts get no row and slot -1.
 typedef struct nfk_moe_permute_params {
   const void* h;             // [T, ld_h]
   long long ld_h;

@@ -36,16 +36,25 @@ __global__ void __launch_bounds__(kRouteWarps * 32)
 moe_route_kernel(nfk_moe_route_params p) {
   extern __shared__ float rsm[];                       // per warp: scores | choice scores | group scores
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int E = p.experts, per = E / p.groups;
+  const int E = p.experts + p.identity, per = E / p.groups;
   float* s_s = rsm + warp * (2 * E + p.groups);
   float* c_s = s_s + E;
   float* g_s = c_s + E;
-  const bool softmax = p.score == NFK_SCORE_SOFTMAX;
+  const bool softmax = p.score == NFK_SCORE_SOFTMAX, whole = p.score == NFK_SCORE_SOFTMAX_ALL;
   for (int t = blockIdx.x * kRouteWarps + warp; t < p.T; t += gridDim.x * kRouteWarps) {
     const float* z = p.logits + t * p.ld;
+    float z_max = -INFINITY, inv = 0.f;
+    if (whole) {
+      for (int e = lane; e < E; e += 32) z_max = fmaxf(z_max, z[e]);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) z_max = fmaxf(z_max, __shfl_xor_sync(0xffffffffu, z_max, o));
+      float all = 0.f;
+      for (int e = lane; e < E; e += 32) all += expf(z[e] - z_max);
+      inv = 1.f / warp_sum(all);
+    }
     for (int e = lane; e < E; e += 32) {
       const float corr = p.correction != nullptr ? p.correction[e] : 0.f;
-      const float s = softmax ? z[e] + corr : 1.f / (1.f + expf(-z[e]));
+      const float s = softmax ? z[e] + corr : whole ? expf(z[e] - z_max) * inv : 1.f / (1.f + expf(-z[e]));
       s_s[e] = s;
       c_s[e] = softmax ? s : s + corr;
     }
@@ -63,7 +72,7 @@ moe_route_kernel(nfk_moe_route_params p) {
             b = c;
           }
         }
-        g_s[g] = per > 1 ? a + b : a;
+        g_s[g] = per > 1 && p.group_max == 0 ? a + b : a;
       }
       __syncwarp();
       // a group stays if fewer than `keep` groups come before it
@@ -99,14 +108,18 @@ moe_route_kernel(nfk_moe_route_params p) {
       const float top = __shfl_sync(0xffffffffu, share, 0);        // the first one chosen has the largest logit
       share = mine >= 0 ? expf(share - top) : 0.f;
       share /= warp_sum(share);
-    } else {
+    } else if (!whole) {
       share /= sum + 1e-20f;
     }
     if (lane < p.top) {
       const long long o = static_cast<long long>(t) * p.top + lane;
       p.expert[o] = mine;
       p.weight[o] = share * p.scale;
-      p.rank[o] = atomicAdd(p.counts + mine, 1);
+      p.rank[o] = mine < p.experts ? atomicAdd(p.counts + mine, 1) : 0;
+    }
+    if (p.identity > 0) {
+      const float kept = warp_sum(lane < p.top && mine >= p.experts ? share * p.scale : 0.f);
+      if (lane == 0) p.gate[t] = kept;
     }
     __syncwarp();
   }
@@ -154,7 +167,8 @@ moe_permute_kernel(nfk_moe_permute_params p, int row_chunks) {
     int slot = 0;
     if (lane < p.top) {
       const long long o = static_cast<long long>(t) * p.top + lane;
-      slot = off[p.expert[o]] + p.rank[o];
+      const int e = p.expert[o];
+      slot = e < p.experts ? off[e] + p.rank[o] : -1;
       p.slot[o] = slot;
     }
     const uint4* src = reinterpret_cast<const uint4*>(p.h) + t * ld_h;
@@ -167,6 +181,7 @@ moe_permute_kernel(nfk_moe_permute_params p, int row_chunks) {
         if (c + j * 32 < row_chunks) v[j] = src[c + j * 32];
       for (int k = 0; k < p.top; ++k) {
         const long long s = __shfl_sync(0xffffffffu, slot, k);
+        if (s < 0) continue;
 #pragma unroll
         for (int j = 0; j < 4; ++j)
           if (c + j * 32 < row_chunks) out[s * ld_o + c + j * 32] = v[j];
@@ -499,11 +514,12 @@ extern "C" int nfk_moe_route(const nfk_moe_route_params* p, cudaStream_t stream)
   if (p == nullptr) return NF_ERR_BAD_ARG;
   if (p->T == 0) return NF_OK;
   if (!p->logits || !p->expert || !p->weight || !p->rank || !p->counts || p->T < 0 || p->experts <= 0 ||
-      p->experts > kMaxExperts || p->groups <= 0 || p->experts % p->groups != 0 || p->keep <= 0 || p->keep > p->groups ||
-      p->top <= 0 || p->top > 32 || p->top > p->keep * (p->experts / p->groups) || (p->gate_col >= 0 && !p->gate) ||
-      p->score < NFK_SCORE_SIGMOID || p->score > NFK_SCORE_SOFTMAX)
+      p->identity < 0 || p->experts + p->identity > kMaxExperts || p->groups <= 0 || (p->experts + p->identity) % p->groups != 0 ||
+      p->keep <= 0 || p->keep > p->groups || p->top <= 0 || p->top > 32 ||
+      p->top > p->keep * ((p->experts + p->identity) / p->groups) || ((p->gate_col >= 0 || p->identity > 0) && !p->gate) ||
+      (p->gate_col >= 0 && p->identity > 0) || p->score < NFK_SCORE_SIGMOID || p->score > NFK_SCORE_SOFTMAX_ALL)
     return NF_ERR_BAD_ARG;
-  const size_t sm = static_cast<size_t>(kRouteWarps) * (2 * p->experts + p->groups) * 4;
+  const size_t sm = static_cast<size_t>(kRouteWarps) * (2 * (p->experts + p->identity) + p->groups) * 4;
   if (sm > 48 * 1024) return NF_ERR_UNSUPPORTED;
   int grid = (p->T + kRouteWarps - 1) / kRouteWarps;
   if (grid > 16 * device_sm_count()) grid = 16 * device_sm_count();
@@ -531,7 +547,7 @@ extern "C" int nfk_moe_gemm(const nfk_moe_gemm_params* p, cudaStream_t stream) {
   if (p->rows == 0) return NF_OK;
   if (!p->A || !p->B || !p->D || !p->counts || p->rows < 0 || p->experts <= 0 || p->experts > kMaxExperts || p->N <= 0 ||
       p->K <= 0 || p->N % 8 != 0 || p->K % 8 != 0 || p->lda % 8 != 0 || p->ldb % 8 != 0 || p->ldd % 8 != 0 ||
-      p->act < NFK_ACT_SILU || p->act > NFK_ACT_CAPPED || p->lin_act < NFK_LIN_NONE || p->lin_act > NFK_LIN_GELU || (reinterpret_cast<uintptr_t>(p->D) & 15) != 0)
+      p->act < NFK_ACT_SILU || p->act > NFK_ACT_CAPPED || p->lin_act < NFK_LIN_NONE || p->lin_act > NFK_LIN_RELU2 || (reinterpret_cast<uintptr_t>(p->D) & 15) != 0)
     return NF_ERR_BAD_ARG;
   if (p->dtype == NFK_F32) {
     const long long m_tiles = p->rows / kFt + (p->rows < p->experts ? p->rows : p->experts);

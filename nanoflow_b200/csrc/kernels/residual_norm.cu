@@ -4,7 +4,8 @@
 //   x <- (table ? 0 : x) + norm_in(src) (+ second output) (+ weighted expert outputs) (+ add);   h = norm_out(x)
 //
 // The norm can also be taken of the whole sum, the source can be the mean of two normed outputs, and the embedding row
-// can join a stream that goes on (see kernels.h). Where the next sublayer reads its input through a convolution over time,
+// can join a stream that goes on (see kernels.h). A position vector can join the embedding row, the "norm" of the source can
+// be a mere scale per column, and what goes on can be a weighted sum of the result and of earlier results. Where the next sublayer reads its input through a convolution over time,
 // rows that are the only token of their request get it here, from the request's state.
 // `src` is the sublayer's output row, or the embedding row of the token (ids as in nfk_embedding, with the
 // previous iteration's tokens fed back on the device). Norms are RMS or layer norms with fp32 weights. The
@@ -35,6 +36,16 @@ template <int NV>
 __device__ __forceinline__ void norm_row(float4 (&v)[NV], int kind, const float* w, const float* b, int cols, int nvec,
                                          float eps, float* red) {
   if (kind == NFK_NORM_NONE) return;
+  if (kind == NFK_NORM_SCALE) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int vi = threadIdx.x + i * kRnThreads;
+      if (vi >= nvec) continue;
+      const float4 ww = load4(w + vi * 4);            // zero past `cols`
+      v[i] = make_float4(v[i].x * ww.x, v[i].y * ww.y, v[i].z * ww.z, v[i].w * ww.w);
+    }
+    return;
+  }
   const float inv_n = 1.f / static_cast<float>(cols);
   float mean = 0.f;
   if (kind == NFK_NORM_LAYER) {
@@ -112,8 +123,42 @@ __device__ __forceinline__ void input_conv(const float4 (&v)[NV], const nfk_resi
   }
 }
 
-// CONV: some rows go through the input convolution.
-template <class T, int NV, bool CONV>
+// sin and cos of pos * (hi + lo), the rounding of the product included.
+__device__ __forceinline__ float2 sin_cos(float pos, float2 f) {
+  const float a = pos * f.x, e = fmaf(pos, f.x, -a) + pos * f.y;
+  float s, c;
+  sincosf(a, &s, &c);
+  return make_float2(fmaf(e, c, s), fmaf(-e, s, c));
+}
+
+// v (the sum of the row) is kept as a result of its own, and replaced by the weighted sum of all results so far.
+template <int NV>
+__device__ __forceinline__ void depth_average(float4 (&v)[NV], const nfk_residual_norm_params& p, long long row_off, int nvec) {
+  if (p.hist_out != nullptr) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int vi = threadIdx.x + i * kRnThreads;
+      if (vi < nvec) store4(p.hist_out + row_off + vi * 4, v[i]);
+    }
+  }
+  if (p.hist_w == nullptr) return;
+  const float own = p.hist_w[p.hist_n];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) v[i] = make_float4(own * v[i].x, own * v[i].y, own * v[i].z, own * v[i].w);
+  const float* src = p.hist + row_off;
+#pragma unroll 4
+  for (int j = 0; j < p.hist_n; ++j, src += p.hist_stride) {
+    const float f = p.hist_w[j];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int vi = threadIdx.x + i * kRnThreads;
+      if (vi < nvec) fma4(v[i], f, load4(src + vi * 4));
+    }
+  }
+}
+
+// CONV: some rows go through the input convolution. DEEP: position vectors and earlier results.
+template <class T, int NV, bool CONV, bool DEEP>
 __global__ void __launch_bounds__(kRnThreads)
 residual_norm_kernel(nfk_residual_norm_params p) {
   __shared__ float red[kRnThreads / 32];
@@ -156,6 +201,20 @@ residual_norm_kernel(nfk_residual_norm_params p) {
         v[i].x *= p.src_scale; v[i].y *= p.src_scale; v[i].z *= p.src_scale; v[i].w *= p.src_scale;
       }
     }
+    if (DEEP && p.pos_freq != nullptr) {
+      const float pos = static_cast<float>(p.positions[row]);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int vi = threadIdx.x + i * kRnThreads;
+        if (vi >= nvec) continue;
+        const int c = vi * 4;
+        const float2* f = reinterpret_cast<const float2*>(p.pos_freq) + vi * 2;
+        const float2 a = sin_cos(pos, f[0]), b = c + 2 < p.cols ? sin_cos(pos, f[1]) : make_float2(0.f, 0.f);
+        v[i].x += a.x; v[i].z += b.x;
+        if (c + 1 < p.cols) v[i].y += a.y;
+        if (c + 3 < p.cols) v[i].w += b.y;
+      }
+    }
     if (p.pair_w != nullptr) {
       const T* y2 = reinterpret_cast<const T*>(p.y2) + static_cast<long long>(src_row) * p.ld_y2;
       float4 o[NV];
@@ -185,7 +244,7 @@ residual_norm_kernel(nfk_residual_norm_params p) {
         const int slot = p.e_slot[static_cast<long long>(src_row) * p.e_top + k];
         const float f = p.e_weight[static_cast<long long>(src_row) * p.e_top + k];
         if (slot < 0 || slot >= p.e_rows) {
-          if (threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
+          if (slot != -1 && threadIdx.x == 0) report_status(p.status, NF_ST_BAD_INDEX);
           continue;
         }
         const T* e = reinterpret_cast<const T*>(p.e_out) + static_cast<long long>(slot) * p.ld_e;
@@ -216,7 +275,15 @@ residual_norm_kernel(nfk_residual_norm_params p) {
           const float4 a = load4(p.add + vi * 4);
           v[i].x += a.x; v[i].y += a.y; v[i].z += a.z; v[i].w += a.w;
         }
-        if (p.rows_idx == nullptr) store4(xr + vi * 4, v[i]);
+        if (!DEEP && p.rows_idx == nullptr) store4(xr + vi * 4, v[i]);
+      }
+    }
+    if (DEEP) {
+      depth_average<NV>(v, p, static_cast<long long>(src_row) * p.ld_x, nvec);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int vi = threadIdx.x + i * kRnThreads;
+        if (vi < nvec && p.rows_idx == nullptr) store4(xr + vi * 4, v[i]);
       }
     }
     if (p.h != nullptr) {
@@ -235,18 +302,25 @@ residual_norm_kernel(nfk_residual_norm_params p) {
   }
 }
 
-template <class T, bool CONV>
+template <class T, bool CONV, bool DEEP>
 int launch_rn(const nfk_residual_norm_params& p, cudaStream_t stream) {
   const int nvec = (p.cols + 3) / 4, per = (nvec + kRnThreads - 1) / kRnThreads;
   const int cap = device_sm_count() * 16;
   const int grid = p.rows < cap ? p.rows : cap;
-  if (per <= 1) residual_norm_kernel<T, 1, CONV><<<grid, kRnThreads, 0, stream>>>(p);
-  else if (per <= 2) residual_norm_kernel<T, 2, CONV><<<grid, kRnThreads, 0, stream>>>(p);
-  else if (per <= 4) residual_norm_kernel<T, 4, CONV><<<grid, kRnThreads, 0, stream>>>(p);
-  else if (per <= 8) residual_norm_kernel<T, 8, CONV><<<grid, kRnThreads, 0, stream>>>(p);
-  else if (per <= 16) residual_norm_kernel<T, 16, CONV><<<grid, kRnThreads, 0, stream>>>(p);
+  if (per <= 1) residual_norm_kernel<T, 1, CONV, DEEP><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 2) residual_norm_kernel<T, 2, CONV, DEEP><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 4) residual_norm_kernel<T, 4, CONV, DEEP><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 8) residual_norm_kernel<T, 8, CONV, DEEP><<<grid, kRnThreads, 0, stream>>>(p);
+  else if (per <= 16) residual_norm_kernel<T, 16, CONV, DEEP><<<grid, kRnThreads, 0, stream>>>(p);
   else return NF_ERR_UNSUPPORTED;
   return cudaGetLastError() == cudaSuccess ? NF_OK : NF_ERR_CUDA;
+}
+
+template <class T>
+int launch_rn_form(const nfk_residual_norm_params& p, cudaStream_t stream) {
+  const bool deep = p.pos_freq != nullptr || p.hist_w != nullptr || p.hist_out != nullptr;
+  if (p.conv_w != nullptr && p.conv_rows > 0) return deep ? launch_rn<T, true, true>(p, stream) : launch_rn<T, true, false>(p, stream);
+  return deep ? launch_rn<T, false, true>(p, stream) : launch_rn<T, false, false>(p, stream);
 }
 
 }  // namespace
@@ -269,10 +343,11 @@ extern "C" int nfk_residual_norm(const nfk_residual_norm_params* p, cudaStream_t
   if (p->pair_w && (!p->pair_w2 || !p->y || !p->y2)) return NF_ERR_BAD_ARG;
   if (p->norm_sum && p->in_kind != NFK_NORM_NONE && !p->in_w) return NF_ERR_BAD_ARG;
   for (int kind : {p->in_kind, p->out_kind})
-    if (kind != NFK_NORM_NONE && kind != NFK_NORM_RMS && kind != NFK_NORM_LAYER) return NF_ERR_BAD_ARG;
+    if (kind < NFK_NORM_NONE || kind > NFK_NORM_SCALE) return NF_ERR_BAD_ARG;
   if ((p->table || p->y) && p->in_kind != NFK_NORM_NONE && !p->in_w) return NF_ERR_BAD_ARG;
   if (p->h && p->out_kind != NFK_NORM_NONE && !p->out_w) return NF_ERR_BAD_ARG;
-  if (p->conv_w && p->conv_rows > 0)
-    return p->dtype == NFK_F32 ? launch_rn<float, true>(*p, stream) : launch_rn<__nv_bfloat16, true>(*p, stream);
-  return p->dtype == NFK_F32 ? launch_rn<float, false>(*p, stream) : launch_rn<__nv_bfloat16, false>(*p, stream);
+  if (p->pos_freq && (!p->table || p->table_add || !p->positions)) return NF_ERR_BAD_ARG;
+  if (p->hist_w && (p->hist_n < 0 || (p->hist_n > 0 && !p->hist))) return NF_ERR_BAD_ARG;
+  if (p->hist_out && p->rows_idx) return NF_ERR_BAD_ARG;
+  return p->dtype == NFK_F32 ? launch_rn_form<float>(*p, stream) : launch_rn_form<__nv_bfloat16>(*p, stream);
 }

@@ -77,14 +77,14 @@ def make_plan(engine, spans, pages: int):
     m = engine.model
     pool = DistKVPool(m.run_layers, m.num_kv_heads, m.head_dim, pages, 16, 1)
     slots = StateSlotPool(len(spans)) if getattr(m, "has_state", False) else None
-    window = getattr(m, "kv_window", 0)
+    first_seen = getattr(m, "first_seen", None)
     parts = []
     for ctx, n in spans:
         kv = DistKVCache(pool, slots)
         if ctx:
             kv.allocate_tokens(ctx)
-        if window:
-            kv.trim(ctx - window + 1)
+        if first_seen is not None:
+            kv.trim(first_seen(ctx))
         kv.allocate_tokens(n)
         parts.append(Portion(kv, np.random.default_rng(len(parts)).integers(0, m.vocab_size, n), [n - 1]))
     return plan_portions(parts, tile_tokens=max(1, 128 // m.group_size))

@@ -2,10 +2,12 @@
 
 A layer is a mixer (one of the registered kinds below, with its own sizes, or two of them side by side) and optionally
 a feed-forward (gated, or a mixture of experts), one after the other or side by side on one normed input; what a
-sublayer reads may first pass a short convolution over time. A contiguous range of layers may run several times in a row
+sublayer reads may first pass a short convolution over time, and what goes on to the next layer may be a weighted sum of
+all results so far. A contiguous range of layers may run several times in a row
 with the same weights, each pass with a cache or state of its own. :class:`LayerListConfig` plays the part
 :class:`~..config.ModelConfig` plays for the Llama family; :class:`LayerListWeights` that of ``RankWeights``. Designs map
-their ``config.json`` and tensor names onto these (``models/volarax.py``, ``models/zubedra.py``, ``models/gupizen.py``).
+their ``config.json`` and tensor names onto these (``models/volarax.py``, ``models/zubedra.py``, ``models/gupizen.py``,
+``models/gimudra.py``).
 
 Kernel layout of the weights: every matrix ``[N, K]`` with both sizes padded with zeros to multiples of 8
 (per head where a matrix is per head), projections of one input packed into one matrix, norm weights,
@@ -27,7 +29,7 @@ WKV_CHUNK_DIM = 128           # largest head size of the chunked WKV kernels
 DELTA_CHUNK_DIM = 128         # ... and of the chunked delta-rule kernels
 PAGE = 16                     # tokens per cache page
 MOE_MAX_EXPERTS, MOE_MAX_TOP = 1024, 32
-LINEAR_ACTS = ("gelu",)       # activations of products without a gate
+LINEAR_ACTS = ("gelu", "relu2")     # activations of products without a gate
 CONV_MAX_TAPS = 8             # taps of the short convolution kernel
 LATENT_LDS = (64, 128, 192, 256, 384, 512)   # row sizes the tensor-core latent attention kernel is built for
 
@@ -104,7 +106,10 @@ class RotarySpec:
 class AttentionSpec:
     """Grouped-query attention, with options: RMS norm over whole query and key rows, rotary positions, a sliding window,
     capped scores, a sink per head. ``value_mix``: values are mixed with those of the first layer that has it set.
-    ``talk``: the heads' softmax weights are mixed by a matrix before they meet the values."""
+    ``talk``: the heads' softmax weights are mixed by a matrix before they meet the values. ``bias``: the projections of
+    queries, keys and values have biases. ``distance_bias``: scores lose a ln(1 + b distance), two numbers per head.
+    ``chunk``: positions see only those of their own run of so many. ``kv_from``: the layer whose cached keys and values
+    are used instead of own ones."""
     heads: int
     kv_heads: int
     dim: int
@@ -117,6 +122,10 @@ class AttentionSpec:
     rotary: Optional[RotarySpec] = None
     window: Optional[int] = None
     talk: bool = False
+    bias: bool = False
+    distance_bias: bool = False
+    chunk: Optional[int] = None
+    kv_from: Optional[int] = None
     kind = "attention"
 
     @property
@@ -142,9 +151,31 @@ class AttentionSpec:
                 _positive(where, factor=s.factor, low=s.low, original=s.original, high_over_low=s.high - s.low)
         if self.talk and (self.softcap is not None or self.value_mix):
             raise ValueError(f"{where}: capped scores and mixed values are not built for mixed heads")
+        if self.chunk is not None:
+            _positive(where, chunk=self.chunk)
+        if self.distance_bias and self.softcap is not None:
+            raise ValueError(f"{where}: capped scores with a distance bias are not built")
+        if self.chunk is not None and self.window is not None:
+            raise ValueError(f"{where}: chunks with a window are not built")
+        if self.talk and (self.distance_bias or self.chunk is not None):
+            raise ValueError(f"{where}: distance biases and chunks are not built for mixed heads")
+        if self.kv_from is not None and (self.qk_norm or self.rotary is not None or self.value_mix or self.talk):
+            raise ValueError(f"{where}: another layer's keys and values are not built with norms, rotations, mixed values or heads")
+
+    def first_seen(self, position: int) -> int:
+        """The first position that a token sees."""
+        if self.window is not None:
+            return max(0, position - self.window + 1)
+        return position // self.chunk * self.chunk if self.chunk is not None else 0
+
+    @property
+    def proj_heads(self) -> int:
+        """Heads that the input projection forms."""
+        return self.heads + (2 * self.kv_heads if self.kv_from is None else 0)
 
     def matrix_params(self, w: int) -> int:
-        return w * (self.heads * (self.dim + self.vdim) + self.kv_heads * (self.dim + self.vdim))
+        own = self.kv_heads * (self.dim + self.vdim) if self.kv_from is None else 0
+        return w * (self.heads * (self.dim + self.vdim) + own)
 
 
 @dataclass(frozen=True)
@@ -278,10 +309,11 @@ class ActSpec:
 
 @dataclass(frozen=True)
 class MlpSpec:
-    """``gated``: act(gate) * up; else act(up)."""
+    """``gated``: act(gate) * up; else act(up). ``bias``: all projections have biases."""
     ff: int
     act: ActSpec
     gated: bool = True
+    bias: bool = False
     kind = "dense"
 
     def check(self, where: str) -> None:
@@ -296,9 +328,11 @@ class MlpSpec:
 @dataclass(frozen=True)
 class MoeSpec:
     """Mixture of experts, of which a token uses ``top``. ``score`` "sigmoid": sigmoid scores, a correction added for the
-    choice, the chosen scores normed and times ``scale``; "softmax": softmax over the chosen logits times ``scale``.
-    Experts in ``groups`` of which only the best ``keep`` can be chosen. ``shared``: an expert that runs for every token,
-    times a sigmoid gate of its own."""
+    choice, the chosen scores normed and times ``scale``; "softmax": softmax over the chosen logits times ``scale``;
+    "softmax_all": softmax over all logits, a correction added for the choice, the chosen scores times ``scale``.
+    Experts in ``groups`` of which only the best ``keep`` can be chosen; a group counts by its two largest choice scores or
+    (``group_score`` "max") its largest. ``shared``: an expert that runs for every token, times a sigmoid gate of its own.
+    ``identity``: so many router outputs behind the experts' stand for the input itself."""
     expert: MlpSpec
     experts: int
     top: int
@@ -307,29 +341,42 @@ class MoeSpec:
     keep: int = 1
     shared: Optional[MlpSpec] = None
     score: str = "sigmoid"
+    identity: int = 0
+    group_score: str = "top2"
     kind = "moe"
+
+    @property
+    def outputs(self) -> int:
+        """Experts to choose from, those that only hand on the input included."""
+        return self.experts + self.identity
 
     def check(self, where: str) -> None:
         _positive(where, experts=self.experts, top=self.top, groups=self.groups, keep=self.keep)
         self.expert.check(where)
         if self.shared is not None:
             self.shared.check(where + " (shared expert)")
-        if self.experts % self.groups or self.keep > self.groups:
-            raise ValueError(f"{where}: {self.experts} experts do not form {self.groups} groups of which {self.keep} are kept")
-        if self.top > self.keep * (self.experts // self.groups):
+        if self.identity < 0 or (self.identity and self.shared is not None):
+            raise ValueError(f"{where}: identity experts beside a shared expert are not built")
+        if self.group_score not in ("top2", "max"):
+            raise ValueError(f"{where}: unknown group score '{self.group_score}'")
+        if self.expert.bias or (self.shared is not None and self.shared.bias):
+            raise ValueError(f"{where}: experts with biases are not built")
+        if self.outputs % self.groups or self.keep > self.groups:
+            raise ValueError(f"{where}: {self.outputs} experts do not form {self.groups} groups of which {self.keep} are kept")
+        if self.top > self.keep * (self.outputs // self.groups):
             raise ValueError(f"{where}: {self.top} experts per token cannot be chosen from {self.keep} groups")
-        if self.score not in ("sigmoid", "softmax"):
+        if self.score not in ("sigmoid", "softmax", "softmax_all"):
             raise ValueError(f"{where}: unknown router score '{self.score}'")
         if self.expert.gated == (self.expert.act.name in LINEAR_ACTS):
             raise ValueError(f"{where}: activation '{self.expert.act.name}' is not built for this kind of expert")
         if self.shared is not None and not self.shared.gated:
             raise ValueError(f"{where}: a shared expert without a gate product is not built")
-        if self.experts > MOE_MAX_EXPERTS or self.top > MOE_MAX_TOP:
+        if self.outputs > MOE_MAX_EXPERTS or self.top > MOE_MAX_TOP:
             raise ValueError(f"{where}: at most {MOE_MAX_EXPERTS} experts and {MOE_MAX_TOP} per token are built")
 
     @property
     def router_cols(self) -> int:
-        return self.experts + (1 if self.shared is not None else 0)
+        return self.outputs + (1 if self.shared is not None else 0)
 
     def matrix_params(self, w: int) -> int:
         return w * self.router_cols + self.experts * self.expert.matrix_params(w) + \
@@ -368,6 +415,10 @@ class LayerListConfig:
     embed_scale: float = 1.0
     logit_scale: float = 1.0            # folded into the final norm's weight
     input_conv: int = 0                 # taps of the convolution over time that a sublayer's input passes (0: none)
+    input_conv_mlp: bool = True         # ... a feed-forward's too
+    sinusoid: float = 0.0               # base of the sinusoidal position vector that joins the embedding row (0: none)
+    layer_scale: bool = False           # every sublayer's output is scaled per column before it joins the stream
+    depth_average: bool = False         # a weighted sum of the embedding output and all layers' results goes on
     tied_head: bool = False             # the embedding table is the output matrix
     loop: Optional[Tuple[int, int, int]] = None      # (start, stop, times)
     loop_add: str = "steps"             # what joins the stream ahead of a pass: a vector per pass, or "embedding": what the
@@ -398,12 +449,27 @@ class LayerListConfig:
             raise ValueError(f"at most {CONV_MAX_TAPS} taps of the input convolution are built, not {self.input_conv}")
         if self.input_conv and self.parallel:
             raise ValueError("input convolutions are not built for parallel layers")
+        if self.layer_scale and (self.parallel or self.output_norms):
+            raise ValueError("scaled sublayer outputs are not built for parallel layers or normed outputs")
+        if self.depth_average and self.loop is not None:
+            raise ValueError("averages over depth are not built for loops")
+        if self.sinusoid and (self.sinusoid < 0 or self.embed_norm or (self.loop is not None and self.loop_add == "embedding")):
+            raise ValueError("position vectors need a positive base, and are not built with normed or repeated embeddings")
         for i, lay in enumerate(self.layers):
             lay.mixer.check(f"layer {i}")
             if lay.mixer.kind == "pair" and (self.parallel or not self.output_norms or self.norm_kind != "rms"):
                 raise ValueError(f"layer {i}: mixers side by side need RMS norms of sublayer outputs")
             if lay.mlp is not None:
                 lay.mlp.check(f"layer {i}")
+            src = getattr(lay.mixer, "kv_from", None)
+            if src is not None:
+                s = self.layers[src].mixer if 0 <= src < i else None
+                if s is None or s.kind != "attention" or s.kv_from is not None:
+                    raise ValueError(f"layer {i}: layer {src} has no keys and values to lend")
+                if (s.kv_heads, s.dim, s.vdim) != (lay.mixer.kv_heads, lay.mixer.dim, lay.mixer.vdim):
+                    raise ValueError(f"layer {i}: the keys and values of layer {src} have other sizes")
+                if self.loop is not None:
+                    raise ValueError(f"layer {i}: lent keys and values are not built for loops")
         mixed = {(l.mixer.kv_heads, l.mixer.vdim) for l in self.layers if getattr(l.mixer, "value_mix", False)}
         if len(mixed) > 1:
             raise ValueError(f"layers that mix values need the same key/value heads and value size, not {sorted(mixed)}")
@@ -457,6 +523,12 @@ class LayerListConfig:
             return 0
         return max(s.window for s in specs)
 
+    def first_seen(self, position: int) -> int:
+        """The first position that any layer sees from ``position``; tokens after it see none before."""
+        latent, attn = self.run_specs("latent_attention"), self.run_specs("attention")
+        firsts = [0 if s.window is None else max(0, position - s.window + 1) for s in latent] + [s.first_seen(position) for s in attn]
+        return min(firsts, default=0)
+
     @property
     def has_state(self) -> bool:
         return any(self.run_specs(kind) for kind in ("mlstm", "wkv", "rglru", "delta")) or self.input_conv > 1
@@ -504,14 +576,15 @@ class LayerListConfig:
 
     def kv_bytes_per_token_local(self, dtype_bytes: int = 0) -> int:
         elems = sum(self.latent_ld(s) for s in self.run_specs("latent_attention")) + \
-            sum(2 * s.kv_heads * self.attn_hd(s) for s in self.run_specs("attention"))
+            sum(2 * s.kv_heads * self.attn_hd(s) for s in self.run_specs("attention") if s.kv_from is None)
         return elems * (dtype_bytes or self.elem_bytes)
 
     def pool_shape(self, spec) -> Optional[Tuple[int, ...]]:
         """Shape of one page of a mixer's cache (None: it keeps none)."""
         if spec.kind == "latent_attention":
             return (PAGE, self.latent_ld(spec))
-        return (2, spec.kv_heads, PAGE, self.attn_hd(spec)) if spec.kind == "attention" else None
+        own = spec.kind == "attention" and spec.kv_from is None
+        return (2, spec.kv_heads, PAGE, self.attn_hd(spec)) if own else None
 
     def state_shapes(self, spec) -> List[Tuple[Tuple[int, ...], torch.dtype]]:
         """What a request keeps of a recurrent mixer, as (shape, type) without the leading slots. Small vectors come in two
@@ -535,6 +608,10 @@ class LayerListConfig:
         """The last inputs of a sublayer's input convolution, in two halves."""
         return (2, max(1, self.input_conv - 1), self.width_p)
 
+    def conv_mlp(self, layer: LayerSpec) -> bool:
+        """Whether a layer's feed-forward reads through an input convolution."""
+        return bool(self.input_conv) and self.input_conv_mlp and layer.mlp is not None
+
     def state_bytes_per_slot(self) -> int:
         n = 0
         for r in self.runs:
@@ -542,7 +619,7 @@ class LayerListConfig:
             for s in parts_of(lay.mixer):
                 n += sum(math.prod(shape) * (4 if dt == torch.float32 else 2) for shape, dt in self.state_shapes(s))
             if self.input_conv:
-                n += (1 if lay.mlp is None else 2) * math.prod(self.conv_state_shape()) * self.elem_bytes
+                n += (2 if self.conv_mlp(lay) else 1) * math.prod(self.conv_state_shape()) * self.elem_bytes
         return n
 
     def param_count(self) -> int:
@@ -563,6 +640,7 @@ class LayerListConfig:
 class NormWeights:
     w: torch.Tensor                      # fp32, padded with zeros
     b: Optional[torch.Tensor] = None
+    kind: Optional[str] = None           # other than the model's: "scale" only multiplies by the weights
 
 
 @dataclass
@@ -587,13 +665,15 @@ class MlstmWeights:
 
 @dataclass
 class AttentionWeights:
-    w_in: torch.Tensor                   # queries | keys | values, per head padded
+    w_in: torch.Tensor                   # queries | keys | values, per head padded (queries only with lent keys and values)
     q_norm: Optional[torch.Tensor]       # fp32 [heads * hd]
     k_norm: Optional[torch.Tensor]       # fp32 [kv_heads * hd]
     w_o: torch.Tensor
     sinks: Optional[torch.Tensor]        # fp32 [heads]
     value_lambda: float
     talk: Optional[torch.Tensor] = None  # fp32 [heads, heads]
+    b_in: Optional[torch.Tensor] = None  # bias of w_in
+    dist: Optional[torch.Tensor] = None  # fp32 [heads, 2]: factor and rate of the distance bias
 
 
 @dataclass
@@ -648,12 +728,15 @@ class MlpWeights:
     w_gate: torch.Tensor
     w_up: torch.Tensor
     w_down: torch.Tensor
+    b_gate: Optional[torch.Tensor] = None
+    b_up: Optional[torch.Tensor] = None
+    b_down: Optional[torch.Tensor] = None
 
 
 @dataclass
 class MoeWeights:
-    router: torch.Tensor                 # experts | gate of the shared expert, rows padded to a multiple of 8
-    correction: Optional[torch.Tensor]   # fp32 [experts]: added for the choice, or to the logits of a softmax router
+    router: torch.Tensor                 # experts | identity experts | gate of the shared expert, rows padded to a multiple of 8
+    correction: Optional[torch.Tensor]   # fp32 [experts | identity experts]: added for the choice, or to the logits of a softmax router
     w_gate: Optional[torch.Tensor]       # [experts * ff_p, width_p], None in experts without a gate product
     w_up: torch.Tensor
     w_down: torch.Tensor                 # [experts * width_p, ff_p]
@@ -670,6 +753,7 @@ class LayerListLayer:
     mlp: Any = None
     conv_in: Optional[torch.Tensor] = None       # fp32 [taps, width_p]: input convolutions of the two sublayers
     conv_mlp: Optional[torch.Tensor] = None
+    depth: Optional[torch.Tensor] = None         # fp32: weights of the embedding output and all results up to this layer's
 
 
 @dataclass
@@ -744,17 +828,23 @@ def pack_mlstm(cfg: LayerListConfig, spec: MlstmSpec, q, k, v, g, i, f, i_b, f_b
 
 
 def pack_attention(cfg: LayerListConfig, spec: AttentionSpec, q, k, v, q_norm, k_norm, sink, o, value_lambda: float,
-                   device, talk=None) -> AttentionWeights:
+                   device, talk=None, biases=None, dist=None) -> AttentionWeights:
+    """``k``, ``v`` None: lent by another layer. ``biases``: of queries, keys and values; ``dist`` [heads, 2]."""
     H, G, wp, hd = spec.heads, spec.kv_heads, cfg.width_p, cfg.attn_hd(spec)
     mv = lambda t: t.to(device=device, dtype=cfg.dtype).contiguous()
     f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
-    w_in = torch.cat([pad_heads(q, H, spec.dim, hd), pad_heads(k, G, spec.dim, hd), pad_heads(v, G, spec.vdim, hd)])
+    def rows(q, k, v):
+        parts = [pad_heads(q, H, spec.dim, hd)]
+        return torch.cat(parts if k is None else parts + [pad_heads(k, G, spec.dim, hd), pad_heads(v, G, spec.vdim, hd)])
+
+    w_in = rows(q, k, v)
     w_o = pad_to(o.reshape(-1, H, spec.vdim), wp, H, hd).reshape(wp, H * hd)
     return AttentionWeights(w_in=mv(pad_to(w_in, w_in.shape[0], wp)),
                             q_norm=None if q_norm is None else f32(pad_heads(q_norm, H, spec.dim, hd)),
                             k_norm=None if k_norm is None else f32(pad_heads(k_norm, G, spec.dim, hd)), w_o=mv(w_o),
                             sinks=None if sink is None else f32(sink), value_lambda=float(value_lambda),
-                            talk=None if talk is None else f32(talk))
+                            talk=None if talk is None else f32(talk), b_in=None if biases is None else mv(rows(*biases)),
+                            dist=None if dist is None else f32(dist))
 
 
 def pack_wkv(cfg: LayerListConfig, spec: WkvSpec, mu, r, k, v, g, w1, w2, w0, u, norm, o, device) -> WkvWeights:
@@ -817,10 +907,12 @@ def pack_pair(cfg: LayerListConfig, spec: PairSpec, left: AttentionWeights, righ
     return PairWeights(w_in=w_in, b_in=b_in, left=left, right=right, left_norm=f32(left_norm), right_norm=f32(right_norm))
 
 
-def pack_mlp(cfg: LayerListConfig, ff: int, gate, up, down, device) -> MlpWeights:
+def pack_mlp(cfg: LayerListConfig, ff: int, gate, up, down, device, biases=None) -> MlpWeights:
+    """``biases``: of the three products."""
     fp, wp = round8(ff), cfg.width_p
     mv = lambda t: t.to(device=device, dtype=cfg.dtype).contiguous()
-    return MlpWeights(mv(pad_to(gate, fp, wp)), mv(pad_to(up, fp, wp)), mv(pad_to(down, wp, fp)))
+    b = [None] * 3 if biases is None else [mv(pad_to(t, n)) for t, n in zip(biases, (fp, fp, wp))]
+    return MlpWeights(mv(pad_to(gate, fp, wp)), mv(pad_to(up, fp, wp)), mv(pad_to(down, wp, fp)), *b)
 
 
 def pack_moe(cfg: LayerListConfig, spec: MoeSpec, router, correction, expert, shared, shared_gate, device) -> MoeWeights:
@@ -843,6 +935,6 @@ def pack_moe(cfg: LayerListConfig, spec: MoeSpec, router, correction, expert, sh
         shared=None if spec.shared is None else pack_mlp(cfg, spec.shared.ff, *shared, device))
 
 
-def pack_norm(cfg: LayerListConfig, w, b, device) -> NormWeights:
+def pack_norm(cfg: LayerListConfig, w, b, device, kind: Optional[str] = None) -> NormWeights:
     f = lambda t: None if t is None else pad_to(t.to(device=device, dtype=torch.float32), cfg.width_p).contiguous()
-    return NormWeights(f(w), f(b))
+    return NormWeights(f(w), f(b), kind)

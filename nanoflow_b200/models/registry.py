@@ -82,8 +82,13 @@ def _gupizen() -> ModelFamily:
     return _layer_list("gupizen", gupizen)
 
 
+def _gimudra() -> ModelFamily:
+    from . import gimudra
+    return _layer_list("gimudra", gimudra)
+
+
 _FAMILIES: Dict[str, Callable[[], ModelFamily]] = {"llama": _llama, "volarax": _volarax, "zubedra": _zubedra,
-                                                    "gupizen": _gupizen}
+                                                    "gupizen": _gupizen, "gimudra": _gimudra}
 _cache: Dict[str, ModelFamily] = {}
 
 

@@ -44,7 +44,7 @@ class GemmParams(Structure):
                 ("rs_staged", c_int), ("gate_flags", c_void_p), ("gate_epoch", c_int), ("gate_nranks", c_int),
                 ("D32", c_void_p), ("ld32", c_longlong), ("f32_col0", c_int), ("act", c_int),
                 ("groups", c_int), ("group_k", c_int), ("lin_act", c_int),
-                ("act_limit", c_float), ("act_alpha", c_float), ("act_shift", c_float)]
+                ("act_limit", c_float), ("act_alpha", c_float), ("act_shift", c_float), ("bias2", c_void_p)]
 
 
 class RopeAppendParams(Structure):
@@ -72,15 +72,16 @@ class AttnParams(Structure):
                 ("chunk_pages", c_int), ("workspace", c_void_p), ("max_chunks", c_int),
                 ("items", c_void_p), ("num_items", c_int), ("status", c_void_p), ("decode_stages", c_int),
                 ("window", c_int), ("sinks", c_void_p), ("kv_ld", c_int), ("k_col", c_int), ("v_col", c_int),
-                ("q_rows", c_int), ("ld_q", c_int), ("softcap", c_float), ("precise", c_int)]
+                ("q_rows", c_int), ("ld_q", c_int), ("softcap", c_float), ("precise", c_int), ("kv_first", c_void_p),
+                ("dist", c_void_p), ("chunk", c_int)]
 
 
 BF16, F32 = 0, 1                                        # storage type of a kernel's activations and weights
 ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "capped": 3}   # activation of the gated GEMM epilogue
-LIN_ACTS = {None: 0, "tanh": 1, "gelu": 2}              # activation of the linear GEMM epilogue
+LIN_ACTS = {None: 0, "tanh": 1, "gelu": 2, "relu2": 3}              # activation of the linear GEMM epilogue
 CONV_ACTS = {None: 0, "silu": 1}                        # activation of the short convolution
-ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
-NORMS = {None: 0, "rms": 1, "layer": 2}
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1, "softmax_all": 2}
+NORMS = {None: 0, "rms": 1, "layer": 2, "scale": 3}
 
 
 def dtype_code(dtype: torch.dtype) -> int:
@@ -102,7 +103,8 @@ class ResidualNormParams(Structure):
                 ("e_slot", c_void_p), ("e_weight", c_void_p), ("e_top", c_int), ("e_rows", c_int), ("norm_sum", c_int),
                 ("pair_w", c_void_p), ("pair_w2", c_void_p), ("table_add", c_int), ("conv_w", c_void_p), ("conv_out", c_void_p),
                 ("conv_state", c_void_p), ("state_slot", c_void_p), ("positions", c_void_p), ("conv_taps", c_int),
-                ("conv_rows", c_int), ("conv_ld", c_int), ("num_slots", c_int)]
+                ("conv_rows", c_int), ("conv_ld", c_int), ("num_slots", c_int), ("pos_freq", c_void_p), ("hist", c_void_p),
+                ("hist_w", c_void_p), ("hist_out", c_void_p), ("hist_stride", c_longlong), ("hist_n", c_int)]
 
 
 class LatentAppendParams(Structure):
@@ -195,14 +197,14 @@ class GqaAttnParams(Structure):
                 ("kv_indptr", c_void_p), ("kv_indices", c_void_p), ("kv_first", c_void_p), ("sinks", c_void_p),
                 ("token_begin", c_int), ("n_tokens", c_int), ("heads", c_int), ("kv_heads", c_int), ("hd", c_int),
                 ("page_size", c_int), ("num_pages", c_int), ("window", c_int), ("scale", c_float), ("softcap", c_float),
-                ("dtype", c_int), ("status", c_void_p)]
+                ("dtype", c_int), ("status", c_void_p), ("dist", c_void_p), ("chunk", c_int), ("ld_q", c_int)]
 
 
 class MoeRouteParams(Structure):
     _fields_ = [("logits", c_void_p), ("ld", c_longlong), ("correction", c_void_p), ("expert", c_void_p),
                 ("weight", c_void_p), ("rank", c_void_p), ("counts", c_void_p), ("gate", c_void_p), ("T", c_int),
                 ("experts", c_int), ("top", c_int), ("groups", c_int), ("keep", c_int), ("gate_col", c_int),
-                ("scale", c_float), ("score", c_int)]
+                ("scale", c_float), ("score", c_int), ("identity", c_int), ("group_max", c_int)]
 
 
 class MoePermuteParams(Structure):

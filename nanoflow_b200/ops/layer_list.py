@@ -23,11 +23,11 @@ def _f32(t: Optional[torch.Tensor], name: str) -> None:
 
 def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None, up: Optional[torch.Tensor] = None,
          act: str = "silu", out32: Optional[torch.Tensor] = None, f32_col0: int = 0, groups: int = 1, group_k: int = 0,
-         k: int = 0, lin_act: Optional[str] = None, bias=None, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0,
+         k: int = 0, lin_act: Optional[str] = None, bias=None, up_bias=None, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0,
          workspace: Optional[torch.Tensor] = None, status=None, **shape) -> Optional[torch.Tensor]:
     """a @ w^T in the storage type of the operands (bf16: tensor cores, fp32: FMA). ``up``: act(a @ w^T) * (a @ up^T).
     ``out32``: columns from ``f32_col0`` on are written there as fp32. ``groups``: block-diagonal product. ``lin_act``:
-    activation of the finished columns; ``limit``, ``alpha``, ``shift``: constants of the "capped" gated form."""
+    activation of the finished columns; ``bias``, ``up_bias``: one per column; ``limit``, ``alpha``, ``shift``: constants of the "capped" gated form."""
     M, N, p = a.shape[0], w.shape[0], GemmParams()
     if a.dtype != w.dtype or a.stride(1) != 1 or w.stride(1) != 1:
         raise RuntimeError("gemm: operands of one type with unit inner stride expected")
@@ -39,6 +39,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
     p.M, p.N, p.K = M, N, k or w.shape[1]
     p.epilogue, p.act, p.groups, p.group_k = (1 if up is not None else 0), ACTS[act], groups, group_k
     p.lin_act, p.bias, p.act_limit, p.act_alpha, p.act_shift = LIN_ACTS[lin_act], _p(bias), limit, alpha, shift
+    p.bias2 = _p(up_bias)
     if out32 is not None:
         p.D32, p.ld32, p.f32_col0 = _p(out32), out32.stride(0), f32_col0
     if workspace is not None:
@@ -54,13 +55,25 @@ def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
 def residual_norm(x: torch.Tensor, *, y=None, table=None, ids=None, feedback_src=None, prev_tokens=None, norm_in=None,
                   add=None, h=None, norm_out=None, rows_idx=None, src_scale: float = 1.0, y2=None, y2_gate=None, experts=None,
                   cols: int, eps: float, rows: Optional[int] = None, norm_sum: bool = False, pair=None, table_add: bool = False,
-                  conv=None, status=None) -> None:
+                  conv=None, pos=None, history=None, status=None) -> None:
     """x <- (table ? 0 : x) + norm_in(src_scale * (y or table[ids])) (+ y2_gate y2) (+ weighted rows of ``experts``:
     outputs, slots, weights) (+ add); h <- norm_out(x). Norms: (kind, weight, bias). ``norm_sum``: norm_in of the whole
     sum; ``pair``: two RMS weights, the source is the mean of the normed y and y2; ``table_add``: the embedding row joins
     the stream instead of being the source; ``conv``: (weights [taps, ld], output, state, state references, positions,
-    rows): the input convolution of the first rows."""
+    rows): the input convolution of the first rows; ``pos``: (positions, frequencies [n, 2] as sums of two floats): the
+    sinusoidal vector that joins the embedding row; ``history``: (earlier results [n, rows, ld], weights [n + 1] or None,
+    where the sum goes or None): what goes on is the weighted sum of the results and this one."""
     p = ResidualNormParams()
+    if pos is not None:
+        _i32(pos[0], "positions"); _f32(pos[1], "frequencies")
+        p.positions, p.pos_freq = _p(pos[0]), _p(pos[1])
+    if history is not None:
+        hist, hw, hout = history
+        _f32(hist, "history"); _f32(hw, "history weights"); _f32(hout, "history output")
+        p.hist, p.hist_w, p.hist_out = _p(hist), _p(hw), _p(hout)
+        if hist is not None:
+            p.hist_n, p.hist_stride = hist.shape[0], hist.stride(0)
+            assert hist.stride(1) == x.stride(0)
     if conv is not None:
         w, out, state, ref, pos, n = conv
         _f32(w, "conv"); _i32(ref, "state references"); _i32(pos, "positions")
@@ -210,7 +223,7 @@ def gqa_append(src, q_out, pool, positions, token_req, kv_indptr, kv_indices, kv
                q_w=None, k_w=None, v_first=None, v_mode: int = 0, v_lambda: float = 0.0, eps: float, rot=None, v_rot=None,
                status=None) -> None:
     """src rows are q | k | v (heads padded to the pool's head size); normed keys and the values go to ``pool`` [pages, 2,
-    kv_heads, page size, head size], normed queries to ``q_out``. ``rot``, ``v_rot``: (table of angles [T, n, 2], pairs per
+    kv_heads, page size, head size], normed queries to ``q_out`` (None: they stay where they are). ``rot``, ``v_rot``: (table of angles [T, n, 2], pairs per
     head) for queries and keys, and for values."""
     for t, nm in ((q_w, "q_w"), (k_w, "k_w"), (rot and rot[0], "rot"), (v_rot and v_rot[0], "v_rot")):
         _f32(t, nm)
@@ -229,30 +242,32 @@ def gqa_append(src, q_out, pool, positions, token_req, kv_indptr, kv_indices, kv
 
 def gqa_attention(q, pool, out, positions, token_req, kv_indptr, kv_indices, kv_first=None, *, heads: int, scale: float,
                   softcap: float = 0.0, window: int = 0, sinks=None, token_begin: int = 0, n_tokens: Optional[int] = None,
-                  status=None) -> None:
+                  dist=None, chunk: int = 0, ld_q: int = 0, status=None) -> None:
     """The simple kernel: any head size, bf16 or fp32; q, out [T, heads * head size]."""
-    _f32(sinks, "sinks")
+    _f32(sinks, "sinks"); _f32(dist, "dist")
     n, _, G, ps, hd = pool.shape
     p = GqaAttnParams(q=_p(q), pool=_p(pool), out=_p(out), positions=_p(positions), token_req=_p(token_req),
                       kv_indptr=_p(kv_indptr), kv_indices=_p(kv_indices), kv_first=_p(kv_first), sinks=_p(sinks),
                       token_begin=token_begin, n_tokens=q.shape[0] - token_begin if n_tokens is None else n_tokens, heads=heads,
                       kv_heads=G, hd=hd, page_size=ps, num_pages=n, window=window, scale=scale, softcap=softcap,
-                      dtype=dtype_code(pool.dtype), status=_p(status))
+                      dtype=dtype_code(pool.dtype), status=_p(status), dist=_p(dist), chunk=chunk, ld_q=ld_q)
     _check(lib().nfk_gqa_attn(byref(p), _stream()), "nfk_gqa_attn")
 
 
 def paged_attention(q, pool, out, qo_indptr, kv_indptr, kv_indices, kv_last_page_len, *, heads: int, scale: float,
                     softcap: float = 0.0, sinks=None, items=None, req_count: int = 0, chunk_pages: int = 0,
-                    max_chunks: int = 1, workspace=None, status=None) -> None:
-    """The tensor-core kernels with capped scores, sinks and probabilities in two parts: portions (``items`` [n, 3]: request,
+                    max_chunks: int = 1, workspace=None, dist=None, chunk: int = 0, kv_first=None, ld_q: int = 0,
+                    status=None) -> None:
+    """The tensor-core kernels with capped scores, sinks, distance biases, chunks and probabilities in two parts: portions (``items`` [n, 3]: request,
     first token, tokens) on the prefill kernel, else single tokens of the first ``req_count`` requests."""
-    _f32(sinks, "sinks")
+    _f32(sinks, "sinks"); _f32(dist, "dist")
     p = AttnParams()
     p.q, p.out, p.kv_pool = _p(q), _p(out), _p(pool)
     p.qo_indptr, p.kv_indptr, p.kv_indices = _p(qo_indptr), _p(kv_indptr), _p(kv_indices)
     p.kv_last_page_len, p.q_heads, p.kv_heads = _p(kv_last_page_len), heads, pool.shape[2]
     p.head_dim, p.page_size, p.num_pages, p.sm_scale = pool.shape[4], pool.shape[3], pool.shape[0], scale
     p.softcap, p.sinks, p.precise, p.status = softcap, _p(sinks), 1, _p(status)
+    p.dist, p.chunk, p.kv_first, p.ld_q = _p(dist), chunk, _p(kv_first), ld_q
     if items is not None:
         p.items, p.num_items = _p(items), items.shape[0]
         _check(lib().nfk_attn_prefill_ws(byref(p), _stream()), "nfk_attn_prefill_ws")
@@ -341,15 +356,16 @@ def delta(qkv, x, beta, g, rate, dt_bias, norm, state, y, positions, qo_indptr, 
 
 
 def moe_route(logits, correction, counts, *, top: int, experts: int, groups: int = 1, keep: int = 1, scale: float,
-              gate_col: int = -1, score: str = "sigmoid"):
-    """(experts [T, top], weights, ranks, gate [T]); ``counts`` [experts] is increased."""
+              gate_col: int = -1, score: str = "sigmoid", identity: int = 0, group_max: bool = False):
+    """(experts [T, top], weights, ranks, gate [T]); ``counts`` [experts] is increased. ``identity``: outputs behind the
+    experts that stand for the input; gate is then the sum of their weights."""
     _f32(logits, "logits"); _f32(correction, "correction"); _i32(counts, "counts")
     T, dev = logits.shape[0], logits.device
     idx, rank = (torch.zeros(T, top, dtype=torch.int32, device=dev) for _ in range(2))
     weight, gate = torch.zeros(T, top, device=dev), torch.zeros(T, device=dev)
     p = MoeRouteParams(logits=_p(logits), ld=logits.stride(0), correction=_p(correction), expert=_p(idx), weight=_p(weight),
                        rank=_p(rank), counts=_p(counts), gate=_p(gate), T=T, experts=experts, top=top, groups=groups, keep=keep,
-                       gate_col=gate_col, scale=scale, score=ROUTER_SCORES[score])
+                       gate_col=gate_col, scale=scale, score=ROUTER_SCORES[score], identity=identity, group_max=int(group_max))
     _check(lib().nfk_moe_route(byref(p), _stream()), "nfk_moe_route")
     return idx, weight, rank, gate
 

@@ -145,8 +145,22 @@ def gated_act(g, u, act: str, limit=0.0, alpha=1.0, shift=0.0):
     return f(g) * u
 
 
-def gated_mlp(h, w_gate, w_up, w_down, act: str, **constants):
-    return gated_act(h.float() @ w_gate.float().t(), h.float() @ w_up.float().t(), act, **constants) @ w_down.float().t()
+def gated_mlp(h, w_gate, w_up, w_down, act: str, biases=(None, None, None), **constants):
+    g, u = h.float() @ w_gate.float().t(), h.float() @ w_up.float().t()
+    plus = lambda t, b: t if b is None else t + b.float()
+    return plus(gated_act(plus(g, biases[0]), plus(u, biases[1]), act, **constants) @ w_down.float().t(), biases[2])
+
+
+def linear_act(x, act: str):
+    """Activation of a product without a gate."""
+    return torch.nn.functional.gelu(x) if act == "gelu" else torch.relu(x) ** 2
+
+
+def sinusoid(positions, width, base):
+    """[T, width]: sine and cosine of position * base^(-2 i / width), next to each other."""
+    f = float(base) ** (-torch.arange(0, width, 2, dtype=torch.float64) / width)
+    a = torch.as_tensor(positions, dtype=torch.float64)[:, None] * f
+    return torch.stack([torch.sin(a), torch.cos(a)], dim=-1).flatten(1)[:, :width].float()
 
 
 def _pool_rows(positions, req, kv_indptr, kv_indices, kv_first, page_size):
@@ -308,19 +322,24 @@ def gqa_append(q, k, v, q_w, k_w, pool, positions, token_req, kv_indptr, kv_indi
     return q
 
 
-def gqa_attention(q, pool, positions, token_req, kv_indptr, kv_indices, kv_first, *, scale, softcap=0.0, window=0, sinks=None):
-    """q [T, H, hd] -> [T, H, hd] over the paged keys and values; capped scores, exp(sink) in the denominator."""
+def gqa_attention(q, pool, positions, token_req, kv_indptr, kv_indices, kv_first, *, scale, softcap=0.0, window=0, sinks=None,
+                  dist=None, chunk=0):
+    """q [T, H, hd] -> [T, H, hd] over the paged keys and values; capped scores, exp(sink) in the denominator, ``dist`` [H, 2]
+    (a, b): scores lose a ln(1 + b distance); ``chunk``: only keys of the position's own run of so many."""
     T, H, hd = q.shape
     G, ps = pool.shape[2], pool.shape[3]
     out = torch.zeros(T, H, hd)
     for t in range(T):
         pos = int(positions[t])
-        keys = torch.arange(max(0, pos - window + 1) if window else 0, pos + 1)
+        first = max(0, pos - window + 1) if window else pos // chunk * chunk if chunk else 0
+        keys = torch.arange(first, pos + 1)
         rows = _pool_rows(keys, int(token_req[t]), kv_indptr, kv_indices, kv_first, ps)
         k, v = (pool[rows // ps, j, :, rows % ps].float() for j in (0, 1))          # [n, G, hd]
         s = torch.einsum("gmd,ngd->gmn", q[t].float().reshape(G, H // G, hd), k).reshape(H, -1) * scale
         if softcap:
             s = softcap * torch.tanh(s / softcap)
+        if dist is not None:
+            s = s - dist[:, :1] * torch.log1p(dist[:, 1:] * (pos - keys).float())
         if sinks is not None:
             s = torch.cat([s, sinks.float()[:, None]], dim=1)
         p = torch.softmax(s, dim=-1)[:, :keys.numel()].reshape(G, H // G, -1)
@@ -361,19 +380,22 @@ def head_norm_silu(o, g, w, dim, eps):
     return o.float() * inv * w.float() * torch.nn.functional.silu(g.float())
 
 
-def moe_route(logits, correction, top, groups, keep, scale, score="sigmoid"):
+def moe_route(logits, correction, top, groups, keep, scale, score="sigmoid", group_score="top2"):
     """(experts [T, top], weights [T, top]) from router logits [T, E]. ``score`` "softmax": of the chosen logits, the
-    correction included."""
-    s = torch.sigmoid(logits.float()) if score == "sigmoid" else logits.float()
+    correction included; "softmax_all": of all logits, the chosen ones not normed."""
+    z = logits.float()
+    s = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, dim=-1) if score == "softmax_all" else z
     choice = s if correction is None else s + correction
     z = choice
     if groups > 1:
         c = choice.reshape(len(s), groups, -1)
-        best = c.topk(min(2, c.shape[-1]), dim=-1).values.sum(-1).topk(keep, dim=-1).indices
+        best = c.topk(min(2 if group_score == "top2" else 1, c.shape[-1]), dim=-1).values.sum(-1).topk(keep, dim=-1).indices
         allowed = torch.zeros(len(s), groups, dtype=torch.bool).scatter_(1, best, True)
         choice = c.masked_fill(~allowed[:, :, None], float("-inf")).reshape(len(s), -1)
     idx = choice.topk(top, dim=-1).indices
     if score == "softmax":
         return idx, torch.softmax(z.gather(1, idx), dim=-1) * scale
     w = s.gather(1, idx)
+    if score == "softmax_all":
+        return idx, w * scale
     return idx, w / (w.sum(-1, keepdim=True) + 1e-20) * scale

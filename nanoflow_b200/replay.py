@@ -35,7 +35,7 @@ class TraceReplay:
         self.engine, self.model = engine, m
         self.pool = DistKVPool(m.run_layers, m.num_kv_heads, m.head_dim, num_pages, engine.eng.page_size, 1)
         self.slots = StateSlotPool(state_slots) if getattr(m, "has_state", False) else None
-        self.window = getattr(m, "kv_window", 0)
+        self.first_seen = getattr(m, "first_seen", None)
         self.live: Dict[str, object] = {}
         self.steps = 0
 
@@ -51,8 +51,8 @@ class TraceReplay:
             kv = self.live.get(e["id"])
             if kv is None:
                 kv = self.live[e["id"]] = DistKVCache(self.pool, self.slots)
-            if self.window > 0:
-                kv.trim(kv.seqlen - self.window + 1)
+            if self.first_seen is not None:
+                kv.trim(self.first_seen(kv.seqlen))
             kv.allocate_tokens(tokens.size)
             portions.append(Portion(kv, tokens, e.get("want") or ()))
         out = None

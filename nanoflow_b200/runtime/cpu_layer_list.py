@@ -36,6 +36,9 @@ class CpuLayerListEngine:
             self.pools.append(torch.zeros(num_pages, *shapes[0]) if shapes else None)
             self.state.append(tuple(torch.zeros(n, *shape) for s in parts for shape, _ in m.state_shapes(s)))
             self.conv_state.append([torch.zeros(n, *m.conv_state_shape()) for _ in range(2)] if m.input_conv else None)
+            src = getattr(m.layers[r.layer].mixer, "kv_from", None)
+            if src is not None:                              # lent keys and values (no loops: runs are layers)
+                self.pools[-1] = self.pools[src]
         self.v_first: Optional[torch.Tensor] = None
         self.sampled = torch.zeros(self.eng.max_sample_rows or self.eng.max_batch_size, dtype=torch.int32)
         self._staged: Optional[BatchPlan] = None
@@ -46,7 +49,8 @@ class CpuLayerListEngine:
     # ---- one iteration --------------------------------------------------------------------------------
     def _norm(self, x, n):
         m = self.model
-        y = ref.layernorm(x, n.w[:m.hidden_size], None if n.b is None else n.b[:m.hidden_size], m.norm_eps) if m.norm_kind == "layer" else \
+        y = x * n.w[:m.hidden_size] if n.kind == "scale" else \
+            ref.layernorm(x, n.w[:m.hidden_size], None if n.b is None else n.b[:m.hidden_size], m.norm_eps) if m.norm_kind == "layer" else \
             ref.rmsnorm(x, n.w[:m.hidden_size], m.norm_eps)
         return torch.nn.functional.pad(y, (0, m.width_p - m.hidden_size))
 
@@ -79,24 +83,26 @@ class CpuLayerListEngine:
     def _attention(self, r, s, lw, h, plan):
         m, T = self.model, h.shape[0]
         H, G, hd = s.heads, s.kv_heads, m.attn_hd(s)
-        q, k, v = (h @ lw.w_in.t()).split([H * hd, G * hd, G * hd], dim=1)
+        proj = h @ lw.w_in.t() if lw.b_in is None else h @ lw.w_in.t() + lw.b_in
+        q, k, v = proj.split([H * hd, G * hd, G * hd], dim=1) if s.kv_from is None else (proj, None, None)
         if s.value_mix and r == m.first_value_run:
             self.v_first = v
         elif s.value_mix:
             v = (1.0 - lw.value_lambda) * v + lw.value_lambda * self.v_first
         pages = (plan.positions, plan.token_req, plan.kv_indptr, plan.kv_indices, plan.kv_first)
         turns = rotations(s)
-        turn = lambda x, n, i, sign=1.0: x if len(turns) <= i else \
+        turn = lambda x, n, i, sign=1.0: x if x is None or len(turns) <= i else \
             ref.turn_pairs(x.reshape(T, n, hd), plan.positions, turns[i], sign).reshape(T, -1)
         q, k, v = turn(q, H, 0), turn(k, G, 0), turn(v, G, 1)
-        q = ref.gqa_append(q, k, v, lw.q_norm, lw.k_norm, self.pools[r], *pages, heads=H, kv_heads=G, dim=s.dim,
-                           eps=m.norm_eps)
+        if k is not None:
+            q = ref.gqa_append(q, k, v, lw.q_norm, lw.k_norm, self.pools[r], *pages, heads=H, kv_heads=G, dim=s.dim,
+                               eps=m.norm_eps)
         if s.talk:
             o = ref.talk_attention(q.reshape(T, H, hd), self.pools[r], *pages, scale=s.scale, talk=lw.talk, window=s.window or 0,
                                    sinks=lw.sinks)
         else:
             o = ref.gqa_attention(q.reshape(T, H, hd), self.pools[r], *pages, scale=s.scale, softcap=s.softcap or 0.0,
-                                  window=s.window or 0, sinks=lw.sinks)
+                                  window=s.window or 0, sinks=lw.sinks, dist=lw.dist, chunk=s.chunk or 0)
         o = turn(o, H, 1, -1.0)
         return o.reshape(T, -1) @ lw.w_o.t()
 
@@ -142,19 +148,22 @@ class CpuLayerListEngine:
     # ---- feed-forwards ----------------------------------------------------------------------------------
     def _dense(self, s, lw, h):
         a = s.act
-        return ref.gated_mlp(h, lw.w_gate, lw.w_up, lw.w_down, a.name, limit=a.limit, alpha=a.alpha, shift=a.shift)
+        return ref.gated_mlp(h, lw.w_gate, lw.w_up, lw.w_down, a.name, biases=(lw.b_gate, lw.b_up, lw.b_down), limit=a.limit,
+                             alpha=a.alpha, shift=a.shift)
 
     def _moe(self, s, lw, h):
         logits = h @ lw.router.t()
-        idx, weight = ref.moe_route(logits[:, :s.experts], lw.correction, s.top, s.groups, s.keep, s.scale, s.score)
+        idx, weight = ref.moe_route(logits[:, :s.outputs], lw.correction, s.top, s.groups, s.keep, s.scale, s.score, s.group_score)
         mats = [None if t is None else t.chunk(s.experts) for t in (lw.w_gate, lw.w_up, lw.w_down)]
         a, out = s.expert.act, torch.zeros_like(h)
         for e in range(s.experts):
             t, k = (idx == e).nonzero(as_tuple=True)
             if t.numel():
-                y = torch.nn.functional.gelu(h[t] @ mats[1][e].t()) @ mats[2][e].t() if not s.expert.gated else \
+                y = ref.linear_act(h[t] @ mats[1][e].t(), a.name) @ mats[2][e].t() if not s.expert.gated else \
                     ref.gated_mlp(h[t], mats[0][e], mats[1][e], mats[2][e], a.name, limit=a.limit, alpha=a.alpha, shift=a.shift)
                 out.index_add_(0, t, y * weight[t, k][:, None])
+        if s.identity:
+            out += (weight * (idx >= s.experts)).sum(-1, keepdim=True) * h
         if s.shared is not None:
             out += torch.sigmoid(logits[:, s.experts:s.experts + 1]) * self._dense(s.shared, lw.shared, h)
         return out
@@ -171,6 +180,9 @@ class CpuLayerListEngine:
         W = m.hidden_size
         after = lambda y, n: y if n is None else self._norm(y[:, :W], n)
         x = start = after(w.embed[ids] * m.embed_scale, w.embed_norm)
+        if m.sinusoid:
+            x = start = x + torch.nn.functional.pad(ref.sinusoid(plan.positions, W, m.sinusoid), (0, m.width_p - W))
+        results = [x]
         for r, run in enumerate(m.runs):
             spec, lw = m.layers[run.layer], w.layers[run.layer]
             if run.step is not None:
@@ -185,6 +197,9 @@ class CpuLayerListEngine:
                 x = x + after(y, lw.norm_out)
                 h = self._input_conv(r, 1, self._norm(x[:, :W], lw.mlp_in), lw.conv_mlp, plan)
                 x = x + after(FEED_FORWARDS[spec.mlp.kind](self, spec.mlp, lw.mlp, h), lw.mlp_out)
+            if m.depth_average:
+                results.append(x)
+                x = sum(a * y for a, y in zip(lw.depth, results))
         rows = torch.from_numpy(plan.sample_rows).long()
         self._logits = (self._norm(x[rows][:, :m.hidden_size], w.final_norm) @ w.lm_head.t())[:, :m.vocab_size]
         toks = self._logits.argmax(dim=-1).int()

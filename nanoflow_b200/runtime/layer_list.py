@@ -12,8 +12,9 @@ one GPU, one stream. Per layer run:
   portions gather the latents they can see, expand them to keys and values of all heads with one GEMM, and
   run the tcgen05 prefill kernel over those;
 * grouped-query attention: queries and keys normed or rotated, values mixed or rotated, both appended to the paged
-  pool; single tokens on the split-KV decode kernel, portions on the tcgen05 prefill kernel (in 32-bit, and for head
-  sizes and options those are not built for, one simple kernel); attention with mixed heads on kernels of its own;
+  pool (or those of an earlier layer read from its pool); single tokens on the split-KV decode kernel, portions on the
+  tcgen05 prefill kernel, both with capped scores, sinks, distance biases and chunks (in 32-bit, and for head sizes and
+  options those are not built for, one simple kernel); attention with mixed heads on kernels of its own;
 * mLSTM: one kernel for requests with one token, one for longer portions, then head norm and output gate;
 * WKV: every stream's mix with the previous token (kept per request), the four projections as one block-diagonal
   product, the low-rank decay, one kernel for single tokens and one for portions (chunks, or token by token),
@@ -25,10 +26,11 @@ one GPU, one stream. Per layer run:
 * two mixers side by side: one input projection for both;
 * output projection;
 * feed-forward: gated, or a mixture of experts (router product, routing, rows in expert order, two products per
-  expert, the shared expert);
-* one kernel for: norm of the sublayer's output, of a pair's outputs, or of the weighted sum of experts and shared
-  expert, residual sum in fp32, the step vector of a loop pass or the embedding row, and the norm the next sublayer
-  reads; a convolution over time after it where the model has one.
+  expert, the shared expert, or experts that hand on the input);
+* one kernel for: norm or scale of the sublayer's output, of a pair's outputs, or of the weighted sum of experts and shared
+  expert, residual sum in fp32, the step vector of a loop pass or the embedding row (with its position vector), the
+  weighted sum with the results of earlier layers, and the norm the next sublayer reads; a convolution over time after
+  it where the model has one.
 
 A new kind of mixer needs a spec and weights in ``models/layer_list.py`` and a builder in ``MIXERS``, a new kind of
 feed-forward one in ``FEED_FORWARDS``.
@@ -151,7 +153,7 @@ class LayerListEngine(Engine):
             lay = m.layers[r.layer]
             self.state.append(tuple(z(n, *shape, dtype=dt) for s in parts_of(lay.mixer) for shape, dt in m.state_shapes(s)))
             conv = lambda used: z(n, *m.conv_state_shape(), dtype=m.dtype) if m.input_conv and used else None
-            self.conv_state.append((conv(True), conv(lay.mlp is not None)))
+            self.conv_state.append((conv(True), conv(m.conv_mlp(lay))))
 
     def _widths(self) -> Dict[str, int]:
         """Columns of the shared activation buffers (the widest layer's)."""
@@ -195,8 +197,9 @@ class LayerListEngine(Engine):
                     up("cg", ld)
             elif s.kind == "attention":
                 hd = m.attn_hd(s)
-                up("proj", (s.heads + 2 * s.kv_heads) * hd)
-                up("qn", s.heads * hd)
+                up("proj", s.proj_heads * hd)
+                if moves_queries(s):
+                    up("qn", s.heads * hd)
                 up("attn", s.heads * hd)
                 if s.value_mix:
                     up("v_first", s.kv_heads * hd)
@@ -237,6 +240,7 @@ class LayerListEngine(Engine):
                                          w["aux"] + 2 * m.width_p) +
                    4 * (w["gates"] + w["o_rec"] + w["router"] + w["beta"] + 5 * w["e_top"] + 2 * sum((len(k) + 7) // 8 * 8 for k in self._rotations())))
         act += self._decode_ws_floats() * 4 + self._chunk_scratch_floats() * 4
+        act += 4 * T * m.width_p * len(m.runs) if m.depth_average else 0
         act += self.x_pages * PAGE * (w["kv"] + w["cg"]) * es + self.S_cap * (es * m.width_p + 4 * m.vocab_p)
         budget = free - total * (1.0 - e.gpu_mem_fraction) - act - (1 << 30)
         per_page = max(1, m.kv_bytes_per_token_local()) * PAGE
@@ -281,6 +285,14 @@ class LayerListEngine(Engine):
         self.h = P(T, m.width_p, dt, "h")
         self.y = P(T, m.width_p, dt, "y")
         self.h_raw = P(T, m.width_p, dt, "h_raw") if m.input_conv else None      # before the input convolution
+        # the embedding output and every layer's result, where later layers read them
+        self.hist = self._plain(len(m.runs) * T, m.width_p, dtype=f32, name="results").view(len(m.runs), T, m.width_p) \
+            if m.depth_average else None
+        self.pos_freq = None
+        if m.sinusoid:
+            i = torch.arange((m.hidden_size + 1) // 2 + 1, dtype=torch.float64)
+            f = m.sinusoid ** (-2.0 * i / m.hidden_size)
+            self.pos_freq = torch.stack([f.float(), (f - f.float().double()).float()], dim=1).contiguous().to(dev)
         pairs = any(lay.mixer.kind == "pair" for lay in m.layers)
         self.y2 = P(T, m.width_p, dt, "y2") if m.parallel or m.run_moes() or pairs else None
         flat = lambda k, dtype, rows=T: P(1, max(8, rows * w[k]), dtype, k).view(-1)
@@ -310,6 +322,10 @@ class LayerListEngine(Engine):
         self.logits = P(self.S_cap, m.vocab_p, f32, "logits")
         self.pools = [next((p for s in parts_of(m.layers[r.layer].mixer) for p in [self._pool(s)] if p is not None), None)
                       for r in m.runs]
+        for r, run in enumerate(m.runs):                 # lent keys and values (no loops: runs are layers)
+            src = getattr(m.layers[run.layer].mixer, "kv_from", None)
+            if src is not None:
+                self.pools[r] = self.pools[src]
         self.arange = torch.arange(self.x_pages + 1, dtype=torch.int32, device=dev)
         heads = max([s.heads * (m.latent_ld(s) + 2) for s in m.run_specs("latent_attention")], default=0)
         self.latent_ws = torch.empty(max(8, 160 * heads), dtype=f32, device=dev)
@@ -358,7 +374,8 @@ class LayerListEngine(Engine):
         # what joins the stream before each run: a step vector, or the embedding row
         step = lambda r: None if m.runs[r].step is None else "embedding" if m.loop_add == "embedding" else \
             w.loop_steps[m.runs[r].step]
-        self._residual("embedding", None, w.embed_norm, w.layers[m.runs[0].layer].norm_in, step(0), embed=True, feeds=(0, 0))
+        self._residual("embedding", None, w.embed_norm, w.layers[m.runs[0].layer].norm_in, step(0), embed=True, feeds=(0, 0),
+                       average=-1 if m.depth_average else None)
         for r, run in enumerate(m.runs):
             spec, lw = m.layers[run.layer], w.layers[run.layer]
             last = r + 1 == len(m.runs)
@@ -373,14 +390,15 @@ class LayerListEngine(Engine):
                 more = FEED_FORWARDS[spec.mlp.kind](self, r, run.layer, spec.mlp, lw.mlp)
                 if not m.parallel:
                     y = more.pop("y2", None) if "y2_gate" not in more else None
+            average = r if m.depth_average else None
             if last and self.taps is None:
                 # only the sampled rows go on
-                self._residual("final", y, out, w.final_norm, None, sampled=True, more=more)
+                self._residual("final", y, out, w.final_norm, None, sampled=True, more=more, average=average)
             else:
                 tap_add = add if self.taps is None else None
                 go_on = not last and self.taps is None
                 self._residual(f"R{r}.out", y, out, nxt if go_on else None, tap_add, layer=r, more=more,
-                               feeds=(r + 1, 0) if go_on else None)
+                               feeds=(r + 1, 0) if go_on else None, average=average)
                 if self.taps is not None:
                     self._op(f"R{r}.tap", MemcpyParams(dst=_ptr(self.taps[r]), src=_ptr(self.x), elem_bytes=4 * m.width_p,
                                                        count=0), dyn=[("count", T)], layer=r)
@@ -404,14 +422,21 @@ class LayerListEngine(Engine):
                                   kernel=kernel, layer=layer, nano=0)
 
     def _residual(self, name, y, norm_in: Optional[NormWeights], norm_out: Optional[NormWeights], add, *, embed=False,
-                  sampled=False, layer=-1, more: Optional[dict] = None, feeds: Optional[Tuple[int, int]] = None) -> None:
+                  sampled=False, layer=-1, more: Optional[dict] = None, feeds: Optional[Tuple[int, int]] = None,
+                  average: Optional[int] = None) -> None:
         """``more``: what a sublayer adds to the sum besides ``y``: ``y2`` with ``y2_gate`` per row, and expert rows
         (``e_out``, ``e_slot``, ``e_weight``, ``e_top``), under the same norm; or ``pair``: the norms of ``y`` and ``y2``
         whose mean is the output. ``add``: a vector, or "embedding". ``feeds``: the run and sublayer (mixer 0, feed-forward
         1) that reads the normed stream, through its input convolution if it has one: single tokens get it here, portions
-        by an op of its own."""
-        m, kind = self.model, NORMS[self.model.norm_kind]
+        by an op of its own. ``average``: the run whose result this is (-1: the embedding output); the weighted sum of all
+        results so far goes on."""
+        m = self.model
+        kind = lambda norm: NORMS[norm.kind or m.norm_kind]
         p = ResidualNormParams()
+        conv, state = None, None
+        if feeds is not None:
+            lw = self.w.layers[m.runs[feeds[0]].layer]
+            conv, state = (lw.conv_mlp if feeds[1] else lw.conv_in), self.conv_state[feeds[0]][feeds[1]]
         p.x, p.ld_x = _ptr(self.x), self.x.stride(0)
         again = isinstance(add, str)
         if embed or again:
@@ -420,10 +445,18 @@ class LayerListEngine(Engine):
             p.host_ids, p.feedback_src = _ptr(self.meta["host_ids"]), _ptr(self.meta["feedback_src"])
             p.prev_tokens = _ptr(self.bufs.sampled)
             p.src_scale = m.embed_scale
+        if embed and self.pos_freq is not None:
+            p.pos_freq, p.positions = _ptr(self.pos_freq), _ptr(self.meta["positions"])
+        if average is not None:
+            if average >= 0:
+                p.hist, p.hist_w = _ptr(self.hist), _ptr(self.w.layers[m.runs[average].layer].depth)
+                p.hist_n, p.hist_stride = average + 1, self.hist.stride(0)
+            if average + 1 < len(m.runs):
+                p.hist_out = _ptr(self.hist[average + 1])
         if y is not None and not embed:
             p.y, p.ld_y = _ptr(y), y.stride(0)
         if norm_in is not None:
-            p.in_w, p.in_b, p.in_kind = _ptr(norm_in.w), _ptr(norm_in.b), kind
+            p.in_w, p.in_b, p.in_kind = _ptr(norm_in.w), _ptr(norm_in.b), kind(norm_in)
         more = more or {}
         if more.get("y2") is not None:
             p.y2, p.ld_y2, p.y2_gate = _ptr(more["y2"]), more["y2"].stride(0), _ptr(more.get("y2_gate"))
@@ -436,24 +469,20 @@ class LayerListEngine(Engine):
             p.norm_sum = 1
         p.add = None if again else _ptr(add)
         if norm_out is not None:
-            h = self.h_s if sampled else self.h if self.h_raw is None else self.h_raw
-            p.h, p.ld_h, p.out_w, p.out_b, p.out_kind = _ptr(h), h.stride(0), _ptr(norm_out.w), _ptr(norm_out.b), kind
+            h = self.h_s if sampled else self.h if conv is None else self.h_raw
+            p.h, p.ld_h, p.out_w, p.out_b, p.out_kind = _ptr(h), h.stride(0), _ptr(norm_out.w), _ptr(norm_out.b), kind(norm_out)
         if sampled:
             p.rows_idx, p.in_rows = _ptr(self.meta["sample_rows"]), self.T
         p.cols, p.eps, p.dtype, p.status = m.hidden_size, m.norm_eps, self.code, _ptr(self.bufs.status)
         dyn = [("rows", "n_sample" if sampled else "T")]
-        w = None
-        if feeds is not None:
-            lw = self.w.layers[m.runs[feeds[0]].layer]
-            w, state = (lw.conv_mlp if feeds[1] else lw.conv_in), self.conv_state[feeds[0]][feeds[1]]
-        if w is not None:
-            p.conv_w, p.conv_out, p.conv_state = _ptr(w), _ptr(self.h), _ptr(state)
+        if conv is not None:
+            p.conv_w, p.conv_out, p.conv_state = _ptr(conv), _ptr(self.h), _ptr(state)
             p.state_slot, p.positions = _ptr(self.meta["state_ref"]), _ptr(self.meta["positions"])
-            p.conv_taps, p.conv_ld, p.num_slots = w.shape[0], w.shape[1], self.num_slots
+            p.conv_taps, p.conv_ld, p.num_slots = conv.shape[0], conv.shape[1], self.num_slots
             dyn.append(("conv_rows", "n_dec"))
         self._op(name, p, dyn=dyn, layer=layer)
-        if w is not None:
-            self._short_conv(f"R{feeds[0]}.input_conv{feeds[1]}", self.h_raw, self.h, w, state, residual=True, portions=True,
+        if conv is not None:
+            self._short_conv(f"R{feeds[0]}.input_conv{feeds[1]}", self.h_raw, self.h, conv, state, residual=True, portions=True,
                              layer=feeds[0])
 
     def _short_conv(self, name, x, out, w, state, *, bias=None, act=None, residual=False, portions=False,
@@ -467,15 +496,15 @@ class LayerListEngine(Engine):
                             num_slots=self.num_slots, dtype=self.code, status=_ptr(self.bufs.status))
         self._op(name, p, dyn=[("T", "T")] + ([("row_begin", "n_dec")] if portions else []), layer=layer)
 
-    def _gemm(self, name, a, wt, out, *, rows: str, up=None, act: ActSpec = ActSpec("silu"), lin_act=None, bias=None, d32=None,
-              f32_col0=0, groups=1, group_k=0, k=0, key="", layer=-1) -> None:
+    def _gemm(self, name, a, wt, out, *, rows: str, up=None, act: ActSpec = ActSpec("silu"), lin_act=None, bias=None, up_bias=None,
+              d32=None, f32_col0=0, groups=1, group_k=0, k=0, key="", layer=-1) -> None:
         """out[rows, N] = a @ wt^T. ``d32``: columns from ``f32_col0`` on leave as fp32; ``groups`` > 1:
         block-diagonal (each group of rows of ``wt`` sees ``k`` columns of ``a``, ``group_k`` apart)."""
         p = GemmParams()
         p.A, p.B, p.B2, p.D = _ptr(a), _ptr(wt), _ptr(up), _ptr(out)
         p.lda, p.ldb, p.ldd = a.stride(0), wt.stride(0), (out.stride(0) if out is not None else wt.shape[0])
         p.N, p.K = wt.shape[0], k or wt.shape[1]
-        p.epilogue, p.lin_act, p.bias = (1 if up is not None else 0), LIN_ACTS[lin_act], _ptr(bias)
+        p.epilogue, p.lin_act, p.bias, p.bias2 = (1 if up is not None else 0), LIN_ACTS[lin_act], _ptr(bias), _ptr(up_bias)
         p.act, p.act_limit, p.act_alpha, p.act_shift = ACTS[act.name], act.limit, act.alpha, act.shift
         if d32 is not None:
             p.D32, p.ld32, p.f32_col0 = _ptr(d32), d32.stride(0), f32_col0
@@ -574,12 +603,14 @@ class LayerListEngine(Engine):
         """``proj``: the projected queries, keys and values, if they are there already."""
         m, g, T, meta, st = self.model, self.g, "T", self.meta, _ptr(self.bufs.status)
         H, G, hd, pool = s.heads, s.kv_heads, m.attn_hd(s), self.pools[r]
-        qn, attn = self.view("qn", H * hd), self.view("attn", H * hd)
+        attn = self.view("attn", H * hd)
         if proj is None:
-            proj = self.view("proj", (H + 2 * G) * hd)
-            self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, key=f"l{layer}.in", layer=r)
+            proj = self.view("proj", s.proj_heads * hd)
+            self._gemm(f"R{r}.in", self.h, lw.w_in, proj, rows=T, bias=lw.b_in, key=f"l{layer}.in", layer=r)
+        # queries that nothing is done to stay in the projection's rows
+        q, ld_q = (self.view("qn", H * hd), 0) if moves_queries(s) else (proj, proj.stride(0))
         mode = 0 if not s.value_mix else 1 if r == m.first_value_run else 2
-        ap = GqaAppendParams(src=_ptr(proj), ld_src=proj.stride(0), q_off=0, k_off=H * hd, v_off=(H + G) * hd, q_out=_ptr(qn),
+        ap = GqaAppendParams(src=_ptr(proj), ld_src=proj.stride(0), q_off=0, k_off=H * hd, v_off=(H + G) * hd, q_out=None if ld_q else _ptr(q),
                              q_w=_ptr(lw.q_norm), k_w=_ptr(lw.k_norm), v_first=_ptr(self.flat["v_first"]), v_mode=mode,
                              v_lambda=lw.value_lambda, pool=_ptr(pool), positions=_ptr(meta["positions"]),
                              token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
@@ -594,11 +625,12 @@ class LayerListEngine(Engine):
             ap.v_rot, ap.v_pairs, ap.v_ld = v_rot, v_pairs, v_ld
         else:
             v_rot, v_pairs, v_ld = None, 0, 0
-        self._op(f"R{r}.gqa_append", ap, dyn=[("T", T)], layer=r)
+        if s.kv_from is None:
+            self._op(f"R{r}.gqa_append", ap, dyn=[("T", T)], layer=r)
         if s.talk:
             def params() -> TalkAttnParams:
                 return TalkAttnParams(
-                    q=_ptr(qn), pool=_ptr(pool), out=_ptr(attn), positions=_ptr(meta["positions"]),
+                    q=_ptr(q), pool=_ptr(pool), out=_ptr(attn), positions=_ptr(meta["positions"]),
                     token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]), kv_indices=_ptr(meta["kv_indices"]),
                     kv_first=_ptr(meta["kv_first"]), sinks=_ptr(lw.sinks), talk=_ptr(lw.talk), v_rot=v_rot, v_pairs=v_pairs,
                     v_ld=v_ld, token_begin=0, n_tokens=0, heads=H, kv_heads=G, hd=hd, page_size=PAGE, num_pages=self.num_pages,
@@ -616,7 +648,8 @@ class LayerListEngine(Engine):
         elif m.attn_on_tensor_cores(s):
             def params() -> AttnParams:
                 p = AttnParams()
-                p.q, p.out, p.kv_pool = _ptr(qn), _ptr(attn), _ptr(pool)
+                p.q, p.ld_q, p.out, p.kv_pool = _ptr(q), ld_q, _ptr(attn), _ptr(pool)
+                p.kv_first, p.dist, p.chunk = _ptr(meta["kv_first"]), _ptr(lw.dist), s.chunk or 0
                 p.qo_indptr, p.kv_indptr = _ptr(meta["qo_indptr"]), _ptr(meta["kv_indptr"])
                 p.kv_indices, p.kv_last_page_len = _ptr(meta["kv_indices"]), _ptr(meta["kv_last_page_len"])
                 p.q_heads, p.kv_heads, p.head_dim, p.page_size, p.num_pages = H, G, hd, PAGE, self.num_pages
@@ -633,7 +666,7 @@ class LayerListEngine(Engine):
             self._op(f"R{r}.attn_prefill", p, kernel="nfk_attn_prefill_ws",
                      dyn=[("num_items", g.symbol(f"n_gitems{s.group}"))], layer=r)
         else:
-            gp = GqaAttnParams(q=_ptr(qn), pool=_ptr(pool), out=_ptr(attn), positions=_ptr(meta["positions"]),
+            gp = GqaAttnParams(q=_ptr(q), ld_q=ld_q, dist=_ptr(lw.dist), chunk=s.chunk or 0, pool=_ptr(pool), out=_ptr(attn), positions=_ptr(meta["positions"]),
                                token_req=_ptr(meta["token_req"]), kv_indptr=_ptr(meta["kv_indptr"]),
                                kv_indices=_ptr(meta["kv_indices"]), kv_first=_ptr(meta["kv_first"]), sinks=_ptr(lw.sinks),
                                token_begin=0, n_tokens=0, heads=H, kv_heads=G, hd=hd, page_size=PAGE,
@@ -745,9 +778,9 @@ class LayerListEngine(Engine):
     def _dense(self, r: int, layer: int, s, lw, key="") -> dict:
         act = self.view("act", round8(s.ff))
         out = self.y2 if self.y2 is not None else self.y
-        self._gemm(f"R{r}.{key}gate_up", self.h, lw.w_gate, act, rows="T", up=lw.w_up, act=s.act, key=f"l{layer}.{key}gate_up",
-                   layer=r)
-        self._gemm(f"R{r}.{key}down", act, lw.w_down, out, rows="T", key=f"l{layer}.{key}down", layer=r)
+        self._gemm(f"R{r}.{key}gate_up", self.h, lw.w_gate, act, rows="T", up=lw.w_up, act=s.act, bias=lw.b_gate, up_bias=lw.b_up,
+                   key=f"l{layer}.{key}gate_up", layer=r)
+        self._gemm(f"R{r}.{key}down", act, lw.w_down, out, rows="T", bias=lw.b_down, key=f"l{layer}.{key}down", layer=r)
         return {"y2": out}
 
     def _moe(self, r: int, layer: int, s, lw) -> dict:
@@ -760,7 +793,8 @@ class LayerListEngine(Engine):
         rp = MoeRouteParams(logits=_ptr(logits), ld=logits.stride(0), correction=_ptr(lw.correction), expert=_ptr(ids["expert"]),
                             weight=_ptr(ids["weight"]), rank=_ptr(ids["rank"]), counts=_ptr(counts), gate=_ptr(self.moe_gate),
                             T=0, experts=s.experts, top=s.top, groups=s.groups, keep=s.keep,
-                            gate_col=s.experts if s.shared is not None else -1, scale=s.scale, score=ROUTER_SCORES[s.score])
+                            gate_col=s.experts if s.shared is not None else -1, scale=s.scale, score=ROUTER_SCORES[s.score],
+                            identity=s.identity, group_max=int(s.group_score == "max"))
         self._op(f"R{r}.moe_route", rp, dyn=[("T", T)], layer=r)
         pp = MoePermuteParams(h=_ptr(self.h), ld_h=wp, out=_ptr(e_in), ld_out=wp, expert=_ptr(ids["expert"]),
                               rank=_ptr(ids["rank"]), counts=_ptr(counts), slot=_ptr(ids["slot"]), T=0, top=s.top,
@@ -781,6 +815,8 @@ class LayerListEngine(Engine):
             product("moe_up", e_in, lw.w_up, None, e_act, round8(s.expert.ff), s.expert.act.name)
         product("moe_down", e_act, lw.w_down, None, e_out, wp)
         out = dict(e_out=e_out, e_slot=ids["slot"], e_weight=ids["weight"], e_top=s.top)
+        if s.identity:
+            out.update(y2=self.h, y2_gate=self.moe_gate)
         if s.shared is not None:
             out.update(self._dense(r, layer, s.shared, lw.shared, key="shared_"), y2_gate=self.moe_gate)
         return out
@@ -869,7 +905,9 @@ class LayerListEngine(Engine):
             put(f"gitem{n}", items.reshape(-1))
             sym[f"n_gitems{n}"] = items.shape[0]
         if self.attn_groups:
-            sym["dec_chunk_pages"], sym["dec_max_chunks"] = self._attn_split(D, plan.max_kv_pages)
+            chunks = [s.chunk for s in m.run_specs("attention") if m.attn_on_tensor_cores(s)]
+            seen = plan.max_kv_pages if None in chunks else min(plan.max_kv_pages, max(chunks) // PAGE + 2)
+            sym["dec_chunk_pages"], sym["dec_max_chunks"] = self._attn_split(D, seen)
         for top in {f.top for f in m.run_moes()}:
             sym[f"e_rows{top}"] = plan.num_tokens * top
         for g in self.groups:
@@ -925,6 +963,11 @@ def delta_item_floats(s) -> int:
     """Scratch of a chunk and head of the chunked delta-rule kernels (nfk_delta_item_floats)."""
     n = 64 if max(round8(s.dim), round8(s.vdim)) <= 64 else 128
     return (6 * CHUNK * (n + 8) + 2 * CHUNK * (CHUNK + 8)) // 2 + n + n // 32 * CHUNK * 36
+
+
+def moves_queries(s) -> bool:
+    """Whether an attention layer's queries pass through the append kernel."""
+    return s.qk_norm or s.rotary is not None or s.talk
 
 
 def rotations(s) -> List[tuple]:

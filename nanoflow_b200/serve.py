@@ -139,7 +139,7 @@ def main(argv=None) -> int:
                     hold_retired_pages=bool(eng_cfg.offload and args.backend == "gpu"),
                     decode_tail_fraction=eng_cfg.decode_tail_fraction,
                     state_pool=StateSlotPool(engine.num_slots) if getattr(engine, "num_slots", 0) else None,
-                    kv_window=getattr(model, "kv_window", 0))
+                    first_seen=getattr(model, "first_seen", None))
     sch.keep_schedule_log = bool(args.output_prefix)
     offload = None
     if eng_cfg.offload and args.backend == "gpu":

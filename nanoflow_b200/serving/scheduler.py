@@ -27,7 +27,7 @@ from __future__ import annotations
 
 import time
 from dataclasses import dataclass, field
-from typing import List, Optional, Sequence, Tuple
+from typing import Callable, List, Optional, Sequence, Tuple
 
 import numpy as np
 
@@ -165,13 +165,14 @@ class Scheduler:
                  average_decode_length: int = 512, group_size: int = 8, eos_token_id: Optional[int] = None,
                  stop_on_eos: bool = False, hold_retired_pages: bool = False, prefill_ctas: int = 296,
                  decode_tail_fraction: float = 0.0, state_pool: Optional[StateSlotPool] = None,
-                 kv_window: int = 0):
+                 kv_window: int = 0, first_seen: Optional[Callable[[int], int]] = None):
         """``state_pool``: slots of recurrent state, one per request in flight (models that carry one).
         ``kv_window``: > 0 if no token of the model sees further back than this many positions; pages that
-        have left the window are then given back while the request runs."""
+        have left the window are then given back while the request runs. ``first_seen`` says the same of models whose tokens
+        do not all see as far: the first position that a token at a position, or any token after it, sees."""
         self._memory_pool = memory_pool
         self._state_pool = state_pool
-        self.kv_window = int(kv_window)
+        self.first_seen = first_seen or ((lambda p: p - int(kv_window) + 1) if kv_window > 0 else None)
         self._request_queue = request_queue
         self.global_batch_size = int(global_batch_size)
         self.nanobatch_sizes = list(nanobatch_sizes) if nanobatch_sizes else [self.global_batch_size]
@@ -452,11 +453,11 @@ class Scheduler:
         sample_rows.extend(range(t, t + Dt))
         sample_reqs.extend(tail)
         kvs = [r.kv_cache for r in head] + [r.kv_cache for r, _, _ in prefill] + [r.kv_cache for r in tail]
-        if self.kv_window > 0:
-            # The step's first token of a request sees kv_window - 1 positions back. Pages before that may
-            # still be read by the iteration in flight; whoever gets them writes them in a later one.
+        if self.first_seen is not None:
+            # Pages before what the step's first token of a request sees. They may still be read by the iteration
+            # in flight; whoever gets them writes them in a later one.
             for kv, n in zip(kvs, np.diff(qo_indptr)):
-                kv.trim(kv.seqlen - int(n) - self.kv_window + 1)
+                kv.trim(self.first_seen(kv.seqlen - int(n)))
         arrays = request_arrays(kvs)
 
         # 5. state transitions for the launched work

@@ -88,7 +88,7 @@ def main(argv=None) -> int:
                     average_decode_length=a.output_len, group_size=m.group_size,
                     decode_tail_fraction=e.decode_tail_fraction,
                     state_pool=StateSlotPool(eng.num_slots) if getattr(eng, "num_slots", 0) else None,
-                    kv_window=getattr(m, "kv_window", 0))
+                    first_seen=getattr(m, "first_seen", None))
     loop = ServingLoop(eng, sch, rm, simulated_time=True, est_cycle_time=1.0)
     loop.skip_cycles(a.skip_cycles)
     loop.step()
