@@ -157,7 +157,7 @@ def main():
                     "captured and launched as CUDA graphs) | python")
     ap.add_argument("--layer-list", default="", help="instead of the headline workload: prefill and decode throughput of the "
                     "layer-list model beside the Llama of equal size, comma-separated sizes out of 2B, 8B")
-    ap.add_argument("--layer-model", default="volarax", help="with --layer-list: volarax, zubedra, gupizen, or several with commas")
+    ap.add_argument("--layer-model", default="volarax", help="with --layer-list: volarax, zubedra, gupizen, gimudra, or several with commas")
     ap.add_argument("--layer-list-only", default="", help="with --layer-list: only workloads whose name holds this text")
     ap.add_argument("--timeline", default="", help="after the timed regions, time every op of one iteration "
                     "with CUDA events and write the aggregate + Chrome trace to this file")

@@ -353,6 +353,11 @@ def _gupizen(*a, **kw):
     return builtin(*a, **kw)
 
 
+def _gimudra(*a, **kw):
+    from .models.gimudra import builtin
+    return builtin(*a, **kw)
+
+
 _LLAMA31_SCALING = {"factor": 8.0, "low_freq_factor": 1.0, "high_freq_factor": 4.0,
                     "original_max_position_embeddings": 8192, "rope_type": "llama3"}
 
@@ -397,6 +402,12 @@ MODEL_ARCHS: Dict[str, Dict[str, Any]] = {
     "gupizen-2B": _gupizen(2048, 32000, "pd" * 12, heads=16, kv_heads=4, dim=128, vdim=128, window=512, rec_width=2048,
                            rec_blocks=16, d_heads=16, d_kv_heads=16, d_dim=128, d_vdim=128, rank=128, experts=64, top=6,
                            ff=2048),
+    "gimudra-tiny": _gimudra(200, 1000, "dmsm", heads=6, kv_heads=2, dim=40, vdim=24, chunks=(37, 60), ff=136, experts=10, top=3,
+                             e_ff=40, groups=4, keep=2, identity=2),
+    "gimudra-8B": _gimudra(4096, 128256, "d" + "m" * 16 + "s" * 15, heads=32, kv_heads=8, dim=128, vdim=128, chunks=(8192,), ff=14336,
+                           experts=60, top=6, e_ff=3584, groups=8, keep=4, identity=4),
+    "gimudra-2B": _gimudra(2048, 32000, "d" + "m" * 12 + "s" * 11, heads=16, kv_heads=4, dim=128, vdim=128, chunks=(1536,), ff=8192,
+                           experts=60, top=6, e_ff=2048, groups=8, keep=4, identity=4),
 }
 
 MODEL_IDS = {
@@ -406,7 +417,7 @@ MODEL_IDS = {
     "deepseek-67B": "deepseek-ai/deepseek-llm-67b-chat", "mixtral-8-7B": "mistralai/Mixtral-8x7B-Instruct-v0.1",
     "tiny": "nanoflow/tiny-llama-test", "tiny8": "nanoflow/tiny8-llama-test",
     "volarax-tiny": "nanoflow/volarax-tiny-test", "zubedra-tiny": "nanoflow/zubedra-tiny-test",
-    "gupizen-tiny": "nanoflow/gupizen-tiny-test",
+    "gupizen-tiny": "nanoflow/gupizen-tiny-test", "gimudra-tiny": "nanoflow/gimudra-tiny-test",
 }
 
 

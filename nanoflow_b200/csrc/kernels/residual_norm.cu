@@ -128,7 +128,8 @@ __device__ __forceinline__ float2 sin_cos(float pos, float2 f) {
   const float a = pos * f.x, e = fmaf(pos, f.x, -a) + pos * f.y;
   float s, c;
   sincosf(a, &s, &c);
-  return make_float2(fmaf(e, c, s), fmaf(-e, s, c));
+  const float h = 0.5f * e * e;
+  return make_float2(fmaf(-h, s, fmaf(e, c, s)), fmaf(-h, c, fmaf(-e, s, c)));
 }
 
 // v (the sum of the row) is kept as a result of its own, and replaced by the weighted sum of all results so far.

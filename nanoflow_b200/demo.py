@@ -23,7 +23,7 @@ from typing import List
 
 MODELS = ["llama2-70B", "llama3-70B", "llama3.1-70B", "llama3-8B", "llama3.1-8B", "qwen2-72B", "tiny",
           "volarax-tiny", "volarax-2B", "volarax-8B", "zubedra-tiny", "zubedra-2B", "zubedra-8B",
-          "gupizen-tiny", "gupizen-2B", "gupizen-8B"]
+          "gupizen-tiny", "gupizen-2B", "gupizen-8B", "gimudra-tiny", "gimudra-2B", "gimudra-8B"]
 
 
 def _serve(a) -> int:

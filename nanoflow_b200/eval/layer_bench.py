@@ -22,13 +22,14 @@ import torch
 SIZES = {
     # name: (width, ff, heads, kv heads of the Llama, vocab, latent rank, window, mLSTM heads, dim, vdim,
     #        WKV decay rank, ff of an expert and of the shared one: 6 experts per token and the shared one make up ff,
-    #        blocks of the linear recurrent unit, ff of an expert without a gate: 6 of them have as many weights as ff)
+    #        blocks of the linear recurrent unit, ff of an expert without a gate: 6 of them have as many weights as ff,
+    #        tokens per chunk of chunked attention)
     "8B": dict(width=4096, ff=14336, heads=32, kv=8, vocab=128256, rank=512, window=1024, mh=8, md=256, mv=512, decay=128,
-               eff=2048, sff=2048, blocks=16, uff=3584),
+               eff=2048, sff=2048, blocks=16, uff=3584, chunk=8192),
     "2B": dict(width=2048, ff=8192, heads=16, kv=4, vocab=32000, rank=256, window=512, mh=4, md=256, mv=512, decay=64,
-               eff=1024, sff=2048, blocks=16, uff=2048),
+               eff=1024, sff=2048, blocks=16, uff=2048, chunk=1536),
 }
-EXPERTS, TOP, GROUPS, KEEP = 64, 6, 8, 4
+EXPERTS, TOP, GROUPS, KEEP, IDENTITY = 64, 6, 8, 4, 4
 WORKLOADS = [("prefill 4 x 1024", [(0, 1024)] * 4), ("prefill 1 x 4096", [(0, 4096)]),
              ("decode 256 at 1280", [(1280, 1)] * 256), ("decode 32 at 4096", [(4096, 1)] * 32)]
 LAYERS = 4
@@ -45,7 +46,7 @@ def peaks() -> Tuple[float, float]:
 
 def model_dict(kind: str, s: Dict[str, int]) -> Dict[str, Any]:
     from ..config import _hf
-    from ..models import gupizen, volarax, zubedra
+    from ..models import gimudra, gupizen, volarax, zubedra
     if kind == "llama":
         return _hf(s["width"], s["ff"], LAYERS, s["heads"], s["kv"], s["vocab"], 500000.0)
     if kind == "zubedra":
@@ -56,6 +57,10 @@ def model_dict(kind: str, s: Dict[str, int]) -> Dict[str, Any]:
         return gupizen.builtin(s["width"], s["vocab"], "pd" * (LAYERS // 2), heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128,
                                window=s["window"], rec_width=s["width"], rec_blocks=s["blocks"], d_heads=s["heads"],
                                d_kv_heads=s["heads"], d_dim=128, d_vdim=128, rank=128, experts=EXPERTS, top=TOP, ff=s["uff"])
+    if kind == "gimudra":
+        return gimudra.builtin(s["width"], s["vocab"], "dmms"[:LAYERS], heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128,
+                               chunks=(s["chunk"],), ff=s["ff"], experts=EXPERTS - IDENTITY, top=TOP, e_ff=s["uff"], groups=GROUPS,
+                               keep=KEEP, identity=IDENTITY)
     return volarax.builtin(s["width"], s["vocab"], "am" * (LAYERS // 2), heads=s["heads"], dim=128, vdim=128, kv_rank=s["rank"],
                    window=s["window"], m_heads=s["mh"], m_dim=s["md"], m_vdim=s["mv"], ff=s["ff"], m_ff=s["ff"])
 
@@ -96,7 +101,9 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
     m, p = engine.model, op.params
     T = sum(n for _, n in spans)
     es = 2
-    sees = lambda w: sum(sum(min(c + t + 1, w or c + t + 1) for t in range(n)) for c, n in spans)
+    def sees(w, chunk=0):
+        """(query, key) pairs, with a window or chunks."""
+        return sum(sum(min(c + t + 1, w or c + t + 1) - ((c + t) // chunk * chunk if chunk else 0) for t in range(n)) for c, n in spans)
     if isinstance(p, G.GemmParams):
         dyn = dict(op.dyn)["M"]
         M = engine._last_sym.get(dyn, 0)
@@ -111,8 +118,8 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
         if (spans[0][1] == 1) == pre:
             return 0.0, 0.0
         w = p.window
-        pairs = sees(w)
-        keys = sum(min(c + n, (w + n - 1) if w else c + n) for c, n in spans)
+        pairs = sees(w, p.chunk)
+        keys = sum(min(c + n, (w + n - 1) if w else c + n) - (c // p.chunk * p.chunk if p.chunk else 0) for c, n in spans)
         return 4.0 * pairs * p.q_heads * p.head_dim, es * (2 * keys * p.kv_heads * p.head_dim + 2 * T * p.q_heads * p.head_dim)
     if isinstance(p, G.LatentAttnParams):
         if spans[0][1] != 1:
@@ -130,9 +137,10 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
     if isinstance(p, G.ResidualNormParams):
         rows = T if not p.rows_idx else len(spans)
         more = (1 if p.y2 else 0) + (p.e_top if p.e_out else 0)
-        return 0.0, rows * p.cols * (8 + (2 + more) * es)
+        earlier = (p.hist_n if p.hist_w else 0) + (1 if p.hist_out else 0)
+        return 0.0, rows * p.cols * (8 + 4 * earlier + (2 + more) * es)
     if isinstance(p, G.GqaAppendParams):
-        return 0.0, T * 2 * (p.heads + 2 * p.kv_heads) * p.hd * es
+        return 0.0, T * 2 * ((p.heads if p.q_out else 0) + 2 * p.kv_heads) * p.hd * es
     if isinstance(p, G.TalkAttnParams):
         if (spans[0][1] == 1) != (dict(op.dyn).get("n_tokens") == "n_dec"):
             return 0.0, 0.0
@@ -168,9 +176,9 @@ def op_work(engine, op, spans) -> Tuple[float, float]:
     if isinstance(p, G.MoeRouteParams):
         return 0.0, T * 4 * (p.experts + 3 * p.top)
     if isinstance(p, G.MoePermuteParams):
-        return 0.0, T * (1 + p.top) * p.cols * es
+        return 0.0, (T + engine._expert_rows) * p.cols * es
     if isinstance(p, G.MoeGemmParams):
-        rows, mats = engine._last_sym.get(dict(op.dyn)["rows"], 0), 2 if p.B2 else 1
+        rows, mats = engine._expert_rows, 2 if p.B2 else 1
         used = min(p.experts, engine._experts_used)
         return 2.0 * rows * p.N * p.K * mats, es * (mats * used * p.N * p.K + rows * (p.K + p.N))
     if isinstance(p, G.HeadNormGateParams):
@@ -206,6 +214,7 @@ def measure(engine, plan, spans, steps: int, warmup: int) -> Dict[str, Any]:
     # experts that got rows in the last iteration (fewest of all layers): their weights have to be read
     counts = [c for c in getattr(engine, "moe_counts_of", []) if c is not None]
     engine._experts_used = min((int((c > 0).sum()) for c in counts), default=0)
+    engine._expert_rows = min((int(c.sum()) for c in counts), default=0)      # (fewer than chosen with identity experts)
     # one op at a time, best of three iterations
     best: Dict[int, float] = {}
     for _ in range(3):
