@@ -243,8 +243,8 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
         for (int e = 0; e < 4; ++e) {
           const float2 f = e < 2 ? far0 : far1;
           const float d = fmaxf(d0 - (e & 1), 0.f), d8 = fmaxf(d0 - (e & 1) - 8.f, 0.f);
-          s0[e] -= f.x * __log2f(fmaf(f.y, d, 1.f));
-          s1[e] -= f.x * __log2f(fmaf(f.y, d8, 1.f));
+          s0[e] -= distance_loss(f, d);
+          s1[e] -= distance_loss(f, d8);
         }
       }
       if (EXT && pslot == rg.skip && p.chunk > 0) {          // the page that the chunk starts in

@@ -124,6 +124,13 @@ __device__ __forceinline__ Item read_item(const nfk_attn_params& p, long long w)
   return it;
 }
 
+// The CTA's work in round k, -1 if there is none. Later items of a request see more keys, so the last ones go first, and every
+// other round deals them out in reverse: each CTA's share is of nearly the same length.
+__device__ __forceinline__ long long work_index(int k, long long total) {
+  const long long g = gridDim.x, i = k * g + ((k & 1) != 0 ? g - 1 - blockIdx.x : blockIdx.x);
+  return i < total ? total - 1 - i : -1;
+}
+
 template <int HD, bool EXT, bool CAP, bool DIST>
 __global__ void __launch_bounds__(kThreads, 2)
 attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
@@ -168,6 +175,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
   const int group = p.q_heads / p.kv_heads;
   const long long total = static_cast<long long>(p.num_items) * p.kv_heads;
+  const int rounds = static_cast<int>((total + gridDim.x - 1) / gridDim.x);
   auto fail = [&](unsigned int code) {
     report_status(p.status, code);
     *abort_flag = 1;
@@ -180,7 +188,9 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       uint32_t issued[NUM_BARS];           // per "full" barrier: loads issued on it
       for (int b = 0; b < NUM_BARS; ++b) issued[b] = 0;
       bool ok = true;
-      for (long long w = blockIdx.x; w < total && ok; w += gridDim.x) {
+      for (int k = 0; k < rounds && ok; ++k) {
+        const long long w = work_index(k, total);
+        if (w < 0) continue;
         const Item it = read_item<EXT>(p, w);
         if (!it.valid) continue;
         if (!mbar_wait(&bars[Q_EMPTY], (n_item & 1) ^ 1) || *abort_flag) { fail(NF_ST_TIMEOUT_SMEM_EMPTY); break; }
@@ -285,7 +295,9 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         return true;
       };
       bool ok = true;
-      for (long long w = blockIdx.x; w < total && ok; w += gridDim.x) {
+      for (int k = 0; k < rounds && ok; ++k) {
+        const long long w = work_index(k, total);
+        if (w < 0) continue;
         const Item it = read_item<EXT>(p, w);
         if (!it.valid) continue;
         if (!mbar_wait(&bars[Q_FULL], n_item & 1) || *abort_flag) { fail(NF_ST_TIMEOUT_SMEM_FULL); break; }
@@ -334,7 +346,9 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const float cap_in = CAP ? p.sm_scale / p.softcap : 0.f, cap_out = CAP ? p.softcap * kLog2e : 0.f;
     uint32_t g = 0, n_item = 0;
     bool ok = true;
-    for (long long w = blockIdx.x; w < total && ok; w += gridDim.x) {
+    for (int k = 0; k < rounds && ok; ++k) {
+        const long long w = work_index(k, total);
+        if (w < 0) continue;
       const Item it = read_item<EXT>(p, w);
       if (!it.valid) continue;
       const int tl = row / group, hh = row % group;
@@ -347,6 +361,13 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       for (int t = 0; t < it.n_tiles; ++t) {
         const uint32_t gt = g + t;
         const int s = gt & 1;
+        const int cbase = (it.t_first + t) * kTile;
+        float loss[DIST ? 64 : 1];                             // does not depend on the scores: while they are formed
+        if (DIST) {
+          const float d0 = static_cast<float>(pos - cbase);
+#pragma unroll
+          for (int j = 0; j < 64; ++j) loss[DIST ? j : 0] = distance_loss(far, d0 - j);     // (keys behind the row are masked below)
+        }
         if (!mbar_wait(&bars[S_FULL0 + s], (gt >> 1) & 1) || *abort_flag) { fail(NF_ST_TIMEOUT_TMEM_FULL); ok = false; break; }
         tc_fence_after();
         uint32_t r0[32], r1[32];
@@ -360,14 +381,12 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             r1[j] = __float_as_uint(cap_out * tanh_by_exp(__uint_as_float(r1[j]) * cap_in));
           }
         }
-        const int cbase = (it.t_first + t) * kTile;
         if (DIST) {
-          const float in = p.sm_scale * kLog2e, d0 = static_cast<float>(pos - cbase);
+          const float in = p.sm_scale * kLog2e;
 #pragma unroll
-          for (int j = 0; j < 32; ++j) {                      // (keys behind the row are masked below)
-            const float a = __log2f(fmaf(far.y, d0 - j, 1.f)), b = __log2f(fmaf(far.y, d0 - (32 + j), 1.f));
-            r0[j] = __float_as_uint(fmaf(__uint_as_float(r0[j]), in, -far.x * a));
-            r1[j] = __float_as_uint(fmaf(__uint_as_float(r1[j]), in, -far.x * b));
+          for (int j = 0; j < 32; ++j) {
+            r0[j] = __float_as_uint(fmaf(__uint_as_float(r0[j]), in, -loss[DIST ? j : 0]));
+            r1[j] = __float_as_uint(fmaf(__uint_as_float(r1[j]), in, -loss[DIST ? 32 + j : 0]));
           }
         }
         if (cbase + kTile - 1 > pos) {                        // only tiles on the diagonal need the mask

@@ -212,7 +212,7 @@ def measure(engine, plan, spans, steps: int, warmup: int) -> Dict[str, Any]:
     ms = e0.elapsed_time(e1) / steps
     engine.check_status()
     # experts that got rows in the last iteration (fewest of all layers): their weights have to be read
-    counts = [c for c in getattr(engine, "moe_counts_of", []) if c is not None]
+    counts = [c for c in getattr(engine, "moe_counts_of", []) if c is not None and c.numel()]
     engine._experts_used = min((int((c > 0).sum()) for c in counts), default=0)
     engine._expert_rows = min((int(c.sum()) for c in counts), default=0)      # (fewer than chosen with identity experts)
     # one op at a time, best of three iterations

@@ -140,8 +140,10 @@ def _random(name: str, shape: Tuple[int, ...], g: torch.Generator, device, dtype
     t = torch.empty(shape, dtype=dtype, device=device).normal_(generator=g)
     if last in ("norm", "norm1", "norm2", "ls1", "ls2"):
         return 1.0 + 0.1 * t
-    if last in ("b", "correction"):
+    if last == "b":
         return 0.1 * t
+    if last == "correction":                     # (scores are shares of one)
+        return 0.1 / shape[0] * t
     if last == "dwa":
         t = 0.1 * t
         t[-1] += 1.0

@@ -3,6 +3,10 @@ import sys
 
 import pytest
 
+# The tests' tensors are small: more threads than one per operation only wait for one another, above all when several
+# processes run side by side.
+os.environ.setdefault("OMP_NUM_THREADS", "1")
+
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 
 
