@@ -188,8 +188,7 @@ __device__ __forceinline__ NBlock n_block(const DevParams& p, int n_blk, int out
 }
 
 // v += the bias of eight columns.
-__device__ __forceinline__ void add_bias8(float* v, const __nv_bfloat16* bias) {
-  const uint4 bv = *reinterpret_cast<const uint4*>(bias);
+__device__ __forceinline__ void add_bias8(float* v, uint4 bv) {
   const uint32_t bw[4] = {bv.x, bv.y, bv.z, bv.w};
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
@@ -197,6 +196,10 @@ __device__ __forceinline__ void add_bias8(float* v, const __nv_bfloat16* bias) {
     v[2 * j] += f.x;
     v[2 * j + 1] += f.y;
   }
+}
+
+__device__ __forceinline__ void add_bias8(float* v, const __nv_bfloat16* bias) {
+  add_bias8(v, *reinterpret_cast<const uint4*>(bias));
 }
 
 // Eight finished columns of one row: bf16 to D, or fp32 to D32 from f32_col0 on (a multiple of 8).
@@ -617,6 +620,17 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             const int nval = tail16 ? 16 : 32;
             if (tail16) tmem_ld_32x32b_x16(t_lane + mt * BN + c * 32, r);
             else tmem_ld_32x32b_x32(t_lane + mt * BN + c * 32, r);
+            // biases are requested while the accumulators are on their way
+            uint4 bias_w[4], bias2_w[EPI == 1 ? 4 : 1];
+            if (EPI != 2 && p.bias != nullptr) {
+#pragma unroll
+              for (int g8 = 0; g8 < 4; ++g8) {
+                const int col = nb.col0 + c * 32 + g8 * 8;
+                bias_w[g8] = col < tile_col_end ? *reinterpret_cast<const uint4*>(p.bias + col) : make_uint4(0, 0, 0, 0);
+                if (EPI == 1)
+                  bias2_w[EPI == 1 ? g8 : 0] = col < tile_col_end ? *reinterpret_cast<const uint4*>(p.bias2 + col) : make_uint4(0, 0, 0, 0);
+              }
+            }
             if (EPI == 1) {
               uint32_t uu[32];
               if (tail16) tmem_ld_32x32b_x16(t_lane + mt * BN + BN / 2 + c * 32, uu);
@@ -645,11 +659,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
               if (p.bias != nullptr) {
 #pragma unroll
                 for (int g8 = 0; g8 < 4; ++g8) {
-                  const int col = nb.col0 + c * 32 + g8 * 8;
-                  if (col < tile_col_end) {
-                    add_bias8(gsum + g8 * 8, p.bias + col);
-                    add_bias8(usum + g8 * 8, p.bias2 + col);
-                  }
+                  add_bias8(gsum + g8 * 8, bias_w[g8]);
+                  add_bias8(usum + g8 * 8, bias2_w[EPI == 1 ? g8 : 0]);
                 }
               }
 #pragma unroll
@@ -752,7 +763,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 if (col < tile_col_end) {  // N is a multiple of 8
                   float* vv = v + g8 * 8;
                   if (EPI == 0) {
-                    if (p.bias != nullptr) add_bias8(vv, p.bias + col);
+                    if (p.bias != nullptr) add_bias8(vv, bias_w[g8]);
                     if (crow != nullptr) {
                       const uint4 cv = *reinterpret_cast<const uint4*>(crow + col);
                       const uint32_t cw[4] = {cv.x, cv.y, cv.z, cv.w};

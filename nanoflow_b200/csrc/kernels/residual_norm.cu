@@ -96,6 +96,27 @@ __device__ __forceinline__ void input_conv(const float4 (&v)[NV], const nfk_resi
   const T* st = reinterpret_cast<const T*>(p.conv_state) + (ok ? ref : 0) * half;
   T* keep = reinterpret_cast<T*>(p.conv_state) + (ok ? ref ^ 1 : 0) * half;
   T* out = reinterpret_cast<T*>(p.conv_out) + static_cast<long long>(row) * p.conv_ld;
+  if (before == 1) {                                     // two taps: everything is requested before anything is stored
+    float4 s[NV], f[NV], w[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int vi = threadIdx.x + i * kRnThreads;
+      if (vi >= nvec) continue;
+      s[i] = older ? load4(st + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      f[i] = load4(p.conv_w + vi * 4);
+      w[i] = load4(p.conv_w + p.conv_ld + vi * 4);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int vi = threadIdx.x + i * kRnThreads;
+      if (vi >= nvec) continue;
+      const float4 x = rounded(v[i], T(0.f));
+      if (ok) store4(keep + vi * 4, x);
+      store4(out + vi * 4, make_float4(x.x + w[i].x * x.x + f[i].x * s[i].x, x.y + w[i].y * x.y + f[i].y * s[i].y,
+                                       x.z + w[i].z * x.z + f[i].z * s[i].z, x.w + w[i].w * x.w + f[i].w * s[i].w));
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int vi = threadIdx.x + i * kRnThreads;
