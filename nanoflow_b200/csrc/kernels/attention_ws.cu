@@ -124,8 +124,9 @@ __device__ __forceinline__ Item read_item(const nfk_attn_params& p, long long w)
   return it;
 }
 
-// The CTA's work in round k, -1 if there is none. Later items of a request see more keys, so the last ones go first, and every
-// other round deals them out in reverse: each CTA's share is of nearly the same length.
+// The CTA's work in round k, -1 if there is none. Later items of a request see more keys (and callers may order all items by
+// that), so the last ones go first, and every other round deals them out in reverse: each CTA's share is of nearly the same
+// length.
 __device__ __forceinline__ long long work_index(int k, long long total) {
   const long long g = gridDim.x, i = k * g + ((k & 1) != 0 ? g - 1 - blockIdx.x : blockIdx.x);
   return i < total ? total - 1 - i : -1;

@@ -901,7 +901,7 @@ class LayerListEngine(Engine):
         if "pre_reqs" in self.meta:
             put("pre_reqs", np.arange(D, D + P, dtype=np.int32))
         for n in self.attn_groups:
-            items = query_items(qo, D, QUERY_TILE // n)
+            items = by_keys(query_items(qo, D, QUERY_TILE // n), plan.positions, m.first_seen)
             put(f"gitem{n}", items.reshape(-1))
             sym[f"n_gitems{n}"] = items.shape[0]
         if self.attn_groups:
@@ -1022,6 +1022,14 @@ def query_items(qo_indptr: np.ndarray, n_dec: int, tile: int) -> np.ndarray:
         q0, q1 = int(qo_indptr[b]), int(qo_indptr[b + 1])
         rows += [(b, t, min(tile, q1 - t)) for t in range(q0, q1, tile)]
     return np.asarray(rows, dtype=np.int32).reshape(-1, 3)
+
+
+def by_keys(items: np.ndarray, positions: np.ndarray, first_seen) -> np.ndarray:
+    """Work items in the order of how many keys they see: the prefill kernel deals out the last ones first."""
+    if items.shape[0] == 0:
+        return items
+    first, last = positions[items[:, 1]], positions[items[:, 1] + items[:, 2] - 1]
+    return items[np.argsort(last - np.asarray([first_seen(int(p)) for p in first]), kind="stable")]
 
 
 def route_attention(plan: BatchPlan, window: int, expands: bool, page_cap: int, min_tokens: int) -> dict:

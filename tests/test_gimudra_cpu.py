@@ -16,6 +16,7 @@ from nanoflow_b200.models.safetensors_io import write_safetensors
 from nanoflow_b200.ops import reference as ref
 from nanoflow_b200.replay import TraceReplay
 from nanoflow_b200.runtime.cpu_layer_list import CpuLayerListEngine
+from nanoflow_b200.runtime.layer_list import by_keys, query_items
 from nanoflow_b200.serving import DistKVPool, RequestManager, Scheduler, StateSlotPool
 from nanoflow_b200.serving.loop import ServingLoop
 from volarax_cases import prompt, row_errors
@@ -118,6 +119,17 @@ def test_first_position_that_any_layer_sees():
         want = min(p // c * c for c in (20, 33, 48, 64, 50))
         assert m.first_seen(p) == want <= m.first_seen(p + 1)
     assert cases.engine_config(cases.CASES["wide_heads"]).model.first_seen(399) == 0
+
+
+def test_work_items_are_ordered_by_the_keys_they_see():
+    """Two prompts from their start and one that goes on behind the start of a chunk."""
+    qo = np.asarray([0, 1, 41, 81, 121])
+    pos = np.concatenate([[500], np.arange(40), np.arange(40), np.arange(90, 130)])
+    items = by_keys(query_items(qo, 1, 16), pos, lambda p: p // 100 * 100)
+    assert sorted(map(tuple, items.tolist())) == sorted(map(tuple, query_items(qo, 1, 16).tolist()))
+    seen = [int(pos[t + n - 1]) - int(pos[t]) // 100 * 100 for _, t, n in items]
+    assert seen == sorted(seen)
+    assert by_keys(query_items(qo, 4, 16), pos, lambda p: 0).shape == (0, 3)
 
 
 # ---- single mechanisms of the CPU backend -------------------------------------------------------------------------
