@@ -338,6 +338,11 @@ struct Walk {
 // per k step into one accumulator of BN columns. A pair MMA takes half of its weight rows from each CTA, so
 // each CTA stages quarter `rank` of both halves, one behind the other, and the accumulator columns come out in
 // the order of the weight rows. A separate instantiation: the common kernel's instruction stream is untouched.
+// Forms of the epilogue as template parameter: NFK_EPI_*, and the gated one with biases on both halves, which has kernels of
+// its own so that the others keep their registers.
+constexpr int kGatedBias = 3;
+constexpr bool gated_epi(int epi) { return epi == 1 || epi == kGatedBias; }
+
 template <int MT, int EPI, int CG, bool WIDE>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB0,
@@ -375,7 +380,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
   const int STAGE_BYTES = MT * A_TILE_BYTES + B_BYTES;
   constexpr int A_BYTES = MT * A_TILE_BYTES;
   // Output tile width: the SwiGLU epilogue folds a gate half and an up half of BN/2 columns each.
-  const int OUT_BN = (EPI == 1) ? BN / 2 : BN;
+  const int OUT_BN = gated_epi(EPI) ? BN / 2 : BN;
   const int m_tiles = (p.M + BM - 1) / BM;
   const int m_groups = (m_tiles + MT * CG - 1) / (MT * CG);
   const int n_blocks = n_block_count(p.groups, p.group_n, OUT_BN);
@@ -397,7 +402,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
     mbar_fence_init();
     tma_prefetch_desc(&tmA);
     tma_prefetch_desc(&tmB0);
-    if (EPI == 1) tma_prefetch_desc(&tmB1);
+    if (gated_epi(EPI)) tma_prefetch_desc(&tmB1);
   }
   if (warp == 1) {
     if (CG == 2) {
@@ -457,7 +462,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
           // A tile past the last row or column is still copied in full (zero filled).
           const uint32_t fb = mapa_shared(smem_u32(&full_bar[s]), 0);
           if (leader) mbar_expect_tx(&full_bar[s], 2 * (A_TILE_BYTES + B_BYTES));
-          if (EPI == 1)
+          if (gated_epi(EPI))
             tma_load_2d_pair(sb, rank == 0 ? &tmB0 : &tmB1, fb, kb * BK, nb.col0);
           else if (WIDE) {
             const int qrows = BN / 4;
@@ -470,7 +475,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
           continue;
         }
         mbar_expect_tx(&full_bar[s], mt_valid * A_TILE_BYTES + B_BYTES);
-        if (EPI == 1) {
+        if (gated_epi(EPI)) {
           tma_load_2d(sb, &tmB0, &full_bar[s], kb * BK, nb.col0);
           tma_load_2d(sb + B_BYTES / 2, &tmB1, &full_bar[s], kb * BK, nb.col0);
         } else {
@@ -621,17 +626,16 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             if (tail16) tmem_ld_32x32b_x16(t_lane + mt * BN + c * 32, r);
             else tmem_ld_32x32b_x32(t_lane + mt * BN + c * 32, r);
             // biases are requested while the accumulators are on their way
-            uint4 bias_w[4], bias2_w[EPI == 1 ? 4 : 1];
-            if (EPI != 2 && p.bias != nullptr) {
+            uint4 bias_w[EPI == kGatedBias ? 4 : 1], bias2_w[EPI == kGatedBias ? 4 : 1];
+            if constexpr (EPI == kGatedBias) {
 #pragma unroll
               for (int g8 = 0; g8 < 4; ++g8) {
                 const int col = nb.col0 + c * 32 + g8 * 8;
                 bias_w[g8] = col < tile_col_end ? *reinterpret_cast<const uint4*>(p.bias + col) : make_uint4(0, 0, 0, 0);
-                if (EPI == 1)
-                  bias2_w[EPI == 1 ? g8 : 0] = col < tile_col_end ? *reinterpret_cast<const uint4*>(p.bias2 + col) : make_uint4(0, 0, 0, 0);
+                bias2_w[g8] = col < tile_col_end ? *reinterpret_cast<const uint4*>(p.bias2 + col) : make_uint4(0, 0, 0, 0);
               }
             }
-            if (EPI == 1) {
+            if (gated_epi(EPI)) {
               uint32_t uu[32];
               if (tail16) tmem_ld_32x32b_x16(t_lane + mt * BN + BN / 2 + c * 32, uu);
               else tmem_ld_32x32b_x32(t_lane + mt * BN + BN / 2 + c * 32, uu);
@@ -656,11 +660,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 }
                 continue;
               }
-              if (p.bias != nullptr) {
+              if constexpr (EPI == kGatedBias) {
 #pragma unroll
                 for (int g8 = 0; g8 < 4; ++g8) {
                   add_bias8(gsum + g8 * 8, bias_w[g8]);
-                  add_bias8(usum + g8 * 8, bias2_w[EPI == 1 ? g8 : 0]);
+                  add_bias8(usum + g8 * 8, bias2_w[g8]);
                 }
               }
 #pragma unroll
@@ -763,7 +767,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 if (col < tile_col_end) {  // N is a multiple of 8
                   float* vv = v + g8 * 8;
                   if (EPI == 0) {
-                    if (p.bias != nullptr) add_bias8(vv, bias_w[g8]);
+                    if (p.bias != nullptr) add_bias8(vv, p.bias + col);
                     if (crow != nullptr) {
                       const uint4 cv = *reinterpret_cast<const uint4*>(crow + col);
                       const uint32_t cw[4] = {cv.x, cv.y, cv.z, cv.w};
@@ -1050,7 +1054,7 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
   int budget = g.smem_budget_kb > 0 ? g.smem_budget_kb * 1024 : kSmemMax;
   if (budget > kSmemMax) budget = kSmemMax;
   const bool rs_staged = EPI == 2 && g.rs_staged != 0;
-  const Geom geo = make_geom(bn, MT, EPI == 1, budget, CG, rs_staged ? kRsStageBytes : 0);
+  const Geom geo = make_geom(bn, MT, gated_epi(EPI), budget, CG, rs_staged ? kRsStageBytes : 0);
   if (geo.stages < 2) return NF_ERR_BAD_ARG;      // shared-memory budget too small for this tile
   CUtensorMap tmA, tmB0, tmB1;
   const int groups = g.groups > 1 ? g.groups : 1;
@@ -1061,10 +1065,10 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
   if (rc != NF_OK) return rc;
   // rows of B that one TMA copy brings in: a whole tile, a SwiGLU half, or a CTA pair's half
   // (wide tiles: a quarter of the tile per copy, two copies per CTA)
-  const int b_box = (EPI == 1) ? geo.out_bn : (WIDE ? bn / 4 : bn / CG);
+  const int b_box = gated_epi(EPI) ? geo.out_bn : (WIDE ? bn / 4 : bn / CG);
   rc = make_tmap_bf16_2d(&tmB0, g.B, g.N, g.K, g.ldb, b_box, BK);
   if (rc != NF_OK) return rc;
-  if (EPI == 1) {
+  if (gated_epi(EPI)) {
     rc = make_tmap_bf16_2d(&tmB1, g.B2, g.N, g.K, g.ldb, b_box, BK);
     if (rc != NF_OK) return rc;
   } else {
@@ -1199,7 +1203,7 @@ int launch_impl(const nfk_gemm_params& g, int bn, int split_k, bool stream_k, cu
     const long long total = static_cast<long long>(sk.rest) * CG * MT * BM * (geo.out_bn / 8);
     long long blocks = (total + 255) / 256;
     if (blocks > sm_count() * 8) blocks = sm_count() * 8;
-    sk_fixup_kernel<EPI == 1 ? 1 : 0><<<static_cast<int>(blocks), 256, 0, stream>>>(p, f);
+    sk_fixup_kernel<gated_epi(EPI) ? 1 : 0><<<static_cast<int>(blocks), 256, 0, stream>>>(p, f);
     if (cudaGetLastError() != cudaSuccess) return NF_ERR_CUDA;
   }
   p.norm_w = reinterpret_cast<const __nv_bfloat16*>(g.norm_w);
@@ -1467,6 +1471,7 @@ extern "C" int nfk_gemm_bf16(const nfk_gemm_params* g, cudaStream_t stream) {
   if (rcs != NF_OK) return rcs;
   if (swiglu) {
     if ((s.bn / 2) % 16 != 0) return NF_ERR_UNSUPPORTED;
+    if (g->bias != nullptr) return launch_mt<kGatedBias>(*g, s.bn, s.mt, s.cg, 1, s.stream_k, stream);
     return launch_mt<1>(*g, s.bn, s.mt, s.cg, 1, s.stream_k, stream);
   }
   if (rs) return launch_mt<2>(*g, s.bn, s.mt, s.cg, 1, false, stream);

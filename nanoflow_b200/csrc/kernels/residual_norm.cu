@@ -96,7 +96,7 @@ __device__ __forceinline__ void input_conv(const float4 (&v)[NV], const nfk_resi
   const T* st = reinterpret_cast<const T*>(p.conv_state) + (ok ? ref : 0) * half;
   T* keep = reinterpret_cast<T*>(p.conv_state) + (ok ? ref ^ 1 : 0) * half;
   T* out = reinterpret_cast<T*>(p.conv_out) + static_cast<long long>(row) * p.conv_ld;
-  if (before == 1) {                                     // two taps: everything is requested before anything is stored
+  if (NV <= 8 && before == 1) {                          // two taps: everything is requested before anything is stored
     float4 s[NV], f[NV], w[NV];
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
