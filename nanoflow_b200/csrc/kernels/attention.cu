@@ -171,11 +171,11 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
     if (c_begin >= c_end) break;  // uniform across the CTA: on to the next item
     const int tok = p.qo_indptr[req];
     const long long ld_q = EXT && p.ld_q > 0 ? p.ld_q : p.q_heads * HD;
-    float2 far0 = make_float2(0.f, 0.f), far1 = far0;        // distance bias of this lane's two rows
+    float2 loss0 = make_float2(0.f, 0.f), loss1 = loss0;        // distance bias of this lane's two rows
     if (EXT && p.dist != nullptr) {
       const float2* dist = reinterpret_cast<const float2*>(p.dist) + kvh * group;
-      if ((lane >> 2) < group) far0 = dist[lane >> 2];
-      if ((lane >> 2) + 8 < group) far1 = dist[(lane >> 2) + 8];
+      if ((lane >> 2) < group) loss0 = dist[lane >> 2];
+      if ((lane >> 2) + 8 < group) loss1 = dist[(lane >> 2) + 8];
     }
 
     uint32_t qa[HD / 16][4];
@@ -241,7 +241,7 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
         const float d0 = static_cast<float>(rg.pos - (rg.first + pslot) * kPage - c0);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float2 f = e < 2 ? far0 : far1;
+          const float2 f = e < 2 ? loss0 : loss1;
           const float d = fmaxf(d0 - (e & 1), 0.f), d8 = fmaxf(d0 - (e & 1) - 8.f, 0.f);
           s0[e] -= distance_loss(f, d);
           s1[e] -= distance_loss(f, d8);

@@ -217,12 +217,10 @@ def test_every_mechanism_shows_in_the_logits(monkeypatch):
         e = row_errors(oracle.forward(raw, t, toks), want)
         monkeypatch.setattr(oracle, name, real[name])
         assert not float(e.max()) <= 0.02, what
-    lent = json.loads(json.dumps(raw))
-    for i, j in ((2, 1), (3, 0)):
+    for i, j in ((2, 1), (3, 0)):                        # keys and values of another layer
         other = json.loads(json.dumps(raw))
         other["layers"][i]["mixer"]["kv_from"] = j
         assert float(row_errors(oracle.forward(other, t, toks), want).max()) > 0.02
-    assert lent == raw
 
 
 # ---- the CPU backend against the oracle ------------------------------------------------------------------------
