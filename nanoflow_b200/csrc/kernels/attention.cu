@@ -171,7 +171,7 @@ attn_decode_kernel(nfk_attn_params p, int slot) {
     if (c_begin >= c_end) break;  // uniform across the CTA: on to the next item
     const int tok = p.qo_indptr[req];
     const long long ld_q = EXT && p.ld_q > 0 ? p.ld_q : p.q_heads * HD;
-    float2 loss0 = make_float2(0.f, 0.f), loss1 = loss0;        // distance bias of this lane's two rows
+    float2 loss0 = make_float2(0.f, 0.f), loss1 = loss0;      // distance bias of this lane's two rows
     if (EXT && p.dist != nullptr) {
       const float2* dist = reinterpret_cast<const float2*>(p.dist) + kvh * group;
       if ((lane >> 2) < group) loss0 = dist[lane >> 2];
